@@ -249,6 +249,60 @@ typedef struct ob_model_desc {
                                  * (i, i + rope_dim/2) -- qwen2, qwen3, qwen3vl (rope_layout_for, E/arch/llama.rs:114-119) */
 } ob_model_desc;
 
+/* ------------------------------------------------- models given as a list of layers
+ * Designs whose layers are not all alike: every layer names its token mixer and carries that mixer's sizes, constants and
+ * tensors; mixer and feed-forward read the same normed input (parallel layers, x += mixer(h) + ff(h), h = norm(x) with one
+ * number as gain).  No counterpart in the reference.  The result is an ob_model like any other: caches, batching, sampling,
+ * captured decode graphs and the slot pool are the same calls.  Matrices are bfloat16, out_dim rows of in_dim; vectors f32. */
+#define OB_TYPE_BF16 30u /* ob_matrix_desc.ggml_type of these matrices */
+#define OB_MIXER_LATENT_ATTENTION 1u
+#define OB_MIXER_RETENTION 2u
+
+typedef struct ob_mixer_desc {
+    uint32_t kind;            /* OB_MIXER_* */
+    uint32_t n_head, dim;     /* query/key dimensions per head (latent attention: the unrotated ones) */
+    uint32_t vdim;            /* value dimensions per head */
+    uint32_t rot_dim;         /* latent attention: rotated query/key dimensions per head, in addition to dim */
+    uint32_t kv_rank;         /* latent attention: size of the cached latent */
+    uint32_t window;          /* latent attention: a position sees itself and window - 1 before it; 0 = all before it */
+    uint32_t rot_dims;        /* entries that rotate, from the first: of q and k (retention), of the rot_dim part (latent attention) */
+    uint32_t rot_interleaved; /* 1: pairs (2i, 2i+1); 0: pairs (i, i + rot_dims/2) */
+    float scale;              /* latent attention: factor of the scores */
+    double rot_base;          /* pair i turns by position * rot_base^(-2i / rot_dims) */
+    const float *decay;       /* retention: [n_head] factor of the state per token */
+    ob_matrix_desc wq;        /* retention [n_head*dim]; latent attention [n_head*(dim+rot_dim)], per head unrotated then rotated */
+    ob_matrix_desc wk, wv;    /* retention [n_head*dim], [n_head*vdim] */
+    ob_matrix_desc w_gate;    /* retention [n_head*vdim] (silu of it scales the normed output); latent attention [n_head] (sigmoid of it scales a head) */
+    ob_matrix_desc w_dkv;     /* latent attention [kv_rank+rot_dim]: latent, then the rotated key part all heads share */
+    const float *kv_norm;     /* latent attention [kv_rank]: RMS-norm weight of the latent */
+    ob_matrix_desc w_uk, w_uv; /* latent attention [n_head*dim], [n_head*vdim] from kv_rank */
+    ob_matrix_desc wo;        /* [n_head*vdim -> n_embd] */
+} ob_mixer_desc;
+
+typedef struct ob_block_desc {
+    float norm_gain;
+    ob_mixer_desc mixer;
+    uint32_t n_ff;            /* 0: no feed-forward */
+    float glu_limit, glu_alpha; /* g = min(gate, limit), u = clamp(up, -limit, limit); g * sigmoid(alpha g) * (u + 1) */
+    ob_matrix_desc w_gate, w_up, w_down;
+    ob_matrix_desc side_gate, side_proj; /* per-layer token input (side_dim > 0): y = side_proj (gelu_tanh(side_gate x) * e), x += y / rms(y) * side_norm */
+    const float *side_norm;   /* [n_embd] */
+} ob_block_desc;
+
+typedef struct ob_layered_desc {
+    uint32_t n_vocab, n_embd, n_layer;
+    uint32_t side_dim;         /* per-layer token input: entries per layer in a row of side_embd; 0 = none */
+    float rms_eps, final_gain;
+    uint32_t compute_f32;      /* 0: bfloat16 activations and cache, fp32 accumulation; 1: fp32 throughout */
+    uint32_t max_seq_len, max_batch_tokens;
+    uint64_t kv_pool_tokens;   /* 0 = max_seq_len */
+    uint32_t n_state_slots;    /* sequences that can hold recurrent state at a time; 0 = 64.  Unused without recurrent layers */
+    ob_matrix_desc token_embd; /* [n_vocab] */
+    ob_matrix_desc side_embd;  /* [n_vocab][n_layer * side_dim] */
+    ob_matrix_desc output;     /* [n_vocab] */
+    const ob_block_desc *layers;
+} ob_layered_desc;
+
 /* ------------------------------------------------- GGUF files
  * GgufFile::open (src/gguf.rs:206-275): header, typed metadata, tensor table; the file is mapped read-only and the
  * tensor data pointers below point into the mapping (valid until ob_gguf_close).  Works without a GPU.  A failed call
@@ -286,6 +340,7 @@ int ob_gguf_model_desc(ob_gguf *g, ob_model_desc *desc);
 /* Stands in for LlamaModel::load_with_backend (E/arch/llama.rs:125-230) on the device side:
  * uploads (and shards) every tensor, sizes scratch, builds the RoPE table. */
 int ob_model_create(ob_ctx *ctx, const ob_model_desc *desc, ob_model **out);
+int ob_layered_model_create(ob_ctx *ctx, const ob_layered_desc *desc, ob_model **out);
 void ob_model_destroy(ob_model *model);
 
 /* ModelForward::new_kv_cache (E/arch/llama.rs:1002-1005): an empty per-sequence cache of fp16
@@ -301,15 +356,20 @@ uint32_t ob_kv_len(const ob_kv *kv);
 uint32_t ob_kv_pages(const ob_kv *kv);              /* pages this cache holds now */
 uint32_t ob_model_pool_pages(const ob_model *model); /* pages in the model's KV pool */
 uint32_t ob_model_free_pages(const ob_model *model); /* of which no cache holds */
+uint32_t ob_model_free_slots(const ob_model *model); /* state slots no sequence holds (models with recurrent layers) */
 uint32_t ob_model_n_vocab(const ob_model *model);
 uint32_t ob_model_tp_size(const ob_model *model);    /* 1 for a single-GPU model */
 ob_ctx *ob_model_ctx(const ob_model *model);
-/* KvCache::truncate (E/kv_cache.rs:496-511): roll back to new_len positions. */
+/* KvCache::truncate (E/kv_cache.rs:496-511): roll back to new_len positions.  A sequence of a model with recurrent layers can
+ * only be emptied (new_len 0); OB_ERR_UNSUPPORTED otherwise. */
 int ob_kv_truncate(ob_kv *kv, uint32_t new_len);
-/* Test hook: reads positions [pos0, pos0+n) of one layer back as f32 [n][n_head_kv*head_dim]. */
+/* Test hook: reads positions [pos0, pos0+n) of one layer back as f32 [n][n_head_kv*head_dim]; a latent-attention layer gives
+ * [n][kv_rank] in k_out and the rotated key part [n][rot_dim] in v_out. */
 int ob_kv_read(ob_kv *kv, uint32_t layer, uint32_t pos0, uint32_t n, float *k_out, float *v_out);
+/* Test hook: the recurrent state of one layer, f32 [n_head][dim][vdim]. */
+int ob_state_read(ob_kv *kv, uint32_t layer, float *out);
 /* KvCache::copy_prefix_from (E/kv_cache.rs:1079-1100): makes dst (empty) hold src's first n positions, by a
- * device-side copy of the pages.  Both caches belong to the same model. */
+ * device-side copy of the pages.  Both caches belong to the same model.  With recurrent layers n must be all of src. */
 int ob_kv_copy_prefix(ob_kv *dst, const ob_kv *src, uint32_t n);
 
 typedef struct ob_greedy { /* GpuArgmaxSampleInput, B/vulkan.rs:6219-6241 */
@@ -329,6 +389,12 @@ typedef struct ob_greedy { /* GpuArgmaxSampleInput, B/vulkan.rs:6219-6241 */
 int ob_forward(ob_model *model, ob_kv *const *kvs, const uint32_t *tokens, const uint32_t *n_tokens,
                const uint32_t *start_pos, uint32_t n_seq, const ob_greedy *greedy,
                uint32_t *out_token, float *out_logits);
+
+/* ob_forward with logits of any of the call's tokens: rows [n_rows] are ascending numbers into the concatenated tokens,
+ * out_logits [n_rows][n_vocab].  Models given as a list of layers run all sequences of the call as one batch, whole prompts,
+ * portions and single tokens side by side; the Llama graph runs them one after the other, as ob_forward does. */
+int ob_forward_rows(ob_model *model, ob_kv *const *kvs, const uint32_t *tokens, const uint32_t *n_tokens,
+                    const uint32_t *start_pos, uint32_t n_seq, const uint32_t *rows, uint32_t n_rows, float *out_logits);
 
 /* One greedy decode step of a single sequence replayed from a captured CUDA graph:
  * the record_decode_chain path (E/arch/llama.rs:302-473), one submission per token and one
@@ -426,6 +492,10 @@ int ob_slot_prefill(ob_slot_pool *pool, uint32_t slot_id, const uint32_t *tokens
  * be NULL (plain argmax); its n_recent[0] ids of `recent` are this sequence's penalty window.  A failed batch fails every
  * member with the same status. */
 int ob_slot_decode(ob_slot_pool *pool, uint32_t slot_id, uint32_t token, const ob_greedy *greedy, uint32_t *out_token, float *out_logits);
+/* One ob_forward_rows call over held slots: slot_ids[i] runs its next n_tokens[i] tokens, all of them in one batch.  rows and
+ * out_logits as in ob_forward_rows. */
+int ob_slot_forward(ob_slot_pool *pool, const uint32_t *slot_ids, uint32_t n_slots, const uint32_t *tokens, const uint32_t *n_tokens,
+                    const uint32_t *rows, uint32_t n_rows, float *out_logits);
 int ob_slot_truncate(ob_slot_pool *pool, uint32_t slot_id, uint32_t new_len);
 uint32_t ob_slot_len(const ob_slot_pool *pool, uint32_t slot_id);
 ob_kv *ob_slot_kv(ob_slot_pool *pool, uint32_t slot_id);

@@ -166,6 +166,10 @@ class LlamaModel {
     LlamaModel(CudaBackend &be, const ob_model_desc &desc) : ctx_(be.raw()) {
         if (ob_model_create(ctx_, &desc, &m_) != OB_OK) throw std::runtime_error(ob_last_error(ctx_));
     }
+    // a model given as a list of layers; every other member is the same
+    LlamaModel(CudaBackend &be, const ob_layered_desc &desc) : ctx_(be.raw()) {
+        if (ob_layered_model_create(ctx_, &desc, &m_) != OB_OK) throw std::runtime_error(ob_last_error(ctx_));
+    }
     LlamaModel(LlamaModel &&o) noexcept : ctx_(o.ctx_), m_(o.m_) { o.m_ = nullptr; }
     LlamaModel(const LlamaModel &) = delete;
     ~LlamaModel() {
@@ -206,6 +210,21 @@ class LlamaModel {
         check(ob_forward(m_, kvs.data(), tokens.data(), ones.data(), start.data(), n, nullptr, out.data(), nullptr));
         return out;
     }
+    // the next tokens of several sequences in one call; logits [rows][n_vocab] of the tokens numbered in `rows`
+    std::vector<float> forward_rows(const std::vector<KvCache *> &caches, const std::vector<std::vector<uint32_t>> &tokens, const std::vector<uint32_t> &rows) {
+        const uint32_t n = (uint32_t)caches.size();
+        std::vector<ob_kv *> kvs(n);
+        std::vector<uint32_t> flat, count(n), start(n);
+        for (uint32_t i = 0; i < n; ++i) {
+            kvs[i] = caches[i]->raw();
+            start[i] = caches[i]->len();
+            count[i] = (uint32_t)tokens[i].size();
+            flat.insert(flat.end(), tokens[i].begin(), tokens[i].end());
+        }
+        std::vector<float> out(rows.size() * ob_model_n_vocab(m_));
+        check(ob_forward_rows(m_, kvs.data(), flat.data(), count.data(), start.data(), n, rows.data(), (uint32_t)rows.size(), out.data()));
+        return out;
+    }
     // record_decode_chain + argmax (arch/llama.rs:302-473): one captured graph per token
     uint32_t decode_greedy(KvCache &cache, uint32_t token) {
         uint32_t out = 0;
@@ -223,6 +242,7 @@ class LlamaModel {
     ob_ctx *ctx_;
     ob_model *m_ = nullptr;
 };
+using Model = LlamaModel;  // whichever description it was made from
 
 // SlotPool (engine/scheduler.rs:36-317) with the decode window of BatchCoordinator (engine/batch.rs:184-324).  One thread per
 // request: acquire, prefill, decode per token, let the guard go.

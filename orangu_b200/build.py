@@ -20,7 +20,9 @@ OBJDIR = os.path.join(LIBDIR, "obj")
 LIB = os.path.join(LIBDIR, "liborangu_b200.so")
 SYNTH_LIB = os.path.join(LIBDIR, "libob_synth.so")
 
-CU_SOURCES = ["formats.cu", "act_quant.cu", "gemv.cu", "glue.cu", "attention.cu", "api.cu", "model.cu", "tp.cu", "noalloc.cu", "stream_gemv.cu", "layer_stream.cu", "gemm_mma.cu", "gemm_tc5.cu", "gguf.cu", "sched.cu", "q5k.cu"]
+CU_SOURCES = ["formats.cu", "act_quant.cu", "gemv.cu", "glue.cu", "attention.cu", "api.cu", "model.cu", "tp.cu", "noalloc.cu", "stream_gemv.cu", "layer_stream.cu", "gemm_mma.cu", "gemm_tc5.cu", "gguf.cu", "sched.cu", "q5k.cu",
+              "linear.cu", "mixers.cu", "layered.cu"]
+FMA_SOURCES = {"linear.cu", "mixers.cu", "layered.cu"}  # no CPU arithmetic to reproduce: the compiler may fuse
 NVCC_FLAGS = [
     "-gencode", "arch=compute_100a,code=sm_100a", "-lineinfo", "-O3", "-std=c++17",
     # The reproduced arithmetic never fuses a*b+c; FMAs are written out where wanted.
@@ -67,7 +69,8 @@ def build_cuda(force: bool = False, verbose: bool = False) -> str:
 
     def compile_one(job):
         s, o = job
-        cmd = [nvcc, *NVCC_FLAGS, "-c", s, "-o", o]
+        flags = [f for f in NVCC_FLAGS if not (f == "-fmad=false" and os.path.basename(s) in FMA_SOURCES)]
+        cmd = [nvcc, *flags, "-c", s, "-o", o]
         if verbose:
             cmd.insert(1, "-Xptxas=-v")
         r = subprocess.run(cmd, capture_output=True, text=True)

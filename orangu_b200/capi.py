@@ -37,6 +37,27 @@ class ModelDesc(C.Structure):
         ("rope_freqs", C.c_void_p), ("tp_presliced", C.c_uint32), ("rope_neox", C.c_uint32)]
 
 
+TYPE_BF16 = 30
+MIXER_LATENT_ATTENTION, MIXER_RETENTION = 1, 2
+
+
+class MixerDesc(C.Structure):
+    _fields_ = [(n, C.c_uint32) for n in ("kind", "n_head", "dim", "vdim", "rot_dim", "kv_rank", "window", "rot_dims", "rot_interleaved")] + [
+        ("scale", C.c_float), ("rot_base", C.c_double), ("decay", C.c_void_p)] + [
+        (n, MatrixDesc) for n in ("wq", "wk", "wv", "w_gate", "w_dkv")] + [("kv_norm", C.c_void_p)] + [(n, MatrixDesc) for n in ("w_uk", "w_uv", "wo")]
+
+
+class BlockDesc(C.Structure):
+    _fields_ = [("norm_gain", C.c_float), ("mixer", MixerDesc), ("n_ff", C.c_uint32), ("glu_limit", C.c_float), ("glu_alpha", C.c_float)] + [
+        (n, MatrixDesc) for n in ("w_gate", "w_up", "w_down", "side_gate", "side_proj")] + [("side_norm", C.c_void_p)]
+
+
+class LayeredDesc(C.Structure):
+    _fields_ = [(n, C.c_uint32) for n in ("n_vocab", "n_embd", "n_layer", "side_dim")] + [("rms_eps", C.c_float), ("final_gain", C.c_float)] + [
+        (n, C.c_uint32) for n in ("compute_f32", "max_seq_len", "max_batch_tokens")] + [("kv_pool_tokens", C.c_uint64), ("n_state_slots", C.c_uint32)] + [
+        (n, MatrixDesc) for n in ("token_embd", "side_embd", "output")] + [("layers", C.POINTER(BlockDesc))]
+
+
 class MatmulOpC(C.Structure):
     _fields_ = [("x", C.c_void_p), ("n_tokens", C.c_uint32), ("w", C.c_void_p), ("y", C.c_void_p)]
 
@@ -90,6 +111,7 @@ SIGNATURES = {
     "ob_attention_decode_static": (_i32, [_vp, _vp, _vp, _vp, _vp, _u32, _u32, _u32, _u32, _f32, _vp, _vp]),
     "ob_argmax": (_i32, [_vp, _vp, _u32, _vp, _u32, _u32, _f32, _vp]),
     "ob_model_create": (_i32, [_vp, C.POINTER(ModelDesc), _PP]),
+    "ob_layered_model_create": (_i32, [_vp, C.POINTER(LayeredDesc), _PP]),
     "ob_model_destroy": (None, [_vp]),
     "ob_kv_create": (_i32, [_vp, _u32, _PP]),
     "ob_kv_create_paged": (_i32, [_vp, _u32, _PP]),
@@ -97,15 +119,18 @@ SIGNATURES = {
     "ob_kv_pages": (_u32, [_vp]),
     "ob_model_pool_pages": (_u32, [_vp]),
     "ob_model_free_pages": (_u32, [_vp]),
+    "ob_model_free_slots": (_u32, [_vp]),
     "ob_model_n_vocab": (_u32, [_vp]),
     "ob_model_tp_size": (_u32, [_vp]),
     "ob_model_ctx": (_vp, [_vp]),
     "ob_kv_len": (_u32, [_vp]),
     "ob_kv_truncate": (_i32, [_vp, _u32]),
     "ob_kv_read": (_i32, [_vp, _u32, _u32, _u32, _vp, _vp]),
+    "ob_state_read": (_i32, [_vp, _u32, _vp]),
     "ob_kv_copy_prefix": (_i32, [_vp, _vp, _u32]),
     "ob_profile_gemv": (_i32, [_vp, _u32, _u32, _u32, _vp, _vp, _vp]),
     "ob_forward": (_i32, [_vp, _vp, _vp, _vp, _vp, _u32, _vp, _vp, _vp]),
+    "ob_forward_rows": (_i32, [_vp, _vp, _vp, _vp, _vp, _u32, _vp, _u32, _vp]),
     "ob_decode_greedy": (_i32, [_vp, _vp, _u32, _vp]),
     "ob_decode_loop": (_i32, [_vp, _vp, _vp, _u32, _u32, _vp]),
     "ob_last_hidden": (_i32, [_vp, _u32, _vp]),
@@ -122,6 +147,7 @@ SIGNATURES = {
     "ob_slot_release": (_i32, [_vp, _u32]),
     "ob_slot_prefill": (_i32, [_vp, _u32, _vp, _u32, _vp, _vp]),
     "ob_slot_decode": (_i32, [_vp, _u32, _u32, _vp, _vp, _vp]),
+    "ob_slot_forward": (_i32, [_vp, _vp, _u32, _vp, _vp, _vp, _u32, _vp]),
     "ob_slot_truncate": (_i32, [_vp, _u32, _u32]),
     "ob_slot_len": (_u32, [_vp, _u32]),
     "ob_slot_kv": (_vp, [_vp, _u32]),

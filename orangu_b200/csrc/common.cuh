@@ -123,6 +123,10 @@ __host__ __device__ inline uint32_t block_bytes_gguf(uint32_t type) {
     return type == TYPE_Q8_0 ? 34u : type == TYPE_Q4_K ? 144u : type == TYPE_Q5_K ? 176u : type == TYPE_Q5_0 ? 22u : is_sym32_source(type) ? 18u : 210u;
 }
 
+struct RowSpan {  // consecutive rows of a step that belong to one sequence, in position order
+    uint32_t row0, n;
+};
+
 // Quantized activations of one token row, natural element order.
 //   q     int8  [in_dim]
 //   d     f32   [in_dim/256] (K types) or [in_dim/32] (Q8_0)

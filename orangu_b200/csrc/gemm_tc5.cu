@@ -13,12 +13,9 @@
 // 32 * (w / 4) ..), warp 8 lane 0 issues the TMA loads, warp 9 allocates tensor memory and its lane 0 issues the MMAs.
 // Stages and accumulator halves are handed over through mbarriers; every wait is bounded -- a wait that runs out sets a
 // status word, makes all roles leave their loops, and the CTA frees its tensor memory and returns.
-#include <atomic>
-
-#include <cuda.h>  // CUtensorMap and its enums; cuTensorMapEncodeTiled is looked up through the runtime, libcuda is not linked
-
 #include "common.cuh"
 #include "kernels.h"
+#include "tc5_common.cuh"
 
 namespace ob {
 
@@ -28,55 +25,6 @@ constexpr int TC_M = 128, TC_N = 64;
 constexpr int TC_EPI_WARPS = 8;
 constexpr int TC_TMA_WARP = 8, TC_MMA_WARP = 9;
 constexpr int TC_THREADS = 10 * 32;
-constexpr uint32_t TC_POLL_LIMIT = 1u << 22;  // polls of one wait before it gives up (tens of milliseconds)
-
-__device__ uint32_t g_tc5_status;  // set to 1 when a wait ran out
-std::atomic<bool> g_tc5_launched{false};  // host: a kernel of this file has been launched since the status was last read
-
-__device__ __forceinline__ uint32_t smem_u32(const void *p) { return (uint32_t)__cvta_generic_to_shared(p); }
-
-// ---- mbarrier ------------------------------------------------------------------------------------------------------
-__device__ __forceinline__ void mbar_init(uint32_t bar, uint32_t count) { asm volatile("mbarrier.init.shared::cta.b64 [%0], %1;" ::"r"(bar), "r"(count) : "memory"); }
-__device__ __forceinline__ void mbar_arrive(uint32_t bar) { asm volatile("mbarrier.arrive.shared::cta.b64 _, [%0];" ::"r"(bar) : "memory"); }
-__device__ __forceinline__ void mbar_expect_tx(uint32_t bar, uint32_t bytes) {
-    asm volatile("mbarrier.arrive.expect_tx.shared::cta.b64 _, [%0], %1;" ::"r"(bar), "r"(bytes) : "memory");
-}
-__device__ __forceinline__ bool mbar_try(uint32_t bar, uint32_t parity) {
-    uint32_t ok;
-    asm volatile("{\n\t.reg .pred p;\n\tmbarrier.try_wait.parity.shared::cta.b64 p, [%1], %2;\n\tselp.u32 %0, 1, 0, p;\n\t}" : "=r"(ok) : "r"(bar), "r"(parity) : "memory");
-    return ok != 0;
-}
-// False when the wait was abandoned: this one ran out of polls, or another role's did (*abort is then set).
-__device__ __forceinline__ bool mbar_wait(uint32_t bar, uint32_t parity, volatile uint32_t *abort) {
-    for (uint32_t i = 0; i < TC_POLL_LIMIT; ++i) {
-        if (mbar_try(bar, parity)) return true;
-        if ((i & 63u) == 63u && *abort) return false;
-    }
-    *abort = 1u;
-    g_tc5_status = 1u;
-    return false;
-}
-
-// ---- TMA -----------------------------------------------------------------------------------------------------------
-// Tile at (x, y) of the tensor `tm` describes -> shared memory; completion counts on `bar`.  x * element size must be a
-// multiple of 16 bytes (all callers pass multiples of 128 bytes or of four floats).
-__device__ __forceinline__ void tma_load_2d(uint32_t dst, const CUtensorMap *tm, int32_t x, int32_t y, uint32_t bar) {
-    asm volatile("cp.async.bulk.tensor.2d.shared::cluster.global.mbarrier::complete_tx::bytes [%0], [%1, {%2, %3}], [%4];" ::"r"(dst),
-                 "l"(reinterpret_cast<uint64_t>(tm)), "r"(x), "r"(y), "r"(bar)
-                 : "memory");
-}
-
-// ---- tensor memory and tcgen05 -----------------------------------------------------------------------------------------
-__device__ __forceinline__ void tmem_alloc(uint32_t slot, uint32_t cols) {  // one whole warp
-    asm volatile("tcgen05.alloc.cta_group::1.sync.aligned.shared::cta.b32 [%0], %1;" ::"r"(slot), "r"(cols) : "memory");
-    asm volatile("tcgen05.relinquish_alloc_permit.cta_group::1.sync.aligned;" ::: "memory");
-}
-__device__ __forceinline__ void tmem_dealloc(uint32_t taddr, uint32_t cols) {  // the same warp
-    asm volatile("tcgen05.dealloc.cta_group::1.sync.aligned.b32 %0, %1;" ::"r"(taddr), "r"(cols) : "memory");
-}
-__device__ __forceinline__ void tc_fence_before() { asm volatile("tcgen05.fence::before_thread_sync;" ::: "memory"); }
-__device__ __forceinline__ void tc_fence_after() { asm volatile("tcgen05.fence::after_thread_sync;" ::: "memory"); }
-
 // D (tensor memory, int32, 128 lanes x N columns) [+]= A (128 x 32 int8, K-major) * B (N x 32 int8, K-major)^T
 __device__ __forceinline__ void umma_i8(uint32_t d_tmem, uint64_t a_desc, uint64_t b_desc, uint32_t idesc, uint32_t accumulate) {
     asm volatile(
@@ -84,36 +32,6 @@ __device__ __forceinline__ void umma_i8(uint32_t d_tmem, uint64_t a_desc, uint64
         "tcgen05.mma.cta_group::1.kind::i8 [%0], %1, %2, %3, p;\n\t}" ::"r"(d_tmem),
         "l"(a_desc), "l"(b_desc), "r"(idesc), "r"(accumulate)
         : "memory");
-}
-// All MMAs this thread has issued so far arrive on `bar` when they have completed.
-__device__ __forceinline__ void umma_commit(uint32_t bar) {
-    asm volatile("tcgen05.commit.cta_group::1.mbarrier::arrive::one.shared::cluster.b64 [%0];" ::"r"(bar) : "memory");
-}
-// This warp's 32 lanes x 32 consecutive columns: thread i gets lane i's words.
-__device__ __forceinline__ void tmem_ld32(uint32_t taddr, uint32_t (&r)[32]) {
-    asm volatile(
-        "tcgen05.ld.sync.aligned.32x32b.x32.b32 {%0, %1, %2, %3, %4, %5, %6, %7, %8, %9, %10, %11, %12, %13, %14, %15, %16, %17, %18, %19, %20, %21, %22, "
-        "%23, %24, %25, %26, %27, %28, %29, %30, %31}, [%32];"
-        : "=r"(r[0]), "=r"(r[1]), "=r"(r[2]), "=r"(r[3]), "=r"(r[4]), "=r"(r[5]), "=r"(r[6]), "=r"(r[7]), "=r"(r[8]), "=r"(r[9]), "=r"(r[10]), "=r"(r[11]),
-          "=r"(r[12]), "=r"(r[13]), "=r"(r[14]), "=r"(r[15]), "=r"(r[16]), "=r"(r[17]), "=r"(r[18]), "=r"(r[19]), "=r"(r[20]), "=r"(r[21]), "=r"(r[22]),
-          "=r"(r[23]), "=r"(r[24]), "=r"(r[25]), "=r"(r[26]), "=r"(r[27]), "=r"(r[28]), "=r"(r[29]), "=r"(r[30]), "=r"(r[31])
-        : "r"(taddr)
-        : "memory");
-}
-__device__ __forceinline__ void tmem_ld16(uint32_t taddr, uint32_t (&r)[16]) {
-    asm volatile("tcgen05.ld.sync.aligned.32x32b.x16.b32 {%0, %1, %2, %3, %4, %5, %6, %7, %8, %9, %10, %11, %12, %13, %14, %15}, [%16];"
-                 : "=r"(r[0]), "=r"(r[1]), "=r"(r[2]), "=r"(r[3]), "=r"(r[4]), "=r"(r[5]), "=r"(r[6]), "=r"(r[7]), "=r"(r[8]), "=r"(r[9]), "=r"(r[10]), "=r"(r[11]),
-                   "=r"(r[12]), "=r"(r[13]), "=r"(r[14]), "=r"(r[15])
-                 : "r"(taddr)
-                 : "memory");
-}
-__device__ __forceinline__ void tmem_ld_wait() { asm volatile("tcgen05.wait::ld.sync.aligned;" ::: "memory"); }
-
-// Shared-memory matrix descriptor of a K-major tile in the 128-byte swizzle: rows of 128 bytes, groups of eight rows 1024
-// bytes apart, tile base 1024-byte aligned.  A K = 32 step inside the 128-byte row advances the start address by 32 bytes.
-__device__ __forceinline__ uint64_t umma_desc_sw128(uint32_t saddr) {
-    return (uint64_t)((saddr >> 4) & 0x3fffu) | (1ull << 16) /* leading byte offset: unused with a swizzle */ | (64ull << 32) /* 1024 B between row groups */ |
-           (1ull << 46) /* descriptor version of this architecture */ | (2ull << 61) /* 128-byte swizzle */;
 }
 // Instruction descriptor: int32 accumulator, A and B signed (1) or unsigned (0) 8-bit, both K-major, N columns, M = 128.
 __host__ __device__ constexpr uint32_t umma_idesc_i8(uint32_t a_signed, uint32_t b_signed, uint32_t n) {
@@ -511,31 +429,6 @@ gemm_tc5_q4k_kernel(const __grid_constant__ CUtensorMap tm_raw0, const __grid_co
     if (warp == K4_MMA_WARP) tmem_dealloc(tmem, 512);
 }
 
-// ---- host ------------------------------------------------------------------------------------------------------------
-using EncodeTiled = CUresult (*)(CUtensorMap *, CUtensorMapDataType, cuuint32_t, void *, const cuuint64_t *, const cuuint64_t *, const cuuint32_t *, const cuuint32_t *,
-                                 CUtensorMapInterleave, CUtensorMapSwizzle, CUtensorMapL2promotion, CUtensorMapFloatOOBfill);
-
-EncodeTiled encode_fn() {
-    static EncodeTiled fn = [] {
-        void *p = nullptr;
-        cudaDriverEntryPointQueryResult q = cudaDriverEntryPointSymbolNotFound;
-        if (cudaGetDriverEntryPoint("cuTensorMapEncodeTiled", &p, cudaEnableDefault, &q) != cudaSuccess || q != cudaDriverEntryPointSuccess) p = nullptr;
-        return reinterpret_cast<EncodeTiled>(p);
-    }();
-    return fn;
-}
-
-// 2-D tensor of `rows` rows of `cols` elements, rows `pitch` bytes apart, read in boxes of box_cols x box_rows.
-bool make_map_2d(CUtensorMap *tm, CUtensorMapDataType type, uint32_t elem_bytes, const void *base, uint64_t cols, uint64_t rows, uint64_t pitch, uint32_t box_cols,
-                 uint32_t box_rows, CUtensorMapSwizzle swz) {
-    EncodeTiled fn = encode_fn();
-    if (!fn || (reinterpret_cast<uintptr_t>(base) & 15) || (pitch & 15) || ((uint64_t)box_cols * elem_bytes & 15)) return false;
-    const cuuint64_t dims[2] = {cols, rows}, strides[1] = {pitch};
-    const cuuint32_t box[2] = {box_cols, box_rows}, estr[2] = {1, 1};
-    return fn(tm, type, 2, const_cast<void *>(base), dims, strides, box, estr, CU_TENSOR_MAP_INTERLEAVE_NONE, swz, CU_TENSOR_MAP_L2_PROMOTION_L2_128B,
-              CU_TENSOR_MAP_FLOAT_OOB_FILL_NONE) == CUDA_SUCCESS;
-}
-
 }  // namespace
 
 bool gemm_tc5_supported(const GemvArgs &a) {
@@ -625,16 +518,6 @@ bool launch_gemm_tc5(const GemvArgs &a, int sm_count, cudaStream_t st) {
     return true;
 }
 
-// 1 when a bounded wait of one of these kernels ran out since the last call (and clears it).  Synchronises with the device.
-int gemm_tc5_take_status() {
-    if (!g_tc5_launched.exchange(false)) return 0;
-    uint32_t v = 0;
-    if (cudaMemcpyFromSymbol(&v, g_tc5_status, 4) != cudaSuccess) return 0;
-    if (v) {
-        const uint32_t z = 0;
-        cudaMemcpyToSymbol(g_tc5_status, &z, 4);
-    }
-    return (int)v;
-}
+int gemm_tc5_take_status() { return tc5_take_status(); }
 
 }  // namespace ob

@@ -1,0 +1,574 @@
+// Models given as a list of layers (ob_layered_desc): weights as padded bfloat16 matrices, a latent-cache pool per
+// latent-attention layer on the model's pages, a state pool per recurrent layer on the model's slots, and the step.
+//
+// A layer is a short chain of launches.  All products that read the normed input are one matrix, its feed-forward rows
+// interleaved (gate, up) so that the activation is the epilogue; the mixer's output and the feed-forward's activations sit side
+// by side in one row, so the two output products and the residual addition are one product too.
+//   in      [mixer projections | gate/up]  <- h
+//   mixer   latent attention: prep (norm, rotate, append), absorbed query (per head), attention, value up-projection with gate
+//           retention: rotate, recurrence, norm with gate
+//   out     x += [W_o | W_down] [mixer | ff]
+//   side    gate (gelu, token entry), proj, then norm + residual + the next layer's norm in one kernel
+#include <math.h>
+#include <string.h>
+
+#include <algorithm>
+#include <cmath>
+#include <memory>
+
+#include "model.h"
+
+namespace {
+
+constexpr uint32_t round_up(uint32_t v, uint32_t m) { return (v + m - 1) / m * m; }
+
+struct Dense {  // rows x kp bfloat16 on the device
+    __nv_bfloat16 *w = nullptr;
+    uint32_t rows = 0, kp = 0;
+};
+
+struct LayerPlan {
+    ob_mixer_desc mx{};  // sizes and constants only
+    float norm_gain = 0.0f, glu_limit = 0.0f, glu_alpha = 0.0f;
+    uint32_t n_ff = 0;
+    Dense in, out, side_gate, side_proj;
+    float *side_norm = nullptr;
+    Rot rot{};
+    // rows of `in`: [activations (unrotated queries) | f32 projections | gate/up]
+    uint32_t act_rows = 0, f32_row0 = 0, f32_rows = 0, glu_row0 = 0, mix_cols = 0;  // mix_cols: columns of the mixer in the out product's input
+    // latent attention
+    Dense uk, uv;        // per head [kv_rank <- dim], [vdim <- kv_rank]
+    uint32_t dim_p = 0, kv_p = 0, dq = 0, kv_w = 0;
+    float *kv_norm = nullptr;
+    void *pool = nullptr;
+    // retention
+    float *decay = nullptr, *state = nullptr;
+};
+
+// A zero-padded bfloat16 matrix put together on the host from parts of others.
+struct HostDense {
+    uint32_t rows, kp;
+    std::vector<uint16_t> v;
+    HostDense(uint32_t r, uint32_t k) : rows(r), kp(k), v((size_t)r * k, 0) {}
+    void copy(uint32_t row, uint32_t col, const ob_matrix_desc &src, uint32_t src_row) {
+        memcpy(v.data() + (size_t)row * kp + col, src.data + (size_t)src_row * src.in_dim * 2, (size_t)src.in_dim * 2);
+    }
+};
+
+struct LayeredGraph : StepGraph {
+    ob_model *m = nullptr;
+    bool f32 = false, has_state = false;
+    uint32_t width = 0, h_pitch = 0, side_dim = 0, side_p = 0, y_pitch = 0, cat_pitch = 0;
+    float eps = 0.0f, final_gain = 0.0f;
+    std::vector<LayerPlan> L;
+    __nv_bfloat16 *embd = nullptr, *side_embd = nullptr;
+    Dense output;
+    void *h = nullptr, *xb = nullptr, *qn = nullptr, *q = nullptr, *o_lat = nullptr, *cat = nullptr, *sg = nullptr;
+    float *y = nullptr, *o_ret = nullptr, *sy = nullptr, *part = nullptr;
+    uint64_t part_cap = 0;
+    bool failed = false;  // a product could not be launched
+
+    size_t es() const { return f32 ? 4 : 2; }
+    bool recurrent() const override { return has_state; }
+    bool take_failure() override {
+        const bool f = failed;
+        failed = false;
+        return f;
+    }
+
+    void linear(const LinArgs &a, cudaStream_t st) {
+        if (!launch_linear(a, f32, m->ctx->sm_count, st)) failed = true;
+        m->ctx->launches++;
+    }
+    LinArgs product(const Dense &w, const void *x, uint32_t x_pitch, uint32_t T) const {
+        LinArgs a{};
+        a.w = w.w;
+        a.n_rows = w.rows;
+        a.kp = w.kp;
+        a.x = x;
+        a.x_pitch = x_pitch;
+        a.T = T;
+        a.n_batch = 1;
+        return a;
+    }
+    static void segment(LinArgs &a, uint32_t row0, uint32_t n, int epi, void *out, uint32_t pitch, uint32_t col0 = 0, uint32_t batch_cols = 0) {
+        if (n) a.seg[a.n_seg++] = LinSegment{row0, n, epi, out, pitch, col0, batch_cols};
+    }
+
+    void layers(uint32_t T, uint32_t n_seq, const RowSpan *spans, uint32_t max_pos, cudaStream_t st) override;
+    void head(const uint32_t *d_rows, uint32_t n, cudaStream_t st) override;
+    void latent(const LayerPlan &P, uint32_t T, uint32_t n_seq, const RowSpan *spans, bool single, uint32_t max_pos, cudaStream_t st);
+    void retention(const LayerPlan &P, uint32_t T, uint32_t n_seq, cudaStream_t st);
+    int copy_prefix(ob_kv *dst, const ob_kv *src, uint32_t n) override;
+    int read_pages(const ob_kv *kv, uint32_t layer, uint32_t pos0, uint32_t n, float *k_out, float *v_out) override;
+    int read_state(const ob_kv *kv, uint32_t layer, float *out) override;
+    size_t state_elems(const LayerPlan &P) const { return (size_t)P.mx.n_head * P.mx.dim * P.mx.vdim; }
+
+    int upload(const HostDense &src, Dense *out) {
+        int rc = dev_alloc(m, &out->w, src.v.size());
+        if (rc) return rc;
+        out->rows = src.rows;
+        out->kp = src.kp;
+        OB_CUDA(m->ctx, cudaMemcpy(out->w, src.v.data(), src.v.size() * 2, cudaMemcpyHostToDevice));
+        return OB_OK;
+    }
+    int scratch(void **p, size_t elems, size_t elem_bytes) {  // zeroed: padding columns stay finite
+        uint8_t *b = nullptr;
+        int rc = dev_alloc(m, &b, elems * elem_bytes);
+        if (rc) return rc;
+        OB_CUDA(m->ctx, cudaMemset(b, 0, std::max<size_t>(elems * elem_bytes, 16)));
+        *p = b;
+        return OB_OK;
+    }
+    int scratch_f32(float **p, size_t elems) {
+        void *v = nullptr;
+        int rc = scratch(&v, elems, 4);
+        *p = static_cast<float *>(v);
+        return rc;
+    }
+    int build(const ob_layered_desc &c);
+    int build_layer(const ob_block_desc &b, LayerPlan &P);
+};
+
+void LayeredGraph::latent(const LayerPlan &P, uint32_t T, uint32_t n_seq, const RowSpan *spans, bool single, uint32_t max_pos, cudaStream_t st) {
+    const MetaLayout ml(m->T);
+    const uint32_t H = P.mx.n_head;
+    LatentArgs a{};
+    a.y = y;
+    a.y_pitch = y_pitch;
+    a.n_head = H;
+    a.kv_rank = P.mx.kv_rank;
+    a.rot_dim = P.mx.rot_dim;
+    a.window = P.mx.window;
+    a.kv_p = P.kv_p;
+    a.dq = P.dq;
+    a.eps = eps;
+    a.scale = P.mx.scale;
+    a.kv_norm = P.kv_norm;
+    a.rot = P.rot;
+    a.q = q;
+    a.cache = P.pool;
+    a.o = o_lat;
+    a.o_head = P.kv_w;
+    a.part = part;
+    a.part_cap = part_cap;
+    a.T = T;
+    a.n_seq = n_seq;
+    a.spans = reinterpret_cast<const RowSpan *>(m->d_meta + ml.off_spans);
+    a.h_spans = spans;
+    a.single = single;
+    a.positions = reinterpret_cast<const uint32_t *>(m->d_meta + ml.off_positions);
+    a.tables = reinterpret_cast<const int32_t *const *>(m->d_meta + ml.off_tables);
+    a.max_pos = max_pos;
+    launch_latent_prep(a, f32, st);
+    LinArgs uk = product(P.uk, qn, H * P.dim_p, T);  // head h: its unrotated query through the key up-projection
+    uk.n_rows = P.uk.rows / H;
+    uk.n_batch = H;
+    uk.x_step = P.dim_p;
+    segment(uk, 0, P.mx.kv_rank, LE_ACT, q, H * P.dq, 0, P.dq);
+    linear(uk, st);
+    m->ctx->launches += 1 + launch_latent_attention(a, f32, m->ctx->sm_count, st);
+    LinArgs uv = product(P.uv, o_lat, H * P.kv_w, T);
+    uv.n_rows = P.uv.rows / H;
+    uv.n_batch = H;
+    uv.x_step = P.kv_w;
+    uv.gate = y + (size_t)H * P.mx.rot_dim + P.mx.kv_rank + P.mx.rot_dim;
+    uv.gate_pitch = y_pitch;
+    segment(uv, 0, P.mx.vdim, LE_GATED, cat, cat_pitch, 0, P.mx.vdim);
+    linear(uv, st);
+}
+
+void LayeredGraph::retention(const LayerPlan &P, uint32_t T, uint32_t n_seq, cudaStream_t st) {
+    const MetaLayout ml(m->T);
+    RetentionArgs a{};
+    a.y = y;
+    a.y_pitch = y_pitch;
+    a.n_head = P.mx.n_head;
+    a.dim = P.mx.dim;
+    a.vdim = P.mx.vdim;
+    a.eps = eps;
+    a.k_scale = 1.0f / sqrtf((float)P.mx.dim);
+    a.decay = P.decay;
+    a.rot = P.rot;
+    a.state = P.state;
+    a.o = o_ret;
+    a.out = cat;
+    a.out_pitch = cat_pitch;
+    a.T = T;
+    a.n_seq = n_seq;
+    a.spans = reinterpret_cast<const RowSpan *>(m->d_meta + ml.off_spans);
+    a.positions = reinterpret_cast<const uint32_t *>(m->d_meta + ml.off_positions);
+    a.slots = reinterpret_cast<const int32_t *>(m->d_meta + ml.off_slots);
+    m->ctx->launches += launch_retention(a, f32, m->ctx->sm_count, st);
+}
+
+void LayeredGraph::layers(uint32_t T, uint32_t n_seq, const RowSpan *spans, uint32_t max_pos, cudaStream_t st) {
+    const MetaLayout ml(m->T);
+    const uint32_t *tokens = reinterpret_cast<const uint32_t *>(m->d_meta + ml.off_tokens);
+    const bool single = n_seq == T;
+    launch_embed_bf16(embd, width, tokens, T, m->x, st);
+    launch_norm_scalar(m->x, width, nullptr, T, eps, L[0].norm_gain, h, h_pitch, f32, st);
+    m->ctx->launches += 2;
+    for (size_t li = 0; li < L.size(); ++li) {
+        const LayerPlan &P = L[li];
+        LinArgs in = product(P.in, h, h_pitch, T);
+        segment(in, 0, P.act_rows, LE_ACT, qn, P.act_rows);
+        segment(in, P.f32_row0, P.f32_rows, LE_F32, y, y_pitch);
+        segment(in, P.glu_row0, 2 * P.n_ff, LE_GLU, cat, cat_pitch, P.mix_cols);
+        in.glu_limit = P.glu_limit;
+        in.glu_alpha = P.glu_alpha;
+        linear(in, st);
+
+        if (P.mx.kind == OB_MIXER_LATENT_ATTENTION) latent(P, T, n_seq, spans, single, max_pos, st);
+        else retention(P, T, n_seq, st);
+
+        LinArgs out = product(P.out, cat, cat_pitch, T);
+        segment(out, 0, width, LE_RESIDUAL, m->x, width);
+        if (side_dim) {
+            out.out2 = xb;
+            out.out2_pitch = h_pitch;
+        }
+        linear(out, st);
+
+        const bool last = li + 1 == L.size();
+        const float gain = last ? 0.0f : L[li + 1].norm_gain;
+        if (side_dim) {
+            LinArgs g = product(P.side_gate, xb, h_pitch, T);
+            segment(g, 0, side_dim, LE_GELU_EMB, sg, side_p);
+            g.tokens = tokens;
+            g.emb = side_embd;
+            g.emb_pitch = (uint32_t)L.size() * side_dim;
+            g.emb_col0 = (uint32_t)li * side_dim;
+            linear(g, st);
+            LinArgs pr = product(P.side_proj, sg, side_p, T);
+            segment(pr, 0, width, LE_F32, sy, width);
+            linear(pr, st);
+            launch_side_finish(m->x, sy, P.side_norm, width, T, eps, gain, last ? nullptr : h, h_pitch, f32, st);
+            m->ctx->launches++;
+        } else if (!last) {
+            launch_norm_scalar(m->x, width, nullptr, T, eps, gain, h, h_pitch, f32, st);
+            m->ctx->launches++;
+        }
+    }
+}
+
+void LayeredGraph::head(const uint32_t *d_rows, uint32_t n, cudaStream_t st) {
+    launch_norm_scalar(m->x, width, d_rows, n, eps, final_gain, h, h_pitch, f32, st);
+    m->ctx->launches++;
+    LinArgs a = product(output, h, h_pitch, n);
+    segment(a, 0, m->cfg.n_vocab, LE_F32, m->logits, m->cfg.n_vocab);
+    linear(a, st);
+}
+
+int LayeredGraph::copy_prefix(ob_kv *dst, const ob_kv *src, uint32_t n) {
+    cudaStream_t st = m->ctx->stream;
+    for (const LayerPlan &P : L) {
+        if (P.pool) {
+            launch_copy_pages(P.pool, (uint64_t)KV_PAGE * P.dq * es(), src->d_table, dst->d_table, (n + KV_PAGE - 1) / KV_PAGE, st);
+            m->ctx->launches++;
+        } else if (P.state && src->slot >= 0 && dst->slot >= 0) {
+            const size_t e = state_elems(P);
+            OB_CUDA(m->ctx, cudaMemcpyAsync(P.state + (size_t)dst->slot * e, P.state + (size_t)src->slot * e, e * 4, cudaMemcpyDeviceToDevice, st));
+        }
+    }
+    return OB_OK;
+}
+
+int LayeredGraph::read_pages(const ob_kv *kv, uint32_t layer, uint32_t pos0, uint32_t n, float *k_out, float *v_out) {
+    const LayerPlan &P = L[layer];
+    if (!P.pool) return fail(m->ctx, OB_ERR_INVALID, "kv_read: the layer caches no positions");
+    std::vector<uint8_t> row(P.dq * es());
+    for (uint32_t i = 0; i < n; ++i) {
+        const uint32_t p = pos0 + i;
+        const uint8_t *src = static_cast<const uint8_t *>(P.pool) + ((size_t)kv->pages[p / KV_PAGE] * KV_PAGE + p % KV_PAGE) * row.size();
+        OB_CUDA(m->ctx, cudaMemcpy(row.data(), src, row.size(), cudaMemcpyDeviceToHost));
+        auto at = [&](uint32_t c) {
+            float v;
+            if (f32) {
+                memcpy(&v, row.data() + 4 * c, 4);
+            } else {
+                uint16_t b;
+                memcpy(&b, row.data() + 2 * c, 2);
+                const uint32_t u = (uint32_t)b << 16;
+                memcpy(&v, &u, 4);
+            }
+            return v;
+        };
+        for (uint32_t c = 0; c < P.mx.kv_rank; ++c) k_out[(size_t)i * P.mx.kv_rank + c] = at(c);
+        for (uint32_t c = 0; c < P.mx.rot_dim; ++c) v_out[(size_t)i * P.mx.rot_dim + c] = at(P.kv_p + c);
+    }
+    return OB_OK;
+}
+
+int LayeredGraph::read_state(const ob_kv *kv, uint32_t layer, float *out) {
+    if (layer >= L.size() || !L[layer].state) return fail(m->ctx, OB_ERR_INVALID, "state_read: the layer has no recurrent state");
+    const size_t e = state_elems(L[layer]);
+    OB_CUDA(m->ctx, cudaMemcpy(out, L[layer].state + (size_t)kv->slot * e, e * 4, cudaMemcpyDeviceToHost));
+    return OB_OK;
+}
+
+int LayeredGraph::build_layer(const ob_block_desc &b, LayerPlan &P) {
+    const ob_mixer_desc &x = b.mixer;
+    const bool latent = x.kind == OB_MIXER_LATENT_ATTENTION;
+    const uint32_t H = x.n_head;
+    int rc;
+    P.mx = x;
+    P.norm_gain = b.norm_gain;
+    P.n_ff = b.n_ff;
+    P.glu_limit = b.glu_limit;
+    P.glu_alpha = b.glu_alpha;
+    // ---- everything that reads the normed input
+    if (latent) {
+        P.dim_p = round_up(x.dim, LIN_K_ALIGN);
+        P.kv_p = round_up(x.kv_rank, 16);
+        P.dq = P.kv_p + round_up(x.rot_dim, 16);
+        P.kv_w = round_up(x.kv_rank, LIN_K_ALIGN);
+        P.act_rows = H * P.dim_p;
+        P.f32_rows = H * x.rot_dim + x.kv_rank + x.rot_dim + H;
+    } else {
+        P.f32_rows = H * (2 * x.dim + 2 * x.vdim);
+    }
+    P.f32_row0 = P.act_rows;
+    P.glu_row0 = P.f32_row0 + round_up(P.f32_rows, LIN_ROW_ALIGN);
+    HostDense in(P.glu_row0 + round_up(2 * b.n_ff, LIN_ROW_ALIGN), h_pitch);
+    uint32_t r = P.f32_row0;
+    auto rows = [&](const ob_matrix_desc &d) {
+        for (uint32_t i = 0; i < d.out_dim; ++i) in.copy(r++, 0, d, i);
+    };
+    if (latent) {
+        for (uint32_t hd = 0; hd < H; ++hd) {
+            for (uint32_t i = 0; i < x.dim; ++i) in.copy(hd * P.dim_p + i, 0, x.wq, hd * (x.dim + x.rot_dim) + i);
+            for (uint32_t i = 0; i < x.rot_dim; ++i) in.copy(r++, 0, x.wq, hd * (x.dim + x.rot_dim) + x.dim + i);
+        }
+        rows(x.w_dkv);
+        rows(x.w_gate);
+    } else {
+        rows(x.wq);
+        rows(x.wk);
+        rows(x.wv);
+        rows(x.w_gate);
+    }
+    for (uint32_t i = 0; i < b.n_ff; ++i) {
+        in.copy(P.glu_row0 + 2 * i, 0, b.w_gate, i);
+        in.copy(P.glu_row0 + 2 * i + 1, 0, b.w_up, i);
+    }
+    if ((rc = upload(in, &P.in))) return rc;
+    // ---- output products side by side
+    P.mix_cols = round_up(H * x.vdim, LIN_K_ALIGN);
+    HostDense out(round_up(width, LIN_ROW_ALIGN), P.mix_cols + round_up(b.n_ff, LIN_K_ALIGN));
+    for (uint32_t i = 0; i < width; ++i) {
+        out.copy(i, 0, x.wo, i);
+        if (b.n_ff) out.copy(i, P.mix_cols, b.w_down, i);
+    }
+    if ((rc = upload(out, &P.out))) return rc;
+    if (side_dim) {
+        HostDense g(round_up(side_dim, LIN_ROW_ALIGN), h_pitch), pr(round_up(width, LIN_ROW_ALIGN), side_p);
+        for (uint32_t i = 0; i < side_dim; ++i) g.copy(i, 0, b.side_gate, i);
+        for (uint32_t i = 0; i < width; ++i) pr.copy(i, 0, b.side_proj, i);
+        if ((rc = upload(g, &P.side_gate)) || (rc = upload(pr, &P.side_proj))) return rc;
+        if ((rc = upload_f32(m, b.side_norm, width, &P.side_norm))) return rc;
+    }
+    // ---- the mixer's own tensors
+    if (latent) {
+        const uint32_t kr = round_up(x.kv_rank, LIN_ROW_ALIGN), vr = round_up(x.vdim, LIN_ROW_ALIGN);
+        HostDense uk(H * kr, P.dim_p), uv(H * vr, P.kv_w);
+        const uint16_t *src = reinterpret_cast<const uint16_t *>(x.w_uk.data);
+        for (uint32_t hd = 0; hd < H; ++hd) {
+            for (uint32_t d = 0; d < x.dim; ++d)  // transposed: the query goes through it
+                for (uint32_t c = 0; c < x.kv_rank; ++c) uk.v[(size_t)(hd * kr + c) * P.dim_p + d] = src[(size_t)(hd * x.dim + d) * x.kv_rank + c];
+            for (uint32_t i = 0; i < x.vdim; ++i) uv.copy(hd * vr + i, 0, x.w_uv, hd * x.vdim + i);
+        }
+        if ((rc = upload(uk, &P.uk)) || (rc = upload(uv, &P.uv))) return rc;
+        if ((rc = upload_f32(m, x.kv_norm, x.kv_rank, &P.kv_norm))) return rc;
+        if ((rc = scratch(&P.pool, (size_t)m->pool_pages * KV_PAGE * P.dq, es()))) return rc;
+    } else {
+        if ((rc = upload_f32(m, x.decay, H, &P.decay))) return rc;
+        if ((rc = scratch_f32(&P.state, (size_t)m->n_state_slots * state_elems(P)))) return rc;
+        has_state = true;
+    }
+    OB_CUDA(m->ctx, cudaStreamSynchronize(m->ctx->stream));  // the host matrices end here
+    P.mx.decay = nullptr;
+    P.mx.kv_norm = nullptr;
+    return OB_OK;
+}
+
+int LayeredGraph::build(const ob_layered_desc &c) {
+    int rc;
+    const size_t T = m->T;
+    f32 = c.compute_f32 != 0;
+    width = c.n_embd;
+    h_pitch = round_up(width, LIN_K_ALIGN);
+    side_dim = c.side_dim;
+    side_p = round_up(side_dim, LIN_K_ALIGN);
+    eps = c.rms_eps;
+    final_gain = c.final_gain;
+    L.resize(c.n_layer);
+    std::map<std::pair<double, uint32_t>, float2 *> tables;
+    size_t act = 0, q_n = 0, o_n = 0, o_r = 0, kvp = 0, heads = 0;
+    for (uint32_t i = 0; i < c.n_layer; ++i) {
+        LayerPlan &P = L[i];
+        if ((rc = build_layer(c.layers[i], P))) return rc;
+        const uint32_t H = P.mx.n_head, half = P.mx.rot_dims / 2;
+        float2 *&tab = tables[{P.mx.rot_base, P.mx.rot_dims}];
+        if (!tab) {  // angles in double on the host: the table is exact to fp32 at any position
+            std::vector<float2> t((size_t)m->cfg.max_seq_len * half);
+            std::vector<double> f(half);
+            for (uint32_t k = 0; k < half; ++k) f[k] = pow(P.mx.rot_base, -2.0 * k / P.mx.rot_dims);
+            for (uint32_t p = 0; p < m->cfg.max_seq_len; ++p)
+                for (uint32_t k = 0; k < half; ++k) t[(size_t)p * half + k] = make_float2((float)cos(p * f[k]), (float)sin(p * f[k]));
+            if ((rc = dev_alloc(m, &tab, t.size()))) return rc;
+            OB_CUDA(m->ctx, cudaMemcpy(tab, t.data(), t.size() * sizeof(float2), cudaMemcpyHostToDevice));
+        }
+        P.rot = Rot{tab, P.mx.rot_dims, P.mx.rot_interleaved != 0};
+        act = std::max<size_t>(act, P.act_rows);
+        y_pitch = std::max(y_pitch, round_up(P.f32_rows, 4));
+        cat_pitch = std::max(cat_pitch, P.out.kp);
+        if (P.pool) {
+            q_n = std::max<size_t>(q_n, (size_t)H * P.dq);
+            o_n = std::max<size_t>(o_n, (size_t)H * P.kv_w);
+            kvp = std::max<size_t>(kvp, P.kv_p);
+            heads = std::max<size_t>(heads, H);
+        } else {
+            o_r = std::max<size_t>(o_r, (size_t)H * P.mx.vdim);
+        }
+    }
+    {
+        if ((rc = dev_alloc(m, &embd, (size_t)c.n_vocab * width))) return rc;
+        OB_CUDA(m->ctx, cudaMemcpy(embd, c.token_embd.data, (size_t)c.n_vocab * width * 2, cudaMemcpyHostToDevice));
+        if (side_dim) {
+            const size_t n = (size_t)c.n_vocab * c.n_layer * side_dim;
+            if ((rc = dev_alloc(m, &side_embd, n))) return rc;
+            OB_CUDA(m->ctx, cudaMemcpy(side_embd, c.side_embd.data, n * 2, cudaMemcpyHostToDevice));
+        }
+        HostDense o(round_up(c.n_vocab, LIN_ROW_ALIGN), h_pitch);
+        for (uint32_t i = 0; i < c.n_vocab; ++i) o.copy(i, 0, c.output, i);
+        if ((rc = upload(o, &output))) return rc;
+    }
+    if ((rc = scratch(&h, T * h_pitch, es())) || (rc = scratch(&xb, T * h_pitch, es())) || (rc = scratch(&cat, T * cat_pitch, es()))) return rc;
+    if ((rc = scratch(&qn, T * act, es())) || (rc = scratch(&q, T * q_n, es())) || (rc = scratch(&o_lat, T * o_n, es()))) return rc;
+    if ((rc = scratch_f32(&y, T * y_pitch)) || (rc = scratch_f32(&o_ret, T * o_r))) return rc;
+    if (side_dim && ((rc = scratch(&sg, T * side_p, es())) || (rc = scratch_f32(&sy, T * width)))) return rc;
+    if (q_n && !f32) {  // at most one CTA per SM, of 64 rows, writes partial results at a time (launch_latent_attention)
+        part_cap = ((uint64_t)m->ctx->sm_count * 64 + 64) * (kvp + 2);
+        if ((rc = scratch_f32(&part, part_cap))) return rc;
+    }
+    return OB_OK;
+}
+
+int check_dense(ob_ctx *ctx, const ob_matrix_desc &d, uint32_t in_dim, uint32_t out_dim, const std::string &name) {
+    if (!d.data) return fail(ctx, OB_ERR_INVALID, "layered model: " + name + " has no data");
+    if (d.ggml_type != OB_TYPE_BF16) return fail(ctx, OB_ERR_UNSUPPORTED, "layered model: " + name + " is not bfloat16");
+    if (d.in_dim != in_dim || d.out_dim != out_dim)
+        return fail(ctx, OB_ERR_INVALID, "layered model: " + name + " is [" + std::to_string(d.in_dim) + " -> " + std::to_string(d.out_dim) + "], expected [" +
+                                             std::to_string(in_dim) + " -> " + std::to_string(out_dim) + "]");
+    return OB_OK;
+}
+
+int check_block(ob_ctx *ctx, const ob_layered_desc &c, uint32_t i) {
+    const ob_block_desc &b = c.layers[i];
+    const ob_mixer_desc &x = b.mixer;
+    const std::string at = "layer " + std::to_string(i) + " ";
+    int rc;
+    if (!x.n_head || !x.dim || !x.vdim) return fail(ctx, OB_ERR_INVALID, "layered model: " + at + "mixer sizes missing");
+    const uint32_t H = x.n_head, E = c.n_embd, rotating = x.kind == OB_MIXER_LATENT_ATTENTION ? x.rot_dim : x.dim;
+    if ((x.rot_dims & 1) || x.rot_dims > rotating) return fail(ctx, OB_ERR_INVALID, "layered model: " + at + "rot_dims must be even and fit the rotated vector");
+    if (x.rot_dims && !(x.rot_base > 0)) return fail(ctx, OB_ERR_INVALID, "layered model: " + at + "rot_base must be positive");
+    if (x.kind == OB_MIXER_LATENT_ATTENTION) {
+        if (!x.kv_rank || !x.kv_norm) return fail(ctx, OB_ERR_INVALID, "layered model: " + at + "latent size or norm missing");
+        if ((uint64_t)(2 * x.kv_rank + x.rot_dim + 256) * 4 > 128 * 1024) return fail(ctx, OB_ERR_UNSUPPORTED, "layered model: " + at + "kv_rank too large");
+        if ((rc = check_dense(ctx, x.wq, E, H * (x.dim + x.rot_dim), at + "wq"))) return rc;
+        if ((rc = check_dense(ctx, x.w_dkv, E, x.kv_rank + x.rot_dim, at + "w_dkv"))) return rc;
+        if ((rc = check_dense(ctx, x.w_uk, x.kv_rank, H * x.dim, at + "w_uk"))) return rc;
+        if ((rc = check_dense(ctx, x.w_uv, x.kv_rank, H * x.vdim, at + "w_uv"))) return rc;
+        if ((rc = check_dense(ctx, x.w_gate, E, H, at + "mixer gate"))) return rc;
+    } else if (x.kind == OB_MIXER_RETENTION) {
+        if (!x.decay) return fail(ctx, OB_ERR_INVALID, "layered model: " + at + "decay missing");
+        if (!retention_supported(x.dim)) return fail(ctx, OB_ERR_UNSUPPORTED, "layered model: " + at + "retention heads have at most 256 key dimensions");
+        if ((rc = check_dense(ctx, x.wq, E, H * x.dim, at + "wq"))) return rc;
+        if ((rc = check_dense(ctx, x.wk, E, H * x.dim, at + "wk"))) return rc;
+        if ((rc = check_dense(ctx, x.wv, E, H * x.vdim, at + "wv"))) return rc;
+        if ((rc = check_dense(ctx, x.w_gate, E, H * x.vdim, at + "mixer gate"))) return rc;
+    } else {
+        return fail(ctx, OB_ERR_UNSUPPORTED, "layered model: " + at + "unknown mixer");
+    }
+    if ((rc = check_dense(ctx, x.wo, H * x.vdim, E, at + "wo"))) return rc;
+    if (b.n_ff) {
+        if ((rc = check_dense(ctx, b.w_gate, E, b.n_ff, at + "ff gate"))) return rc;
+        if ((rc = check_dense(ctx, b.w_up, E, b.n_ff, at + "ff up"))) return rc;
+        if ((rc = check_dense(ctx, b.w_down, b.n_ff, E, at + "ff down"))) return rc;
+    }
+    if (c.side_dim) {
+        if (!b.side_norm) return fail(ctx, OB_ERR_INVALID, "layered model: " + at + "side norm missing");
+        if ((rc = check_dense(ctx, b.side_gate, E, c.side_dim, at + "side gate"))) return rc;
+        if ((rc = check_dense(ctx, b.side_proj, c.side_dim, E, at + "side proj"))) return rc;
+    }
+    return OB_OK;
+}
+
+}  // namespace
+
+extern "C" int ob_layered_model_create(ob_ctx *ctx, const ob_layered_desc *desc, ob_model **out) {
+    if (!ctx || !desc || !out) return fail(ctx, OB_ERR_INVALID, "layered_model_create: null argument");
+    *out = nullptr;
+    const ob_layered_desc &c = *desc;
+    if (!c.n_layer || !c.n_embd || !c.n_vocab || !c.layers) return fail(ctx, OB_ERR_INVALID, "layered_model_create: incomplete description");
+    if (c.n_embd > 32768) return fail(ctx, OB_ERR_UNSUPPORTED, "layered_model_create: n_embd above 32768");
+    int rc;
+    if ((rc = check_dense(ctx, c.token_embd, c.n_embd, c.n_vocab, "token_embd"))) return rc;
+    if ((rc = check_dense(ctx, c.output, c.n_embd, c.n_vocab, "output"))) return rc;
+    if (c.side_dim && (rc = check_dense(ctx, c.side_embd, c.n_layer * c.side_dim, c.n_vocab, "side_embd"))) return rc;
+    bool state = false;
+    for (uint32_t i = 0; i < c.n_layer; ++i) {
+        if ((rc = check_block(ctx, c, i))) return rc;
+        state |= c.layers[i].mixer.kind == OB_MIXER_RETENTION;
+    }
+
+    std::unique_lock<std::mutex> g(ctx->mu);
+    Bind b(ctx);
+    OB_CUDA(ctx, linear_configure());
+    OB_CUDA(ctx, mixers_configure());
+    ob_model *m = new ob_model;
+    m->ctx = ctx;
+    m->cfg.n_vocab = c.n_vocab;
+    m->cfg.n_embd = c.n_embd;
+    m->cfg.n_layer = c.n_layer;
+    m->cfg.rms_eps = c.rms_eps;
+    m->cfg.max_seq_len = c.max_seq_len ? c.max_seq_len : 4096;
+    m->cfg.max_batch_tokens = std::max(1u, c.max_batch_tokens);
+    m->T = m->cfg.max_batch_tokens;
+    auto bail = [&](int code) {
+        g.unlock();
+        ob_model_destroy(m);
+        return code;
+    };
+    const uint64_t tokens = c.kv_pool_tokens ? c.kv_pool_tokens : m->cfg.max_seq_len;
+    m->pool_pages = (uint32_t)((tokens + KV_PAGE - 1) / KV_PAGE);
+    for (int32_t p = (int32_t)m->pool_pages - 1; p >= 0; --p) m->free_pages.push_back(p);
+    if (state) {
+        m->n_state_slots = c.n_state_slots ? c.n_state_slots : 64;
+        for (int32_t s = (int32_t)m->n_state_slots - 1; s >= 0; --s) m->free_slots.push_back(s);
+    }
+    const uint32_t T = m->T;
+    // logits of as many rows at a time as fit 1 GiB (a step's rows come in slices of this many)
+    m->logit_cap = std::min<uint64_t>(T, std::max<uint64_t>(64, (1ull << 30) / (4ull * c.n_vocab)));
+    LayeredGraph *gr = new LayeredGraph;
+    gr->m = m;
+    m->graph = gr;
+    if ((rc = gr->build(c))) return bail(rc);
+    if ((rc = dev_alloc(m, &m->x, (size_t)T * c.n_embd))) return bail(rc);
+    if ((rc = dev_alloc(m, &m->logits, (size_t)m->logit_cap * c.n_vocab))) return bail(rc);
+    const MetaLayout ml(T);
+    if ((rc = dev_alloc(m, &m->d_meta, ml.bytes))) return bail(rc);
+    if ((rc = dev_alloc(m, &m->d_out_tokens, T))) return bail(rc);
+    if ((rc = dev_alloc(m, &m->argmax_scratch, T))) return bail(rc);
+    if ((rc = dev_alloc(m, &m->d_step_counter, 4))) return bail(rc);
+    if (cudaMallocHost(reinterpret_cast<void **>(&m->h_meta), ml.bytes) != cudaSuccess ||
+        cudaMallocHost(reinterpret_cast<void **>(&m->h_out_tokens), (size_t)T * 4) != cudaSuccess)
+        return bail(fail(ctx, OB_ERR_OOM, "layered_model_create: pinned host allocation failed"));
+    memset(m->h_meta, 0, ml.bytes);
+    cudaError_t e = cudaDeviceSynchronize();
+    if (e == cudaSuccess) e = cudaGetLastError();
+    if (e != cudaSuccess) return bail(fail(ctx, OB_ERR_CUDA, std::string("layered_model_create: ") + cudaGetErrorString(e)));
+    *out = m;
+    return OB_OK;
+}

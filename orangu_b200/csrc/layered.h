@@ -1,0 +1,119 @@
+// Launchers of the kernels for models given as a list of layers (layered.cu): bf16-weight products with fused epilogues, norms,
+// latent attention over a paged latent cache, retention with a per-sequence state (internal to the library).
+//
+// Two precisions share every launcher.  bf16: activations that enter a product are bfloat16, accumulation is fp32.  f32:
+// activations are fp32 and every product is plain fp32 multiply-add.  Weights are bfloat16 in both.  The residual stream, norms,
+// rotation, attention scores and weights, gates and recurrent states are fp32 in both.
+#pragma once
+
+#include <cuda_bf16.h>
+#include <cuda_runtime.h>
+#include <stdint.h>
+
+#include "common.cuh"
+
+namespace ob {
+
+// ---- linear.cu -------------------------------------------------------------------------------------------------------
+enum LinEpilogue {
+    LE_F32 = 0,       // out f32
+    LE_ACT = 1,       // out activation
+    LE_GLU = 2,       // rows (2j, 2j+1) are (gate j, up j): out activation j = g sigmoid(alpha g) (u + 1) of the limited pair
+    LE_RESIDUAL = 3,  // x f32 [t][pitch] += v; out2 (optional) gets the sum as activation
+    LE_GELU_EMB = 4,  // out activation = gelu_tanh(v) * emb[token t][emb_col0 + row]
+    LE_GATED = 5      // out activation = v * sigmoid(gate[t * gate_pitch + batch])
+};
+struct LinSegment {       // consecutive rows of the weight with one epilogue; row0 is a multiple of 32
+    uint32_t row0, n;     // rows [row0, row0 + n)
+    int epi;
+    void *out;            // element (t, r) goes to out[t * pitch + col0 + batch * batch_cols + (r - row0)] (LE_GLU: (r - row0) / 2)
+    uint32_t pitch, col0, batch_cols;
+};
+struct LinArgs {
+    const __nv_bfloat16 *w;   // [n_batch][n_rows][kp], zero padded
+    uint32_t n_rows, kp;      // kp: columns, a multiple of 64
+    const void *x;            // activations [T][x_pitch]; batch b reads columns [b * x_step, + kp)
+    uint32_t x_pitch, x_step; // elements; multiples of 8
+    uint32_t T, n_batch;
+    LinSegment seg[3];
+    int n_seg;
+    // epilogue parameters
+    void *out2 = nullptr;
+    uint32_t out2_pitch = 0;
+    float glu_limit = 0.0f, glu_alpha = 0.0f;
+    const uint32_t *tokens = nullptr;
+    const __nv_bfloat16 *emb = nullptr;
+    uint32_t emb_pitch = 0, emb_col0 = 0;
+    const float *gate = nullptr;
+    uint32_t gate_pitch = 0;
+};
+constexpr uint32_t LIN_K_ALIGN = 64, LIN_ROW_ALIGN = 32;
+cudaError_t linear_configure();  // kernel attributes of the current device (outside stream capture)
+bool launch_linear(const LinArgs &a, bool f32, int sm_count, cudaStream_t st);  // false: a tensor map could not be made
+int linear_take_status();        // 1 when a bounded wait inside a product ran out since the last call
+void linear_mark_launched();     // a replayed graph may have run one of the tensor-core products
+
+// ---- mixers.cu -------------------------------------------------------------------------------------------------------
+void launch_embed_bf16(const __nv_bfloat16 *table, uint32_t width, const uint32_t *tokens, uint32_t T, float *x, cudaStream_t st);
+// h[i] = x[row i] / rms(x[row i]) * gain, as activation; rows == nullptr: row i.
+void launch_norm_scalar(const float *x, uint32_t width, const uint32_t *rows, uint32_t n, float eps, float gain, void *h, uint32_t h_pitch, bool f32,
+                        cudaStream_t st);
+// x += y / rms(y) * w, then (h != nullptr) h = x / rms(x) * gain as activation.
+void launch_side_finish(float *x, const float *y, const float *w, uint32_t width, uint32_t T, float eps, float gain, void *h, uint32_t h_pitch, bool f32,
+                        cudaStream_t st);
+
+struct Rot {                 // rotation of the first `dims` entries of a vector by position
+    const float2 *table;     // [position][dims / 2] (cos, sin)
+    uint32_t dims;
+    bool interleaved;        // pairs (2i, 2i+1), else (i, i + dims/2)
+};
+
+struct LatentArgs {          // latent attention of one layer over T rows
+    const float *y;          // projections [T][y_pitch]: rotated query parts [H][rot_dim], latent [kv_rank], shared rotated key part [rot_dim], gates [H]
+    uint32_t y_pitch;
+    uint32_t n_head, kv_rank, rot_dim, window;  // window 0: no limit
+    uint32_t kv_p, dq;       // padded latent width and padded row width (latent | rotated part) of queries and cache rows
+    float eps, scale;
+    const float *kv_norm;    // [kv_rank]
+    Rot rot;
+    void *q;                 // activations [T][H][dq]; the latent part is written by the absorbed-query product
+    void *cache;             // activations [page][16][dq]
+    void *o;                 // activations [T][H * o_pitch_h]: attention output in the latent space
+    uint32_t o_head;         // elements between heads in o
+    float *part;             // [splits][T * H][kv_p + 2] partial results (unnormalised output, max, sum)
+    uint64_t part_cap;       // floats `part` holds
+    // rows
+    uint32_t T, n_seq;
+    const RowSpan *spans;    // device [n_seq]
+    const RowSpan *h_spans;  // the same on the host
+    bool single;             // every span is one row
+    const uint32_t *positions;
+    const int32_t *const *tables;
+    uint32_t max_pos;        // positions are below this
+};
+cudaError_t mixers_configure();
+void launch_latent_prep(const LatentArgs &a, bool f32, cudaStream_t st);   // norms and appends the latent, rotates and stores the query parts
+uint32_t launch_latent_attention(const LatentArgs &a, bool f32, int sm_count, cudaStream_t st);  // returns the kernels launched
+
+struct RetentionArgs {       // retention of one layer over T rows
+    float *y;                // projections [T][y_pitch]: q [H][dim], k [H][dim], v [H][vdim], gate [H][vdim]; q and k are rotated in place
+    uint32_t y_pitch;
+    uint32_t n_head, dim, vdim;
+    float eps, k_scale;
+    const float *decay;      // [H]
+    Rot rot;
+    float *state;            // [slot][H][dim][vdim]
+    float *o;                // [T][H * vdim] before the norm
+    void *out;               // activations [T][out_pitch]: normed, gated
+    uint32_t out_pitch;
+    uint32_t T, n_seq;
+    const RowSpan *spans;
+    const uint32_t *positions;
+    const int32_t *slots;    // [T]
+};
+bool retention_supported(uint32_t dim);
+uint32_t launch_retention(const RetentionArgs &a, bool f32, int sm_count, cudaStream_t st);
+// Pages [0, n_pages) of one sequence's table to another's within a pool of pages of page_bytes (a multiple of 16).
+void launch_copy_pages(void *pool, uint64_t page_bytes, const int32_t *src_table, const int32_t *dst_table, uint32_t n_pages, cudaStream_t st);
+
+}  // namespace ob

@@ -1,0 +1,641 @@
+// Kernels around the products of models given as a list of layers: embedding, norms with a scalar gain, the per-layer token
+// input, latent attention over the paged latent cache, retention over the per-sequence state.
+//
+// Latent attention runs in the latent space: the query is multiplied by the key up-projection once per token and head (a batched
+// product, linear.cu), so a cache row (latent | shared rotated key part) is key and, in its first part, value of every head; the
+// value up-projection follows the attention.  Keys outside a row's window are never weighted, whole tiles outside are not read.
+#include <math.h>
+
+#include <algorithm>
+
+#include "layered.h"
+#include "pdl.cuh"
+
+namespace ob {
+
+namespace {
+
+using bf16 = __nv_bfloat16;
+
+template <typename TA> __device__ __forceinline__ TA to_act(float v);
+template <> __device__ __forceinline__ float to_act<float>(float v) { return v; }
+template <> __device__ __forceinline__ bf16 to_act<bf16>(float v) { return __float2bfloat16_rn(v); }
+__device__ __forceinline__ float from_act(float v) { return v; }
+__device__ __forceinline__ float from_act(bf16 v) { return __bfloat162float(v); }
+
+// Sum over the CTA; every thread gets it.  red: 33 floats.
+__device__ __forceinline__ float block_sum(float v, float *red) {
+    v = warp_sum(v);
+    __syncthreads();
+    if ((threadIdx.x & 31) == 0) red[threadIdx.x >> 5] = v;
+    __syncthreads();
+    if (threadIdx.x < 32) {
+        float s = threadIdx.x < blockDim.x / 32 ? red[threadIdx.x] : 0.0f;
+        s = warp_sum(s);
+        if (threadIdx.x == 0) red[32] = s;
+    }
+    __syncthreads();
+    return red[32];
+}
+
+__device__ __forceinline__ float inv_rms(float sum_sq, uint32_t n, float eps) { return 1.0f / sqrtf(sum_sq / (float)n + eps); }
+
+// (No __restrict__ on what an earlier kernel writes: a load the compiler may take for invariant could move above pdl_wait.)
+// ---- embedding, norms ------------------------------------------------------------------------------------------------------
+__global__ void __launch_bounds__(256) embed_bf16_kernel(const bf16 *table, uint32_t width, const uint32_t *tokens, float *x) {
+    pdl_release();
+    pdl_wait();
+    const bf16 *row = table + (uint64_t)tokens[blockIdx.x] * width;
+    for (uint32_t i = threadIdx.x; i < width; i += blockDim.x) x[(uint64_t)blockIdx.x * width + i] = __bfloat162float(row[i]);
+}
+
+template <typename TA>
+__global__ void __launch_bounds__(256) norm_scalar_kernel(const float *x, uint32_t width, const uint32_t *rows, float eps, float gain, TA *h, uint32_t h_pitch) {
+    __shared__ float red[33];
+    pdl_release();
+    pdl_wait();
+    const float *row = x + (uint64_t)(rows ? rows[blockIdx.x] : blockIdx.x) * width;
+    float s = 0.0f;
+    for (uint32_t i = threadIdx.x; i < width; i += blockDim.x) s += row[i] * row[i];
+    const float f = inv_rms(block_sum(s, red), width, eps) * gain;
+    for (uint32_t i = threadIdx.x; i < width; i += blockDim.x) h[(uint64_t)blockIdx.x * h_pitch + i] = to_act<TA>(row[i] * f);
+}
+
+template <typename TA>
+__global__ void __launch_bounds__(256) side_finish_kernel(float *x, const float *y, const float *w, uint32_t width, float eps, float gain, TA *h,
+                                                          uint32_t h_pitch) {
+    extern __shared__ float row[];
+    __shared__ float red[33];
+    pdl_release();
+    pdl_wait();
+    const uint64_t o = (uint64_t)blockIdx.x * width;
+    float s = 0.0f;
+    for (uint32_t i = threadIdx.x; i < width; i += blockDim.x) s += y[o + i] * y[o + i];
+    const float f = inv_rms(block_sum(s, red), width, eps);
+    s = 0.0f;
+    for (uint32_t i = threadIdx.x; i < width; i += blockDim.x) {
+        const float v = x[o + i] + y[o + i] * f * w[i];
+        x[o + i] = v;
+        row[i] = v;
+        s += v * v;
+    }
+    if (!h) return;
+    const float f2 = inv_rms(block_sum(s, red), width, eps) * gain;
+    for (uint32_t i = threadIdx.x; i < width; i += blockDim.x) h[(uint64_t)blockIdx.x * h_pitch + i] = to_act<TA>(row[i] * f2);
+}
+
+// ---- rotation ----------------------------------------------------------------------------------------------------------------
+// Value d of the rotated vector whose unrotated values are v[0..]; cs: this position's (cos, sin) row.
+__device__ __forceinline__ float rotated(const float *v, uint32_t d, const Rot &r, const float2 *cs) {
+    if (d >= r.dims) return v[d];
+    const uint32_t half = r.dims / 2;
+    if (r.interleaved) {
+        const float2 c = cs[d >> 1];
+        return d & 1 ? v[d] * c.x + v[d - 1] * c.y : v[d] * c.x - v[d + 1] * c.y;
+    }
+    const float2 c = cs[d < half ? d : d - half];
+    return d < half ? v[d] * c.x - v[d + half] * c.y : v[d] * c.x + v[d - half] * c.y;
+}
+
+// ---- latent attention: what a token leaves in the cache, and its rotated query parts -----------------------------------------------
+template <typename TA>
+__global__ void __launch_bounds__(256) latent_prep_kernel(LatentArgs a) {
+    __shared__ float red[33];
+    pdl_release();
+    pdl_wait();
+    const uint32_t t = blockIdx.x, pos = a.positions[t];
+    const float *y = a.y + (uint64_t)t * a.y_pitch;
+    const float *lat = y + (uint64_t)a.n_head * a.rot_dim;
+    const float2 *cs = a.rot.table + (uint64_t)pos * (a.rot.dims / 2);
+    float s = 0.0f;
+    for (uint32_t i = threadIdx.x; i < a.kv_rank; i += blockDim.x) s += lat[i] * lat[i];
+    const float f = inv_rms(block_sum(s, red), a.kv_rank, a.eps);
+    TA *row = static_cast<TA *>(a.cache) + ((uint64_t)a.tables[t][pos / KV_PAGE] * KV_PAGE + pos % KV_PAGE) * a.dq;
+    for (uint32_t i = threadIdx.x; i < a.kv_rank; i += blockDim.x) row[i] = to_act<TA>(lat[i] * f * a.kv_norm[i]);
+    for (uint32_t d = threadIdx.x; d < a.rot_dim; d += blockDim.x) row[a.kv_p + d] = to_act<TA>(rotated(lat + a.kv_rank, d, a.rot, cs));
+    TA *q = static_cast<TA *>(a.q) + (uint64_t)t * a.n_head * a.dq + a.kv_p;
+    for (uint32_t i = threadIdx.x; i < a.n_head * a.rot_dim; i += blockDim.x) {
+        const uint32_t h = i / a.rot_dim, d = i - h * a.rot_dim;
+        q[(uint64_t)h * a.dq + d] = to_act<TA>(rotated(y + (uint64_t)h * a.rot_dim, d, a.rot, cs));
+    }
+}
+
+// First position row t of a sequence sees.
+__device__ __forceinline__ uint32_t first_seen(uint32_t pos, uint32_t window) { return window && pos + 1 > window ? pos + 1 - window : 0u; }
+
+// ---- latent attention, plain form: one CTA per (token, head), any sizes; fp32 throughout when the cache is fp32 ---------------------
+// Keys in blocks of 128: scores by the warps (lanes over the row), online softmax, then every thread adds up its own columns.
+constexpr int LA_KEYS = 128, LA_THREADS = 128;
+template <typename TA>
+__global__ void __launch_bounds__(LA_THREADS) latent_attn_plain_kernel(LatentArgs a) {
+    extern __shared__ float sm[];
+    float *q = sm, *acc = q + a.dq, *p = acc + a.kv_p;  // [dq], [kv_p], [LA_KEYS]
+    __shared__ float red[33];
+    pdl_release();
+    pdl_wait();
+    const uint32_t t = blockIdx.x / a.n_head, h = blockIdx.x % a.n_head, warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
+    const uint32_t pos = a.positions[t], lo = first_seen(pos, a.window), hi = pos + 1;
+    const int32_t *table = a.tables[t];
+    const TA *qg = static_cast<const TA *>(a.q) + ((uint64_t)t * a.n_head + h) * a.dq, *cache = static_cast<const TA *>(a.cache);
+    for (uint32_t i = threadIdx.x; i < a.dq; i += blockDim.x) q[i] = i < a.kv_rank || (i >= a.kv_p && i < a.kv_p + a.rot_dim) ? from_act(qg[i]) : 0.0f;
+    for (uint32_t i = threadIdx.x; i < a.kv_p; i += blockDim.x) acc[i] = 0.0f;
+    auto row_of = [&](uint32_t j) { return cache + ((uint64_t)table[j / KV_PAGE] * KV_PAGE + j % KV_PAGE) * a.dq; };
+    float m = -INFINITY, l = 0.0f;
+    __syncthreads();
+    for (uint32_t j0 = lo; j0 < hi; j0 += LA_KEYS) {
+        const uint32_t n = min((uint32_t)LA_KEYS, hi - j0);
+        for (uint32_t j = warp; j < n; j += LA_THREADS / 32) {
+            const TA *k = row_of(j0 + j);
+            float s = 0.0f;
+            for (uint32_t i = lane; i < a.dq; i += 32) s = fmaf(q[i], from_act(k[i]), s);
+            s = warp_sum(s);
+            if (lane == 0) p[j] = s * a.scale;
+        }
+        __syncthreads();
+        const float own = threadIdx.x < n ? p[threadIdx.x] : -INFINITY;
+        float bm = warp_max(own);
+        if (lane == 0) red[warp] = bm;
+        __syncthreads();
+        bm = fmaxf(fmaxf(red[0], red[1]), fmaxf(red[2], red[3]));
+        const float m_new = fmaxf(m, bm), keep = expf(m - m_new), e = threadIdx.x < n ? expf(own - m_new) : 0.0f;
+        p[threadIdx.x] = e;
+        l = l * keep + block_sum(e, red);  // synchronises: p is complete
+        m = m_new;
+        for (uint32_t i = threadIdx.x; i < a.kv_rank; i += blockDim.x) {
+            float v = acc[i] * keep;
+            for (uint32_t j = 0; j < n; ++j) v = fmaf(p[j], from_act(row_of(j0 + j)[i]), v);
+            acc[i] = v;
+        }
+        __syncthreads();
+    }
+    TA *o = static_cast<TA *>(a.o) + (uint64_t)t * a.n_head * a.o_head + (uint64_t)h * a.o_head;
+    for (uint32_t i = threadIdx.x; i < a.kv_rank; i += blockDim.x) o[i] = to_act<TA>(acc[i] / l);
+}
+
+// ---- latent attention on the tensor cores (bf16 cache) ----------------------------------------------------------------------------
+// A CTA takes 16 * MT consecutive (token, head) rows of one sequence -- all heads share the cache rows, so rows of several tokens
+// and heads make one tile -- and walks the union of their windows in tiles of KT keys, two stages of cp.async.  Scores: a warp has
+// 16 rows x 16 keys over the whole row width.  Softmax statistics, scores and weights are fp32; the weights enter the second
+// product as value plus remainder, two bf16 rows each.  Output: a warp has all rows x its share of the latent columns (16 at a
+// time, LM_PAIRS shares of them).  (mma.sync on purpose: with few tokens M is the number of heads, and 512 output columns for
+// 128 rows would take all of tensor memory.)
+constexpr int LM_THREADS = 256, LM_PAIRS = 4;
+__host__ __device__ constexpr int lm_keys(int mt) { return mt == 4 ? 32 : 64; }
+struct LmPlan {
+    uint32_t q, k, stage, s, ph, pl, stat, bytes;  // byte offsets; stage: bytes of one key stage
+    __host__ __device__ LmPlan(int mt, uint32_t dq) {
+        const uint32_t M = 16 * mt, KT = lm_keys(mt), row = (dq + 8) * 2;
+        q = 0;
+        k = q + M * row;
+        stage = KT * row;
+        s = k + 2 * stage;
+        ph = s + M * (KT + 4) * 4;
+        pl = ph + M * (KT + 8) * 2;
+        stat = pl + M * (KT + 8) * 2;  // m, l, keep [M] f32, position [M]
+        bytes = stat + 4 * M * 4;
+    }
+};
+
+__device__ __forceinline__ uint32_t smem_addr(const void *p) { return (uint32_t)__cvta_generic_to_shared(p); }
+__device__ __forceinline__ void cp16(uint32_t dst, const void *src, bool in) {  // 16 bytes, or zeros
+    asm volatile("cp.async.cg.shared.global [%0], [%1], 16, %2;" ::"r"(dst), "l"(src), "r"(in ? 16 : 0) : "memory");
+}
+__device__ __forceinline__ void cp_commit() { asm volatile("cp.async.commit_group;" ::: "memory"); }
+template <int N> __device__ __forceinline__ void cp_wait() { asm volatile("cp.async.wait_group %0;" ::"n"(N) : "memory"); }
+__device__ __forceinline__ void ldsm4(uint32_t (&r)[4], uint32_t addr) {
+    asm volatile("ldmatrix.sync.aligned.m8n8.x4.shared.b16 {%0, %1, %2, %3}, [%4];" : "=r"(r[0]), "=r"(r[1]), "=r"(r[2]), "=r"(r[3]) : "r"(addr) : "memory");
+}
+__device__ __forceinline__ void ldsm4t(uint32_t (&r)[4], uint32_t addr) {
+    asm volatile("ldmatrix.sync.aligned.m8n8.x4.trans.shared.b16 {%0, %1, %2, %3}, [%4];" : "=r"(r[0]), "=r"(r[1]), "=r"(r[2]), "=r"(r[3]) : "r"(addr) : "memory");
+}
+__device__ __forceinline__ void mma_bf16(float (&c)[4], const uint32_t (&a)[4], uint32_t b0, uint32_t b1) {
+    asm volatile("mma.sync.aligned.m16n8k16.row.col.f32.bf16.bf16.f32 {%0, %1, %2, %3}, {%4, %5, %6, %7}, {%8, %9}, {%0, %1, %2, %3};"
+                 : "+f"(c[0]), "+f"(c[1]), "+f"(c[2]), "+f"(c[3])
+                 : "r"(a[0]), "r"(a[1]), "r"(a[2]), "r"(a[3]), "r"(b0), "r"(b1));
+}
+
+// The tile'th group of `rows` (token, head) rows: its span and first row within the span.  One warp; every lane gets the answer.
+__device__ __forceinline__ void find_tile(const RowSpan *spans, uint32_t n_seq, uint32_t n_head, uint32_t rows, uint32_t tile, RowSpan *span, uint32_t *first) {
+    const uint32_t lane = threadIdx.x & 31;
+    for (uint32_t s0 = 0;; s0 += 32) {
+        const RowSpan sp = s0 + lane < n_seq ? spans[s0 + lane] : RowSpan{0, 0};
+        const uint32_t n = (sp.n * n_head + rows - 1) / rows;
+        uint32_t sum = n;
+#pragma unroll
+        for (int o = 1; o < 32; o <<= 1) {
+            const uint32_t up = __shfl_up_sync(0xffffffffu, sum, o);
+            if (lane >= o) sum += up;
+        }
+        const uint32_t hit = __ballot_sync(0xffffffffu, tile < sum);
+        if (hit || s0 + 32 >= n_seq) {
+            const int src = hit ? __ffs(hit) - 1 : 31;
+            span->row0 = __shfl_sync(0xffffffffu, sp.row0, src);
+            span->n = hit ? __shfl_sync(0xffffffffu, sp.n, src) : 0;
+            *first = (tile - __shfl_sync(0xffffffffu, sum - n, src)) * rows;
+            return;
+        }
+        tile -= __shfl_sync(0xffffffffu, sum, 31);
+    }
+}
+
+template <int MT>
+__global__ void __launch_bounds__(LM_THREADS, 1) latent_attn_mma_kernel(LatentArgs a) {
+    constexpr int M = 16 * MT, KT = lm_keys(MT), SP = KT + 4, PP = KT + 8;
+    extern __shared__ __align__(16) uint8_t smem[];
+    const LmPlan pl(MT, a.dq);
+    float *S = reinterpret_cast<float *>(smem + pl.s), *mx = reinterpret_cast<float *>(smem + pl.stat), *sum = mx + M, *keep = sum + M;
+    int *rpos = reinterpret_cast<int *>(keep + M);
+    bf16 *Ph = reinterpret_cast<bf16 *>(smem + pl.ph), *Pl = reinterpret_cast<bf16 *>(smem + pl.pl);
+    const uint32_t warp = threadIdx.x >> 5, lane = threadIdx.x & 31, row_bytes = (a.dq + 8) * 2, chunks = a.dq / 8;
+    pdl_release();
+    pdl_wait();
+    __shared__ uint32_t tile_info[3];
+    if (warp == 0) {
+        RowSpan sp{blockIdx.x, 1};
+        uint32_t f = 0;
+        const uint32_t per = (a.n_head + M - 1) / M;
+        if (a.single) sp.row0 = blockIdx.x / per, f = blockIdx.x % per * M;
+        else find_tile(a.spans, a.n_seq, a.n_head, M, blockIdx.x, &sp, &f);
+        if (lane == 0) tile_info[0] = sp.row0, tile_info[1] = sp.n, tile_info[2] = f;
+    }
+    __syncthreads();
+    const uint32_t row0 = tile_info[0], f0 = tile_info[2], n_flat = tile_info[1] * a.n_head;
+    if (f0 >= n_flat) return;
+    const uint32_t n_here = min((uint32_t)M, n_flat - f0), pos0 = a.positions[row0];
+    const uint32_t first_tok = f0 / a.n_head, last_tok = (f0 + n_here - 1) / a.n_head;
+    const int32_t *table = a.tables[row0];
+    // this CTA's keys
+    uint32_t lo = first_seen(pos0 + first_tok, a.window), hi = pos0 + last_tok + 1;
+    {
+        const uint32_t per = ((hi - lo + gridDim.y - 1) / gridDim.y + KT - 1) / KT * KT;
+        lo = min(hi, lo + blockIdx.y * per);
+        hi = min(hi, lo + per);
+    }
+    const uint32_t n_tiles = (hi - lo + KT - 1) / KT;
+
+    auto load_keys = [&](uint32_t it) {
+        const uint32_t base = smem_addr(smem + pl.k) + (it & 1u) * pl.stage;
+        for (uint32_t i = threadIdx.x; i < KT * chunks; i += LM_THREADS) {
+            const uint32_t r = i / chunks, c = i - r * chunks, j = lo + it * KT + r;
+            const bool in = j < hi;
+            const bf16 *src = static_cast<const bf16 *>(a.cache) + (in ? ((uint64_t)table[j / KV_PAGE] * KV_PAGE + j % KV_PAGE) * a.dq + 8 * c : 0);
+            cp16(base + r * row_bytes + c * 16, src, in);
+        }
+    };
+    {   // queries: consecutive flat rows are consecutive in memory
+        const bf16 *q = static_cast<const bf16 *>(a.q) + ((uint64_t)row0 * a.n_head + f0) * a.dq;
+        for (uint32_t i = threadIdx.x; i < M * chunks; i += LM_THREADS) {
+            const uint32_t r = i / chunks, c = i - r * chunks;
+            cp16(smem_addr(smem + pl.q) + r * row_bytes + c * 16, q + (r < n_here ? (uint64_t)r * a.dq + 8 * c : 0), r < n_here);
+        }
+    }
+    if (n_tiles) load_keys(0);
+    cp_commit();
+    if (threadIdx.x < M) {
+        mx[threadIdx.x] = -INFINITY;
+        sum[threadIdx.x] = 0.0f;
+        rpos[threadIdx.x] = threadIdx.x < n_here ? (int)(pos0 + (f0 + threadIdx.x) / a.n_head) : -1;
+    }
+    const float scale2 = a.scale * 1.4426950408889634f;  // weights are powers of two of the scaled score
+    const uint32_t n_pair = a.kv_p / 16;
+    float acc[MT][LM_PAIRS][2][4];
+#pragma unroll
+    for (int i = 0; i < MT; ++i)
+#pragma unroll
+        for (int p = 0; p < LM_PAIRS; ++p)
+#pragma unroll
+            for (int n = 0; n < 2; ++n)
+#pragma unroll
+                for (int e = 0; e < 4; ++e) acc[i][p][n][e] = 0.0f;
+
+    const uint32_t qs = smem_addr(smem + pl.q), mt_s = warp % MT, kg = warp / MT;
+    const uint32_t a_off = (lane & 15) * row_bytes + (lane >> 4) * 16, b_off = ((lane & 7) + ((lane >> 4) << 3)) * row_bytes + ((lane >> 3) & 1) * 16;
+    const uint32_t v_off = ((lane & 7) + (((lane >> 3) & 1) << 3)) * row_bytes + (lane >> 4) * 16, p_off = (lane & 15) * (PP * 2) + (lane >> 4) * 16;
+    for (uint32_t it = 0; it < n_tiles; ++it) {
+        if (it + 1 < n_tiles) load_keys(it + 1);
+        cp_commit();
+        cp_wait<1>();
+        __syncthreads();
+        const uint32_t ks = smem_addr(smem + pl.k) + (it & 1u) * pl.stage;
+        if (kg * 16 < KT) {
+            float c[2][4] = {};
+            const uint32_t qa = qs + mt_s * 16 * row_bytes + a_off, kb = ks + kg * 16 * row_bytes + b_off;
+#pragma unroll 4
+            for (uint32_t k = 0; k < a.dq / 16; ++k) {
+                uint32_t fa[4], fb[4];
+                ldsm4(fa, qa + k * 32);
+                ldsm4(fb, kb + k * 32);
+                mma_bf16(c[0], fa, fb[0], fb[1]);
+                mma_bf16(c[1], fa, fb[2], fb[3]);
+            }
+            float *s = S + (mt_s * 16 + lane / 4) * SP + kg * 16 + 2 * (lane & 3);
+#pragma unroll
+            for (int n = 0; n < 2; ++n) {
+                *reinterpret_cast<float2 *>(s + 8 * n) = make_float2(c[n][0], c[n][1]);
+                *reinterpret_cast<float2 *>(s + 8 * SP + 8 * n) = make_float2(c[n][2], c[n][3]);
+            }
+        }
+        __syncthreads();
+#pragma unroll
+        for (int i = 0; i < M / 8; ++i) {  // online softmax, a warp per row
+            const int r = warp * (M / 8) + i, p = rpos[r];
+            float v[KT / 32], best = -INFINITY;
+#pragma unroll
+            for (int u = 0; u < KT / 32; ++u) {
+                const int j = (int)(lo + it * KT) + u * 32 + (int)lane;
+                const bool see = j <= p && j < (int)hi && (a.window == 0 || p - j < (int)a.window);
+                v[u] = see ? S[r * SP + u * 32 + lane] * scale2 : -INFINITY;
+                best = fmaxf(best, v[u]);
+            }
+            best = warp_max(best);
+            const float m_old = mx[r], m_new = fmaxf(m_old, best);
+            float l = 0.0f;
+#pragma unroll
+            for (int u = 0; u < KT / 32; ++u) {
+                const float e = m_new == -INFINITY ? 0.0f : exp2f(v[u] - m_new);
+                const bf16 h = __float2bfloat16_rn(e);
+                Ph[r * PP + u * 32 + lane] = h;
+                Pl[r * PP + u * 32 + lane] = __float2bfloat16_rn(e - __bfloat162float(h));
+                l += e;
+            }
+            l = warp_sum(l);
+            if (lane == 0) {
+                const float f = m_new == -INFINITY ? 1.0f : exp2f(m_old - m_new);
+                keep[r] = f;
+                mx[r] = m_new;
+                sum[r] = sum[r] * f + l;
+            }
+        }
+        __syncthreads();
+#pragma unroll
+        for (int i = 0; i < MT; ++i) {
+            const float f0r = keep[i * 16 + lane / 4], f1r = keep[i * 16 + lane / 4 + 8];
+#pragma unroll
+            for (int p = 0; p < LM_PAIRS; ++p)
+#pragma unroll
+                for (int n = 0; n < 2; ++n) acc[i][p][n][0] *= f0r, acc[i][p][n][1] *= f0r, acc[i][p][n][2] *= f1r, acc[i][p][n][3] *= f1r;
+        }
+#pragma unroll
+        for (int kk = 0; kk < KT / 16; ++kk) {
+            uint32_t fh[MT][4], fl[MT][4];
+#pragma unroll
+            for (int i = 0; i < MT; ++i) {
+                ldsm4(fh[i], smem_addr(Ph) + (i * 16 * PP + kk * 16) * 2 + p_off);
+                ldsm4(fl[i], smem_addr(Pl) + (i * 16 * PP + kk * 16) * 2 + p_off);
+            }
+#pragma unroll
+            for (int p = 0; p < LM_PAIRS; ++p) {
+                if (warp + 8 * p >= n_pair) break;
+                uint32_t fv[4];
+                ldsm4t(fv, ks + kk * 16 * row_bytes + (warp + 8 * p) * 32 + v_off);
+#pragma unroll
+                for (int i = 0; i < MT; ++i) {
+                    mma_bf16(acc[i][p][0], fh[i], fv[0], fv[1]);
+                    mma_bf16(acc[i][p][1], fh[i], fv[2], fv[3]);
+                    mma_bf16(acc[i][p][0], fl[i], fv[0], fv[1]);
+                    mma_bf16(acc[i][p][1], fl[i], fv[2], fv[3]);
+                }
+            }
+        }
+        __syncthreads();
+    }
+    cp_wait<0>();
+    __syncthreads();
+    const bool whole = gridDim.y == 1;
+#pragma unroll
+    for (int i = 0; i < MT; ++i)
+#pragma unroll
+        for (int hf = 0; hf < 2; ++hf) {
+            const uint32_t r = i * 16 + lane / 4 + 8 * hf;
+            if (r >= n_here) continue;
+            const uint64_t flat = (uint64_t)row0 * a.n_head + f0 + r;
+            const float inv = whole ? 1.0f / sum[r] : 1.0f;
+#pragma unroll
+            for (int p = 0; p < LM_PAIRS; ++p) {
+                if (warp + 8 * p >= n_pair) break;
+#pragma unroll
+                for (int n = 0; n < 2; ++n) {
+                    const uint32_t col = (warp + 8 * p) * 16 + n * 8 + 2 * (lane & 3);
+                    const float v0 = acc[i][p][n][2 * hf] * inv, v1 = acc[i][p][n][2 * hf + 1] * inv;
+                    if (whole) *reinterpret_cast<__nv_bfloat162 *>(static_cast<bf16 *>(a.o) + flat * a.o_head + col) = __floats2bfloat162_rn(v0, v1);
+                    else *reinterpret_cast<float2 *>(a.part + ((uint64_t)blockIdx.y * a.T * a.n_head + flat) * (a.kv_p + 2) + col) = make_float2(v0, v1);
+                }
+            }
+            if (!whole && warp == 0 && (lane & 3) == 0)
+                *reinterpret_cast<float2 *>(a.part + ((uint64_t)blockIdx.y * a.T * a.n_head + flat) * (a.kv_p + 2) + a.kv_p) = make_float2(mx[r], sum[r]);
+        }
+}
+
+// The splits of one (token, head) row put together.
+__global__ void __launch_bounds__(128) latent_merge_kernel(LatentArgs a, uint32_t n_splits) {
+    pdl_release();
+    pdl_wait();
+    const uint64_t flat = blockIdx.x, stride = (uint64_t)a.T * a.n_head * (a.kv_p + 2);
+    const float *p = a.part + flat * (a.kv_p + 2);
+    float m = -INFINITY, l = 0.0f;
+    for (uint32_t s = 0; s < n_splits; ++s) m = fmaxf(m, p[s * stride + a.kv_p]);
+    for (uint32_t s = 0; s < n_splits; ++s) l += exp2f(p[s * stride + a.kv_p] - m) * p[s * stride + a.kv_p + 1];
+    const float inv = 1.0f / l;
+    for (uint32_t i = threadIdx.x; i < a.kv_rank; i += blockDim.x) {
+        float v = 0.0f;
+        for (uint32_t s = 0; s < n_splits; ++s) v += exp2f(p[s * stride + a.kv_p] - m) * p[s * stride + i];
+        static_cast<bf16 *>(a.o)[flat * a.o_head + i] = __float2bfloat16_rn(v * inv);
+    }
+}
+
+// ---- retention -------------------------------------------------------------------------------------------------------------------
+// q and k of a token rotated in place, k scaled.
+__global__ void __launch_bounds__(256) retention_prep_kernel(RetentionArgs a) {
+    pdl_release();
+    pdl_wait();
+    const uint32_t t = blockIdx.x, half = a.rot.dims / 2, rest = a.dim - a.rot.dims, per = half + rest;
+    const float2 *cs = a.rot.table + (uint64_t)a.positions[t] * half;
+    float *y = a.y + (uint64_t)t * a.y_pitch;
+    for (uint32_t i = threadIdx.x; i < 2 * a.n_head * per; i += blockDim.x) {
+        const uint32_t v = i / per, e = i - v * per;  // vector (queries, then keys) and pair or unrotated entry within it
+        float *p = y + (uint64_t)v * a.dim;
+        const float s = v >= a.n_head ? a.k_scale : 1.0f;
+        if (e < half) {
+            const uint32_t iu = a.rot.interleaved ? 2 * e : e, iv = a.rot.interleaved ? 2 * e + 1 : e + half;
+            const float u = p[iu], w = p[iv];
+            p[iu] = (u * cs[e].x - w * cs[e].y) * s;
+            p[iv] = (w * cs[e].x + u * cs[e].y) * s;
+        } else {
+            p[a.rot.dims + e - half] *= s;
+        }
+    }
+}
+
+// One CTA carries 32 columns of one head's state through the rows of one sequence, token by token: lane = column, warp = DW of
+// the state's rows, kept in registers.  S = decay S + k v^T, o = S^T q; the warps' parts of o are added up once per block of tokens.
+template <int DW>
+__global__ void __launch_bounds__(256) retention_kernel(RetentionArgs a) {
+    constexpr int D = 8 * DW, RT_BLOCK = DW > 16 ? 8 : 16;
+    __shared__ __align__(16) float qs[RT_BLOCK][D], ks[RT_BLOCK][D];
+    __shared__ float vs[RT_BLOCK][32], part[8][RT_BLOCK][32];
+    pdl_release();
+    pdl_wait();
+    const uint32_t warp = threadIdx.x >> 5, lane = threadIdx.x & 31, h = blockIdx.y, col = blockIdx.x * 32 + lane;
+    const RowSpan sp = a.spans[blockIdx.z];
+    const bool live = col < a.vdim;
+    const float decay = a.decay[h];
+    float *state = a.state + (((uint64_t)a.slots[sp.row0] * a.n_head + h) * a.dim) * a.vdim + col;
+    float S[DW];
+    const bool fresh = a.positions[sp.row0] == 0;
+#pragma unroll
+    for (int i = 0; i < DW; ++i) {
+        const uint32_t d = warp * DW + i;
+        S[i] = !fresh && live && d < a.dim ? state[(uint64_t)d * a.vdim] : 0.0f;
+    }
+    for (uint32_t t0 = 0; t0 < sp.n; t0 += RT_BLOCK) {
+        const uint32_t n = min((uint32_t)RT_BLOCK, sp.n - t0);
+        for (uint32_t i = threadIdx.x; i < n * D; i += 256) {
+            const uint32_t t = i / D, d = i - t * D;
+            const float *y = a.y + (uint64_t)(sp.row0 + t0 + t) * a.y_pitch + (uint64_t)h * a.dim + d;
+            qs[t][d] = d < a.dim ? y[0] : 0.0f;
+            ks[t][d] = d < a.dim ? y[(uint64_t)a.n_head * a.dim] : 0.0f;
+        }
+        for (uint32_t i = threadIdx.x; i < n * 32; i += 256) {
+            const uint32_t t = i / 32;  // i % 32 == lane
+            vs[t][lane] = live ? a.y[(uint64_t)(sp.row0 + t0 + t) * a.y_pitch + 2ull * a.n_head * a.dim + (uint64_t)h * a.vdim + col] : 0.0f;
+        }
+        __syncthreads();
+        for (uint32_t t = 0; t < n; ++t) {
+            const float v = vs[t][lane];
+            float o[4] = {0.0f, 0.0f, 0.0f, 0.0f};
+#pragma unroll
+            for (int i = 0; i < DW; i += 4) {
+                const float4 k = *reinterpret_cast<const float4 *>(&ks[t][warp * DW + i]), q = *reinterpret_cast<const float4 *>(&qs[t][warp * DW + i]);
+                S[i] = fmaf(k.x, v, decay * S[i]), o[0] = fmaf(q.x, S[i], o[0]);
+                S[i + 1] = fmaf(k.y, v, decay * S[i + 1]), o[1] = fmaf(q.y, S[i + 1], o[1]);
+                S[i + 2] = fmaf(k.z, v, decay * S[i + 2]), o[2] = fmaf(q.z, S[i + 2], o[2]);
+                S[i + 3] = fmaf(k.w, v, decay * S[i + 3]), o[3] = fmaf(q.w, S[i + 3], o[3]);
+            }
+            part[warp][t][lane] = (o[0] + o[1]) + (o[2] + o[3]);
+        }
+        __syncthreads();
+        for (uint32_t t = warp; t < n; t += 8) {
+            float o = 0.0f;
+#pragma unroll
+            for (int w = 0; w < 8; ++w) o += part[w][t][lane];
+            if (live) a.o[(uint64_t)(sp.row0 + t0 + t) * a.n_head * a.vdim + (uint64_t)h * a.vdim + col] = o;
+        }
+    }
+#pragma unroll
+    for (int i = 0; i < DW; ++i) {
+        const uint32_t d = warp * DW + i;
+        if (live && d < a.dim) state[(uint64_t)d * a.vdim] = S[i];
+    }
+}
+
+// Every head's output over its root mean square, times silu of its gate.
+template <typename TA>
+__global__ void __launch_bounds__(256) retention_post_kernel(RetentionArgs a) {
+    pdl_release();
+    pdl_wait();
+    const uint32_t t = blockIdx.x, warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
+    const float *g = a.y + (uint64_t)t * a.y_pitch + 2ull * a.n_head * a.dim + (uint64_t)a.n_head * a.vdim;
+    for (uint32_t h = warp; h < a.n_head; h += 8) {
+        const float *o = a.o + ((uint64_t)t * a.n_head + h) * a.vdim;
+        float s = 0.0f;
+        for (uint32_t i = lane; i < a.vdim; i += 32) s += o[i] * o[i];
+        const float f = inv_rms(warp_sum(s), a.vdim, a.eps);
+        for (uint32_t i = lane; i < a.vdim; i += 32) {
+            const float z = g[(uint64_t)h * a.vdim + i];
+            static_cast<TA *>(a.out)[(uint64_t)t * a.out_pitch + (uint64_t)h * a.vdim + i] = to_act<TA>(o[i] * f * (z / (1.0f + expf(-z))));
+        }
+    }
+}
+
+__global__ void __launch_bounds__(256) copy_pool_pages_kernel(uint4 *pool, uint64_t page_vecs, const int32_t *__restrict__ src, const int32_t *__restrict__ dst) {
+    const uint4 *s = pool + (uint64_t)src[blockIdx.x] * page_vecs;
+    uint4 *d = pool + (uint64_t)dst[blockIdx.x] * page_vecs;
+    for (uint64_t i = threadIdx.x; i < page_vecs; i += blockDim.x) d[i] = s[i];
+}
+
+constexpr uint32_t MAX_SMEM = 227 * 1024;
+size_t plain_smem(const LatentArgs &a) { return (size_t)(a.dq + a.kv_p + LA_KEYS) * 4; }
+
+}  // namespace
+
+// ---- launchers ----------------------------------------------------------------------------------------------------------------------
+cudaError_t mixers_configure() {
+    static PerDeviceOnce once;
+    return once.run([] {
+        cudaError_t e = cudaFuncSetAttribute(latent_attn_mma_kernel<1>, cudaFuncAttributeMaxDynamicSharedMemorySize, MAX_SMEM - 64);
+        if (e == cudaSuccess) e = cudaFuncSetAttribute(latent_attn_mma_kernel<2>, cudaFuncAttributeMaxDynamicSharedMemorySize, MAX_SMEM - 64);
+        if (e == cudaSuccess) e = cudaFuncSetAttribute(latent_attn_mma_kernel<4>, cudaFuncAttributeMaxDynamicSharedMemorySize, MAX_SMEM - 64);
+        if (e == cudaSuccess) e = cudaFuncSetAttribute(latent_attn_plain_kernel<float>, cudaFuncAttributeMaxDynamicSharedMemorySize, 128 * 1024);
+        if (e == cudaSuccess) e = cudaFuncSetAttribute(latent_attn_plain_kernel<bf16>, cudaFuncAttributeMaxDynamicSharedMemorySize, 128 * 1024);
+        if (e == cudaSuccess) e = cudaFuncSetAttribute(side_finish_kernel<float>, cudaFuncAttributeMaxDynamicSharedMemorySize, 128 * 1024);
+        if (e == cudaSuccess) e = cudaFuncSetAttribute(side_finish_kernel<bf16>, cudaFuncAttributeMaxDynamicSharedMemorySize, 128 * 1024);
+        return e;
+    });
+}
+
+void launch_embed_bf16(const bf16 *table, uint32_t width, const uint32_t *tokens, uint32_t T, float *x, cudaStream_t st) {
+    launch_pdl(embed_bf16_kernel, T, 256, 0, st, table, width, tokens, x);
+}
+void launch_norm_scalar(const float *x, uint32_t width, const uint32_t *rows, uint32_t n, float eps, float gain, void *h, uint32_t h_pitch, bool f32, cudaStream_t st) {
+    if (f32) launch_pdl(norm_scalar_kernel<float>, n, 256, 0, st, x, width, rows, eps, gain, static_cast<float *>(h), h_pitch);
+    else launch_pdl(norm_scalar_kernel<bf16>, n, 256, 0, st, x, width, rows, eps, gain, static_cast<bf16 *>(h), h_pitch);
+}
+void launch_side_finish(float *x, const float *y, const float *w, uint32_t width, uint32_t T, float eps, float gain, void *h, uint32_t h_pitch, bool f32, cudaStream_t st) {
+    if (f32) launch_pdl(side_finish_kernel<float>, T, 256, (size_t)width * 4, st, x, y, w, width, eps, gain, static_cast<float *>(h), h_pitch);
+    else launch_pdl(side_finish_kernel<bf16>, T, 256, (size_t)width * 4, st, x, y, w, width, eps, gain, static_cast<bf16 *>(h), h_pitch);
+}
+
+void launch_latent_prep(const LatentArgs &a, bool f32, cudaStream_t st) {
+    if (f32) launch_pdl(latent_prep_kernel<float>, a.T, 256, 0, st, a);
+    else launch_pdl(latent_prep_kernel<bf16>, a.T, 256, 0, st, a);
+}
+
+uint32_t launch_latent_attention(const LatentArgs &a, bool f32, int sm_count, cudaStream_t st) {
+    uint32_t longest = 1;
+    if (!a.single)
+        for (uint32_t s = 0; s < a.n_seq; ++s) longest = std::max(longest, a.h_spans[s].n);
+    const uint64_t rows = (uint64_t)longest * a.n_head;
+    const int mt = rows <= 16 ? 1 : rows <= 32 ? 2 : 4;
+    const LmPlan plan(mt, a.dq);
+    if (f32 || a.kv_p > 16 * 8 * LM_PAIRS || plan.bytes > MAX_SMEM - 64) {
+        if (f32) launch_pdl(latent_attn_plain_kernel<float>, a.T * a.n_head, LA_THREADS, plain_smem(a), st, a);
+        else launch_pdl(latent_attn_plain_kernel<bf16>, a.T * a.n_head, LA_THREADS, plain_smem(a), st, a);
+        return 1;
+    }
+    const uint32_t M = 16 * mt, KT = lm_keys(mt);
+    uint32_t tiles = 0;
+    if (a.single) tiles = a.n_seq * ((a.n_head + M - 1) / M);
+    else
+        for (uint32_t s = 0; s < a.n_seq; ++s) tiles += (a.h_spans[s].n * a.n_head + M - 1) / M;
+    // few tiles: their keys are split over CTAs and put together afterwards
+    const uint32_t span = M / a.n_head + 2, reach = a.window ? std::min<uint64_t>(a.max_pos, (uint64_t)a.window + span) : a.max_pos;
+    uint32_t splits = std::max(1u, std::min((uint32_t)sm_count / std::max(1u, tiles), (reach + KT - 1) / KT));
+    while (splits > 1 && (uint64_t)splits * a.T * a.n_head * (a.kv_p + 2) > a.part_cap) --splits;
+    const dim3 grid(tiles, splits);
+    if (mt == 1) launch_pdl(latent_attn_mma_kernel<1>, grid, LM_THREADS, plan.bytes, st, a);
+    else if (mt == 2) launch_pdl(latent_attn_mma_kernel<2>, grid, LM_THREADS, plan.bytes, st, a);
+    else launch_pdl(latent_attn_mma_kernel<4>, grid, LM_THREADS, plan.bytes, st, a);
+    if (splits == 1) return 1;
+    launch_pdl(latent_merge_kernel, a.T * a.n_head, 128, 0, st, a, splits);
+    return 2;
+}
+
+bool retention_supported(uint32_t dim) { return dim >= 1 && dim <= 256; }
+
+uint32_t launch_retention(const RetentionArgs &a, bool f32, int sm_count, cudaStream_t st) {
+    (void)sm_count;
+    launch_pdl(retention_prep_kernel, a.T, 256, 0, st, a);
+    const dim3 grid((a.vdim + 31) / 32, a.n_head, a.n_seq);
+    if (a.dim <= 64) launch_pdl(retention_kernel<8>, grid, 256, 0, st, a);
+    else if (a.dim <= 128) launch_pdl(retention_kernel<16>, grid, 256, 0, st, a);
+    else launch_pdl(retention_kernel<32>, grid, 256, 0, st, a);
+    if (f32) launch_pdl(retention_post_kernel<float>, a.T, 256, 0, st, a);
+    else launch_pdl(retention_post_kernel<bf16>, a.T, 256, 0, st, a);
+    return 3;
+}
+
+void launch_copy_pages(void *pool, uint64_t page_bytes, const int32_t *src, const int32_t *dst, uint32_t n_pages, cudaStream_t st) {
+    if (n_pages) copy_pool_pages_kernel<<<n_pages, 256, 0, st>>>(static_cast<uint4 *>(pool), page_bytes / 16, src, dst);
+}
+
+}  // namespace ob

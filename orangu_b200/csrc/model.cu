@@ -8,39 +8,13 @@
 
 #include <algorithm>
 #include <cmath>
+#include <functional>
 #include <map>
 #include <vector>
 
-#include "runtime.h"
-#include "tp.h"
-
-using namespace obrt;
+#include "model.h"
 
 namespace {
-
-struct LayerDev {
-    float *attn_norm = nullptr, *ffn_norm = nullptr;
-    float *q_bias = nullptr, *k_bias = nullptr, *v_bias = nullptr, *q_norm = nullptr, *k_norm = nullptr;  // this rank's part; null: absent
-    bool variant = false;  // any of the above, or the NEOX pairing: the layer takes the operator-by-operator path
-    ob_weight *wq = nullptr, *wk = nullptr, *wv = nullptr, *wo = nullptr, *gate = nullptr, *up = nullptr, *down = nullptr;
-};
-
-struct ActPair {  // both granularities for one product input
-    ActBuf k, flat;
-};
-
-// Per-step metadata, one pinned host block mirrored by one device block.
-struct MetaLayout {
-    uint32_t T;
-    size_t off_tokens, off_positions, off_npos, off_tables, bytes;
-    explicit MetaLayout(uint32_t t) : T(t) {
-        off_tokens = 0;
-        off_positions = off_tokens + (size_t)t * 4;
-        off_npos = off_positions + (size_t)t * 4;
-        off_tables = (off_npos + (size_t)t * 4 + 15) & ~(size_t)15;
-        bytes = off_tables + (size_t)t * 8;
-    }
-};
 
 __global__ void advance_kernel(uint32_t *tokens, uint32_t *positions, uint32_t *npos, const uint32_t *out_tokens, uint32_t n_seq,
                                uint32_t *history, uint32_t *step_counter) {
@@ -68,95 +42,7 @@ __global__ void __launch_bounds__(256) copy_pages_kernel(__half *k_pool, __half 
 
 }  // namespace
 
-struct ob_model {
-    ob_ctx *ctx = nullptr;
-    ob_model_desc cfg{};
-    uint32_t tp_rank = 0, tp_size = 1;
-    uint32_t n_head_l = 0, n_head_kv_l = 0, n_ff_l = 0, vocab_l = 0, vocab0 = 0;
-    std::vector<LayerDev> layers;
-    ob_weight *token_embd = nullptr, *output = nullptr;
-    float *output_norm = nullptr;
-    float *rope_table = nullptr;
-    std::vector<void *> owned;  // plain cudaMalloc blocks
-
-    // KV pool: [layer][page][n_head_kv_l][16][head_dim] fp16, K and V
-    uint32_t pool_pages = 0;
-    __half *k_pool = nullptr, *v_pool = nullptr;
-    size_t layer_stride = 0;  // elements
-    std::vector<int32_t> free_pages;
-
-    uint32_t T = 0;  // max rows per step
-    float *x = nullptr, *q = nullptr, *k = nullptr, *v = nullptr, *attn = nullptr, *gate = nullptr, *up = nullptr, *proj = nullptr,
-          *logits = nullptr;
-    ActPair act_embd, act_attn, act_ff;
-    float *part_o = nullptr, *part_ml = nullptr;
-    uint32_t *ff_counters = nullptr;    // [n_ff / 256] arrival counters of the SwiGLU outputs, zero between launches
-    uint32_t *attn_counters = nullptr;  // [rows][kv heads] arrival counters of the fused attention kernel, zero between launches
-    float *norm_scale = nullptr;      // [2] RMSNorm scales for the fused decode kernels (attention norm, FFN / output norm)
-    uint8_t *ready_embd = nullptr, *ready_attn = nullptr, *ready_ff = nullptr;  // quantized activations of the single decode token
-    float *scores = nullptr;          // exact-order attention scratch [T][n_head_l][score_stride]
-    uint32_t score_stride = 0, exact_attn_max_pos = 0;
-    uint32_t max_splits = 1;
-    size_t row_splits_cap = 0;  // (row, split) pairs part_o / part_ml hold
-    uint8_t *d_meta = nullptr, *h_meta = nullptr;
-    uint32_t *d_out_tokens = nullptr, *h_out_tokens = nullptr;
-    unsigned long long *argmax_scratch = nullptr;
-    uint32_t *d_history = nullptr, *d_step_counter = nullptr;
-    uint32_t history_cap = 0;
-    uint32_t last_T = 0;
-    std::map<uint64_t, cudaGraphExec_t> graphs;
-    std::map<uint64_t, uint64_t> graph_launches;  // kernels one replay stands for
-    obtp::Comm *comm = nullptr;
-    obtp::PeerXchg px{};         // size > 1: the single-token step exchanges partials through peer memory instead of NCCL
-    obtp::PeerBulk bulk{};       // cap > 0: so do steps of a few rows (decode batches, short prefill chunks)
-    bool use_stream = true;  // OB_STREAM_GEMV=0 keeps batch-1 decode on the unfused kernels
-    bool stream_ok = false;      // every fused decode kernel of this model's shapes fits (shared memory)
-    bool use_fused_attn = true;  // OB_FUSED_ATTN=0 keeps the two-kernel flash-decode
-    bool use_prefill_attn = true;  // OB_PREFILL_ATTN=0: prefill chunks take the decode kernel row by row
-    bool comm_failed = false;    // a collective could not be enqueued during the last step (reported by check_peer)
-    obtp::Rendezvous *rdv = nullptr;  // host-side meeting of the ranks before a step is enqueued (tensor parallel only)
-    uint32_t rdv_timeout_ms = 30000;  // OB_TP_RENDEZVOUS_MS; 0 = off
-    bool out_of_step = false;         // a rendezvous failed: the ranks no longer run the same sequence of steps
-    // Persistent layer kernel (layer_stream.cu): the single-token products between two attention kernels as one launch.
-    // Phase list: [q/k/v of layer 0] then per layer [attention-output, gate/up, down, q/k/v of the next layer | output projection].
-    bool use_persist = false;    // OB_PERSIST=1; measured slower than one launch per product (barrier waits and the synchronous norm outweigh the launches saved)
-    bool persist_ok = false;
-    bool launch_failed = false;  // a launch of the persistent kernel was refused (reported after the step)
-    std::vector<LsPhase> h_phases;
-    LsPhase *d_phases = nullptr;
-    LsLayout ls_layout{};
-    uint32_t *ls_barriers = nullptr;  // one word per launch of a step, zeroed when the step starts
-    uint32_t *ls_status = nullptr;    // set by the kernel when a barrier wait ran out of time
-    uint32_t *h_ls_status = nullptr;  // pinned host copy, fetched with every step's results
-    uint32_t ls_timeout_ms = 2000;
-    bool ls_split = false;            // OB_LS_SPLIT=1: every phase is its own launch
-};
-
-struct ob_kv {
-    ob_model *m = nullptr;
-    uint32_t capacity = 0, len = 0;
-    std::vector<int32_t> pages;   // pages held, in position order
-    int32_t *d_table = nullptr;   // device copy, room for ceil(capacity / 16) entries
-    bool on_demand = false;       // pages are taken from the pool as the sequence grows (ob_kv_create_paged) and go back on truncate
-};
-
 namespace {
-
-template <typename Tp>
-int dev_alloc(ob_model *m, Tp **out, size_t count) {
-    void *p = nullptr;
-    OB_CUDA(m->ctx, cudaMalloc(&p, std::max<size_t>(count * sizeof(Tp), 16)));
-    m->owned.push_back(p);
-    *out = static_cast<Tp *>(p);
-    return OB_OK;
-}
-
-int upload_f32(ob_model *m, const float *src, size_t n, float **out) {
-    int rc = dev_alloc(m, out, n);
-    if (rc) return rc;
-    OB_CUDA(m->ctx, cudaMemcpyAsync(*out, src, n * 4, cudaMemcpyHostToDevice, m->ctx->stream));
-    return OB_OK;
-}
 
 int alloc_act(ob_model *m, ActPair *a, uint32_t rows, uint32_t dim) {
     int rc;
@@ -406,6 +292,36 @@ int grow_pages(ob_kv *kv, uint32_t new_len) {
     return OB_OK;
 }
 
+// Sequences of recurrent models hold a state slot from their first token until they are emptied.  Its contents need no
+// clearing: a sequence's first token starts from zero whatever the slot holds.
+bool slot_missing(const ob_kv *kv) { return kv->m->n_state_slots && kv->slot < 0; }
+void take_slot(ob_kv *kv) {
+    if (!slot_missing(kv)) return;
+    kv->slot = kv->m->free_slots.back();
+    kv->m->free_slots.pop_back();
+}
+void give_slot(ob_kv *kv) {
+    if (kv->slot < 0) return;
+    kv->m->free_slots.push_back(kv->slot);
+    kv->slot = -1;
+}
+
+// Room for every sequence of a call to hold kv->len + n[s] positions: all of it or an error that changes nothing.
+int reserve(ob_model *m, ob_kv *const *kvs, uint32_t n_seq, const std::function<uint32_t(uint32_t)> &n_new, const char *who) {
+    uint64_t pages = 0, slots = 0;
+    for (uint32_t s = 0; s < n_seq; ++s) {
+        pages += pages_missing(kvs[s], kvs[s]->len + n_new(s));
+        slots += slot_missing(kvs[s]);
+    }
+    if (pages > m->free_pages.size()) return fail(m->ctx, OB_ERR_CAPACITY, std::string(who) + ": KV pool exhausted");
+    if (slots > m->free_slots.size()) return fail(m->ctx, OB_ERR_CAPACITY, std::string(who) + ": no free state slot");
+    for (uint32_t s = 0; s < n_seq; ++s) {
+        take_slot(kvs[s]);
+        if (int rc = grow_pages(kvs[s], kvs[s]->len + n_new(s))) return rc;
+    }
+    return OB_OK;
+}
+
 // Returns true when `image` (the quantized output, for the single-token product kernels) has been written.
 // one_sequence: the rows are consecutive tokens of one sequence (a prefill chunk)
 bool run_attention(ob_model *m, uint32_t li, uint32_t T, bool exact_attn, uint32_t pos_bound, uint8_t *image, const int32_t *const *d_tables,
@@ -485,6 +401,24 @@ bool run_attention(ob_model *m, uint32_t li, uint32_t T, bool exact_attn, uint32
     }
 }
 
+std::vector<RowSpan> single_spans(uint32_t T) {
+    std::vector<RowSpan> v(T);
+    for (uint32_t i = 0; i < T; ++i) v[i] = RowSpan{i, 1};
+    return v;
+}
+
+// Greedy token of each of the first n rows of m->logits (single GPU).
+void enqueue_argmax(ob_model *m, uint32_t n, uint32_t *out, cudaStream_t st) {
+    ArgmaxArgs am{};
+    am.logits = m->logits;
+    am.n_seq = n;
+    am.n_vocab = m->cfg.n_vocab;
+    am.out = out;
+    am.scratch = m->argmax_scratch;
+    launch_argmax(am, st);
+    m->ctx->launches += 3;
+}
+
 // Enqueue one forward step over T rows whose metadata is already in d_meta.
 //   gemm_order: the rows are consecutive tokens of one sequence (prefill chunk)
 //   logit_row0 / n_logit_rows: which rows get the output projection
@@ -493,6 +427,14 @@ void enqueue_step(ob_model *m, uint32_t T, bool gemm_order, uint32_t logit_row0,
                   uint32_t pos_bound, cudaStream_t st) {
     const ob_model_desc &c = m->cfg;
     const MetaLayout ml(m->T);
+    if (m->graph) {  // decode batch (captured graphs): every row its own sequence, logits of all rows
+        const std::vector<RowSpan> spans = single_spans(T);
+        m->graph->layers(T, T, spans.data(), pos_bound, st);
+        m->graph->head(nullptr, n_logit_rows, st);
+        if (want_argmax) enqueue_argmax(m, n_logit_rows, m->d_out_tokens, st);
+        m->last_T = T;
+        return;
+    }
     const uint32_t *d_tokens = reinterpret_cast<uint32_t *>(m->d_meta + ml.off_tokens);
     const uint32_t *d_positions = reinterpret_cast<uint32_t *>(m->d_meta + ml.off_positions);
     const uint32_t *d_npos = reinterpret_cast<uint32_t *>(m->d_meta + ml.off_npos);
@@ -712,6 +654,7 @@ void ob_model_destroy(ob_model *m) {
     Bind b(ctx);
     cudaStreamSynchronize(ctx->stream);
     for (auto &kvp : m->graphs) cudaGraphExecDestroy(kvp.second);
+    delete m->graph;
     if (m->rdv) obtp::rendezvous_close(m->rdv);
     if (m->comm) obtp::destroy(m->comm);
     auto rel = [&](ob_weight *w) {
@@ -959,6 +902,7 @@ static int kv_create(ob_model *m, uint32_t capacity_tokens, bool on_demand, ob_k
     if (capacity_tokens > m->cfg.max_seq_len) return fail(ctx, OB_ERR_CAPACITY, "kv_create: capacity exceeds the model's max_seq_len");
     const uint32_t n_pages = (capacity_tokens + KV_PAGE - 1) / KV_PAGE;
     if (!on_demand && n_pages > m->free_pages.size()) return fail(ctx, OB_ERR_CAPACITY, "kv_create: KV pool exhausted");
+    if (!on_demand && m->n_state_slots && m->free_slots.empty()) return fail(ctx, OB_ERR_CAPACITY, "kv_create: no free state slot");
     Bind b(ctx);
     ob_kv *kv = new ob_kv;
     kv->m = m;
@@ -969,12 +913,14 @@ static int kv_create(ob_model *m, uint32_t capacity_tokens, bool on_demand, ob_k
             kv->pages.push_back(m->free_pages.back());
             m->free_pages.pop_back();
         }
+    if (!on_demand) take_slot(kv);
     cudaError_t e = cudaMalloc(reinterpret_cast<void **>(&kv->d_table), (size_t)n_pages * 4);
     if (e == cudaSuccess) e = cudaMemsetAsync(kv->d_table, 0, (size_t)n_pages * 4, ctx->stream);
     if (e == cudaSuccess && !kv->pages.empty()) e = cudaMemcpyAsync(kv->d_table, kv->pages.data(), kv->pages.size() * 4, cudaMemcpyHostToDevice, ctx->stream);
     if (e == cudaSuccess) e = cudaStreamSynchronize(ctx->stream);
     if (e != cudaSuccess) {
         for (int32_t p : kv->pages) m->free_pages.push_back(p);
+        give_slot(kv);
         if (kv->d_table) cudaFree(kv->d_table);
         delete kv;
         return fail(ctx, OB_ERR_CUDA, std::string("kv_create: ") + cudaGetErrorString(e));
@@ -993,6 +939,7 @@ void ob_kv_destroy(ob_kv *kv) {
     Bind b(ctx);
     cudaStreamSynchronize(ctx->stream);
     for (int32_t p : kv->pages) kv->m->free_pages.push_back(p);
+    give_slot(kv);
     cudaFree(kv->d_table);
     delete kv;
 }
@@ -1020,7 +967,10 @@ int ob_kv_truncate(ob_kv *kv, uint32_t new_len) {
     if (!kv) return OB_ERR_INVALID;
     std::lock_guard<std::mutex> g(kv->m->ctx->mu);
     if (new_len > kv->len) return fail(kv->m->ctx, OB_ERR_INVALID, "kv_truncate: new_len exceeds the current length");
+    if (kv->m->graph && kv->m->graph->recurrent() && new_len != 0 && new_len != kv->len)
+        return fail(kv->m->ctx, OB_ERR_UNSUPPORTED, "kv_truncate: a recurrent state can be emptied, not rolled back");
     kv->len = new_len;
+    if (kv->on_demand && new_len == 0) give_slot(kv);
     if (kv->on_demand) {  // whole pages past the new length go back to the pool (the device table keeps stale ids nobody reads)
         const size_t keep = (new_len + KV_PAGE - 1) / KV_PAGE;
         while (kv->pages.size() > keep) {
@@ -1038,6 +988,7 @@ int ob_kv_read(ob_kv *kv, uint32_t layer, uint32_t pos0, uint32_t n, float *k_ou
     std::lock_guard<std::mutex> g(ctx->mu);
     if (layer >= m->cfg.n_layer || (uint64_t)pos0 + n > kv->len) return fail(ctx, OB_ERR_INVALID, "kv_read: out of range");
     Bind b(ctx);
+    if (m->graph) return m->graph->read_pages(kv, layer, pos0, n, k_out, v_out);
     const uint32_t hd = m->cfg.head_dim, nkv = m->n_head_kv_l, kv_dim = nkv * hd;
     std::vector<__half> page((size_t)nkv * KV_PAGE * hd);
     for (int which = 0; which < 2; ++which) {
@@ -1066,9 +1017,16 @@ int ob_kv_copy_prefix(ob_kv *dst, const ob_kv *src, uint32_t n) {
     std::lock_guard<std::mutex> g(ctx->mu);
     if (dst->len != 0) return fail(ctx, OB_ERR_INVALID, "kv_copy_prefix: the destination is not empty");
     if (n > src->len || n > dst->capacity) return fail(ctx, OB_ERR_CAPACITY, "kv_copy_prefix: n exceeds the source length or the destination capacity");
-    if (pages_missing(dst, n) > m->free_pages.size()) return fail(ctx, OB_ERR_CAPACITY, "kv_copy_prefix: KV pool exhausted");
+    if (m->graph && m->graph->recurrent() && n != src->len)
+        return fail(ctx, OB_ERR_UNSUPPORTED, "kv_copy_prefix: a recurrent state can be copied whole, not for a shorter prefix");
     Bind b(ctx);
-    if (int rc = grow_pages(dst, n)) return rc;
+    if (int rc = reserve(m, &dst, 1, [n](uint32_t) { return n; }, "kv_copy_prefix")) return rc;
+    if (m->graph) {
+        if (int rc = m->graph->copy_prefix(dst, src, n)) return rc;
+        OB_CUDA(ctx, cudaStreamSynchronize(ctx->stream));
+        dst->len = n;
+        return OB_OK;
+    }
     const size_t page_elems = (size_t)m->n_head_kv_l * KV_PAGE * m->cfg.head_dim;  // a multiple of 8 halves: head_dim is even and a page holds 16 tokens
     const uint32_t n_pages = (n + KV_PAGE - 1) / KV_PAGE;
     if (n_pages) {
@@ -1080,11 +1038,27 @@ int ob_kv_copy_prefix(ob_kv *dst, const ob_kv *src, uint32_t n) {
     return OB_OK;
 }
 
+int ob_state_read(ob_kv *kv, uint32_t layer, float *out) {
+    if (!kv || !out) return OB_ERR_INVALID;
+    ob_model *m = kv->m;
+    std::lock_guard<std::mutex> g(m->ctx->mu);
+    if (!m->graph || kv->slot < 0 || kv->len == 0) return fail(m->ctx, OB_ERR_INVALID, "state_read: the sequence holds no recurrent state");
+    Bind b(m->ctx);
+    return m->graph->read_state(kv, layer, out);
+}
+
+uint32_t ob_model_free_slots(const ob_model *m) {
+    if (!m) return 0;
+    std::lock_guard<std::mutex> g(m->ctx->mu);
+    return (uint32_t)m->free_slots.size();
+}
+
 int ob_profile_gemv(ob_model *m, uint32_t ggml_type, uint32_t variant, uint32_t iters, float *ms_total, uint64_t *bytes_per_pass,
                     uint32_t *launches_per_pass) {
     if (!m || !ms_total || variant > 5) return OB_ERR_INVALID;
     ob_ctx *ctx = m->ctx;
     std::lock_guard<std::mutex> g(ctx->mu);
+    if (m->graph) return fail(ctx, OB_ERR_UNSUPPORTED, "profile_gemv: the model has no quantized products");
     Bind b(ctx);
     cudaStream_t st = ctx->stream;
     if (variant) {
@@ -1180,56 +1154,85 @@ int ob_profile_gemv(ob_model *m, uint32_t ggml_type, uint32_t variant, uint32_t 
 
 namespace {
 
-// One step on the stream: metadata up, kernels, results down; synchronises.
-int run_rows(ob_model *m, const std::vector<ob_kv *> &row_kv, const uint32_t *tokens, const uint32_t *positions, bool gemm_order,
-             uint32_t logit_row0, uint32_t n_logit_rows, const ob_greedy *greedy, const uint32_t *recent_off, uint32_t seq0,
-             uint32_t *out_token, float *out_logits) {
-    ob_ctx *ctx = m->ctx;
-    const uint32_t T = (uint32_t)row_kv.size();
+// What one step runs: its rows, and which of them get logits.
+struct StepRows {
+    std::vector<ob_kv *> kv;      // [T] sequence of each row
+    const uint32_t *tokens;       // [T]
+    const uint32_t *positions;    // [T]
+    bool gemm_order = false;      // Llama graph: the rows are consecutive tokens of one sequence
+    uint32_t logit_row0 = 0, n_logit_rows = 0;  // Llama graph: a range of rows
+    std::vector<RowSpan> spans;                 // other graphs: the rows of each sequence ...
+    std::vector<uint32_t> logit_rows;           // ... and any rows at all
+};
+
+void fill_meta_row(ob_model *m, uint32_t i, uint32_t token, uint32_t position, const ob_kv *kv) {
     const MetaLayout ml(m->T);
-    uint32_t *h_tokens = reinterpret_cast<uint32_t *>(m->h_meta + ml.off_tokens);
-    uint32_t *h_positions = reinterpret_cast<uint32_t *>(m->h_meta + ml.off_positions);
-    uint32_t *h_npos = reinterpret_cast<uint32_t *>(m->h_meta + ml.off_npos);
-    const int32_t **h_tables = reinterpret_cast<const int32_t **>(m->h_meta + ml.off_tables);
+    reinterpret_cast<uint32_t *>(m->h_meta + ml.off_tokens)[i] = token;
+    reinterpret_cast<uint32_t *>(m->h_meta + ml.off_positions)[i] = position;
+    reinterpret_cast<uint32_t *>(m->h_meta + ml.off_npos)[i] = position + 1;
+    reinterpret_cast<const int32_t **>(m->h_meta + ml.off_tables)[i] = kv->d_table;
+    reinterpret_cast<int32_t *>(m->h_meta + ml.off_slots)[i] = kv->slot;
+    reinterpret_cast<RowSpan *>(m->h_meta + ml.off_spans)[i] = RowSpan{i, 1};
+}
+
+// One step on the stream: metadata up, kernels, results down; synchronises.  seq0: the greedy settings' index of the first
+// row with logits.
+int run_rows(ob_model *m, const StepRows &r, const ob_greedy *greedy, const uint32_t *recent_off, uint32_t seq0, uint32_t *out_token, float *out_logits) {
+    ob_ctx *ctx = m->ctx;
+    const uint32_t T = (uint32_t)r.kv.size();
+    const uint32_t n_logit_rows = m->graph ? (uint32_t)r.logit_rows.size() : r.n_logit_rows;
+    const MetaLayout ml(m->T);
     uint32_t pos_bound = 0;
     for (uint32_t t = 0; t < T; ++t) {
-        h_tokens[t] = tokens[t];
-        h_positions[t] = positions[t];
-        h_npos[t] = positions[t] + 1;
-        h_tables[t] = row_kv[t]->d_table;
-        pos_bound = std::max(pos_bound, positions[t] + 1);
+        fill_meta_row(m, t, r.tokens[t], r.positions[t], r.kv[t]);
+        pos_bound = std::max(pos_bound, r.positions[t] + 1);
+    }
+    if (m->graph) {
+        memcpy(m->h_meta + ml.off_spans, r.spans.data(), r.spans.size() * sizeof(RowSpan));
+        memcpy(m->h_meta + ml.off_logit_rows, r.logit_rows.data(), (size_t)n_logit_rows * 4);
     }
     const bool exact_attn = pos_bound <= m->exact_attn_max_pos;
     cudaStream_t st = ctx->stream;
     OB_CUDA(ctx, cudaEventRecord(ctx->ev0, st));
     OB_CUDA(ctx, cudaMemcpyAsync(m->d_meta, m->h_meta, ml.bytes, cudaMemcpyHostToDevice, st));
     const bool penalise = greedy && greedy->repeat_penalty != 1.0f && greedy->recent && greedy->n_recent;
-    enqueue_step(m, T, gemm_order, logit_row0, n_logit_rows, out_token != nullptr && !penalise, out_logits != nullptr || penalise, exact_attn, pos_bound, st);
-    if (out_token && penalise) {
-        // repeat penalty, then argmax (sampling.rs:345-359); the history comes from the caller per call
-        for (uint32_t r = 0; r < n_logit_rows; ++r) {
-            const uint32_t s = seq0 + r, nr = greedy->n_recent[s];
-            const uint32_t start = nr > greedy->repeat_last_n ? nr - greedy->repeat_last_n : 0, cnt = nr - start;
-            if (!cnt) continue;
-            int rc = ensure(ctx, ctx->saux, (size_t)cnt * 4);
-            if (rc) return rc;
-            OB_CUDA(ctx, cudaMemcpyAsync(ctx->saux.p, greedy->recent + recent_off[s] + start, (size_t)cnt * 4, cudaMemcpyHostToDevice, st));
-            launch_repeat_penalty(m->logits + (size_t)r * m->cfg.n_vocab, m->cfg.n_vocab, static_cast<uint32_t *>(ctx->saux.p), cnt,
-                                  greedy->repeat_penalty, st);
-            ctx->launches++;
-            OB_CUDA(ctx, cudaStreamSynchronize(st));  // saux is reused by the next row
+    // Repeat penalty, argmax and the copies for rows [r0, r0 + n), whose logits are rows 0 .. n-1 of m->logits.
+    auto deliver = [&](uint32_t r0, uint32_t n, bool argmax_done) -> int {
+        if (out_token && penalise) {
+            // repeat penalty, then argmax (sampling.rs:345-359); the history comes from the caller per call
+            for (uint32_t i = 0; i < n; ++i) {
+                const uint32_t s = seq0 + r0 + i, nr = greedy->n_recent[s];
+                const uint32_t start = nr > greedy->repeat_last_n ? nr - greedy->repeat_last_n : 0, cnt = nr - start;
+                if (!cnt) continue;
+                int rc = ensure(ctx, ctx->saux, (size_t)cnt * 4);
+                if (rc) return rc;
+                OB_CUDA(ctx, cudaMemcpyAsync(ctx->saux.p, greedy->recent + recent_off[s] + start, (size_t)cnt * 4, cudaMemcpyHostToDevice, st));
+                launch_repeat_penalty(m->logits + (size_t)i * m->cfg.n_vocab, m->cfg.n_vocab, static_cast<uint32_t *>(ctx->saux.p), cnt,
+                                      greedy->repeat_penalty, st);
+                ctx->launches++;
+                OB_CUDA(ctx, cudaStreamSynchronize(st));  // saux is reused by the next row
+            }
         }
-        ArgmaxArgs am{};
-        am.logits = m->logits;
-        am.n_seq = n_logit_rows;
-        am.n_vocab = m->cfg.n_vocab;
-        am.out = m->d_out_tokens;
-        am.scratch = m->argmax_scratch;
-        launch_argmax(am, st);
-        ctx->launches += 3;
+        if (out_token && !argmax_done) enqueue_argmax(m, n, m->d_out_tokens + r0, st);
+        if (out_token) OB_CUDA(ctx, cudaMemcpyAsync(m->h_out_tokens + r0, m->d_out_tokens + r0, (size_t)n * 4, cudaMemcpyDeviceToHost, st));
+        if (out_logits)
+            OB_CUDA(ctx, cudaMemcpyAsync(out_logits + (size_t)r0 * m->cfg.n_vocab, m->logits, (size_t)n * m->cfg.n_vocab * 4, cudaMemcpyDeviceToHost, st));
+        return OB_OK;
+    };
+    if (m->graph) {
+        m->graph->layers(T, (uint32_t)r.spans.size(), r.spans.data(), pos_bound, st);
+        m->last_T = T;
+        for (uint32_t r0 = 0; r0 < n_logit_rows; r0 += m->logit_cap) {
+            const uint32_t n = std::min(m->logit_cap, n_logit_rows - r0);
+            m->graph->head(reinterpret_cast<const uint32_t *>(m->d_meta + ml.off_logit_rows) + r0, n, st);
+            if (int rc = deliver(r0, n, false)) return rc;
+        }
+    } else {
+        const bool argmax_in_step = out_token != nullptr && !penalise;
+        enqueue_step(m, T, r.gemm_order, r.logit_row0, n_logit_rows, argmax_in_step, out_logits != nullptr || penalise, exact_attn, pos_bound, st);
+        if (n_logit_rows)
+            if (int rc = deliver(0, n_logit_rows, argmax_in_step)) return rc;
     }
-    if (out_token) OB_CUDA(ctx, cudaMemcpyAsync(m->h_out_tokens, m->d_out_tokens, (size_t)n_logit_rows * 4, cudaMemcpyDeviceToHost, st));
-    if (out_logits) OB_CUDA(ctx, cudaMemcpyAsync(out_logits, m->logits, (size_t)n_logit_rows * m->cfg.n_vocab * 4, cudaMemcpyDeviceToHost, st));
     OB_CUDA(ctx, cudaEventRecord(ctx->ev1, st));
     fetch_status(m, st);
     OB_CUDA(ctx, cudaStreamSynchronize(st));
@@ -1239,6 +1242,71 @@ int run_rows(ob_model *m, const std::vector<ob_kv *> &row_kv, const uint32_t *to
     ctx->last_ms += ms;
     if (out_token) memcpy(out_token, m->h_out_tokens, (size_t)n_logit_rows * 4);
     return check_peer(m);
+}
+
+// All sequences of a call as one batch (graphs that take spans), in steps of at most T rows filled in order.  `want` lists
+// flat token numbers in ascending order; out_token / out_logits get one entry per wanted token.
+int forward_spans(ob_model *m, ob_kv *const *kvs, const uint32_t *tokens, const uint32_t *n_tokens, uint32_t n_seq, const std::vector<uint32_t> &want,
+                  const ob_greedy *greedy, const uint32_t *recent_off, uint32_t *out_token, float *out_logits) {
+    StepRows r;
+    std::vector<uint32_t> pos;
+    uint32_t flat0 = 0, flat = 0, done_want = 0, s = 0, in_seq = 0;
+    while (s < n_seq) {
+        r.kv.clear();
+        r.spans.clear();
+        r.logit_rows.clear();
+        pos.clear();
+        flat0 = flat;
+        std::vector<std::pair<ob_kv *, uint32_t>> moved;
+        while (s < n_seq && r.kv.size() < m->T) {
+            const uint32_t n = std::min(m->T - (uint32_t)r.kv.size(), n_tokens[s] - in_seq);
+            r.spans.push_back(RowSpan{(uint32_t)r.kv.size(), n});
+            for (uint32_t i = 0; i < n; ++i) {
+                r.kv.push_back(kvs[s]);
+                pos.push_back(kvs[s]->len + i);
+            }
+            moved.emplace_back(kvs[s], n);
+            flat += n;
+            in_seq += n;
+            if (in_seq == n_tokens[s]) {
+                ++s;
+                in_seq = 0;
+            }
+        }
+        const uint32_t w0 = done_want;
+        while (done_want < want.size() && want[done_want] < flat) r.logit_rows.push_back(want[done_want++] - flat0);
+        r.tokens = tokens + flat0;
+        r.positions = pos.data();
+        const bool any = !r.logit_rows.empty();
+        if (int rc = run_rows(m, r, greedy, recent_off, w0, any && out_token ? out_token + w0 : nullptr,
+                              any && out_logits ? out_logits + (size_t)w0 * m->cfg.n_vocab : nullptr))
+            return rc;
+        for (auto &mv : moved) mv.first->len += mv.second;
+    }
+    return OB_OK;
+}
+
+// What every forward call checks before anything changes.  tok_off[s] is the first flat token of sequence s.
+int check_forward(ob_model *m, ob_kv *const *kvs, const uint32_t *tokens, const uint32_t *n_tokens, const uint32_t *start_pos, uint32_t n_seq,
+                  std::vector<uint32_t> *tok_off, bool *all_single) {
+    ob_ctx *ctx = m->ctx;
+    uint64_t total = 0;
+    *all_single = true;
+    for (uint32_t s = 0; s < n_seq; ++s) {
+        ob_kv *kv = kvs[s];
+        if (!kv || kv->m != m) return fail(ctx, OB_ERR_INVALID, "forward: KV cache missing or from another model");
+        if (n_tokens[s] == 0) return fail(ctx, OB_ERR_INVALID, "forward: a sequence carries no tokens");
+        if (start_pos[s] != kv->len) return fail(ctx, OB_ERR_INVALID, "forward: start_pos does not continue the KV cache");
+        if ((uint64_t)kv->len + n_tokens[s] > kv->capacity) return fail(ctx, OB_ERR_CAPACITY, "forward: KV cache is full");
+        for (uint32_t s2 = 0; s2 < s; ++s2)
+            if (kvs[s2] == kv) return fail(ctx, OB_ERR_INVALID, "forward: the same KV cache appears twice");
+        if (n_tokens[s] != 1) *all_single = false;
+        (*tok_off)[s] = (uint32_t)total;
+        total += n_tokens[s];
+    }
+    for (uint64_t i = 0; i < total; ++i)
+        if (tokens[i] >= m->cfg.n_vocab) return fail(ctx, OB_ERR_INVALID, "forward: token id out of vocabulary range");
+    return OB_OK;
 }
 
 }  // namespace
@@ -1252,43 +1320,30 @@ int ob_forward(ob_model *m, ob_kv *const *kvs, const uint32_t *tokens, const uin
     std::lock_guard<std::mutex> g(ctx->mu);
     if (n_seq == 0) return OB_OK;
     Bind b(ctx);
-    // ---- validate everything before any state changes
     bool all_single = true;
-    uint64_t total = 0;
     std::vector<uint32_t> tok_off(n_seq), recent_off(n_seq, 0);
-    for (uint32_t s = 0; s < n_seq; ++s) {
-        ob_kv *kv = kvs[s];
-        if (!kv || kv->m != m) return fail(ctx, OB_ERR_INVALID, "forward: KV cache missing or from another model");
-        if (n_tokens[s] == 0) return fail(ctx, OB_ERR_INVALID, "forward: a sequence carries no tokens");
-        if (start_pos[s] != kv->len) return fail(ctx, OB_ERR_INVALID, "forward: start_pos does not continue the KV cache");
-        if ((uint64_t)kv->len + n_tokens[s] > kv->capacity) return fail(ctx, OB_ERR_CAPACITY, "forward: KV cache is full");
-        for (uint32_t s2 = 0; s2 < s; ++s2)
-            if (kvs[s2] == kv) return fail(ctx, OB_ERR_INVALID, "forward: the same KV cache appears twice");
-        if (n_tokens[s] != 1) all_single = false;
-        tok_off[s] = (uint32_t)total;
-        total += n_tokens[s];
-        if (s + 1 < n_seq && greedy && greedy->n_recent) recent_off[s + 1] = recent_off[s] + greedy->n_recent[s];
-    }
-    for (uint64_t i = 0; i < total; ++i)
-        if (tokens[i] >= m->cfg.n_vocab) return fail(ctx, OB_ERR_INVALID, "forward: token id out of vocabulary range");
-    {   // on-demand caches: all the pages this call needs, or none of them
-        uint64_t need = 0;
-        for (uint32_t s = 0; s < n_seq; ++s) need += pages_missing(kvs[s], kvs[s]->len + n_tokens[s]);
-        if (need > m->free_pages.size()) return fail(ctx, OB_ERR_CAPACITY, "forward: KV pool exhausted");
-        for (uint32_t s = 0; s < n_seq; ++s) {
-            int rc = grow_pages(kvs[s], kvs[s]->len + n_tokens[s]);
-            if (rc) return rc;
-        }
-    }
+    if (int rc = check_forward(m, kvs, tokens, n_tokens, start_pos, n_seq, &tok_off, &all_single)) return rc;
+    for (uint32_t s = 0; s + 1 < n_seq; ++s)
+        if (greedy && greedy->n_recent) recent_off[s + 1] = recent_off[s] + greedy->n_recent[s];
+    if (int rc = reserve(m, kvs, n_seq, [n_tokens](uint32_t s) { return n_tokens[s]; }, "forward")) return rc;
     if (int rc = pre_step(m)) return rc;
     ctx->last_ms = 0.0f;
 
+    if (m->graph) {
+        std::vector<uint32_t> last(n_seq);
+        for (uint32_t s = 0; s < n_seq; ++s) last[s] = tok_off[s] + n_tokens[s] - 1;
+        return forward_spans(m, kvs, tokens, n_tokens, n_seq, last, greedy, recent_off.data(), out_token, out_logits);
+    }
+    StepRows r;
     if (all_single) {
         // decode batch, in slices of at most max_batch_tokens rows
         for (uint32_t s0 = 0; s0 < n_seq; s0 += m->T) {
             const uint32_t n = std::min(m->T, n_seq - s0);
-            std::vector<ob_kv *> rows(kvs + s0, kvs + s0 + n);
-            int rc = run_rows(m, rows, tokens + s0, start_pos + s0, false, 0, n, greedy, recent_off.data(), s0, out_token ? out_token + s0 : nullptr,
+            r.kv.assign(kvs + s0, kvs + s0 + n);
+            r.tokens = tokens + s0;
+            r.positions = start_pos + s0;
+            r.n_logit_rows = n;
+            int rc = run_rows(m, r, greedy, recent_off.data(), s0, out_token ? out_token + s0 : nullptr,
                               out_logits ? out_logits + (size_t)s0 * m->cfg.n_vocab : nullptr);
             if (rc) return rc;
             for (uint32_t i = 0; i < n; ++i) kvs[s0 + i]->len += 1;
@@ -1302,14 +1357,62 @@ int ob_forward(ob_model *m, ob_kv *const *kvs, const uint32_t *tokens, const uin
         while (done < n_tokens[s]) {
             const uint32_t n = std::min(m->T, n_tokens[s] - done);
             const bool last_chunk = done + n == n_tokens[s];
-            std::vector<ob_kv *> rows(n, kv);
+            r.kv.assign(n, kv);
             std::vector<uint32_t> pos(n);
             for (uint32_t i = 0; i < n; ++i) pos[i] = kv->len + i;
-            // a chunk of one token takes the single-token kernels, exactly as the reference's matmul does
-            int rc = run_rows(m, rows, tokens + tok_off[s] + done, pos.data(), n > 1, n - 1, last_chunk ? 1 : 0, greedy, recent_off.data(), s,
-                              (last_chunk && out_token) ? out_token + s : nullptr,
+            r.tokens = tokens + tok_off[s] + done;
+            r.positions = pos.data();
+            r.gemm_order = n > 1;  // a chunk of one token takes the single-token kernels, exactly as the reference's matmul does
+            r.logit_row0 = n - 1;
+            r.n_logit_rows = last_chunk ? 1 : 0;
+            int rc = run_rows(m, r, greedy, recent_off.data(), s, (last_chunk && out_token) ? out_token + s : nullptr,
                               (last_chunk && out_logits) ? out_logits + (size_t)s * m->cfg.n_vocab : nullptr);
             if (rc) return rc;
+            kv->len += n;
+            done += n;
+        }
+    }
+    return OB_OK;
+}
+
+int ob_forward_rows(ob_model *m, ob_kv *const *kvs, const uint32_t *tokens, const uint32_t *n_tokens, const uint32_t *start_pos, uint32_t n_seq,
+                    const uint32_t *rows, uint32_t n_rows, float *out_logits) {
+    if (!m || !kvs || !tokens || !n_tokens || !start_pos || (n_rows && (!rows || !out_logits))) return fail(m ? m->ctx : nullptr, OB_ERR_INVALID, "forward_rows: null argument");
+    ob_ctx *ctx = m->ctx;
+    std::lock_guard<std::mutex> g(ctx->mu);
+    if (n_seq == 0) return OB_OK;
+    Bind b(ctx);
+    bool all_single = true;
+    std::vector<uint32_t> tok_off(n_seq);
+    if (int rc = check_forward(m, kvs, tokens, n_tokens, start_pos, n_seq, &tok_off, &all_single)) return rc;
+    const uint64_t total = (uint64_t)tok_off[n_seq - 1] + n_tokens[n_seq - 1];
+    for (uint32_t i = 0; i < n_rows; ++i)
+        if (rows[i] >= total || (i && rows[i] <= rows[i - 1])) return fail(ctx, OB_ERR_INVALID, "forward_rows: rows must ascend and name tokens of this call");
+    if (int rc = reserve(m, kvs, n_seq, [n_tokens](uint32_t s) { return n_tokens[s]; }, "forward_rows")) return rc;
+    if (int rc = pre_step(m)) return rc;
+    ctx->last_ms = 0.0f;
+    if (m->graph) return forward_spans(m, kvs, tokens, n_tokens, n_seq, std::vector<uint32_t>(rows, rows + n_rows), nullptr, nullptr, nullptr, out_logits);
+    // the Llama graph: sequence by sequence, all rows of a chunk projected and the wanted ones kept
+    StepRows r;
+    std::vector<float> all;
+    uint32_t w = 0;
+    for (uint32_t s = 0; s < n_seq; ++s) {
+        ob_kv *kv = kvs[s];
+        for (uint32_t done = 0; done < n_tokens[s];) {
+            const uint32_t n = std::min(m->T, n_tokens[s] - done), flat = tok_off[s] + done;
+            uint32_t w1 = w;
+            while (w1 < n_rows && rows[w1] < flat + n) ++w1;
+            std::vector<uint32_t> pos(n);
+            for (uint32_t i = 0; i < n; ++i) pos[i] = kv->len + i;
+            r.kv.assign(n, kv);
+            r.tokens = tokens + flat;
+            r.positions = pos.data();
+            r.gemm_order = n > 1;
+            r.logit_row0 = 0;
+            r.n_logit_rows = w1 > w ? n : 0;
+            all.resize((size_t)r.n_logit_rows * m->cfg.n_vocab);
+            if (int rc = run_rows(m, r, nullptr, nullptr, 0, nullptr, w1 > w ? all.data() : nullptr)) return rc;
+            for (; w < w1; ++w) memcpy(out_logits + (size_t)w * m->cfg.n_vocab, all.data() + (size_t)(rows[w] - flat) * m->cfg.n_vocab, (size_t)m->cfg.n_vocab * 4);
             kv->len += n;
             done += n;
         }
@@ -1349,6 +1452,8 @@ int pre_step(ob_model *m) {
 
 int check_peer(ob_model *m) {
     if (gemm_tc5_take_status()) return fail(m->ctx, OB_ERR_CUDA, "a tensor-core product gave up a bounded wait (pipeline barrier); the step's output is not valid");
+    if (m->graph && m->graph->take_failure()) return fail(m->ctx, OB_ERR_CUDA, "a product of the step could not be launched");
+    if (m->graph && linear_take_status()) return fail(m->ctx, OB_ERR_CUDA, "a tensor-core product gave up a bounded wait (pipeline barrier); the step's output is not valid");
     if (m->launch_failed) {
         m->launch_failed = false;
         return fail(m->ctx, OB_ERR_CUDA, std::string("launching the persistent layer kernel failed: ") + cudaGetErrorString(cudaGetLastError()));
@@ -1390,12 +1495,16 @@ int get_graph(ob_model *m, uint32_t n_seq, int kind, bool exact, cudaGraphExec_t
     // One eager pass first (d_meta must already describe a valid step): it sets the kernels' one-time
     // function attributes outside capture and counts what a step launches.  It rewrites the KV slot of
     // the current position with the values the replay will write again.
+    // A recurrent state would advance twice, so other graphs set their attributes when the model is made and are counted
+    // while they are captured.
     const uint64_t launches_before = ctx->launches;
-    enqueue_step(m, n_seq, false, 0, n_seq, true, false, exact, pos_bound, st);
-    OB_CUDA(ctx, cudaStreamSynchronize(st));
-    OB_CUDA(ctx, cudaGetLastError());
-    m->graph_launches[key] = ctx->launches - launches_before + (kind == 1 ? 1 : 0);
-    ctx->launches = launches_before;
+    if (!m->graph) {
+        enqueue_step(m, n_seq, false, 0, n_seq, true, false, exact, pos_bound, st);
+        OB_CUDA(ctx, cudaStreamSynchronize(st));
+        OB_CUDA(ctx, cudaGetLastError());
+        m->graph_launches[key] = ctx->launches - launches_before + (kind == 1 ? 1 : 0);
+        ctx->launches = launches_before;
+    }
     cudaGraph_t graph = nullptr;
     OB_CUDA(ctx, cudaStreamBeginCapture(st, cudaStreamCaptureModeThreadLocal));
     if (kind == 0) cudaMemcpyAsync(m->d_meta, m->h_meta, ml.bytes, cudaMemcpyHostToDevice, st);
@@ -1412,6 +1521,7 @@ int get_graph(ob_model *m, uint32_t n_seq, int kind, bool exact, cudaGraphExec_t
     }
     cudaError_t e = cudaStreamEndCapture(st, &graph);
     if (e != cudaSuccess || !graph) return fail(ctx, OB_ERR_CUDA, std::string("graph capture: ") + cudaGetErrorString(e));
+    if (m->graph) m->graph_launches[key] = ctx->launches - launches_before;
     m->ctx->launches = launches_before;  // capture enqueued nothing; replays are counted by their callers
     cudaGraphExec_t exec = nullptr;
     e = cudaGraphInstantiate(&exec, graph, 0);
@@ -1432,15 +1542,11 @@ int ob_decode_greedy(ob_model *m, ob_kv *kv, uint32_t token, uint32_t *out_token
     std::lock_guard<std::mutex> g(ctx->mu);
     if (token >= m->cfg.n_vocab) return fail(ctx, OB_ERR_INVALID, "decode_greedy: token id out of vocabulary range");
     if (kv->len >= kv->capacity) return fail(ctx, OB_ERR_CAPACITY, "decode_greedy: KV cache is full");
-    if (pages_missing(kv, kv->len + 1) > m->free_pages.size()) return fail(ctx, OB_ERR_CAPACITY, "decode_greedy: KV pool exhausted");
     Bind b(ctx);
-    if (int rc = grow_pages(kv, kv->len + 1)) return rc;
+    if (int rc = reserve(m, &kv, 1, [](uint32_t) { return 1u; }, "decode_greedy")) return rc;
     if (int rc = pre_step(m)) return rc;
     const MetaLayout ml(m->T);
-    reinterpret_cast<uint32_t *>(m->h_meta + ml.off_tokens)[0] = token;
-    reinterpret_cast<uint32_t *>(m->h_meta + ml.off_positions)[0] = kv->len;
-    reinterpret_cast<uint32_t *>(m->h_meta + ml.off_npos)[0] = kv->len + 1;
-    reinterpret_cast<const int32_t **>(m->h_meta + ml.off_tables)[0] = kv->d_table;
+    fill_meta_row(m, 0, token, kv->len, kv);
     cudaGraphExec_t exec;
     uint64_t key = 0;
     const bool exact = kv->len + 1 <= m->exact_attn_max_pos;
@@ -1472,13 +1578,8 @@ int ob_decode_loop(ob_model *m, ob_kv *const *kvs, const uint32_t *first_tokens,
             if (kvs[s2] == kvs[s]) return fail(ctx, OB_ERR_INVALID, "decode_loop: the same KV cache appears twice");
     }
     Bind b(ctx);
-    {
-        uint64_t need = 0;
-        for (uint32_t s = 0; s < n_seq; ++s) need += pages_missing(kvs[s], kvs[s]->len + n_steps);
-        if (need > m->free_pages.size()) return fail(ctx, OB_ERR_CAPACITY, "decode_loop: KV pool exhausted");
-        for (uint32_t s = 0; s < n_seq; ++s)
-            if (int rc = grow_pages(kvs[s], kvs[s]->len + n_steps)) return rc;
-    }
+    if (m->graph && n_seq > m->logit_cap) return fail(ctx, OB_ERR_CAPACITY, "decode_loop: more sequences than the model has logit rows for");
+    if (int rc = reserve(m, kvs, n_seq, [n_steps](uint32_t) { return n_steps; }, "decode_loop")) return rc;
     if (int rc = pre_step(m)) return rc;
     if ((uint64_t)n_steps * n_seq > m->history_cap) {
         int rc = dev_alloc(m, &m->d_history, (size_t)n_steps * n_seq);
@@ -1498,12 +1599,7 @@ int ob_decode_loop(ob_model *m, ob_kv *const *kvs, const uint32_t *first_tokens,
     bool exact = true;
     for (uint32_t s = 0; s < n_seq; ++s) exact = exact && (uint64_t)kvs[s]->len + n_steps <= m->exact_attn_max_pos;
     const MetaLayout ml(m->T);
-    for (uint32_t s = 0; s < n_seq; ++s) {
-        reinterpret_cast<uint32_t *>(m->h_meta + ml.off_tokens)[s] = first_tokens[s];
-        reinterpret_cast<uint32_t *>(m->h_meta + ml.off_positions)[s] = kvs[s]->len;
-        reinterpret_cast<uint32_t *>(m->h_meta + ml.off_npos)[s] = kvs[s]->len + 1;
-        reinterpret_cast<const int32_t **>(m->h_meta + ml.off_tables)[s] = kvs[s]->d_table;
-    }
+    for (uint32_t s = 0; s < n_seq; ++s) fill_meta_row(m, s, first_tokens[s], kvs[s]->len, kvs[s]);
     OB_CUDA(ctx, cudaMemcpyAsync(m->d_meta, m->h_meta, ml.bytes, cudaMemcpyHostToDevice, ctx->stream));
     cudaGraphExec_t exec;
     int rc = get_graph(m, n_seq, 1, exact, &exec, &key);

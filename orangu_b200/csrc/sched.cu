@@ -393,6 +393,27 @@ int ob_slot_decode(ob_slot_pool *p, uint32_t slot_id, uint32_t token, const ob_g
     return OB_OK;
 }
 
+int ob_slot_forward(ob_slot_pool *p, const uint32_t *slot_ids, uint32_t n_slots, const uint32_t *tokens, const uint32_t *n_tokens, const uint32_t *rows, uint32_t n_rows,
+                    float *out_logits) {
+    if (!p || !slot_ids || !tokens || !n_tokens || n_slots == 0) return pool_fail(p, -1, OB_ERR_INVALID, "slot_forward: bad argument");
+    std::vector<ob_kv *> kvs(n_slots);
+    std::vector<uint32_t> start(n_slots);
+    for (uint32_t i = 0; i < n_slots; ++i) {
+        if (!slot_held(p, slot_ids[i]) || !p->slots[slot_ids[i]].kv) return pool_fail(p, -1, OB_ERR_INVALID, "slot_forward: the slot is not held");
+        kvs[i] = p->slots[slot_ids[i]].kv;
+        start[i] = ob_kv_len(kvs[i]);
+    }
+    const int rc = ob_forward_rows(p->model, kvs.data(), tokens, n_tokens, start.data(), n_slots, rows, n_rows, out_logits);
+    if (rc != OB_OK) return pool_fail(p, -1, rc, ob_last_error(ob_model_ctx(p->model)));
+    std::lock_guard<std::mutex> g(p->mu);
+    for (uint32_t i = 0; i < n_slots; ++i) {
+        Slot &s = p->slots[slot_ids[i]];
+        if (n_tokens[i] == 1 && start[i] > 0) ++s.generated_tokens;
+        else s.prompt_tokens += n_tokens[i];
+    }
+    return OB_OK;
+}
+
 int ob_slot_truncate(ob_slot_pool *p, uint32_t slot_id, uint32_t new_len) {
     if (!p || !slot_held(p, slot_id) || !p->slots[slot_id].kv) return pool_fail(p, -1, OB_ERR_INVALID, "slot_truncate: the slot is not held");
     const int rc = ob_kv_truncate(p->slots[slot_id].kv, new_len);

@@ -41,11 +41,17 @@ class KvCache:
         capi.check(self.model.backend._h, self._lib.ob_kv_truncate(self._h, new_len))
 
     def read(self, layer: int, pos0: int, n: int):
-        kvd = self.model.kv_dim_local
-        k = np.empty((n, kvd), np.float32)
-        v = np.empty((n, kvd), np.float32)
+        kd, vd = self.model.cache_widths(layer)
+        k = np.empty((n, kd), np.float32)
+        v = np.empty((n, vd), np.float32)
         capi.check(self.model.backend._h, self._lib.ob_kv_read(self._h, layer, pos0, n, k.ctypes.data, v.ctypes.data))
         return k, v
+
+    def read_state(self, layer: int) -> np.ndarray:
+        """Recurrent state of a layer, [heads, dim, vdim]."""
+        out = np.empty(self.model.state_shape(layer), np.float32)
+        capi.check(self.model.backend._h, self._lib.ob_state_read(self._h, layer, out.ctypes.data))
+        return out
 
     def copy_prefix_from(self, src: "KvCache", n: int):
         """KvCache::copy_prefix_from (kv_cache.rs:1079-1100)."""
@@ -65,7 +71,109 @@ class KvCache:
             pass
 
 
-class LlamaModel:
+class DeviceModel:
+    """What every model on the device offers (ModelForward, arch/mod.rs:2035-2191): caches, steps, sampling, decode loops.  A
+    subclass makes the handle and sets ``backend``, ``_lib``, ``_h``, ``cfg`` (with ``n_embd``), ``n_vocab``, ``max_batch_tokens``."""
+
+    def new_kv_cache(self, capacity: int, paged: bool = False) -> KvCache:
+        return KvCache(self, capacity, paged)
+
+    @property
+    def free_slots(self) -> int:
+        return int(self._lib.ob_model_free_slots(self._h))
+
+    @property
+    def free_pages(self) -> int:
+        return int(self._lib.ob_model_free_pages(self._h))
+
+    @property
+    def pool_pages(self) -> int:
+        return int(self._lib.ob_model_pool_pages(self._h))
+
+    # ModelForward::forward (arch/llama.rs:1007-1032): logits of the last token
+    def forward(self, cache: KvCache, tokens, start_pos: int) -> np.ndarray:
+        return self._forward([cache], [list(tokens)], [start_pos], want_logits=True)[1][0]
+
+    # ModelForward::forward_maybe_sampling with a greedy sampler (arch/llama.rs:949-1000): next token id
+    def forward_maybe_sampling(self, cache: KvCache, tokens, start_pos: int, recent=None, repeat_penalty: float = 1.0, repeat_last_n: int = 64) -> int:
+        g = None
+        if recent is not None and repeat_penalty != 1.0:
+            g = ([np.ascontiguousarray(recent, np.uint32)], repeat_penalty, repeat_last_n)
+        return int(self._forward([cache], [list(tokens)], [start_pos], want_tokens=True, greedy=g)[0][0])
+
+    # ModelForward::forward_batch_decode (arch/mod.rs:2174-2190): one token per sequence
+    def forward_batch_decode(self, caches, tokens, want_logits: bool = False):
+        toks, logits = self._forward(list(caches), [[int(t)] for t in tokens], [len(c) for c in caches], want_tokens=True, want_logits=want_logits)
+        return (toks, logits) if want_logits else toks
+
+    def _forward(self, caches, token_lists, start_pos, want_tokens=False, want_logits=False, greedy=None):
+        n_seq = len(caches)
+        kvs = (C.c_void_p * n_seq)(*[c._h for c in caches])
+        flat = np.ascontiguousarray([t for l in token_lists for t in l], dtype=np.uint32)
+        n_tok = np.ascontiguousarray([len(l) for l in token_lists], dtype=np.uint32)
+        sp = np.ascontiguousarray(start_pos, dtype=np.uint32)
+        out_tok = np.zeros(n_seq, np.uint32) if want_tokens else None
+        out_log = np.empty((n_seq, self.n_vocab), np.float32) if want_logits else None
+        gptr = None
+        if greedy is not None:
+            recents, penalty, last_n = greedy
+            rec = np.ascontiguousarray(np.concatenate(recents), np.uint32)
+            nrec = np.ascontiguousarray([len(r) for r in recents], np.uint32)
+            gs = capi.Greedy(penalty, last_n, rec.ctypes.data, nrec.ctypes.data)
+            gptr = C.addressof(gs)
+        capi.check(self.backend._h, self._lib.ob_forward(
+            self._h, kvs, flat.ctypes.data, n_tok.ctypes.data, sp.ctypes.data, n_seq, gptr,
+            out_tok.ctypes.data if want_tokens else None, out_log.ctypes.data if want_logits else None))
+        return out_tok, out_log
+
+    def forward_rows(self, caches, token_lists, rows) -> np.ndarray:
+        """One call over all sequences, each continuing its cache; logits of the tokens whose numbers (ascending, counted through
+        the concatenated lists) are in `rows`."""
+        n_seq = len(caches)
+        kvs = (C.c_void_p * n_seq)(*[c._h for c in caches])
+        flat = np.ascontiguousarray([t for l in token_lists for t in l], dtype=np.uint32)
+        n_tok = np.ascontiguousarray([len(l) for l in token_lists], dtype=np.uint32)
+        start = np.ascontiguousarray([len(c) for c in caches], dtype=np.uint32)
+        rows = np.ascontiguousarray(rows, dtype=np.uint32)
+        out = np.empty((rows.size, self.n_vocab), np.float32)
+        capi.check(self.backend._h, self._lib.ob_forward_rows(self._h, kvs, flat.ctypes.data, n_tok.ctypes.data, start.ctypes.data, n_seq,
+                                                             rows.ctypes.data, rows.size, out.ctypes.data))
+        return out
+
+    def decode_greedy(self, cache: KvCache, token: int) -> int:
+        """One greedy step replayed from the captured CUDA graph (record_decode_chain, arch/llama.rs:302-473)."""
+        out = C.c_uint32()
+        capi.check(self.backend._h, self._lib.ob_decode_greedy(self._h, cache._h, int(token), C.byref(out)))
+        return int(out.value)
+
+    def decode_loop(self, caches, first_tokens, n_steps: int) -> np.ndarray:
+        """n_steps greedy steps for every sequence without the host in between; [n_steps, n_seq] token ids."""
+        n_seq = len(caches)
+        kvs = (C.c_void_p * n_seq)(*[c._h for c in caches])
+        ft = np.ascontiguousarray(first_tokens, dtype=np.uint32)
+        out = np.empty((n_steps, n_seq), np.uint32)
+        capi.check(self.backend._h, self._lib.ob_decode_loop(self._h, kvs, ft.ctypes.data, n_seq, n_steps, out.ctypes.data))
+        return out
+
+    def last_hidden(self, n_tokens: int) -> np.ndarray:
+        out = np.empty((n_tokens, self.cfg["n_embd"]), np.float32)
+        capi.check(self.backend._h, self._lib.ob_last_hidden(self._h, n_tokens, out.ctypes.data))
+        return out
+
+    def close(self):
+        if self._h:
+            self._lib.ob_model_destroy(self._h)
+            self._h = None
+
+    def __del__(self):
+        try:
+            if self.backend._h:
+                self.close()
+        except Exception:
+            pass
+
+
+class LlamaModel(DeviceModel):
     """Built from a dict of named tensors (GGUF names, arch/llama.rs:125-183): each value is
     ``{"data": np.ndarray, "type": ggml_type, "in_dim": .., "out_dim": ..}``; norm vectors are f32."""
 
@@ -141,87 +249,11 @@ class LlamaModel:
         self.max_batch_tokens = max_batch_tokens
         return self
 
-    def new_kv_cache(self, capacity: int, paged: bool = False) -> KvCache:
-        return KvCache(self, capacity, paged)
-
-    @property
-    def free_pages(self) -> int:
-        return int(self._lib.ob_model_free_pages(self._h))
-
-    @property
-    def pool_pages(self) -> int:
-        return int(self._lib.ob_model_pool_pages(self._h))
-
-    # ModelForward::forward (arch/llama.rs:1007-1032): logits of the last token
-    def forward(self, cache: KvCache, tokens, start_pos: int) -> np.ndarray:
-        return self._forward([cache], [list(tokens)], [start_pos], want_logits=True)[1][0]
-
-    # ModelForward::forward_maybe_sampling with a greedy sampler (arch/llama.rs:949-1000): next token id
-    def forward_maybe_sampling(self, cache: KvCache, tokens, start_pos: int, recent=None, repeat_penalty: float = 1.0, repeat_last_n: int = 64) -> int:
-        g = None
-        if recent is not None and repeat_penalty != 1.0:
-            g = ([np.ascontiguousarray(recent, np.uint32)], repeat_penalty, repeat_last_n)
-        return int(self._forward([cache], [list(tokens)], [start_pos], want_tokens=True, greedy=g)[0][0])
-
-    # ModelForward::forward_batch_decode (arch/mod.rs:2174-2190): one token per sequence
-    def forward_batch_decode(self, caches, tokens, want_logits: bool = False):
-        toks, logits = self._forward(list(caches), [[int(t)] for t in tokens], [len(c) for c in caches], want_tokens=True, want_logits=want_logits)
-        return (toks, logits) if want_logits else toks
-
-    def _forward(self, caches, token_lists, start_pos, want_tokens=False, want_logits=False, greedy=None):
-        n_seq = len(caches)
-        kvs = (C.c_void_p * n_seq)(*[c._h for c in caches])
-        flat = np.ascontiguousarray([t for l in token_lists for t in l], dtype=np.uint32)
-        n_tok = np.ascontiguousarray([len(l) for l in token_lists], dtype=np.uint32)
-        sp = np.ascontiguousarray(start_pos, dtype=np.uint32)
-        out_tok = np.zeros(n_seq, np.uint32) if want_tokens else None
-        out_log = np.empty((n_seq, self.n_vocab), np.float32) if want_logits else None
-        gptr = None
-        if greedy is not None:
-            recents, penalty, last_n = greedy
-            rec = np.ascontiguousarray(np.concatenate(recents), np.uint32)
-            nrec = np.ascontiguousarray([len(r) for r in recents], np.uint32)
-            gs = capi.Greedy(penalty, last_n, rec.ctypes.data, nrec.ctypes.data)
-            gptr = C.addressof(gs)
-        capi.check(self.backend._h, self._lib.ob_forward(
-            self._h, kvs, flat.ctypes.data, n_tok.ctypes.data, sp.ctypes.data, n_seq, gptr,
-            out_tok.ctypes.data if want_tokens else None, out_log.ctypes.data if want_logits else None))
-        return out_tok, out_log
-
-    def decode_greedy(self, cache: KvCache, token: int) -> int:
-        """One greedy step replayed from the captured CUDA graph (record_decode_chain, arch/llama.rs:302-473)."""
-        out = C.c_uint32()
-        capi.check(self.backend._h, self._lib.ob_decode_greedy(self._h, cache._h, int(token), C.byref(out)))
-        return int(out.value)
-
-    def decode_loop(self, caches, first_tokens, n_steps: int) -> np.ndarray:
-        """n_steps greedy steps for every sequence without the host in between; [n_steps, n_seq] token ids."""
-        n_seq = len(caches)
-        kvs = (C.c_void_p * n_seq)(*[c._h for c in caches])
-        ft = np.ascontiguousarray(first_tokens, dtype=np.uint32)
-        out = np.empty((n_steps, n_seq), np.uint32)
-        capi.check(self.backend._h, self._lib.ob_decode_loop(self._h, kvs, ft.ctypes.data, n_seq, n_steps, out.ctypes.data))
-        return out
+    def cache_widths(self, layer: int):
+        return self.kv_dim_local, self.kv_dim_local
 
     def profile_gemv(self, ggml_type: int, iters: int, variant: int = 0):
         """(ms_total, bytes_per_pass, launches_per_pass) of the single-token GEMVs of one weight type, run alone."""
         ms, nbytes, nl = C.c_float(), C.c_uint64(), C.c_uint32()
         capi.check(self.backend._h, self._lib.ob_profile_gemv(self._h, ggml_type, variant, iters, C.byref(ms), C.byref(nbytes), C.byref(nl)))
         return ms.value, nbytes.value, nl.value
-
-    def last_hidden(self, n_tokens: int) -> np.ndarray:
-        out = np.empty((n_tokens, self.cfg["n_embd"]), np.float32)
-        capi.check(self.backend._h, self._lib.ob_last_hidden(self._h, n_tokens, out.ctypes.data))
-        return out
-
-    def close(self):
-        if self._h:
-            self._lib.ob_model_destroy(self._h)
-            self._h = None
-
-    def __del__(self):
-        try:
-            if self.backend._h:
-                self.close()
-        except Exception:
-            pass

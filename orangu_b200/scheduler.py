@@ -115,6 +115,18 @@ class SlotPool:
         self._check(None, rc)
         return SlotGuard(self, index)
 
+    def forward(self, guards, token_lists, rows) -> np.ndarray:
+        """The next tokens of several held slots -- portions of prompts and single tokens alike -- as one batch; logits of the
+        tokens whose numbers (ascending, counted through the concatenated lists) are in `rows`."""
+        ids = np.ascontiguousarray([g.index for g in guards], np.uint32)
+        flat = np.ascontiguousarray([t for l in token_lists for t in l], np.uint32)
+        n_tok = np.ascontiguousarray([len(l) for l in token_lists], np.uint32)
+        rows = np.ascontiguousarray(rows, np.uint32)
+        out = np.empty((rows.size, self.model.n_vocab), np.float32)
+        self._check(None, self._lib.ob_slot_forward(self._h, ids.ctypes.data, ids.size, flat.ctypes.data, n_tok.ctypes.data, rows.ctypes.data, rows.size,
+                                                    out.ctypes.data))
+        return out
+
     def snapshot(self):
         n = int(self._lib.ob_slot_pool_snapshot(self._h, None, 0))
         arr = (SlotState * n)()

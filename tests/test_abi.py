@@ -125,6 +125,24 @@ def test_struct_layouts_agree_between_header_binding_and_integration_notes(lib):
     assert header
 
 
+def test_layered_struct_layouts_agree(lib):
+    """The structs of models given as a list of layers: C sizes == ctypes sizes, and the written Rust structs name every field."""
+    from orangu_b200 import capi
+
+    out = _compile_and_run(
+        '#include <cstdio>\n#include <cstddef>\n#include "orangu_b200.h"\n'
+        'int main(){ std::printf("%zu %zu %zu %zu %zu %zu\\n", sizeof(ob_mixer_desc), sizeof(ob_block_desc), sizeof(ob_layered_desc),'
+        ' offsetof(ob_mixer_desc, decay), offsetof(ob_block_desc, w_gate), offsetof(ob_layered_desc, token_embd)); }\n')
+    assert [int(v) for v in out.split()] == [C.sizeof(capi.MixerDesc), C.sizeof(capi.BlockDesc), C.sizeof(capi.LayeredDesc),
+                                             capi.MixerDesc.decay.offset, capi.BlockDesc.w_gate.offset, capi.LayeredDesc.token_embd.offset]
+    notes = open(os.path.join(ROOT, "INTEGRATION.md")).read()
+    for name, struct in (("ob_mixer_desc", capi.MixerDesc), ("ob_block_desc", capi.BlockDesc), ("ob_layered_desc", capi.LayeredDesc)):
+        rust = notes[notes.index(f"pub struct {name}"):]
+        rust = rust[:rust.index("}")]
+        for field, _ in struct._fields_:
+            assert f"pub {field}:" in rust, f"INTEGRATION.md's {name} lacks {field}"
+
+
 def test_cpp_model_and_slot_pool_wrappers_compile():
     """The ModelForward / KvCache / SlotPool part of the C++ mirror, compiled with warnings on and linked against the library
     (run without a device: try_init_index gives an empty optional and main returns)."""
@@ -133,7 +151,8 @@ def test_cpp_model_and_slot_pool_wrappers_compile():
            ' try { orangu::LlamaModel m(*be, d); auto kv = m.new_kv_cache(16, true); auto t = m.forward_maybe_sampling(kv, {1, 2, 3}, 0);\n'
            '  (void)m.decode_greedy(kv, t); (void)m.forward(kv, {t}, kv.len()); ob_slot_pool_desc pd{2, 64, 0, 0, 0, 1}; orangu::SlotPool pool(m, pd);\n'
            '  if (auto g = pool.try_acquire(0)) { auto x = g->prefill({1, 2}); (void)g->decode(x); g->truncate(1); }\n'
-           '  (void)pool.snapshot(); (void)pool.stats(); std::vector<orangu::KvCache *> c{&kv}; (void)m.forward_batch_decode(c, {1}); }\n'
+           '  (void)pool.snapshot(); (void)pool.stats(); std::vector<orangu::KvCache *> c{&kv}; (void)m.forward_batch_decode(c, {1}); (void)m.forward_rows(c, {{1, 2}}, {0, 1});\n'
+           '  ob_layered_desc ld{}; orangu::Model lm(*be, ld); (void)lm.n_vocab(); }\n'
            ' catch (const std::exception &) { return 0; } return 0; }\n')
     from orangu_b200 import capi
 
