@@ -38,7 +38,7 @@ class TensorDict:
 
     def f32(self, name, shape=None):
         a = self._get(name, shape)
-        return self._from(a) if a.dtype == np.uint16 else np.ascontiguousarray(a, np.float32)
+        return self._from(a) if a.dtype == np.uint16 else np.array(a, np.float32, order="C")
 
 
 def _latent_attention(d: Describer, t, at: str, mx: dict, width: int) -> capi.MixerDesc:

@@ -57,7 +57,7 @@ class SafetensorsFile:
 
     def f32(self, name: str, shape=None) -> np.ndarray:
         a = self.raw(name, shape)
-        return from_bf16(a) if self.dtype(name) == "BF16" else np.ascontiguousarray(a, np.float32)
+        return from_bf16(a) if self.dtype(name) == "BF16" else np.array(a, np.float32, order="C")
 
 
 def from_bf16(bits: np.ndarray) -> np.ndarray:
@@ -65,7 +65,7 @@ def from_bf16(bits: np.ndarray) -> np.ndarray:
 
 
 def to_bf16(x: np.ndarray) -> np.ndarray:
-    u = np.ascontiguousarray(x, np.float32).view(np.uint32)
+    u = np.array(x, np.float32, order="C").view(np.uint32)
     return ((u + 0x7FFF + ((u >> 16) & 1)) >> 16).astype(np.uint16)
 
 
