@@ -63,6 +63,10 @@ def parse_args():
     ap.add_argument("--context", type=int, default=4096)
     ap.add_argument("--batch64-steps", type=int, default=16, help="steps of the 64-sequence decode measured as an extra (0 = skip)")
     ap.add_argument("--no-cpu-baseline", action="store_true")
+    ap.add_argument("--fenipel", default="", metavar="SIZE[,SIZE]", help="instead of the workload above: prefill and decode of Fenipel at these sizes "
+                    "(1b, 8b; random weights) beside the quantized Llama shape of the same widths")
+    ap.add_argument("--fenipel-layers", type=int, default=8, help="layers of both models in that comparison")
+    ap.add_argument("--fenipel-only", action="store_true", help="leave the Llama shape out")
     return ap.parse_args()
 
 
@@ -317,6 +321,124 @@ def run_reference(args, rank: int, world: int):
 
 
 # ---------------------------------------------------------------------------------------- our arm
+FENIPEL_SIZES = {  # widths and feed-forwards of the Llama shapes of the same name; half of the layers attend, half retain
+    "1b": {"width": 2048, "ff": 8192, "vocab": 32768, "side": 128,
+           "latent": {"heads": 16, "dim": 128, "rot_dim": 64, "vdim": 128, "kv_rank": 384, "window": 1024},
+           "retention": {"heads": 8, "dim": 128, "vdim": 256}},
+    "8b": {"width": 4096, "ff": 14336, "vocab": 32768, "side": 256,
+           "latent": {"heads": 32, "dim": 128, "rot_dim": 64, "vdim": 128, "kv_rank": 512, "window": 1024},
+           "retention": {"heads": 16, "dim": 128, "vdim": 256}},
+}
+
+
+def fenipel_model(size: str, n_layer: int):
+    """Configuration and random bfloat16 tensors (bits); one pool of normal values is dealt out over all of them."""
+    import numpy as np
+    from orangu_b200.safetensors import to_bf16
+
+    z = FENIPEL_SIZES[size]
+    E, V, sd = z["width"], z["vocab"], z["side"]
+    pool = np.random.default_rng(1).normal(size=1 << 22).astype(np.float32)
+    cache = {}
+
+    def lin(o, i):
+        bits = cache.setdefault(i, to_bf16(pool * i ** -0.5))
+        return np.resize(np.roll(bits, (o * 7919) % bits.size), (o, i))
+
+    layers, t = [], {"embed": lin(V, E), "head": lin(V, E), "final.norm": to_bf16(np.float32(1)), "side.embed": lin(V, n_layer * sd)}
+    for n in range(n_layer):
+        at, m = f"l{n}.mix.", dict(z["latent" if n % 2 == 0 else "retention"])
+        H, d, v = m["heads"], m["dim"], m["vdim"]
+        if n % 2 == 0:
+            R, K = m["rot_dim"], m["kv_rank"]
+            m.update(mask={"size": m.pop("window")}, rot={"base": 10000.0, "dims": R}, scale=(d + R) ** -0.5)
+            t.update({at + "q": lin(H * (d + R), E), at + "dkv": lin(K + R, E), at + "dkv.norm": to_bf16(np.ones(K)), at + "uk": lin(H * d, K), at + "uv": lin(H * v, K),
+                      at + "g": lin(H, E)})
+        else:
+            m.update(rot={"base": 10000.0, "dims": d}, decay=[1 - 2.0 ** (-5 - 0.5 * h) for h in range(H)])
+            t.update({at + "q": lin(H * d, E), at + "k": lin(H * d, E), at + "v": lin(H * v, E), at + "g": lin(H * v, E)})
+        t.update({at + "o": lin(E, H * v), f"l{n}.norm1": to_bf16(np.float32(1)), f"l{n}.mlp.gate": lin(z["ff"], E), f"l{n}.mlp.up": lin(z["ff"], E),
+                  f"l{n}.mlp.down": lin(E, z["ff"]), f"l{n}.side.gate": lin(sd, E), f"l{n}.side.proj": lin(E, sd), f"l{n}.side.norm": to_bf16(np.ones(E))})
+        layers.append({"type": "latent_attention" if n % 2 == 0 else "retention", "mixer": m, "mlp": {"kind": "dense", "ff": z["ff"], "limit": 7.0}})
+    return {"architecture": "Fenipel", "vocab": V, "width": E, "norm": {"eps": 1e-6}, "token_side": {"dim": sd}, "layers": layers}, t
+
+
+def time_model(be, model, vocab: int, weight_bytes: int, cache_bytes_per_token: float, flops_per_token: float, steps: int, warmup: int, prompt: int = 4096):
+    """Prefill of one prompt and greedy decode loops at batch 1, 8 and 64 (device time, CUDA events; weights exceed L2).
+    cache_bytes_per_token: cache and state traffic of one decoded token at this context."""
+    import numpy as np
+
+    rng = np.random.default_rng(0)
+    toks = rng.integers(0, vocab, prompt)
+    peaks = json.load(open(os.path.join(ROOT, "MEASURED_PEAKS.json"))) if os.path.exists(os.path.join(ROOT, "MEASURED_PEAKS.json")) else {}
+    hbm, tf = peaks.get("hbm_gbs", 6650.0), peaks.get("bf16_tflops_sustained", 1400.0)
+    out = {"decode": {}}
+    room = prompt + 4 * (steps + warmup)
+    kv, ms = model.new_kv_cache(room, paged=True), []
+    for _ in range(4):
+        kv.truncate(0)
+        model.forward_maybe_sampling(kv, toks, 0)
+        ms.append(be.last_device_ms())
+    best = min(ms[1:])
+    out["prefill"] = {"tokens": prompt, "ms": best, "tok_s": prompt / best * 1e3, "of_bf16_sustained": prompt * flops_per_token / (best * 1e-3) / (tf * 1e12)}
+    kvs = [kv]
+    for batch in (1, 8, 64):
+        while len(kvs) < batch:
+            k = model.new_kv_cache(room, paged=True)
+            k.copy_prefix_from(kv, len(kv))
+            kvs.append(k)
+        first = [int(x) for x in rng.integers(0, vocab, batch)]
+        model.decode_loop(kvs[:batch], first, warmup)
+        model.decode_loop(kvs[:batch], first, steps)
+        t = be.last_device_ms() / steps
+        need = weight_bytes + batch * cache_bytes_per_token
+        out["decode"][str(batch)] = {"ms_per_step": t, "tok_s": batch / t * 1e3, "bytes_per_step": need, "of_hbm": need / (t * 1e-3) / (hbm * 1e9)}
+    for k in kvs:
+        k.close()
+    return out
+
+
+def run_fenipel(args):
+    """--fenipel: one JSON line with both models at every size.  bf16 weights against Q4_K_M: equal parameter counts are not
+    equal bytes, so fractions of the roofline are what compares."""
+    import orangu_b200
+    from orangu_b200 import synth
+
+    be = orangu_b200.CudaBackend.init(0)
+    steps, warmup, L = args.steps, max(3, args.warmup), args.fenipel_layers
+    result = {"bench": "fenipel", "data": "synthetic", "dtype": "bf16", "layers": L, "steps": steps, "warmup": warmup, "sizes": {}}
+    clocks = ClockSampler(0)
+    clocks.start()
+    for size in args.fenipel.split(","):
+        cfg, t = fenipel_model(size, L)
+        n = sum(a.size for k, a in t.items() if not k.endswith("embed"))
+        z, prompt = FENIPEL_SIZES[size], 4096
+        la, re = z["latent"], z["retention"]
+        win = min(la["window"], prompt)
+        n_lat, n_ret = (L + 1) // 2, L // 2
+        cache = n_lat * win * (la["kv_rank"] + la["rot_dim"]) * 2 + n_ret * re["heads"] * re["dim"] * re["vdim"] * 8
+        flops = 2 * n + n_lat * 2 * win * la["heads"] * (la["dim"] + la["rot_dim"] + la["vdim"]) + n_ret * 4 * re["heads"] * re["dim"] * re["vdim"]
+        m = orangu_b200.FenipelModel(be, cfg, t, max_seq_len=8192, max_batch_tokens=prompt, kv_pool_tokens=64 * 4480, state_slots=64)
+        entry = {"fenipel": dict(time_model(be, m, z["vocab"], 2 * n, cache, flops, steps, warmup), parameters=n)}
+        m.close()
+        del t
+        if not args.fenipel_only:
+            c = dict(synth.CONFIGS[size], n_layer=L, n_vocab=z["vocab"])
+            tensors = synth.model_tensors(c, seed=7)
+            wb = sum(x["data"].nbytes for k, x in tensors.items() if not k.startswith("token_embd"))
+            elems = sum(x["in_dim"] * x["out_dim"] for k, x in tensors.items() if not k.startswith("token_embd") and "norm" not in k)
+            kvd = c["n_head_kv"] * c["head_dim"]
+            m = orangu_b200.LlamaModel(be, c, tensors, max_seq_len=8192, max_batch_tokens=512, kv_pool_tokens=64 * 4480)
+            fl = 2 * elems + L * 2 * (prompt / 2) * c["n_head"] * c["head_dim"] * 2
+            entry["llama_q4km"] = dict(time_model(be, m, z["vocab"], wb, L * prompt * kvd * 4, fl, steps, warmup), parameters=elems)
+            m.close()
+            del tensors
+        result["sizes"][size] = entry
+    result["clocks"] = clocks.stop()
+    be.close()
+    print(json.dumps(result))
+
+
 def main():
     args = parse_args()
     rank = int(os.environ.get("RANK", "0"))
@@ -324,6 +446,9 @@ def main():
     local_rank = int(os.environ.get("LOCAL_RANK", "0"))
     if args.impl == "reference":
         run_reference(args, rank, world)
+        return
+    if args.fenipel:
+        run_fenipel(args)
         return
 
     import torch
