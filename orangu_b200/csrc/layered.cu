@@ -206,9 +206,8 @@ void LayeredGraph::layers(uint32_t T, uint32_t n_seq, const RowSpan *spans, uint
     const MetaLayout ml(m->T);
     const uint32_t *tokens = reinterpret_cast<const uint32_t *>(m->d_meta + ml.off_tokens);
     const bool single = n_seq == T;
-    launch_embed_bf16(embd, width, tokens, T, m->x, st);
-    launch_norm_scalar(m->x, width, nullptr, T, eps, L[0].norm_gain, h, h_pitch, f32, st);
-    m->ctx->launches += 2;
+    launch_embed_norm(embd, width, tokens, T, m->x, eps, L[0].norm_gain, h, h_pitch, f32, st);
+    m->ctx->launches++;
     for (size_t li = 0; li < L.size(); ++li) {
         const LayerPlan &P = L[li];
         LinArgs in = product(P.in, h, h_pitch, T);

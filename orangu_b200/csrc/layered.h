@@ -54,7 +54,9 @@ int linear_take_status();        // 1 when a bounded wait inside a product ran o
 void linear_mark_launched();     // a replayed graph may have run one of the tensor-core products
 
 // ---- mixers.cu -------------------------------------------------------------------------------------------------------
-void launch_embed_bf16(const __nv_bfloat16 *table, uint32_t width, const uint32_t *tokens, uint32_t T, float *x, cudaStream_t st);
+// x = embedding rows, h = x / rms(x) * gain as activation.
+void launch_embed_norm(const __nv_bfloat16 *table, uint32_t width, const uint32_t *tokens, uint32_t T, float *x, float eps, float gain, void *h, uint32_t h_pitch,
+                       bool f32, cudaStream_t st);
 // h[i] = x[row i] / rms(x[row i]) * gain, as activation; rows == nullptr: row i.
 void launch_norm_scalar(const float *x, uint32_t width, const uint32_t *rows, uint32_t n, float eps, float gain, void *h, uint32_t h_pitch, bool f32,
                         cudaStream_t st);

@@ -15,10 +15,6 @@ namespace ob {
 namespace {
 
 // ---- activations -------------------------------------------------------------------------------------------------------
-template <typename TA> __device__ __forceinline__ TA to_act(float v);
-template <> __device__ __forceinline__ float to_act<float>(float v) { return v; }
-template <> __device__ __forceinline__ __nv_bfloat16 to_act<__nv_bfloat16>(float v) { return __float2bfloat16_rn(v); }
-
 __device__ __forceinline__ void unpack8(const uint4 &w, float (&f)[8]) {  // eight bfloat16
     const uint32_t u[4] = {w.x, w.y, w.z, w.w};
 #pragma unroll
@@ -256,18 +252,23 @@ __global__ void __launch_bounds__(256) linear_simt_kernel(LinArgs a) {
 }
 
 // ---- tcgen05 ---------------------------------------------------------------------------------------------------------------
-// One CTA: 128 tokens (the lanes of tensor memory) x BN weight rows (its columns), K in steps of 64 columns = one 128-byte
+// Tiles of 128 tokens (the lanes of tensor memory) x BN weight rows (its columns), K in steps of 64 columns = one 128-byte
 // swizzled row per operand row.  Warps 0-3 epilogue (warp w reads lane quadrant w), warp 4 issues the TMA loads, warp 5 owns
 // tensor memory and issues the MMAs.  The weight tiles of the first stages are requested before the wait for the predecessor.
+// BN = 256 is persistent with two accumulators, so a tile's epilogue runs under the next tile's products; narrower tiles are one
+// per CTA, two CTAs per SM.  AR: token rows that are loaded.  With few tokens the other rows of the operand are whatever the
+// shared memory holds -- they only reach tensor-memory lanes nobody reads -- and the room goes into more stages of weights.
 constexpr int LT_M = 128, LT_EPI_WARPS = 4, LT_TMA_WARP = 4, LT_MMA_WARP = 5, LT_THREADS = 6 * 32;
-constexpr uint32_t LT_A_BYTES = LT_M * 128;
+constexpr uint32_t LT_GROUP = 16;  // token tiles that share the weight tiles of a wave: both operands stay in L2
 
-template <int BN>
+template <int BN, int AR>
 struct LtSmem {
-    static constexpr uint32_t STAGES = BN == 256 ? 4 : BN == 128 ? 3 : BN == 64 ? 4 : 5;
-    static constexpr uint32_t B_BYTES = BN * 128;
-    static constexpr uint32_t A = 0, B = STAGES * LT_A_BYTES, FULL = B + STAGES * B_BYTES, EMPTY = FULL + 8 * STAGES, DONE = EMPTY + 8 * STAGES, SLOT = DONE + 8,
-                              ABORT = SLOT + 8, BYTES = ABORT + 8, ALLOC = BYTES + 1024;
+    static constexpr uint32_t A_BYTES = AR * 128, B_BYTES = BN * 128, SLACK = LT_M * 128 - A_BYTES;  // the MMA reads 128 rows from every stage's base
+    static constexpr uint32_t STAGES = BN == 256 ? 4 : (104 * 1024 - SLACK) / (A_BYTES + B_BYTES);
+    static constexpr uint32_t NBUF = BN == 256 ? 2 : 1, COLS = NBUF * BN;
+    static constexpr uint32_t B = 0, A = STAGES * B_BYTES, FULL = A + STAGES * A_BYTES + SLACK, EMPTY = FULL + 8 * STAGES, ACC_FULL = EMPTY + 8 * STAGES,
+                              ACC_EMPTY = ACC_FULL + 8 * NBUF, SLOT = ACC_EMPTY + 8 * NBUF, ABORT = SLOT + 8, BYTES = ABORT + 8, ALLOC = BYTES + 1024;
+    static_assert(STAGES >= 3 && ALLOC <= (BN == 256 ? 227 : 113) * 1024, "shared memory plan does not fit");
 };
 
 // D (tensor memory, fp32, 128 lanes x N columns) [+]= A (128 x 16 bf16, K-major) * B (N x 16 bf16, K-major)^T
@@ -281,15 +282,27 @@ __device__ __forceinline__ void umma_bf16(uint32_t d_tmem, uint64_t a_desc, uint
 // Instruction descriptor: fp32 accumulator, A and B bfloat16, both K-major, N columns, M = 128.
 __host__ __device__ constexpr uint32_t umma_idesc_bf16(uint32_t n) { return (1u << 4) | (1u << 7) | (1u << 10) | ((n >> 3) << 17) | ((128u >> 4) << 24); }
 
-template <int BN>
+struct LtTiles {
+    uint32_t rows, toks, total;  // weight tiles and token tiles of one batch entry, tiles of all
+};
+__device__ __forceinline__ void lt_tile(const LtTiles &g, uint32_t tile, uint32_t *batch, uint32_t *rt, uint32_t *tt) {
+    const uint32_t per = g.rows * g.toks;
+    *batch = tile / per;
+    uint32_t i = tile - *batch * per;
+    const uint32_t grp = i / (LT_GROUP * g.rows), width = min(LT_GROUP, g.toks - grp * LT_GROUP);
+    i -= grp * LT_GROUP * g.rows;
+    *rt = i / width;
+    *tt = grp * LT_GROUP + i % width;
+}
+
+template <int BN, int AR>
 __global__ void __launch_bounds__(LT_THREADS, BN == 256 ? 1 : 2)
-linear_tc5_kernel(const __grid_constant__ CUtensorMap tm_x, const __grid_constant__ CUtensorMap tm_w, const __grid_constant__ LinArgs a) {
-    using S = LtSmem<BN>;
+linear_tc5_kernel(const __grid_constant__ CUtensorMap tm_x, const __grid_constant__ CUtensorMap tm_w, const __grid_constant__ LinArgs a, const LtTiles g) {
+    using S = LtSmem<BN, AR>;
     extern __shared__ uint8_t smem_raw[];
     const uint32_t sbase = (smem_u32(smem_raw) + 1023u) & ~1023u;
     uint8_t *smem = smem_raw + (sbase - smem_u32(smem_raw));
     const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
-    const uint32_t r0 = blockIdx.x * BN, t0 = blockIdx.y * LT_M, batch = blockIdx.z;
     volatile uint32_t *abort = reinterpret_cast<volatile uint32_t *>(smem + S::ABORT);
     const uint32_t n_steps = a.kp / 64;
 
@@ -298,12 +311,15 @@ linear_tc5_kernel(const __grid_constant__ CUtensorMap tm_x, const __grid_constan
             mbar_init(sbase + S::FULL + 8 * s, 1);
             mbar_init(sbase + S::EMPTY + 8 * s, 1);
         }
-        mbar_init(sbase + S::DONE, 1);
+        for (uint32_t b = 0; b < S::NBUF; ++b) {
+            mbar_init(sbase + S::ACC_FULL + 8 * b, 1);
+            mbar_init(sbase + S::ACC_EMPTY + 8 * b, LT_EPI_WARPS);
+        }
         *abort = 0u;
         asm volatile("fence.mbarrier_init.release.cluster;" ::: "memory");
         asm volatile("fence.proxy.async.shared::cta;" ::: "memory");
     }
-    if (warp == LT_MMA_WARP) tmem_alloc(sbase + S::SLOT, BN);
+    if (warp == LT_MMA_WARP) tmem_alloc(sbase + S::SLOT, S::COLS);
     tc_fence_before();
     __syncthreads();
     tc_fence_after();
@@ -312,50 +328,73 @@ linear_tc5_kernel(const __grid_constant__ CUtensorMap tm_x, const __grid_constan
 
     if (warp == LT_TMA_WARP) {
         if (lane == 0) {
-            const int32_t wy = (int32_t)(batch * a.n_rows + r0), xc = (int32_t)(batch * a.x_step);
-            const uint32_t head = min(n_steps, S::STAGES);
-            for (uint32_t it = 0; it < head; ++it) {
-                mbar_expect_tx(sbase + S::FULL + 8 * it, LT_A_BYTES + S::B_BYTES);
-                tma_load_2d(sbase + S::B + it * S::B_BYTES, &tm_w, (int32_t)(it * 64), wy, sbase + S::FULL + 8 * it);
-            }
-            pdl_wait();
-            for (uint32_t it = 0; it < n_steps; ++it) {
-                const uint32_t s = it % S::STAGES, full = sbase + S::FULL + 8 * s;
-                if (it >= S::STAGES) {
-                    if (!mbar_wait(sbase + S::EMPTY + 8 * s, ((it / S::STAGES) & 1u) ^ 1u, abort)) break;
-                    mbar_expect_tx(full, LT_A_BYTES + S::B_BYTES);
-                    tma_load_2d(sbase + S::B + s * S::B_BYTES, &tm_w, (int32_t)(it * 64), wy, full);
+            const uint32_t ahead = min(n_steps, S::STAGES);
+            uint32_t it = 0;
+            bool ok = true;
+            for (uint32_t tile = blockIdx.x; ok && tile < g.total; tile += gridDim.x) {
+                uint32_t batch, rt, tt;
+                lt_tile(g, tile, &batch, &rt, &tt);
+                const int32_t wy = (int32_t)(batch * a.n_rows + rt * BN), xc = (int32_t)(batch * a.x_step), xy = (int32_t)(tt * LT_M);
+                auto weights = [&](uint32_t k, uint32_t s) {
+                    mbar_expect_tx(sbase + S::FULL + 8 * s, S::A_BYTES + S::B_BYTES);
+                    tma_load_2d(sbase + S::B + s * S::B_BYTES, &tm_w, (int32_t)(k * 64), wy, sbase + S::FULL + 8 * s);
+                };
+                if (tile == blockIdx.x) {
+                    for (uint32_t k = 0; k < ahead; ++k) weights(k, k);
+                    pdl_wait();
                 }
-                tma_load_2d(sbase + S::A + s * LT_A_BYTES, &tm_x, xc + (int32_t)(it * 64), (int32_t)t0, full);
+                for (uint32_t k = 0; k < n_steps; ++k, ++it) {
+                    const uint32_t s = it % S::STAGES;
+                    if (it >= S::STAGES && !mbar_wait(sbase + S::EMPTY + 8 * s, ((it / S::STAGES) & 1u) ^ 1u, abort)) {
+                        ok = false;
+                        break;
+                    }
+                    if (it >= ahead) weights(k, s);
+                    tma_load_2d(sbase + S::A + s * S::A_BYTES, &tm_x, xc + (int32_t)(k * 64), xy, sbase + S::FULL + 8 * s);
+                }
             }
         }
     } else if (warp == LT_MMA_WARP) {
         pdl_wait();
         if (lane == 0) {
             constexpr uint32_t idesc = umma_idesc_bf16(BN);
-            for (uint32_t it = 0; it < n_steps; ++it) {
-                const uint32_t s = it % S::STAGES;
-                if (!mbar_wait(sbase + S::FULL + 8 * s, (it / S::STAGES) & 1u, abort)) break;
-                tc_fence_after();
-                const uint64_t da = umma_desc_sw128(sbase + S::A + s * LT_A_BYTES), db = umma_desc_sw128(sbase + S::B + s * S::B_BYTES);
+            uint32_t it = 0, n = 0;
+            bool ok = true;
+            for (uint32_t tile = blockIdx.x; ok && tile < g.total; tile += gridDim.x, ++n) {
+                const uint32_t buf = n % S::NBUF;
+                if (n >= S::NBUF && !mbar_wait(sbase + S::ACC_EMPTY + 8 * buf, ((n / S::NBUF) & 1u) ^ 1u, abort)) break;
+                for (uint32_t k = 0; k < n_steps; ++k, ++it) {
+                    const uint32_t s = it % S::STAGES;
+                    if (!mbar_wait(sbase + S::FULL + 8 * s, (it / S::STAGES) & 1u, abort)) {
+                        ok = false;
+                        break;
+                    }
+                    tc_fence_after();
+                    const uint64_t da = umma_desc_sw128(sbase + S::A + s * S::A_BYTES), db = umma_desc_sw128(sbase + S::B + s * S::B_BYTES);
 #pragma unroll
-                for (uint32_t j = 0; j < 4; ++j) umma_bf16(tmem, da + 2 * j, db + 2 * j, idesc, (it | j) ? 1u : 0u);
-                umma_commit(sbase + S::EMPTY + 8 * s);
+                    for (uint32_t j = 0; j < 4; ++j) umma_bf16(tmem + buf * BN, da + 2 * j, db + 2 * j, idesc, (k | j) ? 1u : 0u);
+                    umma_commit(sbase + S::EMPTY + 8 * s);
+                }
+                if (ok) umma_commit(sbase + S::ACC_FULL + 8 * buf);
             }
-            umma_commit(sbase + S::DONE);
         }
     } else {
         pdl_wait();
-        if (mbar_wait(sbase + S::DONE, 0, abort)) {
+        uint32_t n = 0;
+        for (uint32_t tile = blockIdx.x; tile < g.total; tile += gridDim.x, ++n) {
+            const uint32_t buf = n % S::NBUF;
+            uint32_t batch, rt, tt;
+            lt_tile(g, tile, &batch, &rt, &tt);
+            if (!mbar_wait(sbase + S::ACC_FULL + 8 * buf, (n / S::NBUF) & 1u, abort)) break;
             tc_fence_after();
-            const uint32_t t = t0 + warp * 32 + lane;
+            const uint32_t t = tt * LT_M + warp * 32 + lane;
 #pragma unroll 1
             for (int c = 0; c < BN / 32; ++c) {
                 uint32_t u[32];
                 __syncwarp();
-                tmem_ld32(tmem + ((uint32_t)(warp * 32) << 16) + c * 32, u);
+                tmem_ld32(tmem + ((uint32_t)(warp * 32) << 16) + buf * BN + c * 32, u);
                 tmem_ld_wait();
-                const uint32_t r = r0 + c * 32;
+                const uint32_t r = rt * BN + c * 32;
                 if (t < a.T && r < a.n_rows) {
                     float v[32];
 #pragma unroll
@@ -363,6 +402,9 @@ linear_tc5_kernel(const __grid_constant__ CUtensorMap tm_x, const __grid_constan
                     epilogue_store<__nv_bfloat16, 32>(a, batch, t, r, v);
                 }
             }
+            tc_fence_before();
+            __syncwarp();
+            if (lane == 0) mbar_arrive(sbase + S::ACC_EMPTY + 8 * buf);
         }
     }
     __syncwarp();
@@ -371,17 +413,32 @@ linear_tc5_kernel(const __grid_constant__ CUtensorMap tm_x, const __grid_constan
     }
     tc_fence_before();
     __syncthreads();
-    if (warp == LT_MMA_WARP) tmem_dealloc(tmem, BN);
+    if (warp == LT_MMA_WARP) tmem_dealloc(tmem, S::COLS);
+}
+
+template <int BN, int AR>
+cudaError_t configure_tc5() {
+    return cudaFuncSetAttribute(linear_tc5_kernel<BN, AR>, cudaFuncAttributeMaxDynamicSharedMemorySize, LtSmem<BN, AR>::ALLOC);
+}
+
+template <int BN, int AR>
+bool launch_tc5(const LinArgs &a, int sm_count, cudaStream_t st) {
+    CUtensorMap tm_x, tm_w;
+    if (!make_map_2d(&tm_x, CU_TENSOR_MAP_DATA_TYPE_BFLOAT16, 2, a.x, a.x_pitch, a.T, (uint64_t)a.x_pitch * 2, 64, AR, CU_TENSOR_MAP_SWIZZLE_128B)) return false;
+    if (!make_map_2d(&tm_w, CU_TENSOR_MAP_DATA_TYPE_BFLOAT16, 2, a.w, a.kp, (uint64_t)a.n_batch * a.n_rows, (uint64_t)a.kp * 2, 64, BN, CU_TENSOR_MAP_SWIZZLE_128B)) return false;
+    LtTiles g{(a.n_rows + BN - 1) / BN, (a.T + LT_M - 1) / LT_M, 0};
+    g.total = g.rows * g.toks * a.n_batch;
+    const uint32_t ctas = BN == 256 ? std::min(g.total, (uint32_t)sm_count) : g.total;
+    launch_pdl(linear_tc5_kernel<BN, AR>, ctas, LT_THREADS, LtSmem<BN, AR>::ALLOC, st, tm_x, tm_w, a, g);
+    g_tc5_launched.store(true, std::memory_order_relaxed);
+    return true;
 }
 
 template <int BN>
-bool launch_tc5(const LinArgs &a, cudaStream_t st) {
-    CUtensorMap tm_x, tm_w;
-    if (!make_map_2d(&tm_x, CU_TENSOR_MAP_DATA_TYPE_BFLOAT16, 2, a.x, a.x_pitch, a.T, (uint64_t)a.x_pitch * 2, 64, LT_M, CU_TENSOR_MAP_SWIZZLE_128B)) return false;
-    if (!make_map_2d(&tm_w, CU_TENSOR_MAP_DATA_TYPE_BFLOAT16, 2, a.w, a.kp, (uint64_t)a.n_batch * a.n_rows, (uint64_t)a.kp * 2, 64, BN, CU_TENSOR_MAP_SWIZZLE_128B)) return false;
-    launch_pdl(linear_tc5_kernel<BN>, dim3((a.n_rows + BN - 1) / BN, (a.T + LT_M - 1) / LT_M, a.n_batch), LT_THREADS, LtSmem<BN>::ALLOC, st, tm_x, tm_w, a);
-    g_tc5_launched.store(true, std::memory_order_relaxed);
-    return true;
+bool launch_tc5_rows(const LinArgs &a, int sm_count, cudaStream_t st) {
+    if (a.T <= 16) return launch_tc5<BN, 16>(a, sm_count, st);
+    if (a.T <= 64) return launch_tc5<BN, 64>(a, sm_count, st);
+    return launch_tc5<BN, 128>(a, sm_count, st);
 }
 
 template <typename TA>
@@ -392,7 +449,7 @@ void launch_gemv_act(const LinArgs &a, int sm_count, cudaStream_t st) {
     uint32_t KS = 1;
     const uint32_t pairs = a.n_rows / 2 * a.n_batch;
     if (G == 32)
-        while (KS < 8 && pairs * KS * 2 <= (uint32_t)sm_count * 16 && a.kp / 8 >= 32 * KS * 2) KS *= 2;
+        while (KS < 8 && pairs * KS * 2 <= (uint32_t)sm_count * 32 && a.kp / 8 >= 32 * KS * 2) KS *= 2;
     const uint32_t units = KS > 1 ? 8 / KS : 8 * (32 / G);
     const dim3 grid((a.n_rows / 2 + units - 1) / units, 1, a.n_batch);
     switch (a.T) {
@@ -409,10 +466,10 @@ constexpr uint32_t GV_MAX_TOKENS = 4;
 cudaError_t linear_configure() {
     static PerDeviceOnce once;
     return once.run([] {
-        cudaError_t e = cudaFuncSetAttribute(linear_tc5_kernel<32>, cudaFuncAttributeMaxDynamicSharedMemorySize, LtSmem<32>::ALLOC);
-        if (e == cudaSuccess) e = cudaFuncSetAttribute(linear_tc5_kernel<64>, cudaFuncAttributeMaxDynamicSharedMemorySize, LtSmem<64>::ALLOC);
-        if (e == cudaSuccess) e = cudaFuncSetAttribute(linear_tc5_kernel<128>, cudaFuncAttributeMaxDynamicSharedMemorySize, LtSmem<128>::ALLOC);
-        if (e == cudaSuccess) e = cudaFuncSetAttribute(linear_tc5_kernel<256>, cudaFuncAttributeMaxDynamicSharedMemorySize, LtSmem<256>::ALLOC);
+        cudaError_t e = configure_tc5<256, 128>();
+        for (cudaError_t (*f)() : {configure_tc5<128, 128>, configure_tc5<128, 64>, configure_tc5<128, 16>, configure_tc5<64, 128>, configure_tc5<64, 64>, configure_tc5<64, 16>,
+                                   configure_tc5<32, 128>, configure_tc5<32, 64>, configure_tc5<32, 16>})
+            if (e == cudaSuccess) e = f();
         return e;
     });
 }
@@ -432,10 +489,10 @@ bool launch_linear(const LinArgs &a, bool f32, int sm_count, cudaStream_t st) {
     const uint32_t tok_tiles = (a.T + LT_M - 1) / LT_M * a.n_batch;
     auto ctas = [&](uint32_t bn) { return (a.n_rows + bn - 1) / bn * tok_tiles; };
     const uint32_t sms = (uint32_t)sm_count;
-    if (ctas(256) >= 2 * sms) return launch_tc5<256>(a, st);
-    if (ctas(128) >= sms) return launch_tc5<128>(a, st);
-    if (ctas(64) >= sms) return launch_tc5<64>(a, st);
-    return launch_tc5<32>(a, st);
+    if (a.T > 64 && ctas(256) >= sms) return launch_tc5<256, 128>(a, sm_count, st);
+    if (ctas(128) >= sms) return launch_tc5_rows<128>(a, sm_count, st);
+    if (ctas(64) >= sms) return launch_tc5_rows<64>(a, sm_count, st);
+    return launch_tc5_rows<32>(a, sm_count, st);
 }
 
 int linear_take_status() { return tc5_take_status(); }

@@ -42,46 +42,134 @@ __device__ __forceinline__ float inv_rms(float sum_sq, uint32_t n, float eps) { 
 
 // (No __restrict__ on what an earlier kernel writes: a load the compiler may take for invariant could move above pdl_wait.)
 // ---- embedding, norms ------------------------------------------------------------------------------------------------------
-__global__ void __launch_bounds__(256) embed_bf16_kernel(const bf16 *table, uint32_t width, const uint32_t *tokens, float *x) {
+// A row of activations from four fp32 values per thread and step.
+template <typename TA> __device__ __forceinline__ void store4(TA *p, float4 v);
+template <> __device__ __forceinline__ void store4<float>(float *p, float4 v) { *reinterpret_cast<float4 *>(p) = v; }
+template <> __device__ __forceinline__ void store4<bf16>(bf16 *p, float4 v) {
+    const __nv_bfloat162 lo = __floats2bfloat162_rn(v.x, v.y), hi = __floats2bfloat162_rn(v.z, v.w);
+    *reinterpret_cast<uint2 *>(p) = make_uint2(*reinterpret_cast<const uint32_t *>(&lo), *reinterpret_cast<const uint32_t *>(&hi));
+}
+__device__ __forceinline__ float sq4(float4 v) { return v.x * v.x + v.y * v.y + v.z * v.z + v.w * v.w; }
+__device__ __forceinline__ float4 mul4(float4 v, float f) { return make_float4(v.x * f, v.y * f, v.z * f, v.w * f); }
+
+// A row in registers: element group i of a thread is columns 4 (threadIdx + i blockDim) .. + 3; NV = 0: any width, one column
+// at a time through memory.
+constexpr int ROW_VECS = 4;
+
+// x = the token's embedding, h = x / rms(x) * gain.
+template <typename TA, int NV>
+__global__ void __launch_bounds__(1024) embed_norm_kernel(const bf16 *table, uint32_t width, const uint32_t *tokens, float *x, float eps, float gain, TA *h, uint32_t h_pitch) {
+    __shared__ float red[33];
     pdl_release();
     pdl_wait();
     const bf16 *row = table + (uint64_t)tokens[blockIdx.x] * width;
-    for (uint32_t i = threadIdx.x; i < width; i += blockDim.x) x[(uint64_t)blockIdx.x * width + i] = __bfloat162float(row[i]);
+    float *xr = x + (uint64_t)blockIdx.x * width;
+    TA *hr = h + (uint64_t)blockIdx.x * h_pitch;
+    float s = 0.0f;
+    if constexpr (NV > 0) {
+        float4 v[NV];
+#pragma unroll
+        for (int i = 0; i < NV; ++i) {
+            const uint32_t c = 4 * (threadIdx.x + i * blockDim.x);
+            if (c >= width) continue;
+            const uint2 u = *reinterpret_cast<const uint2 *>(row + c);
+            v[i] = make_float4(__uint_as_float(u.x << 16), __uint_as_float(u.x & 0xffff0000u), __uint_as_float(u.y << 16), __uint_as_float(u.y & 0xffff0000u));
+            *reinterpret_cast<float4 *>(xr + c) = v[i];
+            s += sq4(v[i]);
+        }
+        const float f = inv_rms(block_sum(s, red), width, eps) * gain;
+#pragma unroll
+        for (int i = 0; i < NV; ++i) {
+            const uint32_t c = 4 * (threadIdx.x + i * blockDim.x);
+            if (c < width) store4<TA>(hr + c, mul4(v[i], f));
+        }
+    } else {
+        for (uint32_t i = threadIdx.x; i < width; i += blockDim.x) {
+            const float v = __bfloat162float(row[i]);
+            xr[i] = v;
+            s += v * v;
+        }
+        const float f = inv_rms(block_sum(s, red), width, eps) * gain;
+        for (uint32_t i = threadIdx.x; i < width; i += blockDim.x) hr[i] = to_act<TA>(xr[i] * f);
+    }
 }
 
-template <typename TA>
-__global__ void __launch_bounds__(256) norm_scalar_kernel(const float *x, uint32_t width, const uint32_t *rows, float eps, float gain, TA *h, uint32_t h_pitch) {
+template <typename TA, int NV>
+__global__ void __launch_bounds__(1024) norm_scalar_kernel(const float *x, uint32_t width, const uint32_t *rows, float eps, float gain, TA *h, uint32_t h_pitch) {
     __shared__ float red[33];
     pdl_release();
     pdl_wait();
     const float *row = x + (uint64_t)(rows ? rows[blockIdx.x] : blockIdx.x) * width;
+    TA *hr = h + (uint64_t)blockIdx.x * h_pitch;
     float s = 0.0f;
-    for (uint32_t i = threadIdx.x; i < width; i += blockDim.x) s += row[i] * row[i];
-    const float f = inv_rms(block_sum(s, red), width, eps) * gain;
-    for (uint32_t i = threadIdx.x; i < width; i += blockDim.x) h[(uint64_t)blockIdx.x * h_pitch + i] = to_act<TA>(row[i] * f);
+    if constexpr (NV > 0) {
+        float4 v[NV];
+#pragma unroll
+        for (int i = 0; i < NV; ++i) {
+            const uint32_t c = 4 * (threadIdx.x + i * blockDim.x);
+            v[i] = c < width ? *reinterpret_cast<const float4 *>(row + c) : make_float4(0, 0, 0, 0);
+            s += sq4(v[i]);
+        }
+        const float f = inv_rms(block_sum(s, red), width, eps) * gain;
+#pragma unroll
+        for (int i = 0; i < NV; ++i) {
+            const uint32_t c = 4 * (threadIdx.x + i * blockDim.x);
+            if (c < width) store4<TA>(hr + c, mul4(v[i], f));
+        }
+    } else {
+        for (uint32_t i = threadIdx.x; i < width; i += blockDim.x) s += row[i] * row[i];
+        const float f = inv_rms(block_sum(s, red), width, eps) * gain;
+        for (uint32_t i = threadIdx.x; i < width; i += blockDim.x) hr[i] = to_act<TA>(row[i] * f);
+    }
 }
 
-template <typename TA>
-__global__ void __launch_bounds__(256) side_finish_kernel(float *x, const float *y, const float *w, uint32_t width, float eps, float gain, TA *h,
-                                                          uint32_t h_pitch) {
-    extern __shared__ float row[];
+template <typename TA, int NV>
+__global__ void __launch_bounds__(1024) side_finish_kernel(float *x, const float *y, const float *w, uint32_t width, float eps, float gain, TA *h, uint32_t h_pitch) {
     __shared__ float red[33];
     pdl_release();
     pdl_wait();
-    const uint64_t o = (uint64_t)blockIdx.x * width;
-    float s = 0.0f;
-    for (uint32_t i = threadIdx.x; i < width; i += blockDim.x) s += y[o + i] * y[o + i];
-    const float f = inv_rms(block_sum(s, red), width, eps);
-    s = 0.0f;
-    for (uint32_t i = threadIdx.x; i < width; i += blockDim.x) {
-        const float v = x[o + i] + y[o + i] * f * w[i];
-        x[o + i] = v;
-        row[i] = v;
-        s += v * v;
+    float *xr = x + (uint64_t)blockIdx.x * width;
+    const float *yr = y + (uint64_t)blockIdx.x * width;
+    TA *hr = h + (uint64_t)blockIdx.x * h_pitch;
+    float s = 0.0f, s2 = 0.0f;
+    if constexpr (NV > 0) {
+        float4 v[NV], yv[NV], wv[NV];
+#pragma unroll
+        for (int i = 0; i < NV; ++i) {
+            const uint32_t c = 4 * (threadIdx.x + i * blockDim.x);
+            const bool in = c < width;
+            yv[i] = in ? *reinterpret_cast<const float4 *>(yr + c) : make_float4(0, 0, 0, 0);
+            v[i] = in ? *reinterpret_cast<const float4 *>(xr + c) : make_float4(0, 0, 0, 0);
+            wv[i] = in ? *reinterpret_cast<const float4 *>(w + c) : make_float4(0, 0, 0, 0);
+            s += sq4(yv[i]);
+        }
+        const float f = inv_rms(block_sum(s, red), width, eps);
+#pragma unroll
+        for (int i = 0; i < NV; ++i) {
+            const uint32_t c = 4 * (threadIdx.x + i * blockDim.x);
+            v[i].x += yv[i].x * f * wv[i].x, v[i].y += yv[i].y * f * wv[i].y, v[i].z += yv[i].z * f * wv[i].z, v[i].w += yv[i].w * f * wv[i].w;
+            if (c < width) *reinterpret_cast<float4 *>(xr + c) = v[i];
+            s2 += sq4(v[i]);
+        }
+        if (!h) return;
+        const float f2 = inv_rms(block_sum(s2, red), width, eps) * gain;
+#pragma unroll
+        for (int i = 0; i < NV; ++i) {
+            const uint32_t c = 4 * (threadIdx.x + i * blockDim.x);
+            if (c < width) store4<TA>(hr + c, mul4(v[i], f2));
+        }
+    } else {
+        for (uint32_t i = threadIdx.x; i < width; i += blockDim.x) s += yr[i] * yr[i];
+        const float f = inv_rms(block_sum(s, red), width, eps);
+        for (uint32_t i = threadIdx.x; i < width; i += blockDim.x) {
+            const float v = xr[i] + yr[i] * f * w[i];
+            xr[i] = v;
+            s2 += v * v;
+        }
+        if (!h) return;
+        const float f2 = inv_rms(block_sum(s2, red), width, eps) * gain;
+        for (uint32_t i = threadIdx.x; i < width; i += blockDim.x) hr[i] = to_act<TA>(xr[i] * f2);
     }
-    if (!h) return;
-    const float f2 = inv_rms(block_sum(s, red), width, eps) * gain;
-    for (uint32_t i = threadIdx.x; i < width; i += blockDim.x) h[(uint64_t)blockIdx.x * h_pitch + i] = to_act<TA>(row[i] * f2);
 }
 
 // ---- rotation ----------------------------------------------------------------------------------------------------------------
@@ -98,6 +186,8 @@ __device__ __forceinline__ float rotated(const float *v, uint32_t d, const Rot &
 }
 
 // ---- latent attention: what a token leaves in the cache, and its rotated query parts -----------------------------------------------
+// Part 0 of a token is its cache row, every further part PREP_Q entries of its rotated query parts.
+constexpr uint32_t PREP_Q = 1024;
 template <typename TA>
 __global__ void __launch_bounds__(256) latent_prep_kernel(LatentArgs a) {
     __shared__ float red[33];
@@ -105,19 +195,26 @@ __global__ void __launch_bounds__(256) latent_prep_kernel(LatentArgs a) {
     pdl_wait();
     const uint32_t t = blockIdx.x, pos = a.positions[t];
     const float *y = a.y + (uint64_t)t * a.y_pitch;
-    const float *lat = y + (uint64_t)a.n_head * a.rot_dim;
     const float2 *cs = a.rot.table + (uint64_t)pos * (a.rot.dims / 2);
+    if (blockIdx.y > 0) {
+        TA *q = static_cast<TA *>(a.q) + (uint64_t)t * a.n_head * a.dq + a.kv_p;
+        const uint32_t first = (blockIdx.y - 1) * PREP_Q, n = a.n_head * a.rot_dim;
+#pragma unroll
+        for (uint32_t u = 0; u < PREP_Q / 256; ++u) {
+            const uint32_t i = first + u * 256 + threadIdx.x;
+            if (i >= n) break;
+            const uint32_t h = i / a.rot_dim, d = i - h * a.rot_dim;
+            q[(uint64_t)h * a.dq + d] = to_act<TA>(rotated(y + (uint64_t)h * a.rot_dim, d, a.rot, cs));
+        }
+        return;
+    }
+    const float *lat = y + (uint64_t)a.n_head * a.rot_dim;
+    TA *row = static_cast<TA *>(a.cache) + ((uint64_t)a.tables[t][pos / KV_PAGE] * KV_PAGE + pos % KV_PAGE) * a.dq;
+    for (uint32_t d = threadIdx.x; d < a.rot_dim; d += blockDim.x) row[a.kv_p + d] = to_act<TA>(rotated(lat + a.kv_rank, d, a.rot, cs));
     float s = 0.0f;
     for (uint32_t i = threadIdx.x; i < a.kv_rank; i += blockDim.x) s += lat[i] * lat[i];
     const float f = inv_rms(block_sum(s, red), a.kv_rank, a.eps);
-    TA *row = static_cast<TA *>(a.cache) + ((uint64_t)a.tables[t][pos / KV_PAGE] * KV_PAGE + pos % KV_PAGE) * a.dq;
     for (uint32_t i = threadIdx.x; i < a.kv_rank; i += blockDim.x) row[i] = to_act<TA>(lat[i] * f * a.kv_norm[i]);
-    for (uint32_t d = threadIdx.x; d < a.rot_dim; d += blockDim.x) row[a.kv_p + d] = to_act<TA>(rotated(lat + a.kv_rank, d, a.rot, cs));
-    TA *q = static_cast<TA *>(a.q) + (uint64_t)t * a.n_head * a.dq + a.kv_p;
-    for (uint32_t i = threadIdx.x; i < a.n_head * a.rot_dim; i += blockDim.x) {
-        const uint32_t h = i / a.rot_dim, d = i - h * a.rot_dim;
-        q[(uint64_t)h * a.dq + d] = to_act<TA>(rotated(y + (uint64_t)h * a.rot_dim, d, a.rot, cs));
-    }
 }
 
 // First position row t of a sequence sees.
@@ -427,19 +524,34 @@ __global__ void __launch_bounds__(LM_THREADS, 1) latent_attn_mma_kernel(LatentAr
 }
 
 // The splits of one (token, head) row put together.
+constexpr uint32_t MERGE_MAX = 256;  // splits
 __global__ void __launch_bounds__(128) latent_merge_kernel(LatentArgs a, uint32_t n_splits) {
+    __shared__ float wt[MERGE_MAX];
+    __shared__ float red[33];
     pdl_release();
     pdl_wait();
     const uint64_t flat = blockIdx.x, stride = (uint64_t)a.T * a.n_head * (a.kv_p + 2);
     const float *p = a.part + flat * (a.kv_p + 2);
-    float m = -INFINITY, l = 0.0f;
-    for (uint32_t s = 0; s < n_splits; ++s) m = fmaxf(m, p[s * stride + a.kv_p]);
-    for (uint32_t s = 0; s < n_splits; ++s) l += exp2f(p[s * stride + a.kv_p] - m) * p[s * stride + a.kv_p + 1];
-    const float inv = 1.0f / l;
-    for (uint32_t i = threadIdx.x; i < a.kv_rank; i += blockDim.x) {
-        float v = 0.0f;
-        for (uint32_t s = 0; s < n_splits; ++s) v += exp2f(p[s * stride + a.kv_p] - m) * p[s * stride + i];
-        static_cast<bf16 *>(a.o)[flat * a.o_head + i] = __float2bfloat16_rn(v * inv);
+    float m = -INFINITY;
+    for (uint32_t s = threadIdx.x & 31; s < n_splits; s += 32) m = fmaxf(m, p[s * stride + a.kv_p]);  // every warp for itself
+    m = warp_max(m);
+    float l = 0.0f;
+    for (uint32_t s = threadIdx.x; s < n_splits; s += blockDim.x) {
+        const float2 ml = *reinterpret_cast<const float2 *>(p + s * stride + a.kv_p);
+        const float e = exp2f(ml.x - m);
+        wt[s] = e;
+        l += e * ml.y;
+    }
+    const float inv = 1.0f / block_sum(l, red);  // synchronises: wt is complete
+    bf16 *o = static_cast<bf16 *>(a.o) + flat * a.o_head;
+    for (uint32_t c = 2 * threadIdx.x; c < a.kv_p; c += 2 * blockDim.x) {
+        float2 v = make_float2(0.0f, 0.0f);
+#pragma unroll 8
+        for (uint32_t s = 0; s < n_splits; ++s) {
+            const float2 u = *reinterpret_cast<const float2 *>(p + s * stride + c);
+            v.x = fmaf(wt[s], u.x, v.x), v.y = fmaf(wt[s], u.y, v.y);
+        }
+        *reinterpret_cast<__nv_bfloat162 *>(o + c) = __floats2bfloat162_rn(v.x * inv, v.y * inv);
     }
 }
 
@@ -528,23 +640,32 @@ __global__ void __launch_bounds__(256) retention_kernel(RetentionArgs a) {
     }
 }
 
-// Every head's output over its root mean square, times silu of its gate.
+// Every head's output over its root mean square, times silu of its gate.  A warp per (token, head).
+constexpr int POST_VALUES = 8;  // per lane in registers; wider heads read the rest twice
 template <typename TA>
 __global__ void __launch_bounds__(256) retention_post_kernel(RetentionArgs a) {
     pdl_release();
     pdl_wait();
-    const uint32_t t = blockIdx.x, warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
-    const float *g = a.y + (uint64_t)t * a.y_pitch + 2ull * a.n_head * a.dim + (uint64_t)a.n_head * a.vdim;
-    for (uint32_t h = warp; h < a.n_head; h += 8) {
-        const float *o = a.o + ((uint64_t)t * a.n_head + h) * a.vdim;
-        float s = 0.0f;
-        for (uint32_t i = lane; i < a.vdim; i += 32) s += o[i] * o[i];
-        const float f = inv_rms(warp_sum(s), a.vdim, a.eps);
-        for (uint32_t i = lane; i < a.vdim; i += 32) {
-            const float z = g[(uint64_t)h * a.vdim + i];
-            static_cast<TA *>(a.out)[(uint64_t)t * a.out_pitch + (uint64_t)h * a.vdim + i] = to_act<TA>(o[i] * f * (z / (1.0f + expf(-z))));
-        }
+    const uint32_t t = blockIdx.x, lane = threadIdx.x & 31, h = blockIdx.y * 8 + (threadIdx.x >> 5);
+    if (h >= a.n_head) return;
+    const float *g = a.y + (uint64_t)t * a.y_pitch + 2ull * a.n_head * a.dim + (uint64_t)(a.n_head + h) * a.vdim;
+    const float *o = a.o + ((uint64_t)t * a.n_head + h) * a.vdim;
+    TA *out = static_cast<TA *>(a.out) + (uint64_t)t * a.out_pitch + (uint64_t)h * a.vdim;
+    float v[POST_VALUES], z[POST_VALUES], s = 0.0f;
+#pragma unroll
+    for (int u = 0; u < POST_VALUES; ++u) {
+        const uint32_t i = lane + 32 * u;
+        v[u] = i < a.vdim ? o[i] : 0.0f;
+        z[u] = i < a.vdim ? g[i] : 0.0f;
+        s += v[u] * v[u];
     }
+    for (uint32_t i = lane + 32 * POST_VALUES; i < a.vdim; i += 32) s += o[i] * o[i];
+    const float f = inv_rms(warp_sum(s), a.vdim, a.eps);
+    auto gated = [&](float x, float zz) { return to_act<TA>(x * f * (zz / (1.0f + expf(-zz)))); };
+#pragma unroll
+    for (int u = 0; u < POST_VALUES; ++u)
+        if (lane + 32 * u < a.vdim) out[lane + 32 * u] = gated(v[u], z[u]);
+    for (uint32_t i = lane + 32 * POST_VALUES; i < a.vdim; i += 32) out[i] = gated(o[i], g[i]);
 }
 
 __global__ void __launch_bounds__(256) copy_pool_pages_kernel(uint4 *pool, uint64_t page_vecs, const int32_t *__restrict__ src, const int32_t *__restrict__ dst) {
@@ -567,27 +688,56 @@ cudaError_t mixers_configure() {
         if (e == cudaSuccess) e = cudaFuncSetAttribute(latent_attn_mma_kernel<4>, cudaFuncAttributeMaxDynamicSharedMemorySize, MAX_SMEM - 64);
         if (e == cudaSuccess) e = cudaFuncSetAttribute(latent_attn_plain_kernel<float>, cudaFuncAttributeMaxDynamicSharedMemorySize, 128 * 1024);
         if (e == cudaSuccess) e = cudaFuncSetAttribute(latent_attn_plain_kernel<bf16>, cudaFuncAttributeMaxDynamicSharedMemorySize, 128 * 1024);
-        if (e == cudaSuccess) e = cudaFuncSetAttribute(side_finish_kernel<float>, cudaFuncAttributeMaxDynamicSharedMemorySize, 128 * 1024);
-        if (e == cudaSuccess) e = cudaFuncSetAttribute(side_finish_kernel<bf16>, cudaFuncAttributeMaxDynamicSharedMemorySize, 128 * 1024);
         return e;
     });
 }
 
-void launch_embed_bf16(const bf16 *table, uint32_t width, const uint32_t *tokens, uint32_t T, float *x, cudaStream_t st) {
-    launch_pdl(embed_bf16_kernel, T, 256, 0, st, table, width, tokens, x);
+// Kernel form and threads for rows of `width`: in registers when the columns come in fours and fit, few rows on wide CTAs.
+struct RowShape {
+    bool vec;
+    uint32_t threads;
+    RowShape(uint32_t width, uint32_t rows, int sm_rows = 296) {
+        const uint32_t want = (width / 4 + 31) / 32 * 32;
+        threads = rows <= (uint32_t)sm_rows ? std::min(1024u, std::max(128u, want)) : std::min(1024u, std::max(128u, (want / ROW_VECS + 31) / 32 * 32));
+        vec = width % 4 == 0 && (uint64_t)threads * 4 * ROW_VECS >= width;
+    }
+};
+template <typename TA>
+static void embed_norm(const bf16 *table, uint32_t width, const uint32_t *tokens, uint32_t T, float *x, float eps, float gain, void *h, uint32_t h_pitch, cudaStream_t st) {
+    const RowShape r(width, T);
+    if (r.vec) launch_pdl(embed_norm_kernel<TA, ROW_VECS>, T, r.threads, 0, st, table, width, tokens, x, eps, gain, static_cast<TA *>(h), h_pitch);
+    else launch_pdl(embed_norm_kernel<TA, 0>, T, r.threads, 0, st, table, width, tokens, x, eps, gain, static_cast<TA *>(h), h_pitch);
+}
+void launch_embed_norm(const bf16 *table, uint32_t width, const uint32_t *tokens, uint32_t T, float *x, float eps, float gain, void *h, uint32_t h_pitch, bool f32,
+                       cudaStream_t st) {
+    if (f32) embed_norm<float>(table, width, tokens, T, x, eps, gain, h, h_pitch, st);
+    else embed_norm<bf16>(table, width, tokens, T, x, eps, gain, h, h_pitch, st);
+}
+template <typename TA>
+static void norm_scalar(const float *x, uint32_t width, const uint32_t *rows, uint32_t n, float eps, float gain, void *h, uint32_t h_pitch, cudaStream_t st) {
+    const RowShape r(width, n);
+    if (r.vec) launch_pdl(norm_scalar_kernel<TA, ROW_VECS>, n, r.threads, 0, st, x, width, rows, eps, gain, static_cast<TA *>(h), h_pitch);
+    else launch_pdl(norm_scalar_kernel<TA, 0>, n, r.threads, 0, st, x, width, rows, eps, gain, static_cast<TA *>(h), h_pitch);
 }
 void launch_norm_scalar(const float *x, uint32_t width, const uint32_t *rows, uint32_t n, float eps, float gain, void *h, uint32_t h_pitch, bool f32, cudaStream_t st) {
-    if (f32) launch_pdl(norm_scalar_kernel<float>, n, 256, 0, st, x, width, rows, eps, gain, static_cast<float *>(h), h_pitch);
-    else launch_pdl(norm_scalar_kernel<bf16>, n, 256, 0, st, x, width, rows, eps, gain, static_cast<bf16 *>(h), h_pitch);
+    if (f32) norm_scalar<float>(x, width, rows, n, eps, gain, h, h_pitch, st);
+    else norm_scalar<bf16>(x, width, rows, n, eps, gain, h, h_pitch, st);
+}
+template <typename TA>
+static void side_finish(float *x, const float *y, const float *w, uint32_t width, uint32_t T, float eps, float gain, void *h, uint32_t h_pitch, cudaStream_t st) {
+    const RowShape r(width, T);
+    if (r.vec) launch_pdl(side_finish_kernel<TA, ROW_VECS>, T, r.threads, 0, st, x, y, w, width, eps, gain, static_cast<TA *>(h), h_pitch);
+    else launch_pdl(side_finish_kernel<TA, 0>, T, r.threads, 0, st, x, y, w, width, eps, gain, static_cast<TA *>(h), h_pitch);
 }
 void launch_side_finish(float *x, const float *y, const float *w, uint32_t width, uint32_t T, float eps, float gain, void *h, uint32_t h_pitch, bool f32, cudaStream_t st) {
-    if (f32) launch_pdl(side_finish_kernel<float>, T, 256, (size_t)width * 4, st, x, y, w, width, eps, gain, static_cast<float *>(h), h_pitch);
-    else launch_pdl(side_finish_kernel<bf16>, T, 256, (size_t)width * 4, st, x, y, w, width, eps, gain, static_cast<bf16 *>(h), h_pitch);
+    if (f32) side_finish<float>(x, y, w, width, T, eps, gain, h, h_pitch, st);
+    else side_finish<bf16>(x, y, w, width, T, eps, gain, h, h_pitch, st);
 }
 
 void launch_latent_prep(const LatentArgs &a, bool f32, cudaStream_t st) {
-    if (f32) launch_pdl(latent_prep_kernel<float>, a.T, 256, 0, st, a);
-    else launch_pdl(latent_prep_kernel<bf16>, a.T, 256, 0, st, a);
+    const dim3 grid(a.T, 1 + (a.n_head * a.rot_dim + PREP_Q - 1) / PREP_Q);
+    if (f32) launch_pdl(latent_prep_kernel<float>, grid, 256, 0, st, a);
+    else launch_pdl(latent_prep_kernel<bf16>, grid, 256, 0, st, a);
 }
 
 uint32_t launch_latent_attention(const LatentArgs &a, bool f32, int sm_count, cudaStream_t st) {
@@ -609,7 +759,7 @@ uint32_t launch_latent_attention(const LatentArgs &a, bool f32, int sm_count, cu
         for (uint32_t s = 0; s < a.n_seq; ++s) tiles += (a.h_spans[s].n * a.n_head + M - 1) / M;
     // few tiles: their keys are split over CTAs and put together afterwards
     const uint32_t span = M / a.n_head + 2, reach = a.window ? std::min<uint64_t>(a.max_pos, (uint64_t)a.window + span) : a.max_pos;
-    uint32_t splits = std::max(1u, std::min((uint32_t)sm_count / std::max(1u, tiles), (reach + KT - 1) / KT));
+    uint32_t splits = std::max(1u, std::min(std::min((uint32_t)sm_count, MERGE_MAX) / std::max(1u, tiles), (reach + KT - 1) / KT));
     while (splits > 1 && (uint64_t)splits * a.T * a.n_head * (a.kv_p + 2) > a.part_cap) --splits;
     const dim3 grid(tiles, splits);
     if (mt == 1) launch_pdl(latent_attn_mma_kernel<1>, grid, LM_THREADS, plan.bytes, st, a);
@@ -629,8 +779,9 @@ uint32_t launch_retention(const RetentionArgs &a, bool f32, int sm_count, cudaSt
     if (a.dim <= 64) launch_pdl(retention_kernel<8>, grid, 256, 0, st, a);
     else if (a.dim <= 128) launch_pdl(retention_kernel<16>, grid, 256, 0, st, a);
     else launch_pdl(retention_kernel<32>, grid, 256, 0, st, a);
-    if (f32) launch_pdl(retention_post_kernel<float>, a.T, 256, 0, st, a);
-    else launch_pdl(retention_post_kernel<bf16>, a.T, 256, 0, st, a);
+    const dim3 post(a.T, (a.n_head + 7) / 8);
+    if (f32) launch_pdl(retention_post_kernel<float>, post, 256, 0, st, a);
+    else launch_pdl(retention_post_kernel<bf16>, post, 256, 0, st, a);
     return 3;
 }
 
