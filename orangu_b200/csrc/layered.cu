@@ -38,7 +38,8 @@ struct LayerPlan {
     uint32_t act_rows = 0, f32_row0 = 0, f32_rows = 0, glu_row0 = 0, mix_cols = 0;  // mix_cols: columns of the mixer in the out product's input
     // latent attention
     Dense uk, uv;        // per head [kv_rank <- dim], [vdim <- kv_rank]
-    uint32_t dim_p = 0, kv_p = 0, dq = 0, kv_w = 0;
+    Dense expand;        // latent -> keys [H][dim_k], then (from row ex_v0) values [H][vdim_k]; no rows: prompts attend in the latent space too
+    uint32_t dim_p = 0, kv_p = 0, dq = 0, kv_w = 0, dim_k = 0, vdim_k = 0, ex_v0 = 0;
     float *kv_norm = nullptr;
     void *pool = nullptr;
     // retention
@@ -65,7 +66,10 @@ struct LayeredGraph : StepGraph {
     Dense output;
     void *h = nullptr, *xb = nullptr, *qn = nullptr, *q = nullptr, *o_lat = nullptr, *cat = nullptr, *sg = nullptr;
     float *y = nullptr, *o_ret = nullptr, *sy = nullptr, *part = nullptr;
+    void *lat = nullptr, *expanded = nullptr;  // gathered latents of prompts, their keys and values: key_cap rows
+    uint32_t key_cap = 0;
     uint64_t part_cap = 0;
+    float *split_part = nullptr;
     bool failed = false;  // a product could not be launched
 
     size_t es() const { return f32 ? 4 : 2; }
@@ -77,8 +81,9 @@ struct LayeredGraph : StepGraph {
     }
 
     void linear(const LinArgs &a, cudaStream_t st) {
-        if (!launch_linear(a, f32, m->ctx->sm_count, st)) failed = true;
-        m->ctx->launches++;
+        const uint32_t n = launch_linear(a, f32, m->ctx->sm_count, st);
+        if (!n) failed = true;
+        m->ctx->launches += n;
     }
     LinArgs product(const Dense &w, const void *x, uint32_t x_pitch, uint32_t T) const {
         LinArgs a{};
@@ -89,6 +94,7 @@ struct LayeredGraph : StepGraph {
         a.x_pitch = x_pitch;
         a.T = T;
         a.n_batch = 1;
+        a.split_part = split_part;
         return a;
     }
     static void segment(LinArgs &a, uint32_t row0, uint32_t n, int epi, void *out, uint32_t pitch, uint32_t col0 = 0, uint32_t batch_cols = 0) {
@@ -161,21 +167,69 @@ void LayeredGraph::latent(const LayerPlan &P, uint32_t T, uint32_t n_seq, const 
     a.tables = reinterpret_cast<const int32_t *const *>(m->d_meta + ml.off_tables);
     a.max_pos = max_pos;
     launch_latent_prep(a, f32, st);
-    LinArgs uk = product(P.uk, qn, H * P.dim_p, T);  // head h: its unrotated query through the key up-projection
-    uk.n_rows = P.uk.rows / H;
-    uk.n_batch = H;
-    uk.x_step = P.dim_p;
-    segment(uk, 0, P.mx.kv_rank, LE_ACT, q, H * P.dq, 0, P.dq);
-    linear(uk, st);
-    m->ctx->launches += 1 + launch_latent_attention(a, f32, m->ctx->sm_count, st);
-    LinArgs uv = product(P.uv, o_lat, H * P.kv_w, T);
-    uv.n_rows = P.uv.rows / H;
-    uv.n_batch = H;
-    uv.x_step = P.kv_w;
-    uv.gate = y + (size_t)H * P.mx.rot_dim + P.mx.kv_rank + P.mx.rot_dim;
-    uv.gate_pitch = y_pitch;
-    segment(uv, 0, P.mx.vdim, LE_GATED, cat, cat_pitch, 0, P.mx.vdim);
-    linear(uv, st);
+    m->ctx->launches++;
+    uint32_t n_short = n_seq;  // spans that attend in the latent space; the longer ones follow them
+    if (P.expand.rows)
+        while (n_short && spans[n_short - 1].n >= PREFILL_SPAN) --n_short;
+    const float *gate = y + (size_t)H * P.mx.rot_dim + P.mx.kv_rank + P.mx.rot_dim;
+    if (n_short) {
+        a.n_seq = n_short;
+        LinArgs uk = product(P.uk, qn, H * P.dim_p, T);  // head h: its unrotated query through the key up-projection
+        uk.n_rows = P.uk.rows / H;
+        uk.n_batch = H;
+        uk.x_step = P.dim_p;
+        segment(uk, 0, P.mx.kv_rank, LE_ACT, q, H * P.dq, 0, P.dq);
+        linear(uk, st);
+        m->ctx->launches += launch_latent_attention(a, f32, m->ctx->sm_count, st);
+        LinArgs uv = product(P.uv, o_lat, H * P.kv_w, T);
+        uv.n_rows = P.uv.rows / H;
+        uv.n_batch = H;
+        uv.x_step = P.kv_w;
+        uv.gate = gate;
+        uv.gate_pitch = y_pitch;
+        segment(uv, 0, P.mx.vdim, LE_GATED, cat, cat_pitch, 0, P.mx.vdim);
+        linear(uv, st);
+    }
+    LatentPrefillArgs p{};
+    p.n_head = H;
+    p.vdim = P.mx.vdim;
+    p.window = P.mx.window;
+    p.dim_k = P.dim_k;
+    p.vdim_k = P.vdim_k;
+    p.kv_p = P.kv_p;
+    p.dq = P.dq;
+    p.dim_p = P.dim_p;
+    p.scale = P.mx.scale;
+    p.tables = a.tables;
+    p.cache = P.pool;
+    p.lat = lat;
+    p.expanded = expanded;
+    p.ex_pitch = P.expand.rows;
+    p.ex_v0 = P.ex_v0;
+    p.qn = qn;
+    p.qn_pitch = P.act_rows;
+    p.q = q;
+    p.gate = gate;
+    p.gate_pitch = y_pitch;
+    p.out = cat;
+    p.out_pitch = cat_pitch;
+    const uint32_t *h_pos = reinterpret_cast<const uint32_t *>(m->h_meta + ml.off_positions);
+    for (uint32_t s = n_short; s < n_seq;) {  // as many spans at a time as the buffers hold
+        p.n_span = p.n_keys = p.n_tiles = 0;
+        for (; s < n_seq && p.n_span < PREFILL_GROUP; ++s) {
+            const uint32_t pos0 = h_pos[spans[s].row0], hist = P.mx.window ? std::min(pos0, P.mx.window - 1) : pos0;
+            if (p.n_span && p.n_keys + hist + spans[s].n > key_cap) break;
+            p.span[p.n_span++] = PrefillSpan{spans[s].row0, spans[s].n, pos0, hist, p.n_keys, p.n_tiles};
+            p.n_keys += hist + spans[s].n;
+            p.n_tiles += latent_prefill_tiles(spans[s].n);
+        }
+        launch_latent_gather(p, st);
+        LinArgs ex = product(P.expand, lat, P.dq, p.n_keys);
+        segment(ex, 0, P.expand.rows, LE_ACT, expanded, P.expand.rows);
+        linear(ex, st);
+        launch_latent_prefill(p, st);
+        m->ctx->launches += 2;
+    }
 }
 
 void LayeredGraph::retention(const LayerPlan &P, uint32_t T, uint32_t n_seq, cudaStream_t st) {
@@ -378,6 +432,17 @@ int LayeredGraph::build_layer(const ob_block_desc &b, LayerPlan &P) {
             for (uint32_t i = 0; i < x.vdim; ++i) uv.copy(hd * vr + i, 0, x.w_uv, hd * x.vdim + i);
         }
         if ((rc = upload(uk, &P.uk)) || (rc = upload(uv, &P.uv))) return rc;
+        P.dim_k = round_up(x.dim, 16);
+        P.vdim_k = round_up(x.vdim, 16);
+        if (!f32 && latent_prefill_supported(P.dim_k, P.dq - P.kv_p, P.vdim_k)) {
+            P.ex_v0 = round_up(H * P.dim_k, LIN_ROW_ALIGN);
+            HostDense ex(P.ex_v0 + round_up(H * P.vdim_k, LIN_ROW_ALIGN), P.kv_w);
+            for (uint32_t hd = 0; hd < H; ++hd) {
+                for (uint32_t d = 0; d < x.dim; ++d) ex.copy(hd * P.dim_k + d, 0, x.w_uk, hd * x.dim + d);
+                for (uint32_t d = 0; d < x.vdim; ++d) ex.copy(P.ex_v0 + hd * P.vdim_k + d, 0, x.w_uv, hd * x.vdim + d);
+            }
+            if ((rc = upload(ex, &P.expand))) return rc;
+        }
         if ((rc = upload_f32(m, x.kv_norm, x.kv_rank, &P.kv_norm))) return rc;
         if ((rc = scratch(&P.pool, (size_t)m->pool_pages * KV_PAGE * P.dq, es()))) return rc;
     } else {
@@ -403,7 +468,7 @@ int LayeredGraph::build(const ob_layered_desc &c) {
     final_gain = c.final_gain;
     L.resize(c.n_layer);
     std::map<std::pair<double, uint32_t>, float2 *> tables;
-    size_t act = 0, q_n = 0, o_n = 0, o_r = 0, kvp = 0, heads = 0;
+    size_t act = 0, q_n = 0, o_n = 0, o_r = 0, kvp = 0, dq = 0, ex = 0, reach = 0;
     for (uint32_t i = 0; i < c.n_layer; ++i) {
         LayerPlan &P = L[i];
         if ((rc = build_layer(c.layers[i], P))) return rc;
@@ -426,7 +491,11 @@ int LayeredGraph::build(const ob_layered_desc &c) {
             q_n = std::max<size_t>(q_n, (size_t)H * P.dq);
             o_n = std::max<size_t>(o_n, (size_t)H * P.kv_w);
             kvp = std::max<size_t>(kvp, P.kv_p);
-            heads = std::max<size_t>(heads, H);
+            if (P.expand.rows) {
+                dq = std::max<size_t>(dq, P.dq);
+                ex = std::max<size_t>(ex, P.expand.rows);
+                reach = std::max<size_t>(reach, std::min(P.mx.window ? P.mx.window - 1 : m->cfg.max_seq_len, m->cfg.max_seq_len));
+            }
         } else {
             o_r = std::max<size_t>(o_r, (size_t)H * P.mx.vdim);
         }
@@ -446,7 +515,12 @@ int LayeredGraph::build(const ob_layered_desc &c) {
     if ((rc = scratch(&h, T * h_pitch, es())) || (rc = scratch(&xb, T * h_pitch, es())) || (rc = scratch(&cat, T * cat_pitch, es()))) return rc;
     if ((rc = scratch(&qn, T * act, es())) || (rc = scratch(&q, T * q_n, es())) || (rc = scratch(&o_lat, T * o_n, es()))) return rc;
     if ((rc = scratch_f32(&y, T * y_pitch)) || (rc = scratch_f32(&o_ret, T * o_r))) return rc;
+    if (ex) {
+        key_cap = (uint32_t)(T + reach);
+        if ((rc = scratch(&lat, (size_t)key_cap * dq, 2)) || (rc = scratch(&expanded, (size_t)key_cap * ex, 2))) return rc;
+    }
     if (side_dim && ((rc = scratch(&sg, T * side_p, es())) || (rc = scratch_f32(&sy, T * width)))) return rc;
+    if (!f32 && (rc = scratch_f32(&split_part, linear_split_bytes() / 4))) return rc;
     if (q_n && !f32) {  // at most one CTA per SM, of 64 rows, writes partial results at a time (launch_latent_attention)
         part_cap = ((uint64_t)m->ctx->sm_count * 64 + 64) * (kvp + 2);
         if ((rc = scratch_f32(&part, part_cap))) return rc;

@@ -46,10 +46,12 @@ struct LinArgs {
     uint32_t emb_pitch = 0, emb_col0 = 0;
     const float *gate = nullptr;
     uint32_t gate_pitch = 0;
+    float *split_part = nullptr;  // scratch of products that split K, linear_split_bytes
 };
 constexpr uint32_t LIN_K_ALIGN = 64, LIN_ROW_ALIGN = 32;
 cudaError_t linear_configure();  // kernel attributes of the current device (outside stream capture)
-bool launch_linear(const LinArgs &a, bool f32, int sm_count, cudaStream_t st);  // false: a tensor map could not be made
+uint32_t launch_linear(const LinArgs &a, bool f32, int sm_count, cudaStream_t st);  // kernels launched; 0: a tensor map could not be made
+size_t linear_split_bytes();
 int linear_take_status();        // 1 when a bounded wait inside a product ran out since the last call
 void linear_mark_launched();     // a replayed graph may have run one of the tensor-core products
 
@@ -96,6 +98,37 @@ struct LatentArgs {          // latent attention of one layer over T rows
 cudaError_t mixers_configure();
 void launch_latent_prep(const LatentArgs &a, bool f32, cudaStream_t st);   // norms and appends the latent, rotates and stores the query parts
 uint32_t launch_latent_attention(const LatentArgs &a, bool f32, int sm_count, cudaStream_t st);  // returns the kernels launched
+
+// Prompts: the window's latents are gathered from the pages, multiplied out to keys and values (a product), and attended per head.
+constexpr uint32_t PREFILL_SPAN = 64;     // spans of at least this many rows go this way (bf16); in a step they follow the shorter ones
+constexpr uint32_t PREFILL_GROUP = 8;     // spans of one launch
+struct PrefillSpan {
+    uint32_t row0, n, pos0, hist;         // rows, first position, positions before it that are seen
+    uint32_t key0, tile0;                 // first gathered key, first tile of the launch
+};
+struct LatentPrefillArgs {
+    PrefillSpan span[PREFILL_GROUP];
+    uint32_t n_span, n_keys, n_tiles;
+    uint32_t n_head, vdim, window;
+    uint32_t dim_k, vdim_k;               // per head in `expanded`, multiples of 16
+    uint32_t kv_p, dq, dim_p;
+    float scale;
+    const int32_t *const *tables;
+    const void *cache;                    // [page][16][dq]
+    void *lat;                            // [n_keys][dq] gathered rows
+    const void *expanded;                 // [n_keys][ex_pitch]: keys [H][dim_k], at ex_v0 values [H][vdim_k]
+    uint32_t ex_pitch, ex_v0;
+    const void *qn, *q;                   // unrotated query parts [T][qn_pitch] (head h at h * dim_p), rotated ones in [T][H][dq] at kv_p
+    uint32_t qn_pitch;
+    const float *gate;                    // [T][gate_pitch]: sigmoid of entry h scales head h
+    uint32_t gate_pitch;
+    void *out;                            // activations [T][out_pitch], head h at h * vdim
+    uint32_t out_pitch;
+};
+bool latent_prefill_supported(uint32_t dim_k, uint32_t rot_p, uint32_t vdim_k);
+uint32_t latent_prefill_tiles(uint32_t n);
+void launch_latent_gather(const LatentPrefillArgs &a, cudaStream_t st);
+void launch_latent_prefill(const LatentPrefillArgs &a, cudaStream_t st);
 
 struct RetentionArgs {       // retention of one layer over T rows
     float *y;                // projections [T][y_pitch]: q [H][dim], k [H][dim], v [H][vdim], gate [H][vdim]; q and k are rotated in place

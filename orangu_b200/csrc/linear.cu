@@ -129,7 +129,7 @@ __device__ __forceinline__ void epilogue_store(const LinArgs &a, uint32_t batch,
 constexpr int GV_THREADS = 256, GV_UNROLL = 4;
 
 template <typename TA, int NT>
-__global__ void __launch_bounds__(GV_THREADS) gemv_act_kernel(LinArgs a, uint32_t G, uint32_t KS) {
+__global__ void __launch_bounds__(GV_THREADS, NT == 1 ? 3 : 2) gemv_act_kernel(LinArgs a, uint32_t G, uint32_t KS) {
     const uint32_t warp = threadIdx.x >> 5, lane = threadIdx.x & 31, per_warp = 32 / G;
     const uint32_t ks = KS > 1 ? warp % KS : 0, unit = KS > 1 ? warp / KS : warp * per_warp + lane / G;
     const uint32_t units = KS > 1 ? 8 / KS : 8 * per_warp;
@@ -258,6 +258,8 @@ __global__ void __launch_bounds__(256) linear_simt_kernel(LinArgs a) {
 // BN = 256 is persistent with two accumulators, so a tile's epilogue runs under the next tile's products; narrower tiles are one
 // per CTA, two CTAs per SM.  AR: token rows that are loaded.  With few tokens the other rows of the operand are whatever the
 // shared memory holds -- they only reach tensor-memory lanes nobody reads -- and the room goes into more stages of weights.
+// An MMA costs its 128 token rows however narrow the tile, so small batches keep wide tiles and fill the GPU by splitting K: the
+// splits of a tile leave fp32 partial sums, which linear_finish_kernel adds up in split order before it runs the epilogue.
 constexpr int LT_M = 128, LT_EPI_WARPS = 4, LT_TMA_WARP = 4, LT_MMA_WARP = 5, LT_THREADS = 6 * 32;
 constexpr uint32_t LT_GROUP = 16;  // token tiles that share the weight tiles of a wave: both operands stay in L2
 
@@ -265,7 +267,8 @@ template <int BN, int AR>
 struct LtSmem {
     static constexpr uint32_t A_BYTES = AR * 128, B_BYTES = BN * 128, SLACK = LT_M * 128 - A_BYTES;  // the MMA reads 128 rows from every stage's base
     static constexpr uint32_t STAGES = BN == 256 ? 4 : (104 * 1024 - SLACK) / (A_BYTES + B_BYTES);
-    static constexpr uint32_t NBUF = BN == 256 ? 2 : 1, COLS = NBUF * BN;
+    static constexpr uint32_t NBUF = BN == 256 ? 2 : 1;
+    static constexpr uint32_t COLS = NBUF * BN;
     static constexpr uint32_t B = 0, A = STAGES * B_BYTES, FULL = A + STAGES * A_BYTES + SLACK, EMPTY = FULL + 8 * STAGES, ACC_FULL = EMPTY + 8 * STAGES,
                               ACC_EMPTY = ACC_FULL + 8 * NBUF, SLOT = ACC_EMPTY + 8 * NBUF, ABORT = SLOT + 8, BYTES = ABORT + 8, ALLOC = BYTES + 1024;
     static_assert(STAGES >= 3 && ALLOC <= (BN == 256 ? 227 : 113) * 1024, "shared memory plan does not fit");
@@ -283,8 +286,11 @@ __device__ __forceinline__ void umma_bf16(uint32_t d_tmem, uint64_t a_desc, uint
 __host__ __device__ constexpr uint32_t umma_idesc_bf16(uint32_t n) { return (1u << 4) | (1u << 7) | (1u << 10) | ((n >> 3) << 17) | ((128u >> 4) << 24); }
 
 struct LtTiles {
-    uint32_t rows, toks, total;  // weight tiles and token tiles of one batch entry, tiles of all
+    uint32_t rows, toks, total;  // weight tiles and token tiles of one batch entry, tiles of all (splits counted)
+    uint32_t splits;             // > 1: one token tile of at most LT_SPLIT_TOKENS rows, a CTA per tile and split
+    float *part;                 // [tile][split][LT_SPLIT_TOKENS][BN]
 };
+constexpr uint32_t LT_SPLIT_TOKENS = 64;
 __device__ __forceinline__ void lt_tile(const LtTiles &g, uint32_t tile, uint32_t *batch, uint32_t *rt, uint32_t *tt) {
     const uint32_t per = g.rows * g.toks;
     *batch = tile / per;
@@ -304,7 +310,7 @@ linear_tc5_kernel(const __grid_constant__ CUtensorMap tm_x, const __grid_constan
     uint8_t *smem = smem_raw + (sbase - smem_u32(smem_raw));
     const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
     volatile uint32_t *abort = reinterpret_cast<volatile uint32_t *>(smem + S::ABORT);
-    const uint32_t n_steps = a.kp / 64;
+    const uint32_t split = blockIdx.x % g.splits, k0 = a.kp / 64 * split / g.splits, k1 = a.kp / 64 * (split + 1) / g.splits, n_steps = k1 - k0;
 
     if (threadIdx.x == 0) {
         for (uint32_t s = 0; s < S::STAGES; ++s) {
@@ -333,17 +339,17 @@ linear_tc5_kernel(const __grid_constant__ CUtensorMap tm_x, const __grid_constan
             bool ok = true;
             for (uint32_t tile = blockIdx.x; ok && tile < g.total; tile += gridDim.x) {
                 uint32_t batch, rt, tt;
-                lt_tile(g, tile, &batch, &rt, &tt);
+                lt_tile(g, tile / g.splits, &batch, &rt, &tt);
                 const int32_t wy = (int32_t)(batch * a.n_rows + rt * BN), xc = (int32_t)(batch * a.x_step), xy = (int32_t)(tt * LT_M);
                 auto weights = [&](uint32_t k, uint32_t s) {
                     mbar_expect_tx(sbase + S::FULL + 8 * s, S::A_BYTES + S::B_BYTES);
                     tma_load_2d(sbase + S::B + s * S::B_BYTES, &tm_w, (int32_t)(k * 64), wy, sbase + S::FULL + 8 * s);
                 };
                 if (tile == blockIdx.x) {
-                    for (uint32_t k = 0; k < ahead; ++k) weights(k, k);
+                    for (uint32_t k = 0; k < ahead; ++k) weights(k0 + k, k);
                     pdl_wait();
                 }
-                for (uint32_t k = 0; k < n_steps; ++k, ++it) {
+                for (uint32_t k = k0; k < k1; ++k, ++it) {
                     const uint32_t s = it % S::STAGES;
                     if (it >= S::STAGES && !mbar_wait(sbase + S::EMPTY + 8 * s, ((it / S::STAGES) & 1u) ^ 1u, abort)) {
                         ok = false;
@@ -363,7 +369,7 @@ linear_tc5_kernel(const __grid_constant__ CUtensorMap tm_x, const __grid_constan
             for (uint32_t tile = blockIdx.x; ok && tile < g.total; tile += gridDim.x, ++n) {
                 const uint32_t buf = n % S::NBUF;
                 if (n >= S::NBUF && !mbar_wait(sbase + S::ACC_EMPTY + 8 * buf, ((n / S::NBUF) & 1u) ^ 1u, abort)) break;
-                for (uint32_t k = 0; k < n_steps; ++k, ++it) {
+                for (uint32_t k = k0; k < k1; ++k, ++it) {
                     const uint32_t s = it % S::STAGES;
                     if (!mbar_wait(sbase + S::FULL + 8 * s, (it / S::STAGES) & 1u, abort)) {
                         ok = false;
@@ -372,7 +378,7 @@ linear_tc5_kernel(const __grid_constant__ CUtensorMap tm_x, const __grid_constan
                     tc_fence_after();
                     const uint64_t da = umma_desc_sw128(sbase + S::A + s * S::A_BYTES), db = umma_desc_sw128(sbase + S::B + s * S::B_BYTES);
 #pragma unroll
-                    for (uint32_t j = 0; j < 4; ++j) umma_bf16(tmem + buf * BN, da + 2 * j, db + 2 * j, idesc, (k | j) ? 1u : 0u);
+                    for (uint32_t j = 0; j < 4; ++j) umma_bf16(tmem + buf * BN, da + 2 * j, db + 2 * j, idesc, (k > k0 || j) ? 1u : 0u);
                     umma_commit(sbase + S::EMPTY + 8 * s);
                 }
                 if (ok) umma_commit(sbase + S::ACC_FULL + 8 * buf);
@@ -384,7 +390,7 @@ linear_tc5_kernel(const __grid_constant__ CUtensorMap tm_x, const __grid_constan
         for (uint32_t tile = blockIdx.x; tile < g.total; tile += gridDim.x, ++n) {
             const uint32_t buf = n % S::NBUF;
             uint32_t batch, rt, tt;
-            lt_tile(g, tile, &batch, &rt, &tt);
+            lt_tile(g, tile / g.splits, &batch, &rt, &tt);
             if (!mbar_wait(sbase + S::ACC_FULL + 8 * buf, (n / S::NBUF) & 1u, abort)) break;
             tc_fence_after();
             const uint32_t t = tt * LT_M + warp * 32 + lane;
@@ -394,12 +400,13 @@ linear_tc5_kernel(const __grid_constant__ CUtensorMap tm_x, const __grid_constan
                 __syncwarp();
                 tmem_ld32(tmem + ((uint32_t)(warp * 32) << 16) + buf * BN + c * 32, u);
                 tmem_ld_wait();
+                float v[32];
+#pragma unroll
+                for (int i = 0; i < 32; ++i) v[i] = __uint_as_float(u[i]);
                 const uint32_t r = rt * BN + c * 32;
                 if (t < a.T && r < a.n_rows) {
-                    float v[32];
-#pragma unroll
-                    for (int i = 0; i < 32; ++i) v[i] = __uint_as_float(u[i]);
-                    epilogue_store<__nv_bfloat16, 32>(a, batch, t, r, v);
+                    if (g.splits == 1) epilogue_store<__nv_bfloat16, 32>(a, batch, t, r, v);
+                    else store_row<32>(g.part + ((uint64_t)tile * LT_SPLIT_TOKENS + t) * BN + c * 32, v, 32);
                 }
             }
             tc_fence_before();
@@ -416,29 +423,41 @@ linear_tc5_kernel(const __grid_constant__ CUtensorMap tm_x, const __grid_constan
     if (warp == LT_MMA_WARP) tmem_dealloc(tmem, S::COLS);
 }
 
+// The splits of every (token, 4 weight rows) added up, then the epilogue.
+template <int BN>
+__global__ void __launch_bounds__(256) linear_finish_kernel(const __grid_constant__ LinArgs a, const LtTiles g) {
+    pdl_release();
+    pdl_wait();
+    const uint32_t per = a.n_rows / 4, i = blockIdx.x * 256 + threadIdx.x;
+    if (i >= per * a.T * a.n_batch) return;
+    const uint32_t r = i % per * 4, t = i / per % a.T, batch = i / per / a.T, tile = batch * g.rows + r / BN;
+    const float *p = g.part + ((uint64_t)tile * g.splits * LT_SPLIT_TOKENS + t) * BN + r % BN;
+    float v[4] = {0.0f, 0.0f, 0.0f, 0.0f};
+#pragma unroll 4
+    for (uint32_t k = 0; k < g.splits; ++k) {
+        const float4 u = *reinterpret_cast<const float4 *>(p + (uint64_t)k * LT_SPLIT_TOKENS * BN);
+        v[0] += u.x, v[1] += u.y, v[2] += u.z, v[3] += u.w;
+    }
+    epilogue_store<__nv_bfloat16, 4>(a, batch, t, r, v);
+}
+
 template <int BN, int AR>
 cudaError_t configure_tc5() {
     return cudaFuncSetAttribute(linear_tc5_kernel<BN, AR>, cudaFuncAttributeMaxDynamicSharedMemorySize, LtSmem<BN, AR>::ALLOC);
 }
 
 template <int BN, int AR>
-bool launch_tc5(const LinArgs &a, int sm_count, cudaStream_t st) {
+bool launch_tc5(const LinArgs &a, int sm_count, cudaStream_t st, uint32_t splits = 1) {
     CUtensorMap tm_x, tm_w;
     if (!make_map_2d(&tm_x, CU_TENSOR_MAP_DATA_TYPE_BFLOAT16, 2, a.x, a.x_pitch, a.T, (uint64_t)a.x_pitch * 2, 64, AR, CU_TENSOR_MAP_SWIZZLE_128B)) return false;
     if (!make_map_2d(&tm_w, CU_TENSOR_MAP_DATA_TYPE_BFLOAT16, 2, a.w, a.kp, (uint64_t)a.n_batch * a.n_rows, (uint64_t)a.kp * 2, 64, BN, CU_TENSOR_MAP_SWIZZLE_128B)) return false;
-    LtTiles g{(a.n_rows + BN - 1) / BN, (a.T + LT_M - 1) / LT_M, 0};
-    g.total = g.rows * g.toks * a.n_batch;
+    LtTiles g{(a.n_rows + BN - 1) / BN, (a.T + LT_M - 1) / LT_M, 0, splits, a.split_part};
+    g.total = g.rows * g.toks * a.n_batch * splits;
     const uint32_t ctas = BN == 256 ? std::min(g.total, (uint32_t)sm_count) : g.total;
     launch_pdl(linear_tc5_kernel<BN, AR>, ctas, LT_THREADS, LtSmem<BN, AR>::ALLOC, st, tm_x, tm_w, a, g);
+    if (splits > 1) launch_pdl(linear_finish_kernel<BN>, (a.n_rows / 4 * a.T * a.n_batch + 255) / 256, 256, 0, st, a, g);
     g_tc5_launched.store(true, std::memory_order_relaxed);
     return true;
-}
-
-template <int BN>
-bool launch_tc5_rows(const LinArgs &a, int sm_count, cudaStream_t st) {
-    if (a.T <= 16) return launch_tc5<BN, 16>(a, sm_count, st);
-    if (a.T <= 64) return launch_tc5<BN, 64>(a, sm_count, st);
-    return launch_tc5<BN, 128>(a, sm_count, st);
 }
 
 template <typename TA>
@@ -449,7 +468,7 @@ void launch_gemv_act(const LinArgs &a, int sm_count, cudaStream_t st) {
     uint32_t KS = 1;
     const uint32_t pairs = a.n_rows / 2 * a.n_batch;
     if (G == 32)
-        while (KS < 8 && pairs * KS * 2 <= (uint32_t)sm_count * 32 && a.kp / 8 >= 32 * KS * 2) KS *= 2;
+        while (KS < 8 && pairs * KS * 2 <= (uint32_t)sm_count * 64 && a.kp / 8 >= 32 * KS * 2) KS *= 2;
     const uint32_t units = KS > 1 ? 8 / KS : 8 * (32 / G);
     const dim3 grid((a.n_rows / 2 + units - 1) / units, 1, a.n_batch);
     switch (a.T) {
@@ -460,6 +479,7 @@ void launch_gemv_act(const LinArgs &a, int sm_count, cudaStream_t st) {
     }
 }
 constexpr uint32_t GV_MAX_TOKENS = 4;
+constexpr uint32_t LT_SPLIT_CTAS = 296;  // of a launch that splits K
 
 }  // namespace
 
@@ -467,33 +487,40 @@ cudaError_t linear_configure() {
     static PerDeviceOnce once;
     return once.run([] {
         cudaError_t e = configure_tc5<256, 128>();
-        for (cudaError_t (*f)() : {configure_tc5<128, 128>, configure_tc5<128, 64>, configure_tc5<128, 16>, configure_tc5<64, 128>, configure_tc5<64, 64>, configure_tc5<64, 16>,
-                                   configure_tc5<32, 128>, configure_tc5<32, 64>, configure_tc5<32, 16>})
+        for (cudaError_t (*f)() : {configure_tc5<128, 128>, configure_tc5<128, 64>, configure_tc5<128, 16>, configure_tc5<64, 128>, configure_tc5<32, 128>})
             if (e == cudaSuccess) e = f();
         return e;
     });
 }
 
-bool launch_linear(const LinArgs &a, bool f32, int sm_count, cudaStream_t st) {
-    if (!a.T || !a.n_rows) return true;
+uint32_t launch_linear(const LinArgs &a, bool f32, int sm_count, cudaStream_t st) {
+    if (!a.T || !a.n_rows) return 1;
     if (a.T <= GV_MAX_TOKENS) {
         if (f32) launch_gemv_act<float>(a, sm_count, st);
         else launch_gemv_act<__nv_bfloat16>(a, sm_count, st);
-        return true;
+        return 1;
     }
     if (f32) {
         launch_pdl(linear_simt_kernel<float>, dim3((a.n_rows + 63) / 64, (a.T + 63) / 64, a.n_batch), 256, 0, st, a);
-        return true;
+        return 1;
     }
     // the widest tile that still gives every SM a CTA
     const uint32_t tok_tiles = (a.T + LT_M - 1) / LT_M * a.n_batch;
     auto ctas = [&](uint32_t bn) { return (a.n_rows + bn - 1) / bn * tok_tiles; };
     const uint32_t sms = (uint32_t)sm_count;
-    if (a.T > 64 && ctas(256) >= sms) return launch_tc5<256, 128>(a, sm_count, st);
-    if (ctas(128) >= sms) return launch_tc5_rows<128>(a, sm_count, st);
-    if (ctas(64) >= sms) return launch_tc5_rows<64>(a, sm_count, st);
-    return launch_tc5_rows<32>(a, sm_count, st);
+    if (a.T <= LT_SPLIT_TOKENS) {
+        const uint32_t tiles = ctas(128), steps = a.kp / 64;
+        const uint32_t splits = std::max(1u, std::min({LT_SPLIT_CTAS / tiles, 2 * sms / tiles, steps / 4}));
+        const bool ok = a.T <= 16 ? launch_tc5<128, 16>(a, sm_count, st, splits) : launch_tc5<128, 64>(a, sm_count, st, splits);
+        return ok ? 1 + (splits > 1) : 0;
+    }
+    if (ctas(256) >= sms) return launch_tc5<256, 128>(a, sm_count, st);
+    if (ctas(128) >= sms) return launch_tc5<128, 128>(a, sm_count, st);
+    if (ctas(64) >= sms) return launch_tc5<64, 128>(a, sm_count, st);
+    return launch_tc5<32, 128>(a, sm_count, st);
 }
+
+size_t linear_split_bytes() { return (size_t)LT_SPLIT_CTAS * LT_SPLIT_TOKENS * 128 * 4; }
 
 int linear_take_status() { return tc5_take_status(); }
 void linear_mark_launched() { g_tc5_launched.store(true, std::memory_order_relaxed); }

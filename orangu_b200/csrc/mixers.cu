@@ -274,19 +274,22 @@ __global__ void __launch_bounds__(LA_THREADS) latent_attn_plain_kernel(LatentArg
 // and heads make one tile -- and walks the union of their windows in tiles of KT keys, two stages of cp.async.  Scores: a warp has
 // 16 rows x 16 keys over the whole row width.  Softmax statistics, scores and weights are fp32; the weights enter the second
 // product as value plus remainder, two bf16 rows each.  Output: a warp has all rows x its share of the latent columns (16 at a
-// time, LM_PAIRS shares of them).  (mma.sync on purpose: with few tokens M is the number of heads, and 512 output columns for
+// time, LM_PAIRS shares of them).  With fewer rows the warps also split the row width of the score product.  (mma.sync on purpose: with few tokens M is the number of heads, and 512 output columns for
 // 128 rows would take all of tensor memory.)
-constexpr int LM_THREADS = 256, LM_PAIRS = 4;
-__host__ __device__ constexpr int lm_keys(int mt) { return mt == 4 ? 32 : 64; }
+constexpr int LM_THREADS = 256, LM_PAIRS = 4, LM_KEYS = 32;
 struct LmPlan {
     uint32_t q, k, stage, s, ph, pl, stat, bytes;  // byte offsets; stage: bytes of one key stage
-    __host__ __device__ LmPlan(int mt, uint32_t dq) {
-        const uint32_t M = 16 * mt, KT = lm_keys(mt), row = (dq + 8) * 2;
+    uint32_t stages;  // two, or one where that lets a second CTA onto the SM (its products then cover this one's loads)
+    __host__ __device__ LmPlan(int mt, uint32_t dq) : LmPlan(mt, dq, 2) {
+        if (mt < 4 && 2 * bytes > 224 * 1024) *this = LmPlan(mt, dq, 1);
+    }
+    __host__ __device__ LmPlan(int mt, uint32_t dq, uint32_t n_stage) : stages(n_stage) {
+        const uint32_t M = 16 * mt, KT = LM_KEYS, row = (dq + 8) * 2, parts = 4 / mt;
         q = 0;
         k = q + M * row;
         stage = KT * row;
-        s = k + 2 * stage;
-        ph = s + M * (KT + 4) * 4;
+        s = k + stages * stage;
+        ph = s + parts * M * (KT + 4) * 4;
         pl = ph + M * (KT + 8) * 2;
         stat = pl + M * (KT + 8) * 2;  // m, l, keep [M] f32, position [M]
         bytes = stat + 4 * M * 4;
@@ -336,8 +339,8 @@ __device__ __forceinline__ void find_tile(const RowSpan *spans, uint32_t n_seq, 
 }
 
 template <int MT>
-__global__ void __launch_bounds__(LM_THREADS, 1) latent_attn_mma_kernel(LatentArgs a) {
-    constexpr int M = 16 * MT, KT = lm_keys(MT), SP = KT + 4, PP = KT + 8;
+__global__ void __launch_bounds__(LM_THREADS, MT == 4 ? 1 : 2) latent_attn_mma_kernel(LatentArgs a) {
+    constexpr int M = 16 * MT, KT = LM_KEYS, SP = KT + 4, PP = KT + 8, PARTS = 4 / MT;  // MT row tiles x 2 key groups x PARTS of the row width = 8 warps
     extern __shared__ __align__(16) uint8_t smem[];
     const LmPlan pl(MT, a.dq);
     float *S = reinterpret_cast<float *>(smem + pl.s), *mx = reinterpret_cast<float *>(smem + pl.stat), *sum = mx + M, *keep = sum + M;
@@ -371,7 +374,7 @@ __global__ void __launch_bounds__(LM_THREADS, 1) latent_attn_mma_kernel(LatentAr
     const uint32_t n_tiles = (hi - lo + KT - 1) / KT;
 
     auto load_keys = [&](uint32_t it) {
-        const uint32_t base = smem_addr(smem + pl.k) + (it & 1u) * pl.stage;
+        const uint32_t base = smem_addr(smem + pl.k) + (pl.stages == 2 ? it & 1u : 0u) * pl.stage;
         for (uint32_t i = threadIdx.x; i < KT * chunks; i += LM_THREADS) {
             const uint32_t r = i / chunks, c = i - r * chunks, j = lo + it * KT + r;
             const bool in = j < hi;
@@ -405,27 +408,34 @@ __global__ void __launch_bounds__(LM_THREADS, 1) latent_attn_mma_kernel(LatentAr
 #pragma unroll
                 for (int e = 0; e < 4; ++e) acc[i][p][n][e] = 0.0f;
 
-    const uint32_t qs = smem_addr(smem + pl.q), mt_s = warp % MT, kg = warp / MT;
+    const uint32_t qs = smem_addr(smem + pl.q), mt_s = warp % MT, kg = warp / MT % 2, wp = warp / (2 * MT);
+    const uint32_t k_steps = a.dq / 16, k_first = k_steps * wp / PARTS, k_end = k_steps * (wp + 1) / PARTS;
     const uint32_t a_off = (lane & 15) * row_bytes + (lane >> 4) * 16, b_off = ((lane & 7) + ((lane >> 4) << 3)) * row_bytes + ((lane >> 3) & 1) * 16;
     const uint32_t v_off = ((lane & 7) + (((lane >> 3) & 1) << 3)) * row_bytes + (lane >> 4) * 16, p_off = (lane & 15) * (PP * 2) + (lane >> 4) * 16;
     for (uint32_t it = 0; it < n_tiles; ++it) {
-        if (it + 1 < n_tiles) load_keys(it + 1);
-        cp_commit();
-        cp_wait<1>();
+        if (pl.stages == 2) {
+            if (it + 1 < n_tiles) load_keys(it + 1);
+            cp_commit();
+            cp_wait<1>();
+        } else {
+            if (it) load_keys(it);
+            cp_commit();
+            cp_wait<0>();
+        }
         __syncthreads();
-        const uint32_t ks = smem_addr(smem + pl.k) + (it & 1u) * pl.stage;
-        if (kg * 16 < KT) {
+        const uint32_t ks = smem_addr(smem + pl.k) + (pl.stages == 2 ? it & 1u : 0u) * pl.stage;
+        {
             float c[2][4] = {};
             const uint32_t qa = qs + mt_s * 16 * row_bytes + a_off, kb = ks + kg * 16 * row_bytes + b_off;
 #pragma unroll 4
-            for (uint32_t k = 0; k < a.dq / 16; ++k) {
+            for (uint32_t k = k_first; k < k_end; ++k) {
                 uint32_t fa[4], fb[4];
                 ldsm4(fa, qa + k * 32);
                 ldsm4(fb, kb + k * 32);
                 mma_bf16(c[0], fa, fb[0], fb[1]);
                 mma_bf16(c[1], fa, fb[2], fb[3]);
             }
-            float *s = S + (mt_s * 16 + lane / 4) * SP + kg * 16 + 2 * (lane & 3);
+            float *s = S + (wp * M + mt_s * 16 + lane / 4) * SP + kg * 16 + 2 * (lane & 3);
 #pragma unroll
             for (int n = 0; n < 2; ++n) {
                 *reinterpret_cast<float2 *>(s + 8 * n) = make_float2(c[n][0], c[n][1]);
@@ -441,7 +451,10 @@ __global__ void __launch_bounds__(LM_THREADS, 1) latent_attn_mma_kernel(LatentAr
             for (int u = 0; u < KT / 32; ++u) {
                 const int j = (int)(lo + it * KT) + u * 32 + (int)lane;
                 const bool see = j <= p && j < (int)hi && (a.window == 0 || p - j < (int)a.window);
-                v[u] = see ? S[r * SP + u * 32 + lane] * scale2 : -INFINITY;
+                float sc = S[r * SP + u * 32 + lane];
+#pragma unroll
+                for (int w = 1; w < PARTS; ++w) sc += S[(w * M + r) * SP + u * 32 + lane];
+                v[u] = see ? sc * scale2 : -INFINITY;
                 best = fmaxf(best, v[u]);
             }
             best = warp_max(best);
@@ -552,6 +565,194 @@ __global__ void __launch_bounds__(128) latent_merge_kernel(LatentArgs a, uint32_
             v.x = fmaf(wt[s], u.x, v.x), v.y = fmaf(wt[s], u.y, v.y);
         }
         *reinterpret_cast<__nv_bfloat162 *>(o + c) = __floats2bfloat162_rn(v.x * inv, v.y * inv);
+    }
+}
+
+// ---- latent attention of prompts: keys and values rebuilt from the latent, bf16 -------------------------------------------------------
+// With many tokens per sequence it is cheaper to multiply the window's latents out once (linear.cu) and attend per head: the score
+// product is dim + rot_dim wide and the output vdim wide, against kv_rank each in the latent space.  A CTA takes one head and 64
+// consecutive tokens of a sequence, a warp 16 of them; keys come in tiles of 64 through two stages of cp.async.  Scores, softmax
+// and the weights' two bf16 parts (value and remainder) stay in registers.
+constexpr int PF_TOKENS = 64, PF_KEYS = 64, PF_THREADS = 128;
+struct PfPlan {
+    uint32_t k, v, k_stage, v_stage, bytes;
+    __host__ __device__ PfPlan(uint32_t dqk, uint32_t vd) {
+        k = PF_TOKENS * (dqk + 8) * 2;
+        k_stage = PF_KEYS * (dqk + 8) * 2;
+        v = k + 2 * k_stage;
+        v_stage = PF_KEYS * (vd + 8) * 2;
+        bytes = v + 2 * v_stage;
+    }
+};
+
+__global__ void __launch_bounds__(256) latent_gather_kernel(LatentPrefillArgs a) {
+    pdl_release();
+    pdl_wait();
+    const uint32_t key = blockIdx.x * 8 + (threadIdx.x >> 5), lane = threadIdx.x & 31;
+    if (key >= a.n_keys) return;
+    uint32_t s = 0;
+    while (s + 1 < a.n_span && key >= a.span[s + 1].key0) ++s;
+    const PrefillSpan sp = a.span[s];
+    const uint32_t p = sp.pos0 - sp.hist + (key - sp.key0);
+    const uint4 *src = reinterpret_cast<const uint4 *>(static_cast<const bf16 *>(a.cache) + ((uint64_t)a.tables[sp.row0][p / KV_PAGE] * KV_PAGE + p % KV_PAGE) * a.dq);
+    uint4 *dst = reinterpret_cast<uint4 *>(static_cast<bf16 *>(a.lat) + (uint64_t)key * a.dq);
+    for (uint32_t i = lane; i < a.dq / 8; i += 32) dst[i] = src[i];
+}
+
+template <int NV>  // columns of a value in sixteens, at most
+__global__ void __launch_bounds__(PF_THREADS, NV <= 8 ? 2 : 1) latent_prefill_kernel(LatentPrefillArgs a) {
+    extern __shared__ __align__(16) uint8_t smem[];
+    const uint32_t rot_p = a.dq - a.kv_p, dqk = a.dim_k + rot_p, qrow = (dqk + 8) * 2, vrow = (a.vdim_k + 8) * 2;
+    const PfPlan pl(dqk, a.vdim_k);
+    const uint32_t warp = threadIdx.x >> 5, lane = threadIdx.x & 31, h = blockIdx.y;
+    pdl_release();
+    pdl_wait();
+    uint32_t s = 0;
+    while (s + 1 < a.n_span && blockIdx.x >= a.span[s + 1].tile0) ++s;
+    const PrefillSpan sp = a.span[s];
+    const uint32_t t0 = (blockIdx.x - sp.tile0) * PF_TOKENS, n_tok = min((uint32_t)PF_TOKENS, sp.n - t0);
+    const uint32_t lo = first_seen(sp.pos0 + t0, a.window), hi = sp.pos0 + t0 + n_tok, kbase = sp.pos0 - sp.hist;
+    const uint32_t n_tiles = (hi - lo + PF_KEYS - 1) / PF_KEYS;
+    const uint32_t qs = smem_addr(smem);
+
+    {   // queries: unrotated and rotated parts side by side
+        const uint32_t cn = a.dim_k / 8, cr = rot_p / 8, ct = cn + cr;
+        for (uint32_t i = threadIdx.x; i < PF_TOKENS * ct; i += PF_THREADS) {
+            const uint32_t r = i / ct, c = i - r * ct;
+            const bool in = r < n_tok;
+            const uint64_t t = sp.row0 + t0 + (in ? r : 0);
+            const bf16 *src = c < cn ? static_cast<const bf16 *>(a.qn) + t * a.qn_pitch + (uint64_t)h * a.dim_p + 8 * c
+                                     : static_cast<const bf16 *>(a.q) + (t * a.n_head + h) * a.dq + a.kv_p + 8 * (c - cn);
+            cp16(qs + r * qrow + c * 16, src, in);
+        }
+    }
+    auto load = [&](uint32_t it) {
+        const uint32_t kb = qs + pl.k + (it & 1u) * pl.k_stage, vb = qs + pl.v + (it & 1u) * pl.v_stage, j0 = lo + it * PF_KEYS;
+        const uint32_t cn = a.dim_k / 8, cr = rot_p / 8, cv = a.vdim_k / 8, ct = cn + cr + cv;
+        for (uint32_t i = threadIdx.x; i < PF_KEYS * ct; i += PF_THREADS) {
+            const uint32_t r = i / ct, c = i - r * ct;
+            const bool in = j0 + r < hi;
+            const uint64_t key = sp.key0 + (in ? j0 + r - kbase : 0);
+            const bf16 *ex = static_cast<const bf16 *>(a.expanded) + key * a.ex_pitch;
+            if (c < cn) cp16(kb + r * qrow + c * 16, ex + (uint64_t)h * a.dim_k + 8 * c, in);
+            else if (c < cn + cr) cp16(kb + r * qrow + c * 16, static_cast<const bf16 *>(a.lat) + key * a.dq + a.kv_p + 8 * (c - cn), in);
+            else cp16(vb + r * vrow + (c - cn - cr) * 16, ex + a.ex_v0 + (uint64_t)h * a.vdim_k + 8 * (c - cn - cr), in);
+        }
+    };
+    load(0);
+    cp_commit();
+    const float scale2 = a.scale * 1.4426950408889634f;
+    const int p0 = (int)(sp.pos0 + t0 + warp * 16 + lane / 4), p1 = p0 + 8;  // positions of this thread's two rows
+    const int w_first = (int)(sp.pos0 + t0 + warp * 16), w_last = w_first + 15, win = a.window ? (int)a.window : 0x7fffffff;
+    float o[NV][2][4], m0 = -INFINITY, m1 = -INFINITY, l0 = 0.0f, l1 = 0.0f;
+#pragma unroll
+    for (int v = 0; v < NV; ++v)
+#pragma unroll
+        for (int n = 0; n < 2; ++n)
+#pragma unroll
+            for (int e = 0; e < 4; ++e) o[v][n][e] = 0.0f;
+    const uint32_t qa = qs + (warp * 16 + (lane & 15)) * qrow + (lane >> 4) * 16;
+    const uint32_t b_off = ((lane & 7) + ((lane >> 4) << 3)) * qrow + ((lane >> 3) & 1) * 16, v_off = ((lane & 7) + (((lane >> 3) & 1) << 3)) * vrow + (lane >> 4) * 16;
+    const uint32_t nv = a.vdim_k / 16;
+    for (uint32_t it = 0; it < n_tiles; ++it) {
+        if (it + 1 < n_tiles) load(it + 1);
+        cp_commit();
+        cp_wait<1>();
+        __syncthreads();
+        const int j0 = (int)(lo + it * PF_KEYS);
+        const bool any = j0 <= w_last && (long long)j0 + PF_KEYS - 1 > (long long)w_first - win;  // does one of the warp's tokens see one of these keys?
+        if (any) {
+            const uint32_t kb = qs + pl.k + (it & 1u) * pl.k_stage, vb = qs + pl.v + (it & 1u) * pl.v_stage;
+            float c[PF_KEYS / 8][4];
+#pragma unroll
+            for (int n = 0; n < PF_KEYS / 8; ++n) c[n][0] = c[n][1] = c[n][2] = c[n][3] = 0.0f;
+#pragma unroll 2
+            for (uint32_t k = 0; k < dqk / 16; ++k) {
+                uint32_t fa[4];
+                ldsm4(fa, qa + k * 32);
+#pragma unroll
+                for (int g = 0; g < PF_KEYS / 16; ++g) {
+                    uint32_t fb[4];
+                    ldsm4(fb, kb + g * 16 * qrow + b_off + k * 32);
+                    mma_bf16(c[2 * g], fa, fb[0], fb[1]);
+                    mma_bf16(c[2 * g + 1], fa, fb[2], fb[3]);
+                }
+            }
+            const bool inside = j0 + PF_KEYS - 1 <= w_first && (long long)w_last - j0 < win && j0 + PF_KEYS <= (int)hi;  // nothing to mask
+            float b0 = -INFINITY, b1 = -INFINITY;
+#pragma unroll
+            for (int n = 0; n < PF_KEYS / 8; ++n)
+#pragma unroll
+                for (int e = 0; e < 2; ++e) {
+                    const int j = j0 + 8 * n + 2 * (int)(lane & 3) + e;
+                    c[n][e] = inside || (j <= p0 && p0 - j < win) ? c[n][e] * scale2 : -INFINITY;
+                    c[n][2 + e] = inside || (j <= p1 && p1 - j < win) ? c[n][2 + e] * scale2 : -INFINITY;
+                    b0 = fmaxf(b0, c[n][e]);
+                    b1 = fmaxf(b1, c[n][2 + e]);
+                }
+            b0 = fmaxf(b0, __shfl_xor_sync(0xffffffffu, b0, 1)), b0 = fmaxf(b0, __shfl_xor_sync(0xffffffffu, b0, 2));
+            b1 = fmaxf(b1, __shfl_xor_sync(0xffffffffu, b1, 1)), b1 = fmaxf(b1, __shfl_xor_sync(0xffffffffu, b1, 2));
+            const float n0 = fmaxf(m0, b0), n1 = fmaxf(m1, b1);
+            const float s0 = n0 == -INFINITY ? 0.0f : n0, s1 = n1 == -INFINITY ? 0.0f : n1;  // a row that has seen nothing yet keeps weights of zero
+            const float f0 = exp2f(m0 - s0), f1 = exp2f(m1 - s1);
+            m0 = n0, m1 = n1;
+            l0 *= f0, l1 *= f1;
+#pragma unroll
+            for (int v = 0; v < NV; ++v)
+#pragma unroll
+                for (int n = 0; n < 2; ++n) o[v][n][0] *= f0, o[v][n][1] *= f0, o[v][n][2] *= f1, o[v][n][3] *= f1;
+#pragma unroll
+            for (int kk = 0; kk < PF_KEYS / 16; ++kk) {
+                uint32_t ph[4], pr[4];
+#pragma unroll
+                for (int n = 0; n < 2; ++n)
+#pragma unroll
+                    for (int r = 0; r < 2; ++r) {  // fragment register 2n + r: row half r of key half n
+                        const float mr = r ? s1 : s0;
+                        const float e0 = exp2f(c[2 * kk + n][2 * r] - mr), e1 = exp2f(c[2 * kk + n][2 * r + 1] - mr);
+                        if (r) l1 += e0 + e1;
+                        else l0 += e0 + e1;
+                        const __nv_bfloat162 hi2 = __floats2bfloat162_rn(e0, e1);
+                        const __nv_bfloat162 lo2 = __floats2bfloat162_rn(e0 - __low2float(hi2), e1 - __high2float(hi2));
+                        ph[2 * n + r] = *reinterpret_cast<const uint32_t *>(&hi2);
+                        pr[2 * n + r] = *reinterpret_cast<const uint32_t *>(&lo2);
+                    }
+#pragma unroll
+                for (int v = 0; v < NV; ++v) {
+                    if (v >= (int)nv) break;
+                    uint32_t fv[4];
+                    ldsm4t(fv, vb + kk * 16 * vrow + v * 32 + v_off);
+                    mma_bf16(o[v][0], ph, fv[0], fv[1]);
+                    mma_bf16(o[v][1], ph, fv[2], fv[3]);
+                    mma_bf16(o[v][0], pr, fv[0], fv[1]);
+                    mma_bf16(o[v][1], pr, fv[2], fv[3]);
+                }
+            }
+        }
+        __syncthreads();
+    }
+    cp_wait<0>();
+    l0 += __shfl_xor_sync(0xffffffffu, l0, 1), l0 += __shfl_xor_sync(0xffffffffu, l0, 2);
+    l1 += __shfl_xor_sync(0xffffffffu, l1, 1), l1 += __shfl_xor_sync(0xffffffffu, l1, 2);
+#pragma unroll
+    for (int r = 0; r < 2; ++r) {
+        const uint32_t tl = warp * 16 + lane / 4 + 8 * r;
+        if (tl >= n_tok) continue;
+        const uint64_t t = sp.row0 + t0 + tl;
+        const float f = 1.0f / ((r ? l1 : l0) * (1.0f + expf(-a.gate[t * a.gate_pitch + h])));
+        bf16 *out = static_cast<bf16 *>(a.out) + t * a.out_pitch + (uint64_t)h * a.vdim;
+#pragma unroll
+        for (int v = 0; v < NV; ++v)
+#pragma unroll
+            for (int n = 0; n < 2; ++n) {
+                const uint32_t col = v * 16 + n * 8 + 2 * (lane & 3);
+                if (v >= (int)nv || col >= a.vdim) continue;
+                if ((a.vdim & 1) == 0) *reinterpret_cast<__nv_bfloat162 *>(out + col) = __floats2bfloat162_rn(o[v][n][2 * r] * f, o[v][n][2 * r + 1] * f);
+                else {
+                    out[col] = __float2bfloat16_rn(o[v][n][2 * r] * f);
+                    if (col + 1 < a.vdim) out[col + 1] = __float2bfloat16_rn(o[v][n][2 * r + 1] * f);
+                }
+            }
     }
 }
 
@@ -686,6 +887,8 @@ cudaError_t mixers_configure() {
         cudaError_t e = cudaFuncSetAttribute(latent_attn_mma_kernel<1>, cudaFuncAttributeMaxDynamicSharedMemorySize, MAX_SMEM - 64);
         if (e == cudaSuccess) e = cudaFuncSetAttribute(latent_attn_mma_kernel<2>, cudaFuncAttributeMaxDynamicSharedMemorySize, MAX_SMEM - 64);
         if (e == cudaSuccess) e = cudaFuncSetAttribute(latent_attn_mma_kernel<4>, cudaFuncAttributeMaxDynamicSharedMemorySize, MAX_SMEM - 64);
+        for (auto k : {latent_prefill_kernel<4>, latent_prefill_kernel<8>, latent_prefill_kernel<16>})
+            if (e == cudaSuccess) e = cudaFuncSetAttribute(k, cudaFuncAttributeMaxDynamicSharedMemorySize, MAX_SMEM - 64);
         if (e == cudaSuccess) e = cudaFuncSetAttribute(latent_attn_plain_kernel<float>, cudaFuncAttributeMaxDynamicSharedMemorySize, 128 * 1024);
         if (e == cudaSuccess) e = cudaFuncSetAttribute(latent_attn_plain_kernel<bf16>, cudaFuncAttributeMaxDynamicSharedMemorySize, 128 * 1024);
         return e;
@@ -752,14 +955,15 @@ uint32_t launch_latent_attention(const LatentArgs &a, bool f32, int sm_count, cu
         else launch_pdl(latent_attn_plain_kernel<bf16>, a.T * a.n_head, LA_THREADS, plain_smem(a), st, a);
         return 1;
     }
-    const uint32_t M = 16 * mt, KT = lm_keys(mt);
+    const uint32_t M = 16 * mt, KT = LM_KEYS;
     uint32_t tiles = 0;
     if (a.single) tiles = a.n_seq * ((a.n_head + M - 1) / M);
     else
         for (uint32_t s = 0; s < a.n_seq; ++s) tiles += (a.h_spans[s].n * a.n_head + M - 1) / M;
     // few tiles: their keys are split over CTAs and put together afterwards
     const uint32_t span = M / a.n_head + 2, reach = a.window ? std::min<uint64_t>(a.max_pos, (uint64_t)a.window + span) : a.max_pos;
-    uint32_t splits = std::max(1u, std::min(std::min((uint32_t)sm_count, MERGE_MAX) / std::max(1u, tiles), (reach + KT - 1) / KT));
+    const uint32_t slots = (uint32_t)sm_count * (mt == 4 || 2 * plan.bytes > 224 * 1024 ? 1 : 2);
+    uint32_t splits = std::max(1u, std::min(std::min(slots, MERGE_MAX) / std::max(1u, tiles), (reach + KT - 1) / KT));
     while (splits > 1 && (uint64_t)splits * a.T * a.n_head * (a.kv_p + 2) > a.part_cap) --splits;
     const dim3 grid(tiles, splits);
     if (mt == 1) launch_pdl(latent_attn_mma_kernel<1>, grid, LM_THREADS, plan.bytes, st, a);
@@ -768,6 +972,19 @@ uint32_t launch_latent_attention(const LatentArgs &a, bool f32, int sm_count, cu
     if (splits == 1) return 1;
     launch_pdl(latent_merge_kernel, a.T * a.n_head, 128, 0, st, a, splits);
     return 2;
+}
+
+bool latent_prefill_supported(uint32_t dim_k, uint32_t rot_p, uint32_t vdim_k) {
+    return vdim_k <= 256 && PfPlan(dim_k + rot_p, vdim_k).bytes <= MAX_SMEM - 64;
+}
+uint32_t latent_prefill_tiles(uint32_t n) { return (n + PF_TOKENS - 1) / PF_TOKENS; }
+void launch_latent_gather(const LatentPrefillArgs &a, cudaStream_t st) { launch_pdl(latent_gather_kernel, (a.n_keys + 7) / 8, 256, 0, st, a); }
+void launch_latent_prefill(const LatentPrefillArgs &a, cudaStream_t st) {
+    const PfPlan pl(a.dim_k + a.dq - a.kv_p, a.vdim_k);
+    const dim3 grid(a.n_tiles, a.n_head);
+    if (a.vdim_k <= 64) launch_pdl(latent_prefill_kernel<4>, grid, PF_THREADS, pl.bytes, st, a);
+    else if (a.vdim_k <= 128) launch_pdl(latent_prefill_kernel<8>, grid, PF_THREADS, pl.bytes, st, a);
+    else launch_pdl(latent_prefill_kernel<16>, grid, PF_THREADS, pl.bytes, st, a);
 }
 
 bool retention_supported(uint32_t dim) { return dim >= 1 && dim <= 256; }

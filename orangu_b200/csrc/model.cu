@@ -1273,6 +1273,8 @@ int forward_spans(ob_model *m, ob_kv *const *kvs, const uint32_t *tokens, const 
                 in_seq = 0;
             }
         }
+        // a step's spans are in no particular order for the graph but this: prompts after decoded tokens and short portions
+        std::stable_partition(r.spans.begin(), r.spans.end(), [](const RowSpan &sp) { return sp.n < PREFILL_SPAN; });
         const uint32_t w0 = done_want;
         while (done_want < want.size() && want[done_want] < flat) r.logit_rows.push_back(want[done_want++] - flat0);
         r.tokens = tokens + flat0;
@@ -1614,6 +1616,7 @@ int ob_decode_loop(ob_model *m, ob_kv *const *kvs, const uint32_t *first_tokens,
     fetch_status(m, st);
     OB_CUDA(ctx, cudaStreamSynchronize(st));
     OB_CUDA(ctx, cudaGetLastError());
+    if (m->graph) linear_mark_launched();  // the replayed steps may hold tensor-core products
     cudaEventElapsedTime(&ctx->last_ms, ctx->ev0, ctx->ev1);
     ctx->launches += m->graph_launches[key] * n_steps;
     for (uint32_t s = 0; s < n_seq; ++s) kvs[s]->len += n_steps;
