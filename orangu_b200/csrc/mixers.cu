@@ -780,12 +780,22 @@ __global__ void __launch_bounds__(256) retention_prep_kernel(RetentionArgs a) {
 }
 
 // One CTA carries 32 columns of one head's state through the rows of one sequence, token by token: lane = column, warp = DW of
-// the state's rows, kept in registers.  S = decay S + k v^T, o = S^T q; the warps' parts of o are added up once per block of tokens.
+// the state's rows, kept in registers.  S = decay S + k v^T, o = S^T q; the warps' parts of o are added up once per block of tokens,
+// while the next block's q, k and v are on their way to shared memory.
+template <int DW>
+struct RtPlan {
+    static constexpr int D = 8 * DW, BLOCK = DW > 16 ? 8 : 16;
+    static constexpr uint32_t Q = 0, K = Q + BLOCK * D, V = K + BLOCK * D, STAGE = V + BLOCK * 32, PART = 2 * STAGE, FLOATS = PART + 8 * BLOCK * 32;
+};
+__device__ __forceinline__ void cp4(float *dst, const float *src, bool in) {
+    asm volatile("cp.async.ca.shared.global [%0], [%1], 4, %2;" ::"r"(smem_addr(dst)), "l"(src), "r"(in ? 4 : 0) : "memory");
+}
 template <int DW>
 __global__ void __launch_bounds__(256) retention_kernel(RetentionArgs a) {
-    constexpr int D = 8 * DW, RT_BLOCK = DW > 16 ? 8 : 16;
-    __shared__ __align__(16) float qs[RT_BLOCK][D], ks[RT_BLOCK][D];
-    __shared__ float vs[RT_BLOCK][32], part[8][RT_BLOCK][32];
+    using R = RtPlan<DW>;
+    constexpr int D = R::D, BLOCK = R::BLOCK;
+    extern __shared__ __align__(16) float sm[];
+    float *part = sm + R::PART;  // [8][BLOCK][32]
     pdl_release();
     pdl_wait();
     const uint32_t warp = threadIdx.x >> 5, lane = threadIdx.x & 31, h = blockIdx.y, col = blockIdx.x * 32 + lane;
@@ -793,6 +803,22 @@ __global__ void __launch_bounds__(256) retention_kernel(RetentionArgs a) {
     const bool live = col < a.vdim;
     const float decay = a.decay[h];
     float *state = a.state + (((uint64_t)a.slots[sp.row0] * a.n_head + h) * a.dim) * a.vdim + col;
+    const float *yq = a.y + (uint64_t)sp.row0 * a.y_pitch + (uint64_t)h * a.dim, *yk = yq + (uint64_t)a.n_head * a.dim;
+    const float *yv = a.y + (uint64_t)sp.row0 * a.y_pitch + 2ull * a.n_head * a.dim + (uint64_t)h * a.vdim + col;
+    auto load = [&](uint32_t t0, uint32_t stage) {
+        float *s = sm + stage * R::STAGE;
+        const uint32_t n = min((uint32_t)BLOCK, sp.n - t0);
+        for (uint32_t i = threadIdx.x; i < n * D; i += 256) {
+            const uint32_t t = i / D, d = i % D;
+            const bool in = d < a.dim;
+            const uint64_t o = (uint64_t)(t0 + t) * a.y_pitch + (in ? d : 0);
+            cp4(s + R::Q + i, yq + o, in);
+            cp4(s + R::K + i, yk + o, in);
+        }
+        for (uint32_t t = warp; t < n; t += 8) cp4(s + R::V + t * 32 + lane, live ? yv + (uint64_t)(t0 + t) * a.y_pitch : a.y, live);
+    };
+    load(0, 0);
+    cp_commit();
     float S[DW];
     const bool fresh = a.positions[sp.row0] == 0;
 #pragma unroll
@@ -800,40 +826,42 @@ __global__ void __launch_bounds__(256) retention_kernel(RetentionArgs a) {
         const uint32_t d = warp * DW + i;
         S[i] = !fresh && live && d < a.dim ? state[(uint64_t)d * a.vdim] : 0.0f;
     }
-    for (uint32_t t0 = 0; t0 < sp.n; t0 += RT_BLOCK) {
-        const uint32_t n = min((uint32_t)RT_BLOCK, sp.n - t0);
-        for (uint32_t i = threadIdx.x; i < n * D; i += 256) {
-            const uint32_t t = i / D, d = i - t * D;
-            const float *y = a.y + (uint64_t)(sp.row0 + t0 + t) * a.y_pitch + (uint64_t)h * a.dim + d;
-            qs[t][d] = d < a.dim ? y[0] : 0.0f;
-            ks[t][d] = d < a.dim ? y[(uint64_t)a.n_head * a.dim] : 0.0f;
-        }
-        for (uint32_t i = threadIdx.x; i < n * 32; i += 256) {
-            const uint32_t t = i / 32;  // i % 32 == lane
-            vs[t][lane] = live ? a.y[(uint64_t)(sp.row0 + t0 + t) * a.y_pitch + 2ull * a.n_head * a.dim + (uint64_t)h * a.vdim + col] : 0.0f;
-        }
-        __syncthreads();
-        for (uint32_t t = 0; t < n; ++t) {
-            const float v = vs[t][lane];
+    uint32_t stage = 0;
+    for (uint32_t t0 = 0; t0 < sp.n; t0 += BLOCK, stage ^= 1u) {
+        const uint32_t n = min((uint32_t)BLOCK, sp.n - t0);
+        if (t0 + BLOCK < sp.n) load(t0 + BLOCK, stage ^ 1u);
+        cp_commit();
+        cp_wait<1>();
+        __syncthreads();  // this block's operands are there, and everyone is done with the sums of the last one
+        const float *q = sm + stage * R::STAGE + R::Q + warp * DW, *k = sm + stage * R::STAGE + R::K + warp * DW, *v = sm + stage * R::STAGE + R::V + lane;
+        auto token = [&](uint32_t t) {
+            const float vv = v[t * 32];
             float o[4] = {0.0f, 0.0f, 0.0f, 0.0f};
 #pragma unroll
             for (int i = 0; i < DW; i += 4) {
-                const float4 k = *reinterpret_cast<const float4 *>(&ks[t][warp * DW + i]), q = *reinterpret_cast<const float4 *>(&qs[t][warp * DW + i]);
-                S[i] = fmaf(k.x, v, decay * S[i]), o[0] = fmaf(q.x, S[i], o[0]);
-                S[i + 1] = fmaf(k.y, v, decay * S[i + 1]), o[1] = fmaf(q.y, S[i + 1], o[1]);
-                S[i + 2] = fmaf(k.z, v, decay * S[i + 2]), o[2] = fmaf(q.z, S[i + 2], o[2]);
-                S[i + 3] = fmaf(k.w, v, decay * S[i + 3]), o[3] = fmaf(q.w, S[i + 3], o[3]);
+                const float4 kk = *reinterpret_cast<const float4 *>(k + t * D + i), qq = *reinterpret_cast<const float4 *>(q + t * D + i);
+                S[i] = fmaf(kk.x, vv, decay * S[i]), o[0] = fmaf(qq.x, S[i], o[0]);
+                S[i + 1] = fmaf(kk.y, vv, decay * S[i + 1]), o[1] = fmaf(qq.y, S[i + 1], o[1]);
+                S[i + 2] = fmaf(kk.z, vv, decay * S[i + 2]), o[2] = fmaf(qq.z, S[i + 2], o[2]);
+                S[i + 3] = fmaf(kk.w, vv, decay * S[i + 3]), o[3] = fmaf(qq.w, S[i + 3], o[3]);
             }
-            part[warp][t][lane] = (o[0] + o[1]) + (o[2] + o[3]);
+            part[(warp * BLOCK + t) * 32 + lane] = (o[0] + o[1]) + (o[2] + o[3]);
+        };
+        if (n == BLOCK) {
+#pragma unroll 4
+            for (uint32_t t = 0; t < BLOCK; ++t) token(t);
+        } else {
+            for (uint32_t t = 0; t < n; ++t) token(t);
         }
         __syncthreads();
         for (uint32_t t = warp; t < n; t += 8) {
             float o = 0.0f;
 #pragma unroll
-            for (int w = 0; w < 8; ++w) o += part[w][t][lane];
-            if (live) a.o[(uint64_t)(sp.row0 + t0 + t) * a.n_head * a.vdim + (uint64_t)h * a.vdim + col] = o;
+            for (int w = 0; w < 8; ++w) o += part[(w * BLOCK + t) * 32 + lane];
+            if (live) a.o[((uint64_t)(sp.row0 + t0 + t) * a.n_head + h) * a.vdim + col] = o;
         }
     }
+    cp_wait<0>();
 #pragma unroll
     for (int i = 0; i < DW; ++i) {
         const uint32_t d = warp * DW + i;
@@ -889,6 +917,9 @@ cudaError_t mixers_configure() {
         if (e == cudaSuccess) e = cudaFuncSetAttribute(latent_attn_mma_kernel<4>, cudaFuncAttributeMaxDynamicSharedMemorySize, MAX_SMEM - 64);
         for (auto k : {latent_prefill_kernel<4>, latent_prefill_kernel<8>, latent_prefill_kernel<16>})
             if (e == cudaSuccess) e = cudaFuncSetAttribute(k, cudaFuncAttributeMaxDynamicSharedMemorySize, MAX_SMEM - 64);
+        if (e == cudaSuccess) e = cudaFuncSetAttribute(retention_kernel<8>, cudaFuncAttributeMaxDynamicSharedMemorySize, RtPlan<8>::FLOATS * 4);
+        if (e == cudaSuccess) e = cudaFuncSetAttribute(retention_kernel<16>, cudaFuncAttributeMaxDynamicSharedMemorySize, RtPlan<16>::FLOATS * 4);
+        if (e == cudaSuccess) e = cudaFuncSetAttribute(retention_kernel<32>, cudaFuncAttributeMaxDynamicSharedMemorySize, RtPlan<32>::FLOATS * 4);
         if (e == cudaSuccess) e = cudaFuncSetAttribute(latent_attn_plain_kernel<float>, cudaFuncAttributeMaxDynamicSharedMemorySize, 128 * 1024);
         if (e == cudaSuccess) e = cudaFuncSetAttribute(latent_attn_plain_kernel<bf16>, cudaFuncAttributeMaxDynamicSharedMemorySize, 128 * 1024);
         return e;
@@ -993,9 +1024,9 @@ uint32_t launch_retention(const RetentionArgs &a, bool f32, int sm_count, cudaSt
     (void)sm_count;
     launch_pdl(retention_prep_kernel, a.T, 256, 0, st, a);
     const dim3 grid((a.vdim + 31) / 32, a.n_head, a.n_seq);
-    if (a.dim <= 64) launch_pdl(retention_kernel<8>, grid, 256, 0, st, a);
-    else if (a.dim <= 128) launch_pdl(retention_kernel<16>, grid, 256, 0, st, a);
-    else launch_pdl(retention_kernel<32>, grid, 256, 0, st, a);
+    if (a.dim <= 64) launch_pdl(retention_kernel<8>, grid, 256, RtPlan<8>::FLOATS * 4, st, a);
+    else if (a.dim <= 128) launch_pdl(retention_kernel<16>, grid, 256, RtPlan<16>::FLOATS * 4, st, a);
+    else launch_pdl(retention_kernel<32>, grid, 256, RtPlan<32>::FLOATS * 4, st, a);
     const dim3 post(a.T, (a.n_head + 7) / 8);
     if (f32) launch_pdl(retention_post_kernel<float>, post, 256, 0, st, a);
     else launch_pdl(retention_post_kernel<bf16>, post, 256, 0, st, a);
