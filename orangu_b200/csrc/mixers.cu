@@ -309,9 +309,15 @@ __device__ __forceinline__ void ldsm4t(uint32_t (&r)[4], uint32_t addr) {
     asm volatile("ldmatrix.sync.aligned.m8n8.x4.trans.shared.b16 {%0, %1, %2, %3}, [%4];" : "=r"(r[0]), "=r"(r[1]), "=r"(r[2]), "=r"(r[3]) : "r"(addr) : "memory");
 }
 __device__ __forceinline__ void mma_bf16(float (&c)[4], const uint32_t (&a)[4], uint32_t b0, uint32_t b1) {
-    asm volatile("mma.sync.aligned.m16n8k16.row.col.f32.bf16.bf16.f32 {%0, %1, %2, %3}, {%4, %5, %6, %7}, {%8, %9}, {%0, %1, %2, %3};"
+    asm("mma.sync.aligned.m16n8k16.row.col.f32.bf16.bf16.f32 {%0, %1, %2, %3}, {%4, %5, %6, %7}, {%8, %9}, {%0, %1, %2, %3};"
                  : "+f"(c[0]), "+f"(c[1]), "+f"(c[2]), "+f"(c[3])
                  : "r"(a[0]), "r"(a[1]), "r"(a[2]), "r"(a[3]), "r"(b0), "r"(b1));
+}
+
+__device__ __forceinline__ float pow2(float x) {  // relative error below 2^-22; 0 for -inf
+    float y;
+    asm("ex2.approx.ftz.f32 %0, %1;" : "=f"(y) : "f"(x));
+    return y;
 }
 
 // The tile'th group of `rows` (token, head) rows: its span and first row within the span.  One warp; every lane gets the answer.
@@ -338,7 +344,8 @@ __device__ __forceinline__ void find_tile(const RowSpan *spans, uint32_t n_seq, 
     }
 }
 
-template <int MT>
+// NP: shares of sixteen latent columns per warp; a warp whose last share does not exist repeats another and drops it.
+template <int MT, int NP>
 __global__ void __launch_bounds__(LM_THREADS, MT == 4 ? 1 : 2) latent_attn_mma_kernel(LatentArgs a) {
     constexpr int M = 16 * MT, KT = LM_KEYS, SP = KT + 4, PP = KT + 8, PARTS = 4 / MT;  // MT row tiles x 2 key groups x PARTS of the row width = 8 warps
     extern __shared__ __align__(16) uint8_t smem[];
@@ -398,11 +405,11 @@ __global__ void __launch_bounds__(LM_THREADS, MT == 4 ? 1 : 2) latent_attn_mma_k
     }
     const float scale2 = a.scale * 1.4426950408889634f;  // weights are powers of two of the scaled score
     const uint32_t n_pair = a.kv_p / 16;
-    float acc[MT][LM_PAIRS][2][4];
+    float acc[MT][NP][2][4];
 #pragma unroll
     for (int i = 0; i < MT; ++i)
 #pragma unroll
-        for (int p = 0; p < LM_PAIRS; ++p)
+        for (int p = 0; p < NP; ++p)
 #pragma unroll
             for (int n = 0; n < 2; ++n)
 #pragma unroll
@@ -462,7 +469,7 @@ __global__ void __launch_bounds__(LM_THREADS, MT == 4 ? 1 : 2) latent_attn_mma_k
             float l = 0.0f;
 #pragma unroll
             for (int u = 0; u < KT / 32; ++u) {
-                const float e = m_new == -INFINITY ? 0.0f : exp2f(v[u] - m_new);
+                const float e = m_new == -INFINITY ? 0.0f : pow2(v[u] - m_new);
                 const bf16 h = __float2bfloat16_rn(e);
                 Ph[r * PP + u * 32 + lane] = h;
                 Pl[r * PP + u * 32 + lane] = __float2bfloat16_rn(e - __bfloat162float(h));
@@ -470,7 +477,7 @@ __global__ void __launch_bounds__(LM_THREADS, MT == 4 ? 1 : 2) latent_attn_mma_k
             }
             l = warp_sum(l);
             if (lane == 0) {
-                const float f = m_new == -INFINITY ? 1.0f : exp2f(m_old - m_new);
+                const float f = m_new == -INFINITY ? 1.0f : pow2(m_old - m_new);
                 keep[r] = f;
                 mx[r] = m_new;
                 sum[r] = sum[r] * f + l;
@@ -481,7 +488,7 @@ __global__ void __launch_bounds__(LM_THREADS, MT == 4 ? 1 : 2) latent_attn_mma_k
         for (int i = 0; i < MT; ++i) {
             const float f0r = keep[i * 16 + lane / 4], f1r = keep[i * 16 + lane / 4 + 8];
 #pragma unroll
-            for (int p = 0; p < LM_PAIRS; ++p)
+            for (int p = 0; p < NP; ++p)
 #pragma unroll
                 for (int n = 0; n < 2; ++n) acc[i][p][n][0] *= f0r, acc[i][p][n][1] *= f0r, acc[i][p][n][2] *= f1r, acc[i][p][n][3] *= f1r;
         }
@@ -494,10 +501,9 @@ __global__ void __launch_bounds__(LM_THREADS, MT == 4 ? 1 : 2) latent_attn_mma_k
                 ldsm4(fl[i], smem_addr(Pl) + (i * 16 * PP + kk * 16) * 2 + p_off);
             }
 #pragma unroll
-            for (int p = 0; p < LM_PAIRS; ++p) {
-                if (warp + 8 * p >= n_pair) break;
+            for (int p = 0; p < NP; ++p) {
                 uint32_t fv[4];
-                ldsm4t(fv, ks + kk * 16 * row_bytes + (warp + 8 * p) * 32 + v_off);
+                ldsm4t(fv, ks + kk * 16 * row_bytes + min(warp + 8 * p, n_pair - 1) * 32 + v_off);
 #pragma unroll
                 for (int i = 0; i < MT; ++i) {
                     mma_bf16(acc[i][p][0], fh[i], fv[0], fv[1]);
@@ -521,7 +527,7 @@ __global__ void __launch_bounds__(LM_THREADS, MT == 4 ? 1 : 2) latent_attn_mma_k
             const uint64_t flat = (uint64_t)row0 * a.n_head + f0 + r;
             const float inv = whole ? 1.0f / sum[r] : 1.0f;
 #pragma unroll
-            for (int p = 0; p < LM_PAIRS; ++p) {
+            for (int p = 0; p < NP; ++p) {
                 if (warp + 8 * p >= n_pair) break;
 #pragma unroll
                 for (int n = 0; n < 2; ++n) {
@@ -581,7 +587,7 @@ struct PfPlan {
         k_stage = PF_KEYS * (dqk + 8) * 2;
         v = k + 2 * k_stage;
         v_stage = PF_KEYS * (vd + 8) * 2;
-        bytes = v + 2 * v_stage;
+        bytes = v + 2 * v_stage + 128;  // a row's reads may go up to 64 columns past its end
     }
 };
 
@@ -599,7 +605,7 @@ __global__ void __launch_bounds__(256) latent_gather_kernel(LatentPrefillArgs a)
     for (uint32_t i = lane; i < a.dq / 8; i += 32) dst[i] = src[i];
 }
 
-template <int NV>  // columns of a value in sixteens, at most
+template <int NV>  // columns of a value in sixteens; what goes past vdim_k is computed from whatever follows in shared memory and dropped
 __global__ void __launch_bounds__(PF_THREADS, NV <= 8 ? 2 : 1) latent_prefill_kernel(LatentPrefillArgs a) {
     extern __shared__ __align__(16) uint8_t smem[];
     const uint32_t rot_p = a.dq - a.kv_p, dqk = a.dim_k + rot_p, qrow = (dqk + 8) * 2, vrow = (a.vdim_k + 8) * 2;
@@ -653,7 +659,6 @@ __global__ void __launch_bounds__(PF_THREADS, NV <= 8 ? 2 : 1) latent_prefill_ke
             for (int e = 0; e < 4; ++e) o[v][n][e] = 0.0f;
     const uint32_t qa = qs + (warp * 16 + (lane & 15)) * qrow + (lane >> 4) * 16;
     const uint32_t b_off = ((lane & 7) + ((lane >> 4) << 3)) * qrow + ((lane >> 3) & 1) * 16, v_off = ((lane & 7) + (((lane >> 3) & 1) << 3)) * vrow + (lane >> 4) * 16;
-    const uint32_t nv = a.vdim_k / 16;
     for (uint32_t it = 0; it < n_tiles; ++it) {
         if (it + 1 < n_tiles) load(it + 1);
         cp_commit();
@@ -666,7 +671,7 @@ __global__ void __launch_bounds__(PF_THREADS, NV <= 8 ? 2 : 1) latent_prefill_ke
             float c[PF_KEYS / 8][4];
 #pragma unroll
             for (int n = 0; n < PF_KEYS / 8; ++n) c[n][0] = c[n][1] = c[n][2] = c[n][3] = 0.0f;
-#pragma unroll 2
+#pragma unroll 4
             for (uint32_t k = 0; k < dqk / 16; ++k) {
                 uint32_t fa[4];
                 ldsm4(fa, qa + k * 32);
@@ -694,7 +699,7 @@ __global__ void __launch_bounds__(PF_THREADS, NV <= 8 ? 2 : 1) latent_prefill_ke
             b1 = fmaxf(b1, __shfl_xor_sync(0xffffffffu, b1, 1)), b1 = fmaxf(b1, __shfl_xor_sync(0xffffffffu, b1, 2));
             const float n0 = fmaxf(m0, b0), n1 = fmaxf(m1, b1);
             const float s0 = n0 == -INFINITY ? 0.0f : n0, s1 = n1 == -INFINITY ? 0.0f : n1;  // a row that has seen nothing yet keeps weights of zero
-            const float f0 = exp2f(m0 - s0), f1 = exp2f(m1 - s1);
+            const float f0 = pow2(m0 - s0), f1 = pow2(m1 - s1);
             m0 = n0, m1 = n1;
             l0 *= f0, l1 *= f1;
 #pragma unroll
@@ -709,7 +714,7 @@ __global__ void __launch_bounds__(PF_THREADS, NV <= 8 ? 2 : 1) latent_prefill_ke
 #pragma unroll
                     for (int r = 0; r < 2; ++r) {  // fragment register 2n + r: row half r of key half n
                         const float mr = r ? s1 : s0;
-                        const float e0 = exp2f(c[2 * kk + n][2 * r] - mr), e1 = exp2f(c[2 * kk + n][2 * r + 1] - mr);
+                        const float e0 = pow2(c[2 * kk + n][2 * r] - mr), e1 = pow2(c[2 * kk + n][2 * r + 1] - mr);
                         if (r) l1 += e0 + e1;
                         else l0 += e0 + e1;
                         const __nv_bfloat162 hi2 = __floats2bfloat162_rn(e0, e1);
@@ -719,7 +724,6 @@ __global__ void __launch_bounds__(PF_THREADS, NV <= 8 ? 2 : 1) latent_prefill_ke
                     }
 #pragma unroll
                 for (int v = 0; v < NV; ++v) {
-                    if (v >= (int)nv) break;
                     uint32_t fv[4];
                     ldsm4t(fv, vb + kk * 16 * vrow + v * 32 + v_off);
                     mma_bf16(o[v][0], ph, fv[0], fv[1]);
@@ -746,7 +750,7 @@ __global__ void __launch_bounds__(PF_THREADS, NV <= 8 ? 2 : 1) latent_prefill_ke
 #pragma unroll
             for (int n = 0; n < 2; ++n) {
                 const uint32_t col = v * 16 + n * 8 + 2 * (lane & 3);
-                if (v >= (int)nv || col >= a.vdim) continue;
+                if (col >= a.vdim) continue;
                 if ((a.vdim & 1) == 0) *reinterpret_cast<__nv_bfloat162 *>(out + col) = __floats2bfloat162_rn(o[v][n][2 * r] * f, o[v][n][2 * r + 1] * f);
                 else {
                     out[col] = __float2bfloat16_rn(o[v][n][2 * r] * f);
@@ -824,7 +828,7 @@ __global__ void __launch_bounds__(256) retention_kernel(RetentionArgs a) {
 #pragma unroll
     for (int i = 0; i < DW; ++i) {
         const uint32_t d = warp * DW + i;
-        S[i] = !fresh && live && d < a.dim ? state[(uint64_t)d * a.vdim] : 0.0f;
+        S[i] = !fresh && live && d < a.dim ? state[d * a.vdim] : 0.0f;
     }
     uint32_t stage = 0;
     for (uint32_t t0 = 0; t0 < sp.n; t0 += BLOCK, stage ^= 1u) {
@@ -865,7 +869,7 @@ __global__ void __launch_bounds__(256) retention_kernel(RetentionArgs a) {
 #pragma unroll
     for (int i = 0; i < DW; ++i) {
         const uint32_t d = warp * DW + i;
-        if (live && d < a.dim) state[(uint64_t)d * a.vdim] = S[i];
+        if (live && d < a.dim) state[d * a.vdim] = S[i];
     }
 }
 
@@ -904,6 +908,10 @@ __global__ void __launch_bounds__(256) copy_pool_pages_kernel(uint4 *pool, uint6
 }
 
 constexpr uint32_t MAX_SMEM = 227 * 1024;
+using LmKernel = void (*)(LatentArgs);
+const LmKernel LM_KERNELS[3][LM_PAIRS] = {{latent_attn_mma_kernel<1, 1>, latent_attn_mma_kernel<1, 2>, latent_attn_mma_kernel<1, 3>, latent_attn_mma_kernel<1, 4>},
+                                          {latent_attn_mma_kernel<2, 1>, latent_attn_mma_kernel<2, 2>, latent_attn_mma_kernel<2, 3>, latent_attn_mma_kernel<2, 4>},
+                                          {latent_attn_mma_kernel<4, 1>, latent_attn_mma_kernel<4, 2>, latent_attn_mma_kernel<4, 3>, latent_attn_mma_kernel<4, 4>}};
 size_t plain_smem(const LatentArgs &a) { return (size_t)(a.dq + a.kv_p + LA_KEYS) * 4; }
 
 }  // namespace
@@ -912,10 +920,11 @@ size_t plain_smem(const LatentArgs &a) { return (size_t)(a.dq + a.kv_p + LA_KEYS
 cudaError_t mixers_configure() {
     static PerDeviceOnce once;
     return once.run([] {
-        cudaError_t e = cudaFuncSetAttribute(latent_attn_mma_kernel<1>, cudaFuncAttributeMaxDynamicSharedMemorySize, MAX_SMEM - 64);
-        if (e == cudaSuccess) e = cudaFuncSetAttribute(latent_attn_mma_kernel<2>, cudaFuncAttributeMaxDynamicSharedMemorySize, MAX_SMEM - 64);
-        if (e == cudaSuccess) e = cudaFuncSetAttribute(latent_attn_mma_kernel<4>, cudaFuncAttributeMaxDynamicSharedMemorySize, MAX_SMEM - 64);
-        for (auto k : {latent_prefill_kernel<4>, latent_prefill_kernel<8>, latent_prefill_kernel<16>})
+        cudaError_t e = cudaSuccess;
+        for (int mt = 0; mt < 3; ++mt)
+            for (auto k : LM_KERNELS[mt])
+                if (e == cudaSuccess) e = cudaFuncSetAttribute(k, cudaFuncAttributeMaxDynamicSharedMemorySize, MAX_SMEM - 64);
+        for (auto k : {latent_prefill_kernel<2>, latent_prefill_kernel<4>, latent_prefill_kernel<6>, latent_prefill_kernel<8>, latent_prefill_kernel<12>, latent_prefill_kernel<16>})
             if (e == cudaSuccess) e = cudaFuncSetAttribute(k, cudaFuncAttributeMaxDynamicSharedMemorySize, MAX_SMEM - 64);
         if (e == cudaSuccess) e = cudaFuncSetAttribute(retention_kernel<8>, cudaFuncAttributeMaxDynamicSharedMemorySize, RtPlan<8>::FLOATS * 4);
         if (e == cudaSuccess) e = cudaFuncSetAttribute(retention_kernel<16>, cudaFuncAttributeMaxDynamicSharedMemorySize, RtPlan<16>::FLOATS * 4);
@@ -997,9 +1006,7 @@ uint32_t launch_latent_attention(const LatentArgs &a, bool f32, int sm_count, cu
     uint32_t splits = std::max(1u, std::min(std::min(slots, MERGE_MAX) / std::max(1u, tiles), (reach + KT - 1) / KT));
     while (splits > 1 && (uint64_t)splits * a.T * a.n_head * (a.kv_p + 2) > a.part_cap) --splits;
     const dim3 grid(tiles, splits);
-    if (mt == 1) launch_pdl(latent_attn_mma_kernel<1>, grid, LM_THREADS, plan.bytes, st, a);
-    else if (mt == 2) launch_pdl(latent_attn_mma_kernel<2>, grid, LM_THREADS, plan.bytes, st, a);
-    else launch_pdl(latent_attn_mma_kernel<4>, grid, LM_THREADS, plan.bytes, st, a);
+    launch_pdl(LM_KERNELS[mt == 4 ? 2 : mt - 1][(a.kv_p / 16 + 7) / 8 - 1], grid, LM_THREADS, plan.bytes, st, a);
     if (splits == 1) return 1;
     launch_pdl(latent_merge_kernel, a.T * a.n_head, 128, 0, st, a, splits);
     return 2;
@@ -1013,9 +1020,14 @@ void launch_latent_gather(const LatentPrefillArgs &a, cudaStream_t st) { launch_
 void launch_latent_prefill(const LatentPrefillArgs &a, cudaStream_t st) {
     const PfPlan pl(a.dim_k + a.dq - a.kv_p, a.vdim_k);
     const dim3 grid(a.n_tiles, a.n_head);
-    if (a.vdim_k <= 64) launch_pdl(latent_prefill_kernel<4>, grid, PF_THREADS, pl.bytes, st, a);
-    else if (a.vdim_k <= 128) launch_pdl(latent_prefill_kernel<8>, grid, PF_THREADS, pl.bytes, st, a);
-    else launch_pdl(latent_prefill_kernel<16>, grid, PF_THREADS, pl.bytes, st, a);
+    const uint32_t nv = a.vdim_k / 16;
+    auto run = [&](void (*k)(LatentPrefillArgs)) { launch_pdl(k, grid, PF_THREADS, pl.bytes, st, a); };
+    if (nv <= 2) run(latent_prefill_kernel<2>);
+    else if (nv <= 4) run(latent_prefill_kernel<4>);
+    else if (nv <= 6) run(latent_prefill_kernel<6>);
+    else if (nv <= 8) run(latent_prefill_kernel<8>);
+    else if (nv <= 12) run(latent_prefill_kernel<12>);
+    else run(latent_prefill_kernel<16>);
 }
 
 bool retention_supported(uint32_t dim) { return dim >= 1 && dim <= 256; }
