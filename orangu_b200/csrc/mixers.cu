@@ -577,7 +577,8 @@ __global__ void __launch_bounds__(128) latent_merge_kernel(LatentArgs a, uint32_
 // ---- latent attention of prompts: keys and values rebuilt from the latent, bf16 -------------------------------------------------------
 // With many tokens per sequence it is cheaper to multiply the window's latents out once (linear.cu) and attend per head: the score
 // product is dim + rot_dim wide and the output vdim wide, against kv_rank each in the latent space.  A CTA takes one head and 64
-// consecutive tokens of a sequence, a warp 16 of them; keys come in tiles of 64 through two stages of cp.async.  Scores, softmax
+// consecutive tokens of a sequence, a warp 16 of them; keys come in tiles of 64, the next keys while this tile is
+// weighted, the next values during the next scores.  Scores, softmax
 // and the weights' two bf16 parts (value and remainder) stay in registers.
 constexpr int PF_TOKENS = 64, PF_KEYS = 64, PF_THREADS = 128;
 struct PfPlan {
@@ -585,9 +586,9 @@ struct PfPlan {
     __host__ __device__ PfPlan(uint32_t dqk, uint32_t vd) {
         k = PF_TOKENS * (dqk + 8) * 2;
         k_stage = PF_KEYS * (dqk + 8) * 2;
-        v = k + 2 * k_stage;
+        v = k + k_stage;
         v_stage = PF_KEYS * (vd + 8) * 2;
-        bytes = v + 2 * v_stage + 128;  // a row's reads may go up to 64 columns past its end
+        bytes = v + v_stage + 128;  // a row's reads may go up to 64 columns past its end
     }
 };
 
@@ -606,7 +607,7 @@ __global__ void __launch_bounds__(256) latent_gather_kernel(LatentPrefillArgs a)
 }
 
 template <int NV>  // columns of a value in sixteens; what goes past vdim_k is computed from whatever follows in shared memory and dropped
-__global__ void __launch_bounds__(PF_THREADS, NV <= 8 ? 2 : 1) latent_prefill_kernel(LatentPrefillArgs a) {
+__global__ void __launch_bounds__(PF_THREADS, NV <= 8 ? 3 : 1) latent_prefill_kernel(LatentPrefillArgs a) {
     extern __shared__ __align__(16) uint8_t smem[];
     const uint32_t rot_p = a.dq - a.kv_p, dqk = a.dim_k + rot_p, qrow = (dqk + 8) * 2, vrow = (a.vdim_k + 8) * 2;
     const PfPlan pl(dqk, a.vdim_k);
@@ -632,20 +633,29 @@ __global__ void __launch_bounds__(PF_THREADS, NV <= 8 ? 2 : 1) latent_prefill_ke
             cp16(qs + r * qrow + c * 16, src, in);
         }
     }
-    auto load = [&](uint32_t it) {
-        const uint32_t kb = qs + pl.k + (it & 1u) * pl.k_stage, vb = qs + pl.v + (it & 1u) * pl.v_stage, j0 = lo + it * PF_KEYS;
-        const uint32_t cn = a.dim_k / 8, cr = rot_p / 8, cv = a.vdim_k / 8, ct = cn + cr + cv;
+    auto load_k = [&](uint32_t it) {
+        const uint32_t j0 = lo + it * PF_KEYS, cn = a.dim_k / 8, ct = cn + rot_p / 8;
         for (uint32_t i = threadIdx.x; i < PF_KEYS * ct; i += PF_THREADS) {
             const uint32_t r = i / ct, c = i - r * ct;
             const bool in = j0 + r < hi;
             const uint64_t key = sp.key0 + (in ? j0 + r - kbase : 0);
-            const bf16 *ex = static_cast<const bf16 *>(a.expanded) + key * a.ex_pitch;
-            if (c < cn) cp16(kb + r * qrow + c * 16, ex + (uint64_t)h * a.dim_k + 8 * c, in);
-            else if (c < cn + cr) cp16(kb + r * qrow + c * 16, static_cast<const bf16 *>(a.lat) + key * a.dq + a.kv_p + 8 * (c - cn), in);
-            else cp16(vb + r * vrow + (c - cn - cr) * 16, ex + a.ex_v0 + (uint64_t)h * a.vdim_k + 8 * (c - cn - cr), in);
+            const bf16 *src = c < cn ? static_cast<const bf16 *>(a.expanded) + key * a.ex_pitch + (uint64_t)h * a.dim_k + 8 * c
+                                     : static_cast<const bf16 *>(a.lat) + key * a.dq + a.kv_p + 8 * (c - cn);
+            cp16(qs + pl.k + r * qrow + c * 16, src, in);
         }
     };
-    load(0);
+    auto load_v = [&](uint32_t it) {
+        const uint32_t j0 = lo + it * PF_KEYS, cv = a.vdim_k / 8;
+        for (uint32_t i = threadIdx.x; i < PF_KEYS * cv; i += PF_THREADS) {
+            const uint32_t r = i / cv, c = i - r * cv;
+            const bool in = j0 + r < hi;
+            const uint64_t key = sp.key0 + (in ? j0 + r - kbase : 0);
+            cp16(qs + pl.v + r * vrow + c * 16, static_cast<const bf16 *>(a.expanded) + key * a.ex_pitch + a.ex_v0 + (uint64_t)h * a.vdim_k + 8 * c, in);
+        }
+    };
+    load_k(0);
+    cp_commit();
+    load_v(0);
     cp_commit();
     const float scale2 = a.scale * 1.4426950408889634f;
     const int p0 = (int)(sp.pos0 + t0 + warp * 16 + lane / 4), p1 = p0 + 8;  // positions of this thread's two rows
@@ -660,17 +670,15 @@ __global__ void __launch_bounds__(PF_THREADS, NV <= 8 ? 2 : 1) latent_prefill_ke
     const uint32_t qa = qs + (warp * 16 + (lane & 15)) * qrow + (lane >> 4) * 16;
     const uint32_t b_off = ((lane & 7) + ((lane >> 4) << 3)) * qrow + ((lane >> 3) & 1) * 16, v_off = ((lane & 7) + (((lane >> 3) & 1) << 3)) * vrow + (lane >> 4) * 16;
     for (uint32_t it = 0; it < n_tiles; ++it) {
-        if (it + 1 < n_tiles) load(it + 1);
-        cp_commit();
         cp_wait<1>();
-        __syncthreads();
+        __syncthreads();  // this tile's keys are there
         const int j0 = (int)(lo + it * PF_KEYS);
         const bool any = j0 <= w_last && (long long)j0 + PF_KEYS - 1 > (long long)w_first - win;  // does one of the warp's tokens see one of these keys?
-        if (any) {
-            const uint32_t kb = qs + pl.k + (it & 1u) * pl.k_stage, vb = qs + pl.v + (it & 1u) * pl.v_stage;
-            float c[PF_KEYS / 8][4];
+        const uint32_t kb = qs + pl.k, vb = qs + pl.v;
+        float c[PF_KEYS / 8][4];
 #pragma unroll
-            for (int n = 0; n < PF_KEYS / 8; ++n) c[n][0] = c[n][1] = c[n][2] = c[n][3] = 0.0f;
+        for (int n = 0; n < PF_KEYS / 8; ++n) c[n][0] = c[n][1] = c[n][2] = c[n][3] = 0.0f;
+        if (any) {
 #pragma unroll 4
             for (uint32_t k = 0; k < dqk / 16; ++k) {
                 uint32_t fa[4];
@@ -683,6 +691,11 @@ __global__ void __launch_bounds__(PF_THREADS, NV <= 8 ? 2 : 1) latent_prefill_ke
                     mma_bf16(c[2 * g + 1], fa, fb[2], fb[3]);
                 }
             }
+        }
+        __syncthreads();  // nobody reads them any more: the next tile's may come
+        if (it + 1 < n_tiles) load_k(it + 1);
+        cp_commit();
+        if (any) {
             const bool inside = j0 + PF_KEYS - 1 <= w_first && (long long)w_last - j0 < win && j0 + PF_KEYS <= (int)hi;  // nothing to mask
             float b0 = -INFINITY, b1 = -INFINITY;
 #pragma unroll
@@ -706,6 +719,11 @@ __global__ void __launch_bounds__(PF_THREADS, NV <= 8 ? 2 : 1) latent_prefill_ke
             for (int v = 0; v < NV; ++v)
 #pragma unroll
                 for (int n = 0; n < 2; ++n) o[v][n][0] *= f0, o[v][n][1] *= f0, o[v][n][2] *= f1, o[v][n][3] *= f1;
+        }
+        cp_wait<1>();
+        __syncthreads();  // and the values
+        if (any) {
+            const float s0 = m0 == -INFINITY ? 0.0f : m0, s1 = m1 == -INFINITY ? 0.0f : m1;
 #pragma unroll
             for (int kk = 0; kk < PF_KEYS / 16; ++kk) {
                 uint32_t ph[4], pr[4];
@@ -734,6 +752,8 @@ __global__ void __launch_bounds__(PF_THREADS, NV <= 8 ? 2 : 1) latent_prefill_ke
             }
         }
         __syncthreads();
+        if (it + 1 < n_tiles) load_v(it + 1);
+        cp_commit();
     }
     cp_wait<0>();
     l0 += __shfl_xor_sync(0xffffffffu, l0, 1), l0 += __shfl_xor_sync(0xffffffffu, l0, 2);
