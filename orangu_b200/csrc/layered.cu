@@ -522,7 +522,7 @@ int LayeredGraph::build(const ob_layered_desc &c) {
     if (side_dim && ((rc = scratch(&sg, T * side_p, es())) || (rc = scratch_f32(&sy, T * width)))) return rc;
     if (!f32 && (rc = scratch_f32(&split_part, linear_split_bytes() / 4))) return rc;
     if (q_n && !f32) {  // at most one CTA per SM, of 64 rows, writes partial results at a time (launch_latent_attention)
-        part_cap = ((uint64_t)m->ctx->sm_count * 64 + 64) * (kvp + 2);
+        part_cap = ((uint64_t)m->ctx->sm_count * 64 + 64) * (kvp + 4);
         if ((rc = scratch_f32(&part, part_cap))) return rc;
     }
     return OB_OK;

@@ -84,7 +84,7 @@ struct LatentArgs {          // latent attention of one layer over T rows
     void *cache;             // activations [page][16][dq]
     void *o;                 // activations [T][H * o_pitch_h]: attention output in the latent space
     uint32_t o_head;         // elements between heads in o
-    float *part;             // [splits][T * H][kv_p + 2] partial results (unnormalised output, max, sum)
+    float *part;             // [splits][T * H][kv_p + 4] partial results (unnormalised output, max, sum)
     uint64_t part_cap;       // floats `part` holds
     // rows
     uint32_t T, n_seq;

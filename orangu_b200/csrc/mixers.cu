@@ -277,6 +277,7 @@ __global__ void __launch_bounds__(LA_THREADS) latent_attn_plain_kernel(LatentArg
 // time, LM_PAIRS shares of them).  With fewer rows the warps also split the row width of the score product.  (mma.sync on purpose: with few tokens M is the number of heads, and 512 output columns for
 // 128 rows would take all of tensor memory.)
 constexpr int LM_THREADS = 256, LM_PAIRS = 4, LM_KEYS = 32;
+__host__ __device__ constexpr uint32_t lm_part_row(uint32_t kv_p) { return kv_p + 4; }  // floats of one partial result: output, then maximum and sum
 struct LmPlan {
     uint32_t q, k, stage, s, ph, pl, stat, bytes;  // byte offsets; stage: bytes of one key stage
     uint32_t stages;  // two, or one where that lets a second CTA onto the SM (its products then cover this one's loads)
@@ -319,6 +320,17 @@ __device__ __forceinline__ float pow2(float x) {  // relative error below 2^-22;
     asm("ex2.approx.ftz.f32 %0, %1;" : "=f"(y) : "f"(x));
     return y;
 }
+
+// How a warp copies rows of `chunks` 16-byte pieces: several short rows at a time, or one row in steps of 32 pieces.
+struct RowCopy {
+    uint32_t rows, row, chunk, chunks;  // rows per step of a warp, this lane's row among them and its first piece (chunks: none)
+    __device__ explicit RowCopy(uint32_t n) : chunks(n) {
+        const uint32_t lane = threadIdx.x & 31;
+        rows = n >= 32 ? 1 : 32 / n;
+        row = n >= 32 ? 0 : lane / n;
+        chunk = n >= 32 ? lane : row < rows ? lane - row * n : n;
+    }
+};
 
 // The tile'th group of `rows` (token, head) rows: its span and first row within the span.  One warp; every lane gets the answer.
 __device__ __forceinline__ void find_tile(const RowSpan *spans, uint32_t n_seq, uint32_t n_head, uint32_t rows, uint32_t tile, RowSpan *span, uint32_t *first) {
@@ -380,13 +392,24 @@ __global__ void __launch_bounds__(LM_THREADS, MT == 4 ? 1 : 2) latent_attn_mma_k
     }
     const uint32_t n_tiles = (hi - lo + KT - 1) / KT;
 
+    const RowCopy rc(chunks);
     auto load_keys = [&](uint32_t it) {
-        const uint32_t base = smem_addr(smem + pl.k) + (pl.stages == 2 ? it & 1u : 0u) * pl.stage;
-        for (uint32_t i = threadIdx.x; i < KT * chunks; i += LM_THREADS) {
-            const uint32_t r = i / chunks, c = i - r * chunks, j = lo + it * KT + r;
-            const bool in = j < hi;
-            const bf16 *src = static_cast<const bf16 *>(a.cache) + (in ? ((uint64_t)table[j / KV_PAGE] * KV_PAGE + j % KV_PAGE) * a.dq + 8 * c : 0);
-            cp16(base + r * row_bytes + c * 16, src, in);
+        const uint32_t base = smem_addr(smem + pl.k) + (pl.stages == 2 ? it & 1u : 0u) * pl.stage, step = LM_THREADS / 32 * rc.rows;
+        constexpr uint32_t AT_ONCE = 4;  // rows whose pages are looked up together
+        for (uint32_t r0 = warp * rc.rows + rc.row; r0 < KT; r0 += AT_ONCE * step) {
+            int32_t page[AT_ONCE];
+#pragma unroll
+            for (uint32_t u = 0; u < AT_ONCE; ++u) {
+                const uint32_t j = lo + it * KT + r0 + u * step;
+                page[u] = r0 + u * step < KT && j < hi ? table[j / KV_PAGE] : -1;
+            }
+#pragma unroll
+            for (uint32_t u = 0; u < AT_ONCE; ++u) {
+                const uint32_t r = r0 + u * step, j = lo + it * KT + r;
+                if (r >= KT) break;
+                const bf16 *src = static_cast<const bf16 *>(a.cache) + (page[u] >= 0 ? ((uint64_t)page[u] * KV_PAGE + j % KV_PAGE) * a.dq : 0);
+                for (uint32_t c = rc.chunk; c < chunks; c += 32) cp16(base + r * row_bytes + c * 16, src + 8 * c, page[u] >= 0);
+            }
         }
     };
     {   // queries: consecutive flat rows are consecutive in memory
@@ -534,43 +557,39 @@ __global__ void __launch_bounds__(LM_THREADS, MT == 4 ? 1 : 2) latent_attn_mma_k
                     const uint32_t col = (warp + 8 * p) * 16 + n * 8 + 2 * (lane & 3);
                     const float v0 = acc[i][p][n][2 * hf] * inv, v1 = acc[i][p][n][2 * hf + 1] * inv;
                     if (whole) *reinterpret_cast<__nv_bfloat162 *>(static_cast<bf16 *>(a.o) + flat * a.o_head + col) = __floats2bfloat162_rn(v0, v1);
-                    else *reinterpret_cast<float2 *>(a.part + ((uint64_t)blockIdx.y * a.T * a.n_head + flat) * (a.kv_p + 2) + col) = make_float2(v0, v1);
+                    else *reinterpret_cast<float2 *>(a.part + ((uint64_t)blockIdx.y * a.T * a.n_head + flat) * lm_part_row(a.kv_p) + col) = make_float2(v0, v1);
                 }
             }
             if (!whole && warp == 0 && (lane & 3) == 0)
-                *reinterpret_cast<float2 *>(a.part + ((uint64_t)blockIdx.y * a.T * a.n_head + flat) * (a.kv_p + 2) + a.kv_p) = make_float2(mx[r], sum[r]);
+                *reinterpret_cast<float2 *>(a.part + ((uint64_t)blockIdx.y * a.T * a.n_head + flat) * lm_part_row(a.kv_p) + a.kv_p) = make_float2(mx[r], sum[r]);
         }
 }
 
-// The splits of one (token, head) row put together.
+// The splits of one (token, head) row put together: a CTA per row when there are few, a warp per row when there are many.
 constexpr uint32_t MERGE_MAX = 256;  // splits
-__global__ void __launch_bounds__(128) latent_merge_kernel(LatentArgs a, uint32_t n_splits) {
-    __shared__ float wt[MERGE_MAX];
-    __shared__ float red[33];
+__global__ void __launch_bounds__(128) latent_merge_kernel(LatentArgs a, uint32_t n_splits, uint32_t rows_per_cta) {
     pdl_release();
     pdl_wait();
-    const uint64_t flat = blockIdx.x, stride = (uint64_t)a.T * a.n_head * (a.kv_p + 2);
-    const float *p = a.part + flat * (a.kv_p + 2);
-    float m = -INFINITY;
-    for (uint32_t s = threadIdx.x & 31; s < n_splits; s += 32) m = fmaxf(m, p[s * stride + a.kv_p]);  // every warp for itself
+    const uint32_t lane = threadIdx.x & 31, width = rows_per_cta == 1 ? 128 : 32;
+    const uint64_t flat = (uint64_t)blockIdx.x * rows_per_cta + (rows_per_cta == 1 ? 0 : threadIdx.x >> 5), n_flat = (uint64_t)a.T * a.n_head;
+    if (flat >= n_flat) return;
+    const uint64_t stride = n_flat * lm_part_row(a.kv_p);
+    const float *p = a.part + flat * lm_part_row(a.kv_p), *ml = p + a.kv_p;
+    float m = -INFINITY, l = 0.0f;
+    for (uint32_t s = lane; s < n_splits; s += 32) m = fmaxf(m, ml[s * stride]);
     m = warp_max(m);
-    float l = 0.0f;
-    for (uint32_t s = threadIdx.x; s < n_splits; s += blockDim.x) {
-        const float2 ml = *reinterpret_cast<const float2 *>(p + s * stride + a.kv_p);
-        const float e = exp2f(ml.x - m);
-        wt[s] = e;
-        l += e * ml.y;
-    }
-    const float inv = 1.0f / block_sum(l, red);  // synchronises: wt is complete
+    for (uint32_t s = lane; s < n_splits; s += 32) l += pow2(ml[s * stride] - m) * ml[s * stride + 1];
+    const float inv = 1.0f / warp_sum(l);
     bf16 *o = static_cast<bf16 *>(a.o) + flat * a.o_head;
-    for (uint32_t c = 2 * threadIdx.x; c < a.kv_p; c += 2 * blockDim.x) {
-        float2 v = make_float2(0.0f, 0.0f);
+    for (uint32_t c = 4 * (threadIdx.x % width); c < a.kv_p; c += 4 * width) {
+        float4 v = make_float4(0.0f, 0.0f, 0.0f, 0.0f);
 #pragma unroll 8
         for (uint32_t s = 0; s < n_splits; ++s) {
-            const float2 u = *reinterpret_cast<const float2 *>(p + s * stride + c);
-            v.x = fmaf(wt[s], u.x, v.x), v.y = fmaf(wt[s], u.y, v.y);
+            const float w = pow2(ml[s * stride] - m);
+            const float4 u = *reinterpret_cast<const float4 *>(p + s * stride + c);
+            v.x = fmaf(w, u.x, v.x), v.y = fmaf(w, u.y, v.y), v.z = fmaf(w, u.z, v.z), v.w = fmaf(w, u.w, v.w);
         }
-        *reinterpret_cast<__nv_bfloat162 *>(o + c) = __floats2bfloat162_rn(v.x * inv, v.y * inv);
+        store4<bf16>(o + c, mul4(v, inv));
     }
 }
 
@@ -1024,11 +1043,12 @@ uint32_t launch_latent_attention(const LatentArgs &a, bool f32, int sm_count, cu
     const uint32_t span = M / a.n_head + 2, reach = a.window ? std::min<uint64_t>(a.max_pos, (uint64_t)a.window + span) : a.max_pos;
     const uint32_t slots = (uint32_t)sm_count * (mt == 4 || 2 * plan.bytes > 224 * 1024 ? 1 : 2);
     uint32_t splits = std::max(1u, std::min(std::min(slots, MERGE_MAX) / std::max(1u, tiles), (reach + KT - 1) / KT));
-    while (splits > 1 && (uint64_t)splits * a.T * a.n_head * (a.kv_p + 2) > a.part_cap) --splits;
+    while (splits > 1 && (uint64_t)splits * a.T * a.n_head * lm_part_row(a.kv_p) > a.part_cap) --splits;
     const dim3 grid(tiles, splits);
     launch_pdl(LM_KERNELS[mt == 4 ? 2 : mt - 1][(a.kv_p / 16 + 7) / 8 - 1], grid, LM_THREADS, plan.bytes, st, a);
     if (splits == 1) return 1;
-    launch_pdl(latent_merge_kernel, a.T * a.n_head, 128, 0, st, a, splits);
+    const uint32_t merge_rows = a.T * a.n_head, per = merge_rows >= 1024 ? 4 : 1;
+    launch_pdl(latent_merge_kernel, (merge_rows + per - 1) / per, 128, 0, st, a, splits, per);
     return 2;
 }
 
