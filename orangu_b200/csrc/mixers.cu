@@ -455,56 +455,70 @@ __global__ void __launch_bounds__(LM_THREADS, MT == 4 ? 1 : 2) latent_attn_mma_k
         __syncthreads();
         const uint32_t ks = smem_addr(smem + pl.k) + (pl.stages == 2 ? it & 1u : 0u) * pl.stage;
         {
-            float c[2][4] = {};
+            float c[2][2][4] = {};  // even and odd steps have accumulators of their own: no product waits for the one before
             const uint32_t qa = qs + mt_s * 16 * row_bytes + a_off, kb = ks + kg * 16 * row_bytes + b_off;
-#pragma unroll 4
-            for (uint32_t k = k_first; k < k_end; ++k) {
+            auto step = [&](uint32_t k, float (&d)[2][4]) {
                 uint32_t fa[4], fb[4];
                 ldsm4(fa, qa + k * 32);
                 ldsm4(fb, kb + k * 32);
-                mma_bf16(c[0], fa, fb[0], fb[1]);
-                mma_bf16(c[1], fa, fb[2], fb[3]);
+                mma_bf16(d[0], fa, fb[0], fb[1]);
+                mma_bf16(d[1], fa, fb[2], fb[3]);
+            };
+            uint32_t k = k_first;
+#pragma unroll 3
+            for (; k + 1 < k_end; k += 2) {
+                step(k, c[0]);
+                step(k + 1, c[1]);
             }
+            if (k < k_end) step(k, c[0]);
             float *s = S + (wp * M + mt_s * 16 + lane / 4) * SP + kg * 16 + 2 * (lane & 3);
 #pragma unroll
             for (int n = 0; n < 2; ++n) {
-                *reinterpret_cast<float2 *>(s + 8 * n) = make_float2(c[n][0], c[n][1]);
-                *reinterpret_cast<float2 *>(s + 8 * SP + 8 * n) = make_float2(c[n][2], c[n][3]);
+                *reinterpret_cast<float2 *>(s + 8 * n) = make_float2(c[0][n][0] + c[1][n][0], c[0][n][1] + c[1][n][1]);
+                *reinterpret_cast<float2 *>(s + 8 * SP + 8 * n) = make_float2(c[0][n][2] + c[1][n][2], c[0][n][3] + c[1][n][3]);
             }
         }
         __syncthreads();
+        {   // online softmax: lane = key, the warp's rows side by side
+            constexpr int R = M / 8;
+            const int j = (int)(lo + it * KT) + (int)lane, r0 = warp * R;
+            float v[R], m_old[R], m_new[R], l[R];
 #pragma unroll
-        for (int i = 0; i < M / 8; ++i) {  // online softmax, a warp per row
-            const int r = warp * (M / 8) + i, p = rpos[r];
-            float v[KT / 32], best = -INFINITY;
+            for (int i = 0; i < R; ++i) {
+                const int p = rpos[r0 + i];
+                float sc = S[(r0 + i) * SP + lane];
 #pragma unroll
-            for (int u = 0; u < KT / 32; ++u) {
-                const int j = (int)(lo + it * KT) + u * 32 + (int)lane;
-                const bool see = j <= p && j < (int)hi && (a.window == 0 || p - j < (int)a.window);
-                float sc = S[r * SP + u * 32 + lane];
-#pragma unroll
-                for (int w = 1; w < PARTS; ++w) sc += S[(w * M + r) * SP + u * 32 + lane];
-                v[u] = see ? sc * scale2 : -INFINITY;
-                best = fmaxf(best, v[u]);
+                for (int w = 1; w < PARTS; ++w) sc += S[(w * M + r0 + i) * SP + lane];
+                v[i] = j <= p && j < (int)hi && (a.window == 0 || p - j < (int)a.window) ? sc * scale2 : -INFINITY;
+                m_new[i] = v[i];
+                m_old[i] = mx[r0 + i];
             }
-            best = warp_max(best);
-            const float m_old = mx[r], m_new = fmaxf(m_old, best);
-            float l = 0.0f;
 #pragma unroll
-            for (int u = 0; u < KT / 32; ++u) {
-                const float e = m_new == -INFINITY ? 0.0f : pow2(v[u] - m_new);
+            for (int o = 16; o > 0; o >>= 1)
+#pragma unroll
+                for (int i = 0; i < R; ++i) m_new[i] = fmaxf(m_new[i], __shfl_xor_sync(0xffffffffu, m_new[i], o));
+#pragma unroll
+            for (int i = 0; i < R; ++i) {
+                m_new[i] = fmaxf(m_new[i], m_old[i]);
+                const float e = m_new[i] == -INFINITY ? 0.0f : pow2(v[i] - m_new[i]);
                 const bf16 h = __float2bfloat16_rn(e);
-                Ph[r * PP + u * 32 + lane] = h;
-                Pl[r * PP + u * 32 + lane] = __float2bfloat16_rn(e - __bfloat162float(h));
-                l += e;
+                Ph[(r0 + i) * PP + lane] = h;
+                Pl[(r0 + i) * PP + lane] = __float2bfloat16_rn(e - __bfloat162float(h));
+                l[i] = e;
             }
-            l = warp_sum(l);
-            if (lane == 0) {
-                const float f = m_new == -INFINITY ? 1.0f : pow2(m_old - m_new);
-                keep[r] = f;
-                mx[r] = m_new;
-                sum[r] = sum[r] * f + l;
-            }
+#pragma unroll
+            for (int o = 16; o > 0; o >>= 1)
+#pragma unroll
+                for (int i = 0; i < R; ++i) l[i] += __shfl_xor_sync(0xffffffffu, l[i], o);
+            __syncwarp();  // every lane has read the old maxima
+#pragma unroll
+            for (int i = 0; i < R; ++i)
+                if (lane == i) {
+                    const float f = m_new[i] == -INFINITY ? 1.0f : pow2(m_old[i] - m_new[i]);
+                    keep[r0 + i] = f;
+                    mx[r0 + i] = m_new[i];
+                    sum[r0 + i] = sum[r0 + i] * f + l[i];
+                }
         }
         __syncthreads();
 #pragma unroll
@@ -523,18 +537,18 @@ __global__ void __launch_bounds__(LM_THREADS, MT == 4 ? 1 : 2) latent_attn_mma_k
                 ldsm4(fh[i], smem_addr(Ph) + (i * 16 * PP + kk * 16) * 2 + p_off);
                 ldsm4(fl[i], smem_addr(Pl) + (i * 16 * PP + kk * 16) * 2 + p_off);
             }
+            uint32_t fv[NP][4];
 #pragma unroll
-            for (int p = 0; p < NP; ++p) {
-                uint32_t fv[4];
-                ldsm4t(fv, ks + kk * 16 * row_bytes + min(warp + 8 * p, n_pair - 1) * 32 + v_off);
+            for (int p = 0; p < NP; ++p) ldsm4t(fv[p], ks + kk * 16 * row_bytes + min(warp + 8 * p, n_pair - 1) * 32 + v_off);
 #pragma unroll
-                for (int i = 0; i < MT; ++i) {
-                    mma_bf16(acc[i][p][0], fh[i], fv[0], fv[1]);
-                    mma_bf16(acc[i][p][1], fh[i], fv[2], fv[3]);
-                    mma_bf16(acc[i][p][0], fl[i], fv[0], fv[1]);
-                    mma_bf16(acc[i][p][1], fl[i], fv[2], fv[3]);
-                }
-            }
+            for (int part = 0; part < 2; ++part)
+#pragma unroll
+                for (int p = 0; p < NP; ++p)
+#pragma unroll
+                    for (int i = 0; i < MT; ++i) {
+                        mma_bf16(acc[i][p][0], part ? fl[i] : fh[i], fv[p][0], fv[p][1]);
+                        mma_bf16(acc[i][p][1], part ? fl[i] : fh[i], fv[p][2], fv[p][3]);
+                    }
         }
         __syncthreads();
     }
