@@ -581,12 +581,19 @@ __global__ void __launch_bounds__(LM_THREADS, MT == 4 ? 1 : 2) latent_attn_mma_k
 
 // The splits of one (token, head) row put together: a CTA per row when there are few, a warp per row when there are many.
 constexpr uint32_t MERGE_MAX = 256;  // splits
-__global__ void __launch_bounds__(128) latent_merge_kernel(LatentArgs a, uint32_t n_splits, uint32_t rows_per_cta) {
+__global__ void __launch_bounds__(128) latent_merge_kernel(LatentArgs a, uint32_t n_splits, uint32_t n_rows, uint32_t rows_per_cta) {
     pdl_release();
     pdl_wait();
     const uint32_t lane = threadIdx.x & 31, width = rows_per_cta == 1 ? 128 : 32;
-    const uint64_t flat = (uint64_t)blockIdx.x * rows_per_cta + (rows_per_cta == 1 ? 0 : threadIdx.x >> 5), n_flat = (uint64_t)a.T * a.n_head;
-    if (flat >= n_flat) return;
+    const uint64_t n_flat = (uint64_t)a.T * a.n_head;
+    uint64_t flat = (uint64_t)blockIdx.x * rows_per_cta + (rows_per_cta == 1 ? 0 : threadIdx.x >> 5);
+    if (flat >= n_rows) return;
+    if (!a.single) {  // only the rows of these spans have partial results
+        RowSpan sp;
+        uint32_t f;
+        find_tile(a.spans, a.n_seq, a.n_head, 1, (uint32_t)flat, &sp, &f);
+        flat = (uint64_t)sp.row0 * a.n_head + f;
+    }
     const uint64_t stride = n_flat * lm_part_row(a.kv_p);
     const float *p = a.part + flat * lm_part_row(a.kv_p), *ml = p + a.kv_p;
     float m = -INFINITY, l = 0.0f;
@@ -1061,8 +1068,11 @@ uint32_t launch_latent_attention(const LatentArgs &a, bool f32, int sm_count, cu
     const dim3 grid(tiles, splits);
     launch_pdl(LM_KERNELS[mt == 4 ? 2 : mt - 1][(a.kv_p / 16 + 7) / 8 - 1], grid, LM_THREADS, plan.bytes, st, a);
     if (splits == 1) return 1;
-    const uint32_t merge_rows = a.T * a.n_head, per = merge_rows >= 1024 ? 4 : 1;
-    launch_pdl(latent_merge_kernel, (merge_rows + per - 1) / per, 128, 0, st, a, splits, per);
+    uint32_t merge_rows = a.single ? a.n_seq * a.n_head : 0;
+    if (!a.single)
+        for (uint32_t s = 0; s < a.n_seq; ++s) merge_rows += a.h_spans[s].n * a.n_head;
+    const uint32_t per = merge_rows >= 1024 ? 4 : 1;
+    launch_pdl(latent_merge_kernel, (merge_rows + per - 1) / per, 128, 0, st, a, splits, merge_rows, per);
     return 2;
 }
 

@@ -128,6 +128,48 @@ def test_unequal_requests_in_one_batch(backend, dtype):
 
 
 @pytest.mark.parametrize("dtype", DTYPES)
+@pytest.mark.parametrize("window", (1, 37, 90, 400))
+def test_long_portions(backend, window, dtype):
+    """Portions long enough for the per-head attention of prompts, started anywhere, beside short ones and single tokens."""
+    cfg = F.config([F.latent(window=window, dim=40, vdim=18), F.retention(), F.latent(heads=2, window=window, dim=16, rot_dim=8, vdim=72, kv_rank=24)], ff=[40, 40, None])
+    w = F.weights(cfg, 36, gain=2.0)
+    prompts = [F.tokens(cfg, n, 37 + n) for n in (230, 165, 131)]
+    want = [P.forward(cfg, F.values(w), p)[0] for p in prompts]
+    m = make(backend, cfg, w, dtype, pool=1024, rows=512)
+    kvs = [m.new_kv_cache(256, paged=True) for _ in prompts]
+    got = [[] for _ in prompts]
+    at = [0, 0, 0]
+    for sizes in ((3, 70, 64), (65, 1, 0), (1, 64, 66), (64, 30, 1), (97, 0, 0)):
+        live = [i for i in range(3) if sizes[i]]
+        lg = m.forward_rows([kvs[i] for i in live], [prompts[i][at[i]:at[i] + sizes[i]] for i in live], range(sum(sizes)))
+        o = 0
+        for i in live:
+            got[i].append(lg[o:o + sizes[i]])
+            at[i] += sizes[i]
+            o += sizes[i]
+    assert at == [230, 165, 131]
+    for g, x in zip(got, want):
+        assert error(np.concatenate(g), x) < TOL[dtype]
+    m.close()
+
+
+@pytest.mark.parametrize("dtype", DTYPES)
+def test_many_prompts_in_one_step(backend, dtype):
+    """More long portions than one launch of the prompt attention takes, and more tokens than a step."""
+    cfg = F.config([F.latent(window=50)], ff=None)
+    w = F.weights(cfg, 46)
+    prompts = [F.tokens(cfg, 66 + i, 47 + i) for i in range(11)]
+    m = make(backend, cfg, w, dtype, pool=2048, rows=700, seq=128)
+    kvs = [m.new_kv_cache(128, paged=True) for _ in prompts]
+    ends = np.cumsum([len(p) for p in prompts]) - 1
+    lg = m.forward_rows(kvs, prompts, ends)
+    for g, p in zip(lg, prompts):
+        want = P.forward(cfg, F.values(w), p)[0]
+        assert error(g[None], want[-1:]) < TOL[dtype]
+    m.close()
+
+
+@pytest.mark.parametrize("dtype", DTYPES)
 def test_many_single_tokens(backend, dtype):
     """A decode batch wide enough for the tensor-core products, at unequal lengths."""
     w = F.weights(MIX, 41)
@@ -234,11 +276,13 @@ def test_window_edges(backend, window, dtype):
             want = P.forward(cfg, v, toks)[0]
             wrong = P.forward(other[-1 if inside else 1], v, toks)[0]
             assert error(wrong[i:], want[i:]) > 0.2
-            m = make(backend, cfg, w, dtype)
-            whole, step, two = (m.new_kv_cache(256, paged=True) for _ in range(3))
+            m = make(backend, cfg, w, dtype, pool=1024)
+            whole, step, two, far = (m.new_kv_cache(256, paged=True) for _ in range(4))
             assert error(run(m, whole, toks)[i:], want[i:]) < TOL[dtype]
             assert error(run(m, step, toks, (i,))[i:], want[i:]) < TOL[dtype]
             assert error(run(m, two, toks, (j, i - 1) if i - 1 > j else (j,))[i:], want[i:]) < TOL[dtype]
+            longer = toks + [filler] * 70  # key and question at the start of long portions
+            assert error(run(m, far, longer, (j, i))[i:i + 1], want[i:]) < TOL[dtype]
             m.close()
 
 
