@@ -44,6 +44,7 @@ struct LayerPlan {
     void *pool = nullptr;
     // retention
     float *decay = nullptr, *state = nullptr;
+    float decay_min = 0.0f;
 };
 
 // A zero-padded bfloat16 matrix put together on the host from parts of others.
@@ -104,7 +105,7 @@ struct LayeredGraph : StepGraph {
     void layers(uint32_t T, uint32_t n_seq, const RowSpan *spans, uint32_t max_pos, cudaStream_t st) override;
     void head(const uint32_t *d_rows, uint32_t n, cudaStream_t st) override;
     void latent(const LayerPlan &P, uint32_t T, uint32_t n_seq, const RowSpan *spans, bool single, uint32_t max_pos, cudaStream_t st);
-    void retention(const LayerPlan &P, uint32_t T, uint32_t n_seq, cudaStream_t st);
+    void retention(const LayerPlan &P, uint32_t T, uint32_t n_seq, const RowSpan *spans, cudaStream_t st);
     int copy_prefix(ob_kv *dst, const ob_kv *src, uint32_t n) override;
     int read_pages(const ob_kv *kv, uint32_t layer, uint32_t pos0, uint32_t n, float *k_out, float *v_out) override;
     int read_state(const ob_kv *kv, uint32_t layer, float *out) override;
@@ -135,6 +136,12 @@ struct LayeredGraph : StepGraph {
     int build(const ob_layered_desc &c);
     int build_layer(const ob_block_desc &b, LayerPlan &P);
 };
+
+// Spans of a step come with the long ones last (forward_spans).
+uint32_t first_long(const RowSpan *spans, uint32_t n_seq) {
+    while (n_seq && spans[n_seq - 1].n >= PREFILL_SPAN) --n_seq;
+    return n_seq;
+}
 
 void LayeredGraph::latent(const LayerPlan &P, uint32_t T, uint32_t n_seq, const RowSpan *spans, bool single, uint32_t max_pos, cudaStream_t st) {
     const MetaLayout ml(m->T);
@@ -168,9 +175,7 @@ void LayeredGraph::latent(const LayerPlan &P, uint32_t T, uint32_t n_seq, const 
     a.max_pos = max_pos;
     launch_latent_prep(a, f32, st);
     m->ctx->launches++;
-    uint32_t n_short = n_seq;  // spans that attend in the latent space; the longer ones follow them
-    if (P.expand.rows)
-        while (n_short && spans[n_short - 1].n >= PREFILL_SPAN) --n_short;
+    const uint32_t n_short = P.expand.rows ? first_long(spans, n_seq) : n_seq;  // spans that attend in the latent space
     const float *gate = y + (size_t)H * P.mx.rot_dim + P.mx.kv_rank + P.mx.rot_dim;
     if (n_short) {
         a.n_seq = n_short;
@@ -232,7 +237,7 @@ void LayeredGraph::latent(const LayerPlan &P, uint32_t T, uint32_t n_seq, const 
     }
 }
 
-void LayeredGraph::retention(const LayerPlan &P, uint32_t T, uint32_t n_seq, cudaStream_t st) {
+void LayeredGraph::retention(const LayerPlan &P, uint32_t T, uint32_t n_seq, const RowSpan *spans, cudaStream_t st) {
     const MetaLayout ml(m->T);
     RetentionArgs a{};
     a.y = y;
@@ -253,6 +258,8 @@ void LayeredGraph::retention(const LayerPlan &P, uint32_t T, uint32_t n_seq, cud
     a.spans = reinterpret_cast<const RowSpan *>(m->d_meta + ml.off_spans);
     a.positions = reinterpret_cast<const uint32_t *>(m->d_meta + ml.off_positions);
     a.slots = reinterpret_cast<const int32_t *>(m->d_meta + ml.off_slots);
+    a.first_long = first_long(spans, n_seq);
+    a.decay_min = P.decay_min;
     m->ctx->launches += launch_retention(a, f32, m->ctx->sm_count, st);
 }
 
@@ -273,7 +280,7 @@ void LayeredGraph::layers(uint32_t T, uint32_t n_seq, const RowSpan *spans, uint
         linear(in, st);
 
         if (P.mx.kind == OB_MIXER_LATENT_ATTENTION) latent(P, T, n_seq, spans, single, max_pos, st);
-        else retention(P, T, n_seq, st);
+        else retention(P, T, n_seq, spans, st);
 
         LinArgs out = product(P.out, cat, cat_pitch, T);
         segment(out, 0, width, LE_RESIDUAL, m->x, width);
@@ -447,6 +454,7 @@ int LayeredGraph::build_layer(const ob_block_desc &b, LayerPlan &P) {
         if ((rc = scratch(&P.pool, (size_t)m->pool_pages * KV_PAGE * P.dq, es()))) return rc;
     } else {
         if ((rc = upload_f32(m, x.decay, H, &P.decay))) return rc;
+        P.decay_min = *std::min_element(x.decay, x.decay + H);
         if ((rc = scratch_f32(&P.state, (size_t)m->n_state_slots * state_elems(P)))) return rc;
         has_state = true;
     }

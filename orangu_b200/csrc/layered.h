@@ -145,6 +145,8 @@ struct RetentionArgs {       // retention of one layer over T rows
     const RowSpan *spans;
     const uint32_t *positions;
     const int32_t *slots;    // [T]
+    uint32_t first_long;     // spans from here on are long (PREFILL_SPAN rows or more)
+    float decay_min;         // of decay
 };
 bool retention_supported(uint32_t dim);
 uint32_t launch_retention(const RetentionArgs &a, bool f32, int sm_count, cudaStream_t st);

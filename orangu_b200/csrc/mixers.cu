@@ -933,6 +933,125 @@ __global__ void __launch_bounds__(256) retention_kernel(RetentionArgs a) {
     }
 }
 
+// The same recurrence for long spans.  A thread has R of the state's rows x 2 columns, so that one read of q and k from shared
+// memory serves both: lane = rows, warp = columns, 16 columns per CTA.  Over a block of eight tokens the state is kept without its
+// decay (S' = decay^-t S, the values scaled instead, the outputs scaled back), and the 16 sums of a block (token, column) are added
+// over the lanes by one exchange that leaves every other lane the sum it stores.
+constexpr int RS_BLOCK = 8, RS_COLS = 16;
+template <int R>
+__global__ void __launch_bounds__(256, R <= 4 ? 2 : 1) retention_span_kernel(RetentionArgs a) {
+    constexpr int D = 32 * R, V4 = R <= 4 ? 1 : R / 4, W = R / V4;  // a lane's rows: V4 groups of W neighbours
+    constexpr uint32_t STAGES = R <= 4 ? 4 : 2;
+    __shared__ __align__(16) float qs[STAGES][RS_BLOCK][D], ks[STAGES][RS_BLOCK][D], vs[STAGES][RS_BLOCK][RS_COLS];
+    pdl_release();
+    pdl_wait();
+    const uint32_t warp = threadIdx.x >> 5, lane = threadIdx.x & 31, h = blockIdx.y, col0 = blockIdx.x * RS_COLS;
+    const RowSpan sp = a.spans[a.first_long + blockIdx.z];
+    const float *yq = a.y + (uint64_t)sp.row0 * a.y_pitch + (uint64_t)h * a.dim, *yk = yq + (uint64_t)a.n_head * a.dim;
+    const float *yv = a.y + (uint64_t)sp.row0 * a.y_pitch + 2ull * a.n_head * a.dim + (uint64_t)h * a.vdim + col0;
+    const bool quads = a.dim % 4 == 0;  // rows of y start at multiples of 16 bytes, so do the heads then
+    auto load = [&](uint32_t t0, uint32_t stage) {
+        const uint32_t n = min((uint32_t)RS_BLOCK, sp.n - t0), step = quads ? 4 : 1;
+        for (uint32_t i = threadIdx.x * step; i < RS_BLOCK * D; i += 256 * step) {
+            const uint32_t t = i / D, d = i % D;
+            const bool in = t < n && d < a.dim;
+            const uint64_t o = in ? (uint64_t)(t0 + t) * a.y_pitch + d : 0;
+            if (quads) {
+                cp16(smem_addr(&qs[stage][t][d]), yq + o, in);
+                cp16(smem_addr(&ks[stage][t][d]), yk + o, in);
+            } else {
+                cp4(&qs[stage][t][d], yq + o, in);
+                cp4(&ks[stage][t][d], yk + o, in);
+            }
+        }
+        if (threadIdx.x < RS_BLOCK * RS_COLS) {
+            const uint32_t t = threadIdx.x / RS_COLS, c = threadIdx.x % RS_COLS;
+            const bool in = t < n && col0 + c < a.vdim;
+            cp4(&vs[stage][t][c], in ? yv + (uint64_t)(t0 + t) * a.y_pitch + c : a.y, in);
+        }
+    };
+#pragma unroll
+    for (uint32_t s = 0; s + 1 < STAGES; ++s) {
+        if (s * RS_BLOCK < sp.n) load(s * RS_BLOCK, s);
+        cp_commit();
+    }
+    const float decay = a.decay[h];
+    float up[RS_BLOCK];  // decay^-(t+1)
+    up[0] = 1.0f / decay;
+#pragma unroll
+    for (int t = 1; t < RS_BLOCK; ++t) up[t] = up[t - 1] * up[0];
+    float down = decay, block = decay;  // decay^(t+1) of the token this lane stores, decay^RS_BLOCK
+    for (uint32_t t = 0; t < lane / 4; ++t) down *= decay;
+    for (int t = 1; t < RS_BLOCK; ++t) block *= decay;
+    float *state = a.state + (((uint64_t)a.slots[sp.row0] * a.n_head + h) * a.dim) * a.vdim + col0 + 2 * warp;
+    const bool fresh = a.positions[sp.row0] == 0;
+    float S[R][2];
+    auto row_of = [&](int i) { return (uint32_t)(i / W) * (32 * W) + lane * W + i % W; };
+    auto exists = [&](int i, int c) { return row_of(i) < a.dim && col0 + 2 * warp + c < a.vdim; };
+#pragma unroll
+    for (int i = 0; i < R; ++i)
+#pragma unroll
+        for (int c = 0; c < 2; ++c) S[i][c] = !fresh && exists(i, c) ? state[row_of(i) * a.vdim + c] : 0.0f;
+    uint32_t stage = 0;
+    for (uint32_t t0 = 0; t0 < sp.n; t0 += RS_BLOCK, stage = (stage + 1) % STAGES) {
+        const uint32_t n = min((uint32_t)RS_BLOCK, sp.n - t0);
+        cp_wait<STAGES - 2>();
+        __syncthreads();  // this block's operands are there, and everyone has left the stage that is filled next
+        if (t0 + (STAGES - 1) * RS_BLOCK < sp.n) load(t0 + (STAGES - 1) * RS_BLOCK, (stage + STAGES - 1) % STAGES);
+        cp_commit();
+        float x[RS_BLOCK * 2];
+#pragma unroll
+        for (int t = 0; t < RS_BLOCK; ++t) {  // tokens past the end are zero: they change nothing
+            const float2 v = *reinterpret_cast<const float2 *>(&vs[stage][t][2 * warp]);
+            const float v0 = v.x * up[t], v1 = v.y * up[t];
+            float x0 = 0.0f, x1 = 0.0f;
+#pragma unroll
+            for (int g = 0; g < V4; ++g) {
+                float kk[W], qq[W];
+                const float *kp = &ks[stage][t][g * 32 * W + lane * W], *qp = &qs[stage][t][g * 32 * W + lane * W];
+                if constexpr (W == 4) {
+                    *reinterpret_cast<float4 *>(kk) = *reinterpret_cast<const float4 *>(kp);
+                    *reinterpret_cast<float4 *>(qq) = *reinterpret_cast<const float4 *>(qp);
+                } else {
+                    *reinterpret_cast<float2 *>(kk) = *reinterpret_cast<const float2 *>(kp);
+                    *reinterpret_cast<float2 *>(qq) = *reinterpret_cast<const float2 *>(qp);
+                }
+#pragma unroll
+                for (int e = 0; e < W; ++e) {
+                    float(&s)[2] = S[g * W + e];
+                    s[0] = fmaf(kk[e], v0, s[0]), s[1] = fmaf(kk[e], v1, s[1]);
+                    x0 = fmaf(qq[e], s[0], x0), x1 = fmaf(qq[e], s[1], x1);
+                }
+            }
+            x[2 * t] = x0, x[2 * t + 1] = x1;
+        }
+        float back = block;
+        if (n < RS_BLOCK) {
+            back = 1.0f;
+            for (uint32_t t = 0; t < n; ++t) back *= decay;
+        }
+#pragma unroll
+        for (int i = 0; i < R; ++i) S[i][0] *= back, S[i][1] *= back;
+#pragma unroll
+        for (int o = 8; o > 0; o >>= 1)  // lanes 2 l and 2 l + 1 end with the halves of the sum of x[l] over the lanes
+#pragma unroll
+            for (int i = 0; i < o; ++i) {
+                const bool hi = lane & (2 * o);
+                const float give = hi ? x[i] : x[i + o], mine = hi ? x[i + o] : x[i];
+                x[i] = mine + __shfl_xor_sync(0xffffffffu, give, 2 * o);
+            }
+        x[0] += __shfl_xor_sync(0xffffffffu, x[0], 1);
+        const uint32_t t = lane / 4, col = col0 + 2 * warp + lane / 2 % 2;
+        if ((lane & 1) == 0 && t < n && col < a.vdim) a.o[((uint64_t)(sp.row0 + t0 + t) * a.n_head + h) * a.vdim + col] = x[0] * down;
+    }
+    cp_wait<0>();
+#pragma unroll
+    for (int i = 0; i < R; ++i)
+#pragma unroll
+        for (int c = 0; c < 2; ++c)
+            if (exists(i, c)) state[row_of(i) * a.vdim + c] = S[i][c];
+}
+
 // Every head's output over its root mean square, times silu of its gate.  A warp per (token, head).
 constexpr int POST_VALUES = 8;  // per lane in registers; wider heads read the rest twice
 template <typename TA>
@@ -1099,14 +1218,23 @@ bool retention_supported(uint32_t dim) { return dim >= 1 && dim <= 256; }
 uint32_t launch_retention(const RetentionArgs &a, bool f32, int sm_count, cudaStream_t st) {
     (void)sm_count;
     launch_pdl(retention_prep_kernel, a.T, 256, 0, st, a);
-    const dim3 grid((a.vdim + 31) / 32, a.n_head, a.n_seq);
-    if (a.dim <= 64) launch_pdl(retention_kernel<8>, grid, 256, RtPlan<8>::FLOATS * 4, st, a);
-    else if (a.dim <= 128) launch_pdl(retention_kernel<16>, grid, 256, RtPlan<16>::FLOATS * 4, st, a);
-    else launch_pdl(retention_kernel<32>, grid, 256, RtPlan<32>::FLOATS * 4, st, a);
+    // spans of a few tokens are bound by the state's traffic, long ones by the recurrence (and a block's decay must stay in range)
+    const uint32_t n_long = a.decay_min >= 0.05f ? a.n_seq - a.first_long : 0, n_short = a.n_seq - n_long;
+    const dim3 grid((a.vdim + 31) / 32, a.n_head, n_short), grid_long((a.vdim + RS_COLS - 1) / RS_COLS, a.n_head, n_long);
+    if (n_short) {
+        if (a.dim <= 64) launch_pdl(retention_kernel<8>, grid, 256, RtPlan<8>::FLOATS * 4, st, a);
+        else if (a.dim <= 128) launch_pdl(retention_kernel<16>, grid, 256, RtPlan<16>::FLOATS * 4, st, a);
+        else launch_pdl(retention_kernel<32>, grid, 256, RtPlan<32>::FLOATS * 4, st, a);
+    }
+    if (n_long) {
+        if (a.dim <= 64) launch_pdl(retention_span_kernel<2>, grid_long, 256, 0, st, a);
+        else if (a.dim <= 128) launch_pdl(retention_span_kernel<4>, grid_long, 256, 0, st, a);
+        else launch_pdl(retention_span_kernel<8>, grid_long, 256, 0, st, a);
+    }
     const dim3 post(a.T, (a.n_head + 7) / 8);
     if (f32) launch_pdl(retention_post_kernel<float>, post, 256, 0, st, a);
     else launch_pdl(retention_post_kernel<bf16>, post, 256, 0, st, a);
-    return 3;
+    return 2 + (n_short > 0) + (n_long > 0);
 }
 
 void launch_copy_pages(void *pool, uint64_t page_bytes, const int32_t *src, const int32_t *dst, uint32_t n_pages, cudaStream_t st) {

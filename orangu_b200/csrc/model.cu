@@ -1273,7 +1273,7 @@ int forward_spans(ob_model *m, ob_kv *const *kvs, const uint32_t *tokens, const 
                 in_seq = 0;
             }
         }
-        // a step's spans are in no particular order for the graph but this: prompts after decoded tokens and short portions
+        // spans carry their rows' numbers, so they may come in any order: long portions last, the graph takes them another way
         std::stable_partition(r.spans.begin(), r.spans.end(), [](const RowSpan &sp) { return sp.n < PREFILL_SPAN; });
         const uint32_t w0 = done_want;
         while (done_want < want.size() && want[done_want] < flat) r.logit_rows.push_back(want[done_want++] - flat0);
