@@ -40,12 +40,12 @@ def run(model, kv, toks, cuts=()):
 ALONE = {
     "latent": F.config([F.latent()], ff=None, side=0),
     "latent, one head, window of one": F.config([F.latent(heads=1, window=1, dim=8, rot_dim=2, vdim=8, kv_rank=8)], ff=None, side=0),
-    "latent, window past the sequence": F.config([F.latent(window=400, dim=64, rot_dim=32, vdim=64, kv_rank=64)], ff=None, side=0),
+    "latent, window past the sequence": F.config([F.latent(window=400, dim=80, rot_dim=32, vdim=64, kv_rank=48)], ff=None, side=0),
     "latent, wide": F.config([F.latent(heads=20, window=37, dim=72, rot_dim=40, vdim=56, kv_rank=328)], ff=None, side=0),
     "latent, sizes of a large model": F.config([F.latent(heads=32, window=50, dim=128, rot_dim=64, vdim=128, kv_rank=512)], width=256, ff=None, side=0),
     "latent, beyond the tensor-core kernel": F.config([F.latent(heads=2, window=21, kv_rank=560)], ff=None, side=0),
     "retention": F.config([F.retention()], ff=None, side=0),
-    "retention, everything rotates": F.config([F.retention(heads=2, dim=64, vdim=32, rot_dims=64)], ff=None, side=0),
+    "retention, everything rotates": F.config([F.retention(heads=2, dim=72, vdim=48, rot_dims=72)], ff=None, side=0),
     "retention, 128": F.config([F.retention(heads=5, dim=112, vdim=72, rot_dims=112)], ff=None, side=0),
     "retention, 256": F.config([F.retention(heads=1, dim=250, vdim=130, rot_dims=12, decay=[0.99])], ff=None, side=0),
     "feed-forward": F.config([F.retention(heads=1, dim=2, vdim=2, rot_dims=2)], ff=250, limit=0.35, side=0),
