@@ -20,8 +20,11 @@ OBJDIR = os.path.join(LIBDIR, "obj")
 LIB = os.path.join(LIBDIR, "liborangu_b200.so")
 SYNTH_LIB = os.path.join(LIBDIR, "libob_synth.so")
 
-CU_SOURCES = ["formats.cu", "act_quant.cu", "gemv.cu", "glue.cu", "attention.cu", "api.cu", "model.cu", "tp.cu", "noalloc.cu", "stream_gemv.cu", "layer_stream.cu", "gemm_mma.cu", "gemm_tc5.cu", "gguf.cu", "sched.cu", "q5k.cu",
-              "linear.cu", "mixers.cu", "layered.cu"]
+LAYERED_LIB = os.path.join(LIBDIR, "liborangu_b200_layered.so")  # the same library without the quantized kernels
+
+CORE_SOURCES = ["api.cu", "model.cu", "tp.cu", "noalloc.cu", "gguf.cu", "sched.cu", "glue.cu", "linear.cu", "mixers.cu", "layered.cu"]
+QUANTIZED_SOURCES = ["formats.cu", "act_quant.cu", "gemv.cu", "attention.cu", "stream_gemv.cu", "layer_stream.cu", "gemm_mma.cu", "gemm_tc5.cu", "q5k.cu"]
+CU_SOURCES = CORE_SOURCES + QUANTIZED_SOURCES
 FMA_SOURCES = {"linear.cu", "mixers.cu", "layered.cu"}  # no CPU arithmetic to reproduce: the compiler may fuse
 NVCC_FLAGS = [
     "-gencode", "arch=compute_100a,code=sm_100a", "-lineinfo", "-O3", "-std=c++17",
@@ -56,12 +59,14 @@ def _headers() -> list[str]:
     return hs
 
 
-def build_cuda(force: bool = False, verbose: bool = False) -> str:
+def build_cuda(force: bool = False, verbose: bool = False, quantized: bool = True) -> str:
+    """The whole library, or (quantized=False) what models given as a list of layers need."""
+    sources, lib = (CU_SOURCES, LIB) if quantized else (CORE_SOURCES, LAYERED_LIB)
     os.makedirs(OBJDIR, exist_ok=True)
     nvcc = _nvcc()
     hdrs = _headers()
     jobs = []
-    for src in CU_SOURCES:
+    for src in sources:
         s = os.path.join(CSRC, src)
         o = os.path.join(OBJDIR, src.replace(".cu", ".o"))
         if force or _newer(o, [s] + hdrs):
@@ -83,13 +88,25 @@ def build_cuda(force: bool = False, verbose: bool = False) -> str:
             for log in ex.map(compile_one, jobs):
                 if verbose and log:
                     print(log, file=sys.stderr)
-    objs = [os.path.join(OBJDIR, s.replace(".cu", ".o")) for s in CU_SOURCES]
-    if force or jobs or _newer(LIB, objs):
-        cmd = [nvcc, "-shared", "-o", LIB, *objs, "-gencode", "arch=compute_100a,code=sm_100a", "-Xcompiler", "-fPIC", "-ldl"]
+    objs = [os.path.join(OBJDIR, s.replace(".cu", ".o")) for s in sources]
+    if force or jobs or _newer(lib, objs):
+        cmd = [nvcc, "-shared", "-o", lib, *objs, "-gencode", "arch=compute_100a,code=sm_100a", "-Xcompiler", "-fPIC", "-ldl"]
         r = subprocess.run(cmd, capture_output=True, text=True)
         if r.returncode != 0:
             raise RuntimeError(f"link failed:\n{r.stdout}\n{r.stderr}")
-    return LIB
+    return lib
+
+
+def ensure_for(model_path: str) -> str:
+    """The library a model needs, compiled if it is not there: the whole one when it is up to date or the model is quantized (a
+    .gguf file), else the one without the quantized kernels.  Makes capi load it."""
+    from . import capi
+
+    sources = [os.path.join(CSRC, s) for s in CU_SOURCES] + _headers()
+    whole = not _newer(LIB, sources)
+    lib = LIB if whole else build_cuda(quantized=not os.path.isdir(model_path))
+    capi.select(lib)
+    return lib
 
 
 def build_synth(force: bool = False) -> str:

@@ -164,6 +164,14 @@ def lib_path() -> str:
     return _LIB_PATH
 
 
+def select(path: str) -> None:
+    """Which library load() opens; before the first load()."""
+    global _LIB_PATH
+    if _lib is not None and path != _LIB_PATH:
+        raise OranguError(-1, "the library is loaded already")
+    _LIB_PATH = path
+
+
 def load():
     """The loaded library.  Raises if it has not been built: there is no fallback path."""
     global _lib

@@ -114,7 +114,7 @@ int ob_synchronize(ob_ctx *ctx) {
     if (!ctx) return OB_ERR_INVALID;
     Bind b(ctx);
     OB_CUDA(ctx, cudaStreamSynchronize(ctx->stream));
-    if (gemm_tc5_take_status()) return fail(ctx, OB_ERR_CUDA, "a tensor-core product gave up a bounded wait (pipeline barrier); its output is not valid");
+    if (quantized_built() && gemm_tc5_take_status()) return fail(ctx, OB_ERR_CUDA, "a tensor-core product gave up a bounded wait (pipeline barrier); its output is not valid");
     return OB_OK;
 }
 
@@ -126,6 +126,7 @@ namespace obrt {
 
 int make_weight(ob_ctx *ctx, const uint8_t *raw, uint64_t row_bytes, uint32_t type, uint32_t in_dim, uint32_t out_dim, uint32_t row0,
                 uint32_t n_rows, uint32_t col0, uint32_t n_cols, ob_weight **out) {
+    if (!quantized_built()) return fail(ctx, OB_ERR_UNSUPPORTED, "weight: the library was built without the quantized kernels");
     const bool raw_on_device = false;
     if (!ctx || !raw || !out) return fail(ctx, OB_ERR_INVALID, "weight: null argument");
     *out = nullptr;
@@ -318,7 +319,7 @@ int matmul_host(ob_ctx *ctx, const float *x, uint32_t n_tokens, const ob_weight 
     if (rc) return rc;
     OB_CUDA(ctx, cudaMemcpyAsync(y, ctx->sy.p, yb, cudaMemcpyDeviceToHost, ctx->stream));
     OB_CUDA(ctx, cudaStreamSynchronize(ctx->stream));
-    if (gemm_tc5_take_status()) return fail(ctx, OB_ERR_CUDA, "a tensor-core product gave up a bounded wait (pipeline barrier); its output is not valid");
+    if (quantized_built() && gemm_tc5_take_status()) return fail(ctx, OB_ERR_CUDA, "a tensor-core product gave up a bounded wait (pipeline barrier); its output is not valid");
     OB_CUDA(ctx, cudaGetLastError());
     return OB_OK;
 }
@@ -369,7 +370,7 @@ int ob_matmul_batch(ob_ctx *ctx, const ob_matmul_op *ops, uint32_t n_ops, int de
         yo += yi;
     }
     OB_CUDA(ctx, cudaStreamSynchronize(ctx->stream));
-    if (gemm_tc5_take_status()) return fail(ctx, OB_ERR_CUDA, "a tensor-core product gave up a bounded wait (pipeline barrier); its output is not valid");
+    if (quantized_built() && gemm_tc5_take_status()) return fail(ctx, OB_ERR_CUDA, "a tensor-core product gave up a bounded wait (pipeline barrier); its output is not valid");
     OB_CUDA(ctx, cudaGetLastError());
     return OB_OK;
 }
@@ -477,6 +478,7 @@ int ob_swiglu(ob_ctx *ctx, const float *gate, const float *up, uint32_t n, float
 }
 
 int ob_quantize_act(ob_ctx *ctx, const float *x, uint32_t n, int per_256, int8_t *q, float *d, int32_t *sums) {
+    if (!quantized_built()) return fail(ctx, OB_ERR_UNSUPPORTED, "quantize_act: the library was built without the quantized kernels");
     const uint32_t grp = per_256 ? 256u : 32u;
     if (!ctx || !x || !q || !d || n == 0 || n % grp) return fail(ctx, OB_ERR_INVALID, "quantize_act: bad argument");
     std::lock_guard<std::mutex> g(ctx->mu);
@@ -529,6 +531,7 @@ int ob_argmax(ob_ctx *ctx, const float *logits, uint32_t n_vocab, const uint32_t
 
 int ob_attention_decode(ob_ctx *ctx, const float *q, const float *k, const float *v, uint32_t n_pos, uint32_t n_head, uint32_t n_head_kv,
                         uint32_t head_dim, float scale, int exact_order, float *out) {
+    if (!quantized_built()) return fail(ctx, OB_ERR_UNSUPPORTED, "attention_decode: the library was built without the quantized kernels");
     if (!ctx || !q || !k || !v || !out || n_head == 0 || n_head_kv == 0 || head_dim == 0 || (head_dim & 1) || head_dim > 256)
         return fail(ctx, OB_ERR_INVALID, "attention_decode: bad argument");
     std::lock_guard<std::mutex> g(ctx->mu);

@@ -9,11 +9,15 @@
 
 namespace ob {
 
+// Launchers of the quantized kernels and of their models' attention.  A library may be built without those files (build.py,
+// components); the entry points that need them ask quantized_built() first.
+#define OB_QUANT __attribute__((weak))
+
 // ---- formats.cu
 // src_type: the GGUF type of `src`; w.type is what the device holds (TYPE_Q8_0 for the per-32 symmetric source types).
-void launch_repack(const uint8_t *src, uint64_t src_row_bytes, uint32_t src_type, uint32_t row0, uint32_t blk0, const DevWeight &w, cudaStream_t st);
-void launch_dequant_rows(const DevWeight &w, uint32_t first_row, uint32_t n_rows, float *out, cudaStream_t st);
-void launch_embed(const DevWeight &w, const uint32_t *tokens, uint32_t n_tokens, float *out, cudaStream_t st);
+OB_QUANT void launch_repack(const uint8_t *src, uint64_t src_row_bytes, uint32_t src_type, uint32_t row0, uint32_t blk0, const DevWeight &w, cudaStream_t st);
+OB_QUANT void launch_dequant_rows(const DevWeight &w, uint32_t first_row, uint32_t n_rows, float *out, cudaStream_t st);
+OB_QUANT void launch_embed(const DevWeight &w, const uint32_t *tokens, uint32_t n_tokens, float *out, cudaStream_t st);
 
 // ---- act_quant.cu
 // Writable quantized-activation buffers for up to `rows` token rows of `dim` elements.
@@ -33,7 +37,7 @@ struct QuantArgs {
     ActBuf k;             // per-256 output (q == nullptr: skip)
     ActBuf flat;          // per-32 output  (q == nullptr: skip)
 };
-void launch_quantize(int source, const QuantArgs &a, cudaStream_t st);
+OB_QUANT void launch_quantize(int source, const QuantArgs &a, cudaStream_t st);
 
 // ---- gemv.cu
 enum GemvEpilogue { EPI_STORE = 0, EPI_ADD_RESIDUAL = 1 };
@@ -54,21 +58,21 @@ struct GemvArgs {
     int32_t *isum_out;     // optional debug capture (single segment, token 0): [out_dim][nb]
     int32_t *imin_out;
 };
-void launch_gemv(const GemvArgs &a, int sm_count, cudaStream_t st);
-size_t gemv_smem_bytes(uint32_t type, uint32_t in_dim, uint32_t tile_tokens, bool gemm_order);
-uint32_t gemv_launches(uint32_t type, uint32_t in_dim, uint32_t n_tokens, bool gemm_order);  // kernels launch_gemv issues
+OB_QUANT void launch_gemv(const GemvArgs &a, int sm_count, cudaStream_t st);
+OB_QUANT size_t gemv_smem_bytes(uint32_t type, uint32_t in_dim, uint32_t tile_tokens, bool gemm_order);
+OB_QUANT uint32_t gemv_launches(uint32_t type, uint32_t in_dim, uint32_t n_tokens, bool gemm_order);  // kernels launch_gemv issues
 
 // ---- q5k.cu: Q5_K weights, one kernel for any token count and both fp32 orders
-void launch_q5k(const GemvArgs &a, int sm_count, cudaStream_t st);
+OB_QUANT void launch_q5k(const GemvArgs &a, int sm_count, cudaStream_t st);
 
 // ---- gemm_mma.cu: many-token products on the tensor cores (Q4_K and Q6_K; 9 tokens or more)
-bool gemm_mma_supported(const GemvArgs &a);
-void launch_gemm_mma(const GemvArgs &a, int sm_count, cudaStream_t st);
+OB_QUANT bool gemm_mma_supported(const GemvArgs &a);
+OB_QUANT void launch_gemm_mma(const GemvArgs &a, int sm_count, cudaStream_t st);
 
 // ---- gemm_tc5.cu: many-token products on tcgen05 tensor cores with TMEM accumulators, TMA-fed (16 tokens or more)
-bool gemm_tc5_supported(const GemvArgs &a);
-bool launch_gemm_tc5(const GemvArgs &a, int sm_count, cudaStream_t st);  // false: a tensor map could not be made (nothing was launched)
-int gemm_tc5_take_status();  // 1 when a bounded wait inside one of these kernels ran out since the last call
+OB_QUANT bool gemm_tc5_supported(const GemvArgs &a);
+OB_QUANT bool launch_gemm_tc5(const GemvArgs &a, int sm_count, cudaStream_t st);  // false: a tensor map could not be made (nothing was launched)
+OB_QUANT int gemm_tc5_take_status();  // 1 when a bounded wait inside one of these kernels ran out since the last call
 
 // ---- stream_gemv.cu: fused single-token products for decode (Q4_K / Q6_K weights)
 enum StreamPrologue { SG_PRO_PLAIN = 0, SG_PRO_RMSNORM = 1, SG_PRO_READY = 2 };
@@ -104,18 +108,18 @@ struct StreamArgs {
     obtp::PeerXchg px;
     bool wait_dependency;    // launched with programmatic stream serialisation: wait for the predecessor before reading x
 };
-bool stream_gemv_supported(const StreamArgs &a);
-void launch_stream_gemv(const StreamArgs &a, int sm_count, bool programmatic, cudaStream_t st);
-void launch_norm_scale(const float *x, uint32_t dim, float eps, float *out, bool programmatic, cudaStream_t st);
+OB_QUANT bool stream_gemv_supported(const StreamArgs &a);
+OB_QUANT void launch_stream_gemv(const StreamArgs &a, int sm_count, bool programmatic, cudaStream_t st);
+OB_QUANT void launch_norm_scale(const float *x, uint32_t dim, float eps, float *out, bool programmatic, cudaStream_t st);
 // Bytes of the quantized-activation image of one token row of `dim` elements (dim a multiple of 256).
-size_t act_image_bytes(uint32_t dim);
+OB_QUANT size_t act_image_bytes(uint32_t dim);
 // RMSNorm scale as launch_norm_scale (also stored to *scale_out), then (x * scale) * norm_w quantized per 256 into `image`.
-void launch_norm_quant(const float *x, const float *norm_w, uint32_t dim, float eps, float *scale_out, uint8_t *image, bool programmatic, cudaStream_t st);
+OB_QUANT void launch_norm_quant(const float *x, const float *norm_w, uint32_t dim, float eps, float *scale_out, uint8_t *image, bool programmatic, cudaStream_t st);
 // The same, but first the pending peer exchange is completed: x += the ranks' partials, added in rank order (x is written).
-void launch_norm_quant_consume(float *x, const float *norm_w, uint32_t dim, float eps, float *scale_out, uint8_t *image, const obtp::PeerXchg &px,
+OB_QUANT void launch_norm_quant_consume(float *x, const float *norm_w, uint32_t dim, float eps, float *scale_out, uint8_t *image, const obtp::PeerXchg &px,
                                bool programmatic, cudaStream_t st);
 // x quantized per 256 into `image`.
-void launch_quant_image(const float *x, uint32_t dim, uint8_t *image, bool programmatic, cudaStream_t st);
+OB_QUANT void launch_quant_image(const float *x, uint32_t dim, uint8_t *image, bool programmatic, cudaStream_t st);
 
 // ---- layer_stream.cu: the single-token products between two attention kernels as phases of one persistent launch
 struct alignas(16) LsPhase {
@@ -135,11 +139,11 @@ struct LsLayout {  // byte offsets inside the kernel's dynamic shared memory
     uint32_t off_ring;   // per-warp two-slot weight ring
     uint32_t total;
 };
-bool layer_stream_phase(const StreamArgs &a, LsPhase *out);              // false: the shape does not take this kernel
-LsLayout layer_stream_layout(const LsPhase *phases, uint32_t n);         // host copy of the phases
-bool layer_stream_fits(const LsLayout &L);
+OB_QUANT bool layer_stream_phase(const StreamArgs &a, LsPhase *out);              // false: the shape does not take this kernel
+OB_QUANT LsLayout layer_stream_layout(const LsPhase *phases, uint32_t n);         // host copy of the phases
+OB_QUANT bool layer_stream_fits(const LsLayout &L);
 // barrier: one zeroed word per launch; status: set to 1 when a barrier wait gave up after timeout_ms
-bool launch_layer_stream(const LsPhase *dev_phases, uint32_t n, const LsLayout &L, int sm_count, uint32_t *barrier, uint32_t *status, uint32_t timeout_ms,
+OB_QUANT bool launch_layer_stream(const LsPhase *dev_phases, uint32_t n, const LsLayout &L, int sm_count, uint32_t *barrier, uint32_t *status, uint32_t timeout_ms,
                          bool programmatic, cudaStream_t st);
 
 // ---- glue.cu
@@ -202,14 +206,14 @@ struct AttnDecodeArgs {
     uint8_t *image;            // optional, n_seq == 1: the output quantized per 256 for the product that follows (stream_gemv.cu)
     bool small_ctas;           // many (row, kv head) pairs: CTAs of four warps, two per SM
 };
-void launch_attn_decode(const AttnDecodeArgs &a, cudaStream_t st);
+OB_QUANT void launch_attn_decode(const AttnDecodeArgs &a, cudaStream_t st);
 // One kernel: every warp streams its own pages, the CTAs of a (sequence, kv head) leave partials and the last of them to
 // finish merges them (and quantizes the result when `image` is set).  False when the shape is not covered.
-bool launch_attn_decode_fused(const AttnDecodeArgs &a, bool programmatic, cudaStream_t st);
+OB_QUANT bool launch_attn_decode_fused(const AttnDecodeArgs &a, bool programmatic, cudaStream_t st);
 
 // The rows (n_seq of them) are consecutive tokens of ONE sequence: tiled tensor-core attention, 16 tokens x the query heads of a kv
 // head per CTA, K/V of the window read once per 16 tokens.  Needs no partial buffers.  False when the shape is not covered.
-bool launch_attn_prefill(const AttnDecodeArgs &a, cudaStream_t st);
+OB_QUANT bool launch_attn_prefill(const AttnDecodeArgs &a, cudaStream_t st);
 
 // Exact-order attention (three kernels: scores, softmax, output); see attention.cu.
 struct AttnExactArgs {
@@ -225,6 +229,8 @@ struct AttnExactArgs {
     float scale;
     uint32_t max_pos;          // upper bound of n_pos over the rows (sizes the score grid)
 };
-void launch_attn_exact(const AttnExactArgs &a, cudaStream_t st);
-bool attn_exact_supported(uint32_t n_head, uint32_t n_head_kv, uint32_t head_dim);
+OB_QUANT void launch_attn_exact(const AttnExactArgs &a, cudaStream_t st);
+OB_QUANT bool attn_exact_supported(uint32_t n_head, uint32_t n_head_kv, uint32_t head_dim);
+
+inline bool quantized_built() { return launch_gemv != nullptr; }
 }  // namespace ob

@@ -675,6 +675,7 @@ void ob_model_destroy(ob_model *m) {
 }
 
 int ob_model_create(ob_ctx *ctx, const ob_model_desc *desc, ob_model **out) {
+    if (!quantized_built()) return fail(ctx, OB_ERR_UNSUPPORTED, "model_create: the library was built without the quantized kernels");
     if (!ctx || !desc || !out) return fail(ctx, OB_ERR_INVALID, "model_create: null argument");
     *out = nullptr;
     const ob_model_desc &c = *desc;
@@ -1453,7 +1454,7 @@ int pre_step(ob_model *m) {
 }
 
 int check_peer(ob_model *m) {
-    if (gemm_tc5_take_status()) return fail(m->ctx, OB_ERR_CUDA, "a tensor-core product gave up a bounded wait (pipeline barrier); the step's output is not valid");
+    if (quantized_built() && gemm_tc5_take_status()) return fail(m->ctx, OB_ERR_CUDA, "a tensor-core product gave up a bounded wait (pipeline barrier); the step's output is not valid");
     if (m->graph && m->graph->take_failure()) return fail(m->ctx, OB_ERR_CUDA, "a product of the step could not be launched");
     if (m->graph && linear_take_status()) return fail(m->ctx, OB_ERR_CUDA, "a tensor-core product gave up a bounded wait (pipeline barrier); the step's output is not valid");
     if (m->launch_failed) {
@@ -1631,6 +1632,7 @@ __global__ void selftest_deliver_kernel(uint2 *slot, uint32_t n, float value, ui
 }  // namespace
 
 int ob_tp_exchange_selftest(ob_ctx *ctx, uint32_t n, uint32_t timeout_ms, uint32_t n_rounds, const uint8_t *peer_delivers, float *sums_out) {
+    if (!quantized_built()) return fail(ctx, OB_ERR_UNSUPPORTED, "tp_exchange_selftest: the library was built without the quantized kernels");
     if (!ctx || !peer_delivers || n == 0 || n % 256 || n_rounds == 0 || n_rounds > 64) return fail(ctx, OB_ERR_INVALID, "tp_exchange_selftest: bad argument");
     std::lock_guard<std::mutex> g(ctx->mu);
     Bind b(ctx);

@@ -51,6 +51,7 @@ __global__ void static_meta_kernel(unsigned char *scratch, const int32_t *table,
 extern "C" int ob_attention_decode_static(ob_ctx *ctx, const float *q_dev, const void *k_pages_dev, const void *v_pages_dev,
                                           const int32_t *page_table_dev, uint32_t n_pos, uint32_t n_head, uint32_t n_head_kv,
                                           uint32_t head_dim, float scale, float *out_dev, void *stream) {
+    if (!quantized_built()) return fail(ctx, OB_ERR_UNSUPPORTED, "attention_decode_static: the library was built without the quantized kernels");
     if (!ctx || !q_dev || !k_pages_dev || !v_pages_dev || !page_table_dev || !out_dev)
         return fail(ctx, OB_ERR_INVALID, "attention_decode_static: null argument");
     if (n_pos == 0 || n_head == 0 || n_head_kv == 0 || n_head % n_head_kv || (head_dim != 64 && head_dim != 128))

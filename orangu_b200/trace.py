@@ -67,9 +67,10 @@ def main(argv=None) -> int:
     ap.add_argument("--max-tokens", type=int, required=True, help="most tokens live requests hold at any time")
     a = ap.parse_args(argv)
 
-    from . import CudaBackend
+    from . import CudaBackend, build
     from .registry import load_model
 
+    build.ensure_for(a.model)
     tokens = -(-a.max_tokens // REQUEST_ROUNDING) * REQUEST_ROUNDING
     model = load_model(CudaBackend.init(0), a.model, dtype=a.dtype, max_seq_len=tokens, max_batch_tokens=min(tokens, MAX_STEP_ROWS),
                        kv_pool_tokens=tokens, state_slots=SLOTS)

@@ -112,6 +112,23 @@ def test_command_lines_explain_themselves():
         assert r.returncode == 0 and "--model" in r.stdout
 
 
+def test_library_without_the_quantized_kernels(tmp_path):
+    """The part a layered model needs links, loads and exports everything; what is left out answers with a status."""
+    import subprocess, sys
+
+    from orangu_b200 import build
+
+    root = os.path.dirname(os.path.dirname(os.path.abspath(__file__)))
+    lib = build.build_cuda(quantized=False)
+    code = ("import ctypes as C, sys\nfrom orangu_b200 import capi\ncapi.select(sys.argv[1])\nL = capi.load()\n"
+            "d, h = capi.ModelDesc(), C.c_void_p()\n"
+            "assert L.ob_model_create(None, C.byref(d), C.byref(h)) == -2 and b'without the quantized' in L.ob_last_error(None)\n"
+            "assert L.ob_layered_model_create(None, None, C.byref(h)) == -1 and L.ob_quantize_act(None, None, 1, 0, None, None, None) == -2\n"
+            "print(capi.lib_path())")
+    r = subprocess.run([sys.executable, "-c", code, lib], cwd=root, capture_output=True, text=True)
+    assert r.returncode == 0 and r.stdout.strip() == lib, r.stderr
+
+
 # ---- the plain statement itself
 def test_plain_retention_equals_its_unrolled_sum():
     cfg = F.config([F.retention(heads=2, dim=8, vdim=6, rot_dims=4)], width=16, ff=None, side=0)
