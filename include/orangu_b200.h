@@ -30,8 +30,9 @@ extern "C" {
 #endif
 
 /* 2: ob_model_desc gained rope_freqs (layout change); the GGUF, static-attention and KV-copy entry points were added.
- * 3: ob_model_desc gained tp_presliced. */
-#define OB_ABI_VERSION 4u
+ * 3: ob_model_desc gained tp_presliced.
+ * 5: the layered descriptions gained softmax attention over cached keys and values, sequential blocks and mixtures of experts. */
+#define OB_ABI_VERSION 5u
 
 typedef enum ob_status {
     OB_OK = 0,
@@ -250,13 +251,18 @@ typedef struct ob_model_desc {
 } ob_model_desc;
 
 /* ------------------------------------------------- models given as a list of layers
- * Designs whose layers are not all alike: every layer names its token mixer and carries that mixer's sizes, constants and
- * tensors; mixer and feed-forward read the same normed input (parallel layers, x += mixer(h) + ff(h), h = norm(x) with one
- * number as gain).  No counterpart in the reference.  The result is an ob_model like any other: caches, batching, sampling,
+ * Designs whose layers are not all alike: every layer names its token mixer and its feed-forward and carries their sizes,
+ * constants and tensors.  Two kinds of block: parallel, x += mixer(h) + ff(h) with h = x / rms(x) * norm_gain; and sequential with
+ * normed outputs (post_norm1 given), x += residual_mult * mixer(x) / rms(mixer(x)) * post_norm1, then the same with the
+ * feed-forward and post_norm2.  No counterpart in the reference.  The result is an ob_model like any other: caches, batching, sampling,
  * captured decode graphs and the slot pool are the same calls.  Matrices are bfloat16, out_dim rows of in_dim; vectors f32. */
 #define OB_TYPE_BF16 30u /* ob_matrix_desc.ggml_type of these matrices */
 #define OB_MIXER_LATENT_ATTENTION 1u
 #define OB_MIXER_RETENTION 2u
+#define OB_MIXER_ATTENTION 3u /* softmax attention over cached keys and values, n_head / n_kv_head query heads per key/value head */
+#define OB_FF_CLAMPED_GLU 0u /* g = min(gate, limit), u = clamp(up, -limit, limit); g * sigmoid(alpha g) * (u + 1) */
+#define OB_FF_RELU2 1u       /* max(up, 0)^2 */
+#define OB_FF_EXPERTS 2u     /* n_expert_used of n_expert silu(gate) * up feed-forwards; a chosen one reads the input times its score */
 
 typedef struct ob_mixer_desc {
     uint32_t kind;            /* OB_MIXER_* */
@@ -264,29 +270,43 @@ typedef struct ob_mixer_desc {
     uint32_t vdim;            /* value dimensions per head */
     uint32_t rot_dim;         /* latent attention: rotated query/key dimensions per head, in addition to dim */
     uint32_t kv_rank;         /* latent attention: size of the cached latent */
-    uint32_t window;          /* latent attention: a position sees itself and window - 1 before it; 0 = all before it */
-    uint32_t rot_dims;        /* entries that rotate, from the first: of q and k (retention), of the rot_dim part (latent attention) */
+    uint32_t window;          /* attention: a position sees itself and window - 1 before it; 0 = all before it */
+    uint32_t rot_dims;        /* entries that rotate, from the first: of q and k (retention, attention), of the rot_dim part (latent attention) */
     uint32_t rot_interleaved; /* 1: pairs (2i, 2i+1); 0: pairs (i, i + rot_dims/2) */
-    float scale;              /* latent attention: factor of the scores */
+    float scale;              /* attention: factor of the scores */
     double rot_base;          /* pair i turns by position * rot_base^(-2i / rot_dims) */
     const float *decay;       /* retention: [n_head] factor of the state per token */
-    ob_matrix_desc wq;        /* retention [n_head*dim]; latent attention [n_head*(dim+rot_dim)], per head unrotated then rotated */
-    ob_matrix_desc wk, wv;    /* retention [n_head*dim], [n_head*vdim] */
-    ob_matrix_desc w_gate;    /* retention [n_head*vdim] (silu of it scales the normed output); latent attention [n_head] (sigmoid of it scales a head) */
+    ob_matrix_desc wq;        /* retention [n_head*dim]; latent attention [n_head*(dim+rot_dim)], per head unrotated then rotated;
+                               * attention [n_head*n_map*dim], head by head */
+    ob_matrix_desc wk, wv;    /* retention [n_head*dim], [n_head*vdim]; attention [n_kv_head*n_map*dim], [n_kv_head*vdim] (no data:
+                               * the values are the keys as projected, before norm and rotation; n_map 1, vdim = dim) */
+    ob_matrix_desc w_gate;    /* retention [n_head*vdim] (silu of it scales the normed output); latent attention [n_head] (sigmoid of it scales a head);
+                               * attention [n_head*vdim] (sigmoid of it scales the output; no data: no gate) */
     ob_matrix_desc w_dkv;     /* latent attention [kv_rank+rot_dim]: latent, then the rotated key part all heads share */
     const float *kv_norm;     /* latent attention [kv_rank]: RMS-norm weight of the latent */
     ob_matrix_desc w_uk, w_uv; /* latent attention [n_head*dim], [n_head*vdim] from kv_rank */
     ob_matrix_desc wo;        /* [n_head*vdim -> n_embd] */
+    uint32_t n_kv_head;       /* attention: divides n_head */
+    uint32_t n_map;           /* attention: softmax maps per head over the same values, 1 or 2 */
+    float map_weight;         /* attention with two maps: o = map 1 - map_weight * map 2, then o / rms(o) * head_gain per head */
+    float head_gain;
+    const float *q_norm, *k_norm; /* attention [dim]: RMS-norm weights of every query and key vector before rotation */
+    const float *q_bias, *k_bias, *v_bias, *o_bias; /* attention: added in the projections; NULL: none */
 } ob_mixer_desc;
 
 typedef struct ob_block_desc {
-    float norm_gain;
+    float norm_gain;          /* parallel blocks */
     ob_mixer_desc mixer;
-    uint32_t n_ff;            /* 0: no feed-forward */
-    float glu_limit, glu_alpha; /* g = min(gate, limit), u = clamp(up, -limit, limit); g * sigmoid(alpha g) * (u + 1) */
-    ob_matrix_desc w_gate, w_up, w_down;
+    uint32_t n_ff;            /* of one expert when there are experts; 0: no feed-forward */
+    float glu_limit, glu_alpha; /* OB_FF_CLAMPED_GLU */
+    ob_matrix_desc w_gate, w_up, w_down; /* gate: OB_FF_CLAMPED_GLU only; none with experts */
     ob_matrix_desc side_gate, side_proj; /* per-layer token input (side_dim > 0): y = side_proj (gelu_tanh(side_gate x) * e), x += y / rms(y) * side_norm */
     const float *side_norm;   /* [n_embd] */
+    const float *post_norm1, *post_norm2; /* [n_embd] factors of the normed outputs; post_norm1 makes the block sequential */
+    uint32_t ff_kind;         /* OB_FF_*; parallel blocks have the first kind, sequential ones the others */
+    uint32_t n_expert, n_expert_used; /* OB_FF_EXPERTS: the n_expert_used largest of sigmoid(w_router x) are chosen, scores as they are */
+    ob_matrix_desc w_router;  /* [n_expert] */
+    const ob_matrix_desc *expert_gate, *expert_up, *expert_down; /* [n_expert] matrices each */
 } ob_block_desc;
 
 typedef struct ob_layered_desc {
@@ -301,6 +321,8 @@ typedef struct ob_layered_desc {
     ob_matrix_desc side_embd;  /* [n_vocab][n_layer * side_dim] */
     ob_matrix_desc output;     /* [n_vocab] */
     const ob_block_desc *layers;
+    float residual_mult;       /* sequential blocks */
+    const float *final_norm;   /* [n_embd] factors of the last norm, beside final_gain; NULL: none.  All blocks are of one kind */
 } ob_layered_desc;
 
 /* ------------------------------------------------- GGUF files

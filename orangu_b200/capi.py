@@ -38,24 +38,29 @@ class ModelDesc(C.Structure):
 
 
 TYPE_BF16 = 30
-MIXER_LATENT_ATTENTION, MIXER_RETENTION = 1, 2
+MIXER_LATENT_ATTENTION, MIXER_RETENTION, MIXER_ATTENTION = 1, 2, 3
+FF_CLAMPED_GLU, FF_RELU2, FF_EXPERTS = 0, 1, 2
 
 
 class MixerDesc(C.Structure):
     _fields_ = [(n, C.c_uint32) for n in ("kind", "n_head", "dim", "vdim", "rot_dim", "kv_rank", "window", "rot_dims", "rot_interleaved")] + [
         ("scale", C.c_float), ("rot_base", C.c_double), ("decay", C.c_void_p)] + [
-        (n, MatrixDesc) for n in ("wq", "wk", "wv", "w_gate", "w_dkv")] + [("kv_norm", C.c_void_p)] + [(n, MatrixDesc) for n in ("w_uk", "w_uv", "wo")]
+        (n, MatrixDesc) for n in ("wq", "wk", "wv", "w_gate", "w_dkv")] + [("kv_norm", C.c_void_p)] + [(n, MatrixDesc) for n in ("w_uk", "w_uv", "wo")] + [
+        ("n_kv_head", C.c_uint32), ("n_map", C.c_uint32), ("map_weight", C.c_float), ("head_gain", C.c_float)] + [
+        (n, C.c_void_p) for n in ("q_norm", "k_norm", "q_bias", "k_bias", "v_bias", "o_bias")]
 
 
 class BlockDesc(C.Structure):
     _fields_ = [("norm_gain", C.c_float), ("mixer", MixerDesc), ("n_ff", C.c_uint32), ("glu_limit", C.c_float), ("glu_alpha", C.c_float)] + [
-        (n, MatrixDesc) for n in ("w_gate", "w_up", "w_down", "side_gate", "side_proj")] + [("side_norm", C.c_void_p)]
+        (n, MatrixDesc) for n in ("w_gate", "w_up", "w_down", "side_gate", "side_proj")] + [("side_norm", C.c_void_p)] + [
+        (n, C.c_void_p) for n in ("post_norm1", "post_norm2")] + [(n, C.c_uint32) for n in ("ff_kind", "n_expert", "n_expert_used")] + [
+        ("w_router", MatrixDesc)] + [(n, C.POINTER(MatrixDesc)) for n in ("expert_gate", "expert_up", "expert_down")]
 
 
 class LayeredDesc(C.Structure):
     _fields_ = [(n, C.c_uint32) for n in ("n_vocab", "n_embd", "n_layer", "side_dim")] + [("rms_eps", C.c_float), ("final_gain", C.c_float)] + [
         (n, C.c_uint32) for n in ("compute_f32", "max_seq_len", "max_batch_tokens")] + [("kv_pool_tokens", C.c_uint64), ("n_state_slots", C.c_uint32)] + [
-        (n, MatrixDesc) for n in ("token_embd", "side_embd", "output")] + [("layers", C.POINTER(BlockDesc))]
+        (n, MatrixDesc) for n in ("token_embd", "side_embd", "output")] + [("layers", C.POINTER(BlockDesc)), ("residual_mult", C.c_float), ("final_norm", C.c_void_p)]
 
 
 class MatmulOpC(C.Structure):

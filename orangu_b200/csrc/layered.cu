@@ -1,7 +1,7 @@
-// Models given as a list of layers (ob_layered_desc): weights as padded bfloat16 matrices, a latent-cache pool per
-// latent-attention layer on the model's pages, a state pool per recurrent layer on the model's slots, and the step.
+// Models given as a list of layers (ob_layered_desc): weights as padded bfloat16 matrices, a cache pool per attention layer (latents,
+// or keys and values) on the model's pages, a state pool per recurrent layer on the model's slots, and the step.
 //
-// A layer is a short chain of launches.  All products that read the normed input are one matrix, its feed-forward rows
+// A layer is a short chain of launches.  In a parallel block all products that read the normed input are one matrix, its feed-forward rows
 // interleaved (gate, up) so that the activation is the epilogue; the mixer's output and the feed-forward's activations sit side
 // by side in one row, so the two output products and the residual addition are one product too.
 //   in      [mixer projections | gate/up]  <- h
@@ -9,6 +9,10 @@
 //           retention: rotate, recurrence, norm with gate
 //   out     x += [W_o | W_down] [mixer | ff]
 //   side    gate (gelu, token entry), proj, then norm + residual + the next layer's norm in one kernel
+// A sequential block reads the residual itself (h: its activation form) and norms what it adds:
+//   in      mixer projections <- h; mixer (attention: prep, attention with the heads' epilogue); out product, bias as epilogue
+//   post    x += mult norm(out), h = x in one kernel
+//   ff      dense: up (activation as epilogue), down; experts: routing, grouped gate/up and down (moe.cu); post as above
 #include <math.h>
 #include <string.h>
 
@@ -19,6 +23,8 @@
 #include "model.h"
 
 namespace {
+
+constexpr uint32_t MOE_ROWS_IN_ORDER = 8;  // so many (token, expert) pairs run row by row, more are grouped by expert
 
 constexpr uint32_t round_up(uint32_t v, uint32_t m) { return (v + m - 1) / m * m; }
 
@@ -32,6 +38,14 @@ struct LayerPlan {
     float norm_gain = 0.0f, glu_limit = 0.0f, glu_alpha = 0.0f;
     uint32_t n_ff = 0;
     Dense in, out, side_gate, side_proj;
+    bool sequential = false;
+    float *in_bias = nullptr, *out_bias = nullptr, *post1 = nullptr, *post2 = nullptr;
+    uint32_t ff_kind = 0, n_expert = 0, top = 1;
+    Dense up, down, router;  // feed-forward of a sequential block, one after the other for every expert (gate and up rows interleaved)
+    // attention: rows of `in` are [activations (values, gates) | f32 projections (queries, keys)]
+    float *q_norm = nullptr, *k_norm = nullptr;
+    uint32_t vdim_p = 0, row = 0, gate0 = 0;  // row: elements of a cache row per key/value head
+    bool has_v = false, has_gate = false;
     float *side_norm = nullptr;
     Rot rot{};
     // rows of `in`: [activations (unrotated queries) | f32 projections | gate/up]
@@ -61,7 +75,8 @@ struct LayeredGraph : StepGraph {
     ob_model *m = nullptr;
     bool f32 = false, has_state = false;
     uint32_t width = 0, h_pitch = 0, side_dim = 0, side_p = 0, y_pitch = 0, cat_pitch = 0;
-    float eps = 0.0f, final_gain = 0.0f;
+    float eps = 0.0f, final_gain = 0.0f, residual_mult = 1.0f;
+    float *final_norm = nullptr;
     std::vector<LayerPlan> L;
     __nv_bfloat16 *embd = nullptr, *side_embd = nullptr;
     Dense output;
@@ -69,6 +84,10 @@ struct LayeredGraph : StepGraph {
     float *y = nullptr, *o_ret = nullptr, *sy = nullptr, *part = nullptr;
     void *lat = nullptr, *expanded = nullptr;  // gathered latents of prompts, their keys and values: key_cap rows
     uint32_t key_cap = 0;
+    void *ffa = nullptr;      // feed-forward activations of sequential blocks, a row per token or (token, expert) pair
+    float *yo = nullptr;      // their outputs, and the mixers'
+    MoeArgs moe{};            // routing buffers
+    float *router_logits = nullptr;
     uint64_t part_cap = 0;
     float *split_part = nullptr;
     bool failed = false;  // a product could not be launched
@@ -106,6 +125,11 @@ struct LayeredGraph : StepGraph {
     void head(const uint32_t *d_rows, uint32_t n, cudaStream_t st) override;
     void latent(const LayerPlan &P, uint32_t T, uint32_t n_seq, const RowSpan *spans, bool single, uint32_t max_pos, cudaStream_t st);
     void retention(const LayerPlan &P, uint32_t T, uint32_t n_seq, const RowSpan *spans, cudaStream_t st);
+    void attention(const LayerPlan &P, uint32_t T, uint32_t n_seq, const RowSpan *spans, bool single, uint32_t max_pos, cudaStream_t st);
+    void mixer(const LayerPlan &P, uint32_t T, uint32_t n_seq, const RowSpan *spans, bool single, uint32_t max_pos, cudaStream_t st);
+    void sequential(const LayerPlan &P, bool last, uint32_t T, uint32_t n_seq, const RowSpan *spans, bool single, uint32_t max_pos, cudaStream_t st);
+    void post(const float *w, uint32_t T, bool last, uint32_t top, const uint32_t *rows, uint32_t n_zero, cudaStream_t st);
+    uint32_t cache_elems(const LayerPlan &P) const { return P.mx.kind == OB_MIXER_ATTENTION ? P.mx.n_kv_head * P.row : P.dq; }  // per position
     int copy_prefix(ob_kv *dst, const ob_kv *src, uint32_t n) override;
     int read_pages(const ob_kv *kv, uint32_t layer, uint32_t pos0, uint32_t n, float *k_out, float *v_out) override;
     int read_state(const ob_kv *kv, uint32_t layer, float *out) override;
@@ -135,6 +159,13 @@ struct LayeredGraph : StepGraph {
     }
     int build(const ob_layered_desc &c);
     int build_layer(const ob_block_desc &b, LayerPlan &P);
+    int build_ff(const ob_block_desc &b, LayerPlan &P);
+    int upload_now(const float *src, size_t n, float **out) {  // the source may end with the caller
+        int rc = dev_alloc(m, out, n);
+        if (rc) return rc;
+        OB_CUDA(m->ctx, cudaMemcpy(*out, src, n * 4, cudaMemcpyHostToDevice));
+        return OB_OK;
+    }
 };
 
 // Spans of a step come with the long ones last (forward_spans).
@@ -263,34 +294,174 @@ void LayeredGraph::retention(const LayerPlan &P, uint32_t T, uint32_t n_seq, con
     m->ctx->launches += launch_retention(a, f32, m->ctx->sm_count, st);
 }
 
+void LayeredGraph::attention(const LayerPlan &P, uint32_t T, uint32_t n_seq, const RowSpan *spans, bool single, uint32_t max_pos, cudaStream_t st) {
+    const MetaLayout ml(m->T);
+    AttentionArgs a{};
+    a.y = y;
+    a.y_pitch = y_pitch;
+    a.va = qn;
+    a.va_pitch = P.act_rows;
+    a.gate0 = P.gate0;
+    a.has_v = P.has_v;
+    a.has_gate = P.has_gate;
+    a.n_head = P.mx.n_head;
+    a.n_kv = P.mx.n_kv_head;
+    a.n_map = P.mx.n_map;
+    a.dim = P.mx.dim;
+    a.vdim = P.mx.vdim;
+    a.window = P.mx.window;
+    a.dim_p = P.dim_p;
+    a.vdim_p = P.vdim_p;
+    a.row = P.row;
+    a.eps = eps;
+    a.scale = P.mx.scale;
+    a.map_weight = P.mx.map_weight;
+    a.head_gain = P.mx.head_gain;
+    a.q_norm = P.q_norm;
+    a.k_norm = P.k_norm;
+    a.rot = P.rot;
+    a.q = q;
+    a.cache = P.pool;
+    a.out = cat;
+    a.out_pitch = cat_pitch;
+    a.T = T;
+    a.n_seq = n_seq;
+    a.n_short = first_long(spans, n_seq);
+    a.spans = reinterpret_cast<const RowSpan *>(m->d_meta + ml.off_spans);
+    a.h_spans = spans;
+    a.single = single;
+    a.positions = reinterpret_cast<const uint32_t *>(m->d_meta + ml.off_positions);
+    a.tables = reinterpret_cast<const int32_t *const *>(m->d_meta + ml.off_tables);
+    a.max_pos = max_pos;
+    launch_attention_prep(a, f32, st);
+    m->ctx->launches += 1 + launch_attention(a, f32, m->ctx->sm_count, st);
+}
+
+void LayeredGraph::mixer(const LayerPlan &P, uint32_t T, uint32_t n_seq, const RowSpan *spans, bool single, uint32_t max_pos, cudaStream_t st) {
+    if (P.mx.kind == OB_MIXER_LATENT_ATTENTION) latent(P, T, n_seq, spans, single, max_pos, st);
+    else if (P.mx.kind == OB_MIXER_ATTENTION) attention(P, T, n_seq, spans, single, max_pos, st);
+    else retention(P, T, n_seq, spans, st);
+}
+
+void LayeredGraph::post(const float *w, uint32_t T, bool last, uint32_t top, const uint32_t *rows, uint32_t n_zero, cudaStream_t st) {
+    PostNormArgs p{};
+    p.x = m->x;
+    p.y = yo;
+    p.rows = rows;
+    p.top = top;
+    p.w = w;
+    p.width = width;
+    p.T = T;
+    p.eps = eps;
+    p.mult = residual_mult;
+    p.h = last ? nullptr : h;
+    p.h_pitch = h_pitch;
+    p.zero = n_zero ? moe.count : nullptr;
+    p.n_zero = n_zero;
+    launch_post_norm(p, f32, st);
+    m->ctx->launches++;
+}
+
+void LayeredGraph::sequential(const LayerPlan &P, bool last, uint32_t T, uint32_t n_seq, const RowSpan *spans, bool single, uint32_t max_pos, cudaStream_t st) {
+    LinArgs in = product(P.in, h, h_pitch, T);
+    in.bias = P.in_bias;
+    segment(in, 0, P.act_rows, LE_ACT, qn, P.act_rows);
+    segment(in, P.f32_row0, P.f32_rows, LE_F32, y, y_pitch);
+    linear(in, st);
+    mixer(P, T, n_seq, spans, single, max_pos, st);
+    LinArgs out = product(P.out, cat, cat_pitch, T);
+    out.bias = P.out_bias;
+    segment(out, 0, width, LE_F32, yo, width);
+    linear(out, st);
+    post(P.post1, T, last && !P.n_ff, 1, nullptr, 0, st);
+    if (!P.n_ff) return;
+    if (P.ff_kind != OB_FF_EXPERTS) {
+        LinArgs up = product(P.up, h, h_pitch, T);
+        segment(up, 0, P.n_ff, LE_RELU2, ffa, P.down.kp);
+        linear(up, st);
+        LinArgs down = product(P.down, ffa, P.down.kp, T);
+        segment(down, 0, width, LE_F32, yo, width);
+        linear(down, st);
+        post(P.post2, T, last, 1, nullptr, 0, st);
+        return;
+    }
+    const uint32_t R = T * P.top;
+    const bool in_order = R <= MOE_ROWS_IN_ORDER;
+    MoeArgs r = moe;
+    r.x = h;
+    r.x_pitch = h_pitch;
+    r.w = P.router.w;
+    r.n_expert = P.n_expert;
+    r.top = P.top;
+    r.T = T;
+    r.tile_rows = linear_tile_rows(R, P.n_expert, f32);
+    if (in_order) r.count = nullptr;
+    if (T > MOE_DOT_TOKENS) {
+        LinArgs z = product(P.router, h, h_pitch, T);
+        segment(z, 0, P.n_expert, LE_F32, router_logits, P.n_expert);
+        linear(z, st);
+        r.logits = router_logits;
+        r.logit_pitch = P.n_expert;
+    }
+    m->ctx->launches += launch_moe_route(r, f32, st);
+    auto grouped = [&](const Dense &w, const void *x, uint32_t x_div) {
+        LinArgs a = product(w, x, w.kp, R);
+        a.n_rows = w.rows / P.n_expert;
+        a.n_batch = P.n_expert;
+        if (in_order) {
+            a.row_batch = r.expert;
+            a.x_div = x_div;
+        } else {
+            a.tiles = r.tiles;
+            a.n_tiles = r.n_tiles;
+            a.tile_rows = r.tile_rows;
+            a.max_tiles = R / r.tile_rows + std::min(R, P.n_expert);
+        }
+        return a;
+    };
+    LinArgs up = grouped(P.up, in_order ? h : r.gathered, P.top);
+    up.row_scale = in_order ? r.score : r.row_score;
+    segment(up, 0, 2 * P.n_ff, LE_SWIGLU, ffa, P.down.kp);
+    linear(up, st);
+    LinArgs down = grouped(P.down, ffa, 1);
+    segment(down, 0, width, LE_F32, yo, width);
+    linear(down, st);
+    post(P.post2, T, last, P.top, in_order ? nullptr : r.row, in_order ? 0 : P.n_expert, st);
+}
+
 void LayeredGraph::layers(uint32_t T, uint32_t n_seq, const RowSpan *spans, uint32_t max_pos, cudaStream_t st) {
     const MetaLayout ml(m->T);
     const uint32_t *tokens = reinterpret_cast<const uint32_t *>(m->d_meta + ml.off_tokens);
     const bool single = n_seq == T;
-    launch_embed_norm(embd, width, tokens, T, m->x, eps, L[0].norm_gain, h, h_pitch, f32, st);
+    launch_embed(embd, width, tokens, T, m->x, !L[0].sequential, eps, L[0].norm_gain, h, h_pitch, f32, st);
     m->ctx->launches++;
     for (size_t li = 0; li < L.size(); ++li) {
         const LayerPlan &P = L[li];
+        const bool last = li + 1 == L.size();
+        if (P.sequential) {
+            sequential(P, last, T, n_seq, spans, single, max_pos, st);
+            continue;
+        }
         LinArgs in = product(P.in, h, h_pitch, T);
         segment(in, 0, P.act_rows, LE_ACT, qn, P.act_rows);
         segment(in, P.f32_row0, P.f32_rows, LE_F32, y, y_pitch);
+        in.bias = P.in_bias;
         segment(in, P.glu_row0, 2 * P.n_ff, LE_GLU, cat, cat_pitch, P.mix_cols);
         in.glu_limit = P.glu_limit;
         in.glu_alpha = P.glu_alpha;
         linear(in, st);
 
-        if (P.mx.kind == OB_MIXER_LATENT_ATTENTION) latent(P, T, n_seq, spans, single, max_pos, st);
-        else retention(P, T, n_seq, spans, st);
+        mixer(P, T, n_seq, spans, single, max_pos, st);
 
         LinArgs out = product(P.out, cat, cat_pitch, T);
         segment(out, 0, width, LE_RESIDUAL, m->x, width);
+        out.bias = P.out_bias;
         if (side_dim) {
             out.out2 = xb;
             out.out2_pitch = h_pitch;
         }
         linear(out, st);
 
-        const bool last = li + 1 == L.size();
         const float gain = last ? 0.0f : L[li + 1].norm_gain;
         if (side_dim) {
             LinArgs g = product(P.side_gate, xb, h_pitch, T);
@@ -306,14 +477,14 @@ void LayeredGraph::layers(uint32_t T, uint32_t n_seq, const RowSpan *spans, uint
             launch_side_finish(m->x, sy, P.side_norm, width, T, eps, gain, last ? nullptr : h, h_pitch, f32, st);
             m->ctx->launches++;
         } else if (!last) {
-            launch_norm_scalar(m->x, width, nullptr, T, eps, gain, h, h_pitch, f32, st);
+            launch_norm(m->x, width, nullptr, T, eps, gain, nullptr, h, h_pitch, f32, st);
             m->ctx->launches++;
         }
     }
 }
 
 void LayeredGraph::head(const uint32_t *d_rows, uint32_t n, cudaStream_t st) {
-    launch_norm_scalar(m->x, width, d_rows, n, eps, final_gain, h, h_pitch, f32, st);
+    launch_norm(m->x, width, d_rows, n, eps, final_gain, final_norm, h, h_pitch, f32, st);
     m->ctx->launches++;
     LinArgs a = product(output, h, h_pitch, n);
     segment(a, 0, m->cfg.n_vocab, LE_F32, m->logits, m->cfg.n_vocab);
@@ -324,7 +495,7 @@ int LayeredGraph::copy_prefix(ob_kv *dst, const ob_kv *src, uint32_t n) {
     cudaStream_t st = m->ctx->stream;
     for (const LayerPlan &P : L) {
         if (P.pool) {
-            launch_copy_pages(P.pool, (uint64_t)KV_PAGE * P.dq * es(), src->d_table, dst->d_table, (n + KV_PAGE - 1) / KV_PAGE, st);
+            launch_copy_pages(P.pool, (uint64_t)KV_PAGE * cache_elems(P) * es(), src->d_table, dst->d_table, (n + KV_PAGE - 1) / KV_PAGE, st);
             m->ctx->launches++;
         } else if (P.state && src->slot >= 0 && dst->slot >= 0) {
             const size_t e = state_elems(P);
@@ -337,26 +508,34 @@ int LayeredGraph::copy_prefix(ob_kv *dst, const ob_kv *src, uint32_t n) {
 int LayeredGraph::read_pages(const ob_kv *kv, uint32_t layer, uint32_t pos0, uint32_t n, float *k_out, float *v_out) {
     const LayerPlan &P = L[layer];
     if (!P.pool) return fail(m->ctx, OB_ERR_INVALID, "kv_read: the layer caches no positions");
-    std::vector<uint8_t> row(P.dq * es());
-    for (uint32_t i = 0; i < n; ++i) {
-        const uint32_t p = pos0 + i;
-        const uint8_t *src = static_cast<const uint8_t *>(P.pool) + ((size_t)kv->pages[p / KV_PAGE] * KV_PAGE + p % KV_PAGE) * row.size();
-        OB_CUDA(m->ctx, cudaMemcpy(row.data(), src, row.size(), cudaMemcpyDeviceToHost));
-        auto at = [&](uint32_t c) {
-            float v;
-            if (f32) {
-                memcpy(&v, row.data() + 4 * c, 4);
+    const bool latent = P.mx.kind == OB_MIXER_LATENT_ATTENTION;
+    std::vector<uint8_t> row((latent ? P.dq : P.row) * es());
+    const uint32_t heads = latent ? 1 : P.mx.n_kv_head;  // of a page, KV_PAGE rows each
+    for (uint32_t i = 0; i < n; ++i)
+        for (uint32_t g = 0; g < heads; ++g) {
+            const uint32_t p = pos0 + i;
+            const uint8_t *src = static_cast<const uint8_t *>(P.pool) + (((size_t)kv->pages[p / KV_PAGE] * heads + g) * KV_PAGE + p % KV_PAGE) * row.size();
+            OB_CUDA(m->ctx, cudaMemcpy(row.data(), src, row.size(), cudaMemcpyDeviceToHost));
+            auto copy = [&](float *dst, uint32_t col, uint32_t count) {
+                for (uint32_t c = 0; c < count; ++c) {
+                    if (f32) {
+                        memcpy(dst + c, row.data() + 4 * (col + c), 4);
+                    } else {
+                        uint16_t b;
+                        memcpy(&b, row.data() + 2 * (col + c), 2);
+                        const uint32_t u = (uint32_t)b << 16;
+                        memcpy(dst + c, &u, 4);
+                    }
+                }
+            };
+            if (latent) {
+                copy(k_out + (size_t)i * P.mx.kv_rank, 0, P.mx.kv_rank);
+                copy(v_out + (size_t)i * P.mx.rot_dim, P.kv_p, P.mx.rot_dim);
             } else {
-                uint16_t b;
-                memcpy(&b, row.data() + 2 * c, 2);
-                const uint32_t u = (uint32_t)b << 16;
-                memcpy(&v, &u, 4);
+                for (uint32_t map = 0; map < P.mx.n_map; ++map) copy(k_out + (((size_t)i * heads + g) * P.mx.n_map + map) * P.mx.dim, map * P.dim_p, P.mx.dim);
+                copy(v_out + ((size_t)i * heads + g) * P.mx.vdim, P.mx.n_map * P.dim_p, P.mx.vdim);
             }
-            return v;
-        };
-        for (uint32_t c = 0; c < P.mx.kv_rank; ++c) k_out[(size_t)i * P.mx.kv_rank + c] = at(c);
-        for (uint32_t c = 0; c < P.mx.rot_dim; ++c) v_out[(size_t)i * P.mx.rot_dim + c] = at(P.kv_p + c);
-    }
+        }
     return OB_OK;
 }
 
@@ -369,10 +548,15 @@ int LayeredGraph::read_state(const ob_kv *kv, uint32_t layer, float *out) {
 
 int LayeredGraph::build_layer(const ob_block_desc &b, LayerPlan &P) {
     const ob_mixer_desc &x = b.mixer;
-    const bool latent = x.kind == OB_MIXER_LATENT_ATTENTION;
-    const uint32_t H = x.n_head;
+    const bool latent = x.kind == OB_MIXER_LATENT_ATTENTION, attends = x.kind == OB_MIXER_ATTENTION;
+    const uint32_t H = x.n_head, G = x.n_kv_head;
     int rc;
     P.mx = x;
+    P.sequential = b.post_norm1 != nullptr;
+    P.ff_kind = b.ff_kind;
+    P.n_expert = b.n_expert;
+    P.top = b.ff_kind == OB_FF_EXPERTS ? b.n_expert_used : 1;
+    const uint32_t glu = P.sequential ? 0 : b.n_ff;  // feed-forward inside the mixer's products
     P.norm_gain = b.norm_gain;
     P.n_ff = b.n_ff;
     P.glu_limit = b.glu_limit;
@@ -385,12 +569,21 @@ int LayeredGraph::build_layer(const ob_block_desc &b, LayerPlan &P) {
         P.kv_w = round_up(x.kv_rank, LIN_K_ALIGN);
         P.act_rows = H * P.dim_p;
         P.f32_rows = H * x.rot_dim + x.kv_rank + x.rot_dim + H;
+    } else if (attends) {
+        P.has_v = x.wv.data != nullptr;
+        P.has_gate = x.w_gate.data != nullptr;
+        P.dim_p = round_up(x.dim, 16);
+        P.vdim_p = round_up(x.vdim, 16);
+        P.row = attention_cache_row(x.n_map, P.dim_p, P.vdim_p);
+        P.gate0 = P.has_v ? G * x.vdim : 0;
+        P.act_rows = round_up(P.gate0 + (P.has_gate ? H * x.vdim : 0), LIN_ROW_ALIGN);
+        P.f32_rows = (H + G) * x.n_map * x.dim;
     } else {
         P.f32_rows = H * (2 * x.dim + 2 * x.vdim);
     }
     P.f32_row0 = P.act_rows;
     P.glu_row0 = P.f32_row0 + round_up(P.f32_rows, LIN_ROW_ALIGN);
-    HostDense in(P.glu_row0 + round_up(2 * b.n_ff, LIN_ROW_ALIGN), h_pitch);
+    HostDense in(P.glu_row0 + round_up(2 * glu, LIN_ROW_ALIGN), h_pitch);
     uint32_t r = P.f32_row0;
     auto rows = [&](const ob_matrix_desc &d) {
         for (uint32_t i = 0; i < d.out_dim; ++i) in.copy(r++, 0, d, i);
@@ -402,25 +595,45 @@ int LayeredGraph::build_layer(const ob_block_desc &b, LayerPlan &P) {
         }
         rows(x.w_dkv);
         rows(x.w_gate);
+    } else if (attends) {
+        r = 0;
+        if (P.has_v) rows(x.wv);
+        if (P.has_gate) rows(x.w_gate);
+        r = P.f32_row0;
+        rows(x.wq);
+        rows(x.wk);
+        if (x.q_bias || x.k_bias || x.v_bias) {
+            std::vector<float> bias(in.rows, 0.0f);
+            if (x.v_bias) std::copy(x.v_bias, x.v_bias + G * x.vdim, bias.begin());
+            if (x.q_bias) std::copy(x.q_bias, x.q_bias + H * x.n_map * x.dim, bias.begin() + P.f32_row0);
+            if (x.k_bias) std::copy(x.k_bias, x.k_bias + G * x.n_map * x.dim, bias.begin() + P.f32_row0 + H * x.n_map * x.dim);
+            if ((rc = upload_now(bias.data(), bias.size(), &P.in_bias))) return rc;
+        }
     } else {
         rows(x.wq);
         rows(x.wk);
         rows(x.wv);
         rows(x.w_gate);
     }
-    for (uint32_t i = 0; i < b.n_ff; ++i) {
+    for (uint32_t i = 0; i < glu; ++i) {
         in.copy(P.glu_row0 + 2 * i, 0, b.w_gate, i);
         in.copy(P.glu_row0 + 2 * i + 1, 0, b.w_up, i);
     }
     if ((rc = upload(in, &P.in))) return rc;
     // ---- output products side by side
     P.mix_cols = round_up(H * x.vdim, LIN_K_ALIGN);
-    HostDense out(round_up(width, LIN_ROW_ALIGN), P.mix_cols + round_up(b.n_ff, LIN_K_ALIGN));
+    HostDense out(round_up(width, LIN_ROW_ALIGN), P.mix_cols + round_up(glu, LIN_K_ALIGN));
     for (uint32_t i = 0; i < width; ++i) {
         out.copy(i, 0, x.wo, i);
-        if (b.n_ff) out.copy(i, P.mix_cols, b.w_down, i);
+        if (glu) out.copy(i, P.mix_cols, b.w_down, i);
     }
     if ((rc = upload(out, &P.out))) return rc;
+    if (x.o_bias) {
+        std::vector<float> bias(out.rows, 0.0f);
+        std::copy(x.o_bias, x.o_bias + width, bias.begin());
+        if ((rc = upload_now(bias.data(), bias.size(), &P.out_bias))) return rc;
+    }
+    if (P.sequential && ((rc = upload_now(b.post_norm1, width, &P.post1)) || (rc = build_ff(b, P)))) return rc;
     if (side_dim) {
         HostDense g(round_up(side_dim, LIN_ROW_ALIGN), h_pitch), pr(round_up(width, LIN_ROW_ALIGN), side_p);
         for (uint32_t i = 0; i < side_dim; ++i) g.copy(i, 0, b.side_gate, i);
@@ -452,6 +665,9 @@ int LayeredGraph::build_layer(const ob_block_desc &b, LayerPlan &P) {
         }
         if ((rc = upload_f32(m, x.kv_norm, x.kv_rank, &P.kv_norm))) return rc;
         if ((rc = scratch(&P.pool, (size_t)m->pool_pages * KV_PAGE * P.dq, es()))) return rc;
+    } else if (attends) {
+        if ((rc = upload_now(x.q_norm, x.dim, &P.q_norm)) || (rc = upload_now(x.k_norm, x.dim, &P.k_norm))) return rc;
+        if ((rc = scratch(&P.pool, (size_t)m->pool_pages * KV_PAGE * cache_elems(P), es()))) return rc;
     } else {
         if ((rc = upload_f32(m, x.decay, H, &P.decay))) return rc;
         P.decay_min = *std::min_element(x.decay, x.decay + H);
@@ -460,7 +676,36 @@ int LayeredGraph::build_layer(const ob_block_desc &b, LayerPlan &P) {
     }
     OB_CUDA(m->ctx, cudaStreamSynchronize(m->ctx->stream));  // the host matrices end here
     P.mx.decay = nullptr;
-    P.mx.kv_norm = nullptr;
+    P.mx.kv_norm = P.mx.q_norm = P.mx.k_norm = P.mx.q_bias = P.mx.k_bias = P.mx.v_bias = P.mx.o_bias = nullptr;
+    return OB_OK;
+}
+
+// Feed-forward of a sequential block.
+int LayeredGraph::build_ff(const ob_block_desc &b, LayerPlan &P) {
+    int rc;
+    if (!b.n_ff) return OB_OK;
+    const bool experts = b.ff_kind == OB_FF_EXPERTS;
+    const uint32_t E = experts ? b.n_expert : 1, up_rows = round_up((experts ? 2 : 1) * b.n_ff, LIN_ROW_ALIGN), down_rows = round_up(width, LIN_ROW_ALIGN),
+                   kp = round_up(b.n_ff, LIN_K_ALIGN);
+    if ((rc = upload_now(b.post_norm2, width, &P.post2))) return rc;
+    HostDense up(E * up_rows, h_pitch), down(E * down_rows, kp);
+    for (uint32_t e = 0; e < E; ++e) {
+        for (uint32_t i = 0; i < b.n_ff; ++i) {
+            if (experts) {
+                up.copy(e * up_rows + 2 * i, 0, b.expert_gate[e], i);
+                up.copy(e * up_rows + 2 * i + 1, 0, b.expert_up[e], i);
+            } else {
+                up.copy(i, 0, b.w_up, i);
+            }
+        }
+        for (uint32_t i = 0; i < width; ++i) down.copy(e * down_rows + i, 0, experts ? b.expert_down[e] : b.w_down, i);
+    }
+    if ((rc = upload(up, &P.up)) || (rc = upload(down, &P.down))) return rc;
+    if (experts) {
+        HostDense z(round_up(E, LIN_ROW_ALIGN), h_pitch);
+        for (uint32_t e = 0; e < E; ++e) z.copy(e, 0, b.w_router, e);
+        if ((rc = upload(z, &P.router))) return rc;
+    }
     return OB_OK;
 }
 
@@ -474,9 +719,12 @@ int LayeredGraph::build(const ob_layered_desc &c) {
     side_p = round_up(side_dim, LIN_K_ALIGN);
     eps = c.rms_eps;
     final_gain = c.final_gain;
+    residual_mult = c.residual_mult;
+    if (c.final_norm && (rc = upload_now(c.final_norm, width, &final_norm))) return rc;
     L.resize(c.n_layer);
     std::map<std::pair<double, uint32_t>, float2 *> tables;
-    size_t act = 0, q_n = 0, o_n = 0, o_r = 0, kvp = 0, dq = 0, ex = 0, reach = 0;
+    size_t act = 0, q_n = 0, o_n = 0, o_r = 0, kvp = 0, dq = 0, ex = 0, reach = 0, ff_n = 0, pairs = 0, experts = 0;
+    bool sequential = false;
     for (uint32_t i = 0; i < c.n_layer; ++i) {
         LayerPlan &P = L[i];
         if ((rc = build_layer(c.layers[i], P))) return rc;
@@ -495,7 +743,15 @@ int LayeredGraph::build(const ob_layered_desc &c) {
         act = std::max<size_t>(act, P.act_rows);
         y_pitch = std::max(y_pitch, round_up(P.f32_rows, 4));
         cat_pitch = std::max(cat_pitch, P.out.kp);
-        if (P.pool) {
+        sequential |= P.sequential;
+        if (P.sequential && P.n_ff) ff_n = std::max<size_t>(ff_n, T * P.top * P.down.kp);
+        if (P.n_expert) {
+            pairs = std::max<size_t>(pairs, T * P.top);
+            experts = std::max<size_t>(experts, P.n_expert);
+        }
+        if (P.mx.kind == OB_MIXER_ATTENTION) {
+            q_n = std::max<size_t>(q_n, (size_t)H * P.mx.n_map * P.dim_p);
+        } else if (P.pool) {
             q_n = std::max<size_t>(q_n, (size_t)H * P.dq);
             o_n = std::max<size_t>(o_n, (size_t)H * P.kv_w);
             kvp = std::max<size_t>(kvp, P.kv_p);
@@ -523,13 +779,23 @@ int LayeredGraph::build(const ob_layered_desc &c) {
     if ((rc = scratch(&h, T * h_pitch, es())) || (rc = scratch(&xb, T * h_pitch, es())) || (rc = scratch(&cat, T * cat_pitch, es()))) return rc;
     if ((rc = scratch(&qn, T * act, es())) || (rc = scratch(&q, T * q_n, es())) || (rc = scratch(&o_lat, T * o_n, es()))) return rc;
     if ((rc = scratch_f32(&y, T * y_pitch)) || (rc = scratch_f32(&o_ret, T * o_r))) return rc;
+    if (sequential && ((rc = scratch(&ffa, ff_n, es())) || (rc = scratch_f32(&yo, std::max(T, pairs) * width)))) return rc;
+    if (pairs) {
+        float *row_score;
+        if ((rc = dev_alloc(m, &moe.expert, pairs)) || (rc = dev_alloc(m, &moe.rank, pairs)) || (rc = dev_alloc(m, &moe.row, pairs))) return rc;
+        if ((rc = scratch_f32(&moe.score, pairs)) || (rc = scratch_f32(&row_score, pairs)) || (rc = scratch_f32(&router_logits, T * experts))) return rc;
+        if ((rc = dev_alloc(m, &moe.tiles, pairs / 16 + experts + 1)) || (rc = dev_alloc(m, &moe.n_tiles, 1)) || (rc = dev_alloc(m, &moe.count, experts))) return rc;
+        if ((rc = scratch(&moe.gathered, pairs * h_pitch, es()))) return rc;
+        OB_CUDA(m->ctx, cudaMemset(moe.count, 0, experts * 4));
+        moe.row_score = row_score;
+    }
     if (ex) {
         key_cap = (uint32_t)(T + reach);
         if ((rc = scratch(&lat, (size_t)key_cap * dq, 2)) || (rc = scratch(&expanded, (size_t)key_cap * ex, 2))) return rc;
     }
     if (side_dim && ((rc = scratch(&sg, T * side_p, es())) || (rc = scratch_f32(&sy, T * width)))) return rc;
     if (!f32 && (rc = scratch_f32(&split_part, linear_split_bytes() / 4))) return rc;
-    if (q_n && !f32) {  // at most one CTA per SM, of 64 rows, writes partial results at a time (launch_latent_attention)
+    if (kvp && !f32) {  // at most one CTA per SM, of 64 rows, writes partial results at a time (launch_latent_attention)
         part_cap = ((uint64_t)m->ctx->sm_count * 64 + 64) * (kvp + 4);
         if ((rc = scratch_f32(&part, part_cap))) return rc;
     }
@@ -551,7 +817,7 @@ int check_block(ob_ctx *ctx, const ob_layered_desc &c, uint32_t i) {
     const std::string at = "layer " + std::to_string(i) + " ";
     int rc;
     if (!x.n_head || !x.dim || !x.vdim) return fail(ctx, OB_ERR_INVALID, "layered model: " + at + "mixer sizes missing");
-    const uint32_t H = x.n_head, E = c.n_embd, rotating = x.kind == OB_MIXER_LATENT_ATTENTION ? x.rot_dim : x.dim;
+    const uint32_t H = x.n_head, G = x.n_kv_head, E = c.n_embd, rotating = x.kind == OB_MIXER_LATENT_ATTENTION ? x.rot_dim : x.dim;
     if ((x.rot_dims & 1) || x.rot_dims > rotating) return fail(ctx, OB_ERR_INVALID, "layered model: " + at + "rot_dims must be even and fit the rotated vector");
     if (x.rot_dims && !(x.rot_base > 0)) return fail(ctx, OB_ERR_INVALID, "layered model: " + at + "rot_base must be positive");
     if (x.kind == OB_MIXER_LATENT_ATTENTION) {
@@ -569,10 +835,46 @@ int check_block(ob_ctx *ctx, const ob_layered_desc &c, uint32_t i) {
         if ((rc = check_dense(ctx, x.wk, E, H * x.dim, at + "wk"))) return rc;
         if ((rc = check_dense(ctx, x.wv, E, H * x.vdim, at + "wv"))) return rc;
         if ((rc = check_dense(ctx, x.w_gate, E, H * x.vdim, at + "mixer gate"))) return rc;
+    } else if (x.kind == OB_MIXER_ATTENTION) {
+        if (!G || H % G) return fail(ctx, OB_ERR_INVALID, "layered model: " + at + "n_kv_head does not divide n_head");
+        if (x.n_map != 1 && x.n_map != 2) return fail(ctx, OB_ERR_UNSUPPORTED, "layered model: " + at + "one or two maps per head");
+        if (!x.q_norm || !x.k_norm) return fail(ctx, OB_ERR_INVALID, "layered model: " + at + "query or key norm missing");
+        if (!attention_supported(x.dim, x.vdim)) return fail(ctx, OB_ERR_UNSUPPORTED, "layered model: " + at + "attention head too large");
+        if ((rc = check_dense(ctx, x.wq, E, H * x.n_map * x.dim, at + "wq"))) return rc;
+        if ((rc = check_dense(ctx, x.wk, E, G * x.n_map * x.dim, at + "wk"))) return rc;
+        if (x.wv.data) {
+            if ((rc = check_dense(ctx, x.wv, E, G * x.vdim, at + "wv"))) return rc;
+        } else if (x.n_map != 1 || x.vdim != x.dim || x.v_bias) {
+            return fail(ctx, OB_ERR_INVALID, "layered model: " + at + "keys can be the values of one map of their own size");
+        }
+        if (x.w_gate.data && (rc = check_dense(ctx, x.w_gate, E, H * x.vdim, at + "mixer gate"))) return rc;
     } else {
         return fail(ctx, OB_ERR_UNSUPPORTED, "layered model: " + at + "unknown mixer");
     }
+    if (x.kind != OB_MIXER_ATTENTION && (x.q_bias || x.k_bias || x.v_bias)) return fail(ctx, OB_ERR_UNSUPPORTED, "layered model: " + at + "the mixer has no biases");
+    if ((b.post_norm1 != nullptr) != (c.layers[0].post_norm1 != nullptr)) return fail(ctx, OB_ERR_UNSUPPORTED, "layered model: " + at + "blocks of two kinds");
     if ((rc = check_dense(ctx, x.wo, H * x.vdim, E, at + "wo"))) return rc;
+    if (b.post_norm1) {
+        if (c.side_dim) return fail(ctx, OB_ERR_UNSUPPORTED, "layered model: " + at + "sequential blocks have no per-layer token input");
+        if (!b.n_ff) return OB_OK;
+        if (!b.post_norm2) return fail(ctx, OB_ERR_INVALID, "layered model: " + at + "norm of the feed-forward missing");
+        if (b.ff_kind == OB_FF_RELU2) {
+            if ((rc = check_dense(ctx, b.w_up, E, b.n_ff, at + "ff up"))) return rc;
+            return check_dense(ctx, b.w_down, b.n_ff, E, at + "ff down");
+        }
+        if (b.ff_kind != OB_FF_EXPERTS) return fail(ctx, OB_ERR_UNSUPPORTED, "layered model: " + at + "unknown feed-forward");
+        if (!b.n_expert || !b.n_expert_used || b.n_expert_used > b.n_expert || !b.expert_gate || !b.expert_up || !b.expert_down)
+            return fail(ctx, OB_ERR_INVALID, "layered model: " + at + "experts missing");
+        if (b.n_expert > MOE_MAX_EXPERTS) return fail(ctx, OB_ERR_UNSUPPORTED, "layered model: " + at + "too many experts");
+        if ((rc = check_dense(ctx, b.w_router, E, b.n_expert, at + "router"))) return rc;
+        for (uint32_t e = 0; e < b.n_expert; ++e) {
+            if ((rc = check_dense(ctx, b.expert_gate[e], E, b.n_ff, at + "expert gate"))) return rc;
+            if ((rc = check_dense(ctx, b.expert_up[e], E, b.n_ff, at + "expert up"))) return rc;
+            if ((rc = check_dense(ctx, b.expert_down[e], b.n_ff, E, at + "expert down"))) return rc;
+        }
+        return OB_OK;
+    }
+    if (b.ff_kind != OB_FF_CLAMPED_GLU) return fail(ctx, OB_ERR_UNSUPPORTED, "layered model: " + at + "parallel blocks have the clamped feed-forward");
     if (b.n_ff) {
         if ((rc = check_dense(ctx, b.w_gate, E, b.n_ff, at + "ff gate"))) return rc;
         if ((rc = check_dense(ctx, b.w_up, E, b.n_ff, at + "ff up"))) return rc;
@@ -608,6 +910,7 @@ extern "C" int ob_layered_model_create(ob_ctx *ctx, const ob_layered_desc *desc,
     Bind b(ctx);
     OB_CUDA(ctx, linear_configure());
     OB_CUDA(ctx, mixers_configure());
+    OB_CUDA(ctx, attention_configure());
     ob_model *m = new ob_model;
     m->ctx = ctx;
     m->cfg.n_vocab = c.n_vocab;

@@ -1,5 +1,6 @@
 // Launchers of the kernels for models given as a list of layers (layered.cu): bf16-weight products with fused epilogues, norms,
-// latent attention over a paged latent cache, retention with a per-sequence state (internal to the library).
+// latent attention over a paged latent cache, retention with a per-sequence state, softmax attention over paged keys and values,
+// mixtures of experts (internal to the library).
 //
 // Two precisions share every launcher.  bf16: activations that enter a product are bfloat16, accumulation is fp32.  f32:
 // activations are fp32 and every product is plain fp32 multiply-add.  Weights are bfloat16 in both.  The residual stream, norms,
@@ -21,12 +22,17 @@ enum LinEpilogue {
     LE_GLU = 2,       // rows (2j, 2j+1) are (gate j, up j): out activation j = g sigmoid(alpha g) (u + 1) of the limited pair
     LE_RESIDUAL = 3,  // x f32 [t][pitch] += v; out2 (optional) gets the sum as activation
     LE_GELU_EMB = 4,  // out activation = gelu_tanh(v) * emb[token t][emb_col0 + row]
-    LE_GATED = 5      // out activation = v * sigmoid(gate[t * gate_pitch + batch])
+    LE_GATED = 5,     // out activation = v * sigmoid(gate[t * gate_pitch + batch])
+    LE_RELU2 = 6,     // out activation = max(v, 0)^2
+    LE_SWIGLU = 7     // rows (2j, 2j+1) are (gate j, up j), both times row_scale[t]: out activation j = silu(g) u
+};
+struct LinTile {          // rows of a grouped product that share a batch entry
+    uint32_t batch, row0, n;
 };
 struct LinSegment {       // consecutive rows of the weight with one epilogue; row0 is a multiple of 32
     uint32_t row0, n;     // rows [row0, row0 + n)
     int epi;
-    void *out;            // element (t, r) goes to out[t * pitch + col0 + batch * batch_cols + (r - row0)] (LE_GLU: (r - row0) / 2)
+    void *out;            // element (t, r) goes to out[t * pitch + col0 + batch * batch_cols + (r - row0)] (pairs: (r - row0) / 2)
     uint32_t pitch, col0, batch_cols;
 };
 struct LinArgs {
@@ -47,7 +53,18 @@ struct LinArgs {
     const float *gate = nullptr;
     uint32_t gate_pitch = 0;
     float *split_part = nullptr;  // scratch of products that split K, linear_split_bytes
+    const float *bias = nullptr;  // [n_batch][n_rows] added to the products before the epilogue
+    const float *row_scale = nullptr;  // [T]
+    // Grouped products: every row of x has a batch entry of its own.  Either row by row, or in tiles of rows with one entry each
+    // (rows of one entry next to one another), made on the device: *n_tiles of at most max_tiles, of tile_rows rows or fewer.
+    const uint32_t *row_batch = nullptr;  // [T], row t reads row t / x_div of x
+    uint32_t x_div = 1;
+    const LinTile *tiles = nullptr;
+    const uint32_t *n_tiles = nullptr;
+    uint32_t max_tiles = 0, tile_rows = 0;
 };
+// Rows of a tile that a grouped product of `rows` rows over `batches` entries takes best.
+uint32_t linear_tile_rows(uint32_t rows, uint32_t batches, bool f32);
 constexpr uint32_t LIN_K_ALIGN = 64, LIN_ROW_ALIGN = 32;
 cudaError_t linear_configure();  // kernel attributes of the current device (outside stream capture)
 uint32_t launch_linear(const LinArgs &a, bool f32, int sm_count, cudaStream_t st);  // kernels launched; 0: a tensor map could not be made
@@ -56,12 +73,26 @@ int linear_take_status();        // 1 when a bounded wait inside a product ran o
 void linear_mark_launched();     // a replayed graph may have run one of the tensor-core products
 
 // ---- mixers.cu -------------------------------------------------------------------------------------------------------
-// x = embedding rows, h = x / rms(x) * gain as activation.
-void launch_embed_norm(const __nv_bfloat16 *table, uint32_t width, const uint32_t *tokens, uint32_t T, float *x, float eps, float gain, void *h, uint32_t h_pitch,
-                       bool f32, cudaStream_t st);
-// h[i] = x[row i] / rms(x[row i]) * gain, as activation; rows == nullptr: row i.
-void launch_norm_scalar(const float *x, uint32_t width, const uint32_t *rows, uint32_t n, float eps, float gain, void *h, uint32_t h_pitch, bool f32,
-                        cudaStream_t st);
+// x = embedding rows; h = x / rms(x) * gain as activation, or (normed false) x itself.
+void launch_embed(const __nv_bfloat16 *table, uint32_t width, const uint32_t *tokens, uint32_t T, float *x, bool normed, float eps, float gain, void *h,
+                  uint32_t h_pitch, bool f32, cudaStream_t st);
+// h[i] = x[row i] / rms(x[row i]) * gain (* w), as activation; rows == nullptr: row i; w [width], may be null.
+void launch_norm(const float *x, uint32_t width, const uint32_t *rows, uint32_t n, float eps, float gain, const float *w, void *h, uint32_t h_pitch, bool f32,
+                 cudaStream_t st);
+struct PostNormArgs {        // x += mult * y / rms(y) * w, then h = x as activation
+    float *x;                // [T][width]
+    const float *y;          // [T * top][width]: the `top` rows of a token are added up first
+    const uint32_t *rows;    // where they are, [T * top]; null: in order
+    uint32_t top;
+    const float *w;          // [width]
+    uint32_t width, T;
+    float eps, mult;
+    void *h;                 // null: not needed
+    uint32_t h_pitch;
+    uint32_t *zero;          // set to zero for whoever counts next, n_zero words; may be null
+    uint32_t n_zero;
+};
+void launch_post_norm(const PostNormArgs &a, bool f32, cudaStream_t st);
 // x += y / rms(y) * w, then (h != nullptr) h = x / rms(x) * gain as activation.
 void launch_side_finish(float *x, const float *y, const float *w, uint32_t width, uint32_t T, float eps, float gain, void *h, uint32_t h_pitch, bool f32,
                         cudaStream_t st);
@@ -150,6 +181,58 @@ struct RetentionArgs {       // retention of one layer over T rows
 };
 bool retention_supported(uint32_t dim);
 uint32_t launch_retention(const RetentionArgs &a, bool f32, int sm_count, cudaStream_t st);
+// ---- gqa.cu ----------------------------------------------------------------------------------------------------------
+struct AttentionArgs {       // softmax attention of one layer over T rows
+    const float *y;          // f32 projections [T][y_pitch]: queries [n_head][n_map][dim], keys [n_kv][n_map][dim]
+    uint32_t y_pitch;
+    const void *va;          // activations [T][va_pitch]: values [n_kv][vdim] (has_v; else the values are the keys as projected), gates [n_head][vdim] from gate0
+    uint32_t va_pitch, gate0;
+    bool has_v, has_gate;
+    uint32_t n_head, n_kv, n_map, dim, vdim, window;  // window 0: no limit
+    uint32_t dim_p, vdim_p, row;  // padded sizes; elements of a cache row: keys [n_map][dim_p], value [vdim_p], padding
+    float eps, scale, map_weight, head_gain;
+    const float *q_norm, *k_norm;  // [dim]
+    Rot rot;
+    void *q;                 // activations [T][n_head][n_map][dim_p]
+    void *cache;             // activations [page][n_kv][16][row]
+    void *out;               // activations [T][out_pitch], head h at h * vdim
+    uint32_t out_pitch;
+    uint32_t T, n_seq, n_short;   // spans [0, n_short) are short, the others long (PREFILL_SPAN rows or more)
+    const RowSpan *spans;    // device [n_seq]
+    const RowSpan *h_spans;  // the same on the host
+    bool single;             // every span is one row
+    const uint32_t *positions;
+    const int32_t *const *tables;
+    uint32_t max_pos;        // positions are below this
+};
+cudaError_t attention_configure();
+bool attention_supported(uint32_t dim, uint32_t vdim);
+uint32_t attention_cache_row(uint32_t n_map, uint32_t dim_p, uint32_t vdim_p);  // elements of a cache row
+void launch_attention_prep(const AttentionArgs &a, bool f32, cudaStream_t st);  // norms, rotates and stores queries; appends keys and values
+uint32_t launch_attention(const AttentionArgs &a, bool f32, int sm_count, cudaStream_t st);  // returns the kernels launched
+
+// ---- moe.cu ----------------------------------------------------------------------------------------------------------
+struct MoeArgs {             // routing of T tokens to `top` of n_expert experts; a (token, choice) is a pair, t * top + choice
+    const void *x;           // activations [T][x_pitch], x_pitch a multiple of 64
+    uint32_t x_pitch;
+    const __nv_bfloat16 *w;  // router [n_expert or more][x_pitch]
+    const float *logits;     // [T][logit_pitch]: logits made by a product; null: the routing kernel makes them
+    uint32_t logit_pitch;
+    uint32_t n_expert, top, T;
+    uint32_t *expert;        // [T * top]
+    float *score;            // [T * top]
+    // grouping (null: pairs stay in order): pairs of one expert next to one another
+    uint32_t *count;         // [n_expert], zero before and left for the caller to zero
+    uint32_t *rank, *row;    // [T * top]: place among the expert's pairs; row of the pair
+    void *gathered;          // activations [T * top][x_pitch]
+    float *row_score;        // [T * top], by row
+    LinTile *tiles;          // tiles of tile_rows rows or fewer, *n_tiles of them
+    uint32_t *n_tiles, tile_rows;
+};
+constexpr uint32_t MOE_MAX_EXPERTS = 1024;
+constexpr uint32_t MOE_DOT_TOKENS = 64;  // up to this many tokens the routing kernel makes the logits itself
+uint32_t launch_moe_route(const MoeArgs &a, bool f32, cudaStream_t st);  // returns the kernels launched
+
 // Pages [0, n_pages) of one sequence's table to another's within a pool of pages of page_bytes (a multiple of 16).
 void launch_copy_pages(void *pool, uint64_t page_bytes, const int32_t *src_table, const int32_t *dst_table, uint32_t n_pages, cudaStream_t st);
 

@@ -3,6 +3,7 @@
 //   gemv_act_kernel      a few tokens: a group of lanes per pair of rows streams the weights once, HBM-bound
 //   linear_tc5_kernel    bf16 activations: tcgen05.mma (kind::f16) with fp32 accumulators in tensor memory, operands by TMA
 //   linear_simt_kernel   fp32 activations: plain fp32 multiply-add tiles
+// Each also runs grouped products (a mixture of experts), the rows of which have batch entries of their own.
 // All three end in epilogue_store, so a product means the same whichever kernel runs it.
 #include <algorithm>
 
@@ -68,6 +69,11 @@ __device__ __forceinline__ float gelu_tanhf(float z) {
 // N consecutive weight rows starting at r (within one 32-row group, r even) of token t: v holds the products.
 template <typename TA, int N>
 __device__ __forceinline__ void epilogue_store(const LinArgs &a, uint32_t batch, uint32_t t, uint32_t r, float *v) {
+    if (a.bias) {
+        const float *b = a.bias + (uint64_t)batch * a.n_rows + r;
+#pragma unroll
+        for (int i = 0; i < N; ++i) v[i] += __ldg(b + i);
+    }
 #pragma unroll 1
     for (int s = 0; s < a.n_seg; ++s) {
         const LinSegment &g = a.seg[s];
@@ -112,6 +118,26 @@ __device__ __forceinline__ void epilogue_store(const LinArgs &a, uint32_t batch,
             store_row<N>(static_cast<TA *>(g.out) + base + k, v, n);
             break;
         }
+        case LE_RELU2: {
+#pragma unroll
+            for (int i = 0; i < N; ++i) {
+                const float p = fmaxf(v[i], 0.0f);
+                v[i] = p * p;
+            }
+            store_row<N>(static_cast<TA *>(g.out) + base + k, v, n);
+            break;
+        }
+        case LE_SWIGLU: {
+            const float w = a.row_scale ? a.row_scale[t] : 1.0f;
+            float o[N / 2 > 0 ? N / 2 : 1];
+#pragma unroll
+            for (int j = 0; j < N / 2; ++j) {
+                const float gt = v[2 * j] * w;
+                o[j] = gt * sigmoidf(gt) * (v[2 * j + 1] * w);
+            }
+            store_row<(N / 2 > 0 ? N / 2 : 1)>(static_cast<TA *>(g.out) + base + k / 2, o, n / 2);
+            break;
+        }
         default: {  // LE_GATED
             const float s = sigmoidf(a.gate[(uint64_t)t * a.gate_pitch + batch]);
 #pragma unroll
@@ -133,8 +159,14 @@ __global__ void __launch_bounds__(GV_THREADS, NT == 1 ? 3 : 2) gemv_act_kernel(L
     const uint32_t warp = threadIdx.x >> 5, lane = threadIdx.x & 31, per_warp = 32 / G;
     const uint32_t ks = KS > 1 ? warp % KS : 0, unit = KS > 1 ? warp / KS : warp * per_warp + lane / G;
     const uint32_t units = KS > 1 ? 8 / KS : 8 * per_warp;
-    const uint32_t batch = blockIdx.z, pair = blockIdx.x * units + unit, r = 2 * pair;
-    const bool live = r < a.n_rows;
+    const uint32_t pair = blockIdx.x * units + unit, r = 2 * pair;
+    const bool live = r < a.n_rows, grouped = NT == 1 && a.row_batch != nullptr;  // grouped: a token per blockIdx.z, its weights known once the predecessor is done
+    uint32_t batch = blockIdx.z;
+    if (grouped) {
+        pdl_release();
+        pdl_wait();
+        batch = a.row_batch[blockIdx.z];
+    }
     const uint32_t n_chunk = a.kp / 8, step = G * KS, c_first = ks * G + lane % G;
     const uint4 *wa = reinterpret_cast<const uint4 *>(a.w + ((uint64_t)batch * a.n_rows + (live ? r : 0)) * a.kp);
     const uint4 *wb = wa + n_chunk;
@@ -149,9 +181,11 @@ __global__ void __launch_bounds__(GV_THREADS, NT == 1 ? 3 : 2) gemv_act_kernel(L
         }
     };
     fetch(c_first);
-    pdl_release();
-    pdl_wait();
-    const TA *x = static_cast<const TA *>(a.x) + (uint64_t)batch * a.x_step;
+    if (!grouped) {
+        pdl_release();
+        pdl_wait();
+    }
+    const TA *x = static_cast<const TA *>(a.x) + (grouped ? (uint64_t)(blockIdx.z / a.x_div) * a.x_pitch : (uint64_t)batch * a.x_step);
     float acc[NT][2];
 #pragma unroll
     for (int t = 0; t < NT; ++t) acc[t][0] = acc[t][1] = 0.0f;
@@ -199,7 +233,7 @@ __global__ void __launch_bounds__(GV_THREADS, NT == 1 ? 3 : 2) gemv_act_kernel(L
     if (!live) return;
 #pragma unroll
     for (int t = 0; t < NT; ++t)  // G may be smaller than NT: lanes take tokens in turn
-        if ((t % G) == lane % G) epilogue_store<TA, 2>(a, batch, t, r, acc[t]);
+        if ((t % G) == lane % G) epilogue_store<TA, 2>(a, batch, grouped ? blockIdx.z : t, r, acc[t]);
 }
 
 // ---- fp32 tiles -----------------------------------------------------------------------------------------------------------
@@ -209,9 +243,15 @@ __global__ void __launch_bounds__(256) linear_simt_kernel(LinArgs a) {
     __shared__ float xs[16][68], ws[16][68];
     pdl_release();
     pdl_wait();
-    const uint32_t r0 = blockIdx.x * 64, t0 = blockIdx.y * 64, batch = blockIdx.z;
+    uint32_t t0 = blockIdx.y * 64, batch = blockIdx.z, t_end = a.T;
+    if (a.tiles) {
+        if (blockIdx.y >= *a.n_tiles) return;
+        const LinTile tile = a.tiles[blockIdx.y];
+        t0 = tile.row0, batch = tile.batch, t_end = tile.row0 + tile.n;
+    }
+    const uint32_t r0 = blockIdx.x * 64;
     const uint32_t tx = threadIdx.x % 16, ty = threadIdx.x / 16;
-    const TA *x = static_cast<const TA *>(a.x) + (uint64_t)batch * a.x_step;
+    const TA *x = static_cast<const TA *>(a.x) + (a.tiles ? 0 : (uint64_t)batch * a.x_step);
     const __nv_bfloat16 *w = a.w + (uint64_t)batch * a.n_rows * a.kp;
     float acc[4][4] = {};
     for (uint32_t k0 = 0; k0 < a.kp; k0 += 16) {
@@ -219,7 +259,7 @@ __global__ void __launch_bounds__(256) linear_simt_kernel(LinArgs a) {
             const uint32_t i = threadIdx.x & 127, row = i >> 1, c = (i & 1) * 8;
             float f[8];
             if (threadIdx.x < 128) {
-                if (t0 + row < a.T) load8(x + (uint64_t)(t0 + row) * a.x_pitch + k0 + c, f);
+                if (t0 + row < t_end) load8(x + (uint64_t)(t0 + row) * a.x_pitch + k0 + c, f);
                 else
 #pragma unroll
                     for (int j = 0; j < 8; ++j) f[j] = 0.0f;
@@ -248,7 +288,7 @@ __global__ void __launch_bounds__(256) linear_simt_kernel(LinArgs a) {
     }
 #pragma unroll
     for (int i = 0; i < 4; ++i)
-        if (t0 + 4 * ty + i < a.T && r0 + 4 * tx < a.n_rows) epilogue_store<TA, 4>(a, batch, t0 + 4 * ty + i, r0 + 4 * tx, acc[i]);
+        if (t0 + 4 * ty + i < t_end && r0 + 4 * tx < a.n_rows) epilogue_store<TA, 4>(a, batch, t0 + 4 * ty + i, r0 + 4 * tx, acc[i]);
 }
 
 // ---- tcgen05 ---------------------------------------------------------------------------------------------------------------
@@ -289,6 +329,8 @@ struct LtTiles {
     uint32_t rows, toks, total;  // weight tiles and token tiles of one batch entry, tiles of all (splits counted)
     uint32_t splits;             // > 1: one token tile of at most LT_SPLIT_TOKENS rows, a CTA per tile and split
     float *part;                 // [tile][split][LT_SPLIT_TOKENS][BN]
+    const LinTile *table;        // grouped: the token tiles (rows of x and their batch entry), *n_table of them; toks and total are bounds
+    const uint32_t *n_table;
 };
 constexpr uint32_t LT_SPLIT_TOKENS = 64;
 __device__ __forceinline__ void lt_tile(const LtTiles &g, uint32_t tile, uint32_t *batch, uint32_t *rt, uint32_t *tt) {
@@ -300,16 +342,29 @@ __device__ __forceinline__ void lt_tile(const LtTiles &g, uint32_t tile, uint32_
     *rt = i / width;
     *tt = grp * LT_GROUP + i % width;
 }
+// Grouped: how many tiles there are in truth; then tile -> weight rows of its batch entry and rows [t0, t_end) of x.
+__device__ __forceinline__ void lt_count(LtTiles &g) {
+    if (!g.table) return;
+    g.toks = *g.n_table;
+    g.total = g.rows * g.toks;
+}
+__device__ __forceinline__ void lt_rows(const LtTiles &g, uint32_t T, uint32_t tt, uint32_t *batch, uint32_t *t0, uint32_t *t_end) {
+    *t0 = tt * LT_M, *t_end = T;
+    if (!g.table) return;
+    const LinTile tile = g.table[tt];
+    *batch = tile.batch, *t0 = tile.row0, *t_end = tile.row0 + tile.n;
+}
 
 template <int BN, int AR>
 __global__ void __launch_bounds__(LT_THREADS, BN == 256 ? 1 : 2)
-linear_tc5_kernel(const __grid_constant__ CUtensorMap tm_x, const __grid_constant__ CUtensorMap tm_w, const __grid_constant__ LinArgs a, const LtTiles g) {
+linear_tc5_kernel(const __grid_constant__ CUtensorMap tm_x, const __grid_constant__ CUtensorMap tm_w, const __grid_constant__ LinArgs a, const LtTiles g_in) {
     using S = LtSmem<BN, AR>;
     extern __shared__ uint8_t smem_raw[];
     const uint32_t sbase = (smem_u32(smem_raw) + 1023u) & ~1023u;
     uint8_t *smem = smem_raw + (sbase - smem_u32(smem_raw));
     const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
     volatile uint32_t *abort = reinterpret_cast<volatile uint32_t *>(smem + S::ABORT);
+    LtTiles g = g_in;
     const uint32_t split = blockIdx.x % g.splits, k0 = a.kp / 64 * split / g.splits, k1 = a.kp / 64 * (split + 1) / g.splits, n_steps = k1 - k0;
 
     if (threadIdx.x == 0) {
@@ -334,20 +389,25 @@ linear_tc5_kernel(const __grid_constant__ CUtensorMap tm_x, const __grid_constan
 
     if (warp == LT_TMA_WARP) {
         if (lane == 0) {
+            if (g.table) {  // which weights is known once the predecessor is done
+                pdl_wait();
+                lt_count(g);
+            }
             const uint32_t ahead = min(n_steps, S::STAGES);
             uint32_t it = 0;
             bool ok = true;
             for (uint32_t tile = blockIdx.x; ok && tile < g.total; tile += gridDim.x) {
-                uint32_t batch, rt, tt;
+                uint32_t batch, rt, tt, t0, t_end;
                 lt_tile(g, tile / g.splits, &batch, &rt, &tt);
-                const int32_t wy = (int32_t)(batch * a.n_rows + rt * BN), xc = (int32_t)(batch * a.x_step), xy = (int32_t)(tt * LT_M);
+                lt_rows(g, a.T, tt, &batch, &t0, &t_end);
+                const int32_t wy = (int32_t)(batch * a.n_rows + rt * BN), xc = g.table ? 0 : (int32_t)(batch * a.x_step), xy = (int32_t)t0;
                 auto weights = [&](uint32_t k, uint32_t s) {
                     mbar_expect_tx(sbase + S::FULL + 8 * s, S::A_BYTES + S::B_BYTES);
                     tma_load_2d(sbase + S::B + s * S::B_BYTES, &tm_w, (int32_t)(k * 64), wy, sbase + S::FULL + 8 * s);
                 };
                 if (tile == blockIdx.x) {
                     for (uint32_t k = 0; k < ahead; ++k) weights(k0 + k, k);
-                    pdl_wait();
+                    if (!g.table) pdl_wait();
                 }
                 for (uint32_t k = k0; k < k1; ++k, ++it) {
                     const uint32_t s = it % S::STAGES;
@@ -362,6 +422,7 @@ linear_tc5_kernel(const __grid_constant__ CUtensorMap tm_x, const __grid_constan
         }
     } else if (warp == LT_MMA_WARP) {
         pdl_wait();
+        lt_count(g);
         if (lane == 0) {
             constexpr uint32_t idesc = umma_idesc_bf16(BN);
             uint32_t it = 0, n = 0;
@@ -386,14 +447,16 @@ linear_tc5_kernel(const __grid_constant__ CUtensorMap tm_x, const __grid_constan
         }
     } else {
         pdl_wait();
+        lt_count(g);
         uint32_t n = 0;
         for (uint32_t tile = blockIdx.x; tile < g.total; tile += gridDim.x, ++n) {
             const uint32_t buf = n % S::NBUF;
-            uint32_t batch, rt, tt;
+            uint32_t batch, rt, tt, t0, t_end;
             lt_tile(g, tile / g.splits, &batch, &rt, &tt);
+            lt_rows(g, a.T, tt, &batch, &t0, &t_end);
             if (!mbar_wait(sbase + S::ACC_FULL + 8 * buf, (n / S::NBUF) & 1u, abort)) break;
             tc_fence_after();
-            const uint32_t t = tt * LT_M + warp * 32 + lane;
+            const uint32_t t = t0 + warp * 32 + lane;
 #pragma unroll 1
             for (int c = 0; c < BN / 32; ++c) {
                 uint32_t u[32];
@@ -404,7 +467,7 @@ linear_tc5_kernel(const __grid_constant__ CUtensorMap tm_x, const __grid_constan
 #pragma unroll
                 for (int i = 0; i < 32; ++i) v[i] = __uint_as_float(u[i]);
                 const uint32_t r = rt * BN + c * 32;
-                if (t < a.T && r < a.n_rows) {
+                if (t < t_end && r < a.n_rows) {
                     if (g.splits == 1) epilogue_store<__nv_bfloat16, 32>(a, batch, t, r, v);
                     else store_row<32>(g.part + ((uint64_t)tile * LT_SPLIT_TOKENS + t) * BN + c * 32, v, 32);
                 }
@@ -451,8 +514,8 @@ bool launch_tc5(const LinArgs &a, int sm_count, cudaStream_t st, uint32_t splits
     CUtensorMap tm_x, tm_w;
     if (!make_map_2d(&tm_x, CU_TENSOR_MAP_DATA_TYPE_BFLOAT16, 2, a.x, a.x_pitch, a.T, (uint64_t)a.x_pitch * 2, 64, AR, CU_TENSOR_MAP_SWIZZLE_128B)) return false;
     if (!make_map_2d(&tm_w, CU_TENSOR_MAP_DATA_TYPE_BFLOAT16, 2, a.w, a.kp, (uint64_t)a.n_batch * a.n_rows, (uint64_t)a.kp * 2, 64, BN, CU_TENSOR_MAP_SWIZZLE_128B)) return false;
-    LtTiles g{(a.n_rows + BN - 1) / BN, (a.T + LT_M - 1) / LT_M, 0, splits, a.split_part};
-    g.total = g.rows * g.toks * a.n_batch * splits;
+    LtTiles g{(a.n_rows + BN - 1) / BN, a.tiles ? a.max_tiles : (a.T + LT_M - 1) / LT_M, 0, splits, a.split_part, a.tiles, a.n_tiles};
+    g.total = g.rows * g.toks * (a.tiles ? 1 : a.n_batch) * splits;
     const uint32_t ctas = BN == 256 ? std::min(g.total, (uint32_t)sm_count) : g.total;
     launch_pdl(linear_tc5_kernel<BN, AR>, ctas, LT_THREADS, LtSmem<BN, AR>::ALLOC, st, tm_x, tm_w, a, g);
     if (splits > 1) launch_pdl(linear_finish_kernel<BN>, (a.n_rows / 4 * a.T * a.n_batch + 255) / 256, 256, 0, st, a, g);
@@ -466,12 +529,12 @@ void launch_gemv_act(const LinArgs &a, int sm_count, cudaStream_t st) {
     uint32_t G = 32;
     while (G > 4 && a.kp / 8 <= G / 2) G /= 2;
     uint32_t KS = 1;
-    const uint32_t pairs = a.n_rows / 2 * a.n_batch;
+    const uint32_t n_z = a.row_batch ? a.T : a.n_batch, pairs = a.n_rows / 2 * n_z;
     if (G == 32)
         while (KS < 8 && pairs * KS * 2 <= (uint32_t)sm_count * 64 && a.kp / 8 >= 32 * KS * 2) KS *= 2;
     const uint32_t units = KS > 1 ? 8 / KS : 8 * (32 / G);
-    const dim3 grid((a.n_rows / 2 + units - 1) / units, 1, a.n_batch);
-    switch (a.T) {
+    const dim3 grid((a.n_rows / 2 + units - 1) / units, 1, n_z);
+    switch (a.row_batch ? 1 : a.T) {
     case 1: launch_pdl(gemv_act_kernel<TA, 1>, grid, GV_THREADS, 0, st, a, G, KS); break;
     case 2: launch_pdl(gemv_act_kernel<TA, 2>, grid, GV_THREADS, 0, st, a, G, KS); break;
     case 3: launch_pdl(gemv_act_kernel<TA, 3>, grid, GV_THREADS, 0, st, a, G, KS); break;
@@ -495,7 +558,17 @@ cudaError_t linear_configure() {
 
 uint32_t launch_linear(const LinArgs &a, bool f32, int sm_count, cudaStream_t st) {
     if (!a.T || !a.n_rows) return 1;
-    if (a.T <= GV_MAX_TOKENS) {
+    if (a.tiles) {
+        if (f32) {
+            launch_pdl(linear_simt_kernel<float>, dim3((a.n_rows + 63) / 64, a.max_tiles, 1), 256, 0, st, a);
+            return 1;
+        }
+        if (a.tile_rows == 16) return launch_tc5<128, 16>(a, sm_count, st);
+        if (a.tile_rows == 64) return launch_tc5<128, 64>(a, sm_count, st);
+        // (the real number of tiles is near the lower bound when tiles are full)
+        return (a.n_rows + 255) / 256 * (a.T / LT_M + 1) >= (uint32_t)sm_count ? launch_tc5<256, 128>(a, sm_count, st) : launch_tc5<128, 128>(a, sm_count, st);
+    }
+    if (a.T <= GV_MAX_TOKENS || a.row_batch) {
         if (f32) launch_gemv_act<float>(a, sm_count, st);
         else launch_gemv_act<__nv_bfloat16>(a, sm_count, st);
         return 1;
@@ -518,6 +591,11 @@ uint32_t launch_linear(const LinArgs &a, bool f32, int sm_count, cudaStream_t st
     if (ctas(128) >= sms) return launch_tc5<128, 128>(a, sm_count, st);
     if (ctas(64) >= sms) return launch_tc5<64, 128>(a, sm_count, st);
     return launch_tc5<32, 128>(a, sm_count, st);
+}
+
+uint32_t linear_tile_rows(uint32_t rows, uint32_t batches, bool f32) {
+    if (f32) return 64;
+    return rows <= 12 * batches ? 16 : rows <= 48 * batches ? 64 : 128;
 }
 
 size_t linear_split_bytes() { return (size_t)LT_SPLIT_CTAS * LT_SPLIT_TOKENS * 128 * 4; }

@@ -8,57 +8,21 @@
 
 #include <algorithm>
 
-#include "layered.h"
-#include "pdl.cuh"
+#include "mixers_common.cuh"
 
 namespace ob {
 
 namespace {
 
-using bf16 = __nv_bfloat16;
-
-template <typename TA> __device__ __forceinline__ TA to_act(float v);
-template <> __device__ __forceinline__ float to_act<float>(float v) { return v; }
-template <> __device__ __forceinline__ bf16 to_act<bf16>(float v) { return __float2bfloat16_rn(v); }
-__device__ __forceinline__ float from_act(float v) { return v; }
-__device__ __forceinline__ float from_act(bf16 v) { return __bfloat162float(v); }
-
-// Sum over the CTA; every thread gets it.  red: 33 floats.
-__device__ __forceinline__ float block_sum(float v, float *red) {
-    v = warp_sum(v);
-    __syncthreads();
-    if ((threadIdx.x & 31) == 0) red[threadIdx.x >> 5] = v;
-    __syncthreads();
-    if (threadIdx.x < 32) {
-        float s = threadIdx.x < blockDim.x / 32 ? red[threadIdx.x] : 0.0f;
-        s = warp_sum(s);
-        if (threadIdx.x == 0) red[32] = s;
-    }
-    __syncthreads();
-    return red[32];
-}
-
-__device__ __forceinline__ float inv_rms(float sum_sq, uint32_t n, float eps) { return 1.0f / sqrtf(sum_sq / (float)n + eps); }
-
 // (No __restrict__ on what an earlier kernel writes: a load the compiler may take for invariant could move above pdl_wait.)
 // ---- embedding, norms ------------------------------------------------------------------------------------------------------
-// A row of activations from four fp32 values per thread and step.
-template <typename TA> __device__ __forceinline__ void store4(TA *p, float4 v);
-template <> __device__ __forceinline__ void store4<float>(float *p, float4 v) { *reinterpret_cast<float4 *>(p) = v; }
-template <> __device__ __forceinline__ void store4<bf16>(bf16 *p, float4 v) {
-    const __nv_bfloat162 lo = __floats2bfloat162_rn(v.x, v.y), hi = __floats2bfloat162_rn(v.z, v.w);
-    *reinterpret_cast<uint2 *>(p) = make_uint2(*reinterpret_cast<const uint32_t *>(&lo), *reinterpret_cast<const uint32_t *>(&hi));
-}
-__device__ __forceinline__ float sq4(float4 v) { return v.x * v.x + v.y * v.y + v.z * v.z + v.w * v.w; }
-__device__ __forceinline__ float4 mul4(float4 v, float f) { return make_float4(v.x * f, v.y * f, v.z * f, v.w * f); }
-
 // A row in registers: element group i of a thread is columns 4 (threadIdx + i blockDim) .. + 3; NV = 0: any width, one column
 // at a time through memory.
 constexpr int ROW_VECS = 4;
 
-// x = the token's embedding, h = x / rms(x) * gain.
+// x = the token's embedding, h = x / rms(x) * gain or x.
 template <typename TA, int NV>
-__global__ void __launch_bounds__(1024) embed_norm_kernel(const bf16 *table, uint32_t width, const uint32_t *tokens, float *x, float eps, float gain, TA *h, uint32_t h_pitch) {
+__global__ void __launch_bounds__(1024) embed_kernel(const bf16 *table, uint32_t width, const uint32_t *tokens, float *x, bool normed, float eps, float gain, TA *h, uint32_t h_pitch) {
     __shared__ float red[33];
     pdl_release();
     pdl_wait();
@@ -77,7 +41,7 @@ __global__ void __launch_bounds__(1024) embed_norm_kernel(const bf16 *table, uin
             *reinterpret_cast<float4 *>(xr + c) = v[i];
             s += sq4(v[i]);
         }
-        const float f = inv_rms(block_sum(s, red), width, eps) * gain;
+        const float f = normed ? inv_rms(block_sum(s, red), width, eps) * gain : 1.0f;
 #pragma unroll
         for (int i = 0; i < NV; ++i) {
             const uint32_t c = 4 * (threadIdx.x + i * blockDim.x);
@@ -89,13 +53,13 @@ __global__ void __launch_bounds__(1024) embed_norm_kernel(const bf16 *table, uin
             xr[i] = v;
             s += v * v;
         }
-        const float f = inv_rms(block_sum(s, red), width, eps) * gain;
+        const float f = normed ? inv_rms(block_sum(s, red), width, eps) * gain : 1.0f;
         for (uint32_t i = threadIdx.x; i < width; i += blockDim.x) hr[i] = to_act<TA>(xr[i] * f);
     }
 }
 
 template <typename TA, int NV>
-__global__ void __launch_bounds__(1024) norm_scalar_kernel(const float *x, uint32_t width, const uint32_t *rows, float eps, float gain, TA *h, uint32_t h_pitch) {
+__global__ void __launch_bounds__(1024) norm_kernel(const float *x, uint32_t width, const uint32_t *rows, float eps, float gain, const float *w, TA *h, uint32_t h_pitch) {
     __shared__ float red[33];
     pdl_release();
     pdl_wait();
@@ -114,12 +78,18 @@ __global__ void __launch_bounds__(1024) norm_scalar_kernel(const float *x, uint3
 #pragma unroll
         for (int i = 0; i < NV; ++i) {
             const uint32_t c = 4 * (threadIdx.x + i * blockDim.x);
-            if (c < width) store4<TA>(hr + c, mul4(v[i], f));
+            if (c >= width) continue;
+            float4 o = mul4(v[i], f);
+            if (w) {
+                const float4 g = *reinterpret_cast<const float4 *>(w + c);
+                o = make_float4(o.x * g.x, o.y * g.y, o.z * g.z, o.w * g.w);
+            }
+            store4<TA>(hr + c, o);
         }
     } else {
         for (uint32_t i = threadIdx.x; i < width; i += blockDim.x) s += row[i] * row[i];
         const float f = inv_rms(block_sum(s, red), width, eps) * gain;
-        for (uint32_t i = threadIdx.x; i < width; i += blockDim.x) hr[i] = to_act<TA>(row[i] * f);
+        for (uint32_t i = threadIdx.x; i < width; i += blockDim.x) hr[i] = to_act<TA>(row[i] * f * (w ? w[i] : 1.0f));
     }
 }
 
@@ -172,17 +142,69 @@ __global__ void __launch_bounds__(1024) side_finish_kernel(float *x, const float
     }
 }
 
-// ---- rotation ----------------------------------------------------------------------------------------------------------------
-// Value d of the rotated vector whose unrotated values are v[0..]; cs: this position's (cos, sin) row.
-__device__ __forceinline__ float rotated(const float *v, uint32_t d, const Rot &r, const float2 *cs) {
-    if (d >= r.dims) return v[d];
-    const uint32_t half = r.dims / 2;
-    if (r.interleaved) {
-        const float2 c = cs[d >> 1];
-        return d & 1 ? v[d] * c.x + v[d - 1] * c.y : v[d] * c.x - v[d + 1] * c.y;
+// x += mult * y / rms(y) * w, h = x; y is the sum of a token's `top` rows.
+template <typename TA, int NV>
+__global__ void __launch_bounds__(1024) post_norm_kernel(PostNormArgs a) {
+    __shared__ float red[33];
+    pdl_release();
+    pdl_wait();
+    float *xr = a.x + (uint64_t)blockIdx.x * a.width;
+    TA *hr = a.h ? static_cast<TA *>(a.h) + (uint64_t)blockIdx.x * a.h_pitch : nullptr;
+    auto row = [&](uint32_t i) {
+        const uint32_t p = blockIdx.x * a.top + i;
+        return a.y + (uint64_t)(a.rows ? a.rows[p] : p) * a.width;
+    };
+    if (a.zero && blockIdx.x == 0)
+        for (uint32_t i = threadIdx.x; i < a.n_zero; i += blockDim.x) a.zero[i] = 0;
+    float s = 0.0f;
+    if constexpr (NV > 0) {
+        float4 yv[NV], v[NV], wv[NV];
+#pragma unroll
+        for (int i = 0; i < NV; ++i) {
+            const uint32_t c = 4 * (threadIdx.x + i * blockDim.x);
+            const bool in = c < a.width;
+            yv[i] = in ? *reinterpret_cast<const float4 *>(row(0) + c) : make_float4(0, 0, 0, 0);
+            v[i] = in ? *reinterpret_cast<const float4 *>(xr + c) : make_float4(0, 0, 0, 0);
+            wv[i] = in ? *reinterpret_cast<const float4 *>(a.w + c) : make_float4(0, 0, 0, 0);
+        }
+        for (uint32_t k = 1; k < a.top; ++k) {
+            const float *y = row(k);
+#pragma unroll
+            for (int i = 0; i < NV; ++i) {
+                const uint32_t c = 4 * (threadIdx.x + i * blockDim.x);
+                if (c >= a.width) continue;
+                const float4 u = *reinterpret_cast<const float4 *>(y + c);
+                yv[i].x += u.x, yv[i].y += u.y, yv[i].z += u.z, yv[i].w += u.w;
+            }
+        }
+#pragma unroll
+        for (int i = 0; i < NV; ++i) s += sq4(yv[i]);
+        const float f = inv_rms(block_sum(s, red), a.width, a.eps) * a.mult;
+#pragma unroll
+        for (int i = 0; i < NV; ++i) {
+            const uint32_t c = 4 * (threadIdx.x + i * blockDim.x);
+            if (c >= a.width) continue;
+            v[i].x += yv[i].x * f * wv[i].x, v[i].y += yv[i].y * f * wv[i].y, v[i].z += yv[i].z * f * wv[i].z, v[i].w += yv[i].w * f * wv[i].w;
+            *reinterpret_cast<float4 *>(xr + c) = v[i];
+            if (hr) store4<TA>(hr + c, v[i]);
+        }
+    } else {
+        auto sum = [&](uint32_t c) {
+            float v = row(0)[c];
+            for (uint32_t k = 1; k < a.top; ++k) v += row(k)[c];
+            return v;
+        };
+        for (uint32_t c = threadIdx.x; c < a.width; c += blockDim.x) {
+            const float v = sum(c);
+            s += v * v;
+        }
+        const float f = inv_rms(block_sum(s, red), a.width, a.eps) * a.mult;
+        for (uint32_t c = threadIdx.x; c < a.width; c += blockDim.x) {
+            const float v = xr[c] + sum(c) * f * a.w[c];
+            xr[c] = v;
+            if (hr) hr[c] = to_act<TA>(v);
+        }
     }
-    const float2 c = cs[d < half ? d : d - half];
-    return d < half ? v[d] * c.x - v[d + half] * c.y : v[d] * c.x + v[d - half] * c.y;
 }
 
 // ---- latent attention: what a token leaves in the cache, and its rotated query parts -----------------------------------------------
@@ -216,9 +238,6 @@ __global__ void __launch_bounds__(256) latent_prep_kernel(LatentArgs a) {
     const float f = inv_rms(block_sum(s, red), a.kv_rank, a.eps);
     for (uint32_t i = threadIdx.x; i < a.kv_rank; i += blockDim.x) row[i] = to_act<TA>(lat[i] * f * a.kv_norm[i]);
 }
-
-// First position row t of a sequence sees.
-__device__ __forceinline__ uint32_t first_seen(uint32_t pos, uint32_t window) { return window && pos + 1 > window ? pos + 1 - window : 0u; }
 
 // ---- latent attention, plain form: one CTA per (token, head), any sizes; fp32 throughout when the cache is fp32 ---------------------
 // Keys in blocks of 128: scores by the warps (lanes over the row), online softmax, then every thread adds up its own columns.
@@ -297,30 +316,6 @@ struct LmPlan {
     }
 };
 
-__device__ __forceinline__ uint32_t smem_addr(const void *p) { return (uint32_t)__cvta_generic_to_shared(p); }
-__device__ __forceinline__ void cp16(uint32_t dst, const void *src, bool in) {  // 16 bytes, or zeros
-    asm volatile("cp.async.cg.shared.global [%0], [%1], 16, %2;" ::"r"(dst), "l"(src), "r"(in ? 16 : 0) : "memory");
-}
-__device__ __forceinline__ void cp_commit() { asm volatile("cp.async.commit_group;" ::: "memory"); }
-template <int N> __device__ __forceinline__ void cp_wait() { asm volatile("cp.async.wait_group %0;" ::"n"(N) : "memory"); }
-__device__ __forceinline__ void ldsm4(uint32_t (&r)[4], uint32_t addr) {
-    asm volatile("ldmatrix.sync.aligned.m8n8.x4.shared.b16 {%0, %1, %2, %3}, [%4];" : "=r"(r[0]), "=r"(r[1]), "=r"(r[2]), "=r"(r[3]) : "r"(addr) : "memory");
-}
-__device__ __forceinline__ void ldsm4t(uint32_t (&r)[4], uint32_t addr) {
-    asm volatile("ldmatrix.sync.aligned.m8n8.x4.trans.shared.b16 {%0, %1, %2, %3}, [%4];" : "=r"(r[0]), "=r"(r[1]), "=r"(r[2]), "=r"(r[3]) : "r"(addr) : "memory");
-}
-__device__ __forceinline__ void mma_bf16(float (&c)[4], const uint32_t (&a)[4], uint32_t b0, uint32_t b1) {
-    asm("mma.sync.aligned.m16n8k16.row.col.f32.bf16.bf16.f32 {%0, %1, %2, %3}, {%4, %5, %6, %7}, {%8, %9}, {%0, %1, %2, %3};"
-                 : "+f"(c[0]), "+f"(c[1]), "+f"(c[2]), "+f"(c[3])
-                 : "r"(a[0]), "r"(a[1]), "r"(a[2]), "r"(a[3]), "r"(b0), "r"(b1));
-}
-
-__device__ __forceinline__ float pow2(float x) {  // relative error below 2^-22; 0 for -inf
-    float y;
-    asm("ex2.approx.ftz.f32 %0, %1;" : "=f"(y) : "f"(x));
-    return y;
-}
-
 // How a warp copies rows of `chunks` 16-byte pieces: several short rows at a time, or one row in steps of 32 pieces.
 struct RowCopy {
     uint32_t rows, row, chunk, chunks;  // rows per step of a warp, this lane's row among them and its first piece (chunks: none)
@@ -331,30 +326,6 @@ struct RowCopy {
         chunk = n >= 32 ? lane : row < rows ? lane - row * n : n;
     }
 };
-
-// The tile'th group of `rows` (token, head) rows: its span and first row within the span.  One warp; every lane gets the answer.
-__device__ __forceinline__ void find_tile(const RowSpan *spans, uint32_t n_seq, uint32_t n_head, uint32_t rows, uint32_t tile, RowSpan *span, uint32_t *first) {
-    const uint32_t lane = threadIdx.x & 31;
-    for (uint32_t s0 = 0;; s0 += 32) {
-        const RowSpan sp = s0 + lane < n_seq ? spans[s0 + lane] : RowSpan{0, 0};
-        const uint32_t n = (sp.n * n_head + rows - 1) / rows;
-        uint32_t sum = n;
-#pragma unroll
-        for (int o = 1; o < 32; o <<= 1) {
-            const uint32_t up = __shfl_up_sync(0xffffffffu, sum, o);
-            if (lane >= o) sum += up;
-        }
-        const uint32_t hit = __ballot_sync(0xffffffffu, tile < sum);
-        if (hit || s0 + 32 >= n_seq) {
-            const int src = hit ? __ffs(hit) - 1 : 31;
-            span->row0 = __shfl_sync(0xffffffffu, sp.row0, src);
-            span->n = hit ? __shfl_sync(0xffffffffu, sp.n, src) : 0;
-            *first = (tile - __shfl_sync(0xffffffffu, sum - n, src)) * rows;
-            return;
-        }
-        tile -= __shfl_sync(0xffffffffu, sum, 31);
-    }
-}
 
 // NP: shares of sixteen latent columns per warp; a warp whose last share does not exist repeats another and drops it.
 template <int MT, int NP>
@@ -1125,25 +1096,28 @@ struct RowShape {
     }
 };
 template <typename TA>
-static void embed_norm(const bf16 *table, uint32_t width, const uint32_t *tokens, uint32_t T, float *x, float eps, float gain, void *h, uint32_t h_pitch, cudaStream_t st) {
+static void embed(const bf16 *table, uint32_t width, const uint32_t *tokens, uint32_t T, float *x, bool normed, float eps, float gain, void *h, uint32_t h_pitch, cudaStream_t st) {
     const RowShape r(width, T);
-    if (r.vec) launch_pdl(embed_norm_kernel<TA, ROW_VECS>, T, r.threads, 0, st, table, width, tokens, x, eps, gain, static_cast<TA *>(h), h_pitch);
-    else launch_pdl(embed_norm_kernel<TA, 0>, T, r.threads, 0, st, table, width, tokens, x, eps, gain, static_cast<TA *>(h), h_pitch);
+    launch_pdl(r.vec ? embed_kernel<TA, ROW_VECS> : embed_kernel<TA, 0>, T, r.threads, 0, st, table, width, tokens, x, normed, eps, gain, static_cast<TA *>(h), h_pitch);
 }
-void launch_embed_norm(const bf16 *table, uint32_t width, const uint32_t *tokens, uint32_t T, float *x, float eps, float gain, void *h, uint32_t h_pitch, bool f32,
-                       cudaStream_t st) {
-    if (f32) embed_norm<float>(table, width, tokens, T, x, eps, gain, h, h_pitch, st);
-    else embed_norm<bf16>(table, width, tokens, T, x, eps, gain, h, h_pitch, st);
+void launch_embed(const bf16 *table, uint32_t width, const uint32_t *tokens, uint32_t T, float *x, bool normed, float eps, float gain, void *h, uint32_t h_pitch, bool f32,
+                  cudaStream_t st) {
+    if (f32) embed<float>(table, width, tokens, T, x, normed, eps, gain, h, h_pitch, st);
+    else embed<bf16>(table, width, tokens, T, x, normed, eps, gain, h, h_pitch, st);
 }
 template <typename TA>
-static void norm_scalar(const float *x, uint32_t width, const uint32_t *rows, uint32_t n, float eps, float gain, void *h, uint32_t h_pitch, cudaStream_t st) {
+static void norm(const float *x, uint32_t width, const uint32_t *rows, uint32_t n, float eps, float gain, const float *w, void *h, uint32_t h_pitch, cudaStream_t st) {
     const RowShape r(width, n);
-    if (r.vec) launch_pdl(norm_scalar_kernel<TA, ROW_VECS>, n, r.threads, 0, st, x, width, rows, eps, gain, static_cast<TA *>(h), h_pitch);
-    else launch_pdl(norm_scalar_kernel<TA, 0>, n, r.threads, 0, st, x, width, rows, eps, gain, static_cast<TA *>(h), h_pitch);
+    launch_pdl(r.vec ? norm_kernel<TA, ROW_VECS> : norm_kernel<TA, 0>, n, r.threads, 0, st, x, width, rows, eps, gain, w, static_cast<TA *>(h), h_pitch);
 }
-void launch_norm_scalar(const float *x, uint32_t width, const uint32_t *rows, uint32_t n, float eps, float gain, void *h, uint32_t h_pitch, bool f32, cudaStream_t st) {
-    if (f32) norm_scalar<float>(x, width, rows, n, eps, gain, h, h_pitch, st);
-    else norm_scalar<bf16>(x, width, rows, n, eps, gain, h, h_pitch, st);
+void launch_norm(const float *x, uint32_t width, const uint32_t *rows, uint32_t n, float eps, float gain, const float *w, void *h, uint32_t h_pitch, bool f32, cudaStream_t st) {
+    if (f32) norm<float>(x, width, rows, n, eps, gain, w, h, h_pitch, st);
+    else norm<bf16>(x, width, rows, n, eps, gain, w, h, h_pitch, st);
+}
+void launch_post_norm(const PostNormArgs &a, bool f32, cudaStream_t st) {
+    const RowShape r(a.width, a.T);
+    if (f32) launch_pdl(r.vec ? post_norm_kernel<float, ROW_VECS> : post_norm_kernel<float, 0>, a.T, r.threads, 0, st, a);
+    else launch_pdl(r.vec ? post_norm_kernel<bf16, ROW_VECS> : post_norm_kernel<bf16, 0>, a.T, r.threads, 0, st, a);
 }
 template <typename TA>
 static void side_finish(float *x, const float *y, const float *w, uint32_t width, uint32_t T, float eps, float gain, void *h, uint32_t h_pitch, cudaStream_t st) {

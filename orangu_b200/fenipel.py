@@ -4,41 +4,10 @@ gated feed-forward, followed by a per-layer token input; norms of the residual h
 Reads the design's config.json and tensors into ``ob_layered_desc``; what runs is the library's layered model."""
 from __future__ import annotations
 
-import json
-import os
-
-import numpy as np
-
 from . import capi
-from .layered import Describer, LayeredModel
-from .safetensors import SafetensorsFile
+from .layered import Describer, LayeredModel, tensor_source
 
 GLU_ALPHA = 1.702  # slope of the sigmoid in the feed-forward's gate, fixed by the design
-
-
-class TensorDict:
-    """The reader's interface over a dict: uint16 arrays are bfloat16 bits, other arrays floats."""
-
-    def __init__(self, tensors: dict):
-        from .safetensors import from_bf16, to_bf16
-
-        self._t, self._from, self._to = tensors, from_bf16, to_bf16
-
-    def _get(self, name, shape):
-        if name not in self._t:
-            raise ValueError(f"no tensor {name}")
-        a = np.asarray(self._t[name])
-        if shape is not None and a.shape != tuple(shape):
-            raise ValueError(f"{name} is {list(a.shape)}, expected {list(shape)}")
-        return a
-
-    def bf16(self, name, shape=None):
-        a = self._get(name, shape)
-        return a if a.dtype == np.uint16 else self._to(a)
-
-    def f32(self, name, shape=None):
-        a = self._get(name, shape)
-        return self._from(a) if a.dtype == np.uint16 else np.array(a, np.float32, order="C")
 
 
 def _latent_attention(d: Describer, t, at: str, mx: dict, width: int) -> capi.MixerDesc:
@@ -84,9 +53,7 @@ class FenipelModel(LayeredModel):
 
     def __init__(self, backend, config: dict, tensors, dtype: str = "bfloat16", max_seq_len: int = 4096, max_batch_tokens: int = 512,
                  kv_pool_tokens: int = 0, state_slots: int = 0):
-        if dtype not in ("bfloat16", "float32"):
-            raise ValueError(f"dtype {dtype}: bfloat16 or float32")
-        t = TensorDict(tensors) if isinstance(tensors, dict) else tensors
+        t = tensor_source(tensors)
         d, width, vocab = Describer(), config["width"], config["vocab"]
         side = config.get("token_side")
         side_dim = side["dim"] if side else 0
@@ -94,8 +61,7 @@ class FenipelModel(LayeredModel):
         desc = capi.LayeredDesc()
         desc.n_vocab, desc.n_embd, desc.n_layer, desc.side_dim = vocab, width, len(blocks), side_dim
         desc.rms_eps, desc.final_gain = config["norm"]["eps"], float(t.f32("final.norm", ()).reshape(()))
-        desc.compute_f32 = dtype == "float32"
-        desc.max_seq_len, desc.max_batch_tokens, desc.kv_pool_tokens, desc.n_state_slots = max_seq_len, max_batch_tokens, kv_pool_tokens, state_slots
+        self.size(desc, dtype, max_seq_len, max_batch_tokens, kv_pool_tokens, state_slots)
         desc.token_embd = d.matrix(t.bf16("embed", (vocab, width)))
         desc.output = d.matrix(t.bf16("head", (vocab, width)))
         if side_dim:
@@ -124,9 +90,3 @@ class FenipelModel(LayeredModel):
             b.side_proj = d.matrix(t.bf16(at + "side.proj", (width, side_dim)))
             b.side_norm = d.vector(t.f32(at + "side.norm", (width,)))
         return b
-
-    @classmethod
-    def from_folder(cls, backend, path: str, **sizing) -> "FenipelModel":
-        with open(os.path.join(path, "config.json")) as f:
-            config = json.load(f)
-        return cls(backend, config, SafetensorsFile(os.path.join(path, "model.safetensors")), **sizing)

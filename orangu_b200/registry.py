@@ -6,9 +6,10 @@ import os
 
 from .fenipel import FenipelModel
 from .model import LlamaModel
+from .nenodra import NenodraModel
 
 GGUF_ARCHITECTURES = {a: LlamaModel for a in ("llama", "mistral", "qwen2", "qwen3", "qwen3vl")}
-FOLDER_ARCHITECTURES = {FenipelModel.ARCHITECTURE: FenipelModel}
+FOLDER_ARCHITECTURES = {m.ARCHITECTURE: m for m in (FenipelModel, NenodraModel)}
 
 
 def model_class(path: str):
