@@ -7,7 +7,7 @@ import pytest
 
 import fenipel_make as F
 import fenipel_plain as P
-from gpu_common import backend  # noqa: F401
+from gpu_common import backend, error, greedy_plain, run  # noqa: F401
 
 pytestmark = pytest.mark.gpu
 DTYPES = ("float32", "bfloat16")
@@ -18,22 +18,6 @@ def make(backend, cfg, w, dtype, pool=512, rows=256, slots=4, seq=None):
     from orangu_b200.fenipel import FenipelModel
 
     return FenipelModel(backend, cfg, w, dtype=dtype, max_seq_len=seq or pool, max_batch_tokens=rows, kv_pool_tokens=pool, state_slots=slots)
-
-
-def error(got, want):
-    """Worst position: root mean square of the difference over the root mean square of all expected values."""
-    got, want = np.asarray(got, np.float64), np.asarray(want, np.float64)
-    assert got.shape == want.shape and np.isfinite(got).all()
-    return float(np.sqrt(((got - want) ** 2).mean(-1)).max() / np.sqrt((want ** 2).mean()))
-
-
-def run(model, kv, toks, cuts=()):
-    """Logits at every position, the tokens fed in portions that end at `cuts`."""
-    out, at = [], 0
-    for end in list(cuts) + [len(toks)]:
-        out.append(model.forward_rows([kv], [toks[at:end]], range(end - at)))
-        at = end
-    return np.concatenate(out)
 
 
 # ---- mechanisms ------------------------------------------------------------------------------------------------------------
@@ -311,18 +295,6 @@ def test_far_token_through_retention(backend, dtype):
 
 
 # ---- decoding ------------------------------------------------------------------------------------------------------------------------
-def greedy_plain(cfg, v, prompt, n):
-    """Greedy continuation by the plain statement and, per step, how far the best token is ahead of the next."""
-    toks, out, lead = list(prompt), [], []
-    for _ in range(n):
-        lg = P.forward(cfg, v, toks)[0][-1]
-        top = np.sort(lg)[-2:]
-        lead.append(top[1] - top[0])
-        out.append(int(np.argmax(lg)))
-        toks.append(out[-1])
-    return out, min(lead)
-
-
 def test_long_decoding(backend):
     """Hundreds of decoded tokens through captured graphs; the plain statement then judges every choice at once."""
     w = F.weights(MIX, 91)
@@ -357,7 +329,7 @@ def test_generation_through_scheduler_and_files(backend, tmp_path):
     prompts = [F.tokens(MIX, n, 102 + n) for n in (45, 2, 17, 33, 8)]
     got = generate(m, prompts, 12, prefill_batch=10)
     for p, g in zip(prompts, got):
-        want, lead = greedy_plain(MIX, F.values(w), p, 12)
+        want, lead = greedy_plain(P, MIX, F.values(w), p, 12)
         assert lead > 1e-4 and g == want  # seeds chosen so that no two tokens tie within rounding
     assert (m.free_pages, m.free_slots) == (32, 5)
     # repeat penalty: the penalised argmax of the logits without it
