@@ -67,6 +67,10 @@ def parse_args():
                     "(1b, 8b; random weights) beside the quantized Llama shape of the same widths")
     ap.add_argument("--fenipel-layers", type=int, default=8, help="layers of both models in that comparison")
     ap.add_argument("--fenipel-only", action="store_true", help="leave the Llama shape out")
+    ap.add_argument("--nenodra", default="", metavar="SIZE[,SIZE]", help="instead of the workload above: prefill and decode of Nenodra at these sizes "
+                    "(1b, 8b; random weights) beside Fenipel at the same widths")
+    ap.add_argument("--nenodra-layers", type=int, default=8, help="layers of both models in that comparison")
+    ap.add_argument("--nenodra-only", action="store_true", help="leave Fenipel out")
     return ap.parse_args()
 
 
@@ -331,20 +335,33 @@ FENIPEL_SIZES = {  # widths and feed-forwards of the Llama shapes of the same na
 }
 
 
+def random_matrices():
+    """lin(rows, columns): bfloat16 bits of normal values over the root of the columns (or times std), all dealt out from one pool."""
+    import numpy as np
+    from orangu_b200.safetensors import to_bf16
+
+    pool = np.random.default_rng(1).normal(size=1 << 22).astype(np.float32)
+    cache, turn = {}, [0]
+
+    def lin(o, i, std=None):
+        std = i ** -0.5 if std is None else std
+        if std not in cache:
+            cache[std] = to_bf16(pool * std)
+        bits = cache[std]
+        turn[0] += 1
+        return np.resize(np.roll(bits, (turn[0] * 104729) % bits.size), (o, i))
+
+    return lin
+
+
 def fenipel_model(size: str, n_layer: int):
-    """Configuration and random bfloat16 tensors (bits); one pool of normal values is dealt out over all of them."""
+    """Configuration and random bfloat16 tensors (bits)."""
     import numpy as np
     from orangu_b200.safetensors import to_bf16
 
     z = FENIPEL_SIZES[size]
     E, V, sd = z["width"], z["vocab"], z["side"]
-    pool = np.random.default_rng(1).normal(size=1 << 22).astype(np.float32)
-    cache = {}
-
-    def lin(o, i):
-        bits = cache.setdefault(i, to_bf16(pool * i ** -0.5))
-        return np.resize(np.roll(bits, (o * 7919) % bits.size), (o, i))
-
+    lin = random_matrices()
     layers, t = [], {"embed": lin(V, E), "head": lin(V, E), "final.norm": to_bf16(np.float32(1)), "side.embed": lin(V, n_layer * sd)}
     for n in range(n_layer):
         at, m = f"l{n}.mix.", dict(z["latent" if n % 2 == 0 else "retention"])
@@ -363,9 +380,49 @@ def fenipel_model(size: str, n_layer: int):
     return {"architecture": "Fenipel", "vocab": V, "width": E, "norm": {"eps": 1e-6}, "token_side": {"dim": sd}, "layers": layers}, t
 
 
-def time_model(be, model, vocab: int, weight_bytes: int, cache_bytes_per_token: float, flops_per_token: float, steps: int, warmup: int, prompt: int = 4096):
+NENODRA_SIZES = {  # Fenipel's widths; half of the layers have two maps and a dense feed-forward, half are gated with experts
+    "1b": {"width": 2048, "ff": 8192, "vocab": 32768, "experts": 16, "top": 2, "expert_ff": 1024,
+           "attention": {"heads": 16, "kv_heads": 4, "dim": 64, "vdim": 128, "diff": 0.5}, "attention_2": {"heads": 16, "kv_heads": 4, "dim": 128, "vdim": 128}, "window": 1024},
+    "8b": {"width": 4096, "ff": 14336, "vocab": 32768, "experts": 16, "top": 2, "expert_ff": 2048,
+           "attention": {"heads": 32, "kv_heads": 8, "dim": 64, "vdim": 128, "diff": 0.5}, "attention_2": {"heads": 32, "kv_heads": 8, "dim": 128, "vdim": 128}, "window": 1024},
+}
+
+
+def nenodra_model(size: str, n_layer: int):
+    """Configuration and random bfloat16 tensors (bits)."""
+    import numpy as np
+    from orangu_b200.safetensors import to_bf16
+
+    z = NENODRA_SIZES[size]
+    E, V = z["width"], z["vocab"]
+    lin, const = random_matrices(), lambda v, n: to_bf16(np.full(n, v, np.float32))
+    layers, t = [], {"embed": lin(V, E, 4.0), "head": lin(V, E), "final.norm": const(0, E)}  # (tokens differ enough to choose different experts)
+    for n in range(n_layer):
+        kind = "attention" if n % 2 == 0 else "attention_2"
+        at, m = f"l{n}.mix.", dict(z[kind], mask={"size": z["window"]})
+        H, G, d, v, maps = m["heads"], m["kv_heads"], m["dim"], m["vdim"], 2 - n % 2
+        m.update(rot={"base": 10000.0, "dims": d}, scale=d ** -0.5)
+        t.update({at + "q": lin(H * maps * d, E), at + "k": lin(G * maps * d, E), at + "q.norm": const(1, d), at + "k.norm": const(1, d), at + "o": lin(E, H * v),
+                  f"l{n}.norm1": const(0, E), f"l{n}.norm2": const(0, E)})
+        if maps == 2:
+            t.update({at + "v": lin(G * v, E), at + "q.b": const(0.1, H * 2 * d), at + "k.b": const(0.1, G * 2 * d), at + "v.b": const(0.1, G * v), at + "o.b": const(0.1, E)})
+            t.update({at + x: const(0.05, d) for x in ("lq1", "lk1", "lq2", "lk2")})
+            t.update({f"l{n}.mlp.up": lin(z["ff"], E), f"l{n}.mlp.down": lin(E, z["ff"])})
+            mlp = {"kind": "dense", "ff": z["ff"]}
+        else:
+            X, ff = z["experts"], z["expert_ff"]
+            t.update({at + "g": lin(H * v, E), f"l{n}.mlp.router": lin(X, E)})
+            for e in range(X):
+                t.update({f"l{n}.mlp.e{e}.gate": lin(ff, E), f"l{n}.mlp.e{e}.up": lin(ff, E), f"l{n}.mlp.e{e}.down": lin(E, ff)})
+            mlp = {"kind": "moe", "router": {"experts": X, "top": z["top"]}, "expert": {"ff": ff}}
+        layers.append({"type": kind, "mixer": m, "mlp": mlp})
+    return {"architecture": "Nenodra", "vocab": V, "width": E, "norm": {"eps": 1e-6}, "residual_mult": 1.0, "logit_scale": 1.0, "layers": layers}, t
+
+
+def time_model(be, model, vocab: int, weight_bytes, cache_bytes_per_token: float, flops_per_token: float, steps: int, warmup: int, prompt: int = 4096):
     """Prefill of one prompt and greedy decode loops at batch 1, 8 and 64 (device time, CUDA events; weights exceed L2).
-    cache_bytes_per_token: cache and state traffic of one decoded token at this context."""
+    weight_bytes: read per decoded step, a number or a function of the batch.  cache_bytes_per_token: cache and state traffic of
+    one decoded token at this context."""
     import numpy as np
 
     rng = np.random.default_rng(0)
@@ -391,11 +448,69 @@ def time_model(be, model, vocab: int, weight_bytes: int, cache_bytes_per_token: 
         model.decode_loop(kvs[:batch], first, warmup)
         model.decode_loop(kvs[:batch], first, steps)
         t = be.last_device_ms() / steps
-        need = weight_bytes + batch * cache_bytes_per_token
+        need = (weight_bytes(batch) if callable(weight_bytes) else weight_bytes) + batch * cache_bytes_per_token
         out["decode"][str(batch)] = {"ms_per_step": t, "tok_s": batch / t * 1e3, "bytes_per_step": need, "of_hbm": need / (t * 1e-3) / (hbm * 1e9)}
     for k in kvs:
         k.close()
     return out
+
+
+def time_fenipel(be, size: str, L: int, steps: int, warmup: int):
+    import orangu_b200
+
+    cfg, t = fenipel_model(size, L)
+    n = sum(a.size for k, a in t.items() if not k.endswith("embed"))
+    z, prompt = FENIPEL_SIZES[size], 4096
+    la, re = z["latent"], z["retention"]
+    win = min(la["window"], prompt)
+    n_lat, n_ret = (L + 1) // 2, L // 2
+    cache = n_lat * win * (la["kv_rank"] + la["rot_dim"]) * 2 + n_ret * re["heads"] * re["dim"] * re["vdim"] * 8
+    flops = 2 * n + n_lat * 2 * win * la["heads"] * (la["dim"] + la["rot_dim"] + la["vdim"]) + n_ret * 4 * re["heads"] * re["dim"] * re["vdim"]
+    m = orangu_b200.FenipelModel(be, cfg, t, max_seq_len=8192, max_batch_tokens=prompt, kv_pool_tokens=64 * 4480, state_slots=64)
+    result = dict(time_model(be, m, z["vocab"], 2 * n, cache, flops, steps, warmup), parameters=n)
+    m.close()
+    return result
+
+
+def time_nenodra(be, size: str, L: int, steps: int, warmup: int):
+    import orangu_b200
+
+    cfg, t = nenodra_model(size, L)
+    z, prompt = NENODRA_SIZES[size], 4096
+    expert = 3 * z["width"] * z["expert_ff"]
+    n_moe = sum(x["mlp"]["kind"] == "moe" for x in cfg["layers"])
+    n = sum(a.size for k, a in t.items() if not k.endswith("embed"))
+    shared = n - n_moe * z["experts"] * expert
+    win, cache, flops = min(z["window"], prompt), 0, 2 * (shared + n_moe * z["top"] * expert)
+    for layer in cfg["layers"]:
+        m, maps = layer["mixer"], 2 if layer["type"] == "attention" else 1
+        cache += 2 * win * m["kv_heads"] * (maps * m["dim"] + m["vdim"])
+        flops += 2 * win * m["heads"] * maps * (m["dim"] + m["vdim"])
+    # experts that a step reads when tokens choose independently and evenly
+    weights = lambda batch: 2 * (shared + n_moe * expert * z["experts"] * (1 - (1 - z["top"] / z["experts"]) ** batch))
+    m = orangu_b200.NenodraModel(be, cfg, t, max_seq_len=8192, max_batch_tokens=prompt, kv_pool_tokens=64 * 4480)
+    result = dict(time_model(be, m, z["vocab"], weights, cache, flops, steps, warmup), parameters=n)
+    m.close()
+    return result
+
+
+def run_nenodra(args):
+    """--nenodra: one JSON line with both models at every size."""
+    import orangu_b200
+
+    be = orangu_b200.CudaBackend.init(0)
+    steps, warmup, L = args.steps, max(3, args.warmup), args.nenodra_layers
+    result = {"bench": "nenodra", "data": "synthetic", "dtype": "bf16", "layers": L, "steps": steps, "warmup": warmup, "sizes": {}}
+    clocks = ClockSampler(0)
+    clocks.start()
+    for size in args.nenodra.split(","):
+        entry = {"nenodra": time_nenodra(be, size, L, steps, warmup)}
+        if not args.nenodra_only:
+            entry["fenipel"] = time_fenipel(be, size, L, steps, warmup)
+        result["sizes"][size] = entry
+    result["clocks"] = clocks.stop()
+    be.close()
+    print(json.dumps(result))
 
 
 def run_fenipel(args):
@@ -410,18 +525,8 @@ def run_fenipel(args):
     clocks = ClockSampler(0)
     clocks.start()
     for size in args.fenipel.split(","):
-        cfg, t = fenipel_model(size, L)
-        n = sum(a.size for k, a in t.items() if not k.endswith("embed"))
+        entry = {"fenipel": time_fenipel(be, size, L, steps, warmup)}
         z, prompt = FENIPEL_SIZES[size], 4096
-        la, re = z["latent"], z["retention"]
-        win = min(la["window"], prompt)
-        n_lat, n_ret = (L + 1) // 2, L // 2
-        cache = n_lat * win * (la["kv_rank"] + la["rot_dim"]) * 2 + n_ret * re["heads"] * re["dim"] * re["vdim"] * 8
-        flops = 2 * n + n_lat * 2 * win * la["heads"] * (la["dim"] + la["rot_dim"] + la["vdim"]) + n_ret * 4 * re["heads"] * re["dim"] * re["vdim"]
-        m = orangu_b200.FenipelModel(be, cfg, t, max_seq_len=8192, max_batch_tokens=prompt, kv_pool_tokens=64 * 4480, state_slots=64)
-        entry = {"fenipel": dict(time_model(be, m, z["vocab"], 2 * n, cache, flops, steps, warmup), parameters=n)}
-        m.close()
-        del t
         if not args.fenipel_only:
             c = dict(synth.CONFIGS[size], n_layer=L, n_vocab=z["vocab"])
             tensors = synth.model_tensors(c, seed=7)
@@ -449,6 +554,9 @@ def main():
         return
     if args.fenipel:
         run_fenipel(args)
+        return
+    if args.nenodra:
+        run_nenodra(args)
         return
 
     import torch
