@@ -6,7 +6,9 @@
 //   attention_prep_kernel    norms and rotates queries and keys, appends keys and values to the cache
 //   attention_step_kernel    decoded tokens and short portions: every warp takes pages of its own, a cluster of CTAs shares the
 //                            keys of one tile and adds up over distributed shared memory
-//   attention_span_kernel    portions of prompts: 64 or 128 (token, head) rows of one key/value head, keys in tiles of 64
+//   attention_prompt_kernel  portions of prompts on tcgen05 (gqa_tc5.cu)
+//   attention_span_kernel    portions of prompts whose values are wider than that takes: 64 or 128 (token, head) rows of one
+//                            key/value head, keys in tiles of 64
 //   attention_plain_kernel   any sizes, fp32 cache
 //
 // A page holds 16 positions of every key/value head next to one another.  A cache row is [keys of the maps | value | 8 entries of
@@ -675,7 +677,7 @@ cudaError_t attention_configure() {
             for (int f = 0; f < N_FORM; ++f) set(ST_KERNELS[m][f]), set(SP_KERNELS[m][f]);
         set(attention_plain_kernel<float>), set(attention_plain_kernel<bf16>);
         set(attention_prep_kernel<float>), set(attention_prep_kernel<bf16>);
-        return e;
+        return e != cudaSuccess ? e : attention_prompt_configure();
     });
 }
 
@@ -698,7 +700,8 @@ uint32_t launch_attention(const AttentionArgs &in, bool f32, int sm_count, cudaS
         return 1;
     }
     const SpPlan sp(a.n_map, a.dim_p, a.vdim_p, a.row);
-    if (sp.bytes > MAX_SMEM) a.n_short = a.n_seq;
+    const bool tc5 = attention_prompt_supported(a.n_map, a.dim_p, a.vdim_p);
+    if (!tc5 && sp.bytes > MAX_SMEM) a.n_short = a.n_seq;
     uint32_t launched = 0;
     if (a.n_short) {
         uint32_t tiles = 0;
@@ -724,7 +727,10 @@ uint32_t launch_attention(const AttentionArgs &in, bool f32, int sm_count, cudaS
         cudaLaunchKernelEx(&cfg, ST_KERNELS[a.n_map - 1][form], a, splits, stages);
         ++launched;
     }
-    if (a.n_short < a.n_seq) {
+    if (a.n_short < a.n_seq && tc5) {
+        if (!launch_attention_prompt(a, st)) return 0;
+        ++launched;
+    } else if (a.n_short < a.n_seq) {
         uint32_t tiles = 0;
         for (uint32_t s = a.n_short; s < a.n_seq; ++s) tiles += (a.h_spans[s].n * per + sp.rows - 1) / sp.rows;
         launch_pdl(SP_KERNELS[a.n_map - 1][form], dim3(tiles, a.n_kv), SP_THREADS, sp.bytes, st, a);

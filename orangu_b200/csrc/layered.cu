@@ -322,6 +322,7 @@ void LayeredGraph::attention(const LayerPlan &P, uint32_t T, uint32_t n_seq, con
     a.rot = P.rot;
     a.q = q;
     a.cache = P.pool;
+    a.n_pages = m->pool_pages;
     a.out = cat;
     a.out_pitch = cat_pitch;
     a.T = T;
@@ -334,7 +335,9 @@ void LayeredGraph::attention(const LayerPlan &P, uint32_t T, uint32_t n_seq, con
     a.tables = reinterpret_cast<const int32_t *const *>(m->d_meta + ml.off_tables);
     a.max_pos = max_pos;
     launch_attention_prep(a, f32, st);
-    m->ctx->launches += 1 + launch_attention(a, f32, m->ctx->sm_count, st);
+    const uint32_t n = launch_attention(a, f32, m->ctx->sm_count, st);
+    if (!n) failed = true;
+    m->ctx->launches += 1 + n;
 }
 
 void LayeredGraph::mixer(const LayerPlan &P, uint32_t T, uint32_t n_seq, const RowSpan *spans, bool single, uint32_t max_pos, cudaStream_t st) {

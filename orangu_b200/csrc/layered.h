@@ -195,6 +195,7 @@ struct AttentionArgs {       // softmax attention of one layer over T rows
     Rot rot;
     void *q;                 // activations [T][n_head][n_map][dim_p]
     void *cache;             // activations [page][n_kv][16][row]
+    uint32_t n_pages;        // of the pool
     void *out;               // activations [T][out_pitch], head h at h * vdim
     uint32_t out_pitch;
     uint32_t T, n_seq, n_short;   // spans [0, n_short) are short, the others long (PREFILL_SPAN rows or more)
@@ -209,7 +210,12 @@ cudaError_t attention_configure();
 bool attention_supported(uint32_t dim, uint32_t vdim);
 uint32_t attention_cache_row(uint32_t n_map, uint32_t dim_p, uint32_t vdim_p);  // elements of a cache row
 void launch_attention_prep(const AttentionArgs &a, bool f32, cudaStream_t st);  // norms, rotates and stores queries; appends keys and values
-uint32_t launch_attention(const AttentionArgs &a, bool f32, int sm_count, cudaStream_t st);  // returns the kernels launched
+uint32_t launch_attention(const AttentionArgs &a, bool f32, int sm_count, cudaStream_t st);  // returns the kernels launched; 0: a tensor map could not be made
+// gqa_tc5.cu: the long spans on tcgen05 (bf16)
+cudaError_t attention_prompt_configure();
+bool attention_prompt_supported(uint32_t n_map, uint32_t dim_p, uint32_t vdim_p);
+bool launch_attention_prompt(const AttentionArgs &a, cudaStream_t st);  // false: a tensor map could not be made
+int attention_take_status();  // as linear_take_status
 
 // ---- moe.cu ----------------------------------------------------------------------------------------------------------
 struct MoeArgs {             // routing of T tokens to `top` of n_expert experts; a (token, choice) is a pair, t * top + choice

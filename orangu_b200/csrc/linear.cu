@@ -314,17 +314,6 @@ struct LtSmem {
     static_assert(STAGES >= 3 && ALLOC <= (BN == 256 ? 227 : 113) * 1024, "shared memory plan does not fit");
 };
 
-// D (tensor memory, fp32, 128 lanes x N columns) [+]= A (128 x 16 bf16, K-major) * B (N x 16 bf16, K-major)^T
-__device__ __forceinline__ void umma_bf16(uint32_t d_tmem, uint64_t a_desc, uint64_t b_desc, uint32_t idesc, uint32_t accumulate) {
-    asm volatile(
-        "{\n\t.reg .pred p;\n\tsetp.ne.b32 p, %4, 0;\n\t"
-        "tcgen05.mma.cta_group::1.kind::f16 [%0], %1, %2, %3, p;\n\t}" ::"r"(d_tmem),
-        "l"(a_desc), "l"(b_desc), "r"(idesc), "r"(accumulate)
-        : "memory");
-}
-// Instruction descriptor: fp32 accumulator, A and B bfloat16, both K-major, N columns, M = 128.
-__host__ __device__ constexpr uint32_t umma_idesc_bf16(uint32_t n) { return (1u << 4) | (1u << 7) | (1u << 10) | ((n >> 3) << 17) | ((128u >> 4) << 24); }
-
 struct LtTiles {
     uint32_t rows, toks, total;  // weight tiles and token tiles of one batch entry, tiles of all (splits counted)
     uint32_t splits;             // > 1: one token tile of at most LT_SPLIT_TOKENS rows, a CTA per tile and split

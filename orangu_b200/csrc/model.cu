@@ -1456,7 +1456,7 @@ int pre_step(ob_model *m) {
 int check_peer(ob_model *m) {
     if (quantized_built() && gemm_tc5_take_status()) return fail(m->ctx, OB_ERR_CUDA, "a tensor-core product gave up a bounded wait (pipeline barrier); the step's output is not valid");
     if (m->graph && m->graph->take_failure()) return fail(m->ctx, OB_ERR_CUDA, "a product of the step could not be launched");
-    if (m->graph && linear_take_status()) return fail(m->ctx, OB_ERR_CUDA, "a tensor-core product gave up a bounded wait (pipeline barrier); the step's output is not valid");
+    if (m->graph && linear_take_status() + attention_take_status()) return fail(m->ctx, OB_ERR_CUDA, "a tensor-core product gave up a bounded wait (pipeline barrier); the step's output is not valid");
     if (m->launch_failed) {
         m->launch_failed = false;
         return fail(m->ctx, OB_ERR_CUDA, std::string("launching the persistent layer kernel failed: ") + cudaGetErrorString(cudaGetLastError()));
