@@ -71,6 +71,76 @@ __global__ void __launch_bounds__(PREP_WARPS * 32) attention_prep_kernel(Attenti
     for (uint32_t d = lane; d < a.dim_p; d += 32) dst[d] = to_act<TA>(d < a.dim ? rotated(v, d, a.rot, cs) : 0.0f);
 }
 
+// The same for sizes in eights (head sizes, half of the rotated entries): `group` neighbouring lanes per vector, eight entries each.
+constexpr int PREP_THREADS = 256;
+__device__ __forceinline__ void load_eight(const float *p, float (&v)[8]) {
+    const float4 a = reinterpret_cast<const float4 *>(p)[0], b = reinterpret_cast<const float4 *>(p)[1];
+    v[0] = a.x, v[1] = a.y, v[2] = a.z, v[3] = a.w, v[4] = b.x, v[5] = b.y, v[6] = b.z, v[7] = b.w;
+}
+template <typename TA> __device__ __forceinline__ void store_eight(TA *p, const float (&v)[8]) {
+    store4<TA>(p, make_float4(v[0], v[1], v[2], v[3]));
+    store4<TA>(p + 4, make_float4(v[4], v[5], v[6], v[7]));
+}
+template <typename TA>
+__global__ void __launch_bounds__(PREP_THREADS) attention_prep_vec_kernel(AttentionArgs a, uint32_t group) {
+    pdl_release();
+    pdl_wait();
+    const uint32_t t = blockIdx.x, c = threadIdx.x & (group - 1), i = blockIdx.y * (PREP_THREADS / group) + threadIdx.x / group;
+    const uint32_t n_q = a.n_head * a.n_map, n_k = a.n_kv * a.n_map, d = 8 * c;
+    const bool exists = i < n_q + n_k + a.n_kv, value = i >= n_q + n_k, query = i < n_q;
+    const uint32_t pos = a.positions[t];
+    const float *y = a.y + (uint64_t)t * a.y_pitch;
+    TA *cache = static_cast<TA *>(a.cache) + page_at(a, a.tables[t][pos / KV_PAGE], 0) + (uint64_t)(pos % KV_PAGE) * a.row;
+    const uint64_t head = (uint64_t)KV_PAGE * a.row;  // from one key/value head to the next within a page
+    if (exists && value) {
+        const uint32_t g = i - n_q - n_k;
+        TA *dst = cache + g * head + a.n_map * a.dim_p;
+        for (uint32_t e = d; e < a.vdim; e += 8 * group) {
+            float v[8];
+            if (a.has_v) {
+                constexpr uint32_t P = 16 / sizeof(TA);
+                const TA *src = static_cast<const TA *>(a.va) + (uint64_t)t * a.va_pitch + (uint64_t)g * a.vdim + e;
+#pragma unroll
+                for (uint32_t k = 0; k < 8; k += P) *reinterpret_cast<uint4 *>(dst + e + k) = *reinterpret_cast<const uint4 *>(src + k);
+            } else {
+                load_eight(y + (uint64_t)(n_q + g) * a.dim + e, v);
+                store_eight<TA>(dst + e, v);
+            }
+        }
+    }
+    const bool mine = exists && !value && d < a.dim;
+    float v[8] = {}, s = 0.0f;
+    if (mine) load_eight(y + (uint64_t)i * a.dim + d, v);
+#pragma unroll
+    for (int e = 0; e < 8; ++e) s += v[e] * v[e];
+    for (uint32_t o = group / 2; o > 0; o >>= 1) s += __shfl_xor_sync(0xffffffffu, s, o);
+    const float f = inv_rms(s, a.dim, a.eps);
+    if (mine) {
+        float w[8];
+        load_eight((query ? a.q_norm : a.k_norm) + d, w);
+#pragma unroll
+        for (int e = 0; e < 8; ++e) v[e] *= f * w[e];
+    }
+    const uint32_t half = a.rot.dims / 2;
+    const bool low = d < half, turns = d < a.rot.dims;
+    float other[8];  // the entries half of the rotated ones away
+    const uint32_t lane = threadIdx.x & 31, from = turns ? (low ? lane + half / 8 : lane - half / 8) : lane;
+#pragma unroll
+    for (int e = 0; e < 8; ++e) other[e] = __shfl_sync(0xffffffffu, v[e], from);
+    if (mine && turns) {
+        const float2 *cs = a.rot.table + (uint64_t)pos * half + (low ? d : d - half);
+#pragma unroll
+        for (int e = 0; e < 8; ++e) {
+            const float2 r = cs[e];
+            v[e] = low ? v[e] * r.x - other[e] * r.y : v[e] * r.x + other[e] * r.y;
+        }
+    }
+    if (exists && !value && d < a.dim_p) {  // (zeros from dim on)
+        const uint32_t k = i - n_q;
+        store_eight<TA>((query ? static_cast<TA *>(a.q) + ((uint64_t)t * n_q + i) * a.dim_p : cache + k / a.n_map * head + k % a.n_map * a.dim_p) + d, v);
+    }
+}
+
 // ---- the end of a head: both maps put together, gate, store ----------------------------------------------------------------------
 __device__ __forceinline__ float gate_of(const AttentionArgs &a, uint64_t t, uint32_t h, uint32_t c, bool f32) {
     const uint64_t at = t * a.va_pitch + a.gate0 + (uint64_t)h * a.vdim + c;
@@ -161,9 +231,10 @@ struct StPlan {
         bytes = ST_ROWS * q_row + ST_WARPS * ring + 256 * 2 + 128;  // a page's last row is read up to 256 columns past its values
     }
     static uint32_t best_stages(uint32_t n_map, uint32_t dim_p, uint32_t vdim_p, uint32_t row) {
+        // two CTAs per SM, else one (three with fewer stages, or more splits of a tile, are slower: a CTA's start and end cost)
         for (uint32_t s = 4; s >= 2; --s) {
             const uint32_t b = StPlan(n_map, dim_p, vdim_p, row, s).bytes;
-            if (2 * (b + 1024) <= 226 * 1024 || (s == 2 && b <= MAX_SMEM)) return s;
+            if (2 * (b + 2048) <= 227 * 1024 || (s == 2 && b <= MAX_SMEM)) return s;
         }
         return 0;
     }
@@ -232,19 +303,25 @@ __global__ void __launch_bounds__(ST_THREADS) attention_step_kernel(AttentionArg
             cp16(qs + r * pl.q_row + c * 16, src, r < n_here);
         }
     }
-    auto load = [&](uint32_t n) {  // this warp's n'th page
-        const uint32_t p = unit + n * n_unit;
-        if (p < n_page) {
-            const bf16 *src = static_cast<const bf16 *>(a.cache) + page_at(a, table[page0 + p], g);
-            const uint32_t dst = ring + n % stages * page_bytes;
-            for (uint32_t i = lane; i < pieces; i += 32) cp16(dst + i * 16, src + 8 * i, true);
+    const uint32_t ring_end = ring + stages * page_bytes;
+    uint32_t next_page = unit, next_stage = ring;  // of the next load
+    auto load = [&] {  // this warp's next page
+        if (next_page < n_page) {
+            const bf16 *src = static_cast<const bf16 *>(a.cache) + page_at(a, table[page0 + next_page], g) + 8 * lane;
+            uint32_t dst = next_stage + 16 * lane, i = lane;
+            for (; i + 96 < pieces; i += 128, src += 1024, dst += 2048)
+#pragma unroll
+                for (int k = 0; k < 4; ++k) cp16(dst + 512 * k, src + 256 * k, true);
+            for (; i < pieces; i += 32, src += 256, dst += 512) cp16(dst, src, true);
         }
         cp_commit();
+        next_page += n_unit;
+        next_stage = next_stage + page_bytes == ring_end ? ring : next_stage + page_bytes;
     };
     // (the first group also holds the queries; with fewer than four stages empty groups keep the count)
-    load(0);
-    if (stages > 2) load(1);
-    if (stages > 3) load(2);
+    load();
+    if (stages > 2) load();
+    if (stages > 3) load();
     if (stages == 4) cp_wait<2>();
     else if (stages == 3) cp_wait<1>();
     else cp_wait<0>();
@@ -268,14 +345,14 @@ __global__ void __launch_bounds__(ST_THREADS) attention_step_kernel(AttentionArg
     const uint32_t qa = qs + (lane & 15) * pl.q_row + (lane >> 4) * 16;
     const uint32_t b_off = ((lane & 7) + ((lane >> 4) << 3)) * row_bytes + ((lane >> 3) & 1) * 16;
     const uint32_t v_off = ((lane & 7) + (((lane >> 3) & 1) << 3)) * row_bytes + (lane >> 4) * 16 + NM * a.dim_p * 2;
-    for (uint32_t n = 0; unit + n * n_unit < n_page; ++n) {
-        load(n + stages - 1);
+    uint32_t kb = ring;
+    for (uint32_t page = unit; page < n_page; page += n_unit, kb = kb + page_bytes == ring_end ? ring : kb + page_bytes) {
+        load();
         if (stages == 4) cp_wait<3>();
         else if (stages == 3) cp_wait<2>();
         else cp_wait<1>();
         __syncwarp();
-        const uint32_t kb = ring + n % stages * page_bytes;
-        const int j0 = (int)((page0 + unit + n * n_unit) * KV_PAGE);
+        const int j0 = (int)((page0 + page) * KV_PAGE);
         uint32_t ph[LM][4], pr[LM][4];
 #pragma unroll
         for (int m = 0; m < LM; ++m) {
@@ -308,6 +385,7 @@ __global__ void __launch_bounds__(ST_THREADS) attention_step_kernel(AttentionArg
                 }
             b0 = fmaxf(b0, __shfl_xor_sync(0xffffffffu, b0, 1)), b0 = fmaxf(b0, __shfl_xor_sync(0xffffffffu, b0, 2));
             b1 = fmaxf(b1, __shfl_xor_sync(0xffffffffu, b1, 1)), b1 = fmaxf(b1, __shfl_xor_sync(0xffffffffu, b1, 2));
+            // (rescaling only when the maximum has grown much puts a branch between the maps' products: slower)
             const float n0 = fmaxf(m0[m], b0), n1 = fmaxf(m1[m], b1);
             const float s0 = n0 == -INFINITY ? 0.0f : n0, s1 = n1 == -INFINITY ? 0.0f : n1;  // a row that has seen nothing yet keeps weights of zero
             const float g0 = pow2(m0[m] - s0), g1 = pow2(m1[m] - s1);
@@ -687,6 +765,13 @@ bool attention_supported(uint32_t dim, uint32_t vdim) { return (uint64_t)PREP_WA
 
 void launch_attention_prep(const AttentionArgs &a, bool f32, cudaStream_t st) {
     const uint32_t n = (a.n_head + a.n_kv) * a.n_map + a.n_kv;
+    if (a.dim % 8 == 0 && a.vdim % 8 == 0 && a.rot.dims % 16 == 0 && !a.rot.interleaved && a.dim_p <= 256) {
+        uint32_t group = 1;
+        while (8 * group < a.dim_p) group *= 2;
+        const uint32_t each = PREP_THREADS / group;
+        launch_pdl(f32 ? attention_prep_vec_kernel<float> : attention_prep_vec_kernel<bf16>, dim3(a.T, (n + each - 1) / each), PREP_THREADS, 0, st, a, group);
+        return;
+    }
     const dim3 grid(a.T, (n + PREP_WARPS - 1) / PREP_WARPS);
     launch_pdl(f32 ? attention_prep_kernel<float> : attention_prep_kernel<bf16>, grid, PREP_WARPS * 32, (size_t)PREP_WARPS * a.dim * 4, st, a);
 }
