@@ -4,10 +4,10 @@
 // keys and values, with two maps the maps of the same rows, which share the values.  While one stream's scores go through the
 // softmax, the tensor core works for the other.
 //
-//   warps 0-7  softmax: four warps per stream, a thread per row.  Scores come from tensor memory, weights go back into the same
-//              columns as value plus remainder, two bf16 operands, so that they are not rounded to 8 bits.
-//   warp 8     issues the products: scores = queries (shared memory) x keys, output += weights (tensor memory) x values
-//   warp 9     issues the TMA loads of pages: 16 rows x 64 columns each, straight from the cache into the swizzled operand tiles
+//   warps 0-15 softmax: eight warps per stream, two threads per row with 64 keys each.  Scores come from tensor memory, weights go
+//              back into the same columns as value plus remainder, two bf16 operands, so that they are not rounded to 8 bits.
+//   warp 16    issues the products: scores = queries (shared memory) x keys, output += weights (tensor memory) x values
+//   warp 17    issues the TMA loads of pages: 16 rows x 64 columns each, straight from the cache into the swizzled operand tiles
 //
 // Tensor memory: scores / weights of the streams 2 x 128 columns, outputs 2 x 128.  The output is only rescaled when a row's maximum
 // has grown by more than 2^8 since the last time; until then weights are relative to the older maximum.  All waits are bounded.
@@ -19,26 +19,38 @@ namespace ob {
 namespace {
 
 constexpr uint32_t PT_ROWS = 128, PT_KEYS = 128, PT_PAGES = PT_KEYS / KV_PAGE, PT_BLOCK = PT_KEYS * 128;  // block: 128 rows of 64 columns
-constexpr int PT_SOFTMAX_WARPS = 8, PT_MMA_WARP = 8, PT_TMA_WARP = 9, PT_THREADS = 10 * 32;
+constexpr int PT_SOFTMAX_WARPS = 16, PT_MMA_WARP = 16, PT_TMA_WARP = 17, PT_THREADS = 18 * 32;
 constexpr uint32_t PT_TMEM_S = 0, PT_TMEM_O = 256, PT_TMEM_COLS = 512;
 constexpr float PT_SLACK = 8.0f;  // growth of the maximum (powers of two) that is put up with
 
+constexpr uint32_t PT_SHARED = 256 + 2 * 2 * PT_ROWS * 4;  // mbarriers, then a number per stream, half and row
 struct PtPlan {
     uint32_t nb, nbv, k_bytes, v_bytes, stages, k, v, bar, bytes;  // blocks of 64 columns of a map's keys and of a value; operands of one stage
     __host__ __device__ PtPlan(uint32_t n_map, uint32_t dim_p, uint32_t vdim_p) {
         nb = (dim_p + 63) / 64, nbv = (vdim_p + 63) / 64;
         k_bytes = n_map * nb * PT_BLOCK, v_bytes = nbv * PT_BLOCK;
-        const uint32_t q = 2 * nb * PT_BLOCK, room = 224 * 1024 - 256;
+        const uint32_t q = 2 * nb * PT_BLOCK, room = 225 * 1024 - PT_SHARED;
         stages = q + 2 * (k_bytes + v_bytes) <= room ? 2 : q + k_bytes + v_bytes <= room ? 1 : 0;
         k = q;
         v = k + stages * k_bytes;
         bar = v + stages * v_bytes;
-        bytes = bar + 256 + 1024;
+        bytes = bar + PT_SHARED + 1024;
     }
 };
 // mbarriers, byte offsets from PtPlan::bar
 constexpr uint32_t PT_K_FULL = 0, PT_K_EMPTY = 16, PT_V_FULL = 32, PT_V_EMPTY = 48, PT_S_FULL = 64, PT_P_FULL = 80, PT_O_FULL = 96, PT_Q_FULL = 112, PT_SLOT = 120, PT_ABORT = 124,
-                   PT_INFO = 128;
+                   PT_INFO = 128, PT_EXCHANGE = 256;
+
+// Two fp32 multiply-adds in one instruction.
+__device__ __forceinline__ void fma2(float &d0, float &d1, float a0, float a1, float b, float c) {
+    asm("{\n\t.reg .b64 x, y, z;\n\tmov.b64 x, {%2, %3};\n\tmov.b64 y, {%4, %4};\n\tmov.b64 z, {%5, %5};\n\tfma.rn.f32x2 x, x, y, z;\n\tmov.b64 {%0, %1}, x;\n\t}"
+        : "=f"(d0), "=f"(d1)
+        : "f"(a0), "f"(a1), "f"(b), "f"(c));
+}
+__device__ __forceinline__ void add2(float &d0, float &d1, float a0, float a1) {
+    asm("{\n\t.reg .b64 x, y;\n\tmov.b64 x, {%0, %1};\n\tmov.b64 y, {%2, %3};\n\tadd.rn.f32x2 x, x, y;\n\tmov.b64 {%0, %1}, x;\n\t}" : "+f"(d0), "+f"(d1) : "f"(a0), "f"(a1));
+}
+__device__ __forceinline__ void pair_sync(uint32_t id) { asm volatile("bar.sync %0, 64;" ::"r"(id) : "memory"); }
 
 // Entries [c, c + 16) of a head's output, gated, as activations.
 __device__ __forceinline__ void store_head(const AttentionArgs &a, uint64_t t, uint32_t h, uint32_t c, float (&x)[16]) {
@@ -85,7 +97,7 @@ __global__ void __launch_bounds__(PT_THREADS, 1) attention_prompt_kernel(const _
             mbar_init(bar + PT_V_FULL + 8 * s, 1);
             mbar_init(bar + PT_V_EMPTY + 8 * s, 1);
             mbar_init(bar + PT_S_FULL + 8 * s, 1);
-            mbar_init(bar + PT_P_FULL + 8 * s, 4);
+            mbar_init(bar + PT_P_FULL + 8 * s, 8);
             mbar_init(bar + PT_O_FULL + 8 * s, 1);
         }
         mbar_init(bar + PT_Q_FULL, PT_SOFTMAX_WARPS);
@@ -190,23 +202,24 @@ __global__ void __launch_bounds__(PT_THREADS, 1) attention_prompt_kernel(const _
             }
         }
     } else {
-        const uint32_t s = warp / 4, quad = warp % 4, r = quad * 32 + lane, i_row = (NM == 2 ? 0 : s * PT_ROWS) + r;  // row within the CTA
+        const uint32_t s = warp / 8, part = warp / 4 % 2, quad = warp % 4, r = quad * 32 + lane, i_row = (NM == 2 ? 0 : s * PT_ROWS) + r;  // row within the CTA
         const bool live = i_row < n_here;
-        const uint32_t t0 = first_tile(s), t1 = end_tile(s);
+        const uint32_t t0 = first_tile(s), t1 = end_tile(s), pair = 1 + s * 4 + quad;
         const uint32_t f = f0 + (live ? i_row : 0), h = g * per + f % per;
         const uint64_t t = row0 + f / per;
         const int pos = live ? (int)(pos0 + f / per) : -1, win = a.window ? (int)min(a.window, 0x3fffffffu) : 0x3fffffff;
+        volatile float *xchg = reinterpret_cast<volatile float *>(smem + pl.bar + PT_EXCHANGE) + s * 2 * PT_ROWS + r;  // own half at part * PT_ROWS, the other's beside it
         {   // the row's query into the swizzled operand tile
             const bf16 *q = static_cast<const bf16 *>(a.q) + ((t * a.n_head + h) * NM + (NM == 2 ? s : 0)) * a.dim_p;
             uint8_t *dst = smem + s * pl.nb * PT_BLOCK + r * 128;
-            for (uint32_t c = 0; c < a.dim_p / 8; ++c)
+            for (uint32_t c = part; c < a.dim_p / 8; c += 2)
                 *reinterpret_cast<uint4 *>(dst + c / 8 * PT_BLOCK + (((c & 7) ^ (r & 7)) << 4)) = live ? *reinterpret_cast<const uint4 *>(q + 8 * c) : make_uint4(0, 0, 0, 0);
             asm volatile("fence.proxy.async.shared::cta;" ::: "memory");
             __syncwarp();
             if (lane == 0) mbar_arrive(bar + PT_Q_FULL);
         }
         const float scale2 = a.scale * 1.4426950408889634f;  // weights are powers of two of the scaled score
-        const uint32_t ts = tmem + ((quad * 32) << 16) + PT_TMEM_S + s * PT_KEYS, to = tmem + ((quad * 32) << 16) + PT_TMEM_O + s * 128;
+        const uint32_t lanes = tmem + ((quad * 32) << 16), ts = lanes + PT_TMEM_S + s * PT_KEYS + part * 64, to = lanes + PT_TMEM_O + s * 128;
         // first and last position of the warp's rows (dead rows do not count)
         const uint32_t w0 = (NM == 2 ? 0 : s * PT_ROWS) + quad * 32;
         const bool whole = w0 + 32 <= n_here;
@@ -214,32 +227,40 @@ __global__ void __launch_bounds__(PT_THREADS, 1) attention_prompt_kernel(const _
         float m = -INFINITY, l = 0.0f;
         bool ok = true;
         for (uint32_t i = t0; i < t1; ++i) {
-            if (!(ok = __all_sync(0xffffffffu, mbar_wait(bar + PT_S_FULL + 8 * s, (i - t0) & 1u, abort)))) break;
+            ok = ok && __all_sync(0xffffffffu, mbar_wait(bar + PT_S_FULL + 8 * s, (i - t0) & 1u, abort));
+            if (!ok) {  // a wait was given up: nothing more is computed, but the other half's barriers are kept company
+                pair_sync(pair);
+                continue;
+            }
             tc_fence_after();
-            uint32_t u[4][32];
-#pragma unroll
-            for (int c = 0; c < 4; ++c) tmem_ld32(ts + 32 * c, u[c]);
+            const int j0 = (int)((page0 + i * PT_PAGES) * KV_PAGE + part * 64);
+            const bool masked = !(whole && j0 + 63 <= w_first && w_last - j0 < win);  // keys outside the window of some row
+            const int last = pos - j0, first = last - win + 1;                        // visible columns (pos -1: none)
+            uint32_t u[2][32];
+            tmem_ld32(ts, u[0]);
+            tmem_ld32(ts + 32, u[1]);
             tmem_ld_wait();
-            const int j0 = (int)((page0 + i * PT_PAGES) * KV_PAGE);
-            if (!(whole && j0 + (int)PT_KEYS - 1 <= w_first && w_last - j0 < win)) {  // keys outside the window of some row
-                const int last = pos - j0, first = last - win + 1;  // visible columns (pos -1: none)
+            if (masked) {
 #pragma unroll
-                for (int c = 0; c < 4; ++c)
+                for (int c = 0; c < 2; ++c)
 #pragma unroll
                     for (int e = 0; e < 32; ++e)
                         if (c * 32 + e > last || c * 32 + e < first) u[c][e] = 0xff800000u;
             }
             float top[4] = {-INFINITY, -INFINITY, -INFINITY, -INFINITY};
 #pragma unroll
-            for (int c = 0; c < 4; ++c)
+            for (int c = 0; c < 2; ++c)
 #pragma unroll
-                for (int e = 0; e < 32; ++e) top[c] = fmaxf(top[c], __uint_as_float(u[c][e]));
-            const float now = fmaxf(fmaxf(top[0], top[1]), fmaxf(top[2], top[3])) * scale2;
+                for (int e = 0; e < 32; ++e) top[e % 4] = fmaxf(top[e % 4], __uint_as_float(u[c][e]));
+            const float own = fmaxf(fmaxf(top[0], top[1]), fmaxf(top[2], top[3])) * scale2;
+            xchg[part * PT_ROWS] = own;
+            pair_sync(pair);
+            const float now = fmaxf(own, xchg[(part ^ 1u) * PT_ROWS]);
             const bool grown = m > -INFINITY && now > m + PT_SLACK;
             if (__any_sync(0xffffffffu, grown)) {  // the product before this tile's scores is done: the output may be rescaled
                 const float keep = grown ? pow2(m - now) : 1.0f;
                 if (grown) m = now, l *= keep;
-                for (uint32_t c = 0; c < a.vdim_p; c += 16) {
+                for (uint32_t c = 16 * part; c < a.vdim_p; c += 32) {
                     uint32_t o[16];
                     tmem_ld16(to + c, o);
                     tmem_ld_wait();
@@ -249,16 +270,18 @@ __global__ void __launch_bounds__(PT_THREADS, 1) attention_prompt_kernel(const _
                 }
             }
             if (m == -INFINITY) m = now;
-            const float base = m == -INFINITY ? 0.0f : m;  // a row that has seen nothing yet keeps weights of zero
-            float sum[2] = {0.0f, 0.0f};
+            const float base = m == -INFINITY ? 0.0f : -m;  // a row that has seen nothing yet keeps weights of zero
+            float sum0 = 0.0f, sum1 = 0.0f;
 #pragma unroll
-            for (int c = 0; c < 8; ++c) {  // 16 keys: eight columns of values, eight of remainders
+            for (int c = 0; c < 4; ++c) {  // 16 keys: eight columns of values, eight of remainders
                 uint32_t w[16];
 #pragma unroll
                 for (int e = 0; e < 8; ++e) {
                     const uint32_t(&x)[32] = u[c / 2];
-                    const float e0 = pow2(fmaf(__uint_as_float(x[c % 2 * 16 + 2 * e]), scale2, -base)), e1 = pow2(fmaf(__uint_as_float(x[c % 2 * 16 + 2 * e + 1]), scale2, -base));
-                    sum[0] += e0, sum[1] += e1;
+                    float e0, e1;
+                    fma2(e0, e1, __uint_as_float(x[c % 2 * 16 + 2 * e]), __uint_as_float(x[c % 2 * 16 + 2 * e + 1]), scale2, base);
+                    e0 = pow2(e0), e1 = pow2(e1);
+                    add2(sum0, sum1, e0, e1);
                     const __nv_bfloat162 hi2 = __floats2bfloat162_rn(e0, e1);
                     const uint32_t hw = *reinterpret_cast<const uint32_t *>(&hi2);
                     const __nv_bfloat162 lo2 = __floats2bfloat162_rn(e0 - __uint_as_float(hw << 16), e1 - __uint_as_float(hw & 0xffff0000u));
@@ -266,7 +289,7 @@ __global__ void __launch_bounds__(PT_THREADS, 1) attention_prompt_kernel(const _
                 }
                 tmem_st16(ts + 16 * c, w);
             }
-            l += sum[0] + sum[1];
+            l += sum0 + sum1;
             tmem_st_wait();
             tc_fence_before();
             __syncwarp();
@@ -274,55 +297,55 @@ __global__ void __launch_bounds__(PT_THREADS, 1) attention_prompt_kernel(const _
         }
         if (ok && t1 > t0) ok = mbar_wait(bar + PT_O_FULL + 8 * s, 0, abort);
         tc_fence_after();
-        __syncwarp();
         ok = __all_sync(0xffffffffu, ok) && t1 > t0;
-        float fac = 1.0f / l;
-        const float *ex = reinterpret_cast<const float *>(smem + pl.k) + r * (a.vdim_p + 4);  // [128 rows]: the second map's share
+        pair_sync(pair);
+        xchg[part * PT_ROWS] = l;
+        pair_sync(pair);
+        const float fac = 1.0f / (l + xchg[(part ^ 1u) * PT_ROWS]);
+        float gain = fac;
+        float *ex = reinterpret_cast<float *>(smem + pl.k) + r * (a.vdim_p + 4);  // [128 rows]: the second map's share
+        auto output = [&](uint32_t c, float (&x)[16]) {  // entries [c, c + 16) of the row's output
+            uint32_t o[16];
+            tmem_ld16(to + c, o);
+            tmem_ld_wait();
+#pragma unroll
+            for (int e = 0; e < 16; ++e) x[e] = __uint_as_float(o[e]) * fac;
+        };
         if constexpr (NM == 2) {
             if (s == 1 && ok) {
-                float *mine = reinterpret_cast<float *>(smem + pl.k) + r * (a.vdim_p + 4);
-                const float w = fac * a.map_weight;
-                for (uint32_t c = 0; c < a.vdim_p; c += 16) {
-                    uint32_t o[16];
-                    tmem_ld16(to + c, o);
-                    tmem_ld_wait();
+                for (uint32_t c = 16 * part; c < a.vdim_p; c += 32) {
+                    float x[16];
+                    output(c, x);
 #pragma unroll
                     for (int e = 0; e < 4; ++e)
-                        *reinterpret_cast<float4 *>(mine + c + 4 * e) = make_float4(__uint_as_float(o[4 * e]) * w, __uint_as_float(o[4 * e + 1]) * w, __uint_as_float(o[4 * e + 2]) * w, __uint_as_float(o[4 * e + 3]) * w);
+                        *reinterpret_cast<float4 *>(ex + c + 4 * e) = mul4(make_float4(x[4 * e], x[4 * e + 1], x[4 * e + 2], x[4 * e + 3]), a.map_weight);
                 }
             }
-            asm volatile("bar.sync 1, 256;" ::: "memory");
+            asm volatile("bar.sync 9, 512;" ::: "memory");
+            float q = 0.0f;
             if (s == 0 && ok) {
-                float q = 0.0f;
-                for (uint32_t c = 0; c < a.vdim_p; c += 16) {
-                    uint32_t o[16];
-                    tmem_ld16(to + c, o);
-                    tmem_ld_wait();
+                for (uint32_t c = 16 * part; c < a.vdim_p; c += 32) {
+                    float x[16];
+                    output(c, x);
 #pragma unroll
                     for (int e = 0; e < 16; ++e) {  // columns past vdim are zero: so are the values there
-                        const float x = __uint_as_float(o[e]) * fac - ex[c + e];
-                        q += x * x;
+                        const float d = x[e] - ex[c + e];
+                        q += d * d;
                     }
                 }
-                q = inv_rms(q, a.vdim, a.eps) * a.head_gain;
-                for (uint32_t c = 0; c < a.vdim_p; c += 16) {
-                    uint32_t o[16];
-                    tmem_ld16(to + c, o);
-                    tmem_ld_wait();
-                    float x[16];
-#pragma unroll
-                    for (int e = 0; e < 16; ++e) x[e] = (__uint_as_float(o[e]) * fac - ex[c + e]) * q;
-                    if (live) store_head(a, t, h, c, x);
-                }
             }
-        } else if (ok) {
-            for (uint32_t c = 0; c < a.vdim_p; c += 16) {
-                uint32_t o[16];
-                tmem_ld16(to + c, o);
-                tmem_ld_wait();
+            xchg[part * PT_ROWS] = q;  // (both have read the sums: the barrier above)
+            pair_sync(pair);
+            gain = inv_rms(q + xchg[(part ^ 1u) * PT_ROWS], a.vdim, a.eps) * a.head_gain;
+        }
+        if (ok && (NM == 1 || s == 0)) {
+            for (uint32_t c = 16 * part; c < a.vdim_p; c += 32) {
                 float x[16];
+                output(c, x);
+                if constexpr (NM == 2) {
 #pragma unroll
-                for (int e = 0; e < 16; ++e) x[e] = __uint_as_float(o[e]) * fac;
+                    for (int e = 0; e < 16; ++e) x[e] = (x[e] - ex[c + e]) * gain;
+                }
                 if (live) store_head(a, t, h, c, x);
             }
         }
