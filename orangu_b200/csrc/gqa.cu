@@ -813,7 +813,7 @@ uint32_t launch_attention(const AttentionArgs &in, bool f32, int sm_count, cudaS
         ++launched;
     }
     if (a.n_short < a.n_seq && tc5) {
-        if (!launch_attention_prompt(a, st)) return 0;
+        if (!launch_attention_prompt(a, sm_count, st)) return 0;
         ++launched;
     } else if (a.n_short < a.n_seq) {
         uint32_t tiles = 0;

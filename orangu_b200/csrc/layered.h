@@ -214,7 +214,7 @@ uint32_t launch_attention(const AttentionArgs &a, bool f32, int sm_count, cudaSt
 // gqa_tc5.cu: the long spans on tcgen05 (bf16)
 cudaError_t attention_prompt_configure();
 bool attention_prompt_supported(uint32_t n_map, uint32_t dim_p, uint32_t vdim_p);
-bool launch_attention_prompt(const AttentionArgs &a, cudaStream_t st);  // false: a tensor map could not be made
+bool launch_attention_prompt(const AttentionArgs &a, int sm_count, cudaStream_t st);  // false: a tensor map could not be made
 int attention_take_status();  // as linear_take_status
 
 // ---- moe.cu ----------------------------------------------------------------------------------------------------------
