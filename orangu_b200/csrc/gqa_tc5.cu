@@ -26,7 +26,8 @@ constexpr int PT_MMA_WARP = 16, PT_TMA_WARP = 17, PT_THREADS = 18 * 32;
 constexpr uint32_t PT_TMEM_S = 0, PT_TMEM_O = 256, PT_TMEM_COLS = 512;
 constexpr float PT_SLACK = 8.0f;  // growth of the maximum (powers of two) that is put up with
 
-constexpr uint32_t PT_SHARED = 320 + 2 * 2 * PT_ROWS * 4;  // mbarriers, items, then a number per stream, half and row
+constexpr uint32_t PT_STAGE = 1024;  // of a warp: 32 rows x 16 columns of output on their way from a thread per row to whole sectors
+constexpr uint32_t PT_SHARED = 320 + 2 * 2 * PT_ROWS * 4 + 48 + 16 * PT_STAGE;  // mbarriers, items, a number per stream, half and row, stages
 struct PtPlan {
     uint32_t nb, nbv, k_bytes, v_bytes, stages, k, v, bar, bytes;  // blocks of 64 columns of a map's keys and of a value; operands of one stage
     __host__ __device__ PtPlan(uint32_t n_map, uint32_t dim_p, uint32_t vdim_p) {
@@ -42,7 +43,7 @@ struct PtPlan {
 };
 // mbarriers, byte offsets from PtPlan::bar
 constexpr uint32_t PT_K_FULL = 0, PT_K_EMPTY = 16, PT_V_FULL = 32, PT_V_EMPTY = 48, PT_S_FULL = 64, PT_P_FULL = 80, PT_O_FULL = 96, PT_Q_FULL = 112, PT_SLOT = 128, PT_ABORT = 132,
-                   PT_ITEMS = 160, PT_EXCHANGE = 320;
+                   PT_ITEMS = 160, PT_EXCHANGE = 320, PT_STAGES = PT_EXCHANGE + 2 * 2 * PT_ROWS * 4 + 48;
 
 // Two fp32 multiply-adds in one instruction.
 __device__ __forceinline__ void fma2(float &d0, float &d1, float a0, float a1, float b, float c) {
@@ -58,34 +59,6 @@ __device__ __forceinline__ void quad_sync(uint32_t id) { asm volatile("bar.sync 
 
 // Sigmoid to a few units in the last place.
 __device__ __forceinline__ float gate_factor(float z) { return __fdividef(1.0f, 1.0f + pow2(z * -1.4426950408889634f)); }
-
-// Entries [c, c + 16) of a head's output, gated, as activations.
-__device__ __forceinline__ void store_head(const AttentionArgs &a, uint64_t t, uint32_t h, uint32_t c, float (&x)[16]) {
-    bf16 *out = static_cast<bf16 *>(a.out) + t * a.out_pitch + (uint64_t)h * a.vdim + c;
-    const bf16 *gate = static_cast<const bf16 *>(a.va) + t * a.va_pitch + a.gate0 + (uint64_t)h * a.vdim + c;
-#pragma unroll
-    for (uint32_t b = 0; b < 2; ++b) {
-        float(&v)[8] = *reinterpret_cast<float(*)[8]>(x + 8 * b);
-        if (a.vdim % 8 == 0) {
-            if (c + 8 * b >= a.vdim) return;
-            if (a.has_gate) {
-                const uint4 z = *reinterpret_cast<const uint4 *>(gate + 8 * b);
-                const uint32_t zw[4] = {z.x, z.y, z.z, z.w};
-#pragma unroll
-                for (int e = 0; e < 4; ++e) {
-                    v[2 * e] *= gate_factor(__uint_as_float(zw[e] << 16));
-                    v[2 * e + 1] *= gate_factor(__uint_as_float(zw[e] & 0xffff0000u));
-                }
-            }
-            store4<bf16>(out + 8 * b, make_float4(v[0], v[1], v[2], v[3]));
-            store4<bf16>(out + 8 * b + 4, make_float4(v[4], v[5], v[6], v[7]));
-        } else {
-#pragma unroll
-            for (uint32_t e = 0; e < 8; ++e)
-                if (c + 8 * b + e < a.vdim) out[8 * b + e] = __float2bfloat16_rn(a.has_gate ? v[e] * gate_factor(from_act(gate[8 * b + e])) : v[e]);
-        }
-    }
-}
 
 // A CTA's piece of work: 128 (two maps) or 256 (one map) consecutive (token, head) rows of one key/value head.  The TMA warp looks
 // it up and leaves it in a ring of four (it is never more than two tiles ahead); the others read it when its first keys are there.
@@ -116,6 +89,91 @@ __device__ __forceinline__ PtItem pt_item(const AttentionArgs &a, uint32_t item,
     w.n_page = (hi + KV_PAGE - 1) / KV_PAGE - w.page0;
     w.n_tiles = (w.n_page + PT_PAGES - 1) / PT_PAGES;
     return w;
+}
+// The output of a warp's 32 rows, 16 columns at a time: gates come and activations go by way of the warp's stage, where two lanes
+// share a row.
+struct RowOut {
+    uint64_t at[2];     // this lane's two rows (lane / 2, and 16 on): first entry of their head in the output ...
+    uint64_t gate[2];   // ... and of their gates
+    bool live[2];
+    bool wide;          // entries come in eights
+};
+__device__ __forceinline__ RowOut row_out(const AttentionArgs &a, const PtItem &w, uint32_t warp_row0) {
+    RowOut ro;
+    const uint32_t per = a.n_head / a.n_kv, lane = threadIdx.x & 31;
+#pragma unroll
+    for (uint32_t k = 0; k < 2; ++k) {
+        const uint32_t i = warp_row0 + 16 * k + lane / 2, f = w.f0 + min(i, w.n_here - 1);
+        const uint64_t t = w.row0 + f / per, h = w.g * per + f % per;
+        ro.live[k] = i < w.n_here;
+        ro.at[k] = t * a.out_pitch + h * a.vdim;
+        ro.gate[k] = t * a.va_pitch + a.gate0 + h * a.vdim;
+    }
+    ro.wide = a.vdim % 8 == 0;
+    return ro;
+}
+// Gates of columns [c, c + 16): a lane's eight of either row.
+__device__ __forceinline__ void load_gates(const AttentionArgs &a, const RowOut &ro, uint32_t c, uint4 (&z)[2]) {
+    const uint32_t e = c + 8 * (threadIdx.x & 1);
+#pragma unroll
+    for (uint32_t k = 0; k < 2; ++k) {
+        const bf16 *p = static_cast<const bf16 *>(a.va) + ro.gate[k] + e;
+        z[k] = make_uint4(0, 0, 0, 0);
+        if (ro.wide && ro.live[k] && e < a.vdim) z[k] = *reinterpret_cast<const uint4 *>(p);
+        if (ro.wide) continue;
+        uint32_t u[4] = {0, 0, 0, 0};
+#pragma unroll
+        for (uint32_t i = 0; i < 8; ++i)
+            if (ro.live[k] && e + i < a.vdim) u[i / 2] |= (uint32_t)__bfloat16_as_ushort(p[i]) << (i % 2 * 16);
+        z[k] = make_uint4(u[0], u[1], u[2], u[3]);
+    }
+}
+// x: columns [c, c + 16) of this lane's own row (row `lane` of the warp), z: load_gates of the same columns.
+__device__ __forceinline__ void store_rows(const AttentionArgs &a, const RowOut &ro, uint8_t *stage, uint32_t c, float (&x)[16], const uint4 (&z)[2]) {
+    const uint32_t lane = threadIdx.x & 31;
+    auto place = [&](uint32_t row, uint32_t half) { return reinterpret_cast<uint4 *>(stage + row * 32 + ((half ^ (row >> 2 & 1)) << 4)); };  // (no bank conflicts either way)
+    if (a.has_gate) {
+#pragma unroll
+        for (uint32_t k = 0; k < 2; ++k) *place(16 * k + lane / 2, lane & 1) = z[k];
+        __syncwarp();
+#pragma unroll
+        for (uint32_t b = 0; b < 2; ++b) {
+            const uint4 g = *place(lane, b);
+            const uint32_t gw[4] = {g.x, g.y, g.z, g.w};
+#pragma unroll
+            for (int e = 0; e < 4; ++e) {
+                x[8 * b + 2 * e] *= gate_factor(__uint_as_float(gw[e] << 16));
+                x[8 * b + 2 * e + 1] *= gate_factor(__uint_as_float(gw[e] & 0xffff0000u));
+            }
+        }
+    }
+#pragma unroll
+    for (uint32_t b = 0; b < 2; ++b) {
+        uint32_t o[4];
+#pragma unroll
+        for (int e = 0; e < 4; ++e) {
+            const __nv_bfloat162 v = __floats2bfloat162_rn(x[8 * b + 2 * e], x[8 * b + 2 * e + 1]);
+            o[e] = *reinterpret_cast<const uint32_t *>(&v);
+        }
+        *place(lane, b) = make_uint4(o[0], o[1], o[2], o[3]);
+    }
+    __syncwarp();
+    const uint32_t e = c + 8 * (lane & 1);
+#pragma unroll
+    for (uint32_t k = 0; k < 2; ++k) {
+        const uint4 v = *place(16 * k + lane / 2, lane & 1);
+        bf16 *p = static_cast<bf16 *>(a.out) + ro.at[k] + e;
+        if (!ro.live[k] || e >= a.vdim) continue;
+        if (ro.wide) {
+            *reinterpret_cast<uint4 *>(p) = v;
+        } else {
+            const uint32_t u[4] = {v.x, v.y, v.z, v.w};
+#pragma unroll
+            for (uint32_t i = 0; i < 8; ++i)
+                if (e + i < a.vdim) p[i] = __ushort_as_bfloat16((unsigned short)(u[i / 2] >> (i % 2 * 16)));
+        }
+    }
+    __syncwarp();
 }
 // Tiles of keys that a stream's rows see: [first, end).  Only with one map may the second stream have no rows.
 template <int NM>
@@ -312,13 +370,20 @@ attention_prompt_kernel(const __grid_constant__ CUtensorMap tm, const __grid_con
                 tmem_ld32(ts, u[0]);
                 tmem_ld32(ts + 32, u[1]);
                 tmem_ld_wait();
-                if (!(whole && j0 + 63 <= w_first && w_last - j0 < win)) {  // keys outside the window of some row
-                    const int hi = pos - j0, lo = hi - win + 1;             // visible columns (pos -1: none)
+                const int hi = pos - j0, lo = hi - win + 1;  // visible columns of the row (pos -1: none)
+                if (!whole || j0 + 63 > w_first) {           // keys after some row
 #pragma unroll
                     for (int c = 0; c < 2; ++c)
 #pragma unroll
                         for (int e = 0; e < 32; ++e)
-                            if (c * 32 + e > hi || c * 32 + e < lo) u[c][e] = 0xff800000u;
+                            if (c * 32 + e > hi) u[c][e] = 0xff800000u;
+                }
+                if (w_last - j0 >= win) {  // keys before some row's window
+#pragma unroll
+                    for (int c = 0; c < 2; ++c)
+#pragma unroll
+                        for (int e = 0; e < 32; ++e)
+                            if (c * 32 + e < lo) u[c][e] = 0xff800000u;
                 }
                 float top[4] = {-INFINITY, -INFINITY, -INFINITY, -INFINITY};
 #pragma unroll
@@ -375,6 +440,14 @@ attention_prompt_kernel(const __grid_constant__ CUtensorMap tm, const __grid_con
             n += w.n_tiles;
             if (more) next = item_at(turn + 1, item + gridDim.x);
             const bool idle = end == first;
+            const RowOut ro = row_out(a, w, w0);
+            uint8_t *stage = smem + pl.bar + PT_STAGES + warp * PT_STAGE;
+            const uint32_t c_first = 16 * (NM == 1 ? part : warp / 4), c_step = NM == 1 ? 32 : 64;  // columns of this warp
+            uint4 gates[2][2] = {};
+            if (a.has_gate) {
+                load_gates(a, ro, c_first, gates[0]);
+                load_gates(a, ro, c_first + c_step, gates[1]);
+            }
             if (idle) ok = ok && mbar_wait_warp(bar + PT_O_FULL + 8 * s, turn & 1u, abort);
             if (more) load_query(next);
             if (!idle) ok = ok && mbar_wait_warp(bar + PT_O_FULL + 8 * s, turn & 1u, abort);
@@ -382,50 +455,61 @@ attention_prompt_kernel(const __grid_constant__ CUtensorMap tm, const __grid_con
 
             pair_sync(pair);  // (the last maxima have been read)
             xchg[own] = l;
-            const uint32_t f = w.f0 + (live ? i_row : 0), h = w.g * per + f % per;
-            const uint64_t t = w.row0 + f / per;
+            auto put = [&](uint32_t c, float (&x)[16], uint32_t turn) {
+                store_rows(a, ro, stage, c, x, gates[turn]);
+                if (a.has_gate && c + 2 * c_step < a.vdim_p) load_gates(a, ro, c + 2 * c_step, gates[turn]);
+            };
             if constexpr (NM == 1) {
                 pair_sync(pair);
                 const float fac = 1.0f / (l + xchg[other]);
-                for (uint32_t c = 16 * part; c < a.vdim_p && ok && !idle; c += 32) {
-                    uint32_t o[16];
-                    tmem_ld16(to + s * 128 + c, o);
-                    tmem_ld_wait();
-                    float x[16];
+                if (ok && !idle)
 #pragma unroll
-                    for (int e = 0; e < 16; ++e) x[e] = __uint_as_float(o[e]) * fac;
-                    if (live) store_head(a, t, h, c, x);
-                }
+                    for (uint32_t k = 0; k < 4; ++k) {
+                        const uint32_t c = c_first + k * c_step;
+                        if (c >= a.vdim_p) break;
+                        uint32_t o[16];
+                        tmem_ld16(to + s * 128 + c, o);
+                        tmem_ld_wait();
+                        float x[16];
+#pragma unroll
+                        for (int e = 0; e < 16; ++e) x[e] = __uint_as_float(o[e]) * fac;
+                        put(c, x, k % 2);
+                    }
                 pair_sync(pair);  // (the sums have been read)
             } else {  // four warps share 32 rows: both maps' outputs are in the same lanes of tensor memory
                 quad_sync(9 + quad);
                 const float fac0 = 1.0f / (xchg[0] + xchg[PT_ROWS]), fac1 = a.map_weight / (xchg[2 * PT_ROWS] + xchg[3 * PT_ROWS]);
-                auto difference = [&](uint32_t c, float (&x)[16]) {
-                    uint32_t o0[16], o1[16];
-                    tmem_ld16(to + c, o0);
-                    tmem_ld16(to + 128 + c, o1);
-                    tmem_ld_wait();
+                float q = 0.0f, x[2][16];
+                if (ok)
 #pragma unroll
-                    for (int e = 0; e < 16; ++e) x[e] = __uint_as_float(o0[e]) * fac0 - __uint_as_float(o1[e]) * fac1;
-                };
-                float q = 0.0f, x[16];
-                for (uint32_t c = 16 * (warp / 4); c < a.vdim_p && ok; c += 64) {
-                    difference(c, x);
+                    for (uint32_t k = 0; k < 2; ++k) {
+                        const uint32_t c = c_first + k * c_step;
+                        if (c >= a.vdim_p) break;
+                        uint32_t o0[16], o1[16];
+                        tmem_ld16(to + c, o0);
+                        tmem_ld16(to + 128 + c, o1);
+                        tmem_ld_wait();
 #pragma unroll
-                    for (int e = 0; e < 16; ++e) q += x[e] * x[e];  // columns past vdim are zero: so are the values there
-                }
-                quad_sync(9 + quad);  // (the sums have been read)
+                        for (int e = 0; e < 16; ++e) {  // columns past vdim are zero: so are the values there
+                            x[k][e] = __uint_as_float(o0[e]) * fac0 - __uint_as_float(o1[e]) * fac1;
+                            q += x[k][e] * x[k][e];
+                        }
+                    }
+                tc_fence_before();
+                quad_sync(9 + quad);  // the sums and the outputs have been read: the next weights may come
                 xchg[own] = q;
                 quad_sync(9 + quad);
                 const float gain = inv_rms((xchg[0] + xchg[PT_ROWS]) + (xchg[2 * PT_ROWS] + xchg[3 * PT_ROWS]), a.vdim, a.eps) * a.head_gain;
-                for (uint32_t c = 16 * (warp / 4); c < a.vdim_p && ok; c += 64) {
-                    difference(c, x);
+                if (ok)
 #pragma unroll
-                    for (int e = 0; e < 16; ++e) x[e] *= gain;
-                    if (live) store_head(a, t, h, c, x);
-                }
-                tc_fence_before();
-                quad_sync(9 + quad);  // nobody's next weights come before everyone has read the outputs
+                    for (uint32_t k = 0; k < 2; ++k) {
+                        const uint32_t c = c_first + k * c_step;
+                        if (c >= a.vdim_p) break;
+#pragma unroll
+                        for (int e = 0; e < 16; ++e) x[k][e] *= gain;
+                        put(c, x[k], k);
+                    }
+                quad_sync(9 + quad);  // (the squares have been read)
             }
             tc_fence_before();
             w = next;

@@ -36,8 +36,8 @@ def rotate(x, pos, base, dims):
 
 
 def visible(i, j, window):
-    """Does position i see position j?"""
-    return 0 <= i - j < window
+    """Does position i see position j?  (j may be an array.)"""
+    return (i - j >= 0) & (i - j < window)
 
 
 def normed_rotated(x, w, mx, eps):
@@ -50,7 +50,7 @@ def softmax_average(q, k, v, scale, window):
     """One map of one head: q, k [n, dim], v [n, vdim] -> [n, vdim]."""
     out = np.zeros((len(q), v.shape[1]))
     for i in range(len(q)):
-        js = [j for j in range(len(k)) if visible(i, j, window)]
+        js = np.flatnonzero(visible(i, np.arange(len(k)), window))
         s = (k[js] @ q[i]) * scale
         p = np.exp(s - s.max())
         out[i] = (p / p.sum()) @ v[js]

@@ -174,6 +174,26 @@ def test_many_prompts_and_single_tokens_in_one_step(backend, dtype):
     m.close()
 
 
+@pytest.mark.parametrize("kind", ("differential", "gated"))
+def test_more_pieces_of_prompts_than_processors(backend, kind):
+    """One long prompt, then many short ones (with one map every second stream of rows is empty), on sixteen key/value heads: every
+    CTA of the prompt attention takes several pieces."""
+    layer = N.differential(heads=16, kv_heads=16, dim=16, vdim=24, window=150, rot_dims=16) if kind == "differential" else N.gated(heads=32, kv_heads=16, dim=24, window=150, rot_dims=16)
+    cfg = N.config([layer], width=64)
+    w = N.weights(cfg, 48)
+    long, short = N.tokens(cfg, 1500, 49), [N.tokens(cfg, 64 + i % 9, 50 + i) for i in range(13)]
+    m = make(backend, cfg, w, "bfloat16", pool=4096, rows=2048, seq=2048)
+    want = P.forward(cfg, N.values(w), long)[0]
+    places = list(range(0, 1500, 7)) + [1499]
+    assert error(m.forward_rows([m.new_kv_cache(1536, paged=True)], [long], places), want[places]) < TOL["bfloat16"]
+    kvs = [m.new_kv_cache(96, paged=True) for _ in short]
+    ends = np.cumsum([len(p) for p in short]) - 1
+    got = m.forward_rows(kvs, short, ends)
+    for g, p in zip(got, short):
+        assert error(g[None], P.forward(cfg, N.values(w), p)[0][-1:]) < TOL["bfloat16"]
+    m.close()
+
+
 @pytest.mark.parametrize("dtype", DTYPES)
 def test_many_single_tokens(backend, dtype):
     """A decode batch wide enough for the tensor-core products, at unequal lengths."""
