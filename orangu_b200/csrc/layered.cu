@@ -840,6 +840,7 @@ int check_block(ob_ctx *ctx, const ob_layered_desc &c, uint32_t i) {
         if ((rc = check_dense(ctx, x.w_gate, E, H * x.vdim, at + "mixer gate"))) return rc;
     } else if (x.kind == OB_MIXER_ATTENTION) {
         if (!G || H % G) return fail(ctx, OB_ERR_INVALID, "layered model: " + at + "n_kv_head does not divide n_head");
+        if (!(x.scale > 0)) return fail(ctx, OB_ERR_INVALID, "layered model: " + at + "scale must be positive");
         if (x.n_map != 1 && x.n_map != 2) return fail(ctx, OB_ERR_UNSUPPORTED, "layered model: " + at + "one or two maps per head");
         if (!x.q_norm || !x.k_norm) return fail(ctx, OB_ERR_INVALID, "layered model: " + at + "query or key norm missing");
         if (!attention_supported(x.dim, x.vdim)) return fail(ctx, OB_ERR_UNSUPPORTED, "layered model: " + at + "attention head too large");

@@ -437,6 +437,7 @@ def test_descriptions_the_library_refuses(backend):
         (lambda d, b: setattr(b[0].mixer, "n_kv_head", 3), "divide"),
         (lambda d, b: setattr(b[0].mixer, "n_map", 3), "maps"),
         (lambda d, b: setattr(b[1].mixer, "q_norm", None), "norm missing"),
+        (lambda d, b: setattr(b[1].mixer, "scale", 0.0), "scale"),
         (lambda d, b: setattr(b[1].mixer, "vdim", 24), "wo|keys|gate"),
         (lambda d, b: setattr(b[1].mixer, "rot_dims", 42), "rot_dims"),
         (lambda d, b: setattr(b[1], "post_norm1", None), "two kinds"),
