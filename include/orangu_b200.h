@@ -31,8 +31,10 @@ extern "C" {
 
 /* 2: ob_model_desc gained rope_freqs (layout change); the GGUF, static-attention and KV-copy entry points were added.
  * 3: ob_model_desc gained tp_presliced.
- * 5: the layered descriptions gained softmax attention over cached keys and values, sequential blocks and mixtures of experts. */
-#define OB_ABI_VERSION 5u
+ * 5: the layered descriptions gained softmax attention over cached keys and values, sequential blocks and mixtures of experts.
+ * 6: they gained state-space and time-mixing layers, two mixers in a block, normed inputs, and kept tokens, sinks, soft caps, shared
+ *    keys and values of attention. */
+#define OB_ABI_VERSION 6u
 
 typedef enum ob_status {
     OB_OK = 0,
@@ -253,16 +255,19 @@ typedef struct ob_model_desc {
 /* ------------------------------------------------- models given as a list of layers
  * Designs whose layers are not all alike: every layer names its token mixer and its feed-forward and carries their sizes,
  * constants and tensors.  Two kinds of block: parallel, x += mixer(h) + ff(h) with h = x / rms(x) * norm_gain; and sequential with
- * normed outputs (post_norm1 given), x += residual_mult * mixer(x) / rms(mixer(x)) * post_norm1, then the same with the
- * feed-forward and post_norm2.  No counterpart in the reference.  The result is an ob_model like any other: caches, batching, sampling,
+ * normed outputs (post_norm1 given), x += residual_mult * m / rms(m) * post_norm1 with m = mixer(h), then the same with the
+ * feed-forward and post_norm2; h is x, or (pre_norm1, pre_norm2 given) x / rms(x) * pre_norm.  No counterpart in the reference.  The result is an ob_model like any other: caches, batching, sampling,
  * captured decode graphs and the slot pool are the same calls.  Matrices are bfloat16, out_dim rows of in_dim; vectors f32. */
 #define OB_TYPE_BF16 30u /* ob_matrix_desc.ggml_type of these matrices */
 #define OB_MIXER_LATENT_ATTENTION 1u
 #define OB_MIXER_RETENTION 2u
 #define OB_MIXER_ATTENTION 3u /* softmax attention over cached keys and values, n_head / n_kv_head query heads per key/value head */
+#define OB_MIXER_STATE_SPACE 4u /* short causal convolution, then S = exp(-exp(a_log) dt) S + dt B x^T, y = S^T C + d_skip x per head (state [dim][vdim]) */
+#define OB_MIXER_TIME_MIXING 5u /* projections of h mixed with the previous token's h; o = (S + diag(bonus) k v^T)^T r, S = diag(w) S + k v^T (vdim = dim) */
 #define OB_FF_CLAMPED_GLU 0u /* g = min(gate, limit), u = clamp(up, -limit, limit); g * sigmoid(alpha g) * (u + 1) */
 #define OB_FF_RELU2 1u       /* max(up, 0)^2 */
-#define OB_FF_EXPERTS 2u     /* n_expert_used of n_expert silu(gate) * up feed-forwards; a chosen one reads the input times its score */
+#define OB_FF_EXPERTS 2u     /* n_expert_used of n_expert silu(gate) * up feed-forwards, weighted as router_softmax says */
+#define OB_FF_GELU_GLU 3u    /* gelu(gate) * up, the tanh form */
 
 typedef struct ob_mixer_desc {
     uint32_t kind;            /* OB_MIXER_* */
@@ -270,7 +275,7 @@ typedef struct ob_mixer_desc {
     uint32_t vdim;            /* value dimensions per head */
     uint32_t rot_dim;         /* latent attention: rotated query/key dimensions per head, in addition to dim */
     uint32_t kv_rank;         /* latent attention: size of the cached latent */
-    uint32_t window;          /* attention: a position sees itself and window - 1 before it; 0 = all before it */
+    uint32_t window;          /* attention: a position sees itself and window - 1 before it (and keep_first); 0 = all before it */
     uint32_t rot_dims;        /* entries that rotate, from the first: of q and k (retention, attention), of the rot_dim part (latent attention) */
     uint32_t rot_interleaved; /* 1: pairs (2i, 2i+1); 0: pairs (i, i + rot_dims/2) */
     float scale;              /* attention: factor of the scores */
@@ -281,7 +286,8 @@ typedef struct ob_mixer_desc {
     ob_matrix_desc wk, wv;    /* retention [n_head*dim], [n_head*vdim]; attention [n_kv_head*n_map*dim], [n_kv_head*vdim] (no data:
                                * the values are the keys as projected, before norm and rotation; n_map 1, vdim = dim) */
     ob_matrix_desc w_gate;    /* retention [n_head*vdim] (silu of it scales the normed output); latent attention [n_head] (sigmoid of it scales a head);
-                               * attention [n_head*vdim] (sigmoid of it scales the output; no data: no gate) */
+                               * attention [n_head*vdim] or [n_head] (sigmoid of it scales the output or a head; no data: no gate);
+                               * time mixing [n_head*dim] (silu of it scales the normed output) */
     ob_matrix_desc w_dkv;     /* latent attention [kv_rank+rot_dim]: latent, then the rotated key part all heads share */
     const float *kv_norm;     /* latent attention [kv_rank]: RMS-norm weight of the latent */
     ob_matrix_desc w_uk, w_uv; /* latent attention [n_head*dim], [n_head*vdim] from kv_rank */
@@ -290,8 +296,29 @@ typedef struct ob_mixer_desc {
     uint32_t n_map;           /* attention: softmax maps per head over the same values, 1 or 2 */
     float map_weight;         /* attention with two maps: o = map 1 - map_weight * map 2, then o / rms(o) * head_gain per head */
     float head_gain;
-    const float *q_norm, *k_norm; /* attention [dim]: RMS-norm weights of every query and key vector before rotation */
+    const float *q_norm, *k_norm; /* attention [dim]: RMS-norm weights of every query and key vector before rotation; NULL: no norm */
     const float *q_bias, *k_bias, *v_bias, *o_bias; /* attention: added in the projections; NULL: none */
+    /* attention, one map: */
+    uint32_t qk_norm_whole;   /* 1: the norms go over a token's whole projection, weights [n_head*dim] and [n_kv_head*dim] */
+    uint32_t keep_first;      /* the first tokens of a sequence that stay visible beyond the window */
+    uint32_t kv_layer;        /* 1 + an earlier layer whose cached keys and values are used (wk, wv without data); 0: own ones */
+    float softcap;            /* > 0: score = softcap * tanh(score / softcap) */
+    const float *sink;        /* [n_head]: exp(sink) is added to the softmax denominator; NULL: none */
+    /* attention: frequencies of the pairs instead of the powers of rot_base, and a factor of cos and sin (0: 1) */
+    const double *rot_freqs;  /* [rot_dims/2] or NULL */
+    float rot_gain;
+    /* state space: dim is the state's size, vdim a head's width, inner = n_head*vdim */
+    uint32_t n_group;         /* groups of B and C; divides n_head */
+    uint32_t n_norm_group;    /* equal parts of inner that are normed; divides inner */
+    uint32_t conv_taps;
+    ob_matrix_desc w_in;      /* [z: inner | x: inner | B: n_group*dim | C: n_group*dim | dt: n_head] */
+    const float *conv_w, *conv_b; /* [2 n_group*dim + inner][conv_taps] (the last tap meets the current token), [2 n_group*dim + inner] */
+    const float *dt_bias, *a_log, *d_skip; /* [n_head] */
+    const float *out_norm;    /* state space [inner], time mixing [n_head*dim]: factors of the normed output */
+    /* time mixing: r, k, v, gate are wq, wk, wv, w_gate; input s is h + (h' - h) mu_s with h' the previous token's h */
+    const float *mu_r, *mu_k, *mu_v, *mu_g, *mu_w; /* [n_embd] */
+    ob_matrix_desc w_decay1, w_decay2; /* [rank], [n_head*dim] from rank: decay w = exp(-exp(w_decay2 tanh(w_decay1 mix) + decay0)) */
+    const float *decay0, *bonus;       /* [n_head*dim] */
 } ob_mixer_desc;
 
 typedef struct ob_block_desc {
@@ -299,14 +326,20 @@ typedef struct ob_block_desc {
     ob_mixer_desc mixer;
     uint32_t n_ff;            /* of one expert when there are experts; 0: no feed-forward */
     float glu_limit, glu_alpha; /* OB_FF_CLAMPED_GLU */
-    ob_matrix_desc w_gate, w_up, w_down; /* gate: OB_FF_CLAMPED_GLU only; none with experts */
+    ob_matrix_desc w_gate, w_up, w_down; /* gate: not OB_FF_RELU2; none with experts */
     ob_matrix_desc side_gate, side_proj; /* per-layer token input (side_dim > 0): y = side_proj (gelu_tanh(side_gate x) * e), x += y / rms(y) * side_norm */
     const float *side_norm;   /* [n_embd] */
     const float *post_norm1, *post_norm2; /* [n_embd] factors of the normed outputs; post_norm1 makes the block sequential */
-    uint32_t ff_kind;         /* OB_FF_*; parallel blocks have the first kind, sequential ones the others */
-    uint32_t n_expert, n_expert_used; /* OB_FF_EXPERTS: the n_expert_used largest of sigmoid(w_router x) are chosen, scores as they are */
+    uint32_t ff_kind;         /* OB_FF_*; parallel blocks have OB_FF_CLAMPED_GLU, sequential ones the others */
+    uint32_t n_expert, n_expert_used; /* OB_FF_EXPERTS: the n_expert_used largest of w_router x are chosen */
     ob_matrix_desc w_router;  /* [n_expert] */
     const ob_matrix_desc *expert_gate, *expert_up, *expert_down; /* [n_expert] matrices each */
+    uint32_t router_softmax;  /* 0: a chosen expert reads the input times sigmoid of its logit; 1: outputs are weighted by the softmax over the chosen logits */
+    uint32_t shared_ff;       /* > 0: size of a further expert that every token uses; its output is scaled by sigmoid(w_shared_scale x) (router_softmax 1 only) */
+    ob_matrix_desc shared_gate, shared_up, shared_down, w_shared_scale; /* the last [1] */
+    const float *pre_norm1, *pre_norm2; /* [n_embd] sequential blocks: factors of the normed inputs; NULL: a sublayer reads x itself */
+    ob_mixer_desc mixer2;     /* sequential blocks: a second mixer beside the first, both read the same input; kind 0: none */
+    float mixer_scale, mixer2_scale;    /* with mixer2: factors of the two mixers' outputs */
 } ob_block_desc;
 
 typedef struct ob_layered_desc {

@@ -38,8 +38,8 @@ class ModelDesc(C.Structure):
 
 
 TYPE_BF16 = 30
-MIXER_LATENT_ATTENTION, MIXER_RETENTION, MIXER_ATTENTION = 1, 2, 3
-FF_CLAMPED_GLU, FF_RELU2, FF_EXPERTS = 0, 1, 2
+MIXER_LATENT_ATTENTION, MIXER_RETENTION, MIXER_ATTENTION, MIXER_STATE_SPACE, MIXER_TIME_MIXING = 1, 2, 3, 4, 5
+FF_CLAMPED_GLU, FF_RELU2, FF_EXPERTS, FF_GELU_GLU = 0, 1, 2, 3
 
 
 class MixerDesc(C.Structure):
@@ -47,14 +47,21 @@ class MixerDesc(C.Structure):
         ("scale", C.c_float), ("rot_base", C.c_double), ("decay", C.c_void_p)] + [
         (n, MatrixDesc) for n in ("wq", "wk", "wv", "w_gate", "w_dkv")] + [("kv_norm", C.c_void_p)] + [(n, MatrixDesc) for n in ("w_uk", "w_uv", "wo")] + [
         ("n_kv_head", C.c_uint32), ("n_map", C.c_uint32), ("map_weight", C.c_float), ("head_gain", C.c_float)] + [
-        (n, C.c_void_p) for n in ("q_norm", "k_norm", "q_bias", "k_bias", "v_bias", "o_bias")]
+        (n, C.c_void_p) for n in ("q_norm", "k_norm", "q_bias", "k_bias", "v_bias", "o_bias")] + [
+        (n, C.c_uint32) for n in ("qk_norm_whole", "keep_first", "kv_layer")] + [("softcap", C.c_float), ("sink", C.c_void_p)] + [
+        ("rot_freqs", C.c_void_p), ("rot_gain", C.c_float)] + [(n, C.c_uint32) for n in ("n_group", "n_norm_group", "conv_taps")] + [
+        ("w_in", MatrixDesc)] + [(n, C.c_void_p) for n in ("conv_w", "conv_b", "dt_bias", "a_log", "d_skip", "out_norm")] + [
+        (n, C.c_void_p) for n in ("mu_r", "mu_k", "mu_v", "mu_g", "mu_w")] + [("w_decay1", MatrixDesc), ("w_decay2", MatrixDesc)] + [
+        (n, C.c_void_p) for n in ("decay0", "bonus")]
 
 
 class BlockDesc(C.Structure):
     _fields_ = [("norm_gain", C.c_float), ("mixer", MixerDesc), ("n_ff", C.c_uint32), ("glu_limit", C.c_float), ("glu_alpha", C.c_float)] + [
         (n, MatrixDesc) for n in ("w_gate", "w_up", "w_down", "side_gate", "side_proj")] + [("side_norm", C.c_void_p)] + [
         (n, C.c_void_p) for n in ("post_norm1", "post_norm2")] + [(n, C.c_uint32) for n in ("ff_kind", "n_expert", "n_expert_used")] + [
-        ("w_router", MatrixDesc)] + [(n, C.POINTER(MatrixDesc)) for n in ("expert_gate", "expert_up", "expert_down")]
+        ("w_router", MatrixDesc)] + [(n, C.POINTER(MatrixDesc)) for n in ("expert_gate", "expert_up", "expert_down")] + [
+        (n, C.c_uint32) for n in ("router_softmax", "shared_ff")] + [(n, MatrixDesc) for n in ("shared_gate", "shared_up", "shared_down", "w_shared_scale")] + [
+        (n, C.c_void_p) for n in ("pre_norm1", "pre_norm2")] + [("mixer2", MixerDesc), ("mixer_scale", C.c_float), ("mixer2_scale", C.c_float)]
 
 
 class LayeredDesc(C.Structure):

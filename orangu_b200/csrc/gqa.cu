@@ -36,8 +36,8 @@ __global__ void __launch_bounds__(PREP_WARPS * 32) attention_prep_kernel(Attenti
     pdl_release();
     pdl_wait();
     const uint32_t warp = threadIdx.x >> 5, lane = threadIdx.x & 31, t = blockIdx.x, i = blockIdx.y * PREP_WARPS + warp;
-    const uint32_t n_q = a.n_head * a.n_map, n_k = a.n_kv * a.n_map;
-    if (i >= n_q + n_k + a.n_kv) return;
+    const uint32_t n_q = a.n_head * a.n_map, n_k = a.own_kv ? a.n_kv * a.n_map : 0, n_v = a.own_kv ? a.n_kv : 0;
+    if (i >= n_q + n_k + n_v) return;
     const uint32_t pos = a.positions[t];
     const float *y = a.y + (uint64_t)t * a.y_pitch;
     TA *cache = static_cast<TA *>(a.cache) + page_at(a, a.tables[t][pos / KV_PAGE], 0) + (uint64_t)(pos % KV_PAGE) * a.row;
@@ -64,14 +64,25 @@ __global__ void __launch_bounds__(PREP_WARPS * 32) attention_prep_kernel(Attenti
         v[d] = e;
         s += e * e;
     }
-    const float f = inv_rms(warp_sum(s), a.dim, a.eps);
-    for (uint32_t d = lane; d < a.dim; d += 32) v[d] *= f * w[d];
+    if (w) {
+        uint32_t n = a.dim;
+        if (a.norm_whole) {  // every warp adds up the whole projection
+            n *= query ? n_q : n_k;
+            const float *all = query ? y : y + (uint64_t)n_q * a.dim;
+            s = 0.0f;
+            for (uint32_t d = lane; d < n; d += 32) s += all[d] * all[d];
+            w += (uint64_t)(query ? i : k) * a.dim;
+        }
+        const float f = inv_rms(warp_sum(s), n, a.eps);
+        for (uint32_t d = lane; d < a.dim; d += 32) v[d] *= f * w[d];
+    }
     __syncwarp();
     const float2 *cs = a.rot.table + (uint64_t)pos * (a.rot.dims / 2);
     for (uint32_t d = lane; d < a.dim_p; d += 32) dst[d] = to_act<TA>(d < a.dim ? rotated(v, d, a.rot, cs) : 0.0f);
 }
 
 // The same for sizes in eights (head sizes, half of the rotated entries): `group` neighbouring lanes per vector, eight entries each.
+// With norms over whole projections a CTA has all vectors of its token (gridDim.y 1) and goes over them twice.
 constexpr int PREP_THREADS = 256;
 __device__ __forceinline__ void load_eight(const float *p, float (&v)[8]) {
     const float4 a = reinterpret_cast<const float4 *>(p)[0], b = reinterpret_cast<const float4 *>(p)[1];
@@ -85,67 +96,102 @@ template <typename TA>
 __global__ void __launch_bounds__(PREP_THREADS) attention_prep_vec_kernel(AttentionArgs a, uint32_t group) {
     pdl_release();
     pdl_wait();
-    const uint32_t t = blockIdx.x, c = threadIdx.x & (group - 1), i = blockIdx.y * (PREP_THREADS / group) + threadIdx.x / group;
-    const uint32_t n_q = a.n_head * a.n_map, n_k = a.n_kv * a.n_map, d = 8 * c;
-    const bool exists = i < n_q + n_k + a.n_kv, value = i >= n_q + n_k, query = i < n_q;
+    __shared__ float red[33];
+    const uint32_t t = blockIdx.x, c = threadIdx.x & (group - 1);
+    const uint32_t n_q = a.n_head * a.n_map, n_k = a.own_kv ? a.n_kv * a.n_map : 0, n = n_q + n_k + (a.own_kv ? a.n_kv : 0), d = 8 * c;
     const uint32_t pos = a.positions[t];
     const float *y = a.y + (uint64_t)t * a.y_pitch;
     TA *cache = static_cast<TA *>(a.cache) + page_at(a, a.tables[t][pos / KV_PAGE], 0) + (uint64_t)(pos % KV_PAGE) * a.row;
     const uint64_t head = (uint64_t)KV_PAGE * a.row;  // from one key/value head to the next within a page
-    if (exists && value) {
-        const uint32_t g = i - n_q - n_k;
-        TA *dst = cache + g * head + a.n_map * a.dim_p;
-        for (uint32_t e = d; e < a.vdim; e += 8 * group) {
-            float v[8];
-            if (a.has_v) {
-                constexpr uint32_t P = 16 / sizeof(TA);
-                const TA *src = static_cast<const TA *>(a.va) + (uint64_t)t * a.va_pitch + (uint64_t)g * a.vdim + e;
+    float f_q = 1.0f, f_k = 1.0f;
+    if (a.norm_whole) {
+        float s[2] = {0.0f, 0.0f};
+#pragma unroll 4
+        for (uint32_t e = 4 * threadIdx.x; e < (n_q + n_k) * a.dim; e += 4 * PREP_THREADS) s[e >= n_q * a.dim] += sq4(*reinterpret_cast<const float4 *>(y + e));
+        f_q = inv_rms(block_sum(s[0], red), n_q * a.dim, a.eps);
+        if (n_k) f_k = inv_rms(block_sum(s[1], red), n_k * a.dim, a.eps);
+    }
+    for (uint32_t i0 = blockIdx.y * (PREP_THREADS / group); i0 < n; i0 += gridDim.y * (PREP_THREADS / group)) {
+        const uint32_t i = i0 + threadIdx.x / group;
+        const bool exists = i < n, value = i >= n_q + n_k, query = i < n_q;
+        if (exists && value) {
+            const uint32_t g = i - n_q - n_k;
+            TA *dst = cache + g * head + a.n_map * a.dim_p;
+            for (uint32_t e = d; e < a.vdim; e += 8 * group) {
+                float v[8];
+                if (a.has_v) {
+                    constexpr uint32_t P = 16 / sizeof(TA);
+                    const TA *src = static_cast<const TA *>(a.va) + (uint64_t)t * a.va_pitch + (uint64_t)g * a.vdim + e;
 #pragma unroll
-                for (uint32_t k = 0; k < 8; k += P) *reinterpret_cast<uint4 *>(dst + e + k) = *reinterpret_cast<const uint4 *>(src + k);
-            } else {
-                load_eight(y + (uint64_t)(n_q + g) * a.dim + e, v);
-                store_eight<TA>(dst + e, v);
+                    for (uint32_t k = 0; k < 8; k += P) *reinterpret_cast<uint4 *>(dst + e + k) = *reinterpret_cast<const uint4 *>(src + k);
+                } else {
+                    load_eight(y + (uint64_t)(n_q + g) * a.dim + e, v);
+                    store_eight<TA>(dst + e, v);
+                }
             }
         }
-    }
-    const bool mine = exists && !value && d < a.dim;
-    float v[8] = {}, s = 0.0f;
-    if (mine) load_eight(y + (uint64_t)i * a.dim + d, v);
+        const bool mine = exists && !value && d < a.dim;
+        float v[8] = {}, s = 0.0f;
+        if (mine) load_eight(y + (uint64_t)i * a.dim + d, v);
+        if (a.q_norm) {
+            float f = query ? f_q : f_k;
+            if (!a.norm_whole) {
 #pragma unroll
-    for (int e = 0; e < 8; ++e) s += v[e] * v[e];
-    for (uint32_t o = group / 2; o > 0; o >>= 1) s += __shfl_xor_sync(0xffffffffu, s, o);
-    const float f = inv_rms(s, a.dim, a.eps);
-    if (mine) {
-        float w[8];
-        load_eight((query ? a.q_norm : a.k_norm) + d, w);
+                for (int e = 0; e < 8; ++e) s += v[e] * v[e];
+                for (uint32_t o = group / 2; o > 0; o >>= 1) s += __shfl_xor_sync(0xffffffffu, s, o);
+                f = inv_rms(s, a.dim, a.eps);
+            }
+            if (mine) {
+                float w[8];
+                const float *all = query ? a.q_norm : a.k_norm;
+                load_eight(all + (a.norm_whole ? (uint64_t)(query ? i : i - n_q) * a.dim : 0) + d, w);
 #pragma unroll
-        for (int e = 0; e < 8; ++e) v[e] *= f * w[e];
-    }
-    const uint32_t half = a.rot.dims / 2;
-    const bool low = d < half, turns = d < a.rot.dims;
-    float other[8];  // the entries half of the rotated ones away
-    const uint32_t lane = threadIdx.x & 31, from = turns ? (low ? lane + half / 8 : lane - half / 8) : lane;
-#pragma unroll
-    for (int e = 0; e < 8; ++e) other[e] = __shfl_sync(0xffffffffu, v[e], from);
-    if (mine && turns) {
-        const float2 *cs = a.rot.table + (uint64_t)pos * half + (low ? d : d - half);
-#pragma unroll
-        for (int e = 0; e < 8; ++e) {
-            const float2 r = cs[e];
-            v[e] = low ? v[e] * r.x - other[e] * r.y : v[e] * r.x + other[e] * r.y;
+                for (int e = 0; e < 8; ++e) v[e] *= f * w[e];
+            }
         }
-    }
-    if (exists && !value && d < a.dim_p) {  // (zeros from dim on)
-        const uint32_t k = i - n_q;
-        store_eight<TA>((query ? static_cast<TA *>(a.q) + ((uint64_t)t * n_q + i) * a.dim_p : cache + k / a.n_map * head + k % a.n_map * a.dim_p) + d, v);
+        const uint32_t half = a.rot.dims / 2;
+        const bool low = d < half, turns = d < a.rot.dims;
+        if (a.rot.interleaved) {
+            if (mine && turns) {
+                const float2 *cs = a.rot.table + (uint64_t)pos * half + d / 2;
+#pragma unroll
+                for (int e = 0; e < 8; e += 2) {
+                    const float2 r = cs[e / 2];
+                    const float u = v[e], w = v[e + 1];
+                    v[e] = u * r.x - w * r.y, v[e + 1] = w * r.x + u * r.y;
+                }
+            }
+        } else {
+            float other[8];  // the entries half of the rotated ones away
+            const uint32_t lane = threadIdx.x & 31, from = turns ? (low ? lane + half / 8 : lane - half / 8) : lane;
+#pragma unroll
+            for (int e = 0; e < 8; ++e) other[e] = __shfl_sync(0xffffffffu, v[e], from);
+            if (mine && turns) {
+                const float2 *cs = a.rot.table + (uint64_t)pos * half + (low ? d : d - half);
+#pragma unroll
+                for (int e = 0; e < 8; ++e) {
+                    const float2 r = cs[e];
+                    v[e] = low ? v[e] * r.x - other[e] * r.y : v[e] * r.x + other[e] * r.y;
+                }
+            }
+        }
+        if (exists && !value && d < a.dim_p) {  // (zeros from dim on)
+            const uint32_t k = i - n_q;
+            store_eight<TA>((query ? static_cast<TA *>(a.q) + ((uint64_t)t * n_q + i) * a.dim_p : cache + k / a.n_map * head + k % a.n_map * a.dim_p) + d, v);
+        }
     }
 }
 
-// ---- the end of a head: both maps put together, gate, store ----------------------------------------------------------------------
+// ---- the end of a head: both maps put together, gates, store ----------------------------------------------------------------------
 __device__ __forceinline__ float gate_of(const AttentionArgs &a, uint64_t t, uint32_t h, uint32_t c, bool f32) {
     const uint64_t at = t * a.va_pitch + a.gate0 + (uint64_t)h * a.vdim + c;
     const float z = f32 ? static_cast<const float *>(a.va)[at] : from_act(static_cast<const bf16 *>(a.va)[at]);
     return 1.0f / (1.0f + expf(-z));
+}
+
+// Factor of a whole head of token t (one map).
+__device__ __forceinline__ float head_factor(const AttentionArgs &a, uint64_t t, uint32_t h) {
+    return a.head_gain * (a.head_gate ? 1.0f / (1.0f + expf(-a.head_gate[t * a.y_pitch + h])) : 1.0f);
 }
 
 // ---- plain form: one CTA per (token, head) --------------------------------------------------------------------------------------
@@ -159,9 +205,12 @@ __global__ void __launch_bounds__(AP_THREADS) attention_plain_kernel(AttentionAr
     pdl_release();
     pdl_wait();
     const uint32_t t = blockIdx.x / a.n_head, h = blockIdx.x % a.n_head, g = h / (a.n_head / a.n_kv), warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
-    const uint32_t pos = a.positions[t], lo = first_seen(pos, a.window), hi = pos + 1;
+    const uint32_t pos = a.positions[t], lo = first_seen(pos, a.window), kept = min(a.keep, lo), hi = kept + pos + 1 - lo;
     const int32_t *table = a.tables[t];
-    auto row_of = [&](uint32_t j) { return static_cast<const TA *>(a.cache) + page_at(a, table[j / KV_PAGE], g) + (uint64_t)(j % KV_PAGE) * a.row; };
+    auto row_of = [&](uint32_t i) {  // of the i'th visible position
+        const uint32_t j = i < kept ? i : lo + i - kept;
+        return static_cast<const TA *>(a.cache) + page_at(a, table[j / KV_PAGE], g) + (uint64_t)(j % KV_PAGE) * a.row;
+    };
     for (uint32_t map = 0; map < a.n_map; ++map) {
         const TA *qg = static_cast<const TA *>(a.q) + (((uint64_t)t * a.n_head + h) * a.n_map + map) * a.dim_p;
         float *o = acc + map * a.vdim;
@@ -170,14 +219,15 @@ __global__ void __launch_bounds__(AP_THREADS) attention_plain_kernel(AttentionAr
         for (uint32_t i = threadIdx.x; i < a.vdim; i += blockDim.x) o[i] = 0.0f;
         float m = -INFINITY, l = 0.0f;
         __syncthreads();
-        for (uint32_t j0 = lo; j0 < hi; j0 += AP_KEYS) {
+        for (uint32_t j0 = 0; j0 < hi; j0 += AP_KEYS) {
             const uint32_t n = min((uint32_t)AP_KEYS, hi - j0);
             for (uint32_t j = warp; j < n; j += AP_THREADS / 32) {
                 const TA *k = row_of(j0 + j) + map * a.dim_p;
                 float s = 0.0f;
                 for (uint32_t i = lane; i < a.dim; i += 32) s = fmaf(q[i], from_act(k[i]), s);
                 s = warp_sum(s);
-                if (lane == 0) p[j] = s * a.scale;
+                s *= a.scale;
+                if (lane == 0) p[j] = a.softcap > 0.0f ? a.softcap * tanhf(s / a.softcap) : s;
             }
             __syncthreads();
             const float own = threadIdx.x < n ? p[threadIdx.x] : -INFINITY;
@@ -196,9 +246,14 @@ __global__ void __launch_bounds__(AP_THREADS) attention_plain_kernel(AttentionAr
             }
             __syncthreads();
         }
+        if (a.sink) {
+            const float top = fmaxf(m, a.sink[h]), keep = expf(m - top);
+            l = l * keep + expf(a.sink[h] - top);
+            for (uint32_t i = threadIdx.x; i < a.vdim; i += blockDim.x) o[i] *= keep;
+        }
         for (uint32_t i = threadIdx.x; i < a.vdim; i += blockDim.x) o[i] /= l;
     }
-    float f = 1.0f;
+    float f = a.n_map == 1 ? head_factor(a, t, h) : 1.0f;
     if (a.n_map == 2) {
         float s = 0.0f;
         for (uint32_t i = threadIdx.x; i < a.vdim; i += blockDim.x) {
@@ -265,7 +320,7 @@ __device__ __forceinline__ float2 peer_load2(uint32_t addr) {
 }
 
 // NV: columns of a value in sixteens (what goes past vdim_p is computed from whatever follows in shared memory and dropped).
-template <int NM, int NV>
+template <int NM, int NV, bool CAP>
 __global__ void __launch_bounds__(ST_THREADS) attention_step_kernel(AttentionArgs a, uint32_t splits, uint32_t stages) {
     constexpr bool APART = NM == 2 && NV > 8;  // the maps of wide values are different warps' business: two accumulators would not fit
     constexpr int LM = APART ? 1 : NM;         // maps per warp
@@ -290,8 +345,8 @@ __global__ void __launch_bounds__(ST_THREADS) attention_step_kernel(AttentionArg
     if (f0 >= n_flat) return;  // (the same for the whole cluster)
     const uint32_t n_here = min((uint32_t)ST_ROWS, n_flat - f0), pos0 = a.positions[row0];
     const int32_t *table = a.tables[row0];
-    const uint32_t lo = first_seen(pos0 + f0 / per, a.window), hi = pos0 + (f0 + n_here - 1) / per + 1;
-    const uint32_t page0 = lo / KV_PAGE, n_page = (hi + KV_PAGE - 1) / KV_PAGE - page0;
+    const PageList pages = page_list(pos0 + f0 / per, pos0 + (f0 + n_here - 1) / per, a.window, a.keep, 1);
+    const uint32_t n_page = pages.n;
     const uint32_t unit = rank * UNITS + (APART ? warp >> 1 : warp), n_unit = splits * UNITS, map0 = APART ? warp & 1u : 0u;
     const uint32_t pieces = KV_PAGE * a.row / 8, qs = smem_addr(smem), ring = qs + ST_ROWS * pl.q_row + warp * pl.ring, page_bytes = KV_PAGE * a.row * 2;
 
@@ -307,7 +362,7 @@ __global__ void __launch_bounds__(ST_THREADS) attention_step_kernel(AttentionArg
     uint32_t next_page = unit, next_stage = ring;  // of the next load
     auto load = [&] {  // this warp's next page
         if (next_page < n_page) {
-            const bf16 *src = static_cast<const bf16 *>(a.cache) + page_at(a, table[page0 + next_page], g) + 8 * lane;
+            const bf16 *src = static_cast<const bf16 *>(a.cache) + page_at(a, table[pages[next_page]], g) + 8 * lane;
             uint32_t dst = next_stage + 16 * lane, i = lane;
             for (; i + 96 < pieces; i += 128, src += 1024, dst += 2048)
 #pragma unroll
@@ -327,8 +382,8 @@ __global__ void __launch_bounds__(ST_THREADS) attention_step_kernel(AttentionArg
     else cp_wait<0>();
     __syncthreads();
 
-    const float scale2 = a.scale * LOG2E;
-    const int win = a.window ? (int)a.window : 0x7fffffff;
+    const float scale2 = a.scale * LOG2E, cap = a.softcap * LOG2E, cap_in = CAP ? 2.0f * scale2 / a.softcap : 0.0f;
+    const int win = a.window ? (int)a.window : 0x7fffffff, keep = (int)a.keep;
     const int r0 = (int)(lane / 4), p0 = r0 < (int)n_here ? (int)(pos0 + (f0 + r0) / per) : -1, p1 = r0 + 8 < (int)n_here ? (int)(pos0 + (f0 + r0 + 8) / per) : -1;
     float o[LM][NV][2][4], m0[LM], m1[LM], l0[LM], l1[LM];
 #pragma unroll
@@ -352,7 +407,7 @@ __global__ void __launch_bounds__(ST_THREADS) attention_step_kernel(AttentionArg
         else if (stages == 3) cp_wait<2>();
         else cp_wait<1>();
         __syncwarp();
-        const int j0 = (int)((page0 + page) * KV_PAGE);
+        const int j0 = (int)(pages[page] * KV_PAGE);
         uint32_t ph[LM][4], pr[LM][4];
 #pragma unroll
         for (int m = 0; m < LM; ++m) {
@@ -378,8 +433,11 @@ __global__ void __launch_bounds__(ST_THREADS) attention_step_kernel(AttentionArg
 #pragma unroll
                 for (int e = 0; e < 2; ++e) {
                     const int j = j0 + 8 * h + 2 * (int)(lane & 3) + e;
-                    c[h][e] = j <= p0 && p0 - j < win ? (c[h][e] + d[h][e]) * scale2 : -INFINITY;
-                    c[h][2 + e] = j <= p1 && p1 - j < win ? (c[h][2 + e] + d[h][2 + e]) * scale2 : -INFINITY;
+                    float s0 = c[h][e] + d[h][e], s1 = c[h][2 + e] + d[h][2 + e];
+                    if constexpr (CAP) s0 = soft_cap(s0, cap_in, cap), s1 = soft_cap(s1, cap_in, cap);
+                    else s0 *= scale2, s1 *= scale2;
+                    c[h][e] = j <= p0 && (p0 - j < win || j < keep) ? s0 : -INFINITY;
+                    c[h][2 + e] = j <= p1 && (p1 - j < win || j < keep) ? s1 : -INFINITY;
                     b0 = fmaxf(b0, c[h][e]);
                     b1 = fmaxf(b1, c[h][2 + e]);
                 }
@@ -453,7 +511,10 @@ __global__ void __launch_bounds__(ST_THREADS) attention_step_kernel(AttentionArg
             const bool part = lane < n_unit;
             float2 ml = make_float2(-INFINITY, 0.0f);
             if (part) ml = peer_load2(peer_addr(smem_addr(&stat[part_warp][APART ? 0 : m][r]), part_rank));
-            const float top = warp_max(ml.x), w = part && ml.x > -INFINITY ? pow2(ml.x - top) : 0.0f, inv = 1.0f / warp_sum(w * ml.y);
+            const float top = warp_max(ml.x), w = part && ml.x > -INFINITY ? pow2(ml.x - top) : 0.0f;
+            float sum_w = warp_sum(w * ml.y);
+            if (a.sink) sum_w += pow2(a.sink[g * per + (f0 + r) % per] * LOG2E - top);
+            const float inv = 1.0f / sum_w;
             const uint32_t base = peer_addr(qs + ST_ROWS * pl.q_row + part_warp * pl.ring + (uint32_t)((APART ? 0 : m) * ST_ROWS + r) * pl.o_row * 4, part ? part_rank : 0);
 #pragma unroll
             for (int i = 0; i < NC; ++i) sum[m][i] = make_float4(0, 0, 0, 0);
@@ -471,7 +532,9 @@ __global__ void __launch_bounds__(ST_THREADS) attention_step_kernel(AttentionArg
                 }
             }
         }
-        float f = 1.0f;
+        const uint64_t t = row0 + (f0 + r) / per;
+        const uint32_t h = g * per + (f0 + r) % per;
+        float f = NM == 1 ? head_factor(a, t, h) : 1.0f;
         if constexpr (NM == 2) {
             float s = 0.0f;
 #pragma unroll
@@ -483,8 +546,6 @@ __global__ void __launch_bounds__(ST_THREADS) attention_step_kernel(AttentionArg
             }
             f = inv_rms(warp_sum(s), a.vdim, a.eps) * a.head_gain;
         }
-        const uint64_t t = row0 + (f0 + r) / per;
-        const uint32_t h = g * per + (f0 + r) % per;
         bf16 *out = static_cast<bf16 *>(a.out) + t * a.out_pitch + (uint64_t)h * a.vdim;
 #pragma unroll
         for (int i = 0; i < NC; ++i) {
@@ -514,7 +575,7 @@ struct SpPlan {
     }
 };
 
-template <int NM, int NV>
+template <int NM, int NV, bool CAP>
 __global__ void __launch_bounds__(SP_THREADS, NV <= 8 ? 2 : 1) attention_span_kernel(AttentionArgs a) {
     constexpr int RW = SP_THREADS / 32 / NM, M = 16 * RW;  // warps over the rows
     extern __shared__ __align__(16) uint8_t smem[];
@@ -535,8 +596,8 @@ __global__ void __launch_bounds__(SP_THREADS, NV <= 8 ? 2 : 1) attention_span_ke
     if (f0 >= n_flat) return;
     const uint32_t n_here = min((uint32_t)M, n_flat - f0), pos0 = a.positions[row0];
     const int32_t *table = a.tables[row0];
-    const uint32_t lo = first_seen(pos0 + f0 / per, a.window), hi = pos0 + (f0 + n_here - 1) / per + 1;
-    const uint32_t page0 = lo / KV_PAGE, n_page = (hi + KV_PAGE - 1) / KV_PAGE - page0, n_tiles = (n_page + SP_PAGES - 1) / SP_PAGES;
+    const PageList pages = page_list(pos0 + f0 / per, pos0 + (f0 + n_here - 1) / per, a.window, a.keep, SP_PAGES);
+    const uint32_t n_page = pages.n, n_tiles = (n_page + SP_PAGES - 1) / SP_PAGES;
     const uint32_t qs = smem_addr(smem), pieces = KV_PAGE * a.row / 8;
     {   // queries
         const uint32_t per_row = NM * a.dim_p / 8;
@@ -550,14 +611,14 @@ __global__ void __launch_bounds__(SP_THREADS, NV <= 8 ? 2 : 1) attention_span_ke
         const uint32_t dst = qs + pl.k + (it & 1u) * pl.stage;
 #pragma unroll
         for (uint32_t p = 0; p < SP_PAGES; ++p) {  // past the last page: the last one again, which nobody sees there
-            const bf16 *src = static_cast<const bf16 *>(a.cache) + page_at(a, table[page0 + min(it * SP_PAGES + p, n_page - 1)], g);
+            const bf16 *src = static_cast<const bf16 *>(a.cache) + page_at(a, table[pages[min(it * SP_PAGES + p, n_page - 1)]], g);
             for (uint32_t i = threadIdx.x; i < pieces; i += SP_THREADS) cp16(dst + (p * pieces + i) * 16, src + 8 * i, true);
         }
     };
     load(0);
     cp_commit();
-    const float scale2 = a.scale * LOG2E;
-    const int win = a.window ? (int)a.window : 0x7fffffff;
+    const float scale2 = a.scale * LOG2E, cap = a.softcap * LOG2E, cap_in = CAP ? 2.0f * scale2 / a.softcap : 0.0f;
+    const int win = a.window ? (int)a.window : 0x7fffffff, keep = (int)a.keep;
     const uint32_t wr = rw * 16, ra = wr + lane / 4;
     const int p0 = ra < n_here ? (int)(pos0 + (f0 + ra) / per) : -1, p1 = ra + 8 < n_here ? (int)(pos0 + (f0 + ra + 8) / per) : -1;
     const bool live = wr < n_here;
@@ -579,9 +640,9 @@ __global__ void __launch_bounds__(SP_THREADS, NV <= 8 ? 2 : 1) attention_span_ke
         cp_commit();
         cp_wait<1>();
         __syncthreads();  // this tile is there
-        const int j0 = (int)((page0 + it * SP_PAGES) * KV_PAGE);
+        const int j0 = (int)(pages[it * SP_PAGES] * KV_PAGE);
         const uint32_t kb = qs + pl.k + (it & 1u) * pl.stage;
-        if (live && j0 <= w_last && (long long)j0 + SP_KEYS - 1 > (long long)w_first - win) {  // one of the warp's rows sees one of these keys
+        if (live && j0 <= w_last && (j0 < keep || (long long)j0 + SP_KEYS - 1 > (long long)w_first - win)) {  // one of the warp's rows sees one of these keys
             float c[SP_KEYS / 8][4];
 #pragma unroll
             for (int n = 0; n < SP_KEYS / 8; ++n) c[n][0] = c[n][1] = c[n][2] = c[n][3] = 0.0f;
@@ -604,8 +665,11 @@ __global__ void __launch_bounds__(SP_THREADS, NV <= 8 ? 2 : 1) attention_span_ke
 #pragma unroll
                 for (int e = 0; e < 2; ++e) {
                     const int j = j0 + 8 * n + 2 * (int)(lane & 3) + e;
-                    c[n][e] = inside || (j <= p0 && p0 - j < win) ? c[n][e] * scale2 : -INFINITY;
-                    c[n][2 + e] = inside || (j <= p1 && p1 - j < win) ? c[n][2 + e] * scale2 : -INFINITY;
+                    float s0 = c[n][e], s1 = c[n][2 + e];
+                    if constexpr (CAP) s0 = soft_cap(s0, cap_in, cap), s1 = soft_cap(s1, cap_in, cap);
+                    else s0 *= scale2, s1 *= scale2;
+                    c[n][e] = inside || (j <= p0 && (p0 - j < win || j < keep)) ? s0 : -INFINITY;
+                    c[n][2 + e] = inside || (j <= p1 && (p1 - j < win || j < keep)) ? s1 : -INFINITY;
                     b0 = fmaxf(b0, c[n][e]);
                     b1 = fmaxf(b1, c[n][2 + e]);
                 }
@@ -652,7 +716,14 @@ __global__ void __launch_bounds__(SP_THREADS, NV <= 8 ? 2 : 1) attention_span_ke
     cp_wait<0>();
     l0 += __shfl_xor_sync(0xffffffffu, l0, 1), l0 += __shfl_xor_sync(0xffffffffu, l0, 2);
     l1 += __shfl_xor_sync(0xffffffffu, l1, 1), l1 += __shfl_xor_sync(0xffffffffu, l1, 2);
-    float f[2] = {1.0f / l0, 1.0f / l1};
+    float f[2];
+#pragma unroll
+    for (int r = 0; r < 2; ++r) {
+        const uint32_t i = min(ra + 8 * r, n_here - 1), h = g * per + (f0 + i) % per;
+        float l = r ? l1 : l0;
+        if (a.sink) l += pow2(a.sink[h] * LOG2E - (r ? m1 : m0));
+        f[r] = (NM == 1 ? head_factor(a, row0 + (f0 + i) / per, h) : 1.0f) / l;
+    }
     if constexpr (NM == 2) {  // the second map's rows go to the first map's warps through shared memory
         const uint32_t o_row = a.vdim_p + 8;
         float *ex = reinterpret_cast<float *>(smem + pl.k);
@@ -726,14 +797,12 @@ using StKernel = void (*)(AttentionArgs, uint32_t, uint32_t);
 using SpKernel = void (*)(AttentionArgs);
 constexpr int N_FORM = 6;
 const uint32_t FORMS[N_FORM] = {2, 4, 6, 8, 12, 16};  // columns of a value in sixteens
-const StKernel ST_KERNELS[2][N_FORM] = {{attention_step_kernel<1, 2>, attention_step_kernel<1, 4>, attention_step_kernel<1, 6>, attention_step_kernel<1, 8>,
-                                         attention_step_kernel<1, 12>, attention_step_kernel<1, 16>},
-                                        {attention_step_kernel<2, 2>, attention_step_kernel<2, 4>, attention_step_kernel<2, 6>, attention_step_kernel<2, 8>,
-                                         attention_step_kernel<2, 12>, attention_step_kernel<2, 16>}};
-const SpKernel SP_KERNELS[2][N_FORM] = {{attention_span_kernel<1, 2>, attention_span_kernel<1, 4>, attention_span_kernel<1, 6>, attention_span_kernel<1, 8>,
-                                         attention_span_kernel<1, 12>, attention_span_kernel<1, 16>},
-                                        {attention_span_kernel<2, 2>, attention_span_kernel<2, 4>, attention_span_kernel<2, 6>, attention_span_kernel<2, 8>,
-                                         attention_span_kernel<2, 12>, attention_span_kernel<2, 16>}};
+#define OB_FORMS(KERNEL, NM, CAP) {KERNEL<NM, 2, CAP>, KERNEL<NM, 4, CAP>, KERNEL<NM, 6, CAP>, KERNEL<NM, 8, CAP>, KERNEL<NM, 12, CAP>, KERNEL<NM, 16, CAP>}
+constexpr int N_KIND = 3;  // one map, two maps, one map with a soft cap
+const StKernel ST_KERNELS[N_KIND][N_FORM] = {OB_FORMS(attention_step_kernel, 1, false), OB_FORMS(attention_step_kernel, 2, false), OB_FORMS(attention_step_kernel, 1, true)};
+const SpKernel SP_KERNELS[N_KIND][N_FORM] = {OB_FORMS(attention_span_kernel, 1, false), OB_FORMS(attention_span_kernel, 2, false), OB_FORMS(attention_span_kernel, 1, true)};
+#undef OB_FORMS
+int kind_of(const AttentionArgs &a) { return a.n_map == 2 ? 1 : a.softcap > 0.0f ? 2 : 0; }
 int form_of(uint32_t vdim_p) {
     int f = 0;
     while (f < N_FORM && 16 * FORMS[f] < vdim_p) ++f;
@@ -751,7 +820,7 @@ cudaError_t attention_configure() {
         auto set = [&](auto k) {
             if (e == cudaSuccess) e = cudaFuncSetAttribute(k, cudaFuncAttributeMaxDynamicSharedMemorySize, MAX_SMEM);
         };
-        for (int m = 0; m < 2; ++m)
+        for (int m = 0; m < N_KIND; ++m)
             for (int f = 0; f < N_FORM; ++f) set(ST_KERNELS[m][f]), set(SP_KERNELS[m][f]);
         set(attention_plain_kernel<float>), set(attention_plain_kernel<bf16>);
         set(attention_prep_kernel<float>), set(attention_prep_kernel<bf16>);
@@ -764,12 +833,12 @@ uint32_t attention_cache_row(uint32_t n_map, uint32_t dim_p, uint32_t vdim_p) { 
 bool attention_supported(uint32_t dim, uint32_t vdim) { return (uint64_t)PREP_WARPS * dim * 4 <= MAX_SMEM && (uint64_t)(dim + 2 * vdim + AP_KEYS) * 4 <= MAX_SMEM; }
 
 void launch_attention_prep(const AttentionArgs &a, bool f32, cudaStream_t st) {
-    const uint32_t n = (a.n_head + a.n_kv) * a.n_map + a.n_kv;
-    if (a.dim % 8 == 0 && a.vdim % 8 == 0 && a.rot.dims % 16 == 0 && !a.rot.interleaved && a.dim_p <= 256) {
+    const uint32_t n = a.n_head * a.n_map + (a.own_kv ? a.n_kv * (a.n_map + 1) : 0);
+    if (a.dim % 8 == 0 && a.vdim % 8 == 0 && a.rot.dims % (a.rot.interleaved ? 8 : 16) == 0 && a.dim_p <= 256) {
         uint32_t group = 1;
         while (8 * group < a.dim_p) group *= 2;
         const uint32_t each = PREP_THREADS / group;
-        launch_pdl(f32 ? attention_prep_vec_kernel<float> : attention_prep_vec_kernel<bf16>, dim3(a.T, (n + each - 1) / each), PREP_THREADS, 0, st, a, group);
+        launch_pdl(f32 ? attention_prep_vec_kernel<float> : attention_prep_vec_kernel<bf16>, dim3(a.T, a.norm_whole ? 1 : (n + each - 1) / each), PREP_THREADS, 0, st, a, group);
         return;
     }
     const dim3 grid(a.T, (n + PREP_WARPS - 1) / PREP_WARPS);
@@ -794,7 +863,7 @@ uint32_t launch_attention(const AttentionArgs &in, bool f32, int sm_count, cudaS
         else
             for (uint32_t s = 0; s < a.n_short; ++s) tiles += (a.h_spans[s].n * per + ST_ROWS - 1) / ST_ROWS;
         // few tiles: clusters share their keys, down to two pages per warp
-        const uint32_t units = ST_WARPS, reach = (a.window ? std::min(a.max_pos, a.window) : a.max_pos) / KV_PAGE + 1;
+        const uint32_t units = ST_WARPS, reach = (a.window ? std::min(a.max_pos, a.window + a.keep) : a.max_pos) / KV_PAGE + 1;
         uint32_t splits = 1;
         while (splits < ST_MAX_CLUSTER && (uint64_t)tiles * a.n_kv * splits * 2 <= 2ull * sm_count && reach > units * splits * 2) splits *= 2;
         cudaLaunchAttribute at[2];
@@ -809,7 +878,7 @@ uint32_t launch_attention(const AttentionArgs &in, bool f32, int sm_count, cudaS
         cfg.stream = st;
         cfg.attrs = at;
         cfg.numAttrs = splits > 1 ? 2 : 1;
-        cudaLaunchKernelEx(&cfg, ST_KERNELS[a.n_map - 1][form], a, splits, stages);
+        cudaLaunchKernelEx(&cfg, ST_KERNELS[kind_of(a)][form], a, splits, stages);
         ++launched;
     }
     if (a.n_short < a.n_seq && tc5) {
@@ -818,7 +887,7 @@ uint32_t launch_attention(const AttentionArgs &in, bool f32, int sm_count, cudaS
     } else if (a.n_short < a.n_seq) {
         uint32_t tiles = 0;
         for (uint32_t s = a.n_short; s < a.n_seq; ++s) tiles += (a.h_spans[s].n * per + sp.rows - 1) / sp.rows;
-        launch_pdl(SP_KERNELS[a.n_map - 1][form], dim3(tiles, a.n_kv), SP_THREADS, sp.bytes, st, a);
+        launch_pdl(SP_KERNELS[kind_of(a)][form], dim3(tiles, a.n_kv), SP_THREADS, sp.bytes, st, a);
         ++launched;
     }
     return launched;

@@ -63,15 +63,17 @@ __device__ __forceinline__ float gate_factor(float z) { return __fdividef(1.0f, 
 // A CTA's piece of work: 128 (two maps) or 256 (one map) consecutive (token, head) rows of one key/value head.  The TMA warp looks
 // it up and leaves it in a ring of four (it is never more than two tiles ahead); the others read it when its first keys are there.
 struct PtItem {
-    uint32_t row0, f0, n_here, pos0, page0, n_page, n_tiles, g;
+    uint32_t row0, f0, n_here, pos0, g;
+    PageList pages;  // the kept ones fill whole tiles
+    __device__ __forceinline__ uint32_t n_tiles() const { return (pages.n + PT_PAGES - 1) / PT_PAGES; }
 };
 __device__ __forceinline__ PtItem pt_read(const uint8_t *smem, uint32_t turn) {
     const volatile uint32_t *p = reinterpret_cast<const volatile uint32_t *>(smem + PT_ITEMS) + turn % 4 * 8;
-    return PtItem{p[0], p[1], p[2], p[3], p[4], p[5], p[6], p[7]};
+    return PtItem{p[0], p[1], p[2], p[3], p[4], PageList{p[5], p[6], p[7]}};
 }
 __device__ __forceinline__ void pt_write(uint8_t *smem, uint32_t turn, const PtItem &w) {
     volatile uint32_t *p = reinterpret_cast<volatile uint32_t *>(smem + PT_ITEMS) + turn % 4 * 8;
-    p[0] = w.row0, p[1] = w.f0, p[2] = w.n_here, p[3] = w.pos0, p[4] = w.page0, p[5] = w.n_page, p[6] = w.n_tiles, p[7] = w.g;
+    p[0] = w.row0, p[1] = w.f0, p[2] = w.n_here, p[3] = w.pos0, p[4] = w.g, p[5] = w.pages.kept, p[6] = w.pages.gap, p[7] = w.pages.n;
 }
 template <int NM>
 __device__ __forceinline__ PtItem pt_item(const AttentionArgs &a, uint32_t item, uint32_t n_row_tiles) {  // one warp; every lane gets the answer
@@ -84,10 +86,7 @@ __device__ __forceinline__ PtItem pt_item(const AttentionArgs &a, uint32_t item,
     w.row0 = sp.row0, w.g = item % a.n_kv;
     w.n_here = min(M, sp.n * per - w.f0);
     w.pos0 = a.positions[w.row0];
-    const uint32_t lo = first_seen(w.pos0 + w.f0 / per, a.window), hi = w.pos0 + (w.f0 + w.n_here - 1) / per + 1;
-    w.page0 = lo / KV_PAGE;
-    w.n_page = (hi + KV_PAGE - 1) / KV_PAGE - w.page0;
-    w.n_tiles = (w.n_page + PT_PAGES - 1) / PT_PAGES;
+    w.pages = page_list(w.pos0 + w.f0 / per, w.pos0 + (w.f0 + w.n_here - 1) / per, a.window, a.keep, PT_PAGES);
     return w;
 }
 // The output of a warp's 32 rows, 16 columns at a time: gates come and activations go by way of the warp's stage, where two lanes
@@ -178,17 +177,17 @@ __device__ __forceinline__ void store_rows(const AttentionArgs &a, const RowOut 
 // Tiles of keys that a stream's rows see: [first, end).  Only with one map may the second stream have no rows.
 template <int NM>
 __device__ __forceinline__ uint32_t pt_first(const AttentionArgs &a, const PtItem &w, uint32_t s) {
-    if (NM == 2 || s == 0 || w.n_here <= PT_ROWS) return 0;
-    return (first_seen(w.pos0 + (w.f0 + PT_ROWS) / (a.n_head / a.n_kv), a.window) / KV_PAGE - w.page0) / PT_PAGES;
+    if (NM == 2 || s == 0 || w.n_here <= PT_ROWS || a.keep) return 0;
+    return (first_seen(w.pos0 + (w.f0 + PT_ROWS) / (a.n_head / a.n_kv), a.window) / KV_PAGE - w.pages.gap) / PT_PAGES;
 }
 template <int NM>
 __device__ __forceinline__ uint32_t pt_end(const AttentionArgs &a, const PtItem &w, uint32_t s) {
-    if (NM == 2) return w.n_tiles;
-    if (s == 1) return w.n_here > PT_ROWS ? w.n_tiles : 0;
-    return ((w.pos0 + (w.f0 + min(w.n_here, PT_ROWS) - 1) / (a.n_head / a.n_kv)) / KV_PAGE - w.page0) / PT_PAGES + 1;
+    if (NM == 2) return w.n_tiles();
+    if (s == 1) return w.n_here > PT_ROWS ? w.n_tiles() : 0;
+    return ((w.pos0 + (w.f0 + min(w.n_here, PT_ROWS) - 1) / (a.n_head / a.n_kv)) / KV_PAGE - w.pages.gap) / PT_PAGES + 1;
 }
 
-template <int NM>
+template <int NM, bool CAP>
 __global__ void __launch_bounds__(PT_THREADS, 1)
 attention_prompt_kernel(const __grid_constant__ CUtensorMap tm, const __grid_constant__ AttentionArgs a, uint32_t n_row_tiles) {
     extern __shared__ uint8_t smem_raw[];
@@ -228,12 +227,12 @@ attention_prompt_kernel(const __grid_constant__ CUtensorMap tm, const __grid_con
             if (lane == 0) {
                 const int32_t *table = a.tables[w.row0];
                 pt_write(smem + pl.bar, turn, w);
-                for (uint32_t i = 0; i < w.n_tiles && ok; ++i, ++n) {
+                for (uint32_t i = 0; i < w.n_tiles() && ok; ++i, ++n) {
                     const uint32_t st = n % pl.stages, par = ((n / pl.stages) & 1u) ^ 1u;
                     int32_t y[PT_PAGES];
 #pragma unroll
                     for (uint32_t p = 0; p < PT_PAGES; ++p)  // past the last page: the last one again, which nobody sees there
-                        y[p] = (int32_t)((table[w.page0 + min(i * PT_PAGES + p, w.n_page - 1)] * a.n_kv + w.g) * KV_PAGE);
+                        y[p] = (int32_t)((table[w.pages[min(i * PT_PAGES + p, w.pages.n - 1)]] * a.n_kv + w.g) * KV_PAGE);
                     if (n >= pl.stages && !(ok = mbar_wait(bar + PT_K_EMPTY + 8 * st, par, abort))) break;
                     mbar_expect_tx(bar + PT_K_FULL + 8 * st, pl.k_bytes);
                     for (uint32_t b = 0; b < NM * pl.nb; ++b) {
@@ -277,7 +276,7 @@ attention_prompt_kernel(const __grid_constant__ CUtensorMap tm, const __grid_con
             const PtItem w = pt_read(smem + pl.bar, turn);
             auto uniform = [](uint32_t v) { return __shfl_sync(0xffffffffu, v, 0); };
             const uint32_t first0 = uniform(pt_first<NM>(a, w, 0)), first1 = uniform(pt_first<NM>(a, w, 1)), end0 = uniform(pt_end<NM>(a, w, 0)), end1 = uniform(pt_end<NM>(a, w, 1));
-            const uint32_t n_tiles = uniform(w.n_tiles);
+            const uint32_t n_tiles = uniform(w.n_tiles());
             ok = mbar_wait_warp(bar + PT_Q_FULL, turn & 1u, abort) && mbar_wait_warp(bar + PT_Q_FULL + 8, turn & 1u, abort);
 #pragma unroll
             for (uint32_t s = 0; s < 2; ++s)
@@ -316,7 +315,8 @@ attention_prompt_kernel(const __grid_constant__ CUtensorMap tm, const __grid_con
     } else {
         const uint32_t s = warp / 8, part = warp / 4 % 2, quad = warp % 4, r = quad * 32 + lane, pair = 1 + s * 4 + quad;
         const int win = a.window ? (int)min(a.window, 0x3fffffffu) : 0x3fffffff;
-        const float scale2 = a.scale * 1.4426950408889634f;  // weights are powers of two of the scaled score
+        constexpr float LOG2E = 1.4426950408889634f;  // weights are powers of two of the scaled score
+        const float scale2 = CAP ? 1.0f : a.scale * LOG2E, cap = a.softcap * LOG2E, cap_in = CAP ? 2.0f * LOG2E * a.scale / a.softcap : 0.0f;
         const uint32_t lanes = tmem + ((quad * 32) << 16), ts = lanes + PT_TMEM_S + s * PT_KEYS + part * 64, to = lanes + PT_TMEM_O;
         volatile float *xchg = reinterpret_cast<volatile float *>(smem + pl.bar + PT_EXCHANGE) + r;  // a number per stream, half and row
         const uint32_t own = (2 * s + part) * PT_ROWS, other = (2 * s + (part ^ 1u)) * PT_ROWS;
@@ -365,12 +365,18 @@ attention_prompt_kernel(const __grid_constant__ CUtensorMap tm, const __grid_con
                     continue;
                 }
                 tc_fence_after();
-                const int j0 = (int)((w.page0 + i * PT_PAGES) * KV_PAGE + part * 64);
+                const int j0 = (int)(w.pages[i * PT_PAGES] * KV_PAGE + part * 64);
                 uint32_t u[2][32];
                 tmem_ld32(ts, u[0]);
                 tmem_ld32(ts + 32, u[1]);
                 tmem_ld_wait();
-                const int hi = pos - j0, lo = hi - win + 1;  // visible columns of the row (pos -1: none)
+                if constexpr (CAP) {
+#pragma unroll
+                    for (int c = 0; c < 2; ++c)
+#pragma unroll
+                        for (int e = 0; e < 32; ++e) u[c][e] = __float_as_uint(soft_cap(__uint_as_float(u[c][e]), cap_in, cap));
+                }
+                const int hi = pos - j0, lo = hi - win + 1, kept = (int)a.keep - j0;  // visible columns of the row: [lo, hi] and below kept (pos -1: none)
                 if (!whole || j0 + 63 > w_first) {           // keys after some row
 #pragma unroll
                     for (int c = 0; c < 2; ++c)
@@ -383,7 +389,7 @@ attention_prompt_kernel(const __grid_constant__ CUtensorMap tm, const __grid_con
                     for (int c = 0; c < 2; ++c)
 #pragma unroll
                         for (int e = 0; e < 32; ++e)
-                            if (c * 32 + e < lo) u[c][e] = 0xff800000u;
+                            if (c * 32 + e < lo && c * 32 + e >= kept) u[c][e] = 0xff800000u;
                 }
                 float top[4] = {-INFINITY, -INFINITY, -INFINITY, -INFINITY};
 #pragma unroll
@@ -437,7 +443,7 @@ attention_prompt_kernel(const __grid_constant__ CUtensorMap tm, const __grid_con
             // learns that from the end of the item.
             const bool more = item + gridDim.x < n_items;
             PtItem next{};
-            n += w.n_tiles;
+            n += w.n_tiles();
             if (more) next = item_at(turn + 1, item + gridDim.x);
             const bool idle = end == first;
             const RowOut ro = row_out(a, w, w0);
@@ -454,6 +460,13 @@ attention_prompt_kernel(const __grid_constant__ CUtensorMap tm, const __grid_con
             tc_fence_after();
 
             pair_sync(pair);  // (the last maxima have been read)
+            float gain = 1.0f;  // of the row's head
+            if constexpr (NM == 1) {
+                const uint32_t f = w.f0 + min(i_row, w.n_here - 1), h = w.g * per + f % per;
+                if (a.sink && part == 0) l += pow2(a.sink[h] * LOG2E - m);
+                gain = a.head_gain;
+                if (a.head_gate) gain *= gate_factor(a.head_gate[(uint64_t)(w.row0 + f / per) * a.y_pitch + h]);
+            }
             xchg[own] = l;
             auto put = [&](uint32_t c, float (&x)[16], uint32_t turn) {
                 store_rows(a, ro, stage, c, x, gates[turn]);
@@ -461,7 +474,7 @@ attention_prompt_kernel(const __grid_constant__ CUtensorMap tm, const __grid_con
             };
             if constexpr (NM == 1) {
                 pair_sync(pair);
-                const float fac = 1.0f / (l + xchg[other]);
+                const float fac = gain / (l + xchg[other]);
                 if (ok && !idle)
 #pragma unroll
                     for (uint32_t k = 0; k < 4; ++k) {
@@ -499,7 +512,7 @@ attention_prompt_kernel(const __grid_constant__ CUtensorMap tm, const __grid_con
                 quad_sync(9 + quad);  // the sums and the outputs have been read: the next weights may come
                 xchg[own] = q;
                 quad_sync(9 + quad);
-                const float gain = inv_rms((xchg[0] + xchg[PT_ROWS]) + (xchg[2 * PT_ROWS] + xchg[3 * PT_ROWS]), a.vdim, a.eps) * a.head_gain;
+                gain = inv_rms((xchg[0] + xchg[PT_ROWS]) + (xchg[2 * PT_ROWS] + xchg[3 * PT_ROWS]), a.vdim, a.eps) * a.head_gain;
                 if (ok)
 #pragma unroll
                     for (uint32_t k = 0; k < 2; ++k) {
@@ -529,8 +542,10 @@ attention_prompt_kernel(const __grid_constant__ CUtensorMap tm, const __grid_con
 cudaError_t attention_prompt_configure() {
     static PerDeviceOnce once;
     return once.run([] {
-        cudaError_t e = cudaFuncSetAttribute(attention_prompt_kernel<1>, cudaFuncAttributeMaxDynamicSharedMemorySize, 226 * 1024);
-        return e != cudaSuccess ? e : cudaFuncSetAttribute(attention_prompt_kernel<2>, cudaFuncAttributeMaxDynamicSharedMemorySize, 226 * 1024);
+        cudaError_t e = cudaSuccess;
+        for (auto k : {attention_prompt_kernel<1, false>, attention_prompt_kernel<2, false>, attention_prompt_kernel<1, true>})
+            if (e == cudaSuccess) e = cudaFuncSetAttribute(k, cudaFuncAttributeMaxDynamicSharedMemorySize, 226 * 1024);
+        return e;
     });
 }
 
@@ -543,7 +558,7 @@ bool launch_attention_prompt(const AttentionArgs &a, int sm_count, cudaStream_t 
     CUtensorMap tm;
     if (!make_map_2d(&tm, CU_TENSOR_MAP_DATA_TYPE_BFLOAT16, 2, a.cache, a.row, (uint64_t)a.n_pages * a.n_kv * KV_PAGE, (uint64_t)a.row * 2, 64, KV_PAGE, CU_TENSOR_MAP_SWIZZLE_128B)) return false;
     const PtPlan pl(a.n_map, a.dim_p, a.vdim_p);
-    launch_pdl(a.n_map == 2 ? attention_prompt_kernel<2> : attention_prompt_kernel<1>, std::min(tiles * a.n_kv, (uint32_t)sm_count), PT_THREADS, pl.bytes, st, tm, a, tiles);
+    launch_pdl(a.n_map == 2 ? attention_prompt_kernel<2, false> : a.softcap > 0.0f ? attention_prompt_kernel<1, true> : attention_prompt_kernel<1, false>, std::min(tiles * a.n_kv, (uint32_t)sm_count), PT_THREADS, pl.bytes, st, tm, a, tiles);
     g_tc5_launched.store(true, std::memory_order_relaxed);
     return true;
 }

@@ -9,9 +9,14 @@
 //           retention: rotate, recurrence, norm with gate
 //   out     x += [W_o | W_down] [mixer | ff]
 //   side    gate (gelu, token entry), proj, then norm + residual + the next layer's norm in one kernel
-// A sequential block reads the residual itself (h: its activation form) and norms what it adds:
-//   in      mixer projections <- h; mixer (attention: prep, attention with the heads' epilogue); out product, bias as epilogue
-//   post    x += mult norm(out), h = x in one kernel
+// A sequential block reads the residual itself (h: its activation form) or its norm, and norms what it adds:
+//   in      mixer projections <- h
+//   mixer   attention: prep, attention with the heads' epilogue
+//           state space: convolution and steps, recurrence, gate and norm
+//           time mixing: token shift, projections of the mixes, recurrence, norm and gate
+//           a second mixer leaves its output beside the first one's, so that one product adds up both
+//   out     product, bias as epilogue
+//   post    x += mult norm(out), h = x or norm(x) in one kernel
 //   ff      dense: up (activation as epilogue), down; experts: routing, grouped gate/up and down (moe.cu); post as above
 #include <math.h>
 #include <string.h>
@@ -27,38 +32,62 @@ namespace {
 constexpr uint32_t MOE_ROWS_IN_ORDER = 8;  // so many (token, expert) pairs run row by row, more are grouped by expert
 
 constexpr uint32_t round_up(uint32_t v, uint32_t m) { return (v + m - 1) / m * m; }
+constexpr bool recurrent_kind(uint32_t kind) { return kind == OB_MIXER_RETENTION || kind == OB_MIXER_STATE_SPACE || kind == OB_MIXER_TIME_MIXING; }
 
 struct Dense {  // rows x kp bfloat16 on the device
     __nv_bfloat16 *w = nullptr;
     uint32_t rows = 0, kp = 0;
 };
 
-struct LayerPlan {
+struct MixerPlan {
     ob_mixer_desc mx{};  // sizes and constants only
-    float norm_gain = 0.0f, glu_limit = 0.0f, glu_alpha = 0.0f;
-    uint32_t n_ff = 0;
-    Dense in, out, side_gate, side_proj;
-    bool sequential = false;
-    float *in_bias = nullptr, *out_bias = nullptr, *post1 = nullptr, *post2 = nullptr;
-    uint32_t ff_kind = 0, n_expert = 0, top = 1;
-    Dense up, down, router;  // feed-forward of a sequential block, one after the other for every expert (gate and up rows interleaved)
-    // attention: rows of `in` are [activations (values, gates) | f32 projections (queries, keys)]
-    float *q_norm = nullptr, *k_norm = nullptr;
-    uint32_t vdim_p = 0, row = 0, gate0 = 0;  // row: elements of a cache row per key/value head
-    bool has_v = false, has_gate = false;
-    float *side_norm = nullptr;
+    float scale = 1.0f;  // of its output
+    Dense in;            // projections of the block's input
+    float *in_bias = nullptr;
     Rot rot{};
-    // rows of `in`: [activations (unrotated queries) | f32 projections | gate/up]
-    uint32_t act_rows = 0, f32_row0 = 0, f32_rows = 0, glu_row0 = 0, mix_cols = 0;  // mix_cols: columns of the mixer in the out product's input
+    // rows of `in`: [activations (unrotated queries; values, gates; the state space's gate) | f32 projections]
+    uint32_t act_rows = 0, f32_row0 = 0, f32_rows = 0;
+    uint32_t cols = 0, col0 = 0;  // columns of its output in the out product's input, and the first of them
+    uint32_t out_width = 0;       // of its output
+    // attention
+    float *q_norm = nullptr, *k_norm = nullptr, *sink = nullptr;
+    uint32_t vdim_p = 0, row = 0, gate0 = 0;  // row: elements of a cache row per key/value head
+    bool has_v = false, has_gate = false, head_gate = false, own_kv = true;
     // latent attention
     Dense uk, uv;        // per head [kv_rank <- dim], [vdim <- kv_rank]
     Dense expand;        // latent -> keys [H][dim_k], then (from row ex_v0) values [H][vdim_k]; no rows: prompts attend in the latent space too
     uint32_t dim_p = 0, kv_p = 0, dq = 0, kv_w = 0, dim_k = 0, vdim_k = 0, ex_v0 = 0;
     float *kv_norm = nullptr;
     void *pool = nullptr;
+    // recurrent layers: the state, and the last inputs of the convolution or of the token shift
+    float *state = nullptr, *tail = nullptr;
+    uint32_t tail_elems = 0;  // per slot
     // retention
-    float *decay = nullptr, *state = nullptr;
+    float *decay = nullptr;
     float decay_min = 0.0f;
+    // state space
+    float *conv_w = nullptr, *conv_b = nullptr, *dt_bias = nullptr, *a_log = nullptr, *skip = nullptr, *out_norm = nullptr;
+    // time mixing: r, k, v and gate one after the other, equally many rows each
+    Dense rkvg, decay1, decay2;
+    float *mu[SHIFT_MIXES] = {}, *decay0 = nullptr, *bonus = nullptr;
+
+    uint32_t channels() const { return mx.n_head * mx.vdim + 2 * mx.n_group * mx.dim; }  // of the convolution
+};
+
+struct LayerPlan : MixerPlan {
+    std::unique_ptr<MixerPlan> second;
+    float norm_gain = 0.0f, glu_limit = 0.0f, glu_alpha = 0.0f;
+    uint32_t n_ff = 0, glu_row0 = 0;  // parallel blocks: gate/up rows of `in`, after the mixer's
+    Dense out, side_gate, side_proj;
+    bool sequential = false;
+    float *out_bias = nullptr, *pre1 = nullptr, *pre2 = nullptr, *post1 = nullptr, *post2 = nullptr;
+    uint32_t ff_kind = 0, n_expert = 0, top = 1;
+    uint32_t n_shared = 0;  // pieces of the shared expert, each of an expert's size
+    Dense up, down, router;  // feed-forward of a sequential block, one after the other for every expert (gate and up rows interleaved)
+    bool router_softmax = false;
+    float *side_norm = nullptr;
+
+    uint32_t pairs() const { return top + n_shared; }  // experts of a token
 };
 
 // A zero-padded bfloat16 matrix put together on the host from parts of others.
@@ -66,8 +95,9 @@ struct HostDense {
     uint32_t rows, kp;
     std::vector<uint16_t> v;
     HostDense(uint32_t r, uint32_t k) : rows(r), kp(k), v((size_t)r * k, 0) {}
-    void copy(uint32_t row, uint32_t col, const ob_matrix_desc &src, uint32_t src_row) {
-        memcpy(v.data() + (size_t)row * kp + col, src.data + (size_t)src_row * src.in_dim * 2, (size_t)src.in_dim * 2);
+    void copy(uint32_t row, uint32_t col, const ob_matrix_desc &src, uint32_t src_row) { copy(row, col, src, src_row, 0, src.in_dim); }
+    void copy(uint32_t row, uint32_t col, const ob_matrix_desc &src, uint32_t src_row, uint32_t src_col, uint32_t n) {
+        memcpy(v.data() + (size_t)row * kp + col, src.data + ((size_t)src_row * src.in_dim + src_col) * 2, (size_t)n * 2);
     }
 };
 
@@ -80,6 +110,11 @@ struct LayeredGraph : StepGraph {
     std::vector<LayerPlan> L;
     __nv_bfloat16 *embd = nullptr, *side_embd = nullptr;
     Dense output;
+    void *mix = nullptr;                    // time mixing: the mixes of every row, and the low-rank half of the decay
+    void *low = nullptr;
+    float *conv = nullptr, *decays = nullptr;
+    float2 *steps = nullptr;
+    uint32_t low_p = 0;
     void *h = nullptr, *xb = nullptr, *qn = nullptr, *q = nullptr, *o_lat = nullptr, *cat = nullptr, *sg = nullptr;
     float *y = nullptr, *o_ret = nullptr, *sy = nullptr, *part = nullptr;
     void *lat = nullptr, *expanded = nullptr;  // gathered latents of prompts, their keys and values: key_cap rows
@@ -93,6 +128,7 @@ struct LayeredGraph : StepGraph {
     bool failed = false;  // a product could not be launched
 
     size_t es() const { return f32 ? 4 : 2; }
+    void *column(uint32_t c) const { return static_cast<uint8_t *>(cat) + c * es(); }  // of the out product's input
     bool recurrent() const override { return has_state; }
     bool take_failure() override {
         const bool f = failed;
@@ -123,17 +159,28 @@ struct LayeredGraph : StepGraph {
 
     void layers(uint32_t T, uint32_t n_seq, const RowSpan *spans, uint32_t max_pos, cudaStream_t st) override;
     void head(const uint32_t *d_rows, uint32_t n, cudaStream_t st) override;
-    void latent(const LayerPlan &P, uint32_t T, uint32_t n_seq, const RowSpan *spans, bool single, uint32_t max_pos, cudaStream_t st);
-    void retention(const LayerPlan &P, uint32_t T, uint32_t n_seq, const RowSpan *spans, cudaStream_t st);
-    void attention(const LayerPlan &P, uint32_t T, uint32_t n_seq, const RowSpan *spans, bool single, uint32_t max_pos, cudaStream_t st);
-    void mixer(const LayerPlan &P, uint32_t T, uint32_t n_seq, const RowSpan *spans, bool single, uint32_t max_pos, cudaStream_t st);
-    void sequential(const LayerPlan &P, bool last, uint32_t T, uint32_t n_seq, const RowSpan *spans, bool single, uint32_t max_pos, cudaStream_t st);
-    void post(const float *w, uint32_t T, bool last, uint32_t top, const uint32_t *rows, uint32_t n_zero, cudaStream_t st);
-    uint32_t cache_elems(const LayerPlan &P) const { return P.mx.kind == OB_MIXER_ATTENTION ? P.mx.n_kv_head * P.row : P.dq; }  // per position
+    void latent(const MixerPlan &P, uint32_t T, uint32_t n_seq, const RowSpan *spans, bool single, uint32_t max_pos, cudaStream_t st);
+    void retention(const MixerPlan &P, uint32_t T, uint32_t n_seq, const RowSpan *spans, cudaStream_t st);
+    void state_space(const MixerPlan &P, uint32_t T, uint32_t n_seq, const RowSpan *spans, bool single, cudaStream_t st);
+    void time_mixing(const MixerPlan &P, const float *norm, uint32_t T, uint32_t n_seq, const RowSpan *spans, bool single, cudaStream_t st);
+    void recurrence(const MixerPlan &P, RecurrenceArgs a, uint32_t n_seq, const RowSpan *spans, cudaStream_t st);
+    void attention(const MixerPlan &P, uint32_t T, uint32_t n_seq, const RowSpan *spans, bool single, uint32_t max_pos, cudaStream_t st);
+    void project(const MixerPlan &P, uint32_t T, cudaStream_t st);
+    void mixer(const MixerPlan &P, const float *norm, uint32_t T, uint32_t n_seq, const RowSpan *spans, bool single, uint32_t max_pos, cudaStream_t st);
+    void sequential(const LayerPlan &P, const LayerPlan *next, uint32_t T, uint32_t n_seq, const RowSpan *spans, bool single, uint32_t max_pos, cudaStream_t st);
+    void post(const float *w, uint32_t T, bool last, const float *next, uint32_t top, const uint32_t *rows, uint32_t n_zero, cudaStream_t st);
+    uint32_t cache_elems(const MixerPlan &P) const { return P.mx.kind == OB_MIXER_ATTENTION ? P.mx.n_kv_head * P.row : P.dq; }  // per position
     int copy_prefix(ob_kv *dst, const ob_kv *src, uint32_t n) override;
     int read_pages(const ob_kv *kv, uint32_t layer, uint32_t pos0, uint32_t n, float *k_out, float *v_out) override;
     int read_state(const ob_kv *kv, uint32_t layer, float *out) override;
-    size_t state_elems(const LayerPlan &P) const { return (size_t)P.mx.n_head * P.mx.dim * P.mx.vdim; }
+    size_t state_elems(const MixerPlan &P) const { return (size_t)P.mx.n_head * P.mx.dim * P.mx.vdim; }
+    // The mixers of all layers.
+    template <typename F> void each_mixer(F f) {
+        for (LayerPlan &P : L) {
+            f(static_cast<MixerPlan &>(P));
+            if (P.second) f(*P.second);
+        }
+    }
 
     int upload(const HostDense &src, Dense *out) {
         int rc = dev_alloc(m, &out->w, src.v.size());
@@ -159,11 +206,17 @@ struct LayeredGraph : StepGraph {
     }
     int build(const ob_layered_desc &c);
     int build_layer(const ob_block_desc &b, LayerPlan &P);
+    void size_mixer(const ob_mixer_desc &x, MixerPlan &P) const;
+    int fill_in(const ob_mixer_desc &x, MixerPlan &P, HostDense &in);
+    int build_mixer(const ob_mixer_desc &x, MixerPlan &P);
     int build_ff(const ob_block_desc &b, LayerPlan &P);
-    int upload_now(const float *src, size_t n, float **out) {  // the source may end with the caller
+    int rotation(MixerPlan &P, std::map<std::pair<std::vector<double>, float>, float2 *> &tables);
+    int upload_now(const float *src, size_t n, float **out, float gain = 1.0f) {  // the source may end with the caller
+        std::vector<float> scaled(src, src + n);
+        for (float &v : scaled) v *= gain;
         int rc = dev_alloc(m, out, n);
         if (rc) return rc;
-        OB_CUDA(m->ctx, cudaMemcpy(*out, src, n * 4, cudaMemcpyHostToDevice));
+        OB_CUDA(m->ctx, cudaMemcpy(*out, scaled.data(), n * 4, cudaMemcpyHostToDevice));
         return OB_OK;
     }
 };
@@ -174,7 +227,7 @@ uint32_t first_long(const RowSpan *spans, uint32_t n_seq) {
     return n_seq;
 }
 
-void LayeredGraph::latent(const LayerPlan &P, uint32_t T, uint32_t n_seq, const RowSpan *spans, bool single, uint32_t max_pos, cudaStream_t st) {
+void LayeredGraph::latent(const MixerPlan &P, uint32_t T, uint32_t n_seq, const RowSpan *spans, bool single, uint32_t max_pos, cudaStream_t st) {
     const MetaLayout ml(m->T);
     const uint32_t H = P.mx.n_head;
     LatentArgs a{};
@@ -268,7 +321,7 @@ void LayeredGraph::latent(const LayerPlan &P, uint32_t T, uint32_t n_seq, const 
     }
 }
 
-void LayeredGraph::retention(const LayerPlan &P, uint32_t T, uint32_t n_seq, const RowSpan *spans, cudaStream_t st) {
+void LayeredGraph::retention(const MixerPlan &P, uint32_t T, uint32_t n_seq, const RowSpan *spans, cudaStream_t st) {
     const MetaLayout ml(m->T);
     RetentionArgs a{};
     a.y = y;
@@ -294,7 +347,7 @@ void LayeredGraph::retention(const LayerPlan &P, uint32_t T, uint32_t n_seq, con
     m->ctx->launches += launch_retention(a, f32, m->ctx->sm_count, st);
 }
 
-void LayeredGraph::attention(const LayerPlan &P, uint32_t T, uint32_t n_seq, const RowSpan *spans, bool single, uint32_t max_pos, cudaStream_t st) {
+void LayeredGraph::attention(const MixerPlan &P, uint32_t T, uint32_t n_seq, const RowSpan *spans, bool single, uint32_t max_pos, cudaStream_t st) {
     const MetaLayout ml(m->T);
     AttentionArgs a{};
     a.y = y;
@@ -316,14 +369,20 @@ void LayeredGraph::attention(const LayerPlan &P, uint32_t T, uint32_t n_seq, con
     a.eps = eps;
     a.scale = P.mx.scale;
     a.map_weight = P.mx.map_weight;
-    a.head_gain = P.mx.head_gain;
+    a.head_gain = P.mx.n_map == 2 ? P.mx.head_gain : P.scale;
+    a.norm_whole = P.mx.qk_norm_whole != 0;
+    a.own_kv = P.own_kv;
+    a.keep = P.mx.window ? P.mx.keep_first : 0;
+    a.softcap = P.mx.softcap;
+    a.sink = P.sink;
+    a.head_gate = P.head_gate ? y + P.f32_rows - P.mx.n_head : nullptr;
     a.q_norm = P.q_norm;
     a.k_norm = P.k_norm;
     a.rot = P.rot;
     a.q = q;
     a.cache = P.pool;
     a.n_pages = m->pool_pages;
-    a.out = cat;
+    a.out = column(P.col0);
     a.out_pitch = cat_pitch;
     a.T = T;
     a.n_seq = n_seq;
@@ -340,13 +399,155 @@ void LayeredGraph::attention(const LayerPlan &P, uint32_t T, uint32_t n_seq, con
     m->ctx->launches += 1 + n;
 }
 
-void LayeredGraph::mixer(const LayerPlan &P, uint32_t T, uint32_t n_seq, const RowSpan *spans, bool single, uint32_t max_pos, cudaStream_t st) {
-    if (P.mx.kind == OB_MIXER_LATENT_ATTENTION) latent(P, T, n_seq, spans, single, max_pos, st);
-    else if (P.mx.kind == OB_MIXER_ATTENTION) attention(P, T, n_seq, spans, single, max_pos, st);
-    else retention(P, T, n_seq, spans, st);
+void LayeredGraph::recurrence(const MixerPlan &P, RecurrenceArgs a, uint32_t n_seq, const RowSpan *spans, cudaStream_t st) {
+    const MetaLayout ml(m->T);
+    a.n_head = P.mx.n_head;
+    a.dim = P.mx.dim;
+    a.vdim = P.mx.vdim;
+    a.state = P.state;
+    a.o = o_ret;
+    a.n_seq = n_seq;
+    a.first_long = first_long(spans, n_seq);
+    a.spans = reinterpret_cast<const RowSpan *>(m->d_meta + ml.off_spans);
+    a.positions = reinterpret_cast<const uint32_t *>(m->d_meta + ml.off_positions);
+    a.slots = reinterpret_cast<const int32_t *>(m->d_meta + ml.off_slots);
+    m->ctx->launches += launch_recurrence(a, m->ctx->sm_count, st);
 }
 
-void LayeredGraph::post(const float *w, uint32_t T, bool last, uint32_t top, const uint32_t *rows, uint32_t n_zero, cudaStream_t st) {
+// Rows of `in`: gate as activations; channels of the convolution and raw steps in y.
+void LayeredGraph::state_space(const MixerPlan &P, uint32_t T, uint32_t n_seq, const RowSpan *spans, bool single, cudaStream_t st) {
+    const MetaLayout ml(m->T);
+    const uint32_t inner = P.mx.n_head * P.mx.vdim, n = P.channels();
+    ConvArgs c{};
+    c.y = y;
+    c.y_pitch = y_pitch;
+    c.n_channel = n;
+    c.taps = P.mx.conv_taps;
+    c.n_head = P.mx.n_head;
+    c.w = P.conv_w;
+    c.b = P.conv_b;
+    c.state = P.tail;
+    c.u = conv;
+    c.dt_bias = P.dt_bias;
+    c.a_log = P.a_log;
+    c.step = steps;
+    c.T = T;
+    c.n_seq = n_seq;
+    c.spans = reinterpret_cast<const RowSpan *>(m->d_meta + ml.off_spans);
+    c.h_spans = spans;
+    c.single = single;
+    c.positions = reinterpret_cast<const uint32_t *>(m->d_meta + ml.off_positions);
+    c.slots = reinterpret_cast<const int32_t *>(m->d_meta + ml.off_slots);
+    launch_conv(c, st);
+    RecurrenceArgs r{};
+    r.v = conv;
+    r.k = conv + inner;
+    r.q = conv + inner + (size_t)P.mx.n_group * P.mx.dim;
+    r.pitch = n;
+    r.share = P.mx.n_head / P.mx.n_group;
+    r.step = steps;
+    recurrence(P, r, n_seq, spans, st);
+    StateSpaceOutArgs o{};
+    o.o = o_ret;
+    o.x = conv;
+    o.x_pitch = n;
+    o.z = qn;
+    o.z_pitch = P.act_rows;
+    o.inner = inner;
+    o.vdim = P.mx.vdim;
+    o.n_part = P.mx.n_norm_group;
+    o.T = T;
+    o.skip = P.skip;
+    o.norm = P.out_norm;
+    o.eps = eps;
+    o.out = column(P.col0);
+    o.out_pitch = cat_pitch;
+    launch_state_space_out(o, f32, st);
+    m->ctx->launches += 2;
+}
+
+void LayeredGraph::time_mixing(const MixerPlan &P, const float *norm, uint32_t T, uint32_t n_seq, const RowSpan *spans, bool single, cudaStream_t st) {
+    const MetaLayout ml(m->T);
+    const uint32_t n = P.mx.n_head * P.mx.dim;
+    ShiftMixArgs s{};
+    s.x = m->x;
+    s.norm = norm;
+    for (uint32_t i = 0; i < SHIFT_MIXES; ++i) s.mu[i] = P.mu[i];
+    s.state = P.tail;
+    s.mix = mix;
+    s.width = width;
+    s.pitch = h_pitch;
+    s.T = T;
+    s.n_seq = n_seq;
+    s.eps = eps;
+    s.spans = reinterpret_cast<const RowSpan *>(m->d_meta + ml.off_spans);
+    s.single = single;
+    s.positions = reinterpret_cast<const uint32_t *>(m->d_meta + ml.off_positions);
+    s.slots = reinterpret_cast<const int32_t *>(m->d_meta + ml.off_slots);
+    launch_shift_mix(s, f32, st);
+    LinArgs p = product(P.rkvg, mix, SHIFT_MIXES * h_pitch, T);  // mixes of r, k, v, gate with a matrix each
+    p.n_rows = P.rkvg.rows / 4;
+    p.n_batch = 4;
+    p.x_step = h_pitch;
+    segment(p, 0, n, LE_F32, y, y_pitch, 0, n);
+    linear(p, st);
+    LinArgs d1 = product(P.decay1, static_cast<uint8_t *>(mix) + 4 * h_pitch * es(), SHIFT_MIXES * h_pitch, T);
+    segment(d1, 0, P.mx.w_decay1.out_dim, LE_TANH, low, P.decay2.kp);
+    linear(d1, st);
+    LinArgs d2 = product(P.decay2, low, P.decay2.kp, T);
+    d2.bias = P.decay0;
+    segment(d2, 0, n, LE_DECAY, decays, n);
+    linear(d2, st);
+    RecurrenceArgs r{};
+    r.q = y;
+    r.k = y + n;
+    r.v = y + 2 * n;
+    r.pitch = y_pitch;
+    r.share = 1;
+    r.w = decays;
+    r.w_pitch = n;
+    recurrence(P, r, n_seq, spans, st);
+    TimeMixOutArgs o{};
+    o.o = o_ret;
+    o.r = y;
+    o.k = y + n;
+    o.v = y + 2 * n;
+    o.gate = y + 3 * n;
+    o.pitch = y_pitch;
+    o.n_head = P.mx.n_head;
+    o.dim = P.mx.dim;
+    o.T = T;
+    o.bonus = P.bonus;
+    o.norm = P.out_norm;
+    o.eps = eps;
+    o.out = column(P.col0);
+    o.out_pitch = cat_pitch;
+    launch_time_mix_out(o, f32, st);
+    m->ctx->launches += 2;
+}
+
+// The projections of a sequential block's input.
+void LayeredGraph::project(const MixerPlan &P, uint32_t T, cudaStream_t st) {
+    if (!P.in.rows) return;
+    LinArgs in = product(P.in, h, h_pitch, T);
+    in.bias = P.in_bias;
+    segment(in, 0, P.act_rows, LE_ACT, qn, P.act_rows);
+    segment(in, P.f32_row0, P.f32_rows, LE_F32, y, y_pitch);
+    linear(in, st);
+}
+
+// norm: of the block's input h, which a time-mixing layer makes itself.
+void LayeredGraph::mixer(const MixerPlan &P, const float *norm, uint32_t T, uint32_t n_seq, const RowSpan *spans, bool single, uint32_t max_pos, cudaStream_t st) {
+    switch (P.mx.kind) {
+    case OB_MIXER_LATENT_ATTENTION: return latent(P, T, n_seq, spans, single, max_pos, st);
+    case OB_MIXER_ATTENTION: return attention(P, T, n_seq, spans, single, max_pos, st);
+    case OB_MIXER_STATE_SPACE: return state_space(P, T, n_seq, spans, single, st);
+    case OB_MIXER_TIME_MIXING: return time_mixing(P, norm, T, n_seq, spans, single, st);
+    default: return retention(P, T, n_seq, spans, st);
+    }
+}
+
+void LayeredGraph::post(const float *w, uint32_t T, bool last, const float *next, uint32_t top, const uint32_t *rows, uint32_t n_zero, cudaStream_t st) {
     PostNormArgs p{};
     p.x = m->x;
     p.y = yo;
@@ -359,58 +560,64 @@ void LayeredGraph::post(const float *w, uint32_t T, bool last, uint32_t top, con
     p.mult = residual_mult;
     p.h = last ? nullptr : h;
     p.h_pitch = h_pitch;
+    p.next_w = next;
     p.zero = n_zero ? moe.count : nullptr;
     p.n_zero = n_zero;
     launch_post_norm(p, f32, st);
     m->ctx->launches++;
 }
 
-void LayeredGraph::sequential(const LayerPlan &P, bool last, uint32_t T, uint32_t n_seq, const RowSpan *spans, bool single, uint32_t max_pos, cudaStream_t st) {
-    LinArgs in = product(P.in, h, h_pitch, T);
-    in.bias = P.in_bias;
-    segment(in, 0, P.act_rows, LE_ACT, qn, P.act_rows);
-    segment(in, P.f32_row0, P.f32_rows, LE_F32, y, y_pitch);
-    linear(in, st);
-    mixer(P, T, n_seq, spans, single, max_pos, st);
+// next: the block that follows, null after the last one.
+void LayeredGraph::sequential(const LayerPlan &P, const LayerPlan *next, uint32_t T, uint32_t n_seq, const RowSpan *spans, bool single, uint32_t max_pos, cudaStream_t st) {
+    const float *next_pre = next ? next->pre1 : nullptr;
+    project(P, T, st);
+    mixer(P, P.pre1, T, n_seq, spans, single, max_pos, st);
+    if (P.second) {
+        project(*P.second, T, st);
+        mixer(*P.second, P.pre1, T, n_seq, spans, single, max_pos, st);
+    }
     LinArgs out = product(P.out, cat, cat_pitch, T);
     out.bias = P.out_bias;
     segment(out, 0, width, LE_F32, yo, width);
     linear(out, st);
-    post(P.post1, T, last && !P.n_ff, 1, nullptr, 0, st);
+    post(P.post1, T, !next && !P.n_ff, P.n_ff ? P.pre2 : next_pre, 1, nullptr, 0, st);
     if (!P.n_ff) return;
     if (P.ff_kind != OB_FF_EXPERTS) {
         LinArgs up = product(P.up, h, h_pitch, T);
-        segment(up, 0, P.n_ff, LE_RELU2, ffa, P.down.kp);
+        if (P.ff_kind == OB_FF_GELU_GLU) segment(up, 0, 2 * P.n_ff, LE_GELU_GLU, ffa, P.down.kp);
+        else segment(up, 0, P.n_ff, LE_RELU2, ffa, P.down.kp);
         linear(up, st);
         LinArgs down = product(P.down, ffa, P.down.kp, T);
         segment(down, 0, width, LE_F32, yo, width);
         linear(down, st);
-        post(P.post2, T, last, 1, nullptr, 0, st);
+        post(P.post2, T, !next, next_pre, 1, nullptr, 0, st);
         return;
     }
-    const uint32_t R = T * P.top;
-    const bool in_order = R <= MOE_ROWS_IN_ORDER;
+    const uint32_t R = T * P.pairs(), E = P.n_expert + P.n_shared, n_logit = P.n_expert + (P.n_shared > 0);
+    const bool in_order = T == 1 || R <= MOE_ROWS_IN_ORDER;
     MoeArgs r = moe;
     r.x = h;
     r.x_pitch = h_pitch;
     r.w = P.router.w;
     r.n_expert = P.n_expert;
     r.top = P.top;
+    r.n_shared = P.n_shared;
+    r.softmax = P.router_softmax;
     r.T = T;
-    r.tile_rows = linear_tile_rows(R, P.n_expert, f32);
+    r.tile_rows = linear_tile_rows(R, E, f32);
     if (in_order) r.count = nullptr;
     if (T > MOE_DOT_TOKENS) {
         LinArgs z = product(P.router, h, h_pitch, T);
-        segment(z, 0, P.n_expert, LE_F32, router_logits, P.n_expert);
+        segment(z, 0, n_logit, LE_F32, router_logits, n_logit);
         linear(z, st);
         r.logits = router_logits;
-        r.logit_pitch = P.n_expert;
+        r.logit_pitch = n_logit;
     }
     m->ctx->launches += launch_moe_route(r, f32, st);
     auto grouped = [&](const Dense &w, const void *x, uint32_t x_div) {
         LinArgs a = product(w, x, w.kp, R);
-        a.n_rows = w.rows / P.n_expert;
-        a.n_batch = P.n_expert;
+        a.n_rows = w.rows / E;
+        a.n_batch = E;
         if (in_order) {
             a.row_batch = r.expert;
             a.x_div = x_div;
@@ -418,43 +625,43 @@ void LayeredGraph::sequential(const LayerPlan &P, bool last, uint32_t T, uint32_
             a.tiles = r.tiles;
             a.n_tiles = r.n_tiles;
             a.tile_rows = r.tile_rows;
-            a.max_tiles = R / r.tile_rows + std::min(R, P.n_expert);
+            a.max_tiles = R / r.tile_rows + std::min(R, E);
         }
         return a;
     };
-    LinArgs up = grouped(P.up, in_order ? h : r.gathered, P.top);
-    up.row_scale = in_order ? r.score : r.row_score;
+    LinArgs up = grouped(P.up, in_order ? h : r.gathered, P.pairs());
+    (P.router_softmax ? up.out_scale : up.row_scale) = in_order ? r.score : r.row_score;
     segment(up, 0, 2 * P.n_ff, LE_SWIGLU, ffa, P.down.kp);
     linear(up, st);
     LinArgs down = grouped(P.down, ffa, 1);
     segment(down, 0, width, LE_F32, yo, width);
     linear(down, st);
-    post(P.post2, T, last, P.top, in_order ? nullptr : r.row, in_order ? 0 : P.n_expert, st);
+    post(P.post2, T, !next, next_pre, P.pairs(), in_order ? nullptr : r.row, in_order ? 0 : E, st);
 }
 
 void LayeredGraph::layers(uint32_t T, uint32_t n_seq, const RowSpan *spans, uint32_t max_pos, cudaStream_t st) {
     const MetaLayout ml(m->T);
     const uint32_t *tokens = reinterpret_cast<const uint32_t *>(m->d_meta + ml.off_tokens);
     const bool single = n_seq == T;
-    launch_embed(embd, width, tokens, T, m->x, !L[0].sequential, eps, L[0].norm_gain, h, h_pitch, f32, st);
+    launch_embed(embd, width, tokens, T, m->x, !L[0].sequential || L[0].pre1, eps, L[0].sequential ? 1.0f : L[0].norm_gain, L[0].pre1, h, h_pitch, f32, st);
     m->ctx->launches++;
     for (size_t li = 0; li < L.size(); ++li) {
         const LayerPlan &P = L[li];
         const bool last = li + 1 == L.size();
         if (P.sequential) {
-            sequential(P, last, T, n_seq, spans, single, max_pos, st);
+            sequential(P, last ? nullptr : &L[li + 1], T, n_seq, spans, single, max_pos, st);
             continue;
         }
         LinArgs in = product(P.in, h, h_pitch, T);
         segment(in, 0, P.act_rows, LE_ACT, qn, P.act_rows);
         segment(in, P.f32_row0, P.f32_rows, LE_F32, y, y_pitch);
         in.bias = P.in_bias;
-        segment(in, P.glu_row0, 2 * P.n_ff, LE_GLU, cat, cat_pitch, P.mix_cols);
+        segment(in, P.glu_row0, 2 * P.n_ff, LE_GLU, cat, cat_pitch, P.cols);
         in.glu_limit = P.glu_limit;
         in.glu_alpha = P.glu_alpha;
         linear(in, st);
 
-        mixer(P, T, n_seq, spans, single, max_pos, st);
+        mixer(P, nullptr, T, n_seq, spans, single, max_pos, st);
 
         LinArgs out = product(P.out, cat, cat_pitch, T);
         segment(out, 0, width, LE_RESIDUAL, m->x, width);
@@ -496,20 +703,25 @@ void LayeredGraph::head(const uint32_t *d_rows, uint32_t n, cudaStream_t st) {
 
 int LayeredGraph::copy_prefix(ob_kv *dst, const ob_kv *src, uint32_t n) {
     cudaStream_t st = m->ctx->stream;
-    for (const LayerPlan &P : L) {
-        if (P.pool) {
+    int rc = OB_OK;
+    each_mixer([&](MixerPlan &P) {
+        if (P.pool && P.own_kv) {
             launch_copy_pages(P.pool, (uint64_t)KV_PAGE * cache_elems(P) * es(), src->d_table, dst->d_table, (n + KV_PAGE - 1) / KV_PAGE, st);
             m->ctx->launches++;
-        } else if (P.state && src->slot >= 0 && dst->slot >= 0) {
-            const size_t e = state_elems(P);
-            OB_CUDA(m->ctx, cudaMemcpyAsync(P.state + (size_t)dst->slot * e, P.state + (size_t)src->slot * e, e * 4, cudaMemcpyDeviceToDevice, st));
+        } else if (P.state && src->slot >= 0 && dst->slot >= 0 && !rc) {
+            auto copy = [&](float *p, size_t e) -> int {
+                if (e) OB_CUDA(m->ctx, cudaMemcpyAsync(p + (size_t)dst->slot * e, p + (size_t)src->slot * e, e * 4, cudaMemcpyDeviceToDevice, st));
+                return OB_OK;
+            };
+            rc = copy(P.state, state_elems(P));
+            if (!rc) rc = copy(P.tail, P.tail_elems);
         }
-    }
-    return OB_OK;
+    });
+    return rc;
 }
 
 int LayeredGraph::read_pages(const ob_kv *kv, uint32_t layer, uint32_t pos0, uint32_t n, float *k_out, float *v_out) {
-    const LayerPlan &P = L[layer];
+    const MixerPlan &P = L[layer].pool || !L[layer].second ? L[layer] : *L[layer].second;
     if (!P.pool) return fail(m->ctx, OB_ERR_INVALID, "kv_read: the layer caches no positions");
     const bool latent = P.mx.kind == OB_MIXER_LATENT_ATTENTION;
     std::vector<uint8_t> row((latent ? P.dq : P.row) * es());
@@ -543,92 +755,133 @@ int LayeredGraph::read_pages(const ob_kv *kv, uint32_t layer, uint32_t pos0, uin
 }
 
 int LayeredGraph::read_state(const ob_kv *kv, uint32_t layer, float *out) {
-    if (layer >= L.size() || !L[layer].state) return fail(m->ctx, OB_ERR_INVALID, "state_read: the layer has no recurrent state");
-    const size_t e = state_elems(L[layer]);
-    OB_CUDA(m->ctx, cudaMemcpy(out, L[layer].state + (size_t)kv->slot * e, e * 4, cudaMemcpyDeviceToHost));
+    const MixerPlan *P = layer < L.size() ? &L[layer] : nullptr;
+    if (P && !P->state) P = L[layer].second.get();
+    if (!P || !P->state) return fail(m->ctx, OB_ERR_INVALID, "state_read: the layer has no recurrent state");
+    const size_t e = state_elems(*P);
+    OB_CUDA(m->ctx, cudaMemcpy(out, P->state + (size_t)kv->slot * e, e * 4, cudaMemcpyDeviceToHost));
     return OB_OK;
 }
 
-int LayeredGraph::build_layer(const ob_block_desc &b, LayerPlan &P) {
-    const ob_mixer_desc &x = b.mixer;
-    const bool latent = x.kind == OB_MIXER_LATENT_ATTENTION, attends = x.kind == OB_MIXER_ATTENTION;
+// Sizes of a mixer's parts; nothing is allocated.
+void LayeredGraph::size_mixer(const ob_mixer_desc &x, MixerPlan &P) const {
     const uint32_t H = x.n_head, G = x.n_kv_head;
-    int rc;
     P.mx = x;
-    P.sequential = b.post_norm1 != nullptr;
-    P.ff_kind = b.ff_kind;
-    P.n_expert = b.n_expert;
-    P.top = b.ff_kind == OB_FF_EXPERTS ? b.n_expert_used : 1;
-    const uint32_t glu = P.sequential ? 0 : b.n_ff;  // feed-forward inside the mixer's products
-    P.norm_gain = b.norm_gain;
-    P.n_ff = b.n_ff;
-    P.glu_limit = b.glu_limit;
-    P.glu_alpha = b.glu_alpha;
-    // ---- everything that reads the normed input
-    if (latent) {
+    switch (x.kind) {
+    case OB_MIXER_LATENT_ATTENTION:
         P.dim_p = round_up(x.dim, LIN_K_ALIGN);
         P.kv_p = round_up(x.kv_rank, 16);
         P.dq = P.kv_p + round_up(x.rot_dim, 16);
         P.kv_w = round_up(x.kv_rank, LIN_K_ALIGN);
         P.act_rows = H * P.dim_p;
         P.f32_rows = H * x.rot_dim + x.kv_rank + x.rot_dim + H;
-    } else if (attends) {
+        break;
+    case OB_MIXER_ATTENTION:
+        P.own_kv = !x.kv_layer;
         P.has_v = x.wv.data != nullptr;
-        P.has_gate = x.w_gate.data != nullptr;
+        P.head_gate = x.w_gate.data && x.w_gate.out_dim == H && x.vdim != 1;
+        P.has_gate = x.w_gate.data && !P.head_gate;
         P.dim_p = round_up(x.dim, 16);
         P.vdim_p = round_up(x.vdim, 16);
         P.row = attention_cache_row(x.n_map, P.dim_p, P.vdim_p);
         P.gate0 = P.has_v ? G * x.vdim : 0;
         P.act_rows = round_up(P.gate0 + (P.has_gate ? H * x.vdim : 0), LIN_ROW_ALIGN);
-        P.f32_rows = (H + G) * x.n_map * x.dim;
-    } else {
-        P.f32_rows = H * (2 * x.dim + 2 * x.vdim);
+        P.f32_rows = (H + (P.own_kv ? G : 0)) * x.n_map * x.dim + (P.head_gate ? H : 0);
+        break;
+    case OB_MIXER_STATE_SPACE:
+        P.act_rows = round_up(H * x.vdim, LIN_ROW_ALIGN);
+        P.f32_rows = P.channels() + H;
+        P.tail_elems = (x.conv_taps - 1) * P.channels();
+        break;
+    case OB_MIXER_TIME_MIXING:
+        P.f32_rows = 4 * H * x.dim;
+        P.tail_elems = width;
+        break;
+    default: P.f32_rows = H * (2 * x.dim + 2 * x.vdim);
     }
     P.f32_row0 = P.act_rows;
-    P.glu_row0 = P.f32_row0 + round_up(P.f32_rows, LIN_ROW_ALIGN);
-    HostDense in(P.glu_row0 + round_up(2 * glu, LIN_ROW_ALIGN), h_pitch);
+    P.out_width = H * x.vdim;
+    P.cols = round_up(P.out_width, LIN_K_ALIGN);
+}
+
+// The projections of the block's input.
+int LayeredGraph::fill_in(const ob_mixer_desc &x, MixerPlan &P, HostDense &in) {
+    const uint32_t H = x.n_head, G = x.n_kv_head, inner = H * x.vdim;
     uint32_t r = P.f32_row0;
     auto rows = [&](const ob_matrix_desc &d) {
         for (uint32_t i = 0; i < d.out_dim; ++i) in.copy(r++, 0, d, i);
     };
-    if (latent) {
+    if (x.kind == OB_MIXER_LATENT_ATTENTION) {
         for (uint32_t hd = 0; hd < H; ++hd) {
             for (uint32_t i = 0; i < x.dim; ++i) in.copy(hd * P.dim_p + i, 0, x.wq, hd * (x.dim + x.rot_dim) + i);
             for (uint32_t i = 0; i < x.rot_dim; ++i) in.copy(r++, 0, x.wq, hd * (x.dim + x.rot_dim) + x.dim + i);
         }
         rows(x.w_dkv);
         rows(x.w_gate);
-    } else if (attends) {
+    } else if (x.kind == OB_MIXER_ATTENTION) {
         r = 0;
         if (P.has_v) rows(x.wv);
         if (P.has_gate) rows(x.w_gate);
         r = P.f32_row0;
         rows(x.wq);
-        rows(x.wk);
+        if (P.own_kv) rows(x.wk);
+        if (P.head_gate) rows(x.w_gate);
         if (x.q_bias || x.k_bias || x.v_bias) {
             std::vector<float> bias(in.rows, 0.0f);
             if (x.v_bias) std::copy(x.v_bias, x.v_bias + G * x.vdim, bias.begin());
             if (x.q_bias) std::copy(x.q_bias, x.q_bias + H * x.n_map * x.dim, bias.begin() + P.f32_row0);
             if (x.k_bias) std::copy(x.k_bias, x.k_bias + G * x.n_map * x.dim, bias.begin() + P.f32_row0 + H * x.n_map * x.dim);
-            if ((rc = upload_now(bias.data(), bias.size(), &P.in_bias))) return rc;
+            if (int rc = upload_now(bias.data(), bias.size(), &P.in_bias)) return rc;
         }
-    } else {
+    } else if (x.kind == OB_MIXER_STATE_SPACE) {  // gate | channels, steps
+        for (uint32_t i = 0; i < inner; ++i) in.copy(i, 0, x.w_in, i);
+        for (uint32_t i = 0; i < P.f32_rows; ++i) in.copy(r++, 0, x.w_in, inner + i);
+    } else if (x.kind == OB_MIXER_RETENTION) {
         rows(x.wq);
         rows(x.wk);
         rows(x.wv);
         rows(x.w_gate);
     }
-    for (uint32_t i = 0; i < glu; ++i) {
-        in.copy(P.glu_row0 + 2 * i, 0, b.w_gate, i);
-        in.copy(P.glu_row0 + 2 * i + 1, 0, b.w_up, i);
+    return OB_OK;
+}
+
+int LayeredGraph::build_layer(const ob_block_desc &b, LayerPlan &P) {
+    const ob_mixer_desc &x = b.mixer;
+    int rc;
+    size_mixer(x, P);
+    P.sequential = b.post_norm1 != nullptr;
+    P.ff_kind = b.ff_kind;
+    const uint32_t glu = P.sequential ? 0 : b.n_ff;  // feed-forward inside the mixer's products
+    P.norm_gain = b.norm_gain;
+    P.n_ff = b.n_ff;
+    P.glu_limit = b.glu_limit;
+    P.glu_alpha = b.glu_alpha;
+    if (b.mixer2.kind) {
+        P.second = std::make_unique<MixerPlan>();
+        size_mixer(b.mixer2, *P.second);
+        P.scale = b.mixer_scale;
+        P.second->scale = b.mixer2_scale;
+        P.second->col0 = P.cols;
     }
-    if ((rc = upload(in, &P.in))) return rc;
+    // ---- everything that reads the normed input
+    P.glu_row0 = P.f32_row0 + round_up(P.f32_rows, LIN_ROW_ALIGN);
+    for (MixerPlan *q : {static_cast<MixerPlan *>(&P), P.second.get()}) {
+        if (!q || q->mx.kind == OB_MIXER_TIME_MIXING) continue;
+        HostDense in(q->f32_row0 + round_up(q->f32_rows, LIN_ROW_ALIGN) + (q == &P ? round_up(2 * glu, LIN_ROW_ALIGN) : 0), h_pitch);
+        if ((rc = fill_in(q == &P ? x : b.mixer2, *q, in))) return rc;
+        for (uint32_t i = 0; q == &P && i < glu; ++i) {
+            in.copy(P.glu_row0 + 2 * i, 0, b.w_gate, i);
+            in.copy(P.glu_row0 + 2 * i + 1, 0, b.w_up, i);
+        }
+        if ((rc = upload(in, &q->in))) return rc;
+    }
     // ---- output products side by side
-    P.mix_cols = round_up(H * x.vdim, LIN_K_ALIGN);
-    HostDense out(round_up(width, LIN_ROW_ALIGN), P.mix_cols + round_up(glu, LIN_K_ALIGN));
+    const uint32_t mix_cols = P.cols + (P.second ? P.second->cols : 0);
+    HostDense out(round_up(width, LIN_ROW_ALIGN), mix_cols + round_up(glu, LIN_K_ALIGN));
     for (uint32_t i = 0; i < width; ++i) {
         out.copy(i, 0, x.wo, i);
-        if (glu) out.copy(i, P.mix_cols, b.w_down, i);
+        if (P.second) out.copy(i, P.cols, b.mixer2.wo, i);
+        if (glu) out.copy(i, P.cols, b.w_down, i);
     }
     if ((rc = upload(out, &P.out))) return rc;
     if (x.o_bias) {
@@ -637,6 +890,7 @@ int LayeredGraph::build_layer(const ob_block_desc &b, LayerPlan &P) {
         if ((rc = upload_now(bias.data(), bias.size(), &P.out_bias))) return rc;
     }
     if (P.sequential && ((rc = upload_now(b.post_norm1, width, &P.post1)) || (rc = build_ff(b, P)))) return rc;
+    if (b.pre_norm1 && (rc = upload_now(b.pre_norm1, width, &P.pre1))) return rc;
     if (side_dim) {
         HostDense g(round_up(side_dim, LIN_ROW_ALIGN), h_pitch), pr(round_up(width, LIN_ROW_ALIGN), side_p);
         for (uint32_t i = 0; i < side_dim; ++i) g.copy(i, 0, b.side_gate, i);
@@ -644,8 +898,16 @@ int LayeredGraph::build_layer(const ob_block_desc &b, LayerPlan &P) {
         if ((rc = upload(g, &P.side_gate)) || (rc = upload(pr, &P.side_proj))) return rc;
         if ((rc = upload_f32(m, b.side_norm, width, &P.side_norm))) return rc;
     }
-    // ---- the mixer's own tensors
-    if (latent) {
+    if ((rc = build_mixer(x, P)) || (P.second && (rc = build_mixer(b.mixer2, *P.second)))) return rc;
+    OB_CUDA(m->ctx, cudaStreamSynchronize(m->ctx->stream));  // the host matrices end here
+    return OB_OK;
+}
+
+// The mixer's own tensors, cache and state.
+int LayeredGraph::build_mixer(const ob_mixer_desc &x, MixerPlan &P) {
+    const uint32_t H = x.n_head, G = x.n_kv_head;
+    int rc;
+    if (x.kind == OB_MIXER_LATENT_ATTENTION) {
         const uint32_t kr = round_up(x.kv_rank, LIN_ROW_ALIGN), vr = round_up(x.vdim, LIN_ROW_ALIGN);
         HostDense uk(H * kr, P.dim_p), uv(H * vr, P.kv_w);
         const uint16_t *src = reinterpret_cast<const uint16_t *>(x.w_uk.data);
@@ -668,18 +930,47 @@ int LayeredGraph::build_layer(const ob_block_desc &b, LayerPlan &P) {
         }
         if ((rc = upload_f32(m, x.kv_norm, x.kv_rank, &P.kv_norm))) return rc;
         if ((rc = scratch(&P.pool, (size_t)m->pool_pages * KV_PAGE * P.dq, es()))) return rc;
-    } else if (attends) {
-        if ((rc = upload_now(x.q_norm, x.dim, &P.q_norm)) || (rc = upload_now(x.k_norm, x.dim, &P.k_norm))) return rc;
-        if ((rc = scratch(&P.pool, (size_t)m->pool_pages * KV_PAGE * cache_elems(P), es()))) return rc;
+    } else if (x.kind == OB_MIXER_ATTENTION) {
+        const uint32_t whole_q = x.qk_norm_whole ? H : 1, whole_k = x.qk_norm_whole ? G : 1;
+        if (x.q_norm && (rc = upload_now(x.q_norm, whole_q * x.dim, &P.q_norm))) return rc;
+        if (x.k_norm && (rc = upload_now(x.k_norm, whole_k * x.dim, &P.k_norm))) return rc;
+        if (x.sink && (rc = upload_now(x.sink, H, &P.sink))) return rc;
+        if (!P.own_kv) P.pool = L[x.kv_layer - 1].pool;
+        else if ((rc = scratch(&P.pool, (size_t)m->pool_pages * KV_PAGE * cache_elems(P), es()))) return rc;
+    } else if (x.kind == OB_MIXER_STATE_SPACE) {
+        const uint32_t n = P.channels(), inner = H * x.vdim;
+        if ((rc = upload_now(x.conv_w, (size_t)n * x.conv_taps, &P.conv_w)) || (rc = upload_now(x.conv_b, n, &P.conv_b))) return rc;
+        if ((rc = upload_now(x.dt_bias, H, &P.dt_bias)) || (rc = upload_now(x.a_log, H, &P.a_log)) || (rc = upload_now(x.d_skip, H, &P.skip))) return rc;
+        if ((rc = upload_now(x.out_norm, inner, &P.out_norm, P.scale))) return rc;
+    } else if (x.kind == OB_MIXER_TIME_MIXING) {
+        const uint32_t n = H * x.dim, np = round_up(n, LIN_ROW_ALIGN), rank = x.w_decay1.out_dim;
+        HostDense rkvg(4 * np, h_pitch), d1(round_up(rank, LIN_ROW_ALIGN), h_pitch), d2(np, round_up(rank, LIN_K_ALIGN));
+        const ob_matrix_desc *each[4] = {&x.wq, &x.wk, &x.wv, &x.w_gate};
+        for (uint32_t k = 0; k < 4; ++k)
+            for (uint32_t i = 0; i < n; ++i) rkvg.copy(k * np + i, 0, *each[k], i);
+        for (uint32_t i = 0; i < rank; ++i) d1.copy(i, 0, x.w_decay1, i);
+        for (uint32_t i = 0; i < n; ++i) d2.copy(i, 0, x.w_decay2, i);
+        if ((rc = upload(rkvg, &P.rkvg)) || (rc = upload(d1, &P.decay1)) || (rc = upload(d2, &P.decay2))) return rc;
+        std::vector<float> d0(np, 0.0f);
+        std::copy(x.decay0, x.decay0 + n, d0.begin());
+        const float *mu[SHIFT_MIXES] = {x.mu_r, x.mu_k, x.mu_v, x.mu_g, x.mu_w};
+        for (uint32_t i = 0; i < SHIFT_MIXES; ++i)
+            if ((rc = upload_now(mu[i], width, &P.mu[i]))) return rc;
+        if ((rc = upload_now(d0.data(), np, &P.decay0)) || (rc = upload_now(x.bonus, n, &P.bonus)) || (rc = upload_now(x.out_norm, n, &P.out_norm, P.scale))) return rc;
     } else {
         if ((rc = upload_f32(m, x.decay, H, &P.decay))) return rc;
         P.decay_min = *std::min_element(x.decay, x.decay + H);
+    }
+    if (recurrent_kind(x.kind)) {
         if ((rc = scratch_f32(&P.state, (size_t)m->n_state_slots * state_elems(P)))) return rc;
+        if (P.tail_elems && (rc = scratch_f32(&P.tail, (size_t)m->n_state_slots * P.tail_elems))) return rc;
         has_state = true;
     }
-    OB_CUDA(m->ctx, cudaStreamSynchronize(m->ctx->stream));  // the host matrices end here
+    OB_CUDA(m->ctx, cudaStreamSynchronize(m->ctx->stream));
     P.mx.decay = nullptr;
-    P.mx.kv_norm = P.mx.q_norm = P.mx.k_norm = P.mx.q_bias = P.mx.k_bias = P.mx.v_bias = P.mx.o_bias = nullptr;
+    P.mx.kv_norm = P.mx.q_norm = P.mx.k_norm = P.mx.q_bias = P.mx.k_bias = P.mx.v_bias = P.mx.o_bias = P.mx.sink = nullptr;
+    P.mx.conv_w = P.mx.conv_b = P.mx.dt_bias = P.mx.a_log = P.mx.d_skip = P.mx.out_norm = P.mx.decay0 = P.mx.bonus = nullptr;
+    P.mx.mu_r = P.mx.mu_k = P.mx.mu_v = P.mx.mu_g = P.mx.mu_w = nullptr;
     return OB_OK;
 }
 
@@ -687,33 +978,60 @@ int LayeredGraph::build_layer(const ob_block_desc &b, LayerPlan &P) {
 int LayeredGraph::build_ff(const ob_block_desc &b, LayerPlan &P) {
     int rc;
     if (!b.n_ff) return OB_OK;
-    const bool experts = b.ff_kind == OB_FF_EXPERTS;
-    const uint32_t E = experts ? b.n_expert : 1, up_rows = round_up((experts ? 2 : 1) * b.n_ff, LIN_ROW_ALIGN), down_rows = round_up(width, LIN_ROW_ALIGN),
+    const bool experts = b.ff_kind == OB_FF_EXPERTS, gated = experts || b.ff_kind == OB_FF_GELU_GLU;
+    P.n_expert = experts ? b.n_expert : 0;
+    P.top = experts ? b.n_expert_used : 1;
+    P.router_softmax = b.router_softmax != 0;
+    // A shared expert in pieces of an expert's size: a gated feed-forward is the sum of its parts.
+    P.n_shared = experts ? (b.shared_ff + b.n_ff - 1) / b.n_ff : 0;
+    const uint32_t E = experts ? P.n_expert + P.n_shared : 1, up_rows = round_up((gated ? 2 : 1) * b.n_ff, LIN_ROW_ALIGN), down_rows = round_up(width, LIN_ROW_ALIGN),
                    kp = round_up(b.n_ff, LIN_K_ALIGN);
     if ((rc = upload_now(b.post_norm2, width, &P.post2))) return rc;
+    if (b.pre_norm2 && (rc = upload_now(b.pre_norm2, width, &P.pre2))) return rc;
     HostDense up(E * up_rows, h_pitch), down(E * down_rows, kp);
     for (uint32_t e = 0; e < E; ++e) {
-        for (uint32_t i = 0; i < b.n_ff; ++i) {
-            if (experts) {
-                up.copy(e * up_rows + 2 * i, 0, b.expert_gate[e], i);
-                up.copy(e * up_rows + 2 * i + 1, 0, b.expert_up[e], i);
-            } else {
-                up.copy(i, 0, b.w_up, i);
-            }
+        const bool shared = experts && e >= P.n_expert;
+        const uint32_t c0 = shared ? (e - P.n_expert) * b.n_ff : 0, n = shared ? std::min(b.n_ff, b.shared_ff - c0) : b.n_ff;
+        const ob_matrix_desc &g = !experts ? b.w_gate : shared ? b.shared_gate : b.expert_gate[e], &u = !experts ? b.w_up : shared ? b.shared_up : b.expert_up[e],
+                             &d = !experts ? b.w_down : shared ? b.shared_down : b.expert_down[e];
+        for (uint32_t i = 0; i < n; ++i) {
+            if (gated) up.copy(e * up_rows + 2 * i, 0, g, c0 + i);
+            up.copy(e * up_rows + (gated ? 2 * i + 1 : i), 0, u, c0 + i);
         }
-        for (uint32_t i = 0; i < width; ++i) down.copy(e * down_rows + i, 0, experts ? b.expert_down[e] : b.w_down, i);
+        for (uint32_t i = 0; i < width; ++i) down.copy(e * down_rows + i, 0, d, i, c0, n);
     }
     if ((rc = upload(up, &P.up)) || (rc = upload(down, &P.down))) return rc;
     if (experts) {
-        HostDense z(round_up(E, LIN_ROW_ALIGN), h_pitch);
-        for (uint32_t e = 0; e < E; ++e) z.copy(e, 0, b.w_router, e);
+        HostDense z(round_up(P.n_expert + 1, LIN_ROW_ALIGN), h_pitch);
+        for (uint32_t e = 0; e < P.n_expert; ++e) z.copy(e, 0, b.w_router, e);
+        if (P.n_shared) z.copy(P.n_expert, 0, b.w_shared_scale, 0);
         if ((rc = upload(z, &P.router))) return rc;
     }
     return OB_OK;
 }
 
+// The mixer's (cos, sin) by position.  Angles in double on the host: the table is exact to fp32 at any position.
+int LayeredGraph::rotation(MixerPlan &P, std::map<std::pair<std::vector<double>, float>, float2 *> &tables) {
+    const uint32_t half = P.mx.rot_dims / 2;
+    const float gain = P.mx.rot_gain != 0.0f ? P.mx.rot_gain : 1.0f;
+    std::vector<double> f(half);
+    for (uint32_t k = 0; k < half; ++k) f[k] = P.mx.rot_freqs ? P.mx.rot_freqs[k] : pow(P.mx.rot_base, -2.0 * k / P.mx.rot_dims);
+    P.mx.rot_freqs = nullptr;
+    float2 *&tab = tables[{f, gain}];
+    if (!tab) {
+        std::vector<float2> t((size_t)m->cfg.max_seq_len * half);
+        for (uint32_t p = 0; p < m->cfg.max_seq_len; ++p)
+            for (uint32_t k = 0; k < half; ++k) t[(size_t)p * half + k] = make_float2((float)(gain * cos(p * f[k])), (float)(gain * sin(p * f[k])));
+        int rc = dev_alloc(m, &tab, t.size());
+        if (rc) return rc;
+        OB_CUDA(m->ctx, cudaMemcpy(tab, t.data(), t.size() * sizeof(float2), cudaMemcpyHostToDevice));
+    }
+    P.rot = Rot{tab, P.mx.rot_dims, P.mx.rot_interleaved != 0};
+    return OB_OK;
+}
+
 int LayeredGraph::build(const ob_layered_desc &c) {
-    int rc;
+    int rc = OB_OK;
     const size_t T = m->T;
     f32 = c.compute_f32 != 0;
     width = c.n_embd;
@@ -725,33 +1043,25 @@ int LayeredGraph::build(const ob_layered_desc &c) {
     residual_mult = c.residual_mult;
     if (c.final_norm && (rc = upload_now(c.final_norm, width, &final_norm))) return rc;
     L.resize(c.n_layer);
-    std::map<std::pair<double, uint32_t>, float2 *> tables;
-    size_t act = 0, q_n = 0, o_n = 0, o_r = 0, kvp = 0, dq = 0, ex = 0, reach = 0, ff_n = 0, pairs = 0, experts = 0;
+    std::map<std::pair<std::vector<double>, float>, float2 *> tables;
+    size_t act = 0, q_n = 0, o_n = 0, o_r = 0, kvp = 0, dq = 0, ex = 0, reach = 0, ff_n = 0, pairs = 0, experts = 0, channels = 0, heads = 0, mixed = 0;
     bool sequential = false;
     for (uint32_t i = 0; i < c.n_layer; ++i) {
         LayerPlan &P = L[i];
         if ((rc = build_layer(c.layers[i], P))) return rc;
-        const uint32_t H = P.mx.n_head, half = P.mx.rot_dims / 2;
-        float2 *&tab = tables[{P.mx.rot_base, P.mx.rot_dims}];
-        if (!tab) {  // angles in double on the host: the table is exact to fp32 at any position
-            std::vector<float2> t((size_t)m->cfg.max_seq_len * half);
-            std::vector<double> f(half);
-            for (uint32_t k = 0; k < half; ++k) f[k] = pow(P.mx.rot_base, -2.0 * k / P.mx.rot_dims);
-            for (uint32_t p = 0; p < m->cfg.max_seq_len; ++p)
-                for (uint32_t k = 0; k < half; ++k) t[(size_t)p * half + k] = make_float2((float)cos(p * f[k]), (float)sin(p * f[k]));
-            if ((rc = dev_alloc(m, &tab, t.size()))) return rc;
-            OB_CUDA(m->ctx, cudaMemcpy(tab, t.data(), t.size() * sizeof(float2), cudaMemcpyHostToDevice));
-        }
-        P.rot = Rot{tab, P.mx.rot_dims, P.mx.rot_interleaved != 0};
-        act = std::max<size_t>(act, P.act_rows);
-        y_pitch = std::max(y_pitch, round_up(P.f32_rows, 4));
         cat_pitch = std::max(cat_pitch, P.out.kp);
         sequential |= P.sequential;
-        if (P.sequential && P.n_ff) ff_n = std::max<size_t>(ff_n, T * P.top * P.down.kp);
+        if (P.sequential && P.n_ff) ff_n = std::max<size_t>(ff_n, T * P.pairs() * P.down.kp);
         if (P.n_expert) {
-            pairs = std::max<size_t>(pairs, T * P.top);
-            experts = std::max<size_t>(experts, P.n_expert);
+            pairs = std::max<size_t>(pairs, T * P.pairs());
+            experts = std::max<size_t>(experts, P.n_expert + P.n_shared + 1);
         }
+    }
+    each_mixer([&](MixerPlan &P) {
+        const uint32_t H = P.mx.n_head;
+        if (!rc) rc = rotation(P, tables);
+        act = std::max<size_t>(act, P.act_rows);
+        y_pitch = std::max(y_pitch, round_up(P.f32_rows, 4));
         if (P.mx.kind == OB_MIXER_ATTENTION) {
             q_n = std::max<size_t>(q_n, (size_t)H * P.mx.n_map * P.dim_p);
         } else if (P.pool) {
@@ -765,8 +1075,16 @@ int LayeredGraph::build(const ob_layered_desc &c) {
             }
         } else {
             o_r = std::max<size_t>(o_r, (size_t)H * P.mx.vdim);
+            if (P.mx.kind == OB_MIXER_STATE_SPACE) {
+                channels = std::max<size_t>(channels, P.channels());
+                heads = std::max<size_t>(heads, H);
+            } else if (P.mx.kind == OB_MIXER_TIME_MIXING) {
+                mixed = std::max<size_t>(mixed, (size_t)H * P.mx.dim);
+                low_p = std::max(low_p, P.decay2.kp);
+            }
         }
-    }
+    });
+    if (rc) return rc;
     {
         if ((rc = dev_alloc(m, &embd, (size_t)c.n_vocab * width))) return rc;
         OB_CUDA(m->ctx, cudaMemcpy(embd, c.token_embd.data, (size_t)c.n_vocab * width * 2, cudaMemcpyHostToDevice));
@@ -796,6 +1114,8 @@ int LayeredGraph::build(const ob_layered_desc &c) {
         key_cap = (uint32_t)(T + reach);
         if ((rc = scratch(&lat, (size_t)key_cap * dq, 2)) || (rc = scratch(&expanded, (size_t)key_cap * ex, 2))) return rc;
     }
+    if (channels && ((rc = scratch_f32(&conv, T * channels)) || (rc = dev_alloc(m, &steps, T * heads)))) return rc;
+    if (mixed && ((rc = scratch(&mix, T * SHIFT_MIXES * h_pitch, es())) || (rc = scratch(&low, T * low_p, es())) || (rc = scratch_f32(&decays, T * mixed)))) return rc;
     if (side_dim && ((rc = scratch(&sg, T * side_p, es())) || (rc = scratch_f32(&sy, T * width)))) return rc;
     if (!f32 && (rc = scratch_f32(&split_part, linear_split_bytes() / 4))) return rc;
     if (kvp && !f32) {  // at most one CTA per SM, of 64 rows, writes partial results at a time (launch_latent_attention)
@@ -814,15 +1134,13 @@ int check_dense(ob_ctx *ctx, const ob_matrix_desc &d, uint32_t in_dim, uint32_t 
     return OB_OK;
 }
 
-int check_block(ob_ctx *ctx, const ob_layered_desc &c, uint32_t i) {
-    const ob_block_desc &b = c.layers[i];
-    const ob_mixer_desc &x = b.mixer;
+int check_mixer(ob_ctx *ctx, const ob_layered_desc &c, uint32_t i, const ob_mixer_desc &x) {
     const std::string at = "layer " + std::to_string(i) + " ";
     int rc;
     if (!x.n_head || !x.dim || !x.vdim) return fail(ctx, OB_ERR_INVALID, "layered model: " + at + "mixer sizes missing");
     const uint32_t H = x.n_head, G = x.n_kv_head, E = c.n_embd, rotating = x.kind == OB_MIXER_LATENT_ATTENTION ? x.rot_dim : x.dim;
     if ((x.rot_dims & 1) || x.rot_dims > rotating) return fail(ctx, OB_ERR_INVALID, "layered model: " + at + "rot_dims must be even and fit the rotated vector");
-    if (x.rot_dims && !(x.rot_base > 0)) return fail(ctx, OB_ERR_INVALID, "layered model: " + at + "rot_base must be positive");
+    if (x.rot_dims && !x.rot_freqs && !(x.rot_base > 0)) return fail(ctx, OB_ERR_INVALID, "layered model: " + at + "rot_base must be positive");
     if (x.kind == OB_MIXER_LATENT_ATTENTION) {
         if (!x.kv_rank || !x.kv_norm) return fail(ctx, OB_ERR_INVALID, "layered model: " + at + "latent size or norm missing");
         if ((uint64_t)(2 * x.kv_rank + x.rot_dim + 256) * 4 > 128 * 1024) return fail(ctx, OB_ERR_UNSUPPORTED, "layered model: " + at + "kv_rank too large");
@@ -842,34 +1160,93 @@ int check_block(ob_ctx *ctx, const ob_layered_desc &c, uint32_t i) {
         if (!G || H % G) return fail(ctx, OB_ERR_INVALID, "layered model: " + at + "n_kv_head does not divide n_head");
         if (!(x.scale > 0)) return fail(ctx, OB_ERR_INVALID, "layered model: " + at + "scale must be positive");
         if (x.n_map != 1 && x.n_map != 2) return fail(ctx, OB_ERR_UNSUPPORTED, "layered model: " + at + "one or two maps per head");
-        if (!x.q_norm || !x.k_norm) return fail(ctx, OB_ERR_INVALID, "layered model: " + at + "query or key norm missing");
+        const bool own = !x.kv_layer;
+        if ((x.q_norm != nullptr) != (x.k_norm != nullptr) && own) return fail(ctx, OB_ERR_INVALID, "layered model: " + at + "query or key norm missing");
+        if (x.n_map != 1 && (x.qk_norm_whole || x.keep_first || x.kv_layer || x.softcap > 0 || x.sink))
+            return fail(ctx, OB_ERR_UNSUPPORTED, "layered model: " + at + "norms of whole projections, kept tokens, shared keys, soft caps and sinks go with one map");
+        if (!own) {
+            if (x.kv_layer > i) return fail(ctx, OB_ERR_INVALID, "layered model: " + at + "keys and values come from an earlier layer");
+            const ob_mixer_desc &o = c.layers[x.kv_layer - 1].mixer;
+            if (o.kind != OB_MIXER_ATTENTION || o.kv_layer || o.n_kv_head != G || o.dim != x.dim || o.vdim != x.vdim || o.n_map != x.n_map)
+                return fail(ctx, OB_ERR_INVALID, "layered model: " + at + "the layer of its keys and values has other ones");
+            if (x.wk.data || x.wv.data || x.k_norm || x.k_bias || x.v_bias) return fail(ctx, OB_ERR_INVALID, "layered model: " + at + "has keys and values of another layer and of its own");
+        }
         if (!attention_supported(x.dim, x.vdim)) return fail(ctx, OB_ERR_UNSUPPORTED, "layered model: " + at + "attention head too large");
         if ((rc = check_dense(ctx, x.wq, E, H * x.n_map * x.dim, at + "wq"))) return rc;
-        if ((rc = check_dense(ctx, x.wk, E, G * x.n_map * x.dim, at + "wk"))) return rc;
-        if (x.wv.data) {
+        if (own && (rc = check_dense(ctx, x.wk, E, G * x.n_map * x.dim, at + "wk"))) return rc;
+        if (!own) {
+        } else if (x.wv.data) {
             if ((rc = check_dense(ctx, x.wv, E, G * x.vdim, at + "wv"))) return rc;
         } else if (x.n_map != 1 || x.vdim != x.dim || x.v_bias) {
             return fail(ctx, OB_ERR_INVALID, "layered model: " + at + "keys can be the values of one map of their own size");
         }
-        if (x.w_gate.data && (rc = check_dense(ctx, x.w_gate, E, H * x.vdim, at + "mixer gate"))) return rc;
+        if (x.w_gate.data && x.w_gate.out_dim == H && x.n_map != 1) return fail(ctx, OB_ERR_UNSUPPORTED, "layered model: " + at + "gates of whole heads go with one map");
+        if (x.w_gate.data && (rc = check_dense(ctx, x.w_gate, E, x.w_gate.out_dim == H ? H : H * x.vdim, at + "mixer gate"))) return rc;
+    } else if (x.kind == OB_MIXER_STATE_SPACE) {
+        const uint32_t inner = H * x.vdim, n = inner + 2 * x.n_group * x.dim;
+        if (!x.n_group || H % x.n_group) return fail(ctx, OB_ERR_INVALID, "layered model: " + at + "n_group does not divide n_head");
+        if (!x.n_norm_group || inner % x.n_norm_group) return fail(ctx, OB_ERR_INVALID, "layered model: " + at + "n_norm_group does not divide the inner width");
+        if (!x.conv_taps || x.conv_taps > CONV_MAX_TAPS) return fail(ctx, OB_ERR_UNSUPPORTED, "layered model: " + at + "the convolution has 1 to 16 taps");
+        if (!recurrence_supported(x.dim)) return fail(ctx, OB_ERR_UNSUPPORTED, "layered model: " + at + "a state has at most 256 entries per value");
+        if (!state_space_out_supported(inner / x.n_norm_group)) return fail(ctx, OB_ERR_UNSUPPORTED, "layered model: " + at + "norm group too large");
+        if (!x.conv_w || !x.conv_b || !x.dt_bias || !x.a_log || !x.d_skip || !x.out_norm) return fail(ctx, OB_ERR_INVALID, "layered model: " + at + "state-space vectors missing");
+        if ((rc = check_dense(ctx, x.w_in, E, inner + n + H, at + "w_in"))) return rc;
+    } else if (x.kind == OB_MIXER_TIME_MIXING) {
+        const uint32_t n = H * x.dim;
+        if (x.vdim != x.dim) return fail(ctx, OB_ERR_INVALID, "layered model: " + at + "time mixing has values of its keys' size");
+        if (!c.layers[i].post_norm1) return fail(ctx, OB_ERR_UNSUPPORTED, "layered model: " + at + "time mixing belongs in sequential blocks");
+        if (!recurrence_supported(x.dim)) return fail(ctx, OB_ERR_UNSUPPORTED, "layered model: " + at + "a state has at most 256 entries per value");
+        if (!x.mu_r || !x.mu_k || !x.mu_v || !x.mu_g || !x.mu_w || !x.decay0 || !x.bonus || !x.out_norm)
+            return fail(ctx, OB_ERR_INVALID, "layered model: " + at + "time-mixing vectors missing");
+        if ((rc = check_dense(ctx, x.wq, E, n, at + "wq")) || (rc = check_dense(ctx, x.wk, E, n, at + "wk")) || (rc = check_dense(ctx, x.wv, E, n, at + "wv"))) return rc;
+        if ((rc = check_dense(ctx, x.w_gate, E, n, at + "mixer gate"))) return rc;
+        if (!x.w_decay1.out_dim) return fail(ctx, OB_ERR_INVALID, "layered model: " + at + "w_decay1 missing");
+        if ((rc = check_dense(ctx, x.w_decay1, E, x.w_decay1.out_dim, at + "w_decay1"))) return rc;
+        if ((rc = check_dense(ctx, x.w_decay2, x.w_decay1.out_dim, n, at + "w_decay2"))) return rc;
     } else {
         return fail(ctx, OB_ERR_UNSUPPORTED, "layered model: " + at + "unknown mixer");
     }
     if (x.kind != OB_MIXER_ATTENTION && (x.q_bias || x.k_bias || x.v_bias)) return fail(ctx, OB_ERR_UNSUPPORTED, "layered model: " + at + "the mixer has no biases");
+    if (x.kind != OB_MIXER_ATTENTION && x.o_bias) return fail(ctx, OB_ERR_UNSUPPORTED, "layered model: " + at + "the mixer has no biases");
+    return check_dense(ctx, x.wo, H * x.vdim, E, at + "wo");
+}
+
+int check_block(ob_ctx *ctx, const ob_layered_desc &c, uint32_t i) {
+    const ob_block_desc &b = c.layers[i];
+    const std::string at = "layer " + std::to_string(i) + " ";
+    const uint32_t E = c.n_embd;
+    int rc;
+    if ((rc = check_mixer(ctx, c, i, b.mixer))) return rc;
+    if (b.mixer2.kind) {
+        auto scales = [](uint32_t kind) { return kind == OB_MIXER_ATTENTION || kind == OB_MIXER_STATE_SPACE || kind == OB_MIXER_TIME_MIXING; };
+        if (!b.post_norm1 || !scales(b.mixer.kind) || !scales(b.mixer2.kind) || b.mixer.o_bias || b.mixer2.o_bias || b.mixer.n_map > 1 || b.mixer2.n_map > 1 ||
+            b.mixer2.kv_layer || (b.mixer.kind != OB_MIXER_ATTENTION) == (b.mixer2.kind != OB_MIXER_ATTENTION))
+            return fail(ctx, OB_ERR_UNSUPPORTED, "layered model: " + at + "two mixers: attention with one map beside a recurrent layer, in a sequential block");
+        if ((rc = check_mixer(ctx, c, i, b.mixer2))) return rc;
+    }
     if ((b.post_norm1 != nullptr) != (c.layers[0].post_norm1 != nullptr)) return fail(ctx, OB_ERR_UNSUPPORTED, "layered model: " + at + "blocks of two kinds");
-    if ((rc = check_dense(ctx, x.wo, H * x.vdim, E, at + "wo"))) return rc;
+    if ((b.pre_norm1 != nullptr) != (c.layers[0].pre_norm1 != nullptr)) return fail(ctx, OB_ERR_UNSUPPORTED, "layered model: " + at + "blocks with and without normed inputs");
+    if (b.pre_norm1 && !b.post_norm1) return fail(ctx, OB_ERR_UNSUPPORTED, "layered model: " + at + "norms of inputs belong in sequential blocks");
     if (b.post_norm1) {
         if (c.side_dim) return fail(ctx, OB_ERR_UNSUPPORTED, "layered model: " + at + "sequential blocks have no per-layer token input");
         if (!b.n_ff) return OB_OK;
         if (!b.post_norm2) return fail(ctx, OB_ERR_INVALID, "layered model: " + at + "norm of the feed-forward missing");
-        if (b.ff_kind == OB_FF_RELU2) {
+        if ((b.pre_norm2 != nullptr) != (b.pre_norm1 != nullptr)) return fail(ctx, OB_ERR_INVALID, "layered model: " + at + "norm of the feed-forward's input");
+        if (b.ff_kind == OB_FF_GELU_GLU && (rc = check_dense(ctx, b.w_gate, E, b.n_ff, at + "ff gate"))) return rc;
+        if (b.ff_kind == OB_FF_RELU2 || b.ff_kind == OB_FF_GELU_GLU) {
             if ((rc = check_dense(ctx, b.w_up, E, b.n_ff, at + "ff up"))) return rc;
             return check_dense(ctx, b.w_down, b.n_ff, E, at + "ff down");
         }
         if (b.ff_kind != OB_FF_EXPERTS) return fail(ctx, OB_ERR_UNSUPPORTED, "layered model: " + at + "unknown feed-forward");
         if (!b.n_expert || !b.n_expert_used || b.n_expert_used > b.n_expert || !b.expert_gate || !b.expert_up || !b.expert_down)
             return fail(ctx, OB_ERR_INVALID, "layered model: " + at + "experts missing");
-        if (b.n_expert > MOE_MAX_EXPERTS) return fail(ctx, OB_ERR_UNSUPPORTED, "layered model: " + at + "too many experts");
+        if (b.shared_ff && !b.router_softmax) return fail(ctx, OB_ERR_UNSUPPORTED, "layered model: " + at + "a shared expert goes with weighted outputs");
+        if (b.shared_ff) {
+            if ((rc = check_dense(ctx, b.shared_gate, E, b.shared_ff, at + "shared gate")) || (rc = check_dense(ctx, b.shared_up, E, b.shared_ff, at + "shared up")) ||
+                (rc = check_dense(ctx, b.shared_down, b.shared_ff, E, at + "shared down")) || (rc = check_dense(ctx, b.w_shared_scale, E, 1, at + "scale of the shared expert")))
+                return rc;
+        }
+        if ((uint64_t)b.n_expert + (b.shared_ff + b.n_ff - 1) / b.n_ff > MOE_MAX_EXPERTS) return fail(ctx, OB_ERR_UNSUPPORTED, "layered model: " + at + "too many experts");
         if ((rc = check_dense(ctx, b.w_router, E, b.n_expert, at + "router"))) return rc;
         for (uint32_t e = 0; e < b.n_expert; ++e) {
             if ((rc = check_dense(ctx, b.expert_gate[e], E, b.n_ff, at + "expert gate"))) return rc;
@@ -907,7 +1284,7 @@ extern "C" int ob_layered_model_create(ob_ctx *ctx, const ob_layered_desc *desc,
     bool state = false;
     for (uint32_t i = 0; i < c.n_layer; ++i) {
         if ((rc = check_block(ctx, c, i))) return rc;
-        state |= c.layers[i].mixer.kind == OB_MIXER_RETENTION;
+        state |= recurrent_kind(c.layers[i].mixer.kind) || recurrent_kind(c.layers[i].mixer2.kind);
     }
 
     std::unique_lock<std::mutex> g(ctx->mu);
@@ -915,6 +1292,7 @@ extern "C" int ob_layered_model_create(ob_ctx *ctx, const ob_layered_desc *desc,
     OB_CUDA(ctx, linear_configure());
     OB_CUDA(ctx, mixers_configure());
     OB_CUDA(ctx, attention_configure());
+    OB_CUDA(ctx, recurrence_configure());
     ob_model *m = new ob_model;
     m->ctx = ctx;
     m->cfg.n_vocab = c.n_vocab;

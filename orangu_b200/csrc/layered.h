@@ -24,7 +24,10 @@ enum LinEpilogue {
     LE_GELU_EMB = 4,  // out activation = gelu_tanh(v) * emb[token t][emb_col0 + row]
     LE_GATED = 5,     // out activation = v * sigmoid(gate[t * gate_pitch + batch])
     LE_RELU2 = 6,     // out activation = max(v, 0)^2
-    LE_SWIGLU = 7     // rows (2j, 2j+1) are (gate j, up j), both times row_scale[t]: out activation j = silu(g) u
+    LE_SWIGLU = 7,    // rows (2j, 2j+1) are (gate j, up j), both times row_scale[t]: out activation j = silu(g) u, times out_scale[t]
+    LE_GELU_GLU = 8,  // rows (2j, 2j+1) are (gate j, up j): out activation j = gelu_tanh(g) u
+    LE_TANH = 9,      // out activation = tanh(v)
+    LE_DECAY = 10     // out f32 = exp(-exp(v))
 };
 struct LinTile {          // rows of a grouped product that share a batch entry
     uint32_t batch, row0, n;
@@ -54,7 +57,7 @@ struct LinArgs {
     uint32_t gate_pitch = 0;
     float *split_part = nullptr;  // scratch of products that split K, linear_split_bytes
     const float *bias = nullptr;  // [n_batch][n_rows] added to the products before the epilogue
-    const float *row_scale = nullptr;  // [T]
+    const float *row_scale = nullptr, *out_scale = nullptr;  // [T]
     // Grouped products: every row of x has a batch entry of its own.  Either row by row, or in tiles of rows with one entry each
     // (rows of one entry next to one another), made on the device: *n_tiles of at most max_tiles, of tile_rows rows or fewer.
     const uint32_t *row_batch = nullptr;  // [T], row t reads row t / x_div of x
@@ -73,13 +76,13 @@ int linear_take_status();        // 1 when a bounded wait inside a product ran o
 void linear_mark_launched();     // a replayed graph may have run one of the tensor-core products
 
 // ---- mixers.cu -------------------------------------------------------------------------------------------------------
-// x = embedding rows; h = x / rms(x) * gain as activation, or (normed false) x itself.
-void launch_embed(const __nv_bfloat16 *table, uint32_t width, const uint32_t *tokens, uint32_t T, float *x, bool normed, float eps, float gain, void *h,
-                  uint32_t h_pitch, bool f32, cudaStream_t st);
+// x = embedding rows; h = x / rms(x) * gain (* w) as activation, or (normed false) x itself; w [width], may be null.
+void launch_embed(const __nv_bfloat16 *table, uint32_t width, const uint32_t *tokens, uint32_t T, float *x, bool normed, float eps, float gain, const float *w,
+                  void *h, uint32_t h_pitch, bool f32, cudaStream_t st);
 // h[i] = x[row i] / rms(x[row i]) * gain (* w), as activation; rows == nullptr: row i; w [width], may be null.
 void launch_norm(const float *x, uint32_t width, const uint32_t *rows, uint32_t n, float eps, float gain, const float *w, void *h, uint32_t h_pitch, bool f32,
                  cudaStream_t st);
-struct PostNormArgs {        // x += mult * y / rms(y) * w, then h = x as activation
+struct PostNormArgs {        // x += mult * y / rms(y) * w, then h = x, or x / rms(x) * next_w, as activation
     float *x;                // [T][width]
     const float *y;          // [T * top][width]: the `top` rows of a token are added up first
     const uint32_t *rows;    // where they are, [T * top]; null: in order
@@ -89,6 +92,7 @@ struct PostNormArgs {        // x += mult * y / rms(y) * w, then h = x as activa
     float eps, mult;
     void *h;                 // null: not needed
     uint32_t h_pitch;
+    const float *next_w;     // [width]; null: h is x itself
     uint32_t *zero;          // set to zero for whoever counts next, n_zero words; may be null
     uint32_t n_zero;
 };
@@ -183,15 +187,21 @@ bool retention_supported(uint32_t dim);
 uint32_t launch_retention(const RetentionArgs &a, bool f32, int sm_count, cudaStream_t st);
 // ---- gqa.cu ----------------------------------------------------------------------------------------------------------
 struct AttentionArgs {       // softmax attention of one layer over T rows
-    const float *y;          // f32 projections [T][y_pitch]: queries [n_head][n_map][dim], keys [n_kv][n_map][dim]
+    const float *y;          // f32 projections [T][y_pitch]: queries [n_head][n_map][dim], keys [n_kv][n_map][dim] (own_kv)
     uint32_t y_pitch;
     const void *va;          // activations [T][va_pitch]: values [n_kv][vdim] (has_v; else the values are the keys as projected), gates [n_head][vdim] from gate0
     uint32_t va_pitch, gate0;
     bool has_v, has_gate;
     uint32_t n_head, n_kv, n_map, dim, vdim, window;  // window 0: no limit
     uint32_t dim_p, vdim_p, row;  // padded sizes; elements of a cache row: keys [n_map][dim_p], value [vdim_p], padding
-    float eps, scale, map_weight, head_gain;
-    const float *q_norm, *k_norm;  // [dim]
+    float eps, scale, map_weight, head_gain;  // head_gain: of every head's output
+    const float *q_norm, *k_norm;  // [dim], with norm_whole [n_head * dim] and [n_kv * dim]; null: no norm
+    bool norm_whole;         // a token's queries (keys) are normed all together
+    bool own_kv;             // keys and values are appended to the cache; else another layer has done so
+    uint32_t keep;           // first positions that stay visible beyond the window
+    float softcap;           // > 0: score = softcap tanh(score / softcap)
+    const float *sink;       // [n_head]: exp of it is added to the softmax's denominator; null: none
+    const float *head_gate;  // f32 [T][y_pitch]: sigmoid of entry h scales head h; null: none.  These four: one map
     Rot rot;
     void *q;                 // activations [T][n_head][n_map][dim_p]
     void *cache;             // activations [page][n_kv][16][row]
@@ -218,26 +228,107 @@ bool launch_attention_prompt(const AttentionArgs &a, int sm_count, cudaStream_t 
 int attention_take_status();  // as linear_take_status
 
 // ---- moe.cu ----------------------------------------------------------------------------------------------------------
-struct MoeArgs {             // routing of T tokens to `top` of n_expert experts; a (token, choice) is a pair, t * top + choice
+struct MoeArgs {             // routing of T tokens to `top` of n_expert experts; a (token, choice) is a pair, t * (top + n_shared) + choice
     const void *x;           // activations [T][x_pitch], x_pitch a multiple of 64
     uint32_t x_pitch;
-    const __nv_bfloat16 *w;  // router [n_expert or more][x_pitch]
+    const __nv_bfloat16 *w;  // router [n_expert (+ 1 with n_shared) or more][x_pitch]
     const float *logits;     // [T][logit_pitch]: logits made by a product; null: the routing kernel makes them
     uint32_t logit_pitch;
     uint32_t n_expert, top, T;
-    uint32_t *expert;        // [T * top]
-    float *score;            // [T * top]
+    uint32_t n_shared;       // experts n_expert .. that every token uses after its chosen ones; their score is the sigmoid of logit n_expert
+    bool softmax;            // scores of the chosen experts: the softmax over their logits, else the sigmoid of each
+    uint32_t *expert;        // [pairs]
+    float *score;            // [pairs]
     // grouping (null: pairs stay in order): pairs of one expert next to one another
-    uint32_t *count;         // [n_expert], zero before and left for the caller to zero
-    uint32_t *rank, *row;    // [T * top]: place among the expert's pairs; row of the pair
-    void *gathered;          // activations [T * top][x_pitch]
-    float *row_score;        // [T * top], by row
+    uint32_t *count;         // [n_expert + n_shared], zero before and left for the caller to zero
+    uint32_t *rank, *row;    // [pairs]: place among the expert's pairs; row of the pair
+    void *gathered;          // activations [pairs][x_pitch]
+    float *row_score;        // [pairs], by row
     LinTile *tiles;          // tiles of tile_rows rows or fewer, *n_tiles of them
     uint32_t *n_tiles, tile_rows;
 };
 constexpr uint32_t MOE_MAX_EXPERTS = 1024;
 constexpr uint32_t MOE_DOT_TOKENS = 64;  // up to this many tokens the routing kernel makes the logits itself
 uint32_t launch_moe_route(const MoeArgs &a, bool f32, cudaStream_t st);  // returns the kernels launched
+
+// ---- recurrence.cu ---------------------------------------------------------------------------------------------------
+// Per head a state S [dim][vdim] in fp32.  With a decay per token: S = a S + k (s v)^T, o = S^T q.  With a decay per key entry:
+// o = S^T q, then S = diag(w) S + k v^T.
+struct RecurrenceArgs {
+    const float *q, *k, *v;  // rows of [n_head / share][dim], the same, [n_head][vdim]
+    uint32_t pitch;          // of all three
+    uint32_t share;          // consecutive heads that share q and k
+    const float2 *step;      // [T][n_head] (a, s); null: decay per key entry
+    const float *w;          // rows of [n_head][dim]
+    uint32_t w_pitch;
+    uint32_t n_head, dim, vdim;
+    float *state;            // [slot][n_head][dim][vdim]
+    float *o;                // [T][n_head * vdim]
+    uint32_t n_seq, first_long;  // spans from first_long on are long (PREFILL_SPAN rows or more)
+    const RowSpan *spans;
+    const uint32_t *positions;
+    const int32_t *slots;    // [T]
+};
+cudaError_t recurrence_configure();
+bool recurrence_supported(uint32_t dim);
+uint32_t launch_recurrence(const RecurrenceArgs &a, int sm_count, cudaStream_t st);  // returns the kernels launched
+
+struct ConvArgs {            // causal convolution per channel, silu; and the steps of a state-space layer
+    const float *y;          // projections [T][y_pitch]: inputs of the channels, then [n_head] raw step sizes
+    uint32_t y_pitch, n_channel, taps, n_head;
+    const float *w, *b;      // [n_channel][taps] (the last tap meets the current token), [n_channel]
+    float *state;            // [slot][taps - 1][n_channel]: the last inputs, the oldest first
+    float *u;                // [T][n_channel]
+    const float *dt_bias, *a_log;  // [n_head]
+    float2 *step;            // [T][n_head]: (exp(-exp(a_log) dt), dt) with dt = softplus(raw + dt_bias)
+    uint32_t T, n_seq;
+    const RowSpan *spans, *h_spans;
+    bool single;
+    const uint32_t *positions;
+    const int32_t *slots;
+};
+constexpr uint32_t CONV_MAX_TAPS = 16;
+void launch_conv(const ConvArgs &a, cudaStream_t st);
+
+struct StateSpaceOutArgs {   // (o + skip x) silu(z), normed in n_part equal parts, times norm
+    const float *o, *x;      // [T][inner]; rows of [inner]
+    uint32_t x_pitch;
+    const void *z;           // activations [T][z_pitch]
+    uint32_t z_pitch, inner, vdim, n_part, T;
+    const float *skip, *norm;  // [inner / vdim], [inner]
+    float eps;
+    void *out;               // activations [T][out_pitch]
+    uint32_t out_pitch;
+};
+bool state_space_out_supported(uint32_t part);
+void launch_state_space_out(const StateSpaceOutArgs &a, bool f32, cudaStream_t st);
+
+constexpr uint32_t SHIFT_MIXES = 5;
+struct ShiftMixArgs {        // h = x / rms(x) * norm; mix i = h + (h' - h) mu[i], h' the previous token's h
+    const float *x;          // [T][width]
+    const float *norm;       // null: h is x
+    const float *mu[SHIFT_MIXES];
+    float *state;            // [slot][width]: the last token's h
+    void *mix;               // activations [T][SHIFT_MIXES * pitch]
+    uint32_t width, pitch, T, n_seq;
+    float eps;
+    const RowSpan *spans;
+    bool single;
+    const uint32_t *positions;
+    const int32_t *slots;
+};
+void launch_shift_mix(const ShiftMixArgs &a, bool f32, cudaStream_t st);
+
+struct TimeMixOutArgs {      // per head: (o + (sum r bonus k) v) over its root mean square, times norm, times silu(gate)
+    const float *o;          // [T][n_head * dim]
+    const float *r, *k, *v, *gate;  // rows of [n_head * dim]
+    uint32_t pitch, n_head, dim, T;
+    const float *bonus, *norm;  // [n_head * dim]
+    float eps;
+    void *out;
+    uint32_t out_pitch;
+};
+void launch_time_mix_out(const TimeMixOutArgs &a, bool f32, cudaStream_t st);
 
 // Pages [0, n_pages) of one sequence's table to another's within a pool of pages of page_bytes (a multiple of 16).
 void launch_copy_pages(void *pool, uint64_t page_bytes, const int32_t *src_table, const int32_t *dst_table, uint32_t n_pages, cudaStream_t st);

@@ -135,7 +135,31 @@ __device__ __forceinline__ void epilogue_store(const LinArgs &a, uint32_t batch,
                 const float gt = v[2 * j] * w;
                 o[j] = gt * sigmoidf(gt) * (v[2 * j + 1] * w);
             }
+            if (a.out_scale) {
+                const float f = a.out_scale[t];
+#pragma unroll
+                for (int j = 0; j < N / 2; ++j) o[j] *= f;
+            }
             store_row<(N / 2 > 0 ? N / 2 : 1)>(static_cast<TA *>(g.out) + base + k / 2, o, n / 2);
+            break;
+        }
+        case LE_GELU_GLU: {
+            float o[N / 2 > 0 ? N / 2 : 1];
+#pragma unroll
+            for (int j = 0; j < N / 2; ++j) o[j] = gelu_tanhf(v[2 * j]) * v[2 * j + 1];
+            store_row<(N / 2 > 0 ? N / 2 : 1)>(static_cast<TA *>(g.out) + base + k / 2, o, n / 2);
+            break;
+        }
+        case LE_TANH: {
+#pragma unroll
+            for (int i = 0; i < N; ++i) v[i] = tanhf(v[i]);
+            store_row<N>(static_cast<TA *>(g.out) + base + k, v, n);
+            break;
+        }
+        case LE_DECAY: {
+#pragma unroll
+            for (int i = 0; i < N; ++i) v[i] = expf(-expf(v[i]));
+            store_row<N>(static_cast<float *>(g.out) + base + k, v, n);
             break;
         }
         default: {  // LE_GATED

@@ -20,9 +20,10 @@ namespace {
 // at a time through memory.
 constexpr int ROW_VECS = 4;
 
-// x = the token's embedding, h = x / rms(x) * gain or x.
+// x = the token's embedding, h = x / rms(x) * gain (* w) or x.
 template <typename TA, int NV>
-__global__ void __launch_bounds__(1024) embed_kernel(const bf16 *table, uint32_t width, const uint32_t *tokens, float *x, bool normed, float eps, float gain, TA *h, uint32_t h_pitch) {
+__global__ void __launch_bounds__(1024) embed_kernel(const bf16 *table, uint32_t width, const uint32_t *tokens, float *x, bool normed, float eps, float gain, const float *w, TA *h,
+                                                     uint32_t h_pitch) {
     __shared__ float red[33];
     pdl_release();
     pdl_wait();
@@ -45,7 +46,7 @@ __global__ void __launch_bounds__(1024) embed_kernel(const bf16 *table, uint32_t
 #pragma unroll
         for (int i = 0; i < NV; ++i) {
             const uint32_t c = 4 * (threadIdx.x + i * blockDim.x);
-            if (c < width) store4<TA>(hr + c, mul4(v[i], f));
+            if (c < width) store4<TA>(hr + c, w ? mul44(mul4(v[i], f), *reinterpret_cast<const float4 *>(w + c)) : mul4(v[i], f));
         }
     } else {
         for (uint32_t i = threadIdx.x; i < width; i += blockDim.x) {
@@ -54,7 +55,7 @@ __global__ void __launch_bounds__(1024) embed_kernel(const bf16 *table, uint32_t
             s += v * v;
         }
         const float f = normed ? inv_rms(block_sum(s, red), width, eps) * gain : 1.0f;
-        for (uint32_t i = threadIdx.x; i < width; i += blockDim.x) hr[i] = to_act<TA>(xr[i] * f);
+        for (uint32_t i = threadIdx.x; i < width; i += blockDim.x) hr[i] = to_act<TA>(xr[i] * f * (w ? w[i] : 1.0f));
     }
 }
 
@@ -80,10 +81,7 @@ __global__ void __launch_bounds__(1024) norm_kernel(const float *x, uint32_t wid
             const uint32_t c = 4 * (threadIdx.x + i * blockDim.x);
             if (c >= width) continue;
             float4 o = mul4(v[i], f);
-            if (w) {
-                const float4 g = *reinterpret_cast<const float4 *>(w + c);
-                o = make_float4(o.x * g.x, o.y * g.y, o.z * g.z, o.w * g.w);
-            }
+            if (w) o = mul44(o, *reinterpret_cast<const float4 *>(w + c));
             store4<TA>(hr + c, o);
         }
     } else {
@@ -142,7 +140,7 @@ __global__ void __launch_bounds__(1024) side_finish_kernel(float *x, const float
     }
 }
 
-// x += mult * y / rms(y) * w, h = x; y is the sum of a token's `top` rows.
+// x += mult * y / rms(y) * w, h = x or x / rms(x) * next_w; y is the sum of a token's `top` rows.
 template <typename TA, int NV>
 __global__ void __launch_bounds__(1024) post_norm_kernel(PostNormArgs a) {
     __shared__ float red[33];
@@ -186,7 +184,17 @@ __global__ void __launch_bounds__(1024) post_norm_kernel(PostNormArgs a) {
             if (c >= a.width) continue;
             v[i].x += yv[i].x * f * wv[i].x, v[i].y += yv[i].y * f * wv[i].y, v[i].z += yv[i].z * f * wv[i].z, v[i].w += yv[i].w * f * wv[i].w;
             *reinterpret_cast<float4 *>(xr + c) = v[i];
-            if (hr) store4<TA>(hr + c, v[i]);
+            if (hr && !a.next_w) store4<TA>(hr + c, v[i]);
+        }
+        if (!hr || !a.next_w) return;
+        float s2 = 0.0f;
+#pragma unroll
+        for (int i = 0; i < NV; ++i) s2 += sq4(v[i]);  // (zero past the end)
+        const float f2 = inv_rms(block_sum(s2, red), a.width, a.eps);
+#pragma unroll
+        for (int i = 0; i < NV; ++i) {
+            const uint32_t c = 4 * (threadIdx.x + i * blockDim.x);
+            if (c < a.width) store4<TA>(hr + c, mul44(mul4(v[i], f2), *reinterpret_cast<const float4 *>(a.next_w + c)));
         }
     } else {
         auto sum = [&](uint32_t c) {
@@ -199,11 +207,16 @@ __global__ void __launch_bounds__(1024) post_norm_kernel(PostNormArgs a) {
             s += v * v;
         }
         const float f = inv_rms(block_sum(s, red), a.width, a.eps) * a.mult;
+        float s2 = 0.0f;
         for (uint32_t c = threadIdx.x; c < a.width; c += blockDim.x) {
             const float v = xr[c] + sum(c) * f * a.w[c];
             xr[c] = v;
-            if (hr) hr[c] = to_act<TA>(v);
+            s2 += v * v;
+            if (hr && !a.next_w) hr[c] = to_act<TA>(v);
         }
+        if (!hr || !a.next_w) return;
+        const float f2 = inv_rms(block_sum(s2, red), a.width, a.eps);
+        for (uint32_t c = threadIdx.x; c < a.width; c += blockDim.x) hr[c] = to_act<TA>(xr[c] * f2 * a.next_w[c]);
     }
 }
 
@@ -1096,14 +1109,15 @@ struct RowShape {
     }
 };
 template <typename TA>
-static void embed(const bf16 *table, uint32_t width, const uint32_t *tokens, uint32_t T, float *x, bool normed, float eps, float gain, void *h, uint32_t h_pitch, cudaStream_t st) {
-    const RowShape r(width, T);
-    launch_pdl(r.vec ? embed_kernel<TA, ROW_VECS> : embed_kernel<TA, 0>, T, r.threads, 0, st, table, width, tokens, x, normed, eps, gain, static_cast<TA *>(h), h_pitch);
-}
-void launch_embed(const bf16 *table, uint32_t width, const uint32_t *tokens, uint32_t T, float *x, bool normed, float eps, float gain, void *h, uint32_t h_pitch, bool f32,
+static void embed(const bf16 *table, uint32_t width, const uint32_t *tokens, uint32_t T, float *x, bool normed, float eps, float gain, const float *w, void *h, uint32_t h_pitch,
                   cudaStream_t st) {
-    if (f32) embed<float>(table, width, tokens, T, x, normed, eps, gain, h, h_pitch, st);
-    else embed<bf16>(table, width, tokens, T, x, normed, eps, gain, h, h_pitch, st);
+    const RowShape r(width, T);
+    launch_pdl(r.vec ? embed_kernel<TA, ROW_VECS> : embed_kernel<TA, 0>, T, r.threads, 0, st, table, width, tokens, x, normed, eps, gain, w, static_cast<TA *>(h), h_pitch);
+}
+void launch_embed(const bf16 *table, uint32_t width, const uint32_t *tokens, uint32_t T, float *x, bool normed, float eps, float gain, const float *w, void *h,
+                  uint32_t h_pitch, bool f32, cudaStream_t st) {
+    if (f32) embed<float>(table, width, tokens, T, x, normed, eps, gain, w, h, h_pitch, st);
+    else embed<bf16>(table, width, tokens, T, x, normed, eps, gain, w, h, h_pitch, st);
 }
 template <typename TA>
 static void norm(const float *x, uint32_t width, const uint32_t *rows, uint32_t n, float eps, float gain, const float *w, void *h, uint32_t h_pitch, cudaStream_t st) {

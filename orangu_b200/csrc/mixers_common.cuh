@@ -43,6 +43,7 @@ template <> __device__ __forceinline__ void store4<bf16>(bf16 *p, float4 v) {
 }
 __device__ __forceinline__ float sq4(float4 v) { return v.x * v.x + v.y * v.y + v.z * v.z + v.w * v.w; }
 __device__ __forceinline__ float4 mul4(float4 v, float f) { return make_float4(v.x * f, v.y * f, v.z * f, v.w * f); }
+__device__ __forceinline__ float4 mul44(float4 a, float4 b) { return make_float4(a.x * b.x, a.y * b.y, a.z * b.z, a.w * b.w); }
 
 // Value d of the rotated vector whose unrotated values are v[0..]; cs: this position's (cos, sin) row.
 __device__ __forceinline__ float rotated(const float *v, uint32_t d, const Rot &r, const float2 *cs) {
@@ -58,6 +59,27 @@ __device__ __forceinline__ float rotated(const float *v, uint32_t d, const Rot &
 
 // First position row t of a sequence sees.
 __device__ __forceinline__ uint32_t first_seen(uint32_t pos, uint32_t window) { return window && pos + 1 > window ? pos + 1 - window : 0u; }
+
+// Pages a group of rows of one sequence reads: the kept first ones, then those from the window's start on.  Counted from 0 to `n`.
+struct PageList {
+    uint32_t kept, gap, n;  // page i < kept is page i, the others page i + gap
+    __device__ __forceinline__ uint32_t operator[](uint32_t i) const { return i < kept ? i : i + gap; }
+};
+// Rows at positions [first, last]; the kept pages come in multiples of `unit`.
+__device__ __forceinline__ PageList page_list(uint32_t first, uint32_t last, uint32_t window, uint32_t keep, uint32_t unit) {
+    const uint32_t from = first_seen(first, window) / KV_PAGE, end = last / KV_PAGE + 1;
+    const uint32_t kept = (keep + KV_PAGE - 1) / KV_PAGE, whole = (kept + unit - 1) / unit * unit;
+    if (from <= whole && keep) return PageList{0, 0, end};  // nothing between them
+    return PageList{whole, from - whole, whole + end - from};
+}
+
+// softcap tanh(s / softcap) with c = 2 log2(e) / softcap times s's factor: exact to fp32 where it counts, absolutely.
+__device__ __forceinline__ float soft_cap(float s, float c, float cap) {
+    float e, r;
+    asm("ex2.approx.ftz.f32 %0, %1;" : "=f"(e) : "f"(s * c));
+    asm("rcp.approx.ftz.f32 %0, %1;" : "=f"(r) : "f"(e + 1.0f));
+    return fmaf(-2.0f * cap, r, cap);
+}
 
 __device__ __forceinline__ uint32_t smem_addr(const void *p) { return (uint32_t)__cvta_generic_to_shared(p); }
 __device__ __forceinline__ void cp16(uint32_t dst, const void *src, bool in) {  // 16 bytes, or zeros

@@ -25,7 +25,9 @@ __device__ __forceinline__ void eight(const float *p, float (&f)[8]) {
 // One warp: the `top` largest of z[0 .. n) (the first of equals), best first.  Sigmoid is monotonic, so logits decide.
 __device__ __forceinline__ void choose(const MoeArgs &a, uint32_t t, const float *z) {
     const uint32_t lane = threadIdx.x & 31;
+    const uint32_t p0 = t * (a.top + a.n_shared);
     uint32_t taken = 0;  // of this lane's logits z[lane + 32 j]: bit j
+    float first = 0.0f, sum = 0.0f;  // softmax: the largest logit, and the sum of exponentials below it
     for (uint32_t i = 0; i < a.top; ++i) {
         float best = -INFINITY;
         uint32_t at = 0xffffffffu;
@@ -39,10 +41,23 @@ __device__ __forceinline__ void choose(const MoeArgs &a, uint32_t t, const float
         }
         if (at % 32 == lane) taken |= 1u << (at / 32);
         if (lane == 0) {
-            const uint32_t p = t * a.top + i;
+            const uint32_t p = p0 + i;
             a.expert[p] = at;
-            a.score[p] = 1.0f / (1.0f + expf(-best));
+            if (i == 0) first = best;
+            sum += expf(best - first);
+            a.score[p] = a.softmax ? best : 1.0f / (1.0f + expf(-best));
             if (a.count) a.rank[p] = atomicAdd(a.count + at, 1u);
+        }
+    }
+    if (a.softmax && lane == 0)
+        for (uint32_t i = 0; i < a.top; ++i) a.score[p0 + i] = expf(a.score[p0 + i] - first) / sum;
+    for (uint32_t i = lane; i < a.n_shared; i += 32) {
+        const uint32_t p = p0 + a.top + i, e = a.n_expert + i;
+        a.expert[p] = e;
+        a.score[p] = 1.0f / (1.0f + expf(-z[a.n_expert]));
+        if (a.count) {
+            a.rank[p] = t;
+            if (t == 0) a.count[e] = a.T;
         }
     }
 }
@@ -50,12 +65,12 @@ __device__ __forceinline__ void choose(const MoeArgs &a, uint32_t t, const float
 // A CTA per token: logits, then the choice.
 template <typename TA>
 __global__ void __launch_bounds__(512) moe_route_dot_kernel(MoeArgs a) {
-    __shared__ float z[MOE_MAX_EXPERTS];
+    __shared__ float z[MOE_MAX_EXPERTS + 1];
     pdl_release();
     pdl_wait();
     const uint32_t t = blockIdx.x, warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
     const TA *x = static_cast<const TA *>(a.x) + (uint64_t)t * a.x_pitch;
-    for (uint32_t e = warp; e < a.n_expert; e += blockDim.x / 32) {
+    for (uint32_t e = warp; e < a.n_expert + (a.n_shared > 0); e += blockDim.x / 32) {
         const bf16 *w = a.w + (uint64_t)e * a.x_pitch;
         float s = 0.0f;
 #pragma unroll 4
@@ -87,33 +102,33 @@ __global__ void __launch_bounds__(256) moe_gather_kernel(MoeArgs a) {
     __shared__ uint32_t first[MOE_MAX_EXPERTS], tile0[MOE_MAX_EXPERTS];
     pdl_release();
     pdl_wait();
-    const uint32_t warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
+    const uint32_t warp = threadIdx.x >> 5, lane = threadIdx.x & 31, n_all = a.n_expert + a.n_shared, per = a.top + a.n_shared;
     if (warp == 0) {
         uint32_t rows = 0, tiles = 0;
-        for (uint32_t e0 = 0; e0 < a.n_expert; e0 += 32) {
-            const uint32_t e = e0 + lane, n = e < a.n_expert ? a.count[e] : 0, k = (n + a.tile_rows - 1) / a.tile_rows;
+        for (uint32_t e0 = 0; e0 < n_all; e0 += 32) {
+            const uint32_t e = e0 + lane, n = e < n_all ? a.count[e] : 0, k = (n + a.tile_rows - 1) / a.tile_rows;
             uint32_t rs = n, ts = k;
 #pragma unroll
             for (int o = 1; o < 32; o <<= 1) {
                 const uint32_t ru = __shfl_up_sync(0xffffffffu, rs, o), tu = __shfl_up_sync(0xffffffffu, ts, o);
                 if (lane >= o) rs += ru, ts += tu;
             }
-            if (e < a.n_expert) first[e] = rows + rs - n, tile0[e] = tiles + ts - k;
+            if (e < n_all) first[e] = rows + rs - n, tile0[e] = tiles + ts - k;
             rows += __shfl_sync(0xffffffffu, rs, 31), tiles += __shfl_sync(0xffffffffu, ts, 31);
         }
         if (blockIdx.x == 0 && lane == 0) *a.n_tiles = tiles;
     }
     __syncthreads();
     if (blockIdx.x == 0)
-        for (uint32_t e = threadIdx.x; e < a.n_expert; e += blockDim.x) {
+        for (uint32_t e = threadIdx.x; e < n_all; e += blockDim.x) {
             const uint32_t n = a.count[e];
             for (uint32_t r = 0, k = tile0[e]; r < n; r += a.tile_rows, ++k) a.tiles[k] = LinTile{e, first[e] + r, min(a.tile_rows, n - r)};
         }
     const uint32_t p = blockIdx.x * 8 + warp;
-    if (p >= a.T * a.top) return;
+    if (p >= a.T * per) return;
     const uint32_t row = first[a.expert[p]] + a.rank[p];
     if (lane == 0) a.row[p] = row, a.row_score[row] = a.score[p];
-    const uint4 *src = reinterpret_cast<const uint4 *>(static_cast<const TA *>(a.x) + (uint64_t)(p / a.top) * a.x_pitch);
+    const uint4 *src = reinterpret_cast<const uint4 *>(static_cast<const TA *>(a.x) + (uint64_t)(p / per) * a.x_pitch);
     uint4 *dst = reinterpret_cast<uint4 *>(static_cast<TA *>(a.gathered) + (uint64_t)row * a.x_pitch);
     const uint32_t n = a.x_pitch * (uint32_t)sizeof(TA) / 16;
 #pragma unroll 4
@@ -125,7 +140,7 @@ uint32_t route(const MoeArgs &a, cudaStream_t st) {
     if (a.logits) launch_pdl(moe_route_kernel, (a.T + 7) / 8, 256, 0, st, a);
     else launch_pdl(moe_route_dot_kernel<TA>, a.T, 512, 0, st, a);
     if (!a.count) return 1;
-    launch_pdl(moe_gather_kernel<TA>, (a.T * a.top + 7) / 8, 256, 0, st, a);
+    launch_pdl(moe_gather_kernel<TA>, (a.T * (a.top + a.n_shared) + 7) / 8, 256, 0, st, a);
     return 2;
 }
 

@@ -1,5 +1,5 @@
 """Models given as a list of layers (``ob_layered_desc``), each layer with its own token mixer.  A design's reader (fenipel.py,
-nenodra.py) turns its configuration and tensors into blocks; this class owns the description and the handle."""
+nenodra.py, senuvik.py) turns its configuration and tensors into blocks; this class owns the description and the handle."""
 from __future__ import annotations
 
 import ctypes as C
@@ -29,6 +29,11 @@ class Describer:
         arr = (capi.MatrixDesc * len(each))(*each)
         self.keep.append(arr)
         return arr
+
+    def doubles(self, v) -> int:
+        a = np.ascontiguousarray(v, np.float64)
+        self.keep.append(a)
+        return a.ctypes.data
 
     def vector(self, v) -> int:
         a = np.ascontiguousarray(v, np.float32)
@@ -82,6 +87,7 @@ class LayeredModel(DeviceModel):
     def __init__(self, backend, desc: capi.LayeredDesc, blocks):
         self.backend, self._lib = backend, backend._lib
         self._mixers = [b.mixer for b in blocks]
+        self._states = [b.mixer2 if b.mixer2.kind and b.mixer.kind == capi.MIXER_ATTENTION else b.mixer for b in blocks]
         arr = (capi.BlockDesc * len(blocks))(*blocks)
         desc.layers = arr
         self._h = C.c_void_p()
@@ -96,5 +102,5 @@ class LayeredModel(DeviceModel):
         return m.kv_rank, m.rot_dim
 
     def state_shape(self, layer: int):
-        m = self._mixers[layer]
+        m = self._states[layer]
         return m.n_head, m.dim, m.vdim

@@ -7,9 +7,10 @@ import os
 from .fenipel import FenipelModel
 from .model import LlamaModel
 from .nenodra import NenodraModel
+from .senuvik import SenuvikModel
 
 GGUF_ARCHITECTURES = {a: LlamaModel for a in ("llama", "mistral", "qwen2", "qwen3", "qwen3vl")}
-FOLDER_ARCHITECTURES = {m.ARCHITECTURE: m for m in (FenipelModel, NenodraModel)}
+FOLDER_ARCHITECTURES = {m.ARCHITECTURE: m for m in (FenipelModel, NenodraModel, SenuvikModel)}
 
 
 def model_class(path: str):
