@@ -71,6 +71,10 @@ def parse_args():
                     "(1b, 8b; random weights) beside Fenipel at the same widths")
     ap.add_argument("--nenodra-layers", type=int, default=8, help="layers of both models in that comparison")
     ap.add_argument("--nenodra-only", action="store_true", help="leave Fenipel out")
+    ap.add_argument("--senuvik", default="", metavar="SIZE[,SIZE]", help="instead of the workload above: prefill and decode of Senuvik at these sizes "
+                    "(1b, 8b: widths) beside Nenodra at the same widths; one JSON line of its own")
+    ap.add_argument("--senuvik-layers", type=int, default=8, help="layers of both models in that comparison")
+    ap.add_argument("--senuvik-only", action="store_true", help="leave Nenodra out")
     return ap.parse_args()
 
 
@@ -419,6 +423,63 @@ def nenodra_model(size: str, n_layer: int):
     return {"architecture": "Nenodra", "vocab": V, "width": E, "norm": {"eps": 1e-6}, "residual_mult": 1.0, "logit_scale": 1.0, "layers": layers}, t
 
 
+SENUVIK_SIZES = {  # Nenodra's widths, heads and experts; of four layers one attends within a window (dense), two are parallel, one is a state space
+    "1b": {"width": 2048, "ff": 8192, "vocab": 32768, "experts": 16, "top": 2, "expert_ff": 1024, "window": 1024, "keep": 4,
+           "attention": {"heads": 16, "kv_heads": 4, "dim": 128, "vdim": 128}, "space": {"heads": 64, "vdim": 64, "state": 128, "groups": 4, "norm_groups": 4, "conv": 4},
+           "time": {"heads": 32, "dim": 64}, "rank": 64},
+    "8b": {"width": 4096, "ff": 14336, "vocab": 32768, "experts": 16, "top": 2, "expert_ff": 2048, "window": 1024, "keep": 4,
+           "attention": {"heads": 32, "kv_heads": 8, "dim": 128, "vdim": 128}, "space": {"heads": 128, "vdim": 64, "state": 128, "groups": 8, "norm_groups": 8, "conv": 4},
+           "time": {"heads": 64, "dim": 64}, "rank": 128},
+}
+
+
+def senuvik_model(size: str, n_layer: int):
+    """Configuration and random bfloat16 tensors (bits)."""
+    import numpy as np
+    from orangu_b200.safetensors import to_bf16
+
+    z = SENUVIK_SIZES[size]
+    E, V = z["width"], z["vocab"]
+    lin, const = random_matrices(), lambda v, *n: to_bf16(np.full(n, v, np.float32))
+    layers, t = [], {"embed": lin(V, E, 4.0), "head": lin(V, E), "final.norm": const(1, E)}  # (tokens differ enough to choose different experts)
+    a = z["attention"]
+    H, G, d, v = a["heads"], a["kv_heads"], a["dim"], a["vdim"]
+    for n in range(n_layer):
+        kind = ("attention", "parallel", "mamba2", "parallel")[n % 4]
+        at = f"l{n}.mix."
+        t.update({f"l{n}.{x}": const(1, E) for x in ("norm1", "norm2", "norm1b", "norm2b", "ls1", "ls2")})
+        if kind == "attention":
+            mixer = dict(a, mask={"size": z["window"], "keep_first": z["keep"]}, rot={"base": 10000.0, "dims": d, "scaling": {"factor": 4.0}}, scale=d ** -0.5)
+            t.update({at + "q": lin(H * d, E), at + "q.b": const(0.1, H * d), at + "q.norm": const(1, H * d), at + "k": lin(G * d, E), at + "k.b": const(0.1, G * d),
+                      at + "k.norm": const(1, G * d), at + "v": lin(G * v, E), at + "v.b": const(0.1, G * v), at + "sink": const(0.5, H), at + "o": lin(E, H * v)})
+        elif kind == "mamba2":
+            mixer = s = dict(z["space"])
+            inner = s["heads"] * s["vdim"]
+            ch = inner + 2 * s["groups"] * s["state"]
+            t.update({at + "in": lin(inner + ch + s["heads"], E), at + "conv": lin(ch, s["conv"]), at + "conv.b": const(0.1, ch), at + "dt_bias": const(-2, s["heads"]),
+                      at + "A_log": const(0.5, s["heads"]), at + "D": const(1, s["heads"]), at + "norm": const(1, inner), at + "o": lin(E, inner)})
+        else:
+            r, m = z["time"], z["time"]["heads"] * z["time"]["dim"]
+            mixer = {"left": dict(a, rot={"base": 1e6, "dims": d, "scaling": {"factor": 4.0, "original": 1024, "fast": 32.0, "slow": 1.0}}, scale=d ** -0.5, softcap=50.0),
+                     "right": dict(r), "left_scale": 1.0, "right_scale": 1.0}
+            t.update({at + "left.q": lin(H * d, E), at + "left.k": lin(G * d, E), at + "left.v": lin(G * v, E), at + "left.g": lin(H, E), at + "left.o": lin(E, H * v)})
+            t.update({at + "right." + c: lin(m, E) for c in "rkvg"})
+            t.update({at + "right.mu." + c: const(0.5, E) for c in "rkvgw"})
+            t.update({at + "right.w1": lin(z["rank"], E), at + "right.w2": lin(m, z["rank"]), at + "right.w0": const(-3, m), at + "right.u": const(0.5, r["heads"], r["dim"]),
+                      at + "right.norm": const(1, m), at + "right.o": lin(E, m)})
+        if n % 4 == 0:
+            mlp = {"kind": "dense", "ff": z["ff"]}
+            t.update({f"l{n}.mlp.gate": lin(z["ff"], E), f"l{n}.mlp.up": lin(z["ff"], E), f"l{n}.mlp.down": lin(E, z["ff"])})
+        else:
+            X, ff = z["experts"], z["expert_ff"]
+            mlp = {"kind": "moe", "router": {"experts": X, "top": z["top"]}, "expert": {"ff": ff}, "shared": {"ff": ff}}
+            t.update({f"l{n}.mlp.router": lin(X, E), f"l{n}.mlp.shared.sg": lin(1, E)})
+            for e in [f"e{e}." for e in range(X)] + ["shared."]:
+                t.update({f"l{n}.mlp.{e}gate": lin(ff, E), f"l{n}.mlp.{e}up": lin(ff, E), f"l{n}.mlp.{e}down": lin(E, ff)})
+        layers.append({"type": kind, "mixer": mixer, "mlp": mlp})
+    return {"architecture": "Senuvik", "vocab": V, "width": E, "norm": {"eps": 1e-6}, "layers": layers}, t
+
+
 def time_model(be, model, vocab: int, weight_bytes, cache_bytes_per_token: float, flops_per_token: float, steps: int, warmup: int, prompt: int = 4096):
     """Prefill of one prompt and greedy decode loops at batch 1, 8 and 64 (device time, CUDA events; weights exceed L2).
     weight_bytes: read per decoded step, a number or a function of the batch.  cache_bytes_per_token: cache and state traffic of
@@ -494,6 +555,55 @@ def time_nenodra(be, size: str, L: int, steps: int, warmup: int):
     return result
 
 
+def time_senuvik(be, size: str, L: int, steps: int, warmup: int):
+    import orangu_b200
+
+    cfg, t = senuvik_model(size, L)
+    z, prompt = SENUVIK_SIZES[size], 4096
+    expert = 3 * z["width"] * z["expert_ff"]
+    n_moe = sum(x["mlp"]["kind"] == "moe" for x in cfg["layers"])
+    n = sum(a.size for k, a in t.items() if not k.endswith("embed"))
+    every = n - n_moe * z["experts"] * expert
+    a, s, r = z["attention"], z["space"], z["time"]
+    cache, flops = 0, 2 * (every + n_moe * z["top"] * expert)
+    for layer in cfg["layers"]:
+        if layer["type"] == "mamba2":
+            state = s["heads"] * s["state"] * s["vdim"]
+            cache, flops = cache + 8 * state, flops + 6 * state
+            continue
+        seen = min(z["window"], prompt) if layer["type"] == "attention" else prompt
+        cache += 2 * seen * a["kv_heads"] * (a["dim"] + a["vdim"])
+        flops += 2 * (seen if layer["type"] == "attention" else prompt // 2) * a["heads"] * (a["dim"] + a["vdim"])
+        if layer["type"] == "parallel":
+            state = r["heads"] * r["dim"] ** 2
+            cache, flops = cache + 8 * state, flops + 6 * state
+    # experts that a step reads when tokens choose independently and evenly
+    weights = lambda batch: 2 * (every + n_moe * expert * z["experts"] * (1 - (1 - z["top"] / z["experts"]) ** batch))
+    m = orangu_b200.SenuvikModel(be, cfg, t, max_seq_len=8192, max_batch_tokens=prompt, kv_pool_tokens=64 * 4480, state_slots=64)
+    result = dict(time_model(be, m, z["vocab"], weights, cache, flops, steps, warmup), parameters=n)
+    m.close()
+    return result
+
+
+def run_senuvik(args):
+    """--senuvik: one JSON line with both models at every size."""
+    import orangu_b200
+
+    be = orangu_b200.CudaBackend.init(0)
+    steps, warmup, L = args.steps, max(3, args.warmup), args.senuvik_layers
+    result = {"bench": "senuvik", "data": "synthetic", "dtype": "bf16", "layers": L, "steps": steps, "warmup": warmup, "sizes": {}}
+    clocks = ClockSampler(0)
+    clocks.start()
+    for size in args.senuvik.split(","):
+        entry = {"senuvik": time_senuvik(be, size, L, steps, warmup)}
+        if not args.senuvik_only:
+            entry["nenodra"] = time_nenodra(be, size, L, steps, warmup)
+        result["sizes"][size] = entry
+    result["clocks"] = clocks.stop()
+    be.close()
+    print(json.dumps(result))
+
+
 def run_nenodra(args):
     """--nenodra: one JSON line with both models at every size."""
     import orangu_b200
@@ -554,6 +664,9 @@ def main():
         return
     if args.fenipel:
         run_fenipel(args)
+        return
+    if args.senuvik:
+        run_senuvik(args)
         return
     if args.nenodra:
         run_nenodra(args)

@@ -10,6 +10,7 @@ from .backend import CudaBackend, QuantMatrix, MatmulOp  # noqa: F401
 from .model import LlamaModel, KvCache  # noqa: F401
 from .fenipel import FenipelModel  # noqa: F401
 from .nenodra import NenodraModel  # noqa: F401
+from .senuvik import SenuvikModel  # noqa: F401
 from .registry import load_model  # noqa: F401
 from .scheduler import SlotPool, SlotGuard  # noqa: F401
 
