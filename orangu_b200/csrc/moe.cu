@@ -64,7 +64,7 @@ __device__ __forceinline__ void choose(const MoeArgs &a, uint32_t t, const float
 
 // A CTA per token: logits, then the choice.
 template <typename TA>
-__global__ void __launch_bounds__(512) moe_route_dot_kernel(MoeArgs a) {
+__global__ void __launch_bounds__(1024) moe_route_dot_kernel(MoeArgs a) {
     __shared__ float z[MOE_MAX_EXPERTS + 1];
     pdl_release();
     pdl_wait();
@@ -138,7 +138,7 @@ __global__ void __launch_bounds__(256) moe_gather_kernel(MoeArgs a) {
 template <typename TA>
 uint32_t route(const MoeArgs &a, cudaStream_t st) {
     if (a.logits) launch_pdl(moe_route_kernel, (a.T + 7) / 8, 256, 0, st, a);
-    else launch_pdl(moe_route_dot_kernel<TA>, a.T, 512, 0, st, a);
+    else launch_pdl(moe_route_dot_kernel<TA>, a.T, a.n_expert + (a.n_shared > 0) > 16 ? 1024 : 512, 0, st, a);
     if (!a.count) return 1;
     launch_pdl(moe_gather_kernel<TA>, (a.T * (a.top + a.n_shared) + 7) / 8, 256, 0, st, a);
     return 2;

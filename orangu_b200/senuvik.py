@@ -58,7 +58,7 @@ def _rotation(d: Describer, m: capi.MixerDesc, freqs: np.ndarray, gain: float = 
 def _window_attention(d: Describer, t, at: str, mx: dict, width: int) -> capi.MixerDesc:
     m = _attention(d, t, at, mx, width)
     H, G, dim, vdim = m.n_head, m.n_kv_head, m.dim, m.vdim
-    m.window, m.keep_first, m.rot_interleaved = mx["mask"]["size"], mx["mask"]["keep_first"], 1
+    m.window, m.keep_first, m.rot_interleaved = mx["mask"]["size"], mx["mask"].get("keep_first", 0), 1
     _rotation(d, m, linear_frequencies(mx["rot"]))
     m.qk_norm_whole = 1
     m.q_bias, m.q_norm = d.vector(t.f32(at + "q.b", (H * dim,))), d.vector(t.f32(at + "q.norm", (H * dim,)))
