@@ -3,6 +3,9 @@
 // With two maps per head (differential attention) both maps have queries and keys of their own and share the values; the head's
 // output is map 1 - map_weight * map 2, brought to unit root mean square and scaled.  An elementwise sigmoid gate may follow.
 //
+// With one map, the first positions may stay visible beyond the window, scores may be capped, a sink per head may enter the softmax's
+// denominator, a gate may scale whole heads, and keys and values may be another layer's.
+//
 //   attention_prep_kernel    norms and rotates queries and keys, appends keys and values to the cache
 //   attention_step_kernel    decoded tokens and short portions: every warp takes pages of its own, a cluster of CTAs shares the
 //                            keys of one tile and adds up over distributed shared memory
