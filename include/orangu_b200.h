@@ -34,7 +34,7 @@ extern "C" {
  * 5: the layered descriptions gained softmax attention over cached keys and values, sequential blocks and mixtures of experts.
  * 6: they gained state-space and time-mixing layers, two mixers in a block, normed inputs, and kept tokens, sinks, soft caps, shared
  *    keys and values of attention. */
-#define OB_ABI_VERSION 6u
+#define OB_ABI_VERSION 7u
 
 typedef enum ob_status {
     OB_OK = 0,
@@ -254,9 +254,10 @@ typedef struct ob_model_desc {
 
 /* ------------------------------------------------- models given as a list of layers
  * Designs whose layers are not all alike: every layer names its token mixer and its feed-forward and carries their sizes,
- * constants and tensors.  Two kinds of block: parallel, x += mixer(h) + ff(h) with h = x / rms(x) * norm_gain; and sequential with
+ * constants and tensors.  Three kinds of block: parallel, x += mixer(h) + ff(h) with h = x / rms(x) * norm_gain; sequential with
  * normed outputs (post_norm1 given), x += residual_mult * m / rms(m) * post_norm1 with m = mixer(h), then the same with the
- * feed-forward and post_norm2; h is x, or (pre_norm1, pre_norm2 given) x / rms(x) * pre_norm.  No counterpart in the reference.  The result is an ob_model like any other: caches, batching, sampling,
+ * feed-forward and post_norm2; h is x, or (pre_norm1, pre_norm2 given) x / rms(x) * pre_norm; and sequential with plain sums (only
+ * pre_norm1 given), x += residual_mult * mixer(h), then the same with the feed-forward.  No counterpart in the reference.  The result is an ob_model like any other: caches, batching, sampling,
  * captured decode graphs and the slot pool are the same calls.  Matrices are bfloat16, out_dim rows of in_dim; vectors f32. */
 #define OB_TYPE_BF16 30u /* ob_matrix_desc.ggml_type of these matrices */
 #define OB_MIXER_LATENT_ATTENTION 1u
@@ -268,12 +269,15 @@ typedef struct ob_model_desc {
 #define OB_FF_RELU2 1u       /* max(up, 0)^2 */
 #define OB_FF_EXPERTS 2u     /* n_expert_used of n_expert silu(gate) * up feed-forwards, weighted as router_softmax says */
 #define OB_FF_GELU_GLU 3u    /* gelu(gate) * up, the tanh form */
+#define OB_ROUTER_SIGMOID 0u     /* router_softmax: a chosen expert reads the input times the sigmoid of its logit */
+#define OB_ROUTER_SOFTMAX 1u     /* outputs are weighted by the softmax over the chosen logits */
+#define OB_ROUTER_SOFTMAX_ALL 2u /* outputs are weighted by the softmax over all logits, times router_scale */
 
 typedef struct ob_mixer_desc {
     uint32_t kind;            /* OB_MIXER_* */
     uint32_t n_head, dim;     /* query/key dimensions per head (latent attention: the unrotated ones) */
     uint32_t vdim;            /* value dimensions per head */
-    uint32_t rot_dim;         /* latent attention: rotated query/key dimensions per head, in addition to dim */
+    uint32_t rot_dim;         /* latent attention: rotated query/key dimensions per head, in addition to dim; may be 0 */
     uint32_t kv_rank;         /* latent attention: size of the cached latent */
     uint32_t window;          /* attention: a position sees itself and window - 1 before it (and keep_first); 0 = all before it */
     uint32_t rot_dims;        /* entries that rotate, from the first: of q and k (retention, attention), of the rot_dim part (latent attention) */
@@ -285,8 +289,8 @@ typedef struct ob_mixer_desc {
                                * attention [n_head*n_map*dim], head by head */
     ob_matrix_desc wk, wv;    /* retention [n_head*dim], [n_head*vdim]; attention [n_kv_head*n_map*dim], [n_kv_head*vdim] (no data:
                                * the values are the keys as projected, before norm and rotation; n_map 1, vdim = dim) */
-    ob_matrix_desc w_gate;    /* retention [n_head*vdim] (silu of it scales the normed output); latent attention [n_head] (sigmoid of it scales a head);
-                               * attention [n_head*vdim] or [n_head] (sigmoid of it scales the output or a head; no data: no gate);
+    ob_matrix_desc w_gate;    /* retention [n_head*vdim] (silu of it scales the normed output);
+                               * attention and latent attention [n_head*vdim] or [n_head] (sigmoid of it scales the output or a head; no data: no gate);
                                * time mixing [n_head*dim] (silu of it scales the normed output) */
     ob_matrix_desc w_dkv;     /* latent attention [kv_rank+rot_dim]: latent, then the rotated key part all heads share */
     const float *kv_norm;     /* latent attention [kv_rank]: RMS-norm weight of the latent */
@@ -303,7 +307,7 @@ typedef struct ob_mixer_desc {
     uint32_t keep_first;      /* the first tokens of a sequence that stay visible beyond the window */
     uint32_t kv_layer;        /* 1 + an earlier layer whose cached keys and values are used (wk, wv without data); 0: own ones */
     float softcap;            /* > 0: score = softcap * tanh(score / softcap) */
-    const float *sink;        /* [n_head]: exp(sink) is added to the softmax denominator; NULL: none */
+    const float *sink;        /* (also latent attention) [n_head]: exp(sink) is added to the softmax denominator; NULL: none */
     /* attention: frequencies of the pairs instead of the powers of rot_base, and a factor of cos and sin (0: 1) */
     const double *rot_freqs;  /* [rot_dims/2] or NULL */
     float rot_gain;
@@ -334,12 +338,18 @@ typedef struct ob_block_desc {
     uint32_t n_expert, n_expert_used; /* OB_FF_EXPERTS: the n_expert_used largest of w_router x are chosen */
     ob_matrix_desc w_router;  /* [n_expert] */
     const ob_matrix_desc *expert_gate, *expert_up, *expert_down; /* [n_expert] matrices each */
-    uint32_t router_softmax;  /* 0: a chosen expert reads the input times sigmoid of its logit; 1: outputs are weighted by the softmax over the chosen logits */
-    uint32_t shared_ff;       /* > 0: size of a further expert that every token uses; its output is scaled by sigmoid(w_shared_scale x) (router_softmax 1 only) */
+    uint32_t router_softmax;  /* OB_ROUTER_* */
+    uint32_t shared_ff;       /* > 0: size of a further expert that every token uses; its output is scaled by sigmoid(w_shared_scale x) (not OB_ROUTER_SIGMOID) */
     ob_matrix_desc shared_gate, shared_up, shared_down, w_shared_scale; /* the last [1] */
     const float *pre_norm1, *pre_norm2; /* [n_embd] sequential blocks: factors of the normed inputs; NULL: a sublayer reads x itself */
     ob_mixer_desc mixer2;     /* sequential blocks: a second mixer beside the first, both read the same input; kind 0: none */
     float mixer_scale, mixer2_scale;    /* with mixer2: factors of the two mixers' outputs */
+    float router_scale;       /* OB_ROUTER_SOFTMAX_ALL */
+    uint32_t n_expert_group, n_group_used; /* experts in n_expert_group equal groups of neighbours, of which only the n_group_used with the largest logits
+                               * can be chosen from; 0: no groups */
+    const float *conv1, *conv2; /* with conv_taps: [n_embd][conv_taps] of the mixer's and of the feed-forward's input */
+    const float *depth;       /* layer i, plain sums: [i + 2] factors of the embeddings and of the results of layers 0 .. i; their sum is what goes on.
+                               * NULL: the layer's result goes on */
 } ob_block_desc;
 
 typedef struct ob_layered_desc {
@@ -356,6 +366,9 @@ typedef struct ob_layered_desc {
     const ob_block_desc *layers;
     float residual_mult;       /* sequential blocks */
     const float *final_norm;   /* [n_embd] factors of the last norm, beside final_gain; NULL: none.  All blocks are of one kind */
+    /* plain sums: */
+    uint32_t norm_groups;      /* equal parts of the residual that are normed each by itself, in the last norm too; 0 = 1 */
+    uint32_t conv_taps;        /* > 0: a normed input n becomes n + causal convolution of n over time, a channel by itself (the last tap meets the current token) */
 } ob_layered_desc;
 
 /* ------------------------------------------------- GGUF files
@@ -421,7 +434,8 @@ int ob_kv_truncate(ob_kv *kv, uint32_t new_len);
 /* Test hook: reads positions [pos0, pos0+n) of one layer back as f32 [n][n_head_kv*head_dim]; a latent-attention layer gives
  * [n][kv_rank] in k_out and the rotated key part [n][rot_dim] in v_out. */
 int ob_kv_read(ob_kv *kv, uint32_t layer, uint32_t pos0, uint32_t n, float *k_out, float *v_out);
-/* Test hook: the recurrent state of one layer, f32 [n_head][dim][vdim]. */
+/* Test hook: the recurrent state of one layer, f32 [n_head][dim][vdim]; of a layer without one whose inputs are convolved, the last
+ * conv_taps - 1 normed inputs of its sublayers, the oldest first, [1 or 2][conv_taps - 1][n_embd]. */
 int ob_state_read(ob_kv *kv, uint32_t layer, float *out);
 /* KvCache::copy_prefix_from (E/kv_cache.rs:1079-1100): makes dst (empty) hold src's first n positions, by a
  * device-side copy of the pages.  Both caches belong to the same model.  With recurrent layers n must be all of src. */

@@ -9,6 +9,7 @@ from .capi import OranguError, lib_path, load  # noqa: F401
 from .backend import CudaBackend, QuantMatrix, MatmulOp  # noqa: F401
 from .model import LlamaModel, KvCache  # noqa: F401
 from .fenipel import FenipelModel  # noqa: F401
+from .filorax import FiloraxModel  # noqa: F401
 from .nenodra import NenodraModel  # noqa: F401
 from .senuvik import SenuvikModel  # noqa: F401
 from .registry import load_model  # noqa: F401

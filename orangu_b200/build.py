@@ -22,10 +22,10 @@ SYNTH_LIB = os.path.join(LIBDIR, "libob_synth.so")
 
 LAYERED_LIB = os.path.join(LIBDIR, "liborangu_b200_layered.so")  # the same library without the quantized kernels
 
-CORE_SOURCES = ["api.cu", "model.cu", "tp.cu", "noalloc.cu", "gguf.cu", "sched.cu", "glue.cu", "linear.cu", "mixers.cu", "gqa.cu", "gqa_tc5.cu", "moe.cu", "recurrence.cu", "layered.cu"]
+CORE_SOURCES = ["api.cu", "model.cu", "tp.cu", "noalloc.cu", "gguf.cu", "sched.cu", "glue.cu", "linear.cu", "mixers.cu", "gqa.cu", "gqa_tc5.cu", "moe.cu", "recurrence.cu", "residual.cu", "layered.cu"]
 QUANTIZED_SOURCES = ["formats.cu", "act_quant.cu", "gemv.cu", "attention.cu", "stream_gemv.cu", "layer_stream.cu", "gemm_mma.cu", "gemm_tc5.cu", "q5k.cu"]
 CU_SOURCES = CORE_SOURCES + QUANTIZED_SOURCES
-FMA_SOURCES = {"linear.cu", "mixers.cu", "gqa.cu", "gqa_tc5.cu", "moe.cu", "recurrence.cu", "layered.cu"}  # no CPU arithmetic to reproduce: the compiler may fuse
+FMA_SOURCES = {"linear.cu", "mixers.cu", "gqa.cu", "gqa_tc5.cu", "moe.cu", "recurrence.cu", "residual.cu", "layered.cu"}  # no CPU arithmetic to reproduce: the compiler may fuse
 NVCC_FLAGS = [
     "-gencode", "arch=compute_100a,code=sm_100a", "-lineinfo", "-O3", "-std=c++17",
     # The reproduced arithmetic never fuses a*b+c; FMAs are written out where wanted.

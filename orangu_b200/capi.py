@@ -40,6 +40,7 @@ class ModelDesc(C.Structure):
 TYPE_BF16 = 30
 MIXER_LATENT_ATTENTION, MIXER_RETENTION, MIXER_ATTENTION, MIXER_STATE_SPACE, MIXER_TIME_MIXING = 1, 2, 3, 4, 5
 FF_CLAMPED_GLU, FF_RELU2, FF_EXPERTS, FF_GELU_GLU = 0, 1, 2, 3
+ROUTER_SIGMOID, ROUTER_SOFTMAX, ROUTER_SOFTMAX_ALL = 0, 1, 2
 
 
 class MixerDesc(C.Structure):
@@ -61,13 +62,15 @@ class BlockDesc(C.Structure):
         (n, C.c_void_p) for n in ("post_norm1", "post_norm2")] + [(n, C.c_uint32) for n in ("ff_kind", "n_expert", "n_expert_used")] + [
         ("w_router", MatrixDesc)] + [(n, C.POINTER(MatrixDesc)) for n in ("expert_gate", "expert_up", "expert_down")] + [
         (n, C.c_uint32) for n in ("router_softmax", "shared_ff")] + [(n, MatrixDesc) for n in ("shared_gate", "shared_up", "shared_down", "w_shared_scale")] + [
-        (n, C.c_void_p) for n in ("pre_norm1", "pre_norm2")] + [("mixer2", MixerDesc), ("mixer_scale", C.c_float), ("mixer2_scale", C.c_float)]
+        (n, C.c_void_p) for n in ("pre_norm1", "pre_norm2")] + [("mixer2", MixerDesc), ("mixer_scale", C.c_float), ("mixer2_scale", C.c_float)] + [
+        ("router_scale", C.c_float), ("n_expert_group", C.c_uint32), ("n_group_used", C.c_uint32)] + [(n, C.c_void_p) for n in ("conv1", "conv2", "depth")]
 
 
 class LayeredDesc(C.Structure):
     _fields_ = [(n, C.c_uint32) for n in ("n_vocab", "n_embd", "n_layer", "side_dim")] + [("rms_eps", C.c_float), ("final_gain", C.c_float)] + [
         (n, C.c_uint32) for n in ("compute_f32", "max_seq_len", "max_batch_tokens")] + [("kv_pool_tokens", C.c_uint64), ("n_state_slots", C.c_uint32)] + [
-        (n, MatrixDesc) for n in ("token_embd", "side_embd", "output")] + [("layers", C.POINTER(BlockDesc)), ("residual_mult", C.c_float), ("final_norm", C.c_void_p)]
+        (n, MatrixDesc) for n in ("token_embd", "side_embd", "output")] + [("layers", C.POINTER(BlockDesc)), ("residual_mult", C.c_float), ("final_norm", C.c_void_p)] + [
+        (n, C.c_uint32) for n in ("norm_groups", "conv_taps")]
 
 
 class MatmulOpC(C.Structure):

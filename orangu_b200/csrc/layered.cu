@@ -9,14 +9,15 @@
 //           retention: rotate, recurrence, norm with gate
 //   out     x += [W_o | W_down] [mixer | ff]
 //   side    gate (gelu, token entry), proj, then norm + residual + the next layer's norm in one kernel
-// A sequential block reads the residual itself (h: its activation form) or its norm, and norms what it adds:
+// A sequential block reads the residual itself (h: its activation form) or its norm, and norms what it adds or adds it as it is:
 //   in      mixer projections <- h
 //   mixer   attention: prep, attention with the heads' epilogue
 //           state space: convolution and steps, recurrence, gate and norm
 //           time mixing: token shift, projections of the mixes, recurrence, norm and gate
 //           a second mixer leaves its output beside the first one's, so that one product adds up both
 //   out     product, bias as epilogue
-//   post    x += mult norm(out), h = x or norm(x) in one kernel
+//   post    x += mult norm(out), h = x or norm(x) in one kernel; plain sums: x += mult out, average over depth, grouped norm and
+//           convolution over time in one kernel (residual.cu)
 //   ff      dense: up (activation as epilogue), down; experts: routing, grouped gate/up and down (moe.cu); post as above
 #include <math.h>
 #include <string.h>
@@ -52,7 +53,7 @@ struct MixerPlan {
     // attention
     float *q_norm = nullptr, *k_norm = nullptr, *sink = nullptr;
     uint32_t vdim_p = 0, row = 0, gate0 = 0;  // row: elements of a cache row per key/value head
-    bool has_v = false, has_gate = false, head_gate = false, own_kv = true;
+    bool has_v = false, has_gate = false, head_gate = false, own_kv = true;  // gates: of every output, or of whole heads
     // latent attention
     Dense uk, uv;        // per head [kv_rank <- dim], [vdim <- kv_rank]
     Dense expand;        // latent -> keys [H][dim_k], then (from row ex_v0) values [H][vdim_k]; no rows: prompts attend in the latent space too
@@ -81,10 +82,13 @@ struct LayerPlan : MixerPlan {
     Dense out, side_gate, side_proj;
     bool sequential = false;
     float *out_bias = nullptr, *pre1 = nullptr, *pre2 = nullptr, *post1 = nullptr, *post2 = nullptr;
+    // plain sums: convolution of the two sublayers' inputs [taps][width] and its last inputs per slot; factors of the average over depth
+    float *conv_in[2] = {}, *tail_in[2] = {}, *depth = nullptr;
     uint32_t ff_kind = 0, n_expert = 0, top = 1;
     uint32_t n_shared = 0;  // pieces of the shared expert, each of an expert's size
     Dense up, down, router;  // feed-forward of a sequential block, one after the other for every expert (gate and up rows interleaved)
-    bool router_softmax = false;
+    uint32_t score_of = 0, n_group = 1, keep_group = 1;
+    float router_scale = 1.0f;
     float *side_norm = nullptr;
 
     uint32_t pairs() const { return top + n_shared; }  // experts of a token
@@ -106,6 +110,10 @@ struct LayeredGraph : StepGraph {
     bool f32 = false, has_state = false;
     uint32_t width = 0, h_pitch = 0, side_dim = 0, side_p = 0, y_pitch = 0, cat_pitch = 0;
     float eps = 0.0f, final_gain = 0.0f, residual_mult = 1.0f;
+    // plain sums: the residual alternates between m->x and x2 (cur), results of the layers, normed inputs where they are not fused away
+    bool plain = false;
+    uint32_t n_group = 1, taps = 0;
+    float *x2 = nullptr, *cur = nullptr, *history = nullptr, *normed = nullptr;
     float *final_norm = nullptr;
     std::vector<LayerPlan> L;
     __nv_bfloat16 *embd = nullptr, *side_embd = nullptr;
@@ -168,7 +176,24 @@ struct LayeredGraph : StepGraph {
     void project(const MixerPlan &P, uint32_t T, cudaStream_t st);
     void mixer(const MixerPlan &P, const float *norm, uint32_t T, uint32_t n_seq, const RowSpan *spans, bool single, uint32_t max_pos, cudaStream_t st);
     void sequential(const LayerPlan &P, const LayerPlan *next, uint32_t T, uint32_t n_seq, const RowSpan *spans, bool single, uint32_t max_pos, cudaStream_t st);
-    void post(const float *w, uint32_t T, bool last, const float *next, uint32_t top, const uint32_t *rows, uint32_t n_zero, cudaStream_t st);
+    struct Added {  // what a sublayer leaves in yo: `top` rows per token
+        uint32_t top = 1;
+        const uint32_t *rows = nullptr;  // where they are; null: in order
+        uint32_t n_zero = 0;             // of moe.count, to be zeroed
+    };
+    struct Step {
+        uint32_t T, n_seq;
+        const RowSpan *spans;
+        bool single;
+    };
+    Added feed_forward(const LayerPlan &P, uint32_t T, cudaStream_t st);
+    void post(const float *w, uint32_t T, bool last, const float *next, const Added &y, cudaStream_t st);
+    ResidualArgs residual_step(const Step &s) const;
+    void read_by(ResidualArgs &r, const LayerPlan &P, int sublayer) const;
+    void add(const LayerPlan &P, const LayerPlan *next, int sublayer, const Added &y, const Step &s, cudaStream_t st);
+    void residual(const ResidualArgs &r, cudaStream_t st) { m->ctx->launches += launch_residual(r, f32, m->ctx->sm_count, st); }
+    float *result(size_t i) const { return history + i * (size_t)m->T * width; }  // embeddings, then the results of the layers
+    uint32_t in_state() const { return taps > 1 ? (taps - 1) * width : 0; }         // of one input's convolution, per slot
     uint32_t cache_elems(const MixerPlan &P) const { return P.mx.kind == OB_MIXER_ATTENTION ? P.mx.n_kv_head * P.row : P.dq; }  // per position
     int copy_prefix(ob_kv *dst, const ob_kv *src, uint32_t n) override;
     int read_pages(const ob_kv *kv, uint32_t layer, uint32_t pos0, uint32_t n, float *k_out, float *v_out) override;
@@ -241,6 +266,7 @@ void LayeredGraph::latent(const MixerPlan &P, uint32_t T, uint32_t n_seq, const 
     a.dq = P.dq;
     a.eps = eps;
     a.scale = P.mx.scale;
+    a.sink = P.sink;
     a.kv_norm = P.kv_norm;
     a.rot = P.rot;
     a.q = q;
@@ -260,10 +286,12 @@ void LayeredGraph::latent(const MixerPlan &P, uint32_t T, uint32_t n_seq, const 
     launch_latent_prep(a, f32, st);
     m->ctx->launches++;
     const uint32_t n_short = P.expand.rows ? first_long(spans, n_seq) : n_seq;  // spans that attend in the latent space
-    const float *gate = y + (size_t)H * P.mx.rot_dim + P.mx.kv_rank + P.mx.rot_dim;
+    const float *gate = P.head_gate ? y + (size_t)H * P.mx.rot_dim + P.mx.kv_rank + P.mx.rot_dim : nullptr;
+    const void *gate_act = P.has_gate ? static_cast<const uint8_t *>(qn) + P.gate0 * es() : nullptr;
+    const uint32_t gate_pitch = P.has_gate ? P.act_rows : y_pitch;
     if (n_short) {
         a.n_seq = n_short;
-        LinArgs uk = product(P.uk, qn, H * P.dim_p, T);  // head h: its unrotated query through the key up-projection
+        LinArgs uk = product(P.uk, qn, P.act_rows, T);  // head h: its unrotated query through the key up-projection
         uk.n_rows = P.uk.rows / H;
         uk.n_batch = H;
         uk.x_step = P.dim_p;
@@ -275,8 +303,9 @@ void LayeredGraph::latent(const MixerPlan &P, uint32_t T, uint32_t n_seq, const 
         uv.n_batch = H;
         uv.x_step = P.kv_w;
         uv.gate = gate;
-        uv.gate_pitch = y_pitch;
-        segment(uv, 0, P.mx.vdim, LE_GATED, cat, cat_pitch, 0, P.mx.vdim);
+        uv.gate_act = gate_act;
+        uv.gate_pitch = gate_pitch;
+        segment(uv, 0, P.mx.vdim, gate ? LE_GATED : gate_act ? LE_GATED_EACH : LE_ACT, cat, cat_pitch, 0, P.mx.vdim);
         linear(uv, st);
     }
     LatentPrefillArgs p{};
@@ -299,7 +328,9 @@ void LayeredGraph::latent(const MixerPlan &P, uint32_t T, uint32_t n_seq, const 
     p.qn_pitch = P.act_rows;
     p.q = q;
     p.gate = gate;
-    p.gate_pitch = y_pitch;
+    p.gate_act = gate_act;
+    p.gate_pitch = gate_pitch;
+    p.sink = P.sink;
     p.out = cat;
     p.out_pitch = cat_pitch;
     const uint32_t *h_pos = reinterpret_cast<const uint32_t *>(m->h_meta + ml.off_positions);
@@ -438,7 +469,7 @@ void LayeredGraph::state_space(const MixerPlan &P, uint32_t T, uint32_t n_seq, c
     c.single = single;
     c.positions = reinterpret_cast<const uint32_t *>(m->d_meta + ml.off_positions);
     c.slots = reinterpret_cast<const int32_t *>(m->d_meta + ml.off_slots);
-    launch_conv(c, st);
+    launch_conv(c, f32, st);
     RecurrenceArgs r{};
     r.v = conv;
     r.k = conv + inner;
@@ -547,12 +578,12 @@ void LayeredGraph::mixer(const MixerPlan &P, const float *norm, uint32_t T, uint
     }
 }
 
-void LayeredGraph::post(const float *w, uint32_t T, bool last, const float *next, uint32_t top, const uint32_t *rows, uint32_t n_zero, cudaStream_t st) {
+void LayeredGraph::post(const float *w, uint32_t T, bool last, const float *next, const Added &y, cudaStream_t st) {
     PostNormArgs p{};
     p.x = m->x;
     p.y = yo;
-    p.rows = rows;
-    p.top = top;
+    p.rows = y.rows;
+    p.top = y.top;
     p.w = w;
     p.width = width;
     p.T = T;
@@ -561,15 +592,73 @@ void LayeredGraph::post(const float *w, uint32_t T, bool last, const float *next
     p.h = last ? nullptr : h;
     p.h_pitch = h_pitch;
     p.next_w = next;
-    p.zero = n_zero ? moe.count : nullptr;
-    p.n_zero = n_zero;
+    p.zero = y.n_zero ? moe.count : nullptr;
+    p.n_zero = y.n_zero;
     launch_post_norm(p, f32, st);
     m->ctx->launches++;
+}
+
+ResidualArgs LayeredGraph::residual_step(const Step &s) const {
+    const MetaLayout ml(m->T);
+    ResidualArgs r{};
+    r.mult = residual_mult;
+    r.n_group = n_group;
+    r.eps = eps;
+    r.normed = normed;
+    r.h = h;
+    r.h_pitch = h_pitch;
+    r.width = width;
+    r.T = s.T;
+    r.n_seq = s.n_seq;
+    r.spans = reinterpret_cast<const RowSpan *>(m->d_meta + ml.off_spans);
+    r.h_spans = s.spans;
+    r.single = s.single;
+    r.positions = reinterpret_cast<const uint32_t *>(m->d_meta + ml.off_positions);
+    r.slots = reinterpret_cast<const int32_t *>(m->d_meta + ml.off_slots);
+    return r;
+}
+
+// The input of a sublayer: 0 the mixer, 1 the feed-forward.
+void LayeredGraph::read_by(ResidualArgs &r, const LayerPlan &P, int sublayer) const {
+    r.norm = sublayer ? P.pre2 : P.pre1;
+    r.conv = P.conv_in[sublayer];
+    r.taps = taps;
+    r.state = P.tail_in[sublayer];
+}
+
+// Plain sums: a sublayer's output joins the residual, which becomes the input of the next one.
+void LayeredGraph::add(const LayerPlan &P, const LayerPlan *next, int sublayer, const Added &y, const Step &s, cudaStream_t st) {
+    const bool end = sublayer == 1 || !P.n_ff;
+    ResidualArgs r = residual_step(s);
+    r.x = cur;
+    r.y = yo;
+    r.top = y.top;
+    r.rows = y.rows;
+    r.zero = y.n_zero ? moe.count : nullptr;
+    r.n_zero = y.n_zero;
+    float *to = cur == m->x ? x2 : m->x;
+    if (end && !next) to = m->x;  // no convolution follows: the residual may stay where it is
+    if (end && P.depth) {
+        const size_t i = &P - L.data();
+        r.depth = P.depth;
+        r.history = history;
+        r.history_step = (uint64_t)m->T * width;
+        r.n_history = (uint32_t)i + 1;
+        r.sum = next ? result(i + 1) : nullptr;
+        r.average = to;
+    } else {
+        r.sum = to;
+    }
+    if (!end) read_by(r, P, 1);
+    else if (next) read_by(r, *next, 0);
+    residual(r, st);
+    cur = to;
 }
 
 // next: the block that follows, null after the last one.
 void LayeredGraph::sequential(const LayerPlan &P, const LayerPlan *next, uint32_t T, uint32_t n_seq, const RowSpan *spans, bool single, uint32_t max_pos, cudaStream_t st) {
     const float *next_pre = next ? next->pre1 : nullptr;
+    const Step step{T, n_seq, spans, single};
     project(P, T, st);
     mixer(P, P.pre1, T, n_seq, spans, single, max_pos, st);
     if (P.second) {
@@ -580,8 +669,16 @@ void LayeredGraph::sequential(const LayerPlan &P, const LayerPlan *next, uint32_
     out.bias = P.out_bias;
     segment(out, 0, width, LE_F32, yo, width);
     linear(out, st);
-    post(P.post1, T, !next && !P.n_ff, P.n_ff ? P.pre2 : next_pre, 1, nullptr, 0, st);
+    if (plain) add(P, next, 0, Added{}, step, st);
+    else post(P.post1, T, !next && !P.n_ff, P.n_ff ? P.pre2 : next_pre, Added{}, st);
     if (!P.n_ff) return;
+    const Added y = feed_forward(P, T, st);
+    if (plain) add(P, next, 1, y, step, st);
+    else post(P.post2, T, !next, next_pre, y, st);
+}
+
+// h through the feed-forward of a sequential block.
+LayeredGraph::Added LayeredGraph::feed_forward(const LayerPlan &P, uint32_t T, cudaStream_t st) {
     if (P.ff_kind != OB_FF_EXPERTS) {
         LinArgs up = product(P.up, h, h_pitch, T);
         if (P.ff_kind == OB_FF_GELU_GLU) segment(up, 0, 2 * P.n_ff, LE_GELU_GLU, ffa, P.down.kp);
@@ -590,8 +687,7 @@ void LayeredGraph::sequential(const LayerPlan &P, const LayerPlan *next, uint32_
         LinArgs down = product(P.down, ffa, P.down.kp, T);
         segment(down, 0, width, LE_F32, yo, width);
         linear(down, st);
-        post(P.post2, T, !next, next_pre, 1, nullptr, 0, st);
-        return;
+        return Added{};
     }
     const uint32_t R = T * P.pairs(), E = P.n_expert + P.n_shared, n_logit = P.n_expert + (P.n_shared > 0);
     const bool in_order = T == 1 || R <= MOE_ROWS_IN_ORDER;
@@ -602,7 +698,10 @@ void LayeredGraph::sequential(const LayerPlan &P, const LayerPlan *next, uint32_
     r.n_expert = P.n_expert;
     r.top = P.top;
     r.n_shared = P.n_shared;
-    r.softmax = P.router_softmax;
+    r.score_of = P.score_of;
+    r.scale = P.router_scale;
+    r.n_group = P.n_group;
+    r.keep = P.keep_group;
     r.T = T;
     r.tile_rows = linear_tile_rows(R, E, f32);
     if (in_order) r.count = nullptr;
@@ -630,21 +729,33 @@ void LayeredGraph::sequential(const LayerPlan &P, const LayerPlan *next, uint32_
         return a;
     };
     LinArgs up = grouped(P.up, in_order ? h : r.gathered, P.pairs());
-    (P.router_softmax ? up.out_scale : up.row_scale) = in_order ? r.score : r.row_score;
+    (P.score_of != OB_ROUTER_SIGMOID ? up.out_scale : up.row_scale) = in_order ? r.score : r.row_score;
     segment(up, 0, 2 * P.n_ff, LE_SWIGLU, ffa, P.down.kp);
     linear(up, st);
     LinArgs down = grouped(P.down, ffa, 1);
     segment(down, 0, width, LE_F32, yo, width);
     linear(down, st);
-    post(P.post2, T, !next, next_pre, P.pairs(), in_order ? nullptr : r.row, in_order ? 0 : E, st);
+    return Added{P.pairs(), in_order ? nullptr : r.row, in_order ? 0 : E};
 }
 
 void LayeredGraph::layers(uint32_t T, uint32_t n_seq, const RowSpan *spans, uint32_t max_pos, cudaStream_t st) {
     const MetaLayout ml(m->T);
     const uint32_t *tokens = reinterpret_cast<const uint32_t *>(m->d_meta + ml.off_tokens);
     const bool single = n_seq == T;
-    launch_embed(embd, width, tokens, T, m->x, !L[0].sequential || L[0].pre1, eps, L[0].sequential ? 1.0f : L[0].norm_gain, L[0].pre1, h, h_pitch, f32, st);
-    m->ctx->launches++;
+    if (plain) {
+        cur = m->x;
+        ResidualArgs r = residual_step(Step{T, n_seq, spans, single});
+        r.table = embd;
+        r.tokens = tokens;
+        r.sum = cur;
+        r.average = nullptr;
+        if (history) r.sum = cur = result(0);
+        read_by(r, L[0], 0);
+        residual(r, st);
+    } else {
+        launch_embed(embd, width, tokens, T, m->x, !L[0].sequential || L[0].pre1, eps, L[0].sequential ? 1.0f : L[0].norm_gain, L[0].pre1, h, h_pitch, f32, st);
+        m->ctx->launches++;
+    }
     for (size_t li = 0; li < L.size(); ++li) {
         const LayerPlan &P = L[li];
         const bool last = li + 1 == L.size();
@@ -694,8 +805,16 @@ void LayeredGraph::layers(uint32_t T, uint32_t n_seq, const RowSpan *spans, uint
 }
 
 void LayeredGraph::head(const uint32_t *d_rows, uint32_t n, cudaStream_t st) {
-    launch_norm(m->x, width, d_rows, n, eps, final_gain, final_norm, h, h_pitch, f32, st);
-    m->ctx->launches++;
+    if (plain) {
+        ResidualArgs r = residual_step(Step{n, n, nullptr, true});
+        r.x = m->x;
+        r.x_rows = d_rows;
+        r.norm = final_norm;
+        residual(r, st);
+    } else {
+        launch_norm(m->x, width, d_rows, n, eps, final_gain, final_norm, h, h_pitch, f32, st);
+        m->ctx->launches++;
+    }
     LinArgs a = product(output, h, h_pitch, n);
     segment(a, 0, m->cfg.n_vocab, LE_F32, m->logits, m->cfg.n_vocab);
     linear(a, st);
@@ -704,19 +823,23 @@ void LayeredGraph::head(const uint32_t *d_rows, uint32_t n, cudaStream_t st) {
 int LayeredGraph::copy_prefix(ob_kv *dst, const ob_kv *src, uint32_t n) {
     cudaStream_t st = m->ctx->stream;
     int rc = OB_OK;
+    auto copy = [&](float *p, size_t e) -> int {  // of one slot
+        if (p && e && src->slot >= 0 && dst->slot >= 0)
+            OB_CUDA(m->ctx, cudaMemcpyAsync(p + (size_t)dst->slot * e, p + (size_t)src->slot * e, e * 4, cudaMemcpyDeviceToDevice, st));
+        return OB_OK;
+    };
     each_mixer([&](MixerPlan &P) {
         if (P.pool && P.own_kv) {
             launch_copy_pages(P.pool, (uint64_t)KV_PAGE * cache_elems(P) * es(), src->d_table, dst->d_table, (n + KV_PAGE - 1) / KV_PAGE, st);
             m->ctx->launches++;
-        } else if (P.state && src->slot >= 0 && dst->slot >= 0 && !rc) {
-            auto copy = [&](float *p, size_t e) -> int {
-                if (e) OB_CUDA(m->ctx, cudaMemcpyAsync(p + (size_t)dst->slot * e, p + (size_t)src->slot * e, e * 4, cudaMemcpyDeviceToDevice, st));
-                return OB_OK;
-            };
+        } else if (!rc) {
             rc = copy(P.state, state_elems(P));
             if (!rc) rc = copy(P.tail, P.tail_elems);
         }
     });
+    for (LayerPlan &P : L)
+        for (float *tail : P.tail_in)
+            if (!rc) rc = copy(tail, in_state());
     return rc;
 }
 
@@ -757,6 +880,11 @@ int LayeredGraph::read_pages(const ob_kv *kv, uint32_t layer, uint32_t pos0, uin
 int LayeredGraph::read_state(const ob_kv *kv, uint32_t layer, float *out) {
     const MixerPlan *P = layer < L.size() ? &L[layer] : nullptr;
     if (P && !P->state) P = L[layer].second.get();
+    if (!P && layer < L.size() && L[layer].tail_in[0]) {  // the last inputs of both sublayers
+        const size_t e = in_state();
+        for (int k = 0; k < 2 && L[layer].tail_in[k]; ++k) OB_CUDA(m->ctx, cudaMemcpy(out + k * e, L[layer].tail_in[k] + (size_t)kv->slot * e, e * 4, cudaMemcpyDeviceToHost));
+        return OB_OK;
+    }
     if (!P || !P->state) return fail(m->ctx, OB_ERR_INVALID, "state_read: the layer has no recurrent state");
     const size_t e = state_elems(*P);
     OB_CUDA(m->ctx, cudaMemcpy(out, P->state + (size_t)kv->slot * e, e * 4, cudaMemcpyDeviceToHost));
@@ -773,8 +901,11 @@ void LayeredGraph::size_mixer(const ob_mixer_desc &x, MixerPlan &P) const {
         P.kv_p = round_up(x.kv_rank, 16);
         P.dq = P.kv_p + round_up(x.rot_dim, 16);
         P.kv_w = round_up(x.kv_rank, LIN_K_ALIGN);
-        P.act_rows = H * P.dim_p;
-        P.f32_rows = H * x.rot_dim + x.kv_rank + x.rot_dim + H;
+        P.head_gate = x.w_gate.data && x.w_gate.out_dim == H && x.vdim != 1;
+        P.has_gate = x.w_gate.data && !P.head_gate;
+        P.gate0 = H * P.dim_p;
+        P.act_rows = P.gate0 + (P.has_gate ? round_up(H * x.vdim, LIN_ROW_ALIGN) : 0);
+        P.f32_rows = H * x.rot_dim + x.kv_rank + x.rot_dim + (P.head_gate ? H : 0);
         break;
     case OB_MIXER_ATTENTION:
         P.own_kv = !x.kv_layer;
@@ -817,7 +948,8 @@ int LayeredGraph::fill_in(const ob_mixer_desc &x, MixerPlan &P, HostDense &in) {
             for (uint32_t i = 0; i < x.rot_dim; ++i) in.copy(r++, 0, x.wq, hd * (x.dim + x.rot_dim) + x.dim + i);
         }
         rows(x.w_dkv);
-        rows(x.w_gate);
+        if (P.has_gate) r = P.gate0;
+        if (x.w_gate.data) rows(x.w_gate);
     } else if (x.kind == OB_MIXER_ATTENTION) {
         r = 0;
         if (P.has_v) rows(x.wv);
@@ -849,7 +981,7 @@ int LayeredGraph::build_layer(const ob_block_desc &b, LayerPlan &P) {
     const ob_mixer_desc &x = b.mixer;
     int rc;
     size_mixer(x, P);
-    P.sequential = b.post_norm1 != nullptr;
+    P.sequential = b.post_norm1 || b.pre_norm1;
     P.ff_kind = b.ff_kind;
     const uint32_t glu = P.sequential ? 0 : b.n_ff;  // feed-forward inside the mixer's products
     P.norm_gain = b.norm_gain;
@@ -889,8 +1021,19 @@ int LayeredGraph::build_layer(const ob_block_desc &b, LayerPlan &P) {
         std::copy(x.o_bias, x.o_bias + width, bias.begin());
         if ((rc = upload_now(bias.data(), bias.size(), &P.out_bias))) return rc;
     }
-    if (P.sequential && ((rc = upload_now(b.post_norm1, width, &P.post1)) || (rc = build_ff(b, P)))) return rc;
+    if (b.post_norm1 && (rc = upload_now(b.post_norm1, width, &P.post1))) return rc;
+    if (P.sequential && (rc = build_ff(b, P))) return rc;
     if (b.pre_norm1 && (rc = upload_now(b.pre_norm1, width, &P.pre1))) return rc;
+    const float *conv[2] = {b.conv1, P.n_ff ? b.conv2 : nullptr};
+    for (int k = 0; taps && k < 2; ++k) {
+        if (!conv[k]) continue;
+        std::vector<float> w((size_t)taps * width);
+        for (uint32_t c = 0; c < width; ++c)
+            for (uint32_t i = 0; i < taps; ++i) w[(size_t)i * width + c] = conv[k][(size_t)c * taps + i];
+        if ((rc = upload_now(w.data(), w.size(), &P.conv_in[k]))) return rc;
+        if (in_state() && (rc = scratch_f32(&P.tail_in[k], (size_t)m->n_state_slots * in_state()))) return rc;
+    }
+    if (b.depth && (rc = upload_now(b.depth, &P - L.data() + 2, &P.depth))) return rc;
     if (side_dim) {
         HostDense g(round_up(side_dim, LIN_ROW_ALIGN), h_pitch), pr(round_up(width, LIN_ROW_ALIGN), side_p);
         for (uint32_t i = 0; i < side_dim; ++i) g.copy(i, 0, b.side_gate, i);
@@ -929,6 +1072,7 @@ int LayeredGraph::build_mixer(const ob_mixer_desc &x, MixerPlan &P) {
             if ((rc = upload(ex, &P.expand))) return rc;
         }
         if ((rc = upload_f32(m, x.kv_norm, x.kv_rank, &P.kv_norm))) return rc;
+        if (x.sink && (rc = upload_now(x.sink, H, &P.sink))) return rc;
         if ((rc = scratch(&P.pool, (size_t)m->pool_pages * KV_PAGE * P.dq, es()))) return rc;
     } else if (x.kind == OB_MIXER_ATTENTION) {
         const uint32_t whole_q = x.qk_norm_whole ? H : 1, whole_k = x.qk_norm_whole ? G : 1;
@@ -981,12 +1125,14 @@ int LayeredGraph::build_ff(const ob_block_desc &b, LayerPlan &P) {
     const bool experts = b.ff_kind == OB_FF_EXPERTS, gated = experts || b.ff_kind == OB_FF_GELU_GLU;
     P.n_expert = experts ? b.n_expert : 0;
     P.top = experts ? b.n_expert_used : 1;
-    P.router_softmax = b.router_softmax != 0;
+    P.score_of = b.router_softmax;
+    P.router_scale = b.router_scale;
+    if (b.n_expert_group) P.n_group = b.n_expert_group, P.keep_group = b.n_group_used;
     // A shared expert in pieces of an expert's size: a gated feed-forward is the sum of its parts.
     P.n_shared = experts ? (b.shared_ff + b.n_ff - 1) / b.n_ff : 0;
     const uint32_t E = experts ? P.n_expert + P.n_shared : 1, up_rows = round_up((gated ? 2 : 1) * b.n_ff, LIN_ROW_ALIGN), down_rows = round_up(width, LIN_ROW_ALIGN),
                    kp = round_up(b.n_ff, LIN_K_ALIGN);
-    if ((rc = upload_now(b.post_norm2, width, &P.post2))) return rc;
+    if (b.post_norm2 && (rc = upload_now(b.post_norm2, width, &P.post2))) return rc;
     if (b.pre_norm2 && (rc = upload_now(b.pre_norm2, width, &P.pre2))) return rc;
     HostDense up(E * up_rows, h_pitch), down(E * down_rows, kp);
     for (uint32_t e = 0; e < E; ++e) {
@@ -1041,7 +1187,10 @@ int LayeredGraph::build(const ob_layered_desc &c) {
     eps = c.rms_eps;
     final_gain = c.final_gain;
     residual_mult = c.residual_mult;
-    if (c.final_norm && (rc = upload_now(c.final_norm, width, &final_norm))) return rc;
+    plain = c.layers[0].pre_norm1 && !c.layers[0].post_norm1;
+    n_group = std::max(1u, c.norm_groups);
+    taps = c.conv_taps;
+    if (c.final_norm && (rc = upload_now(c.final_norm, width, &final_norm, plain ? final_gain : 1.0f))) return rc;
     L.resize(c.n_layer);
     std::map<std::pair<std::vector<double>, float>, float2 *> tables;
     size_t act = 0, q_n = 0, o_n = 0, o_r = 0, kvp = 0, dq = 0, ex = 0, reach = 0, ff_n = 0, pairs = 0, experts = 0, channels = 0, heads = 0, mixed = 0;
@@ -1114,6 +1263,12 @@ int LayeredGraph::build(const ob_layered_desc &c) {
         key_cap = (uint32_t)(T + reach);
         if ((rc = scratch(&lat, (size_t)key_cap * dq, 2)) || (rc = scratch(&expanded, (size_t)key_cap * ex, 2))) return rc;
     }
+    if (plain) {
+        if ((rc = scratch_f32(&x2, T * width))) return rc;
+        if (taps && (rc = scratch_f32(&normed, T * width))) return rc;
+        if (L[0].depth && (rc = scratch_f32(&history, (size_t)c.n_layer * T * width))) return rc;
+        if (in_state()) has_state = true;
+    }
     if (channels && ((rc = scratch_f32(&conv, T * channels)) || (rc = dev_alloc(m, &steps, T * heads)))) return rc;
     if (mixed && ((rc = scratch(&mix, T * SHIFT_MIXES * h_pitch, es())) || (rc = scratch(&low, T * low_p, es())) || (rc = scratch_f32(&decays, T * mixed)))) return rc;
     if (side_dim && ((rc = scratch(&sg, T * side_p, es())) || (rc = scratch_f32(&sy, T * width)))) return rc;
@@ -1148,7 +1303,7 @@ int check_mixer(ob_ctx *ctx, const ob_layered_desc &c, uint32_t i, const ob_mixe
         if ((rc = check_dense(ctx, x.w_dkv, E, x.kv_rank + x.rot_dim, at + "w_dkv"))) return rc;
         if ((rc = check_dense(ctx, x.w_uk, x.kv_rank, H * x.dim, at + "w_uk"))) return rc;
         if ((rc = check_dense(ctx, x.w_uv, x.kv_rank, H * x.vdim, at + "w_uv"))) return rc;
-        if ((rc = check_dense(ctx, x.w_gate, E, H, at + "mixer gate"))) return rc;
+        if (x.w_gate.data && (rc = check_dense(ctx, x.w_gate, E, x.w_gate.out_dim == H ? H : H * x.vdim, at + "mixer gate"))) return rc;
     } else if (x.kind == OB_MIXER_RETENTION) {
         if (!x.decay) return fail(ctx, OB_ERR_INVALID, "layered model: " + at + "decay missing");
         if (!retention_supported(x.dim)) return fail(ctx, OB_ERR_UNSUPPORTED, "layered model: " + at + "retention heads have at most 256 key dimensions");
@@ -1226,11 +1381,18 @@ int check_block(ob_ctx *ctx, const ob_layered_desc &c, uint32_t i) {
     }
     if ((b.post_norm1 != nullptr) != (c.layers[0].post_norm1 != nullptr)) return fail(ctx, OB_ERR_UNSUPPORTED, "layered model: " + at + "blocks of two kinds");
     if ((b.pre_norm1 != nullptr) != (c.layers[0].pre_norm1 != nullptr)) return fail(ctx, OB_ERR_UNSUPPORTED, "layered model: " + at + "blocks with and without normed inputs");
-    if (b.pre_norm1 && !b.post_norm1) return fail(ctx, OB_ERR_UNSUPPORTED, "layered model: " + at + "norms of inputs belong in sequential blocks");
-    if (b.post_norm1) {
+    const bool plain = b.pre_norm1 && !b.post_norm1;  // outputs are added as they are
+    if (plain && !c.final_norm) return fail(ctx, OB_ERR_UNSUPPORTED, "layered model: " + at + "plain sums go with factors of the last norm");
+    if (plain && b.mixer2.kind) return fail(ctx, OB_ERR_UNSUPPORTED, "layered model: " + at + "two mixers go with normed outputs");
+    if (!plain && (c.norm_groups > 1 || c.conv_taps || b.depth)) return fail(ctx, OB_ERR_UNSUPPORTED, "layered model: " + at + "norms in groups, convolved inputs and averages over depth go with plain sums");
+    if (c.conv_taps > CONV_MAX_TAPS) return fail(ctx, OB_ERR_UNSUPPORTED, "layered model: " + at + "the convolution has 1 to 16 taps");
+    if (c.norm_groups && E % c.norm_groups) return fail(ctx, OB_ERR_INVALID, "layered model: " + at + "norm_groups does not divide the width");
+    if (c.conv_taps && (!b.conv1 || (b.n_ff && !b.conv2))) return fail(ctx, OB_ERR_INVALID, "layered model: " + at + "convolution of an input missing");
+    if ((b.depth != nullptr) != (c.layers[0].depth != nullptr)) return fail(ctx, OB_ERR_UNSUPPORTED, "layered model: " + at + "layers with and without an average over depth");
+    if (plain || b.post_norm1) {
         if (c.side_dim) return fail(ctx, OB_ERR_UNSUPPORTED, "layered model: " + at + "sequential blocks have no per-layer token input");
         if (!b.n_ff) return OB_OK;
-        if (!b.post_norm2) return fail(ctx, OB_ERR_INVALID, "layered model: " + at + "norm of the feed-forward missing");
+        if (!plain && !b.post_norm2) return fail(ctx, OB_ERR_INVALID, "layered model: " + at + "norm of the feed-forward missing");
         if ((b.pre_norm2 != nullptr) != (b.pre_norm1 != nullptr)) return fail(ctx, OB_ERR_INVALID, "layered model: " + at + "norm of the feed-forward's input");
         if (b.ff_kind == OB_FF_GELU_GLU && (rc = check_dense(ctx, b.w_gate, E, b.n_ff, at + "ff gate"))) return rc;
         if (b.ff_kind == OB_FF_RELU2 || b.ff_kind == OB_FF_GELU_GLU) {
@@ -1240,6 +1402,11 @@ int check_block(ob_ctx *ctx, const ob_layered_desc &c, uint32_t i) {
         if (b.ff_kind != OB_FF_EXPERTS) return fail(ctx, OB_ERR_UNSUPPORTED, "layered model: " + at + "unknown feed-forward");
         if (!b.n_expert || !b.n_expert_used || b.n_expert_used > b.n_expert || !b.expert_gate || !b.expert_up || !b.expert_down)
             return fail(ctx, OB_ERR_INVALID, "layered model: " + at + "experts missing");
+        if (b.router_softmax > OB_ROUTER_SOFTMAX_ALL) return fail(ctx, OB_ERR_UNSUPPORTED, "layered model: " + at + "unknown scores of the router");
+        if (b.n_expert_group && (b.n_expert % b.n_expert_group || !b.n_group_used || b.n_group_used > b.n_expert_group))
+            return fail(ctx, OB_ERR_INVALID, "layered model: " + at + "groups do not divide the experts");
+        if (b.n_expert_group && b.n_expert_used > b.n_expert / b.n_expert_group * b.n_group_used)
+            return fail(ctx, OB_ERR_INVALID, "layered model: " + at + "more experts of a token than its groups hold");
         if (b.shared_ff && !b.router_softmax) return fail(ctx, OB_ERR_UNSUPPORTED, "layered model: " + at + "a shared expert goes with weighted outputs");
         if (b.shared_ff) {
             if ((rc = check_dense(ctx, b.shared_gate, E, b.shared_ff, at + "shared gate")) || (rc = check_dense(ctx, b.shared_up, E, b.shared_ff, at + "shared up")) ||
@@ -1281,7 +1448,7 @@ extern "C" int ob_layered_model_create(ob_ctx *ctx, const ob_layered_desc *desc,
     if ((rc = check_dense(ctx, c.token_embd, c.n_embd, c.n_vocab, "token_embd"))) return rc;
     if ((rc = check_dense(ctx, c.output, c.n_embd, c.n_vocab, "output"))) return rc;
     if (c.side_dim && (rc = check_dense(ctx, c.side_embd, c.n_layer * c.side_dim, c.n_vocab, "side_embd"))) return rc;
-    bool state = false;
+    bool state = c.conv_taps > 1;
     for (uint32_t i = 0; i < c.n_layer; ++i) {
         if ((rc = check_block(ctx, c, i))) return rc;
         state |= recurrent_kind(c.layers[i].mixer.kind) || recurrent_kind(c.layers[i].mixer2.kind);

@@ -1,6 +1,6 @@
 // Launchers of the kernels for models given as a list of layers (layered.cu): bf16-weight products with fused epilogues, norms,
 // latent attention over a paged latent cache, retention with a per-sequence state, softmax attention over paged keys and values,
-// mixtures of experts (internal to the library).
+// mixtures of experts, residuals averaged over depth with convolved inputs (internal to the library).
 //
 // Two precisions share every launcher.  bf16: activations that enter a product are bfloat16, accumulation is fp32.  f32:
 // activations are fp32 and every product is plain fp32 multiply-add.  Weights are bfloat16 in both.  The residual stream, norms,
@@ -27,7 +27,8 @@ enum LinEpilogue {
     LE_SWIGLU = 7,    // rows (2j, 2j+1) are (gate j, up j), both times row_scale[t]: out activation j = silu(g) u, times out_scale[t]
     LE_GELU_GLU = 8,  // rows (2j, 2j+1) are (gate j, up j): out activation j = gelu_tanh(g) u
     LE_TANH = 9,      // out activation = tanh(v)
-    LE_DECAY = 10     // out f32 = exp(-exp(v))
+    LE_DECAY = 10,    // out f32 = exp(-exp(v))
+    LE_GATED_EACH = 11  // out activation = v * sigmoid(gate_act[t * gate_pitch + column of the output])
 };
 struct LinTile {          // rows of a grouped product that share a batch entry
     uint32_t batch, row0, n;
@@ -54,6 +55,7 @@ struct LinArgs {
     const __nv_bfloat16 *emb = nullptr;
     uint32_t emb_pitch = 0, emb_col0 = 0;
     const float *gate = nullptr;
+    const void *gate_act = nullptr;  // activations
     uint32_t gate_pitch = 0;
     float *split_part = nullptr;  // scratch of products that split K, linear_split_bytes
     const float *bias = nullptr;  // [n_batch][n_rows] added to the products before the epilogue
@@ -108,11 +110,12 @@ struct Rot {                 // rotation of the first `dims` entries of a vector
 };
 
 struct LatentArgs {          // latent attention of one layer over T rows
-    const float *y;          // projections [T][y_pitch]: rotated query parts [H][rot_dim], latent [kv_rank], shared rotated key part [rot_dim], gates [H]
+    const float *y;          // projections [T][y_pitch]: rotated query parts [H][rot_dim], latent [kv_rank], shared rotated key part [rot_dim]
     uint32_t y_pitch;
     uint32_t n_head, kv_rank, rot_dim, window;  // window 0: no limit
     uint32_t kv_p, dq;       // padded latent width and padded row width (latent | rotated part) of queries and cache rows
     float eps, scale;
+    const float *sink;       // [n_head]: exp of it is added to the softmax's denominator; null: none
     const float *kv_norm;    // [kv_rank]
     Rot rot;
     void *q;                 // activations [T][H][dq]; the latent part is written by the absorbed-query product
@@ -155,8 +158,10 @@ struct LatentPrefillArgs {
     uint32_t ex_pitch, ex_v0;
     const void *qn, *q;                   // unrotated query parts [T][qn_pitch] (head h at h * dim_p), rotated ones in [T][H][dq] at kv_p
     uint32_t qn_pitch;
-    const float *gate;                    // [T][gate_pitch]: sigmoid of entry h scales head h
+    const float *gate;                    // [T][gate_pitch]: sigmoid of entry h scales head h; null: none
+    const void *gate_act;                 // activations [T][gate_pitch]: sigmoid of entry h * vdim + i scales entry i of head h; null: none
     uint32_t gate_pitch;
+    const float *sink;                    // as in LatentArgs
     void *out;                            // activations [T][out_pitch], head h at h * vdim
     uint32_t out_pitch;
 };
@@ -236,7 +241,9 @@ struct MoeArgs {             // routing of T tokens to `top` of n_expert experts
     uint32_t logit_pitch;
     uint32_t n_expert, top, T;
     uint32_t n_shared;       // experts n_expert .. that every token uses after its chosen ones; their score is the sigmoid of logit n_expert
-    bool softmax;            // scores of the chosen experts: the softmax over their logits, else the sigmoid of each
+    uint32_t score_of;       // OB_ROUTER_*: what a chosen expert's logit becomes
+    float scale;             // OB_ROUTER_SOFTMAX_ALL: factor of the scores
+    uint32_t n_group, keep;  // n_group equal groups of neighbours: only the experts of the `keep` groups with the largest logits can be chosen
     uint32_t *expert;        // [pairs]
     float *score;            // [pairs]
     // grouping (null: pairs stay in order): pairs of one expert next to one another
@@ -273,10 +280,13 @@ cudaError_t recurrence_configure();
 bool recurrence_supported(uint32_t dim);
 uint32_t launch_recurrence(const RecurrenceArgs &a, int sm_count, cudaStream_t st);  // returns the kernels launched
 
-struct ConvArgs {            // causal convolution per channel, silu; and the steps of a state-space layer
+struct ConvArgs {            // causal convolution per channel, silu; and the steps of a state-space layer.  With h: input + convolution, no silu
     const float *y;          // projections [T][y_pitch]: inputs of the channels, then [n_head] raw step sizes
     uint32_t y_pitch, n_channel, taps, n_head;
-    const float *w, *b;      // [n_channel][taps] (the last tap meets the current token), [n_channel]
+    const float *w, *b;      // [n_channel][taps] (the last tap meets the current token), or [taps][tap_step]; [n_channel], may be null
+    uint32_t tap_step;       // 0: a channel's taps are next to one another
+    void *h;                 // activations [T][h_pitch]; null: u gets the outputs
+    uint32_t h_pitch;
     float *state;            // [slot][taps - 1][n_channel]: the last inputs, the oldest first
     float *u;                // [T][n_channel]
     const float *dt_bias, *a_log;  // [n_head]
@@ -288,7 +298,7 @@ struct ConvArgs {            // causal convolution per channel, silu; and the st
     const int32_t *slots;
 };
 constexpr uint32_t CONV_MAX_TAPS = 16;
-void launch_conv(const ConvArgs &a, cudaStream_t st);
+void launch_conv(const ConvArgs &a, bool f32, cudaStream_t st);
 
 struct StateSpaceOutArgs {   // (o + skip x) silu(z), normed in n_part equal parts, times norm
     const float *o, *x;      // [T][inner]; rows of [inner]
@@ -329,6 +339,41 @@ struct TimeMixOutArgs {      // per head: (o + (sum r bonus k) v) over its root 
     uint32_t out_pitch;
 };
 void launch_time_mix_out(const TimeMixOutArgs &a, bool f32, cudaStream_t st);
+
+// ---- residual.cu -----------------------------------------------------------------------------------------------------
+struct ResidualArgs {        // s = x + mult y; v = depth average of s, or s; n = grouped norm of v; h = n + causal convolution of n (or n)
+    const float *x;          // [..][width]; null: the tokens' embeddings
+    const uint32_t *x_rows;  // row of x of each token; null: in order
+    const __nv_bfloat16 *table;
+    const uint32_t *tokens;
+    const float *y;          // null: nothing is added; else the sum of a token's `top` rows, as in PostNormArgs
+    const uint32_t *rows;
+    uint32_t top;
+    float mult;
+    float *sum;              // [T][width] gets s; may be null.  With a convolution neither this nor average may be x
+    const float *depth;      // [n_history + 1]: factors of the rows of `history`, then of s; null: no average
+    const float *history;    // n_history arrays [T][width], history_step apart
+    uint64_t history_step;
+    uint32_t n_history;
+    float *average;          // [T][width] gets v; may be null
+    const float *norm;       // [width]; null: h is not made
+    uint32_t n_group;        // equal parts of the width that are normed each by itself; at least 1
+    float eps;
+    const float *conv;       // [taps][width], the last tap meets the current token
+    uint32_t taps;           // 0: no convolution
+    float *state;            // [slot][taps - 1][width]: the last n, the oldest first
+    float *normed;           // scratch [T][width]
+    void *h;                 // activations [T][h_pitch]
+    uint32_t h_pitch;
+    uint32_t *zero;          // as in PostNormArgs
+    uint32_t n_zero;
+    uint32_t width, T, n_seq;
+    const RowSpan *spans, *h_spans;
+    bool single;             // every span is one row
+    const uint32_t *positions;
+    const int32_t *slots;
+};
+uint32_t launch_residual(const ResidualArgs &a, bool f32, int sm_count, cudaStream_t st);  // returns the kernels launched
 
 // Pages [0, n_pages) of one sequence's table to another's within a pool of pages of page_bytes (a multiple of 16).
 void launch_copy_pages(void *pool, uint64_t page_bytes, const int32_t *src_table, const int32_t *dst_table, uint32_t n_pages, cudaStream_t st);

@@ -162,6 +162,24 @@ __device__ __forceinline__ void epilogue_store(const LinArgs &a, uint32_t batch,
             store_row<N>(static_cast<float *>(g.out) + base + k, v, n);
             break;
         }
+        case LE_GATED_EACH: {
+            const TA *gate = static_cast<const TA *>(a.gate_act) + (uint64_t)t * a.gate_pitch + (uint64_t)batch * g.batch_cols + k;
+            if (N % 8 == 0 && n == N && (reinterpret_cast<uintptr_t>(gate) & 15) == 0) {
+#pragma unroll
+                for (int i = 0; i < N / 8; ++i) {
+                    float f[8];
+                    load8(gate + 8 * i, f);
+#pragma unroll
+                    for (int j = 0; j < 8; ++j) v[8 * i + j] *= sigmoidf(f[j]);
+                }
+            } else {
+#pragma unroll
+                for (int i = 0; i < N; ++i)
+                    if (i < n) v[i] *= sigmoidf((float)gate[i]);
+            }
+            store_row<N>(static_cast<TA *>(g.out) + base + k, v, n);
+            break;
+        }
         default: {  // LE_GATED
             const float s = sigmoidf(a.gate[(uint64_t)t * a.gate_pitch + batch]);
 #pragma unroll

@@ -269,7 +269,7 @@ __global__ void __launch_bounds__(LA_THREADS) latent_attn_plain_kernel(LatentArg
     for (uint32_t i = threadIdx.x; i < a.dq; i += blockDim.x) q[i] = i < a.kv_rank || (i >= a.kv_p && i < a.kv_p + a.rot_dim) ? from_act(qg[i]) : 0.0f;
     for (uint32_t i = threadIdx.x; i < a.kv_p; i += blockDim.x) acc[i] = 0.0f;
     auto row_of = [&](uint32_t j) { return cache + ((uint64_t)table[j / KV_PAGE] * KV_PAGE + j % KV_PAGE) * a.dq; };
-    float m = -INFINITY, l = 0.0f;
+    float m = a.sink ? a.sink[h] : -INFINITY, l = a.sink ? 1.0f : 0.0f;  // a sink is a key seen before all others, without a value
     __syncthreads();
     for (uint32_t j0 = lo; j0 < hi; j0 += LA_KEYS) {
         const uint32_t n = min((uint32_t)LA_KEYS, hi - j0);
@@ -339,6 +339,9 @@ struct RowCopy {
         chunk = n >= 32 ? lane : row < rows ? lane - row * n : n;
     }
 };
+
+// What a sink adds to a sum of powers of two below `top` (the largest scaled score times log2(e)).
+__device__ __forceinline__ float sink_weight(float sink, float top) { return pow2(sink * 1.4426950408889634f - top); }
 
 // NP: shares of sixteen latent columns per warp; a warp whose last share does not exist repeats another and drops it.
 template <int MT, int NP>
@@ -546,7 +549,7 @@ __global__ void __launch_bounds__(LM_THREADS, MT == 4 ? 1 : 2) latent_attn_mma_k
             const uint32_t r = i * 16 + lane / 4 + 8 * hf;
             if (r >= n_here) continue;
             const uint64_t flat = (uint64_t)row0 * a.n_head + f0 + r;
-            const float inv = whole ? 1.0f / sum[r] : 1.0f;
+            const float inv = whole ? 1.0f / (sum[r] + (a.sink ? sink_weight(a.sink[(f0 + r) % a.n_head], mx[r]) : 0.0f)) : 1.0f;
 #pragma unroll
             for (int p = 0; p < NP; ++p) {
                 if (warp + 8 * p >= n_pair) break;
@@ -584,7 +587,9 @@ __global__ void __launch_bounds__(128) latent_merge_kernel(LatentArgs a, uint32_
     for (uint32_t s = lane; s < n_splits; s += 32) m = fmaxf(m, ml[s * stride]);
     m = warp_max(m);
     for (uint32_t s = lane; s < n_splits; s += 32) l += pow2(ml[s * stride] - m) * ml[s * stride + 1];
-    const float inv = 1.0f / warp_sum(l);
+    l = warp_sum(l);
+    if (a.sink) l += sink_weight(a.sink[flat % a.n_head], m);
+    const float inv = 1.0f / l;
     bf16 *o = static_cast<bf16 *>(a.o) + flat * a.o_head;
     for (uint32_t c = 4 * (threadIdx.x % width); c < a.kv_p; c += 4 * width) {
         float4 v = make_float4(0.0f, 0.0f, 0.0f, 0.0f);
@@ -787,18 +792,27 @@ __global__ void __launch_bounds__(PF_THREADS, NV <= 8 ? 3 : 1) latent_prefill_ke
         const uint32_t tl = warp * 16 + lane / 4 + 8 * r;
         if (tl >= n_tok) continue;
         const uint64_t t = sp.row0 + t0 + tl;
-        const float f = 1.0f / ((r ? l1 : l0) * (1.0f + expf(-a.gate[t * a.gate_pitch + h])));
+        float sum = r ? l1 : l0;
+        if (a.sink) sum += sink_weight(a.sink[h], r ? m1 : m0);
+        if (a.gate) sum *= 1.0f + expf(-a.gate[t * a.gate_pitch + h]);
+        const float f = 1.0f / sum;
         bf16 *out = static_cast<bf16 *>(a.out) + t * a.out_pitch + (uint64_t)h * a.vdim;
+        const bf16 *gate = a.gate_act ? static_cast<const bf16 *>(a.gate_act) + t * a.gate_pitch + (uint64_t)h * a.vdim : nullptr;
 #pragma unroll
         for (int v = 0; v < NV; ++v)
 #pragma unroll
             for (int n = 0; n < 2; ++n) {
                 const uint32_t col = v * 16 + n * 8 + 2 * (lane & 3);
                 if (col >= a.vdim) continue;
-                if ((a.vdim & 1) == 0) *reinterpret_cast<__nv_bfloat162 *>(out + col) = __floats2bfloat162_rn(o[v][n][2 * r] * f, o[v][n][2 * r + 1] * f);
+                float o0 = o[v][n][2 * r] * f, o1 = o[v][n][2 * r + 1] * f;
+                if (gate) {
+                    o0 /= 1.0f + expf(-__bfloat162float(gate[col]));
+                    if (col + 1 < a.vdim) o1 /= 1.0f + expf(-__bfloat162float(gate[col + 1]));
+                }
+                if ((a.vdim & 1) == 0) *reinterpret_cast<__nv_bfloat162 *>(out + col) = __floats2bfloat162_rn(o0, o1);
                 else {
-                    out[col] = __float2bfloat16_rn(o[v][n][2 * r] * f);
-                    if (col + 1 < a.vdim) out[col + 1] = __float2bfloat16_rn(o[v][n][2 * r + 1] * f);
+                    out[col] = __float2bfloat16_rn(o0);
+                    if (col + 1 < a.vdim) out[col + 1] = __float2bfloat16_rn(o1);
                 }
             }
     }

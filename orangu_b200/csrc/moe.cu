@@ -5,6 +5,7 @@
 // each pair its place among them, the gathering kernel turns counts into offsets and copies the inputs.  Which place a pair gets
 // depends on timing, what is computed for it does not.
 #include "mixers_common.cuh"
+#include "../../include/orangu_b200.h"
 
 namespace ob {
 
@@ -22,35 +23,62 @@ __device__ __forceinline__ void eight(const float *p, float (&f)[8]) {
     f[0] = a.x, f[1] = a.y, f[2] = a.z, f[3] = a.w, f[4] = b.x, f[5] = b.y, f[6] = b.z, f[7] = b.w;
 }
 
-// One warp: the `top` largest of z[0 .. n) (the first of equals), best first.  Sigmoid is monotonic, so logits decide.
+// One warp: the largest of the z[0 .. n) whose lane's bit (z[lane + 32 j]: bit j) is not set, the first of equals.
+__device__ __forceinline__ void largest(const float *z, uint32_t n, uint32_t closed, float *value, uint32_t *place) {
+    float best = -INFINITY;
+    uint32_t at = 0xffffffffu;
+    for (uint32_t e = threadIdx.x & 31, j = 0; e < n; e += 32, ++j)
+        if (!(closed >> j & 1u) && (z[e] > best || at == 0xffffffffu)) best = z[e], at = e;
+#pragma unroll
+    for (int o = 16; o > 0; o >>= 1) {
+        const float v = __shfl_xor_sync(0xffffffffu, best, o);
+        const uint32_t w = __shfl_xor_sync(0xffffffffu, at, o);
+        if (w != 0xffffffffu && (at == 0xffffffffu || v > best || (v == best && w < at))) best = v, at = w;
+    }
+    *value = best, *place = at;
+}
+
+// One warp: the `top` largest of z[0 .. n) (the first of equals), best first.  Sigmoid and softmax are monotonic, so logits decide.
 __device__ __forceinline__ void choose(const MoeArgs &a, uint32_t t, const float *z) {
     const uint32_t lane = threadIdx.x & 31;
     const uint32_t p0 = t * (a.top + a.n_shared);
-    uint32_t taken = 0;  // of this lane's logits z[lane + 32 j]: bit j
+    uint32_t taken = 0;  // of this lane's logits: bit j, as in largest()
+    if (a.n_group > a.keep) {
+        const uint32_t size = a.n_expert / a.n_group;
+        uint32_t seen = 0;  // the best logit outside the groups found so far is in the next best group
+        for (uint32_t i = 0; i < a.keep; ++i) {
+            float best;
+            uint32_t at;
+            largest(z, a.n_expert, seen, &best, &at);
+            const uint32_t lo = at / size * size;
+            for (uint32_t e = lane, j = 0; e < a.n_expert; e += 32, ++j)
+                if (e - lo < size) seen |= 1u << j;
+        }
+        taken = ~seen;
+    }
     float first = 0.0f, sum = 0.0f;  // softmax: the largest logit, and the sum of exponentials below it
     for (uint32_t i = 0; i < a.top; ++i) {
-        float best = -INFINITY;
-        uint32_t at = 0xffffffffu;
-        for (uint32_t e = lane, j = 0; e < a.n_expert; e += 32, ++j)
-            if (!(taken >> j & 1u) && (z[e] > best || at == 0xffffffffu)) best = z[e], at = e;
-#pragma unroll
-        for (int o = 16; o > 0; o >>= 1) {
-            const float v = __shfl_xor_sync(0xffffffffu, best, o);
-            const uint32_t w = __shfl_xor_sync(0xffffffffu, at, o);
-            if (w != 0xffffffffu && (at == 0xffffffffu || v > best || (v == best && w < at))) best = v, at = w;
-        }
+        float best;
+        uint32_t at;
+        largest(z, a.n_expert, taken, &best, &at);
         if (at % 32 == lane) taken |= 1u << (at / 32);
         if (lane == 0) {
             const uint32_t p = p0 + i;
             a.expert[p] = at;
             if (i == 0) first = best;
             sum += expf(best - first);
-            a.score[p] = a.softmax ? best : 1.0f / (1.0f + expf(-best));
+            a.score[p] = a.score_of != OB_ROUTER_SIGMOID ? best : 1.0f / (1.0f + expf(-best));
             if (a.count) a.rank[p] = atomicAdd(a.count + at, 1u);
         }
     }
-    if (a.softmax && lane == 0)
-        for (uint32_t i = 0; i < a.top; ++i) a.score[p0 + i] = expf(a.score[p0 + i] - first) / sum;
+    if (a.score_of == OB_ROUTER_SOFTMAX_ALL) {  // (the largest logit of all has been chosen)
+        first = __shfl_sync(0xffffffffu, first, 0);
+        sum = 0.0f;
+        for (uint32_t e = lane; e < a.n_expert; e += 32) sum += expf(z[e] - first);
+        sum = warp_sum(sum);
+    }
+    if (a.score_of != OB_ROUTER_SIGMOID && lane == 0)
+        for (uint32_t i = 0; i < a.top; ++i) a.score[p0 + i] = expf(a.score[p0 + i] - first) / sum * (a.score_of == OB_ROUTER_SOFTMAX_ALL ? a.scale : 1.0f);
     for (uint32_t i = lane; i < a.n_shared; i += 32) {
         const uint32_t p = p0 + a.top + i, e = a.n_expert + i;
         a.expert[p] = e;

@@ -1,5 +1,5 @@
 """Models given as a list of layers (``ob_layered_desc``), each layer with its own token mixer.  A design's reader (fenipel.py,
-nenodra.py, senuvik.py) turns its configuration and tensors into blocks; this class owns the description and the handle."""
+nenodra.py, senuvik.py, filorax.py) turns its configuration and tensors into blocks; this class owns the description and the handle."""
 from __future__ import annotations
 
 import ctypes as C
@@ -88,6 +88,7 @@ class LayeredModel(DeviceModel):
         self.backend, self._lib = backend, backend._lib
         self._mixers = [b.mixer for b in blocks]
         self._states = [b.mixer2 if b.mixer2.kind and b.mixer.kind == capi.MIXER_ATTENTION else b.mixer for b in blocks]
+        self._inputs = [(1 + (b.n_ff > 0), max(desc.conv_taps, 1) - 1, desc.n_embd) for b in blocks]
         arr = (capi.BlockDesc * len(blocks))(*blocks)
         desc.layers = arr
         self._h = C.c_void_p()
@@ -103,4 +104,6 @@ class LayeredModel(DeviceModel):
 
     def state_shape(self, layer: int):
         m = self._states[layer]
+        if m.kind in (capi.MIXER_ATTENTION, capi.MIXER_LATENT_ATTENTION):
+            return self._inputs[layer]  # last inputs of the sublayers' convolutions, the oldest first
         return m.n_head, m.dim, m.vdim

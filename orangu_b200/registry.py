@@ -5,12 +5,13 @@ import json
 import os
 
 from .fenipel import FenipelModel
+from .filorax import FiloraxModel
 from .model import LlamaModel
 from .nenodra import NenodraModel
 from .senuvik import SenuvikModel
 
 GGUF_ARCHITECTURES = {a: LlamaModel for a in ("llama", "mistral", "qwen2", "qwen3", "qwen3vl")}
-FOLDER_ARCHITECTURES = {m.ARCHITECTURE: m for m in (FenipelModel, NenodraModel, SenuvikModel)}
+FOLDER_ARCHITECTURES = {m.ARCHITECTURE: m for m in (FenipelModel, NenodraModel, SenuvikModel, FiloraxModel)}
 
 
 def model_class(path: str):
