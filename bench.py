@@ -75,6 +75,10 @@ def parse_args():
                     "(1b, 8b: widths) beside Nenodra at the same widths; one JSON line of its own")
     ap.add_argument("--senuvik-layers", type=int, default=8, help="layers of both models in that comparison")
     ap.add_argument("--senuvik-only", action="store_true", help="leave Nenodra out")
+    ap.add_argument("--filorax", default="", metavar="SIZE[,SIZE]", help="instead of the workload above: prefill and decode of Filorax at these sizes "
+                    "(1b, 8b: widths) beside Fenipel at the same widths; one JSON line of its own")
+    ap.add_argument("--filorax-layers", type=int, default=8, help="layers of both models in that comparison")
+    ap.add_argument("--filorax-only", action="store_true", help="leave Fenipel out")
     return ap.parse_args()
 
 
@@ -480,6 +484,43 @@ def senuvik_model(size: str, n_layer: int):
     return {"architecture": "Senuvik", "vocab": V, "width": E, "norm": {"eps": 1e-6}, "layers": layers}, t
 
 
+FILORAX_SIZES = {  # Fenipel's widths, heads and latents, Senuvik's experts; two layers of three attend within a window, one is causal and rotated
+    "1b": {"width": 2048, "vocab": 32768, "experts": 16, "top": 2, "groups": 4, "keep": 2, "expert_ff": 1024, "taps": 4, "norm_groups": 8,
+           "latent": {"heads": 16, "dim": 128, "vdim": 128, "kv_rank": 384}, "rot_dim": 64, "windows": (512, 1024)},
+    "8b": {"width": 4096, "vocab": 32768, "experts": 16, "top": 2, "groups": 4, "keep": 2, "expert_ff": 2048, "taps": 4, "norm_groups": 16,
+           "latent": {"heads": 32, "dim": 128, "vdim": 128, "kv_rank": 512}, "rot_dim": 64, "windows": (512, 1024)},
+}
+
+
+def filorax_model(size: str, n_layer: int):
+    """Configuration and random bfloat16 tensors (bits)."""
+    import numpy as np
+    from orangu_b200.safetensors import to_bf16
+
+    z = FILORAX_SIZES[size]
+    E, V, X, ff, taps = z["width"], z["vocab"], z["experts"], z["expert_ff"], z["taps"]
+    lin, const = random_matrices(), lambda v, *n: to_bf16(np.full(n, v, np.float32))
+    layers, t = [], {"embed": lin(V, E, 4.0), "head": lin(V, E), "final.norm": const(1, E)}  # (tokens differ enough to choose different experts)
+    for n in range(n_layer):
+        kind = ("latent_attention_3", "latent_attention", "latent_attention_2")[n % 3]
+        at, m = f"l{n}.mix.", dict(z["latent"])
+        H, d, v, K = m["heads"], m["dim"], m["vdim"], m["kv_rank"]
+        R = z["rot_dim"] if n % 3 == 2 else 0
+        m.update(scale=(d + R) ** -0.5)
+        m.update({"rot_dim": R, "rot": {"base": 10000.0, "dims": R}} if R else {"mask": {"size": z["windows"][n % 3]}})
+        t.update({at + "q": lin(H * (d + R), E), at + "dkv": lin(K + R, E), at + "dkv.norm": const(1, K), at + "uk": lin(H * d, K), at + "uv": lin(H * v, K), at + "o": lin(E, H * v)})
+        if n % 3:
+            t.update({at + "sink": const(0.5, H), at + "g": lin(H * v, E)})
+        t.update({f"l{n}.norm1": const(1, E), f"l{n}.norm2": const(1, E), f"l{n}.canon1": lin(E, taps, 0.25), f"l{n}.canon2": lin(E, taps, 0.25), f"l{n}.dwa": const(1 / (n + 2), n + 2)})
+        t.update({f"l{n}.mlp.router": lin(X, E), f"l{n}.mlp.shared.sg": lin(1, E)})
+        for e in [f"e{e}." for e in range(X)] + ["shared."]:
+            t.update({f"l{n}.mlp.{e}gate": lin(ff, E), f"l{n}.mlp.{e}up": lin(ff, E), f"l{n}.mlp.{e}down": lin(E, ff)})
+        router = {"experts": X, "top": z["top"], "scale": 1.0, "groups": {"count": z["groups"], "keep": z["keep"]}}
+        layers.append({"type": kind, "mixer": m, "mlp": {"kind": "moe", "router": router, "expert": {"ff": ff}, "shared": {"ff": ff}}})
+    return {"architecture": "Filorax", "vocab": V, "width": E, "norm": {"eps": 1e-6, "groups": z["norm_groups"]}, "canon": {"taps": taps}, "residual_mult": 1.0,
+            "layers": layers}, t
+
+
 def time_model(be, model, vocab: int, weight_bytes, cache_bytes_per_token: float, flops_per_token: float, steps: int, warmup: int, prompt: int = 4096):
     """Prefill of one prompt and greedy decode loops at batch 1, 8 and 64 (device time, CUDA events; weights exceed L2).
     weight_bytes: read per decoded step, a number or a function of the batch.  cache_bytes_per_token: cache and state traffic of
@@ -585,6 +626,47 @@ def time_senuvik(be, size: str, L: int, steps: int, warmup: int):
     return result
 
 
+def time_filorax(be, size: str, L: int, steps: int, warmup: int):
+    import orangu_b200
+
+    cfg, t = filorax_model(size, L)
+    z, prompt = FILORAX_SIZES[size], 4096
+    expert = 3 * z["width"] * z["expert_ff"]
+    n = sum(a.size for k, a in t.items() if not k.endswith("embed"))
+    every = n - L * z["experts"] * expert
+    cache, flops = L * 2 * (z["taps"] - 1) * z["width"] * 8, 2 * (every + L * z["top"] * expert)  # (last inputs of both sublayers, read and written)
+    for layer in cfg["layers"]:
+        m = layer["mixer"]
+        R, win = m.get("rot_dim", 0), min(m["mask"]["size"], prompt) if "mask" in m else 0
+        cache += 2 * (win or prompt) * (m["kv_rank"] + R)
+        flops += 2 * (win or prompt // 2) * m["heads"] * (m["dim"] + R + m["vdim"])
+    # experts that a step reads when tokens choose independently and evenly
+    weights = lambda batch: 2 * (every + L * expert * z["experts"] * (1 - (1 - z["top"] / z["experts"]) ** batch))
+    m = orangu_b200.FiloraxModel(be, cfg, t, max_seq_len=8192, max_batch_tokens=prompt, kv_pool_tokens=64 * 4480, state_slots=64)
+    result = dict(time_model(be, m, z["vocab"], weights, cache, flops, steps, warmup), parameters=n)
+    m.close()
+    return result
+
+
+def run_filorax(args):
+    """--filorax: one JSON line with both models at every size."""
+    import orangu_b200
+
+    be = orangu_b200.CudaBackend.init(0)
+    steps, warmup, L = args.steps, max(3, args.warmup), args.filorax_layers
+    result = {"bench": "filorax", "data": "synthetic", "dtype": "bf16", "layers": L, "steps": steps, "warmup": warmup, "sizes": {}}
+    clocks = ClockSampler(0)
+    clocks.start()
+    for size in args.filorax.split(","):
+        entry = {"filorax": time_filorax(be, size, L, steps, warmup)}
+        if not args.filorax_only:
+            entry["fenipel"] = time_fenipel(be, size, L, steps, warmup)
+        result["sizes"][size] = entry
+    result["clocks"] = clocks.stop()
+    be.close()
+    print(json.dumps(result))
+
+
 def run_senuvik(args):
     """--senuvik: one JSON line with both models at every size."""
     import orangu_b200
@@ -667,6 +749,9 @@ def main():
         return
     if args.senuvik:
         run_senuvik(args)
+        return
+    if args.filorax:
+        run_filorax(args)
         return
     if args.nenodra:
         run_nenodra(args)

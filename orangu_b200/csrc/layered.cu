@@ -110,10 +110,10 @@ struct LayeredGraph : StepGraph {
     bool f32 = false, has_state = false;
     uint32_t width = 0, h_pitch = 0, side_dim = 0, side_p = 0, y_pitch = 0, cat_pitch = 0;
     float eps = 0.0f, final_gain = 0.0f, residual_mult = 1.0f;
-    // plain sums: the residual alternates between m->x and x2 (cur), results of the layers, normed inputs where they are not fused away
+    // plain sums: embeddings and results of the layers, inverse root mean squares of groups
     bool plain = false;
     uint32_t n_group = 1, taps = 0;
-    float *x2 = nullptr, *cur = nullptr, *history = nullptr, *normed = nullptr;
+    float *history = nullptr, *inverse = nullptr;
     float *final_norm = nullptr;
     std::vector<LayerPlan> L;
     __nv_bfloat16 *embd = nullptr, *side_embd = nullptr;
@@ -191,7 +191,7 @@ struct LayeredGraph : StepGraph {
     ResidualArgs residual_step(const Step &s) const;
     void read_by(ResidualArgs &r, const LayerPlan &P, int sublayer) const;
     void add(const LayerPlan &P, const LayerPlan *next, int sublayer, const Added &y, const Step &s, cudaStream_t st);
-    void residual(const ResidualArgs &r, cudaStream_t st) { m->ctx->launches += launch_residual(r, f32, m->ctx->sm_count, st); }
+    void residual(const ResidualArgs &r, cudaStream_t st) { m->ctx->launches += launch_residual(r, f32, st); }
     float *result(size_t i) const { return history + i * (size_t)m->T * width; }  // embeddings, then the results of the layers
     uint32_t in_state() const { return taps > 1 ? (taps - 1) * width : 0; }         // of one input's convolution, per slot
     uint32_t cache_elems(const MixerPlan &P) const { return P.mx.kind == OB_MIXER_ATTENTION ? P.mx.n_kv_head * P.row : P.dq; }  // per position
@@ -469,7 +469,7 @@ void LayeredGraph::state_space(const MixerPlan &P, uint32_t T, uint32_t n_seq, c
     c.single = single;
     c.positions = reinterpret_cast<const uint32_t *>(m->d_meta + ml.off_positions);
     c.slots = reinterpret_cast<const int32_t *>(m->d_meta + ml.off_slots);
-    launch_conv(c, f32, st);
+    launch_conv(c, st);
     RecurrenceArgs r{};
     r.v = conv;
     r.k = conv + inner;
@@ -604,7 +604,7 @@ ResidualArgs LayeredGraph::residual_step(const Step &s) const {
     r.mult = residual_mult;
     r.n_group = n_group;
     r.eps = eps;
-    r.normed = normed;
+    r.inverse = inverse;
     r.h = h;
     r.h_pitch = h_pitch;
     r.width = width;
@@ -630,29 +630,26 @@ void LayeredGraph::read_by(ResidualArgs &r, const LayerPlan &P, int sublayer) co
 void LayeredGraph::add(const LayerPlan &P, const LayerPlan *next, int sublayer, const Added &y, const Step &s, cudaStream_t st) {
     const bool end = sublayer == 1 || !P.n_ff;
     ResidualArgs r = residual_step(s);
-    r.x = cur;
+    const size_t i = &P - L.data();
+    r.x = i == 0 && sublayer == 0 && history ? history : m->x;
     r.y = yo;
     r.top = y.top;
     r.rows = y.rows;
     r.zero = y.n_zero ? moe.count : nullptr;
     r.n_zero = y.n_zero;
-    float *to = cur == m->x ? x2 : m->x;
-    if (end && !next) to = m->x;  // no convolution follows: the residual may stay where it is
     if (end && P.depth) {
-        const size_t i = &P - L.data();
         r.depth = P.depth;
         r.history = history;
         r.history_step = (uint64_t)m->T * width;
         r.n_history = (uint32_t)i + 1;
         r.sum = next ? result(i + 1) : nullptr;
-        r.average = to;
+        r.average = m->x;
     } else {
-        r.sum = to;
+        r.sum = m->x;
     }
     if (!end) read_by(r, P, 1);
     else if (next) read_by(r, *next, 0);
     residual(r, st);
-    cur = to;
 }
 
 // next: the block that follows, null after the last one.
@@ -743,13 +740,10 @@ void LayeredGraph::layers(uint32_t T, uint32_t n_seq, const RowSpan *spans, uint
     const uint32_t *tokens = reinterpret_cast<const uint32_t *>(m->d_meta + ml.off_tokens);
     const bool single = n_seq == T;
     if (plain) {
-        cur = m->x;
         ResidualArgs r = residual_step(Step{T, n_seq, spans, single});
         r.table = embd;
         r.tokens = tokens;
-        r.sum = cur;
-        r.average = nullptr;
-        if (history) r.sum = cur = result(0);
+        r.sum = history ? history : m->x;
         read_by(r, L[0], 0);
         residual(r, st);
     } else {
@@ -1264,8 +1258,7 @@ int LayeredGraph::build(const ob_layered_desc &c) {
         if ((rc = scratch(&lat, (size_t)key_cap * dq, 2)) || (rc = scratch(&expanded, (size_t)key_cap * ex, 2))) return rc;
     }
     if (plain) {
-        if ((rc = scratch_f32(&x2, T * width))) return rc;
-        if (taps && (rc = scratch_f32(&normed, T * width))) return rc;
+        if ((rc = scratch_f32(&inverse, T * n_group))) return rc;
         if (L[0].depth && (rc = scratch_f32(&history, (size_t)c.n_layer * T * width))) return rc;
         if (in_state()) has_state = true;
     }

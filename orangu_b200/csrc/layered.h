@@ -280,13 +280,10 @@ cudaError_t recurrence_configure();
 bool recurrence_supported(uint32_t dim);
 uint32_t launch_recurrence(const RecurrenceArgs &a, int sm_count, cudaStream_t st);  // returns the kernels launched
 
-struct ConvArgs {            // causal convolution per channel, silu; and the steps of a state-space layer.  With h: input + convolution, no silu
+struct ConvArgs {            // causal convolution per channel, silu; and the steps of a state-space layer
     const float *y;          // projections [T][y_pitch]: inputs of the channels, then [n_head] raw step sizes
     uint32_t y_pitch, n_channel, taps, n_head;
-    const float *w, *b;      // [n_channel][taps] (the last tap meets the current token), or [taps][tap_step]; [n_channel], may be null
-    uint32_t tap_step;       // 0: a channel's taps are next to one another
-    void *h;                 // activations [T][h_pitch]; null: u gets the outputs
-    uint32_t h_pitch;
+    const float *w, *b;      // [n_channel][taps] (the last tap meets the current token), [n_channel]
     float *state;            // [slot][taps - 1][n_channel]: the last inputs, the oldest first
     float *u;                // [T][n_channel]
     const float *dt_bias, *a_log;  // [n_head]
@@ -298,7 +295,7 @@ struct ConvArgs {            // causal convolution per channel, silu; and the st
     const int32_t *slots;
 };
 constexpr uint32_t CONV_MAX_TAPS = 16;
-void launch_conv(const ConvArgs &a, bool f32, cudaStream_t st);
+void launch_conv(const ConvArgs &a, cudaStream_t st);
 
 struct StateSpaceOutArgs {   // (o + skip x) silu(z), normed in n_part equal parts, times norm
     const float *o, *x;      // [T][inner]; rows of [inner]
@@ -350,7 +347,7 @@ struct ResidualArgs {        // s = x + mult y; v = depth average of s, or s; n 
     const uint32_t *rows;
     uint32_t top;
     float mult;
-    float *sum;              // [T][width] gets s; may be null.  With a convolution neither this nor average may be x
+    float *sum;              // [T][width] gets s; may be null, may be x.  With a convolution one of this and average is given
     const float *depth;      // [n_history + 1]: factors of the rows of `history`, then of s; null: no average
     const float *history;    // n_history arrays [T][width], history_step apart
     uint64_t history_step;
@@ -362,7 +359,7 @@ struct ResidualArgs {        // s = x + mult y; v = depth average of s, or s; n 
     const float *conv;       // [taps][width], the last tap meets the current token
     uint32_t taps;           // 0: no convolution
     float *state;            // [slot][taps - 1][width]: the last n, the oldest first
-    float *normed;           // scratch [T][width]
+    float *inverse;          // scratch [T][n_group]
     void *h;                 // activations [T][h_pitch]
     uint32_t h_pitch;
     uint32_t *zero;          // as in PostNormArgs
@@ -373,7 +370,7 @@ struct ResidualArgs {        // s = x + mult y; v = depth average of s, or s; n 
     const uint32_t *positions;
     const int32_t *slots;
 };
-uint32_t launch_residual(const ResidualArgs &a, bool f32, int sm_count, cudaStream_t st);  // returns the kernels launched
+uint32_t launch_residual(const ResidualArgs &a, bool f32, cudaStream_t st);  // returns the kernels launched
 
 // Pages [0, n_pages) of one sequence's table to another's within a pool of pages of page_bytes (a multiple of 16).
 void launch_copy_pages(void *pool, uint64_t page_bytes, const int32_t *src_table, const int32_t *dst_table, uint32_t n_pages, cudaStream_t st);

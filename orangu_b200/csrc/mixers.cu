@@ -16,10 +16,6 @@ namespace {
 
 // (No __restrict__ on what an earlier kernel writes: a load the compiler may take for invariant could move above pdl_wait.)
 // ---- embedding, norms ------------------------------------------------------------------------------------------------------
-// A row in registers: element group i of a thread is columns 4 (threadIdx + i blockDim) .. + 3; NV = 0: any width, one column
-// at a time through memory.
-constexpr int ROW_VECS = 4;
-
 // x = the token's embedding, h = x / rms(x) * gain (* w) or x.
 template <typename TA, int NV>
 __global__ void __launch_bounds__(1024) embed_kernel(const bf16 *table, uint32_t width, const uint32_t *tokens, float *x, bool normed, float eps, float gain, const float *w, TA *h,
@@ -1112,16 +1108,6 @@ cudaError_t mixers_configure() {
     });
 }
 
-// Kernel form and threads for rows of `width`: in registers when the columns come in fours and fit, few rows on wide CTAs.
-struct RowShape {
-    bool vec;
-    uint32_t threads;
-    RowShape(uint32_t width, uint32_t rows, int sm_rows = 296) {
-        const uint32_t want = (width / 4 + 31) / 32 * 32;
-        threads = rows <= (uint32_t)sm_rows ? std::min(1024u, std::max(128u, want)) : std::min(1024u, std::max(128u, (want / ROW_VECS + 31) / 32 * 32));
-        vec = width % 4 == 0 && (uint64_t)threads * 4 * ROW_VECS >= width;
-    }
-};
 template <typename TA>
 static void embed(const bf16 *table, uint32_t width, const uint32_t *tokens, uint32_t T, float *x, bool normed, float eps, float gain, const float *w, void *h, uint32_t h_pitch,
                   cudaStream_t st) {

@@ -4,6 +4,8 @@
 
 #include <math.h>
 
+#include <algorithm>
+
 #include "layered.h"
 #include "pdl.cuh"
 
@@ -33,6 +35,21 @@ __device__ __forceinline__ float block_sum(float v, float *red) {
 }
 
 __device__ __forceinline__ float inv_rms(float sum_sq, uint32_t n, float eps) { return 1.0f / sqrtf(sum_sq / (float)n + eps); }
+
+// A row in registers: element group i of a thread is columns 4 (threadIdx + i blockDim) .. + 3; NV = 0: any width, one column
+// at a time through memory.
+constexpr int ROW_VECS = 4;
+
+// Kernel form and threads for rows of `width`: in registers when the columns come in fours and fit, few rows on wide CTAs.
+struct RowShape {
+    bool vec;
+    uint32_t threads;
+    RowShape(uint32_t width, uint32_t rows, int sm_rows = 296) {
+        const uint32_t want = (width / 4 + 31) / 32 * 32;
+        threads = rows <= (uint32_t)sm_rows ? std::min(1024u, std::max(128u, want)) : std::min(1024u, std::max(128u, (want / ROW_VECS + 31) / 32 * 32));
+        vec = width % 4 == 0 && (uint64_t)threads * 4 * ROW_VECS >= width;
+    }
+};
 
 // A row of activations from four fp32 values per thread and step.
 template <typename TA> __device__ __forceinline__ void store4(TA *p, float4 v);

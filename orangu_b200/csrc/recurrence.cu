@@ -358,11 +358,11 @@ __global__ void __launch_bounds__(32 * NW) recurrence_span_kernel(RecurrenceArgs
         }
 }
 
-// ---- convolution over time; state space: and steps -----------------------------------------------------------------------------------
+// ---- state space: convolution and steps ---------------------------------------------------------------------------------------------
 // A thread has one channel of CV_TOKENS consecutive tokens of a span; threads past the channels have a head's step sizes.  The
 // thread with the first tokens of a span is the only one that reads the state, and replaces it when it has.
 constexpr int CV_THREADS = 128, CV_TOKENS = 16;  // (a decoded token: one)
-template <int K, int TOKENS, typename TA = void>  // taps (0: a.taps), tokens of a thread; TA: the sum of input and convolution is left as activation
+template <int K, int TOKENS>  // taps (0: a.taps), tokens of a thread
 __global__ void __launch_bounds__(CV_THREADS) conv_kernel(ConvArgs a) {
     pdl_release();
     pdl_wait();
@@ -386,17 +386,13 @@ __global__ void __launch_bounds__(CV_THREADS) conv_kernel(ConvArgs a) {
     float *state = a.state + (uint64_t)a.slots[sp.row0] * back * a.n_channel + c;
     const bool fresh = a.positions[sp.row0] == 0;
     auto input = [&](int t) { return t >= 0 ? y[(uint64_t)t * a.y_pitch] : fresh ? 0.0f : state[(uint64_t)(t + back) * a.n_channel]; };
-    const uint32_t w_step = a.tap_step ? a.tap_step : 1;
-    const float *w = a.w + (a.tap_step ? c : (uint64_t)c * taps);
-    const float bias = a.b ? a.b[c] : 0.0f;
-    auto out = [&](int t, float s, float x) {
-        if constexpr (std::is_void_v<TA>) a.u[(uint64_t)(sp.row0 + t) * a.n_channel + c] = silu(s);
-        else static_cast<TA *>(a.h)[(uint64_t)(sp.row0 + t) * a.h_pitch + c] = to_act<TA>(x + s);
-    };
+    const float *w = a.w + (uint64_t)c * taps;
+    const float bias = a.b[c];
+    float *u = a.u + (uint64_t)sp.row0 * a.n_channel + c;
     if constexpr (K > 0) {
         float wk[K], x[K - 1 + TOKENS];  // all inputs are requested before the first is used
 #pragma unroll
-        for (int i = 0; i < K; ++i) wk[i] = w[i * w_step];
+        for (int i = 0; i < K; ++i) wk[i] = w[i];
 #pragma unroll
         for (int i = 0; i + 1 < K; ++i) x[i] = input(first - back + i);
 #pragma unroll
@@ -406,13 +402,13 @@ __global__ void __launch_bounds__(CV_THREADS) conv_kernel(ConvArgs a) {
             float s = bias;
 #pragma unroll
             for (int k = 0; k < K; ++k) s = fmaf(wk[k], x[i + k], s);
-            if (first + i < last) out(first + i, s, x[i + K - 1]);
+            if (first + i < last) u[(uint64_t)(first + i) * a.n_channel] = silu(s);
         }
     } else {
         for (int t = first; t < last; ++t) {
             float s = bias;
-            for (int i = 0; i < taps; ++i) s = fmaf(w[i * w_step], input(t - back + i), s);
-            out(t, s, input(t));
+            for (int i = 0; i < taps; ++i) s = fmaf(w[i], input(t - back + i), s);
+            u[(uint64_t)t * a.n_channel] = silu(s);
         }
     }
     if (first == 0)  // (an entry that is read here has a higher number than the one it goes to: it has not been replaced yet)
@@ -654,8 +650,7 @@ uint32_t launch_recurrence(const RecurrenceArgs &a, int sm_count, cudaStream_t s
     return a.step ? run<false>(a, sm_count, st) : run<true>(a, sm_count, st);
 }
 
-template <typename TA>
-static void conv(const ConvArgs &a, cudaStream_t st) {
+void launch_conv(const ConvArgs &a, cudaStream_t st) {
     uint32_t tiles = a.T;
     if (!a.single) {
         tiles = 0;
@@ -664,15 +659,10 @@ static void conv(const ConvArgs &a, cudaStream_t st) {
     const dim3 grid(tiles, (a.n_channel + a.n_head + CV_THREADS - 1) / CV_THREADS);
     auto run = [&](auto tokens) {
         constexpr int N = decltype(tokens)::value;
-        launch_pdl(a.taps == 4 ? conv_kernel<4, N, TA> : a.taps == 3 ? conv_kernel<3, N, TA> : a.taps == 2 ? conv_kernel<2, N, TA> : conv_kernel<0, N, TA>, grid, CV_THREADS, 0, st, a);
+        launch_pdl(a.taps == 4 ? conv_kernel<4, N> : a.taps == 3 ? conv_kernel<3, N> : a.taps == 2 ? conv_kernel<2, N> : conv_kernel<0, N>, grid, CV_THREADS, 0, st, a);
     };
     if (a.single) run(std::integral_constant<int, 1>{});
     else run(std::integral_constant<int, CV_TOKENS>{});
-}
-void launch_conv(const ConvArgs &a, bool f32, cudaStream_t st) {
-    if (!a.h) conv<void>(a, st);
-    else if (f32) conv<float>(a, st);
-    else conv<bf16>(a, st);
 }
 
 bool state_space_out_supported(uint32_t part) { return (uint64_t)part * 4 <= OUT_SMEM; }

@@ -1,16 +1,16 @@
 // Between two sublayers of a block that adds their outputs as they are: the output joins the residual, a layer's result is averaged
 // with the results of the layers before it, the sum is normed in groups, and a short causal convolution over time is added to it.
-// One kernel makes all of it, so what the next sublayer reads is written once:
 //   s = x + mult * (rows of y of the token)        or the token's embedding
 //   v = depth[n] s + sum_j depth[j] history[j]     or s
 //   n = v over the root mean square of its group, times the norm's factors
 //   h = n + sum_k conv[k] n of the token taps - 1 - k before
 // The last taps - 1 rows n of a sequence are its state.
 //
-// residual_run_kernel   a CTA takes consecutive tokens of a span with the rows n the convolution reaches back to in registers; it
-//                       makes the ones before its first token again (nothing it reads is overwritten: sums go elsewhere)
-// residual_row_kernel   any width, group and number of taps: a CTA per token up to n, then the convolution (recurrence.cu)
+// residual_kernel     a CTA per token: s, v, and n or (every token from another sequence) h.  For spans it leaves the inverse root mean
+//                     squares instead: n is then a product of three numbers, and is made where it is used
+// input_conv_kernel   h of spans: a few channels of several tokens per thread, no exchange between threads
 #include <algorithm>
+#include <type_traits>
 
 #include "mixers_common.cuh"
 
@@ -30,148 +30,123 @@ __device__ __forceinline__ float4 f4(const float *p) { return *reinterpret_cast<
 // Squares are summed in units: a warp's 128 columns when groups consist of such, else a thread's four.
 __host__ __device__ constexpr uint32_t unit_columns(uint32_t group) { return group % 128 ? 4 : 128; }
 
-// NV: float4 of a thread; TAPS: of the convolution, 0: none.
-template <typename TA, int NV, int TAPS>
-__global__ void __launch_bounds__(1024) residual_run_kernel(ResidualArgs a, uint32_t run) {
+enum Leave { LEAVE_INPUT = 0, LEAVE_INVERSE = 1 };  // h; the inverse root mean squares
+
+// Conv of one token alone: n of the tokens before it are the state, which moves on by one.
+template <int V, typename F>
+__device__ __forceinline__ void conv_step(const ResidualArgs &a, float *state, bool fresh, uint32_t c, const float (&n)[V], F store) {
+    float o[V];
+    const uint32_t back = a.taps - 1;
+#pragma unroll
+    for (int e = 0; e < V; ++e) o[e] = fmaf(a.conv[(uint64_t)back * a.width + c + e], n[e], n[e]);
+    for (uint32_t k = 0; k < back; ++k) {
+        float *p = state + (uint64_t)k * a.width + c;
+#pragma unroll
+        for (int e = 0; e < V; ++e) {
+            const float before = fresh ? 0.0f : p[e];
+            o[e] = fmaf(a.conv[(uint64_t)k * a.width + c + e], before, o[e]);
+            if (k) p[e - (int)a.width] = before;
+            if (k + 1 == back) p[e] = n[e];
+        }
+    }
+    store(o);
+}
+
+template <typename TA, int NV, Leave LEAVE>
+__global__ void __launch_bounds__(1024) residual_kernel(ResidualArgs a) {
     extern __shared__ float sm[];
-    constexpr int BACK = TAPS > 1 ? TAPS - 1 : 0;
-    const uint32_t warp = threadIdx.x >> 5, lane = threadIdx.x & 31, warps = blockDim.x >> 5;
+    const uint32_t warp = threadIdx.x >> 5, lane = threadIdx.x & 31, warps = blockDim.x >> 5, t = blockIdx.x;
     const uint32_t group = a.width / a.n_group, unit = unit_columns(group), per_group = group / unit;
     float *units = sm, *inv = sm + a.width / unit;
     pdl_release();
     pdl_wait();
-    RowSpan sp{blockIdx.x, 1};
-    uint32_t f0 = 0;
-    if (run > 1) find_tile(a.spans, a.n_seq, 1, run, blockIdx.x, &sp, &f0);
-    if (f0 >= sp.n) return;
-    if (a.zero && blockIdx.x == 0)
+    if (a.zero && t == 0)
         for (uint32_t i = threadIdx.x; i < a.n_zero; i += blockDim.x) a.zero[i] = 0;
-    const int n = (int)sp.n, first = (int)f0, last = min(first + (int)run, n);
-    float *state = nullptr;
-    bool fresh = true;
-    if (BACK) {
-        state = a.state + (uint64_t)a.slots[sp.row0] * BACK * a.width;
-        fresh = a.positions[sp.row0] == 0;
+    const uint64_t at = (uint64_t)t * a.width;
+    const float *x = a.x ? a.x + (uint64_t)(a.x_rows ? a.x_rows[t] : t) * a.width : nullptr;
+    const bf16 *embedding = a.x ? nullptr : a.table + (uint64_t)a.tokens[t] * a.width;
+    float4 v[NV];
+    auto each = [&](auto f) {
+#pragma unroll
+        for (int i = 0; i < NV; ++i) {
+            const uint32_t c = 4 * (threadIdx.x + i * blockDim.x);
+            if (c < a.width) f(i, c);
+        }
+    };
+#pragma unroll
+    for (int i = 0; i < NV; ++i) v[i] = make_float4(0.0f, 0.0f, 0.0f, 0.0f);
+    each([&](int i, uint32_t c) { v[i] = x ? f4(x + c) : bf16x4(embedding + c); });
+    if (a.y) {
+        float4 y[NV];
+        const float *row = a.y + (uint64_t)(a.rows ? a.rows[t * a.top] : t * a.top) * a.width;
+        each([&](int i, uint32_t c) { y[i] = f4(row + c); });
+        for (uint32_t k = 1; k < a.top; ++k) {
+            const float *more = a.y + (uint64_t)(a.rows ? a.rows[t * a.top + k] : t * a.top + k) * a.width;
+            each([&](int i, uint32_t c) { y[i] = add4(y[i], f4(more + c)); });
+        }
+        each([&](int i, uint32_t c) { v[i] = fma4(a.mult, y[i], v[i]); });
     }
-    auto col = [&](int i) { return 4 * (threadIdx.x + i * blockDim.x); };
-    // The row before the norm; stored where the token is this CTA's own.
-    auto value = [&](uint32_t t, bool own, float4 (&v)[NV]) {
-        const uint64_t at = (uint64_t)t * a.width;
-        const float *x = a.x ? a.x + (uint64_t)(a.x_rows ? a.x_rows[t] : t) * a.width : nullptr;
-        const bf16 *e = a.x ? nullptr : a.table + (uint64_t)a.tokens[t] * a.width;
-        const float last_weight = a.depth ? a.depth[a.n_history] : 1.0f;
-#pragma unroll
-        for (int i = 0; i < NV; ++i) {
-            const uint32_t c = col(i);
-            v[i] = make_float4(0.0f, 0.0f, 0.0f, 0.0f);
-            if (c >= a.width) continue;
-            v[i] = x ? f4(x + c) : bf16x4(e + c);
-            if (a.y) {
-                float4 y = make_float4(0.0f, 0.0f, 0.0f, 0.0f);
-#pragma unroll 4
-                for (uint32_t k = 0; k < a.top; ++k) {
-                    const uint32_t p = t * a.top + k;
-                    y = add4(y, f4(a.y + (uint64_t)(a.rows ? a.rows[p] : p) * a.width + c));
-                }
-                v[i] = fma4(a.mult, y, v[i]);
-            }
-            if (own && a.sum) *reinterpret_cast<float4 *>(a.sum + at + c) = v[i];
-            if (a.depth) {
-                float4 s = mul4(v[i], last_weight);
-#pragma unroll 8
-                for (uint32_t j = 0; j < a.n_history; ++j) s = fma4(a.depth[j], f4(a.history + j * a.history_step + at + c), s);
-                v[i] = s;
-                if (own && a.average) *reinterpret_cast<float4 *>(a.average + at + c) = s;
-            }
+    if (a.sum) each([&](int i, uint32_t c) { *reinterpret_cast<float4 *>(a.sum + at + c) = v[i]; });
+    if (a.depth) {
+        const float own = a.depth[a.n_history];
+        each([&](int i, uint32_t) { v[i] = mul4(v[i], own); });
+#pragma unroll 2
+        for (uint32_t j = 0; j < a.n_history; ++j) {
+            const float f = a.depth[j];
+            const float *past = a.history + j * a.history_step + at;
+            each([&](int i, uint32_t c) { v[i] = fma4(f, f4(past + c), v[i]); });
         }
-    };
-    auto normed = [&](float4 (&v)[NV]) {
-#pragma unroll
-        for (int i = 0; i < NV; ++i) {
-            const uint32_t c = col(i);
-            const float s = sq4(v[i]);
-            if (unit == 128) {
-                const float w = warp_sum(s);
-                if (lane == 0 && c < a.width) units[c / 128] = w;
-            } else if (c < a.width) {
-                units[c / 4] = s;
-            }
-        }
-        __syncthreads();
-        for (uint32_t g = warp; g < a.n_group; g += warps) {
-            float s = 0.0f;
-            for (uint32_t u = lane; u < per_group; u += 32) s += units[g * per_group + u];
-            s = warp_sum(s);
-            if (lane == 0) inv[g] = inv_rms(s, group, a.eps);
-        }
-        __syncthreads();
-#pragma unroll
-        for (int i = 0; i < NV; ++i) {
-            const uint32_t c = col(i);
-            if (c < a.width) v[i] = mul44(mul4(v[i], inv[c / group]), f4(a.norm + c));
-        }
-    };
-    float4 ring[BACK > 0 ? BACK : 1][NV];  // the rows n before the current one, the oldest first
-    auto push = [&](const float4 (&v)[NV]) {
-        if constexpr (BACK > 0) {
-#pragma unroll
-            for (int i = 0; i < NV; ++i) {
-#pragma unroll
-                for (int k = 0; k + 1 < BACK; ++k) ring[k][i] = ring[k + 1][i];
-                ring[BACK - 1][i] = v[i];
-            }
-        }
-    };
-    TA *h = static_cast<TA *>(a.h);
-    for (int t = first - BACK; t < last; ++t) {
-        float4 v[NV];
-        if (t < 0) {
-#pragma unroll
-            for (int i = 0; i < NV; ++i) {
-                const uint32_t c = col(i);
-                v[i] = fresh || c >= a.width ? make_float4(0.0f, 0.0f, 0.0f, 0.0f) : f4(state + (uint64_t)(t + BACK) * a.width + c);
-            }
-        } else {
-            value(sp.row0 + t, t >= first, v);
-            if (!a.norm) continue;
-            normed(v);
-        }
-        if (t >= first) {
-#pragma unroll
-            for (int i = 0; i < NV; ++i) {
-                const uint32_t c = col(i);
-                if (c >= a.width) continue;
-                float4 o = v[i];
-                if constexpr (TAPS > 0) {
-                    const float *w = a.conv + c;  // [taps][width]
-                    o = fma44(f4(w + (uint64_t)BACK * a.width), v[i], o);
-#pragma unroll
-                    for (int k = 0; k < BACK; ++k) o = fma44(f4(w + (uint64_t)k * a.width), ring[k][i], o);
-                }
-                store4<TA>(h + (uint64_t)(sp.row0 + t) * a.h_pitch + c, o);
-            }
-        }
-        push(v);
+        if (a.average) each([&](int i, uint32_t c) { *reinterpret_cast<float4 *>(a.average + at + c) = v[i]; });
     }
-    if constexpr (BACK > 0) {
-        if (first > 0) return;  // the CTA that has read the state replaces it
-        if (n > last)           // (a run is not shorter than the convolution reaches back)
-            for (int t = n - BACK; t < n; ++t) {
-                float4 v[NV];
-                value(sp.row0 + t, false, v);
-                normed(v);
-                push(v);
+    if (!a.norm) return;
+#pragma unroll
+    for (int i = 0; i < NV; ++i) {
+        const uint32_t c = 4 * (threadIdx.x + i * blockDim.x);
+        const float s = sq4(v[i]);
+        if (unit == 128) {
+            const float w = warp_sum(s);
+            if (lane == 0 && c < a.width) units[c / 128] = w;
+        } else if (c < a.width) {
+            units[c / 4] = s;
+        }
+    }
+    __syncthreads();
+    for (uint32_t g = warp; g < a.n_group; g += warps) {
+        float s = 0.0f;
+        for (uint32_t u = lane; u < per_group; u += 32) s += units[g * per_group + u];
+        s = warp_sum(s);
+        if (lane == 0) (LEAVE == LEAVE_INVERSE ? a.inverse + (uint64_t)t * a.n_group : inv)[g] = inv_rms(s, group, a.eps);
+    }
+    if constexpr (LEAVE == LEAVE_INPUT) {
+        __syncthreads();
+        TA *h = static_cast<TA *>(a.h) + (uint64_t)t * a.h_pitch;
+        float *state = a.taps > 1 ? a.state + (uint64_t)a.slots[t] * (a.taps - 1) * a.width : nullptr;
+        const bool fresh = a.taps > 1 && a.positions[t] == 0;
+        each([&](int i, uint32_t c) {
+            const float4 n = mul44(mul4(v[i], inv[c / group]), f4(a.norm + c));
+            if (!a.taps) {
+                store4<TA>(h + c, n);
+            } else if (a.taps == 4) {  // all of the state is requested at once
+                float *p = state + c;
+                const uint32_t w = a.width;
+                float4 b[3] = {};
+                if (!fresh) b[0] = f4(p), b[1] = f4(p + w), b[2] = f4(p + 2 * w);
+                float4 o = fma44(f4(a.conv + 3 * w + c), n, n);
+#pragma unroll
+                for (int k = 0; k < 3; ++k) o = fma44(f4(a.conv + k * w + c), b[k], o);
+                *reinterpret_cast<float4 *>(p) = b[1], *reinterpret_cast<float4 *>(p + w) = b[2], *reinterpret_cast<float4 *>(p + 2 * w) = n;
+                store4<TA>(h + c, o);
+            } else {
+                const float e[4] = {n.x, n.y, n.z, n.w};
+                conv_step<4>(a, state, fresh, c, e, [&](const float(&o)[4]) { store4<TA>(h + c, make_float4(o[0], o[1], o[2], o[3])); });
             }
-#pragma unroll
-        for (int i = 0; i < NV; ++i)
-            if (col(i) < a.width)
-#pragma unroll
-                for (int k = 0; k < BACK; ++k) *reinterpret_cast<float4 *>(state + (uint64_t)k * a.width + col(i)) = ring[k][i];
+        });
     }
 }
 
-template <typename TA>
-__global__ void __launch_bounds__(512) residual_row_kernel(ResidualArgs a) {
+// Any width and groups: columns one at a time through memory.
+template <typename TA, Leave LEAVE>
+__global__ void __launch_bounds__(512) residual_any_kernel(ResidualArgs a) {
     __shared__ float red[33];
     pdl_release();
     pdl_wait();
@@ -179,100 +154,161 @@ __global__ void __launch_bounds__(512) residual_row_kernel(ResidualArgs a) {
         for (uint32_t i = threadIdx.x; i < a.n_zero; i += blockDim.x) a.zero[i] = 0;
     const uint32_t t = blockIdx.x, group = a.width / a.n_group;
     const uint64_t at = (uint64_t)t * a.width;
-    auto value = [&](uint32_t c, bool store) {
+    auto sum = [&](uint32_t c) {
         float v = a.x ? a.x[(uint64_t)(a.x_rows ? a.x_rows[t] : t) * a.width + c] : __bfloat162float(a.table[(uint64_t)a.tokens[t] * a.width + c]);
-        if (a.y) {
-            float y = 0.0f;
-            for (uint32_t k = 0; k < a.top; ++k) {
-                const uint32_t p = t * a.top + k;
-                y += a.y[(uint64_t)(a.rows ? a.rows[p] : p) * a.width + c];
-            }
-            v = fmaf(a.mult, y, v);
+        if (!a.y) return v;
+        float y = 0.0f;
+        for (uint32_t k = 0; k < a.top; ++k) {
+            const uint32_t p = t * a.top + k;
+            y += a.y[(uint64_t)(a.rows ? a.rows[p] : p) * a.width + c];
         }
-        float s = v;
-        if (a.depth) {
-            s = v * a.depth[a.n_history];
-            for (uint32_t j = 0; j < a.n_history; ++j) s = fmaf(a.depth[j], a.history[j * a.history_step + at + c], s);
-        }
-        if (store) {
-            if (a.sum) a.sum[at + c] = v;
-            if (a.depth && a.average) a.average[at + c] = s;
-        }
-        return s;
+        return fmaf(a.mult, y, v);
     };
+    auto averaged = [&](uint32_t c, float s) {
+        if (!a.depth) return s;
+        float v = s * a.depth[a.n_history];
+        for (uint32_t j = 0; j < a.n_history; ++j) v = fmaf(a.depth[j], a.history[j * a.history_step + at + c], v);
+        return v;
+    };
+    float *state = LEAVE == LEAVE_INPUT && a.norm && a.taps > 1 ? a.state + (uint64_t)a.slots[t] * (a.taps - 1) * a.width : nullptr;
+    const bool fresh = state && a.positions[t] == 0;
+    TA *h = static_cast<TA *>(a.h) + (uint64_t)t * a.h_pitch;
     for (uint32_t g = 0; g < a.n_group; ++g) {
-        float s = 0.0f;
-        for (uint32_t c = g * group + threadIdx.x; a.norm && c < (g + 1) * group; c += blockDim.x) {
-            const float v = value(c, false);
-            s += v * v;
+        const uint32_t c0 = g * group + threadIdx.x, c1 = (g + 1) * group;
+        float q = 0.0f;
+        for (uint32_t c = c0; a.norm && c < c1; c += blockDim.x) {
+            const float v = averaged(c, sum(c));
+            q += v * v;
         }
-        const float f = a.norm ? inv_rms(block_sum(s, red), group, a.eps) : 0.0f;
-        for (uint32_t c = g * group + threadIdx.x; c < (g + 1) * group; c += blockDim.x) {  // (a sum may replace its own x)
-            const float v = value(c, true);
-            if (!a.norm) continue;
-            if (a.taps) a.normed[at + c] = v * f * a.norm[c];
-            else static_cast<TA *>(a.h)[(uint64_t)t * a.h_pitch + c] = to_act<TA>(v * f * a.norm[c]);
+        const float f = a.norm ? inv_rms(block_sum(q, red), group, a.eps) : 0.0f;
+        if (LEAVE == LEAVE_INVERSE && threadIdx.x == 0) a.inverse[(uint64_t)t * a.n_group + g] = f;
+        for (uint32_t c = c0; c < c1; c += blockDim.x) {  // (each x is read before it is replaced)
+            const float s = sum(c), v = averaged(c, s);
+            if (a.sum) a.sum[at + c] = s;
+            if (a.depth && a.average) a.average[at + c] = v;
+            if (LEAVE == LEAVE_INVERSE || !a.norm) continue;
+            const float n[1] = {v * f * a.norm[c]};
+            if (!a.taps) h[c] = to_act<TA>(n[0]);
+            else conv_step<1>(a, state, fresh, c, n, [&](const float(&o)[1]) { h[c] = to_act<TA>(o[0]); });
         }
     }
 }
 
-constexpr uint32_t RUN_MAX_TAPS = 4, RUN_MAX = 32;
+// A thread has V channels of TOKENS consecutive tokens of a span.  The thread with a span's first tokens is the only one that reads
+// the state (a thread's tokens are not fewer than the convolution reaches back), and replaces it when it has.
+template <int V> struct Channels { float v[V]; };
+template <int V>
+__device__ __forceinline__ Channels<V> channels(const float *p) {
+    Channels<V> r;
+    if constexpr (V == 4) {
+        const float4 u = f4(p);
+        r.v[0] = u.x, r.v[1] = u.y, r.v[2] = u.z, r.v[3] = u.w;
+    } else {
+        r.v[0] = *p;
+    }
+    return r;
+}
+template <typename TA, int V>
+__device__ __forceinline__ void put(TA *p, const Channels<V> &x) {
+    if constexpr (V == 4) store4<TA>(p, make_float4(x.v[0], x.v[1], x.v[2], x.v[3]));
+    else *p = to_act<TA>(x.v[0]);
+}
+constexpr int IC_THREADS = 128;
+template <int K> constexpr int IC_TOKENS = K ? 8 : 16;
+static_assert(IC_TOKENS<0> >= (int)CONV_MAX_TAPS - 1, "a thread's tokens reach over the state");
 
-template <typename TA, int NV>
-void run_form(const ResidualArgs &a, uint32_t grid, uint32_t threads, uint32_t run, size_t smem, cudaStream_t st) {
-    auto launch = [&](void (*k)(ResidualArgs, uint32_t)) { launch_pdl(k, grid, threads, smem, st, a, run); };
-    switch (a.norm ? a.taps : 0) {
-    case 0: launch(residual_run_kernel<TA, NV, 0>); break;
-    case 1: launch(residual_run_kernel<TA, NV, 1>); break;
-    case 2: launch(residual_run_kernel<TA, NV, 2>); break;
-    case 3: launch(residual_run_kernel<TA, NV, 3>); break;
-    default: launch(residual_run_kernel<TA, NV, 4>); break;
+template <typename TA, int K, int V>  // taps (0: a.taps)
+__global__ void __launch_bounds__(IC_THREADS) input_conv_kernel(ResidualArgs a, const float *v) {
+    constexpr int TOKENS = IC_TOKENS<K>;
+    pdl_release();
+    pdl_wait();
+    RowSpan sp;
+    uint32_t f0;
+    find_tile(a.spans, a.n_seq, 1, TOKENS, blockIdx.x, &sp, &f0);
+    const uint32_t c = V * (blockIdx.y * IC_THREADS + threadIdx.x);
+    if (f0 >= sp.n || c >= a.width) return;
+    const int n = (int)sp.n, first = (int)f0, last = min(first + TOKENS, n), taps = K ? K : (int)a.taps, back = taps - 1;
+    const uint32_t g = c / (a.width / a.n_group);
+    const float *x = v + (uint64_t)sp.row0 * a.width + c, *inv = a.inverse + (uint64_t)sp.row0 * a.n_group + g;
+    float *state = back ? a.state + (uint64_t)a.slots[sp.row0] * back * a.width + c : nullptr;
+    const bool fresh = a.positions[sp.row0] == 0;
+    const Channels<V> factor = channels<V>(a.norm + c);
+    auto normed = [&](int t) {
+        Channels<V> r = channels<V>(x + (uint64_t)t * a.width);
+        const float f = inv[(uint64_t)t * a.n_group];
+#pragma unroll
+        for (int e = 0; e < V; ++e) r.v[e] = r.v[e] * f * factor.v[e];
+        return r;
+    };
+    auto input = [&](int t) {
+        if (t >= 0) return normed(t);
+        return fresh ? Channels<V>{} : channels<V>(state + (uint64_t)(t + back) * a.width);
+    };
+    TA *h = static_cast<TA *>(a.h) + (uint64_t)sp.row0 * a.h_pitch + c;
+    auto add = [&](Channels<V> &o, int k, const Channels<V> &before) {
+        const Channels<V> w = channels<V>(a.conv + (uint64_t)k * a.width + c);
+#pragma unroll
+        for (int e = 0; e < V; ++e) o.v[e] = fmaf(w.v[e], before.v[e], o.v[e]);
+    };
+    if constexpr (K > 0) {
+        Channels<V> in[K - 1 + TOKENS];  // all of them are requested before the first is used
+#pragma unroll
+        for (int i = 0; i + 1 < K; ++i) in[i] = input(first - back + i);
+#pragma unroll
+        for (int i = 0; i < TOKENS; ++i) in[K - 1 + i] = first + i < last ? normed(first + i) : Channels<V>{};
+#pragma unroll
+        for (int i = 0; i < TOKENS; ++i) {
+            Channels<V> o = in[K - 1 + i];
+#pragma unroll
+            for (int k = 0; k < K; ++k) add(o, k, in[i + k]);
+            if (first + i < last) put<TA, V>(h + (uint64_t)(first + i) * a.h_pitch, o);
+        }
+    } else {
+        for (int t = first; t < last; ++t) {
+            Channels<V> o = normed(t);
+            for (int k = 0; k < taps; ++k) add(o, k, input(t - back + k));
+            put<TA, V>(h + (uint64_t)t * a.h_pitch, o);
+        }
+    }
+    if (first == 0)  // (an entry that is read here has a higher number than the one it goes to: it has not been replaced yet)
+        for (int i = 0; i < back; ++i) put<float, V>(state + (uint64_t)i * a.width, input(n - back + i));
+}
+
+template <typename TA, int V>
+void input_conv(const ResidualArgs &a, const float *v, cudaStream_t st) {
+    auto run = [&](void (*k)(ResidualArgs, const float *), uint32_t tokens) {
+        uint32_t tiles = 0;
+        for (uint32_t s = 0; s < a.n_seq; ++s) tiles += (a.h_spans[s].n + tokens - 1) / tokens;
+        launch_pdl(k, dim3(tiles, (a.width / V + IC_THREADS - 1) / IC_THREADS), IC_THREADS, 0, st, a, v);
+    };
+    switch (a.taps) {
+    case 2: return run(input_conv_kernel<TA, 2, V>, IC_TOKENS<2>);
+    case 3: return run(input_conv_kernel<TA, 3, V>, IC_TOKENS<3>);
+    case 4: return run(input_conv_kernel<TA, 4, V>, IC_TOKENS<4>);
+    default: return run(input_conv_kernel<TA, 0, V>, IC_TOKENS<0>);
     }
 }
 
 template <typename TA>
-uint32_t residual(const ResidualArgs &a, bool f32, int sm_count, cudaStream_t st) {
-    const uint32_t group = a.width / a.n_group, taps = a.norm ? a.taps : 0;
-    if (a.width % 4 == 0 && group % 4 == 0 && a.width <= 8192 && taps <= RUN_MAX_TAPS) {
-        // as many tokens per CTA as give every SM two CTAs
-        uint32_t run = 1, grid = a.T;
-        if (!a.single && taps > 1) {
-            run = std::min(RUN_MAX, std::max(RUN_MAX_TAPS, (a.T + 2 * (uint32_t)sm_count - 1) / (2 * (uint32_t)sm_count)));
-            grid = 0;
-            for (uint32_t s = 0; s < a.n_seq; ++s) grid += (a.h_spans[s].n + run - 1) / run;
-        }
-        const uint32_t nv = a.width > 4096 ? 2 : 1, threads = (a.width / 4 / nv + 31) / 32 * 32;
+uint32_t residual(const ResidualArgs &a, cudaStream_t st) {
+    const uint32_t group = a.width / a.n_group;
+    const RowShape r(a.width, a.T);
+    const bool conv = a.norm && a.taps > 1 && !a.single;  // else a token's convolution needs its own row and the state
+    if (r.vec && group % 4 == 0) {
         const size_t smem = (a.width / unit_columns(group) + a.n_group) * sizeof(float);
-        if (nv == 1) run_form<TA, 1>(a, grid, threads, run, smem, st);
-        else run_form<TA, 2>(a, grid, threads, run, smem, st);
-        return 1;
+        launch_pdl(conv ? residual_kernel<TA, ROW_VECS, LEAVE_INVERSE> : residual_kernel<TA, ROW_VECS, LEAVE_INPUT>, a.T, r.threads, smem, st, a);
+    } else {
+        launch_pdl(conv ? residual_any_kernel<TA, LEAVE_INVERSE> : residual_any_kernel<TA, LEAVE_INPUT>, a.T, 512, 0, st, a);
     }
-    launch_pdl(residual_row_kernel<TA>, a.T, 512, 0, st, a);
-    if (!taps) return 1;
-    ConvArgs c{};
-    c.y = a.normed;
-    c.y_pitch = c.n_channel = a.width;
-    c.taps = taps;
-    c.w = a.conv;
-    c.tap_step = a.width;
-    c.state = a.state;
-    c.h = a.h;
-    c.h_pitch = a.h_pitch;
-    c.T = a.T;
-    c.n_seq = a.n_seq;
-    c.spans = a.spans;
-    c.h_spans = a.h_spans;
-    c.single = a.single;
-    c.positions = a.positions;
-    c.slots = a.slots;
-    launch_conv(c, f32, st);
+    if (!conv) return 1;
+    const float *v = a.depth ? a.average : a.sum;
+    if (a.width % 4 == 0 && group % 4 == 0) input_conv<TA, 4>(a, v, st);
+    else input_conv<TA, 1>(a, v, st);
     return 2;
 }
 
 }  // namespace
 
-uint32_t launch_residual(const ResidualArgs &a, bool f32, int sm_count, cudaStream_t st) {
-    return f32 ? residual<float>(a, f32, sm_count, st) : residual<bf16>(a, f32, sm_count, st);
-}
+uint32_t launch_residual(const ResidualArgs &a, bool f32, cudaStream_t st) { return f32 ? residual<float>(a, st) : residual<bf16>(a, st); }
 
 }  // namespace ob
