@@ -43,7 +43,7 @@ struct PtPlan {
 };
 // mbarriers, byte offsets from PtPlan::bar
 constexpr uint32_t PT_K_FULL = 0, PT_K_EMPTY = 16, PT_V_FULL = 32, PT_V_EMPTY = 48, PT_S_FULL = 64, PT_P_FULL = 80, PT_O_FULL = 96, PT_Q_FULL = 112, PT_SLOT = 128, PT_ABORT = 132,
-                   PT_ITEMS = 160, PT_EXCHANGE = 320, PT_STAGES = PT_EXCHANGE + 2 * 2 * PT_ROWS * 4 + 48;
+                   PT_ITEMS = 160, PT_ITEM_FULL = 288, PT_EXCHANGE = 320, PT_STAGES = PT_EXCHANGE + 2 * 2 * PT_ROWS * 4 + 48;
 
 // Two fp32 multiply-adds in one instruction.
 __device__ __forceinline__ void fma2(float &d0, float &d1, float a0, float a1, float b, float c) {
@@ -61,7 +61,7 @@ __device__ __forceinline__ void quad_sync(uint32_t id) { asm volatile("bar.sync 
 __device__ __forceinline__ float gate_factor(float z) { return __fdividef(1.0f, 1.0f + pow2(z * -1.4426950408889634f)); }
 
 // A CTA's piece of work: 128 (two maps) or 256 (one map) consecutive (token, head) rows of one key/value head.  The TMA warp looks
-// it up and leaves it in a ring of four (it is never more than two tiles ahead); the others read it when its first keys are there.
+// it up and leaves it in a ring of four with an mbarrier each (it is never more than three items ahead).
 struct PtItem {
     uint32_t row0, f0, n_here, pos0, g;
     PageList pages;  // the kept ones fill whole tiles
@@ -207,6 +207,7 @@ attention_prompt_kernel(const __grid_constant__ CUtensorMap tm, const __grid_con
             mbar_init(bar + PT_O_FULL + 8 * s, 1);
             mbar_init(bar + PT_Q_FULL + 8 * s, 8);
         }
+        for (uint32_t i = 0; i < 4; ++i) mbar_init(bar + PT_ITEM_FULL + 8 * i, 1);
         *abort = 0u;
         asm volatile("fence.mbarrier_init.release.cluster;" ::: "memory");
         asm volatile("fence.proxy.async.shared::cta;" ::: "memory");
@@ -227,6 +228,7 @@ attention_prompt_kernel(const __grid_constant__ CUtensorMap tm, const __grid_con
             if (lane == 0) {
                 const int32_t *table = a.tables[w.row0];
                 pt_write(smem + pl.bar, turn, w);
+                mbar_arrive(bar + PT_ITEM_FULL + 8 * (turn % 4));
                 for (uint32_t i = 0; i < w.n_tiles() && ok; ++i, ++n) {
                     const uint32_t st = n % pl.stages, par = ((n / pl.stages) & 1u) ^ 1u;
                     int32_t y[PT_PAGES];
@@ -323,14 +325,18 @@ attention_prompt_kernel(const __grid_constant__ CUtensorMap tm, const __grid_con
         bool ok = true;
         auto load_query = [&](const PtItem &w) {  // the row's query (this half of it) into the swizzled operand tile
             const uint32_t i = (NM == 2 ? 0 : s * PT_ROWS) + r, f = w.f0 + min(i, w.n_here - 1);
-            const bf16 *q = static_cast<const bf16 *>(a.q) + (((uint64_t)(w.row0 + f / per) * a.n_head + w.g * per + f % per) * NM + (NM == 2 ? s : 0)) * a.dim_p;
+            const uint64_t t = w.row0 + f / per, h = w.g * per + f % per;
+            const bool two = NM == 1 && a.q2;
+            const bf16 *q = static_cast<const bf16 *>(a.q) + (two ? t * a.q_pitch + h * a.q_head : ((t * a.n_head + h) * NM + (NM == 2 ? s : 0)) * a.dim_p);
+            const bf16 *q2 = two ? static_cast<const bf16 *>(a.q2) + t * a.q2_pitch + h * a.q2_head - a.q_split : q;
+            const uint32_t split = two ? a.q_split / 8 : 0;
             uint8_t *dst = smem + s * pl.nb * PT_BLOCK + r * 128;
             for (uint32_t c0 = part; c0 < a.dim_p / 8; c0 += 8) {
                 uint4 v[4];
 #pragma unroll
                 for (uint32_t k = 0; k < 4; ++k) {
                     const uint32_t c = c0 + 2 * k;
-                    v[k] = i < w.n_here && c < a.dim_p / 8 ? *reinterpret_cast<const uint4 *>(q + 8 * c) : make_uint4(0, 0, 0, 0);
+                    v[k] = i < w.n_here && c < a.dim_p / 8 ? *reinterpret_cast<const uint4 *>((c < split ? q : q2) + 8 * c) : make_uint4(0, 0, 0, 0);
                 }
 #pragma unroll
                 for (uint32_t k = 0; k < 4; ++k) {
@@ -342,9 +348,11 @@ attention_prompt_kernel(const __grid_constant__ CUtensorMap tm, const __grid_con
             __syncwarp();
             if (lane == 0) mbar_arrive(bar + PT_Q_FULL + 8 * s);
         };
-        uint32_t turn = 0, used = 0, n = 0;  // items, tiles of scores and tiles of keys so far
-        auto item_at = [&](uint32_t at, uint32_t item) {  // the item of turn `at`, whose first tile of keys is tile n
-            ok = ok && mbar_wait_warp(bar + PT_K_FULL + 8 * (n % pl.stages), (n / pl.stages) & 1u, abort);
+        uint32_t turn = 0, used = 0;  // items and tiles of scores so far
+        // The item of turn `at`.  (Not by its first keys' barrier: a stream that is done with the item before while that one's last
+        // keys are still to come would, with one stage, take the keys two tiles back for them.)
+        auto item_at = [&](uint32_t at, uint32_t item) {
+            ok = ok && mbar_wait_warp(bar + PT_ITEM_FULL + 8 * (at % 4), (at / 4) & 1u, abort);
             return ok ? pt_read(smem + pl.bar, at) : pt_item<NM>(a, item, n_row_tiles);
         };
         PtItem w{};
@@ -443,7 +451,6 @@ attention_prompt_kernel(const __grid_constant__ CUtensorMap tm, const __grid_con
             // learns that from the end of the item.
             const bool more = item + gridDim.x < n_items;
             PtItem next{};
-            n += w.n_tiles();
             if (more) next = item_at(turn + 1, item + gridDim.x);
             const bool idle = end == first;
             const RowOut ro = row_out(a, w, w0);

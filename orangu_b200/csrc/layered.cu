@@ -57,6 +57,7 @@ struct MixerPlan {
     // latent attention
     Dense uk, uv;        // per head [kv_rank <- dim], [vdim <- kv_rank]
     Dense expand;        // latent -> keys [H][dim_k], then (from row ex_v0) values [H][vdim_k]; no rows: prompts attend in the latent space too
+    bool paged = false;  // prompts' keys and values go into pages, per head (keys, from row ex_v0 values)
     uint32_t dim_p = 0, kv_p = 0, dq = 0, kv_w = 0, dim_k = 0, vdim_k = 0, ex_v0 = 0;
     float *kv_norm = nullptr;
     void *pool = nullptr;
@@ -127,6 +128,8 @@ struct LayeredGraph : StepGraph {
     float *y = nullptr, *o_ret = nullptr, *sy = nullptr, *part = nullptr;
     void *lat = nullptr, *expanded = nullptr;  // gathered latents of prompts, their keys and values: key_cap rows
     uint32_t key_cap = 0;
+    int32_t *numbers = nullptr;                // tables of pages that lie in order
+    const int32_t **page_tables = nullptr;
     void *ffa = nullptr;      // feed-forward activations of sequential blocks, a row per token or (token, expert) pair
     float *yo = nullptr;      // their outputs, and the mixers'
     MoeArgs moe{};            // routing buffers
@@ -168,6 +171,7 @@ struct LayeredGraph : StepGraph {
     void layers(uint32_t T, uint32_t n_seq, const RowSpan *spans, uint32_t max_pos, cudaStream_t st) override;
     void head(const uint32_t *d_rows, uint32_t n, cudaStream_t st) override;
     void latent(const MixerPlan &P, uint32_t T, uint32_t n_seq, const RowSpan *spans, bool single, uint32_t max_pos, cudaStream_t st);
+    void prompt_in_pages(const MixerPlan &P, const float *head_gate, const LatentArgs &l, uint32_t n_keys, uint32_t s0, uint32_t s1, cudaStream_t st);
     void retention(const MixerPlan &P, uint32_t T, uint32_t n_seq, const RowSpan *spans, cudaStream_t st);
     void state_space(const MixerPlan &P, uint32_t T, uint32_t n_seq, const RowSpan *spans, bool single, cudaStream_t st);
     void time_mixing(const MixerPlan &P, const float *norm, uint32_t T, uint32_t n_seq, const RowSpan *spans, bool single, cudaStream_t st);
@@ -334,22 +338,86 @@ void LayeredGraph::latent(const MixerPlan &P, uint32_t T, uint32_t n_seq, const 
     p.out = cat;
     p.out_pitch = cat_pitch;
     const uint32_t *h_pos = reinterpret_cast<const uint32_t *>(m->h_meta + ml.off_positions);
+    if (P.paged) {
+        p.pages = expanded;
+        p.page_row = P.row;
+        p.page_rot0 = P.dim_k;
+        p.numbers = numbers;
+        p.page_tables = page_tables;
+    }
+    const uint32_t unit = P.paged ? KV_PAGE : 1;
     for (uint32_t s = n_short; s < n_seq;) {  // as many spans at a time as the buffers hold
+        const uint32_t s0 = s;
         p.n_span = p.n_keys = p.n_tiles = 0;
         for (; s < n_seq && p.n_span < PREFILL_GROUP; ++s) {
-            const uint32_t pos0 = h_pos[spans[s].row0], hist = P.mx.window ? std::min(pos0, P.mx.window - 1) : pos0;
-            if (p.n_span && p.n_keys + hist + spans[s].n > key_cap) break;
+            const uint32_t pos0 = h_pos[spans[s].row0], from = P.mx.window && pos0 >= P.mx.window ? pos0 - P.mx.window + 1 : 0, hist = pos0 - from / unit * unit;
+            const uint32_t keys = round_up(hist + spans[s].n, unit);
+            if (p.n_span && p.n_keys + keys > key_cap) break;
             p.span[p.n_span++] = PrefillSpan{spans[s].row0, spans[s].n, pos0, hist, p.n_keys, p.n_tiles};
-            p.n_keys += hist + spans[s].n;
+            p.n_keys += keys;
             p.n_tiles += latent_prefill_tiles(spans[s].n);
         }
         launch_latent_gather(p, st);
+        if (P.paged) {
+            prompt_in_pages(P, gate, a, p.n_keys, s0, s, st);
+            continue;
+        }
         LinArgs ex = product(P.expand, lat, P.dq, p.n_keys);
         segment(ex, 0, P.expand.rows, LE_ACT, expanded, P.expand.rows);
         linear(ex, st);
         launch_latent_prefill(p, st);
         m->ctx->launches += 2;
     }
+}
+
+// Latent attention of spans [s0, s1): the gathered latents become pages of one key/value head per head, which are attended as such.
+void LayeredGraph::prompt_in_pages(const MixerPlan &P, const float *head_gate, const LatentArgs &l, uint32_t n_keys, uint32_t s0, uint32_t s1, cudaStream_t st) {
+    const uint32_t H = P.mx.n_head;
+    LinArgs ex = product(P.expand, lat, P.dq, n_keys);
+    ex.n_rows = P.expand.rows / H;
+    ex.n_batch = H;
+    segment(ex, 0, P.dim_k, LE_ACT, expanded, P.row, 0, KV_PAGE * P.row);
+    segment(ex, P.ex_v0, P.vdim_k, LE_ACT, expanded, P.row, P.dim_k + P.dq - P.kv_p, KV_PAGE * P.row);
+    for (int i = 0; i < 2; ++i) ex.seg[i].page_pitch = H * KV_PAGE * P.row;
+    linear(ex, st);
+    AttentionArgs a{};
+    a.y_pitch = y_pitch;
+    a.va = qn;
+    a.va_pitch = P.act_rows;
+    a.gate0 = P.gate0;
+    a.has_gate = P.has_gate;
+    a.n_head = a.n_kv = H;
+    a.n_map = 1;
+    a.vdim = P.mx.vdim;
+    a.window = P.mx.window;
+    a.dim_p = P.dim_k + P.dq - P.kv_p;
+    a.vdim_p = P.vdim_k;
+    a.row = P.row;
+    a.scale = P.mx.scale;
+    a.head_gain = 1.0f;
+    a.sink = P.sink;
+    a.head_gate = head_gate;
+    a.q = qn;
+    a.q2 = static_cast<uint8_t *>(q) + P.kv_p * es();
+    a.q_split = P.dim_k;
+    a.q_pitch = P.act_rows;
+    a.q_head = P.dim_p;
+    a.q2_pitch = H * P.dq;
+    a.q2_head = P.dq;
+    a.cache = expanded;
+    a.n_pages = key_cap / KV_PAGE;
+    a.out = cat;
+    a.out_pitch = cat_pitch;
+    a.T = l.T;
+    a.n_seq = s1;
+    a.n_short = s0;
+    a.spans = l.spans;
+    a.h_spans = l.h_spans;
+    a.positions = l.positions;
+    a.tables = page_tables;
+    a.max_pos = l.max_pos;
+    if (!launch_attention_prompt(a, m->ctx->sm_count, st)) failed = true;
+    m->ctx->launches += 2;
 }
 
 void LayeredGraph::retention(const MixerPlan &P, uint32_t T, uint32_t n_seq, const RowSpan *spans, cudaStream_t st) {
@@ -1056,7 +1124,18 @@ int LayeredGraph::build_mixer(const ob_mixer_desc &x, MixerPlan &P) {
         if ((rc = upload(uk, &P.uk)) || (rc = upload(uv, &P.uv))) return rc;
         P.dim_k = round_up(x.dim, 16);
         P.vdim_k = round_up(x.vdim, 16);
-        if (!f32 && latent_prefill_supported(P.dim_k, P.dq - P.kv_p, P.vdim_k)) {
+        P.paged = !f32 && x.scale > 0 && attention_prompt_supported(1, P.dim_k + P.dq - P.kv_p, P.vdim_k);
+        if (P.paged) {
+            P.row = P.dim_k + P.dq - P.kv_p + P.vdim_k;
+            P.ex_v0 = round_up(P.dim_k, LIN_ROW_ALIGN);
+            const uint32_t per = P.ex_v0 + round_up(P.vdim_k, LIN_ROW_ALIGN);
+            HostDense ex(H * per, P.kv_w);
+            for (uint32_t hd = 0; hd < H; ++hd) {
+                for (uint32_t d = 0; d < x.dim; ++d) ex.copy(hd * per + d, 0, x.w_uk, hd * x.dim + d);
+                for (uint32_t d = 0; d < x.vdim; ++d) ex.copy(hd * per + P.ex_v0 + d, 0, x.w_uv, hd * x.vdim + d);
+            }
+            if ((rc = upload(ex, &P.expand))) return rc;
+        } else if (!f32 && latent_prefill_supported(P.dim_k, P.dq - P.kv_p, P.vdim_k)) {
             P.ex_v0 = round_up(H * P.dim_k, LIN_ROW_ALIGN);
             HostDense ex(P.ex_v0 + round_up(H * P.vdim_k, LIN_ROW_ALIGN), P.kv_w);
             for (uint32_t hd = 0; hd < H; ++hd) {
@@ -1213,7 +1292,7 @@ int LayeredGraph::build(const ob_layered_desc &c) {
             kvp = std::max<size_t>(kvp, P.kv_p);
             if (P.expand.rows) {
                 dq = std::max<size_t>(dq, P.dq);
-                ex = std::max<size_t>(ex, P.expand.rows);
+                ex = std::max<size_t>(ex, P.paged ? H * P.row : P.expand.rows);
                 reach = std::max<size_t>(reach, std::min(P.mx.window ? P.mx.window - 1 : m->cfg.max_seq_len, m->cfg.max_seq_len));
             }
         } else {
@@ -1254,7 +1333,11 @@ int LayeredGraph::build(const ob_layered_desc &c) {
         moe.row_score = row_score;
     }
     if (ex) {
-        key_cap = (uint32_t)(T + reach);
+        key_cap = round_up((uint32_t)(T + reach), KV_PAGE) + (PREFILL_GROUP + 1) * KV_PAGE;  // (spans in pages begin and end at sixteens)
+        std::vector<int32_t> order(key_cap / KV_PAGE);
+        for (size_t i = 0; i < order.size(); ++i) order[i] = (int32_t)i;
+        if ((rc = dev_alloc(m, &numbers, order.size())) || (rc = dev_alloc(m, &page_tables, T))) return rc;
+        OB_CUDA(m->ctx, cudaMemcpy(numbers, order.data(), order.size() * 4, cudaMemcpyHostToDevice));
         if ((rc = scratch(&lat, (size_t)key_cap * dq, 2)) || (rc = scratch(&expanded, (size_t)key_cap * ex, 2))) return rc;
     }
     if (plain) {

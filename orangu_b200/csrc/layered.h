@@ -38,6 +38,7 @@ struct LinSegment {       // consecutive rows of the weight with one epilogue; r
     int epi;
     void *out;            // element (t, r) goes to out[t * pitch + col0 + batch * batch_cols + (r - row0)] (pairs: (r - row0) / 2)
     uint32_t pitch, col0, batch_cols;
+    uint32_t page_pitch = 0;  // > 0: sixteen t's are pitch apart, the sixteens page_pitch
 };
 struct LinArgs {
     const __nv_bfloat16 *w;   // [n_batch][n_rows][kp], zero padded
@@ -137,7 +138,9 @@ cudaError_t mixers_configure();
 void launch_latent_prep(const LatentArgs &a, bool f32, cudaStream_t st);   // norms and appends the latent, rotates and stores the query parts
 uint32_t launch_latent_attention(const LatentArgs &a, bool f32, int sm_count, cudaStream_t st);  // returns the kernels launched
 
-// Prompts: the window's latents are gathered from the pages, multiplied out to keys and values (a product), and attended per head.
+// Prompts: the window's latents are gathered from the pages, multiplied out to keys and values (a product), and attended per head:
+// on tcgen05 as attention over pages of one key/value head per head (gqa_tc5.cu), or, where that does not take the sizes, by
+// latent_prefill_kernel.
 constexpr uint32_t PREFILL_SPAN = 64;     // spans of at least this many rows go this way (bf16); in a step they follow the shorter ones
 constexpr uint32_t PREFILL_GROUP = 8;     // spans of one launch
 struct PrefillSpan {
@@ -154,6 +157,11 @@ struct LatentPrefillArgs {
     const int32_t *const *tables;
     const void *cache;                    // [page][16][dq]
     void *lat;                            // [n_keys][dq] gathered rows
+    // gathered into pages: spans begin at sixteens, what is past a span's end is zero
+    void *pages;                          // [page][n_head][16][page_row]: gets the rotated key part from page_rot0 on; null: no pages
+    uint32_t page_row, page_rot0;
+    const int32_t *numbers;               // 0, 1, 2 ..
+    const int32_t **page_tables;          // [T]: the first row of a span gets its table
     const void *expanded;                 // [n_keys][ex_pitch]: keys [H][dim_k], at ex_v0 values [H][vdim_k]
     uint32_t ex_pitch, ex_v0;
     const void *qn, *q;                   // unrotated query parts [T][qn_pitch] (head h at h * dim_p), rotated ones in [T][H][dq] at kv_p
@@ -209,6 +217,8 @@ struct AttentionArgs {       // softmax attention of one layer over T rows
     const float *head_gate;  // f32 [T][y_pitch]: sigmoid of entry h scales head h; null: none.  These four: one map
     Rot rot;
     void *q;                 // activations [T][n_head][n_map][dim_p]
+    const void *q2 = nullptr;  // prompts on tcgen05, one map: columns from q_split on come from here
+    uint32_t q_split = 0, q_pitch = 0, q_head = 0, q2_pitch = 0, q2_head = 0;  // with q2: pitches of a token and of a head, of both
     void *cache;             // activations [page][n_kv][16][row]
     uint32_t n_pages;        // of the pool
     void *out;               // activations [T][out_pitch], head h at h * vdim

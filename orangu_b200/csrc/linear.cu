@@ -79,7 +79,8 @@ __device__ __forceinline__ void epilogue_store(const LinArgs &a, uint32_t batch,
         const LinSegment &g = a.seg[s];
         if (r < g.row0 || r >= g.row0 + g.n) continue;
         const uint32_t k = r - g.row0, n = min((uint32_t)N, g.n - k);
-        const uint64_t base = (uint64_t)t * g.pitch + g.col0 + (uint64_t)batch * g.batch_cols;
+        const uint64_t row = g.page_pitch ? (uint64_t)(t / KV_PAGE) * g.page_pitch + t % KV_PAGE * g.pitch : (uint64_t)t * g.pitch;
+        const uint64_t base = row + g.col0 + (uint64_t)batch * g.batch_cols;
         switch (g.epi) {
         case LE_F32: store_row<N>(static_cast<float *>(g.out) + base + k, v, n); break;
         case LE_ACT: store_row<N>(static_cast<TA *>(g.out) + base + k, v, n); break;

@@ -626,9 +626,20 @@ __global__ void __launch_bounds__(256) latent_gather_kernel(LatentPrefillArgs a)
     while (s + 1 < a.n_span && key >= a.span[s + 1].key0) ++s;
     const PrefillSpan sp = a.span[s];
     const uint32_t p = sp.pos0 - sp.hist + (key - sp.key0);
-    const uint4 *src = reinterpret_cast<const uint4 *>(static_cast<const bf16 *>(a.cache) + ((uint64_t)a.tables[sp.row0][p / KV_PAGE] * KV_PAGE + p % KV_PAGE) * a.dq);
+    const bool live = p < sp.pos0 + sp.n;
+    const uint4 *src = reinterpret_cast<const uint4 *>(static_cast<const bf16 *>(a.cache) + (live ? ((uint64_t)a.tables[sp.row0][p / KV_PAGE] * KV_PAGE + p % KV_PAGE) * a.dq : 0));
     uint4 *dst = reinterpret_cast<uint4 *>(static_cast<bf16 *>(a.lat) + (uint64_t)key * a.dq);
-    for (uint32_t i = lane; i < a.dq / 8; i += 32) dst[i] = src[i];
+    for (uint32_t i = lane; i < a.dq / 8; i += 32) dst[i] = live ? src[i] : make_uint4(0, 0, 0, 0);
+    if (!a.pages) return;
+    if (key == sp.key0 && lane == 0) a.page_tables[sp.row0] = a.numbers + ((int64_t)(sp.key0 / KV_PAGE) - (int64_t)(p / KV_PAGE));
+    const uint32_t chunks = (a.dq - a.kv_p) / 8;  // of the rotated part, which every head's row gets
+    if (!chunks) return;
+    const RowCopy rc(chunks);
+    bf16 *page = static_cast<bf16 *>(a.pages) + ((uint64_t)(key / KV_PAGE) * a.n_head * KV_PAGE + key % KV_PAGE) * a.page_row + a.page_rot0;
+    for (uint32_t c = rc.chunk; c < chunks; c += 32) {
+        const uint4 v = live ? src[a.kv_p / 8 + c] : make_uint4(0, 0, 0, 0);
+        for (uint32_t h = rc.row; h < a.n_head; h += rc.rows) reinterpret_cast<uint4 *>(page + (uint64_t)h * KV_PAGE * a.page_row)[c] = v;
+    }
 }
 
 template <int NV>  // columns of a value in sixteens; what goes past vdim_k is computed from whatever follows in shared memory and dropped

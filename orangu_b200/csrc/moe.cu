@@ -23,12 +23,13 @@ __device__ __forceinline__ void eight(const float *p, float (&f)[8]) {
     f[0] = a.x, f[1] = a.y, f[2] = a.z, f[3] = a.w, f[4] = b.x, f[5] = b.y, f[6] = b.z, f[7] = b.w;
 }
 
-// One warp: the largest of the z[0 .. n) whose lane's bit (z[lane + 32 j]: bit j) is not set, the first of equals.
+// One warp: the largest of the z[0 .. n) whose lane's bit (z[lane + 32 j]: bit j) is not set, the first of equals.  What is not a
+// number counts as the smallest: whatever the logits are, the lanes agree on one that exists.
 __device__ __forceinline__ void largest(const float *z, uint32_t n, uint32_t closed, float *value, uint32_t *place) {
     float best = -INFINITY;
     uint32_t at = 0xffffffffu;
     for (uint32_t e = threadIdx.x & 31, j = 0; e < n; e += 32, ++j)
-        if (!(closed >> j & 1u) && (z[e] > best || at == 0xffffffffu)) best = z[e], at = e;
+        if (!(closed >> j & 1u) && (z[e] > best || at == 0xffffffffu)) best = fmaxf(z[e], -INFINITY), at = e;
 #pragma unroll
     for (int o = 16; o > 0; o >>= 1) {
         const float v = __shfl_xor_sync(0xffffffffu, best, o);

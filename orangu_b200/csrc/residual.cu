@@ -220,24 +220,29 @@ static_assert(IC_TOKENS<0> >= (int)CONV_MAX_TAPS - 1, "a thread's tokens reach o
 template <typename TA, int K, int V>  // taps (0: a.taps)
 __global__ void __launch_bounds__(IC_THREADS) input_conv_kernel(ResidualArgs a, const float *v) {
     constexpr int TOKENS = IC_TOKENS<K>;
+    const uint32_t c = V * (blockIdx.y * IC_THREADS + threadIdx.x), c_in = min(c, a.width - V);
+    const Channels<V> factor = channels<V>(a.norm + c_in);
+    Channels<V> w[K > 0 ? K : 1];
+#pragma unroll
+    for (int k = 0; k < K; ++k) w[k] = channels<V>(a.conv + (uint64_t)k * a.width + c_in);
     pdl_release();
     pdl_wait();
     RowSpan sp;
     uint32_t f0;
     find_tile(a.spans, a.n_seq, 1, TOKENS, blockIdx.x, &sp, &f0);
-    const uint32_t c = V * (blockIdx.y * IC_THREADS + threadIdx.x);
     if (f0 >= sp.n || c >= a.width) return;
     const int n = (int)sp.n, first = (int)f0, last = min(first + TOKENS, n), taps = K ? K : (int)a.taps, back = taps - 1;
     const uint32_t g = c / (a.width / a.n_group);
     const float *x = v + (uint64_t)sp.row0 * a.width + c, *inv = a.inverse + (uint64_t)sp.row0 * a.n_group + g;
     float *state = back ? a.state + (uint64_t)a.slots[sp.row0] * back * a.width + c : nullptr;
     const bool fresh = a.positions[sp.row0] == 0;
-    const Channels<V> factor = channels<V>(a.norm + c);
-    auto normed = [&](int t) {
-        Channels<V> r = channels<V>(x + (uint64_t)t * a.width);
-        const float f = inv[(uint64_t)t * a.n_group];
+    auto scaled = [&](Channels<V> &r, float f) {
 #pragma unroll
         for (int e = 0; e < V; ++e) r.v[e] = r.v[e] * f * factor.v[e];
+    };
+    auto normed = [&](int t) {
+        Channels<V> r = channels<V>(x + (uint64_t)t * a.width);
+        scaled(r, inv[(uint64_t)t * a.n_group]);
         return r;
     };
     auto input = [&](int t) {
@@ -245,28 +250,36 @@ __global__ void __launch_bounds__(IC_THREADS) input_conv_kernel(ResidualArgs a, 
         return fresh ? Channels<V>{} : channels<V>(state + (uint64_t)(t + back) * a.width);
     };
     TA *h = static_cast<TA *>(a.h) + (uint64_t)sp.row0 * a.h_pitch + c;
-    auto add = [&](Channels<V> &o, int k, const Channels<V> &before) {
-        const Channels<V> w = channels<V>(a.conv + (uint64_t)k * a.width + c);
+    auto add = [&](Channels<V> &o, const Channels<V> &tap, const Channels<V> &before) {
 #pragma unroll
-        for (int e = 0; e < V; ++e) o.v[e] = fmaf(w.v[e], before.v[e], o.v[e]);
+        for (int e = 0; e < V; ++e) o.v[e] = fmaf(tap.v[e], before.v[e], o.v[e]);
     };
     if constexpr (K > 0) {
-        Channels<V> in[K - 1 + TOKENS];  // all of them are requested before the first is used
+        Channels<V> in[K - 1 + TOKENS];  // all of them are requested before the first is used (past the ends: the last one and the first again)
+        float f[K - 1 + TOKENS];
 #pragma unroll
-        for (int i = 0; i + 1 < K; ++i) in[i] = input(first - back + i);
+        for (int i = 0; i < K - 1 + TOKENS; ++i) {
+            const int t = max(min(first - back + i, last - 1), 0);
+            in[i] = channels<V>(x + (uint64_t)t * a.width);
+            f[i] = inv[(uint64_t)t * a.n_group];
+        }
 #pragma unroll
-        for (int i = 0; i < TOKENS; ++i) in[K - 1 + i] = first + i < last ? normed(first + i) : Channels<V>{};
+        for (int i = 0; i < K - 1 + TOKENS; ++i) scaled(in[i], f[i]);
+        if (first == 0) {
+#pragma unroll
+            for (int i = 0; i + 1 < K; ++i) in[i] = input(i - back);
+        }
 #pragma unroll
         for (int i = 0; i < TOKENS; ++i) {
             Channels<V> o = in[K - 1 + i];
 #pragma unroll
-            for (int k = 0; k < K; ++k) add(o, k, in[i + k]);
+            for (int k = 0; k < K; ++k) add(o, w[k], in[i + k]);
             if (first + i < last) put<TA, V>(h + (uint64_t)(first + i) * a.h_pitch, o);
         }
     } else {
         for (int t = first; t < last; ++t) {
             Channels<V> o = normed(t);
-            for (int k = 0; k < taps; ++k) add(o, k, input(t - back + k));
+            for (int k = 0; k < taps; ++k) add(o, channels<V>(a.conv + (uint64_t)k * a.width + c), input(t - back + k));
             put<TA, V>(h + (uint64_t)t * a.h_pitch, o);
         }
     }
