@@ -562,40 +562,83 @@ __global__ void __launch_bounds__(LM_THREADS, MT == 4 ? 1 : 2) latent_attn_mma_k
         }
 }
 
-// The splits of one (token, head) row put together: a CTA per row when there are few, a warp per row when there are many.
-constexpr uint32_t MERGE_MAX = 256;  // splits
-__global__ void __launch_bounds__(128) latent_merge_kernel(LatentArgs a, uint32_t n_splits, uint32_t n_rows, uint32_t rows_per_cta) {
+// The splits of one (token, head) row put together, a CTA per row: `groups` groups of 128 threads take splits in turn, a thread four
+// columns (and every 512th).  What the first splits hold is requested before their weights are known.
+constexpr uint32_t MERGE_MAX = 256, MERGE_AT_ONCE = 8, MERGE_GROUPS = 8;  // splits; loads of a thread in flight
+__global__ void __launch_bounds__(128 * MERGE_GROUPS) latent_merge_kernel(LatentArgs a, uint32_t n_splits) {
+    extern __shared__ float sums[];  // [groups - 1][512]
+    __shared__ float weight[MERGE_MAX], total;
+    const uint32_t lane = threadIdx.x & 31, group = threadIdx.x / 128, groups = blockDim.x / 128;
     pdl_release();
     pdl_wait();
-    const uint32_t lane = threadIdx.x & 31, width = rows_per_cta == 1 ? 128 : 32;
-    const uint64_t n_flat = (uint64_t)a.T * a.n_head;
-    uint64_t flat = (uint64_t)blockIdx.x * rows_per_cta + (rows_per_cta == 1 ? 0 : threadIdx.x >> 5);
-    if (flat >= n_rows) return;
+    uint64_t flat = blockIdx.x;
     if (!a.single) {  // only the rows of these spans have partial results
         RowSpan sp;
         uint32_t f;
         find_tile(a.spans, a.n_seq, a.n_head, 1, (uint32_t)flat, &sp, &f);
         flat = (uint64_t)sp.row0 * a.n_head + f;
     }
-    const uint64_t stride = n_flat * lm_part_row(a.kv_p);
+    const uint64_t stride = (uint64_t)a.T * a.n_head * lm_part_row(a.kv_p);
     const float *p = a.part + flat * lm_part_row(a.kv_p), *ml = p + a.kv_p;
-    float m = -INFINITY, l = 0.0f;
-    for (uint32_t s = lane; s < n_splits; s += 32) m = fmaxf(m, ml[s * stride]);
-    m = warp_max(m);
-    for (uint32_t s = lane; s < n_splits; s += 32) l += pow2(ml[s * stride] - m) * ml[s * stride + 1];
-    l = warp_sum(l);
-    if (a.sink) l += sink_weight(a.sink[flat % a.n_head], m);
-    const float inv = 1.0f / l;
     bf16 *o = static_cast<bf16 *>(a.o) + flat * a.o_head;
-    for (uint32_t c = 4 * (threadIdx.x % width); c < a.kv_p; c += 4 * width) {
-        float4 v = make_float4(0.0f, 0.0f, 0.0f, 0.0f);
-#pragma unroll 8
-        for (uint32_t s = 0; s < n_splits; ++s) {
-            const float w = pow2(ml[s * stride] - m);
-            const float4 u = *reinterpret_cast<const float4 *>(p + s * stride + c);
-            v.x = fmaf(w, u.x, v.x), v.y = fmaf(w, u.y, v.y), v.z = fmaf(w, u.z, v.z), v.w = fmaf(w, u.w, v.w);
+    const uint32_t steps = (a.kv_p + 511) / 512;
+    for (uint32_t k = 0; k < steps; ++k) {
+        const uint32_t c = 512 * k + 4 * (threadIdx.x % 128);
+        const bool in = c < a.kv_p;
+        float4 u[MERGE_AT_ONCE];
+        auto request = [&](uint32_t s0) {
+#pragma unroll
+            for (uint32_t i = 0; i < MERGE_AT_ONCE; ++i) {
+                const uint32_t s = s0 + i * groups;
+                u[i] = in && s < n_splits ? *reinterpret_cast<const float4 *>(p + s * stride + c) : make_float4(0.0f, 0.0f, 0.0f, 0.0f);
+            }
+        };
+        request(group);
+        if (k == 0) {
+            if (threadIdx.x < 32) {
+                float2 t[MERGE_MAX / 32];
+                float m = -INFINITY, l = 0.0f;
+#pragma unroll
+                for (uint32_t i = 0; i < MERGE_MAX / 32; ++i) {
+                    const uint32_t s = lane + 32 * i;
+                    t[i] = s < n_splits ? *reinterpret_cast<const float2 *>(ml + s * stride) : make_float2(-INFINITY, 0.0f);
+                    m = fmaxf(m, t[i].x);
+                }
+                m = warp_max(m);
+#pragma unroll
+                for (uint32_t i = 0; i < MERGE_MAX / 32; ++i) {
+                    const float w = pow2(t[i].x - m);
+                    weight[lane + 32 * i] = w;
+                    l += w * t[i].y;
+                }
+                l = warp_sum(l);
+                if (a.sink) l += sink_weight(a.sink[flat % a.n_head], m);
+                if (lane == 0) total = l;
+            }
+            __syncthreads();
         }
-        store4<bf16>(o + c, mul4(v, inv));
+        float4 v = make_float4(0.0f, 0.0f, 0.0f, 0.0f);
+        for (uint32_t s0 = group; s0 < n_splits; s0 += MERGE_AT_ONCE * groups) {
+            if (s0 != group) request(s0);
+#pragma unroll
+            for (uint32_t i = 0; i < MERGE_AT_ONCE; ++i) {
+                const uint32_t s = s0 + i * groups;
+                const float w = s < n_splits ? weight[s] : 0.0f;
+                v.x = fmaf(w, u[i].x, v.x), v.y = fmaf(w, u[i].y, v.y), v.z = fmaf(w, u[i].z, v.z), v.w = fmaf(w, u[i].w, v.w);
+            }
+        }
+        if (groups > 1) {
+            if (k) __syncthreads();  // (the sums before have been read)
+            float4 *mine = reinterpret_cast<float4 *>(sums) + threadIdx.x % 128;
+            if (group) mine[(group - 1) * 128] = v;
+            __syncthreads();
+            if (group) continue;
+            for (uint32_t g = 0; g + 1 < groups; ++g) {
+                const float4 w = mine[g * 128];
+                v.x += w.x, v.y += w.y, v.z += w.z, v.w += w.w;
+            }
+        }
+        if (in) store4<bf16>(o + c, mul4(v, 1.0f / total));
     }
 }
 
@@ -1189,8 +1232,8 @@ uint32_t launch_latent_attention(const LatentArgs &a, bool f32, int sm_count, cu
     uint32_t merge_rows = a.single ? a.n_seq * a.n_head : 0;
     if (!a.single)
         for (uint32_t s = 0; s < a.n_seq; ++s) merge_rows += a.h_spans[s].n * a.n_head;
-    const uint32_t per = merge_rows >= 1024 ? 4 : 1;
-    launch_pdl(latent_merge_kernel, (merge_rows + per - 1) / per, 128, 0, st, a, splits, merge_rows, per);
+    const uint32_t groups = std::min(MERGE_GROUPS, (splits + MERGE_AT_ONCE - 1) / MERGE_AT_ONCE);
+    launch_pdl(latent_merge_kernel, merge_rows, 128 * groups, (groups - 1) * 512 * sizeof(float), st, a, splits);
     return 2;
 }
 

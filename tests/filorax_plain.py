@@ -59,16 +59,19 @@ def visible(i, j, window=None):
 
 
 def attend(q, k, v, scale, window=None, sink=None):
-    """One head: q, k [n, d], v [n, d2].  A sink is one more term of the denominator, exp(sink), that brings no value."""
-    outs = []
-    for i in range(len(q)):
-        js = [j for j in range(len(q)) if visible(i, j, window)]
-        s = (k[js] @ q[i]) * scale
-        top = s.max() if sink is None else max(s.max(), sink)
-        p = np.exp(s - top)
-        total = p.sum() + (0.0 if sink is None else np.exp(sink - top))
-        outs.append(p @ v[js] / total)
-    return np.array(outs)
+    """q, k [n, heads, d], v [n, heads, d2] -> [n, heads, d2].  A head's sink is one more term of its denominator, exp(sink), that
+    brings no value."""
+    n, heads = q.shape[:2]
+    out = np.zeros((n, heads, v.shape[2]))
+    for i in range(n):
+        js = [j for j in range(n) if visible(i, j, window)]
+        for a in range(heads):
+            s = (k[js, a] @ q[i, a]) * scale
+            top = s.max() if sink is None else max(s.max(), sink[a])
+            p = np.exp(s - top)
+            total = p.sum() + (0.0 if sink is None else np.exp(sink[a] - top))
+            out[i, a] = p @ v[js, a] / total
+    return out
 
 
 def latent(h, w, mx, eps):
@@ -87,14 +90,11 @@ def latent_attention(h, w, mx, eps, rotated, sink, gated):
     c, kr = latent(h, w, mx, eps)
     k = (c @ w["uk"].T).reshape(n, H, D)
     v = (c @ w["uv"].T).reshape(n, H, V)
-    heads = []
-    for a in range(H):
-        qa, ka = q[:, a, :D], k[:, a]
-        if R:
-            turn = lambda x: np.stack([rotate(x[p], p, mx["rot"]["base"]) for p in range(n)])
-            qa, ka = np.concatenate([qa, turn(q[:, a, D:])], -1), np.concatenate([ka, turn(kr)], -1)
-        heads.append(attend(qa, ka, v[:, a], mx["scale"], window, w["sink"][a] if sink else None))
-    o = np.concatenate(heads, -1)
+    if R:
+        q = np.concatenate([q[..., :D], np.stack([rotate(q[p, :, D:], p, mx["rot"]["base"]) for p in range(n)])], -1)
+        shared = np.stack([rotate(kr[p], p, mx["rot"]["base"]) for p in range(n)])
+        k = np.concatenate([k, np.repeat(shared[:, None], H, 1)], -1)
+    o = attend(q, k, v, mx["scale"], window, w["sink"] if sink else None).reshape(n, H * V)
     if gated:
         o = o * sigmoid(h @ w["g"].T)
     return o @ w["o"].T
