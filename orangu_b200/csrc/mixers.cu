@@ -217,35 +217,77 @@ __global__ void __launch_bounds__(1024) post_norm_kernel(PostNormArgs a) {
 }
 
 // ---- latent attention: what a token leaves in the cache, and its rotated query parts -----------------------------------------------
-// Part 0 of a token is its cache row, every further part PREP_Q entries of its rotated query parts.
-constexpr uint32_t PREP_Q = 1024;
-template <typename TA>
-__global__ void __launch_bounds__(256) latent_prep_kernel(LatentArgs a) {
-    __shared__ float red[33];
+// A warp per token.  Part 0 is the token's cache row, every further part PREP_Q entries of its rotated query parts.
+constexpr uint32_t PREP_Q = 256, PREP_TOKENS = 8;
+
+// Entries [d, d + 4) of a rotated vector (rotated() has them one by one); d and half the rotated width are multiples of four.
+__device__ __forceinline__ float4 rotated4(const float *v, uint32_t d, const Rot &r, const float2 *cs) {
+    const float4 x = *reinterpret_cast<const float4 *>(v + d);
+    if (d >= r.dims) return x;
+    const uint32_t half = r.dims / 2;
+    if (r.interleaved) {
+        const float4 c = *reinterpret_cast<const float4 *>(cs + d / 2);
+        return make_float4(x.x * c.x - x.y * c.y, x.y * c.x + x.x * c.y, x.z * c.z - x.w * c.w, x.w * c.z + x.z * c.w);
+    }
+    const bool low = d < half;
+    const float2 *q = cs + (low ? d : d - half);
+    const float4 y = *reinterpret_cast<const float4 *>(v + (low ? d + half : d - half)), c0 = *reinterpret_cast<const float4 *>(q), c1 = *reinterpret_cast<const float4 *>(q + 2);
+    const float s = low ? -1.0f : 1.0f;
+    return make_float4(x.x * c0.x + s * y.x * c0.y, x.y * c0.z + s * y.y * c0.w, x.z * c1.x + s * y.z * c1.y, x.w * c1.z + s * y.w * c1.w);
+}
+
+template <typename TA, bool FOURS>  // FOURS: all sizes and pitches are multiples of four, half the rotated width too
+__global__ void __launch_bounds__(32 * PREP_TOKENS) latent_prep_kernel(LatentArgs a) {
     pdl_release();
     pdl_wait();
-    const uint32_t t = blockIdx.x, pos = a.positions[t];
+    const uint32_t t = blockIdx.x * PREP_TOKENS + threadIdx.x / 32, lane = threadIdx.x & 31;
+    if (t >= a.T) return;
+    constexpr uint32_t V = FOURS ? 4 : 1;
+    const uint32_t pos = a.positions[t];
     const float *y = a.y + (uint64_t)t * a.y_pitch;
     const float2 *cs = a.rot.table + (uint64_t)pos * (a.rot.dims / 2);
+    auto turn = [&](TA *to, const float *v, uint32_t d) {
+        if constexpr (FOURS) store4<TA>(to + d, rotated4(v, d, a.rot, cs));
+        else to[d] = to_act<TA>(rotated(v, d, a.rot, cs));
+    };
     if (blockIdx.y > 0) {
         TA *q = static_cast<TA *>(a.q) + (uint64_t)t * a.n_head * a.dq + a.kv_p;
         const uint32_t first = (blockIdx.y - 1) * PREP_Q, n = a.n_head * a.rot_dim;
-#pragma unroll
-        for (uint32_t u = 0; u < PREP_Q / 256; ++u) {
-            const uint32_t i = first + u * 256 + threadIdx.x;
+#pragma unroll 4
+        for (uint32_t u = V * lane; u < PREP_Q; u += 32 * V) {
+            const uint32_t i = first + u;
             if (i >= n) break;
-            const uint32_t h = i / a.rot_dim, d = i - h * a.rot_dim;
-            q[(uint64_t)h * a.dq + d] = to_act<TA>(rotated(y + (uint64_t)h * a.rot_dim, d, a.rot, cs));
+            const uint32_t h = i / a.rot_dim;
+            turn(q + (uint64_t)h * a.dq, y + (uint64_t)h * a.rot_dim, i - h * a.rot_dim);
         }
         return;
     }
     const float *lat = y + (uint64_t)a.n_head * a.rot_dim;
     TA *row = static_cast<TA *>(a.cache) + ((uint64_t)a.tables[t][pos / KV_PAGE] * KV_PAGE + pos % KV_PAGE) * a.dq;
-    for (uint32_t d = threadIdx.x; d < a.rot_dim; d += blockDim.x) row[a.kv_p + d] = to_act<TA>(rotated(lat + a.kv_rank, d, a.rot, cs));
+    for (uint32_t d = V * lane; d < a.rot_dim; d += 32 * V) turn(row + a.kv_p, lat + a.kv_rank, d);
     float s = 0.0f;
-    for (uint32_t i = threadIdx.x; i < a.kv_rank; i += blockDim.x) s += lat[i] * lat[i];
-    const float f = inv_rms(block_sum(s, red), a.kv_rank, a.eps);
-    for (uint32_t i = threadIdx.x; i < a.kv_rank; i += blockDim.x) row[i] = to_act<TA>(lat[i] * f * a.kv_norm[i]);
+    if constexpr (FOURS) {
+        constexpr uint32_t KEEP = 4;  // rows of up to 512 stay in registers
+        float4 x[KEEP];
+#pragma unroll
+        for (uint32_t k = 0; k < KEEP; ++k) {
+            const uint32_t i = 4 * lane + 128 * k;
+            x[k] = i < a.kv_rank ? *reinterpret_cast<const float4 *>(lat + i) : make_float4(0.0f, 0.0f, 0.0f, 0.0f);
+            s += sq4(x[k]);
+        }
+        for (uint32_t i = 4 * lane + 128 * KEEP; i < a.kv_rank; i += 128) s += sq4(*reinterpret_cast<const float4 *>(lat + i));
+        const float f = inv_rms(warp_sum(s), a.kv_rank, a.eps);
+#pragma unroll
+        for (uint32_t k = 0; k < KEEP; ++k) {
+            const uint32_t i = 4 * lane + 128 * k;
+            if (i < a.kv_rank) store4<TA>(row + i, mul44(mul4(x[k], f), *reinterpret_cast<const float4 *>(a.kv_norm + i)));
+        }
+        for (uint32_t i = 4 * lane + 128 * KEEP; i < a.kv_rank; i += 128) store4<TA>(row + i, mul44(mul4(*reinterpret_cast<const float4 *>(lat + i), f), *reinterpret_cast<const float4 *>(a.kv_norm + i)));
+    } else {
+        for (uint32_t i = lane; i < a.kv_rank; i += 32) s += lat[i] * lat[i];
+        const float f = inv_rms(warp_sum(s), a.kv_rank, a.eps);
+        for (uint32_t i = lane; i < a.kv_rank; i += 32) row[i] = to_act<TA>(lat[i] * f * a.kv_norm[i]);
+    }
 }
 
 // ---- latent attention, plain form: one CTA per (token, head), any sizes; fp32 throughout when the cache is fp32 ---------------------
@@ -1199,9 +1241,10 @@ void launch_side_finish(float *x, const float *y, const float *w, uint32_t width
 }
 
 void launch_latent_prep(const LatentArgs &a, bool f32, cudaStream_t st) {
-    const dim3 grid(a.T, 1 + (a.n_head * a.rot_dim + PREP_Q - 1) / PREP_Q);
-    if (f32) launch_pdl(latent_prep_kernel<float>, grid, 256, 0, st, a);
-    else launch_pdl(latent_prep_kernel<bf16>, grid, 256, 0, st, a);
+    const dim3 grid((a.T + PREP_TOKENS - 1) / PREP_TOKENS, 1 + (a.n_head * a.rot_dim + PREP_Q - 1) / PREP_Q);
+    const bool fours = a.y_pitch % 4 == 0 && a.kv_rank % 4 == 0 && a.rot_dim % 4 == 0 && a.rot.dims % (a.rot.interleaved ? 4 : 8) == 0;
+    if (f32) launch_pdl(fours ? latent_prep_kernel<float, true> : latent_prep_kernel<float, false>, grid, 32 * PREP_TOKENS, 0, st, a);
+    else launch_pdl(fours ? latent_prep_kernel<bf16, true> : latent_prep_kernel<bf16, false>, grid, 32 * PREP_TOKENS, 0, st, a);
 }
 
 uint32_t launch_latent_attention(const LatentArgs &a, bool f32, int sm_count, cudaStream_t st) {
