@@ -10,7 +10,6 @@
 //                     squares instead: n is then a product of three numbers, and is made where it is used
 // input_conv_kernel   h of spans: a few channels of several tokens per thread, no exchange between threads
 #include <algorithm>
-#include <type_traits>
 
 #include "mixers_common.cuh"
 

@@ -311,8 +311,8 @@ def test_short_starts_in_used_slots(backend, first, taps):
     got = m.forward_rows([a, b], [y[:first], z[:1]], range(first + 1))
     got_a, got_b = [got[:first]], [got[first:]]
     for i in range(8):  # one by one beside portions of two
-        lg = m.forward_rows([b, a], [z[1 + 2 * i:3 + 2 * i], y[first + i:first + i + 1]] if first + i < 12 else [z[1 + 2 * i:3 + 2 * i]], range(3)) if first + i < 12 \
-            else m.forward_rows([b], [z[1 + 2 * i:3 + 2 * i]], range(2))
+        more, pair = y[first + i:first + i + 1], z[1 + 2 * i:3 + 2 * i]
+        lg = m.forward_rows([b, a], [pair, more], range(3)) if more else m.forward_rows([b], [pair], range(2))
         got_b.append(lg[:2])
         got_a.append(lg[2:])
     got_a = np.concatenate(got_a)
